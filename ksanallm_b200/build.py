@@ -57,7 +57,14 @@ def engine_lib_path() -> Path:
     return LIB / f"_ksana_engine{suffix}"
 
 
-def build_kernels(force: bool = False, verbose: bool = False) -> Path:
+# what a dense decoder in bf16 or fp32 calls (no FP8 / FP4 / 4-bit weights, experts, latent attention or peer memory)
+DENSE_KERNELS = ("attention", "attention_f32", "attention_tc", "elementwise", "gemm_f32", "gemm_smallm", "gemm_tcgen05",
+                 "residual_stream", "sampler")
+
+
+def build_kernels(force: bool = False, verbose: bool = False, only=None) -> Path:
+    """``only``: names of the kernel sources to compile; the library then holds these and whatever other objects are
+    already built and current (a later full build adds the rest)."""
     LIB.mkdir(exist_ok=True)
     OBJ.mkdir(exist_ok=True)
     kdir = CSRC / "kernels"
@@ -67,8 +74,11 @@ def build_kernels(force: bool = False, verbose: bool = False) -> Path:
     jobs = []
     for s in srcs:
         o = OBJ / (s.stem + ".o")
+        stale = force or _newer(o, [s, *hdrs])
+        if only is not None and s.stem not in only and stale:
+            continue
         objs.append(o)
-        if force or _newer(o, [s, *hdrs]):
+        if stale:
             cmd = [_nvcc(), *NVCC_FLAGS, "-I", str(kdir), "-c", str(s), "-o", str(o)]
             if verbose:
                 cmd.insert(1, "-Xptxas")
@@ -107,6 +117,17 @@ def build_engine(force: bool = False) -> Path:
     if force or jobs or not out.exists():
         _run(["g++", "-shared", "-pthread", "-o", str(out), *map(str, objs), "-ldl"])
     return out
+
+
+def ensure_built(only=None) -> None:
+    """Builds what is missing or out of date; concurrent callers wait for one another."""
+    import fcntl
+    OBJ.mkdir(exist_ok=True)
+    with open(OBJ / ".lock", "w") as f:
+        fcntl.flock(f, fcntl.LOCK_EX)
+        with ThreadPoolExecutor(max_workers=2) as ex:
+            for r in [ex.submit(build_kernels, only=only), ex.submit(build_engine)]:
+                r.result()
 
 
 def build_host_stress(sanitizer: str = "thread") -> Path:

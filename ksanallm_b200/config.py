@@ -191,6 +191,57 @@ def load_yaml_config(path_or_dict) -> EngineConfig:
 
 
 # --------------------------------------------------------------------------------- model config
+# Descriptions of layers that are configured one by one (families whose config.json lists its layers)
+@dataclass
+class RotarySpec:
+    dims: int                             # leading dimensions of a head that rotate (halves: i with i + dims/2)
+    base: float
+    scaling: Optional[dict] = None        # Hugging Face style rope_scaling dict
+
+
+@dataclass
+class AttentionSpec:
+    heads: int
+    kv_heads: int
+    dim: int                              # query / key head size
+    vdim: int                             # value head size
+    scale: float
+    window: int = 0                       # sliding window in tokens, 0: full causal attention
+    keep_first: int = 0                   # first tokens that stay visible behind the window
+    sink: bool = False                    # learned per-head logit in the softmax denominator
+    rotary: Optional[RotarySpec] = None
+
+
+@dataclass
+class MlpSpec:
+    size: int
+    limit: float                          # clamp of the gate (from above) and of the linear part (both sides)
+    alpha: float = 1.702                  # slope inside the gate's sigmoid
+    offset: float = 1.0                   # added to the linear part
+
+
+@dataclass
+class LayerSpec:
+    mixer: AttentionSpec
+    mlp: Optional[MlpSpec]
+
+
+@dataclass
+class LoopSpec:
+    """Layers start .. stop-1 run ``times`` times with the same weights and a cache per pass."""
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass
+class PairEmbeddingSpec:
+    """Hashed embedding of (previous token, token): row (prev * mul_prev + token * mul_cur) mod buckets."""
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+
 @dataclass
 class ModelConfig:
     model_type: str = "llama"
@@ -217,7 +268,7 @@ class ModelConfig:
     gated_mlp: bool = True
     norm_type: str = "rmsnorm"            # rmsnorm | layernorm
     post_norm: bool = False               # GPT-1 / fairseq style
-    position_embedding: str = "rope"      # rope | alibi | learned | sinusoidal | mrope
+    position_embedding: str = "rope"      # rope | alibi | learned | sinusoidal | mrope | per_layer (layer_specs)
     mrope_section: Optional[List[int]] = None
     emb_scale: float = 1.0
     lm_head_norm: bool = False            # Baichuan2 normalised lm_head
@@ -254,6 +305,10 @@ class ModelConfig:
     weight_block_size: Optional[List[int]] = None
     is_visual: bool = False
     kv_scales: Optional[List[List[float]]] = None     # per layer (k_scale, v_scale)
+    # layers configured one by one
+    layer_specs: Optional[List[LayerSpec]] = None
+    loop: Optional[LoopSpec] = None
+    pair_embedding: Optional[PairEmbeddingSpec] = None
 
     @property
     def is_moe(self) -> bool:
@@ -268,8 +323,10 @@ _ARCH_ALIASES = {
     "llama": "llama", "mistral": "llama", "qwen2": "qwen", "qwen": "qwen", "qwen2_vl": "qwen2_vl", "baichuan": "baichuan",
     "chatglm": "chatglm", "glm": "chatglm", "gpt2": "gpt", "openai-gpt": "gpt", "fairseq-transformer": "gpt", "mixtral": "mixtral",
     "qwen2_moe": "qwen2_moe", "deepseek_v3": "deepseek_v3", "deepseek_v2": "deepseek_v3", "internlm2": "llama",
-    "yi": "llama",
+    "yi": "llama", "lenolix": "lenolix",
 }
+# No position limit is part of the Lenolix design: the serving configuration's max_token_len decides
+_UNBOUNDED_POSITIONS = 1 << 20
 
 
 def parse_model_max_length(hf: dict, max_pos: int) -> int:
@@ -343,8 +400,11 @@ def model_config_from_hf(hf: dict, generation: Optional[dict] = None, model_dir:
             hf["rope_scaling"] = {k: v for k, v in rp.items() if k != "rope_theta"}
         elif hf.get("rope_scaling") is None and rp.get("mrope_section"):
             hf["rope_scaling"] = {"mrope_section": rp["mrope_section"]}
-    mt = hf.get("model_type", "llama")
+    # families with a configuration format of their own name themselves in "architecture"
+    mt = hf.get("model_type") or str(hf.get("architecture", "llama")).lower()
     arch = resolve_architecture(mt, model_dir)
+    if arch == "lenolix":
+        return lenolix_config(hf, generation)
     c = ModelConfig(model_type=arch, hf_model_type=mt)
     if arch == "gpt":
         c.hidden_size = hf.get("n_embd", hf.get("hidden_size", hf.get("decoder_embed_dim", 768)))
@@ -445,6 +505,71 @@ def model_config_from_hf(hf: dict, generation: Optional[dict] = None, model_dir:
     c.pad_token_id = int(pad) if pad is not None else (1 if mt == "fairseq-transformer" else 0)   # fairseq dictionaries put <pad> at 1
     if c.num_heads % max(c.num_kv_heads, 1):
         raise ValueError("num_attention_heads must be a multiple of num_key_value_heads")
+    return c
+
+
+def _positive(d: dict, key: str, where: str) -> int:
+    v = int(d[key])
+    if v <= 0:
+        raise ValueError(f"{where}.{key} must be positive, not {v}")
+    return v
+
+
+def _lenolix_attention(m: dict, where: str) -> AttentionSpec:
+    a = AttentionSpec(_positive(m, "heads", where), _positive(m, "kv_heads", where), _positive(m, "dim", where),
+                      _positive(m, "vdim", where), float(m["scale"]), sink=True)
+    if a.heads % a.kv_heads:
+        raise ValueError(f"{where}: heads must be a multiple of kv_heads")
+    mask = m.get("mask")
+    if mask:
+        a.window, a.keep_first = _positive(mask, "size", where + ".mask"), int(mask.get("keep_first", 0))
+    rot = m.get("rot")
+    if rot and int(rot["dims"]) > 0:
+        dims = int(rot["dims"])
+        if dims % 2 or dims > a.dim:
+            raise ValueError(f"{where}.rot.dims must be even and at most dim")
+        sc = rot.get("scaling")
+        a.rotary = RotarySpec(dims, float(rot["base"]), {
+            "rope_type": "llama3", "factor": float(sc["factor"]), "low_freq_factor": float(sc["low"]),
+            "high_freq_factor": float(sc["high"]), "original_max_position_embeddings": float(sc["original"])} if sc else None)
+    return a
+
+
+def lenolix_config(hf: dict, generation: Optional[dict] = None) -> ModelConfig:
+    """config.json of a Lenolix model: ``vocab``, ``width``, ``norm.eps``, ``embedding`` (``scale``, ``bigram``), ``layers``
+    (``type``, ``mixer``, ``mlp``) and ``loop``."""
+    layers = []
+    for i, e in enumerate(hf["layers"]):
+        where = f"layers[{i}]"
+        if e.get("type", "attention") != "attention":
+            raise ValueError(f"{where}: unknown mixer type {e['type']!r}")
+        mlp = e.get("mlp")
+        if mlp and mlp.get("kind", "dense") != "dense":
+            raise ValueError(f"{where}: unknown feed-forward kind {mlp['kind']!r}")
+        layers.append(LayerSpec(_lenolix_attention(e["mixer"], where + ".mixer"),
+                                MlpSpec(_positive(mlp, "ff", where + ".mlp"), float(mlp["limit"])) if mlp else None))
+    if not layers:
+        raise ValueError("layers is empty")
+    emb = hf.get("embedding") or {}
+    first = layers[0].mixer
+    c = ModelConfig(model_type="lenolix", hf_model_type="lenolix", hidden_size=_positive(hf, "width", "config"), num_layers=len(layers),
+                    num_heads=first.heads, num_kv_heads=first.kv_heads, head_dim=first.dim, v_head_dim=first.vdim,
+                    intermediate_size=max([s.mlp.size for s in layers if s.mlp] or [0]), vocab_size=_positive(hf, "vocab", "config"),
+                    rms_norm_eps=float(hf["norm"]["eps"]), norm_type="layernorm", tie_word_embeddings=True,
+                    position_embedding="per_layer",
+                    emb_scale=float(emb.get("scale", 1.0)), layer_specs=layers)
+    c.max_position_embeddings = c.max_token_len = int(hf.get("max_position_embeddings", _UNBOUNDED_POSITIONS))
+    if emb.get("bigram"):
+        b = emb["bigram"]
+        c.pair_embedding = PairEmbeddingSpec(_positive(b, "buckets", "embedding.bigram"), int(b["mul_prev"]), int(b["mul_cur"]))
+    loop = hf.get("loop")
+    if loop:
+        c.loop = LoopSpec(int(loop["start"]), int(loop["stop"]), _positive(loop, "times", "loop"))
+        if not 0 <= c.loop.start < c.loop.stop <= len(layers):
+            raise ValueError("loop must cover at least one of the layers")
+    eos = (generation or {}).get("eos_token_id", hf.get("eos_token_id"))
+    if eos is not None:
+        c.eos_token_ids = [int(e) for e in (eos if isinstance(eos, (list, tuple)) else [eos])]
     return c
 
 

@@ -186,6 +186,7 @@ PYBIND11_MODULE(_ksana_engine, m) {
       .def_property_readonly("q_lens", [](const StepPlan& p) { return ToArray(p.q_lens); })
       .def_property_readonly("kv_lens", [](const StepPlan& p) { return ToArray(p.kv_lens); })
       .def_property_readonly("input_ids", [](const StepPlan& p) { return ToArray(p.input_ids); })
+      .def_property_readonly("prev_ids", [](const StepPlan& p) { return ToArray(p.prev_ids); })
       .def_property_readonly("positions", [](const StepPlan& p) { return ToArray(p.positions); })
       .def_property_readonly("slots", [](const StepPlan& p) { return ToArray(p.slots); })
       .def_property_readonly("cu_q", [](const StepPlan& p) { return ToArray(p.cu_q); })
@@ -270,6 +271,16 @@ PYBIND11_MODULE(_ksana_engine, m) {
         }
         return EventsToList(ev);
       }, py::arg("plan"), py::arg("tokens"), py::arg("parents") = std::vector<int64_t>())
+      .def("open_given", &Scheduler::OpenGiven)
+      .def("plan_given", [](Scheduler& s, const std::vector<std::tuple<int64_t, std::vector<int>, std::vector<int>>>& in) {
+        // entries (seq_id, tokens, wanted places) -> (code, message, plan, wanted rows' places in the entries' order)
+        std::vector<Scheduler::GivenEntry> entries;
+        for (auto& e : in) entries.push_back({std::get<0>(e), std::get<1>(e), std::get<2>(e)});
+        StepPlan p;
+        std::vector<int> order;
+        const Status st = s.PlanGiven(entries, &p, &order);
+        return py::make_tuple(static_cast<int>(st.code), st.message, std::move(p), ToArray(order));
+      })
       .def("can_pipeline", &Scheduler::CanPipeline)
       .def("advance", [](Scheduler& s, const StepPlan& plan) {
         py::gil_scoped_release rel;

@@ -16,7 +16,7 @@ inline int CeilMul(int bs, float thr) { return static_cast<int>(std::ceil(static
 // ---------------------------------------------------------------------------------- StepPlan
 std::vector<int32_t> StepPlan::Pack() const {
   // header: magic, nseq, ntok, num_multi, num_single, num_multi_tokens, max_q_len, max_blocks,
-  //         nsample, nswap_out, nswap_in, ncopies, npre_copies, sample_k, sample_full, reserved
+  //         nsample, nswap_out, nswap_in, ncopies, npre_copies, sample_k, sample_full, has_prev_ids
   std::vector<int32_t> out;
   const int nseq = static_cast<int>(seq_ids.size());
   out.reserve(16 + nseq * (4 + max_blocks) + num_tokens * 3 + 64);
@@ -35,7 +35,8 @@ std::vector<int32_t> StepPlan::Pack() const {
   out.push_back(static_cast<int>(pre_copies.size()));
   out.push_back(sample_k);
   out.push_back(sample_full ? 1 : 0);
-  out.push_back(0);
+  const bool has_prev = static_cast<int>(prev_ids.size()) == num_tokens;
+  out.push_back(has_prev ? 1 : 0);
   auto put = [&](const std::vector<int>& v) { out.insert(out.end(), v.begin(), v.end()); };
   auto put64 = [&](const std::vector<int64_t>& v) {
     for (int64_t x : v) { out.push_back(static_cast<int32_t>(x & 0xffffffff)); out.push_back(static_cast<int32_t>(x >> 32)); }
@@ -47,6 +48,7 @@ std::vector<int32_t> StepPlan::Pack() const {
   for (auto& s : swap_in) { out.push_back(s.device_block); out.push_back(s.host_block); }
   for (auto& c : copies) { out.push_back(c.src); out.push_back(c.dst); out.push_back(c.pos_delta); }
   for (auto& c : pre_copies) { out.push_back(c.src); out.push_back(c.dst); out.push_back(c.pos_delta); }
+  if (has_prev) put(prev_ids);
   return out;
 }
 
@@ -63,7 +65,7 @@ bool StepPlan::Unpack(const int32_t* d, size_t n, StepPlan* p) {
     return false;
   size_t need = 16 + static_cast<size_t>(p->num_tokens) * 3 + (nseq + 1) + nseq * 2 +
                 static_cast<size_t>(nseq) * p->max_blocks + nsample + 2 * nseq + 2 * nsample + 2 * nso + 2 * nsi +
-                3 * ncp + 3 * npre;
+                3 * ncp + 3 * npre + (d[15] ? static_cast<size_t>(p->num_tokens) : 0);
   if (n < need) return false;
   const int32_t* c = d + 16;
   auto get = [&](std::vector<int>* v, size_t cnt) { v->assign(c, c + cnt); c += cnt; };
@@ -83,6 +85,7 @@ bool StepPlan::Unpack(const int32_t* d, size_t n, StepPlan* p) {
   for (int i = 0; i < nsi; ++i) { p->swap_in.push_back({c[0], c[1]}); c += 2; }
   for (int i = 0; i < ncp; ++i) { p->copies.push_back({c[0], c[1], c[2]}); c += 3; }
   for (int i = 0; i < npre; ++i) { p->pre_copies.push_back({c[0], c[1], c[2]}); c += 3; }
+  if (d[15]) get(&p->prev_ids, p->num_tokens);
   return true;
 }
 
@@ -273,19 +276,116 @@ void Scheduler::PreemptLocked(const SeqPtr& v, StepPlan* plan) {
   ++stats_.preempt_recompute;
 }
 
-void Scheduler::EmitSequence(const SeqPtr& s, StepPlan* plan) {
+void Scheduler::EmitRows(const Sequence& s, StepPlan* plan) {
   const int B = cfg_.block_token_num;
-  plan->seq_ids.push_back(s->seq_id);
-  plan->q_lens.push_back(s->chunk);
-  plan->kv_lens.push_back(s->kv_cached + s->chunk);
-  for (int i = 0; i < s->chunk; ++i) {
-    const int pos = s->kv_cached + i;
-    plan->input_ids.push_back(s->tokens[pos]);
+  plan->seq_ids.push_back(s.seq_id);
+  plan->q_lens.push_back(s.chunk);
+  plan->kv_lens.push_back(s.kv_cached + s.chunk);
+  for (int i = 0; i < s.chunk; ++i) {
+    const int pos = s.kv_cached + i;
+    plan->input_ids.push_back(s.tokens[pos]);
+    // only the last element of `tokens` can be a placeholder, so the token before a row is always a real one
+    plan->prev_ids.push_back(pos > 0 ? s.tokens[pos - 1] : -1);
     plan->positions.push_back(pos);
-    plan->slots.push_back(s->blocks[pos / B] * B + pos % B);
+    plan->slots.push_back(s.blocks[pos / B] * B + pos % B);
   }
-  plan->num_tokens += s->chunk;
-  plan->max_q_len = std::max(plan->max_q_len, s->chunk);
+  plan->num_tokens += s.chunk;
+  plan->max_q_len = std::max(plan->max_q_len, s.chunk);
+}
+
+void Scheduler::FillTable(const std::vector<SeqPtr>& multi, const std::vector<SeqPtr>& single, StepPlan* plan) {
+  int max_blocks = 1;
+  for (auto& s : multi) max_blocks = std::max(max_blocks, static_cast<int>(s->blocks.size()));
+  for (auto& s : single) max_blocks = std::max(max_blocks, static_cast<int>(s->blocks.size()));
+  plan->max_blocks = max_blocks;
+  plan->block_table.assign(static_cast<size_t>(plan->seq_ids.size()) * max_blocks, 0);
+  size_t row = 0;
+  auto fill = [&](const SeqPtr& s) {
+    std::copy(s->blocks.begin(), s->blocks.end(), plan->block_table.begin() + row * max_blocks);
+    ++row;
+  };
+  for (auto& s : multi) fill(s);
+  for (auto& s : single) fill(s);
+}
+
+int64_t Scheduler::OpenGiven(int64_t req_id) {
+  std::lock_guard<std::mutex> g(mu_);
+  auto s = std::make_shared<Sequence>();
+  s->seq_id = next_seq_id_++;
+  s->req_id = req_id;
+  s->cfg = std::make_shared<SamplingConfig>();
+  s->arrive_ms = NowMs();
+  s->state = SeqState::RUNNING;
+  by_id_[s->seq_id] = s;
+  return s->seq_id;
+}
+
+Status Scheduler::PlanGiven(const std::vector<GivenEntry>& entries, StepPlan* plan, std::vector<int>* order) {
+  std::lock_guard<std::mutex> g(mu_);
+  plan->Clear();
+  order->clear();
+  const int B = cfg_.block_token_num;
+  std::vector<SeqPtr> seqs;
+  std::vector<int> need(caches_.size(), 0);
+  for (auto& e : entries) {
+    auto it = by_id_.find(e.seq_id);
+    if (it == by_id_.end() || it->second->state != SeqState::RUNNING)
+      return Status(RET_INVALID_ARGUMENT, "unknown sequence " + std::to_string(e.seq_id));
+    if (e.tokens.empty()) return Status(RET_INVALID_ARGUMENT, "an entry without tokens");
+    for (int w : e.want)
+      if (w < 0 || w >= static_cast<int>(e.tokens.size()))
+        return Status(RET_INVALID_ARGUMENT, "a wanted row outside its entry");
+    if (std::find(seqs.begin(), seqs.end(), it->second) != seqs.end())
+      return Status(RET_INVALID_ARGUMENT, "a sequence named twice in one step");
+    const Sequence& s = *it->second;
+    const int total = static_cast<int>(s.tokens.size() + e.tokens.size());
+    if (total > cfg_.max_token_len)
+      return Status(RET_EXCEED_LENGTH, "sequence longer than max_token_len " + std::to_string(cfg_.max_token_len));
+    need[RankOf(s)] += std::max(0, CeilDiv(total, B) - static_cast<int>(s.blocks.size()));
+    seqs.push_back(it->second);
+  }
+  for (size_t r = 0; r < caches_.size(); ++r)
+    if (need[r] > caches_[r]->usable_blocks())
+      return Status(RET_OUT_OF_MEMORY, "not enough KV cache blocks for this step");
+  std::vector<SeqPtr> multi, single;
+  std::vector<size_t> at;                                        // plan order -> entry
+  std::vector<int> first(entries.size() + 1, 0);                 // where an entry's wanted rows start, entries' order
+  for (size_t i = 0; i < entries.size(); ++i) {
+    Sequence& s = *seqs[i];
+    s.tokens.insert(s.tokens.end(), entries[i].tokens.begin(), entries[i].tokens.end());
+    s.prompt_len = static_cast<int>(s.tokens.size());
+    s.chunk = static_cast<int>(entries[i].tokens.size());
+    CacheOf(s).Allocate(BlocksNeeded(s), &s.blocks);
+    first[i + 1] = first[i] + static_cast<int>(entries[i].want.size());
+  }
+  for (int pass = 0; pass < 2; ++pass)
+    for (size_t i = 0; i < entries.size(); ++i)
+      if ((seqs[i]->chunk > 1) == (pass == 0)) {
+        (pass == 0 ? multi : single).push_back(seqs[i]);
+        at.push_back(i);
+      }
+  plan->cu_q.push_back(0);
+  for (size_t i : at) {
+    const int row0 = plan->num_tokens;
+    EmitRows(*seqs[i], plan);
+    plan->cu_q.push_back(plan->num_tokens);
+    for (size_t k = 0; k < entries[i].want.size(); ++k) {
+      plan->sample_rows.push_back(row0 + entries[i].want[k]);
+      order->push_back(first[i] + static_cast<int>(k));
+    }
+    if (seqs[i]->chunk > 1) plan->num_multi_tokens = plan->num_tokens;
+  }
+  plan->num_multi = static_cast<int>(multi.size());
+  plan->num_single = static_cast<int>(single.size());
+  plan->sample_full = true;                                      // the caller reads whole logits rows
+  FillTable(multi, single, plan);
+  ++stats_.steps;
+  stats_.step_tokens += plan->num_tokens;
+  return Status();
+}
+
+void Scheduler::EmitSequence(const SeqPtr& s, StepPlan* plan) {
+  EmitRows(*s, plan);
   if (s->kv_cached + s->chunk == static_cast<int>(s->tokens.size())) {
     const int row = plan->num_tokens - 1;
     plan->sample_seq_ids.push_back(s->seq_id);
@@ -468,18 +568,7 @@ bool Scheduler::Schedule(StepPlan* plan) {
   plan->num_multi_tokens = plan->num_tokens;
   for (auto& s : single) { EmitSequence(s, plan); plan->cu_q.push_back(plan->num_tokens); }
   plan->num_single = static_cast<int>(single.size());
-  int max_blocks = 1;
-  for (auto& s : multi) max_blocks = std::max(max_blocks, static_cast<int>(s->blocks.size()));
-  for (auto& s : single) max_blocks = std::max(max_blocks, static_cast<int>(s->blocks.size()));
-  plan->max_blocks = max_blocks;
-  plan->block_table.assign(static_cast<size_t>(plan->seq_ids.size()) * max_blocks, 0);
-  size_t row = 0;
-  auto fill = [&](const SeqPtr& s) {
-    std::copy(s->blocks.begin(), s->blocks.end(), plan->block_table.begin() + row * max_blocks);
-    ++row;
-  };
-  for (auto& s : multi) fill(s);
-  for (auto& s : single) fill(s);
+  FillTable(multi, single, plan);
 
   if (!pending_copies_.empty()) {
     // Forks decided after the previous step: their tail-block copies run first, before this step's swap-outs,

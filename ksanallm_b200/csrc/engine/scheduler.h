@@ -87,6 +87,7 @@ struct StepPlan {
   std::vector<int64_t> seq_ids;            // multi-token sequences first, then single-token ones
   std::vector<int> q_lens, kv_lens;
   std::vector<int> input_ids, positions, slots, cu_q;
+  std::vector<int> prev_ids;               // the token before each row's token in its sequence (-1: the first token)
   std::vector<int> block_table; int max_blocks = 0;
   std::vector<int64_t> sample_seq_ids;     // sequences that sample this step ...
   std::vector<int> sample_rows;            // ... and the token row whose logits they use
@@ -161,6 +162,16 @@ class Scheduler {
   void Advance(const StepPlan& plan);
   void Resolve(const StepPlan& plan, const std::vector<int>& tokens, std::vector<SeqEvent>* events);
 
+  // Given-token stepping (replaying a trace, scoring given text): the caller names each step's sequences, their next
+  // tokens and the rows whose logits it wants, instead of the queues and the sampler. The sequences use the same
+  // block pool and the same StepPlan as generation; Advance(plan) moves their cached lengths forward after the step
+  // and FinishSequence gives their blocks back. They never enter the running queue, so Schedule() leaves them alone.
+  int64_t OpenGiven(int64_t req_id);
+  struct GivenEntry { int64_t seq_id; std::vector<int> tokens; std::vector<int> want; };
+  // RET_OUT_OF_MEMORY when the pool cannot hold the step's tokens; nothing is changed in that case. ``order``: for
+  // every wanted row of the plan (plan rows put multi-token entries first), its index in the entries' order.
+  Status PlanGiven(const std::vector<GivenEntry>& entries, StepPlan* plan, std::vector<int>* order);
+
   // Runtime hooks: stop strings and structured output need the tokenizer, which lives outside.
   void FinishSequence(int64_t seq_id, int keep_tokens, int code, const std::string& message,
                       std::vector<SeqEvent>* events);
@@ -181,6 +192,8 @@ class Scheduler {
   int BlocksNeeded(const Sequence& s) const;
   bool CheckFinishLocked(const SeqPtr& s, int token, std::vector<SeqEvent>* ev);
   void EmitSequence(const SeqPtr& s, StepPlan* plan);
+  void EmitRows(const Sequence& s, StepPlan* plan);
+  void FillTable(const std::vector<SeqPtr>& multi, const std::vector<SeqPtr>& single, StepPlan* plan);
   int StepTokenCap(int num_decodes) const;
 
   CacheManager& CacheOf(const Sequence& s) { return *caches_[static_cast<size_t>(s.seq_id % static_cast<int64_t>(caches_.size()))]; }

@@ -18,6 +18,12 @@
 //
 // FP8 (e4m3) caches are dequantised with a per-layer scale while staging tiles.
 //
+// Head sizes: a kernel is compiled for a padded head size DP (64, 128, 192, 256); the real query/key size D and value
+// size Dv are run-time values up to DP (multiples of 8), padded with zeros in shared memory only (TMA fills the
+// columns past the row's end). K and V lie in panels of their own: [block][Hkv][block_tokens][D] and [...][Dv].
+// Sliding window: position i sees j <= i with i - j < window or j < keep; tiles between the kept tokens and the
+// window are not visited. Sink: an extra logit per head in the softmax denominator, without a value.
+//
 // Functional counterpart of the reference's decode kernels
 // (3rdparty/LLM_kernels/csrc/kernels/nvidia/paged_attention/paged_attention.cu:81-640)
 // and of its FlashAttention-2 call (src/ksana_llm/kernels/nvidia/kernel_wrapper.cpp:437-588),
@@ -40,14 +46,17 @@ enum KvMode { kKvCpAsync = 0, kKvFp8 = 1, kKvTma = 2 };
 typedef __nv_bfloat16 bf16;
 constexpr int kTileTok = 64;     // KV tokens per shared-memory tile
 constexpr int kAttnThreads = 128;
-constexpr int kKvStages = 3;      // K/V tile ring: two tiles in flight while one is consumed
+__host__ __device__ constexpr int kv_stages(int dp) { return dp <= 192 ? 3 : 2; }    // K/V tile ring: all but one tile in flight while one is consumed
 
 struct AttnParams {
   const bf16* q; long long q_stride;     // [T, q_stride] ; head h at column h*D
   bf16* out; long long out_stride;       // [T, out_stride]
-  const void* cache;                     // layer base: [block][2][Hkv][block_tokens][D]
+  const void* kc; const void* vc;        // panels of block 0: K [Hkv][block_tokens][D], V [Hkv][block_tokens][Dv]
   long long block_stride;                // elements between blocks
   int block_tokens;
+  int D, Dv;                             // real head sizes
+  int window, keep;                      // sliding window in tokens (0: none) and first tokens every row sees
+  const float* sinks;                    // [Hq] logits added to the softmax denominator, or null
   const int* block_table; int table_stride;   // [B][table_stride]
   const int* cu_q;                       // [B+1] query row offsets (prefill) or null (decode: row = s)
   const int* kv_lens;                    // [B]
@@ -82,6 +91,18 @@ __device__ __forceinline__ void store_head_row_q(const AttnParams& p, int s, int
   p.outq[(static_cast<size_t>(s) * p.Hq + head) * 128 + d] = q;
   if (d == 0) p.oscale[static_cast<size_t>(head) * p.oscale_ld + s] = sc;
 }
+
+// Tiles of `tile` tokens a range of rows visits, in order: those that hold kept first tokens, then the window's. `lo` is
+// the first position inside the window of the range's first row, `total` the tile count up to the last visible token.
+struct TileRange { int nkeep, first, count; };
+__device__ __forceinline__ TileRange visited_tiles(int lo, int keep, int total, int tile) {
+  TileRange r;
+  r.first = lo > 0 ? lo / tile : 0;
+  r.nkeep = min((keep + tile - 1) / tile, r.first);
+  r.count = r.nkeep + total - r.first;
+  return r;
+}
+__device__ __forceinline__ int tile_at(const TileRange& r, int i) { return i < r.nkeep ? i : r.first + i - r.nkeep; }
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
 __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
@@ -122,16 +143,18 @@ template <int D, bool FP8>
 __device__ __forceinline__ void load_kv_tile(bf16* dst, const AttnParams& p, const int* table, int g, int which,
                                              int tok0, int kv_len, float dq) {
   constexpr int CH = D / 8;
+  const int rd = which ? p.Dv : p.D;
+  const void* base = which ? p.vc : p.kc;
   for (int i = threadIdx.x; i < kTileTok * CH; i += kAttnThreads) {
     const int r = i / CH, c = i % CH;
     const int tok = tok0 + r;
     bf16* d = tile_ptr<D, kTileTok>(dst, r, c);
-    if (tok < kv_len) {
+    if (tok < kv_len && c * 8 < rd) {
       const int blk = table[tok / p.block_tokens];
       const size_t off = static_cast<size_t>(blk) * p.block_stride +
-                         ((static_cast<size_t>(which) * p.Hkv + g) * p.block_tokens + tok % p.block_tokens) * D + c * 8;
+                         (static_cast<size_t>(g) * p.block_tokens + tok % p.block_tokens) * rd + c * 8;
       if (FP8) {
-        const uint2 raw = *reinterpret_cast<const uint2*>(static_cast<const uint8_t*>(p.cache) + off);
+        const uint2 raw = *reinterpret_cast<const uint2*>(static_cast<const uint8_t*>(base) + off);
         const uint8_t* b = reinterpret_cast<const uint8_t*>(&raw);
         uint4 o;
         uint32_t* ow = reinterpret_cast<uint32_t*>(&o);
@@ -143,7 +166,7 @@ __device__ __forceinline__ void load_kv_tile(bf16* dst, const AttnParams& p, con
         }
         *reinterpret_cast<uint4*>(d) = o;
       } else {
-        cp_async16(d, static_cast<const bf16*>(p.cache) + off);
+        cp_async16(d, static_cast<const bf16*>(base) + off);
       }
     } else {
       *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
@@ -155,20 +178,20 @@ __device__ __forceinline__ void load_kv_tile(bf16* dst, const AttnParams& p, con
 // 64-column panel. Tokens past kv_len inside the last block are loaded as they are (finite cache contents)
 // and masked by the softmax; blocks past the sequence are not loaded at all.
 template <int D>
-__device__ __forceinline__ void tma_issue_kv(bf16* ks, bf16* vs, uint64_t* bar, const CUtensorMap* map, const AttnParams& p,
-                                             const int* table, int g, int tok0, int kv_len, long long rows_per_block) {
+__device__ __forceinline__ void tma_issue_kv(bf16* ks, bf16* vs, uint64_t* bar, const CUtensorMap* kmap, const CUtensorMap* vmap,
+                                             const AttnParams& p, const int* table, int g, int tok0, int kv_len) {
   const int bt = p.block_tokens;
   const int nblk = min(kTileTok / bt, (kv_len - tok0 + bt - 1) / bt);
   constexpr int PANELS = D / 64;
   mbar_expect_tx(bar, static_cast<uint32_t>(nblk) * 2 * PANELS * bt * 128);
   for (int b = 0; b < nblk; ++b) {
-    const long long row0 = static_cast<long long>(table[tok0 / bt + b]) * rows_per_block;
+    const int blk = table[tok0 / bt + b];
 #pragma unroll
     for (int which = 0; which < 2; ++which) {
       bf16* dst = which ? vs : ks;
-      const int y = static_cast<int>(row0 + (static_cast<long long>(which) * p.Hkv + g) * bt);
 #pragma unroll
-      for (int h = 0; h < PANELS; ++h) tma_load_2d(dst + h * (kTileTok * 64) + b * bt * 64, map, bar, h * 64, y);
+      for (int h = 0; h < PANELS; ++h)      // columns past the row's end arrive as zeros
+        tma_load_3d(dst + h * (kTileTok * 64) + b * bt * 64, which ? vmap : kmap, bar, h * 64, g * bt, blk);
     }
   }
 }
@@ -229,11 +252,12 @@ __device__ __forceinline__ void warp_pv(float (&o)[D / 8][4], const float (&s)[N
 }
 
 // Mask + online-softmax update for one warp's 16 x (NT*8) score tile.
-// Rows lane/4 and lane/4+8; limit[i] = last visible kv position of that row (-1 = row inactive).
+// Rows lane/4 and lane/4+8; limit[i] = last visible kv position of that row (-1 = row inactive), lo[i] = first position
+// inside its window (tokens below `keep` are seen as well).
 template <int D, int NT>
 __device__ __forceinline__ void softmax_update(float (&s)[NT][4], float (&o)[D / 8][4], float (&m)[2], float (&l)[2],
-                                               const int (&limit)[2], const float (&slope)[2], int tok0, int lane,
-                                               float scale_log2) {
+                                               const int (&limit)[2], const int (&lo)[2], int keep, const float (&slope)[2],
+                                               int tok0, int lane, float scale_log2) {
   float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
   for (int j = 0; j < NT; ++j) {
@@ -243,7 +267,7 @@ __device__ __forceinline__ void softmax_update(float (&s)[NT][4], float (&o)[D /
       const int tok = tok0 + j * 8 + (lane & 3) * 2 + (e & 1);
       float v = s[j][e] * scale_log2;
       if (slope[i] != 0.f) v += slope[i] * 1.44269504f * static_cast<float>(tok - limit[i]);
-      v = tok <= limit[i] ? v : -INFINITY;
+      v = (tok <= limit[i] && (tok >= lo[i] || tok < keep)) ? v : -INFINITY;
       s[j][e] = v;
       mx[i] = fmaxf(mx[i], v);
     }
@@ -275,11 +299,17 @@ __device__ __forceinline__ void softmax_update(float (&s)[NT][4], float (&o)[D /
   }
 }
 
+// exp(sink - m) of the softmax denominator; m is the row's reference maximum in the log2 domain
+__device__ __forceinline__ float sink_term(const AttnParams& p, int head, float m) {
+  return (p.sinks && m != -INFINITY) ? exp2f(p.sinks[head] * 1.44269504f - m) : 0.f;
+}
+
 // ----------------------------------------------------------------------------- prefill
 template <int D, int MODE>
 __global__ void __launch_bounds__(kAttnThreads)
-paged_prefill_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnParams p, const long long rows_per_block) {
+paged_prefill_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, const AttnParams p) {
   constexpr bool FP8 = MODE == kKvFp8;
+  constexpr int kKvStages = kv_stages(D);
   extern __shared__ uint8_t smem_attn_raw[];
   uint8_t* smem_attn = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_attn_raw) + 1023) & ~uintptr_t(1023));
   __shared__ uint64_t full_bar[kKvStages];
@@ -304,16 +334,18 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnParam
     const int r = i / CH, c = i % CH;
     const int vr = row0 + r;
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (vr < q_len * G) {
+    if (vr < q_len * G && c * 8 < p.D) {
       const int tok = vr / G, head = g * G + vr % G;
-      v = *reinterpret_cast<const uint4*>(p.q + static_cast<size_t>(q0 + tok) * p.q_stride + head * D + c * 8);
+      v = *reinterpret_cast<const uint4*>(p.q + static_cast<size_t>(q0 + tok) * p.q_stride + head * p.D + c * 8);
     }
     *reinterpret_cast<uint4*>(tile_ptr<D, 64>(qs, r, c)) = v;
   }
   // causal bound of this CTA's rows
   const int last_row = min(row0 + 63, q_len * G - 1);
   const int kv_end = min(kv_len, past + last_row / G + 1);
-  const int ntiles = (kv_end + kTileTok - 1) / kTileTok;
+  const TileRange tiles = visited_tiles(p.window > 0 ? past + row0 / G - p.window + 1 : 0, p.keep, (kv_end + kTileTok - 1) / kTileTok,
+                                        kTileTok);
+  const int ntiles = tiles.count;
 
   if (MODE == kKvTma && threadIdx.x == 0) {
     for (int i = 0; i < kKvStages; ++i) mbar_init(&full_bar[i], 1);
@@ -322,21 +354,20 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnParam
   }
   __syncthreads();
   auto issue = [&](int t) {      // cp.async modes always commit a group so that the wait counts stay uniform
-    const int st = t % kKvStages;
+    const int st = t % kKvStages, tok0 = tile_at(tiles, t) * kTileTok;
     if (MODE == kKvTma) {
       if (threadIdx.x == 0 && t < ntiles)
-        tma_issue_kv<D>(ks + st * kTileTok * D, vs + st * kTileTok * D, &full_bar[st], &kv_map, p, table, g,
-                        t * kTileTok, kv_len, rows_per_block);
+        tma_issue_kv<D>(ks + st * kTileTok * D, vs + st * kTileTok * D, &full_bar[st], &k_map, &v_map, p, table, g, tok0, kv_len);
       return;
     }
     if (t < ntiles) {
-      load_kv_tile<D, FP8>(ks + st * kTileTok * D, p, table, g, 0, t * kTileTok, kv_len, p.k_scale);
-      load_kv_tile<D, FP8>(vs + st * kTileTok * D, p, table, g, 1, t * kTileTok, kv_len, p.v_scale);
+      load_kv_tile<D, FP8>(ks + st * kTileTok * D, p, table, g, 0, tok0, kv_len, p.k_scale);
+      load_kv_tile<D, FP8>(vs + st * kTileTok * D, p, table, g, 1, tok0, kv_len, p.v_scale);
     }
     cp_commit();
   };
-  issue(0);
-  issue(1);
+#pragma unroll
+  for (int i = 0; i < kKvStages - 1; ++i) issue(i);
   __syncthreads();
 
   uint32_t qf[D / 16][4];
@@ -346,11 +377,12 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnParam
     const int c = kk * 2 + (lane >> 4);
     ldsm_x4(qf[kk], smem_addr(tile_ptr<D, 64>(qs, r, c)));
   }
-  int limit[2]; float slope[2];
+  int limit[2], lo[2]; float slope[2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int vr = row0 + warp * 16 + (lane >> 2) + i * 8;
     limit[i] = vr < q_len * G ? past + vr / G : -1;
+    lo[i] = p.window > 0 ? limit[i] - p.window + 1 : 0;
     slope[i] = (p.alibi && vr < q_len * G) ? p.alibi[g * G + vr % G] : 0.f;
   }
   float o[D / 8][4];
@@ -360,18 +392,18 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnParam
 
   bool ok = true;
   for (int t = 0; t < ntiles; ++t) {
-    const int buf = t % kKvStages;
+    const int buf = t % kKvStages, tok0 = tile_at(tiles, t) * kTileTok;
     if (MODE == kKvTma) {
       if (!mbar_wait(&full_bar[buf], (t / kKvStages) & 1, &abort_word)) { ok = false; break; }
-      zero_v_tail<D>(vs + buf * kTileTok * D, kv_len - t * kTileTok);
+      zero_v_tail<D>(vs + buf * kTileTok * D, kv_len - tok0);
     } else {
-      cp_wait<1>();               // tile t has landed (only the newest group may still be in flight)
+      cp_wait<kKvStages - 2>();   // tile t has landed (only newer groups may still be in flight)
     }
     __syncthreads();              // ... for every thread, and everyone is done with tile t-1
-    issue(t + 2);                 // refill the stage tile t-1 used
+    issue(t + kKvStages - 1);     // refill the stage tile t-1 used
     float sc[8][4];
     warp_qk<D, 8>(sc, qf, ks + buf * kTileTok * D, 0, lane);
-    softmax_update<D, 8>(sc, o, m, l, limit, slope, t * kTileTok, lane, p.scale_log2);
+    softmax_update<D, 8>(sc, o, m, l, limit, lo, p.keep, slope, tok0, lane, p.scale_log2);
     warp_pv<D, 8>(o, sc, vs + buf * kTileTok * D, 0, lane);
   }
   if (!ok) {                      // a bounded wait gave up: leave the output untouched, report through the error word
@@ -388,21 +420,23 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnParam
     const int vr = row0 + warp * 16 + (lane >> 2) + i * 8;
     if (vr >= q_len * G) continue;
     const int tok = vr / G, head = g * G + vr % G;
+    l[i] += sink_term(p, head, m[i]);
     const float inv = l[i] > 0.f ? 1.f / l[i] : 0.f;
-    bf16* dst = p.out + static_cast<size_t>(q0 + tok) * p.out_stride + head * D + (lane & 3) * 2;
+    bf16* dst = p.out + static_cast<size_t>(q0 + tok) * p.out_stride + head * p.Dv + (lane & 3) * 2;
 #pragma unroll
     for (int n = 0; n < D / 8; ++n) {
-      *reinterpret_cast<uint32_t*>(dst + n * 8) = pack_bf16(o[n][2 * i] * inv, o[n][2 * i + 1] * inv);
+      if (n * 8 < p.Dv) *reinterpret_cast<uint32_t*>(dst + n * 8) = pack_bf16(o[n][2 * i] * inv, o[n][2 * i + 1] * inv);
     }
   }
 }
 
 // ------------------------------------------------------------------------------ decode
-// grid (Hkv, B, splits). Rows = the G query heads of kv head g (G <= 16), one new token each.
+// grid (Hkv x row groups, B, splits). Rows = up to 16 of the G query heads of kv head g, one new token each.
 template <int D, int MODE>
 __global__ void __launch_bounds__(kAttnThreads)
-paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnParams p, const long long rows_per_block) {
+paged_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, const AttnParams p) {
   constexpr bool FP8 = MODE == kKvFp8;
+  constexpr int kKvStages = kv_stages(D);
   extern __shared__ uint8_t smem_attn_raw[];
   uint8_t* smem_attn = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_attn_raw) + 1023) & ~uintptr_t(1023));
   __shared__ uint64_t full_bar[kKvStages];
@@ -415,12 +449,16 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnParams
 
   pdl_trigger();
   pdl_wait();
-  const int g = blockIdx.x, s = blockIdx.y, split = blockIdx.z;
-  const int G = p.Hq / p.Hkv;
+  const int GA = p.Hq / p.Hkv, groups = (GA + 15) / 16;
+  const int g = blockIdx.x / groups, head0 = g * GA + (blockIdx.x % groups) * 16;
+  const int G = min(16, (g + 1) * GA - head0);               // query heads of this CTA: head0 .. head0 + G
+  const int s = blockIdx.y, split = blockIdx.z;
   const int kv_len = p.kv_lens[s];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int* table = p.block_table + static_cast<size_t>(s) * p.table_stride;
-  const int total_tiles = (kv_len + kTileTok - 1) / kTileTok;
+  const int win_lo = p.window > 0 ? kv_len - p.window : 0;
+  const TileRange tiles = visited_tiles(win_lo, p.keep, (kv_len + kTileTok - 1) / kTileTok, kTileTok);
+  const int total_tiles = tiles.count;
   const int tiles_per = (total_tiles + p.num_splits - 1) / p.num_splits;
   const int t_begin = split * tiles_per, t_end = min(total_tiles, t_begin + tiles_per);
 
@@ -428,7 +466,8 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnParams
   for (int i = threadIdx.x; i < 16 * CH; i += kAttnThreads) {
     const int r = i / CH, c = i % CH;
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (r < G) v = *reinterpret_cast<const uint4*>(p.q + static_cast<size_t>(s) * p.q_stride + (g * G + r) * D + c * 8);
+    if (r < G && c * 8 < p.D)
+      v = *reinterpret_cast<const uint4*>(p.q + static_cast<size_t>(s) * p.q_stride + (head0 + r) * p.D + c * 8);
     *reinterpret_cast<uint4*>(tile_ptr<D, 16>(qs, r, c)) = v;
   }
   if (MODE == kKvTma && threadIdx.x == 0) {
@@ -438,21 +477,20 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnParams
   }
   __syncthreads();
   auto issue = [&](int t) {
-    const int st = (t - t_begin) % kKvStages;
+    const int st = (t - t_begin) % kKvStages, tok0 = tile_at(tiles, t) * kTileTok;
     if (MODE == kKvTma) {
       if (threadIdx.x == 0 && t < t_end)
-        tma_issue_kv<D>(ks + st * kTileTok * D, vs + st * kTileTok * D, &full_bar[st], &kv_map, p, table, g,
-                        t * kTileTok, kv_len, rows_per_block);
+        tma_issue_kv<D>(ks + st * kTileTok * D, vs + st * kTileTok * D, &full_bar[st], &k_map, &v_map, p, table, g, tok0, kv_len);
       return;
     }
     if (t < t_end) {
-      load_kv_tile<D, FP8>(ks + st * kTileTok * D, p, table, g, 0, t * kTileTok, kv_len, p.k_scale);
-      load_kv_tile<D, FP8>(vs + st * kTileTok * D, p, table, g, 1, t * kTileTok, kv_len, p.v_scale);
+      load_kv_tile<D, FP8>(ks + st * kTileTok * D, p, table, g, 0, tok0, kv_len, p.k_scale);
+      load_kv_tile<D, FP8>(vs + st * kTileTok * D, p, table, g, 1, tok0, kv_len, p.v_scale);
     }
     cp_commit();
   };
-  issue(t_begin);
-  issue(t_begin + 1);
+#pragma unroll
+  for (int i = 0; i < kKvStages - 1; ++i) issue(t_begin + i);
   __syncthreads();
   uint32_t qf[D / 16][4];
 #pragma unroll
@@ -461,12 +499,13 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnParams
     const int c = kk * 2 + (lane >> 4);
     ldsm_x4(qf[kk], smem_addr(tile_ptr<D, 16>(qs, r, c)));
   }
-  int limit[2]; float slope[2];
+  int limit[2], lo[2]; float slope[2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int r = (lane >> 2) + i * 8;
     limit[i] = r < G ? kv_len - 1 : -1;
-    slope[i] = (p.alibi && r < G) ? p.alibi[g * G + r] : 0.f;
+    lo[i] = win_lo;
+    slope[i] = (p.alibi && r < G) ? p.alibi[head0 + r] : 0.f;
   }
   float o[D / 8][4];
 #pragma unroll
@@ -475,18 +514,18 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnParams
 
   bool ok = true;
   for (int t = t_begin; t < t_end; ++t) {
-    const int buf = (t - t_begin) % kKvStages;
+    const int buf = (t - t_begin) % kKvStages, tok0 = tile_at(tiles, t) * kTileTok;
     if (MODE == kKvTma) {
       if (!mbar_wait(&full_bar[buf], ((t - t_begin) / kKvStages) & 1, &abort_word)) { ok = false; break; }
-      zero_v_tail<D>(vs + buf * kTileTok * D, kv_len - t * kTileTok);
+      zero_v_tail<D>(vs + buf * kTileTok * D, kv_len - tok0);
     } else {
-      cp_wait<1>();
+      cp_wait<kKvStages - 2>();
     }
     __syncthreads();
-    issue(t + 2);
+    issue(t + kKvStages - 1);
     float sc[2][4];
     warp_qk<D, 2>(sc, qf, ks + buf * kTileTok * D, warp * 16, lane);
-    softmax_update<D, 2>(sc, o, m, l, limit, slope, t * kTileTok + warp * 16, lane, p.scale_log2);
+    softmax_update<D, 2>(sc, o, m, l, limit, lo, p.keep, slope, tok0 + warp * 16, lane, p.scale_log2);
     warp_pv<D, 2>(o, sc, vs + buf * kTileTok * D, warp * 16, lane);
   }
   cp_wait<0>();
@@ -514,8 +553,9 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnParams
     }
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < G * D; i += kAttnThreads) {
-    const int r = i / D, d = i % D;
+  const int Dv = p.Dv;
+  for (int i = threadIdx.x; i < G * Dv; i += kAttnThreads) {
+    const int r = i / Dv, d = i % Dv;
     float mm = -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; ++w) mm = fmaxf(mm, merge[(w * 16 + r) * MS + D]);
@@ -527,16 +567,17 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnParams
       acc += src[d] * f;
       ll += src[D + 1] * f;
     }
-    const int head = g * G + r;
+    const int head = head0 + r;
     if (p.num_splits == 1) {
+      ll += sink_term(p, head, mm);
       const float v = ll > 0.f ? acc / ll : 0.f;
       if constexpr (D == 128) {
-        if (p.outq) { store_head_row_q(p, s, head, d, v, red4); continue; }   // (D == blockDim: r is uniform per pass)
+        if (p.outq) { store_head_row_q(p, s, head, d, v, red4); continue; }   // (Dv == blockDim: r is uniform per pass)
       }
-      p.out[static_cast<size_t>(s) * p.out_stride + head * D + d] = __float2bfloat16(v);
+      p.out[static_cast<size_t>(s) * p.out_stride + head * Dv + d] = __float2bfloat16(v);
     } else {
       const size_t base = (static_cast<size_t>(s) * p.Hq + head) * p.num_splits + split;
-      p.part_o[base * D + d] = acc;
+      p.part_o[base * Dv + d] = acc;
       if (d == 0) { p.part_ml[base * 2] = mm; p.part_ml[base * 2 + 1] = ll; }
     }
   }
@@ -552,19 +593,22 @@ __global__ void decode_reduce_kernel(const AttnParams p) {
   const size_t base = (static_cast<size_t>(s) * p.Hq + head) * p.num_splits;
   float mm = -INFINITY;
   for (int k = 0; k < p.num_splits; ++k) mm = fmaxf(mm, p.part_ml[(base + k) * 2]);
-  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+  const float sink = sink_term(p, head, mm);
+  const int Dv = p.Dv;
+  for (int d = threadIdx.x; d < Dv; d += blockDim.x) {
     float acc = 0.f, ll = 0.f;
     for (int k = 0; k < p.num_splits; ++k) {
       const float mk = p.part_ml[(base + k) * 2];
       const float f = (mk == -INFINITY) ? 0.f : exp2f(mk - mm);
-      acc += p.part_o[(base + k) * D + d] * f;
+      acc += p.part_o[(base + k) * Dv + d] * f;
       ll += p.part_ml[(base + k) * 2 + 1] * f;
     }
+    ll += sink;
     const float v = ll > 0.f ? acc / ll : 0.f;
     if constexpr (D == 128) {
       if (p.outq) { store_head_row_q(p, s, head, d, v, red4); continue; }     // 128 threads: one pass, every thread in it
     }
-    p.out[static_cast<size_t>(s) * p.out_stride + head * D + d] = __float2bfloat16(v);
+    p.out[static_cast<size_t>(s) * p.out_stride + head * Dv + d] = __float2bfloat16(v);
   }
 }
 
@@ -584,29 +628,31 @@ static AttnEncodeFn attn_encode_fn() {
   return fn;
 }
 
-// The layer's cache seen as rows of D bf16 (row = one token of one head of K or V of one block); box = one
-// cache block's tokens x 64 columns, 128-byte swizzle.
-static bool make_kv_map(CUtensorMap* map, const void* cache, long long rows, int D, int block_tokens) {
+// A K or V panel of every block seen as [block][row = head x token][D] bf16; box = one cache block's tokens x 64 columns,
+// 128-byte swizzle. Columns past D arrive as zeros.
+static bool make_kv_map(CUtensorMap* map, const void* panel, long long block_stride, int num_blocks, int Hkv, int D, int block_tokens) {
   AttnEncodeFn enc = attn_encode_fn();
-  if (!enc || (reinterpret_cast<uintptr_t>(cache) & 15)) return false;
-  cuuint64_t dims[2] = {static_cast<cuuint64_t>(D), static_cast<cuuint64_t>(rows)};
-  cuuint64_t strides[1] = {static_cast<cuuint64_t>(D) * 2};
-  cuuint32_t box[2] = {64, static_cast<cuuint32_t>(block_tokens)};
-  cuuint32_t estr[2] = {1, 1};
-  return enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(cache), dims, strides, box, estr,
+  if (!enc || (reinterpret_cast<uintptr_t>(panel) & 15)) return false;
+  cuuint64_t dims[3] = {static_cast<cuuint64_t>(D), static_cast<cuuint64_t>(Hkv) * block_tokens, static_cast<cuuint64_t>(num_blocks)};
+  cuuint64_t strides[2] = {static_cast<cuuint64_t>(D) * 2, static_cast<cuuint64_t>(block_stride) * 2};
+  cuuint32_t box[3] = {64, static_cast<cuuint32_t>(block_tokens), 1};
+  cuuint32_t estr[3] = {1, 1, 1};
+  return enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(panel), dims, strides, box, estr,
              CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-static bool tma_ok(const AttnParams& p, int D) {
+// The maps of both panels, where the TMA path covers the cache (block sizes that divide a tile, 16-byte strides).
+static bool tma_maps(const AttnParams& p, int num_blocks, CUtensorMap* km, CUtensorMap* vm) {
   const int bt = p.block_tokens;
-  return (bt == 8 || bt == 16 || bt == 32 || bt == 64) && p.block_stride % D == 0;
+  if (!(bt == 8 || bt == 16 || bt == 32 || bt == 64) || p.block_stride % 8 || num_blocks <= 0) return false;
+  return make_kv_map(km, p.kc, p.block_stride, num_blocks, p.Hkv, p.D, bt) &&
+         make_kv_map(vm, p.vc, p.block_stride, num_blocks, p.Hkv, p.Dv, bt);
 }
 
 template <int D, int MODE>
-static int launch_prefill(const AttnParams& p, const CUtensorMap& map, long long rows_per_block, int B, int max_q_len,
-                          cudaStream_t st) {
-  const int smem = (64 + 2 * kKvStages * kTileTok) * D * 2 + 1024;
+static int launch_prefill(const AttnParams& p, const CUtensorMap& km, const CUtensorMap& vm, int B, int max_q_len, cudaStream_t st) {
+  const int smem = (64 + 2 * kv_stages(D) * kTileTok) * D * 2 + 1024;
   static bool set = false;
   if (!set) {
     if (cudaFuncSetAttribute(paged_prefill_kernel<D, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) !=
@@ -615,21 +661,22 @@ static int launch_prefill(const AttnParams& p, const CUtensorMap& map, long long
   }
   const int G = p.Hq / p.Hkv;
   dim3 grid((max_q_len * G + 63) / 64, p.Hkv, B);
-  paged_prefill_kernel<D, MODE><<<grid, kAttnThreads, smem, st>>>(map, p, rows_per_block);
+  paged_prefill_kernel<D, MODE><<<grid, kAttnThreads, smem, st>>>(km, vm, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
 template <int D, int MODE>
-static int launch_decode(const AttnParams& p, const CUtensorMap& map, long long rows_per_block, int B, cudaStream_t st) {
-  const int smem = (16 + 2 * kKvStages * kTileTok) * D * 2 + 1024;   // the fp32 merge area fits inside the K ring
+static int launch_decode(const AttnParams& p, const CUtensorMap& km, const CUtensorMap& vm, int B, cudaStream_t st) {
+  const int smem = (16 + 2 * kv_stages(D) * kTileTok) * D * 2 + 1024;   // the fp32 merge area fits inside the K and V rings
+  static_assert(4 * 16 * (D + 2) * 4 <= 2 * kv_stages(D) * kTileTok * D * 2, "merge area");
   static bool set = false;
   if (!set) {
     if (cudaFuncSetAttribute(paged_decode_kernel<D, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) !=
         cudaSuccess) return -3;
     set = true;
   }
-  dim3 grid(p.Hkv, B, p.num_splits);
-  if (launch_pdl(paged_decode_kernel<D, MODE>, grid, dim3(kAttnThreads), smem, st, map, p, rows_per_block) != cudaSuccess)
+  dim3 grid(p.Hkv * ((p.Hq / p.Hkv + 15) / 16), B, p.num_splits);
+  if (launch_pdl(paged_decode_kernel<D, MODE>, grid, dim3(kAttnThreads), smem, st, km, vm, p) != cudaSuccess)
     return -4;
   if (p.num_splits > 1) {
     if (launch_pdl(decode_reduce_kernel<D>, dim3(p.Hq, B), dim3(D < 128 ? 64 : 128), 0, st, p) != cudaSuccess) return -5;
@@ -638,69 +685,92 @@ static int launch_decode(const AttnParams& p, const CUtensorMap& map, long long 
 }
 
 template <int D>
-static int dispatch_prefill(const AttnParams& p, int cache_fp8, long long cache_rows, int B, int max_q_len, cudaStream_t st) {
-  CUtensorMap map{};
-  const long long rpb = p.block_stride / D;
-  if (cache_fp8) return launch_prefill<D, kKvFp8>(p, map, rpb, B, max_q_len, st);
-  if (tma_ok(p, D) && cache_rows > 0 && make_kv_map(&map, p.cache, cache_rows, D, p.block_tokens))
-    return launch_prefill<D, kKvTma>(p, map, rpb, B, max_q_len, st);
-  return launch_prefill<D, kKvCpAsync>(p, map, rpb, B, max_q_len, st);
+static int dispatch_prefill(const AttnParams& p, int cache_fp8, int num_blocks, int B, int max_q_len, cudaStream_t st) {
+  CUtensorMap km{}, vm{};
+  if constexpr (D <= 128) {
+    if (cache_fp8) return launch_prefill<D, kKvFp8>(p, km, vm, B, max_q_len, st);
+  } else if (cache_fp8) {
+    return -11;
+  }
+  if (tma_maps(p, num_blocks, &km, &vm)) return launch_prefill<D, kKvTma>(p, km, vm, B, max_q_len, st);
+  return launch_prefill<D, kKvCpAsync>(p, km, vm, B, max_q_len, st);
 }
 
 template <int D>
-static int dispatch_decode(const AttnParams& p, int cache_fp8, long long cache_rows, int B, cudaStream_t st) {
-  CUtensorMap map{};
-  const long long rpb = p.block_stride / D;
-  if (cache_fp8) return launch_decode<D, kKvFp8>(p, map, rpb, B, st);
-  if (tma_ok(p, D) && cache_rows > 0 && make_kv_map(&map, p.cache, cache_rows, D, p.block_tokens))
-    return launch_decode<D, kKvTma>(p, map, rpb, B, st);
-  return launch_decode<D, kKvCpAsync>(p, map, rpb, B, st);
+static int dispatch_decode(const AttnParams& p, int cache_fp8, int num_blocks, int B, cudaStream_t st) {
+  CUtensorMap km{}, vm{};
+  if constexpr (D <= 128) {
+    if (cache_fp8) return launch_decode<D, kKvFp8>(p, km, vm, B, st);
+  } else if (cache_fp8) {
+    return -11;
+  }
+  if (tma_maps(p, num_blocks, &km, &vm)) return launch_decode<D, kKvTma>(p, km, vm, B, st);
+  return launch_decode<D, kKvCpAsync>(p, km, vm, B, st);
+}
+
+// The padded head size that serves (D, Dv), 0 when none does.
+static int padded_head(int D, int Dv) {
+  const int m = D > Dv ? D : Dv;
+  if (D <= 0 || Dv <= 0 || D % 8 || Dv % 8 || m > 256) return 0;
+  return (m + 63) / 64 * 64;
 }
 
 }  // namespace ksana
 
 using namespace ksana;
 
-// Causal attention of new query rows against the paged cache (which already holds their K/V).
-// cache_rows: number of D-wide rows addressable from `cache` (blocks * block_stride / D); 0 disables the TMA path.
+// Causal attention of new query rows against the paged cache (which already holds their K/V). kc / vc: the layer's K and
+// V panels of block 0; block_stride: elements between blocks; num_blocks: blocks addressable (0 disables the TMA path).
+// window 0: no sliding window. sinks: [Hq] fp32 or null. D, Dv: query/key and value head size (out rows: Hq * Dv).
 extern "C" int ksana_paged_prefill(const void* q, long long q_stride, void* out, long long out_stride,
-                                   const void* cache, long long block_stride, int block_tokens, const int* block_table,
-                                   int table_stride, const int* cu_q, const int* kv_lens, const float* alibi, int B,
-                                   int max_q_len, int Hq, int Hkv, int D, float scale, int cache_fp8, float k_scale,
-                                   float v_scale, long long cache_rows, int* err, cudaStream_t st) {
+                                   const void* kc, const void* vc, long long block_stride, int block_tokens,
+                                   const int* block_table, int table_stride, const int* cu_q, const int* kv_lens,
+                                   const float* alibi, const float* sinks, int B, int max_q_len, int Hq, int Hkv, int D, int Dv,
+                                   int window, int keep, float scale, int cache_fp8, float k_scale, float v_scale,
+                                   int num_blocks, int* err, cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0) return 0;
-  if (Hq % Hkv) return -10;
+  if (Hkv <= 0 || Hq % Hkv || q_stride % 8 || (reinterpret_cast<uintptr_t>(q) & 15)) return -10;
   AttnParams p{};
   p.q = (const bf16*)q; p.q_stride = q_stride; p.out = (bf16*)out; p.out_stride = out_stride;
-  p.cache = cache; p.block_stride = block_stride; p.block_tokens = block_tokens;
+  p.kc = kc; p.vc = vc; p.block_stride = block_stride; p.block_tokens = block_tokens; p.D = D; p.Dv = Dv;
+  p.window = window; p.keep = window > 0 ? keep : 0; p.sinks = sinks;
   p.block_table = block_table; p.table_stride = table_stride; p.cu_q = cu_q; p.kv_lens = kv_lens; p.alibi = alibi;
   p.Hq = Hq; p.Hkv = Hkv; p.scale_log2 = scale * 1.44269504f; p.k_scale = k_scale; p.v_scale = v_scale;
   p.num_splits = 1; p.err = err;
-  if (D == 128) return dispatch_prefill<128>(p, cache_fp8, cache_rows, B, max_q_len, st);
-  if (D == 64) return dispatch_prefill<64>(p, cache_fp8, cache_rows, B, max_q_len, st);
+  switch (padded_head(D, Dv)) {
+    case 64: return dispatch_prefill<64>(p, cache_fp8, num_blocks, B, max_q_len, st);
+    case 128: return dispatch_prefill<128>(p, cache_fp8, num_blocks, B, max_q_len, st);
+    case 192: return dispatch_prefill<192>(p, cache_fp8, num_blocks, B, max_q_len, st);
+    case 256: return dispatch_prefill<256>(p, cache_fp8, num_blocks, B, max_q_len, st);
+  }
   return -11;
 }
 
-// One new token per sequence. workspace: part_o [B*Hq*splits*D] fp32, part_ml [B*Hq*splits*2] fp32 (splits > 1).
+// One new token per sequence. workspace: part_o [B*Hq*splits*Dv] fp32, part_ml [B*Hq*splits*2] fp32 (splits > 1).
 extern "C" int ksana_paged_decode(const void* q, long long q_stride, void* out, long long out_stride,
-                                  const void* cache, long long block_stride, int block_tokens, const int* block_table,
-                                  int table_stride, const int* kv_lens, const float* alibi, int B, int Hq, int Hkv,
-                                  int D, float scale, int cache_fp8, float k_scale, float v_scale, int num_splits,
-                                  float* part_o, float* part_ml, long long cache_rows, void* outq, float* oscale,
-                                  int oscale_ld, int* err, cudaStream_t st) {
+                                  const void* kc, const void* vc, long long block_stride, int block_tokens,
+                                  const int* block_table, int table_stride, const int* kv_lens, const float* alibi,
+                                  const float* sinks, int B, int Hq, int Hkv, int D, int Dv, int window, int keep, float scale,
+                                  int cache_fp8, float k_scale, float v_scale, int num_splits, float* part_o, float* part_ml,
+                                  int num_blocks, void* outq, float* oscale, int oscale_ld, int* err, cudaStream_t st) {
   if (B <= 0) return 0;
-  if (outq && (D != 128 || !oscale)) return -13;
-  if (Hq % Hkv || Hq / Hkv > 16) return -10;
+  if (outq && (D != 128 || Dv != 128 || !oscale)) return -13;
+  if (Hkv <= 0 || Hq % Hkv || q_stride % 8 || (reinterpret_cast<uintptr_t>(q) & 15)) return -10;
   if (num_splits < 1) num_splits = 1;
   if (num_splits > 1 && (!part_o || !part_ml)) return -12;
   AttnParams p{};
   p.q = (const bf16*)q; p.q_stride = q_stride; p.out = (bf16*)out; p.out_stride = out_stride;
-  p.cache = cache; p.block_stride = block_stride; p.block_tokens = block_tokens;
+  p.kc = kc; p.vc = vc; p.block_stride = block_stride; p.block_tokens = block_tokens; p.D = D; p.Dv = Dv;
+  p.window = window; p.keep = window > 0 ? keep : 0; p.sinks = sinks;
   p.block_table = block_table; p.table_stride = table_stride; p.cu_q = nullptr; p.kv_lens = kv_lens; p.alibi = alibi;
   p.Hq = Hq; p.Hkv = Hkv; p.scale_log2 = scale * 1.44269504f; p.k_scale = k_scale; p.v_scale = v_scale;
   p.num_splits = num_splits; p.part_o = part_o; p.part_ml = part_ml; p.err = err;
   p.outq = static_cast<uint8_t*>(outq); p.oscale = oscale; p.oscale_ld = oscale_ld;
-  if (D == 128) return dispatch_decode<128>(p, cache_fp8, cache_rows, B, st);
-  if (D == 64) return dispatch_decode<64>(p, cache_fp8, cache_rows, B, st);
+  switch (padded_head(D, Dv)) {
+    case 64: return dispatch_decode<64>(p, cache_fp8, num_blocks, B, st);
+    case 128: return dispatch_decode<128>(p, cache_fp8, num_blocks, B, st);
+    case 192: return dispatch_decode<192>(p, cache_fp8, num_blocks, B, st);
+    case 256: return dispatch_decode<256>(p, cache_fp8, num_blocks, B, st);
+  }
   return -11;
 }

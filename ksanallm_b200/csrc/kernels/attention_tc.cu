@@ -1,5 +1,6 @@
 // Prefill (and chunked-prefill) attention on the tcgen05 tensor cores: causal attention of new query rows
-// against the paged KV cache, head dimension 128, bf16 cache.
+// against the paged KV cache, head sizes up to 128 (query/key and value sizes may differ; both padded with zeros in shared
+// memory only), bf16 cache, optionally a sliding window with kept first tokens and a per-head sink logit.
 //
 // One CTA owns 128 packed query rows of one KV head group: row = (token, head inside the group), so the G query
 // heads that share a KV head reuse every staged K/V tile (G must divide 128). Per 128-token KV tile:
@@ -26,7 +27,7 @@ namespace ksana {
 typedef __nv_bfloat16 bf16;
 constexpr int kFaThreads = 192;
 constexpr int kFaTile = 128;                 // query rows per CTA and KV tokens per tile
-constexpr int kFaD = 128;
+constexpr int kFaD = 128;                    // padded head size
 constexpr int kFaPanelBytes = kFaTile * 128; // one 64-column panel of a 128-row tile
 constexpr int kFaTileBytes = 2 * kFaPanelBytes;
 constexpr int kFaSmemBytes = 3 * kFaTileBytes + 1024 + 256;
@@ -37,8 +38,10 @@ struct FaParams {
   bf16* out; long long out_stride;
   const int* block_table; int table_stride;
   const int* cu_q; const int* kv_lens; const float* alibi;
+  const float* sinks;                        // [Hq] logits added to the softmax denominator, or null
   int Hq, Hkv, G, block_tokens;
-  long long rows_per_block;                  // cache rows (of D elements) between consecutive blocks
+  int D, Dv;                                 // real head sizes
+  int window, keep;                          // sliding window in tokens (0: none), first tokens every row sees
   float scale_log2;
   int* err;
 };
@@ -49,8 +52,11 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
+// WIN: sliding window (p.window > 0); without it the window's tests are not compiled in
+template <bool WIN>
 __global__ void __launch_bounds__(kFaThreads, 2)
-prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap kv_map, const FaParams p) {
+prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
+                  const __grid_constant__ CUtensorMap v_map, const FaParams p) {
   extern __shared__ uint8_t fa_smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(fa_smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* q_s = smem;
@@ -79,7 +85,13 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
   const int past = kv_len - q_len;
   const int last_row = min(row0 + kFaTile - 1, q_len * G - 1);
   const int kv_end = min(kv_len, past + last_row / G + 1);
-  const int ntiles = (kv_end + kFaTile - 1) / kFaTile;
+  // tiles visited: those with kept first tokens, then from the first position in the window of this CTA's first row on
+  const int first_lo = WIN ? past + row0 / G - p.window + 1 : 0;
+  const int win_tile = WIN ? max(first_lo, 0) / kFaTile : 0;
+  const int keep_tiles = WIN ? min((p.keep + kFaTile - 1) / kFaTile, win_tile) : 0;
+  const int ntiles = keep_tiles + (kv_end + kFaTile - 1) / kFaTile - win_tile;
+  auto tile_start = [&](int j) { return (j < keep_tiles ? j : win_tile + j - keep_tiles) * kFaTile; };
+  const int kpanels = (p.D + 63) >> 6, vpanels = (p.Dv + 63) >> 6;
   const int* table = p.block_table + static_cast<size_t>(s) * p.table_stride;
 
   if (threadIdx.x == 0) {
@@ -99,29 +111,28 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     // ------------------------------------------------------------------ TMA producer
     if (lane == 0) {
       tma_prefetch_desc(&q_map);
-      tma_prefetch_desc(&kv_map);
-      mbar_expect_tx(q_full, kFaTileBytes);
+      tma_prefetch_desc(&k_map);
+      tma_prefetch_desc(&v_map);
+      mbar_expect_tx(q_full, kpanels * kFaPanelBytes);
       const int tok0 = q0 + row0 / G;
-      tma_load_3d(q_s, &q_map, q_full, 0, g * G, tok0);
-      tma_load_3d(q_s + kFaPanelBytes, &q_map, q_full, 64, g * G, tok0);
+      for (int h = 0; h < kpanels; ++h) tma_load_3d(q_s + h * kFaPanelBytes, &q_map, q_full, h * 64, g * G, tok0);
       const int bt = p.block_tokens;
       bool ok = true;
       for (int j = 0; j < ntiles && ok; ++j) {
-        const int t0 = j * kFaTile;
+        const int t0 = tile_start(j);
         const int nblk = min(kFaTile / bt, (kv_len - t0 + bt - 1) / bt);
-        const uint32_t bytes = static_cast<uint32_t>(nblk) * 2 * bt * 128;
 #pragma unroll
         for (int which = 0; which < 2; ++which) {
           uint64_t* full = which ? v_full : k_full;
           uint64_t* empty = which ? v_empty : k_empty;
           uint8_t* dst = which ? v_s : k_s;
           if (!mbar_wait(empty, (j & 1) ^ 1, abort_flag)) { ok = false; break; }
-          mbar_expect_tx(full, bytes);
+          const int panels = which ? vpanels : kpanels;
+          mbar_expect_tx(full, static_cast<uint32_t>(nblk) * panels * bt * 128);
           for (int b = 0; b < nblk; ++b) {
-            const long long r0 = static_cast<long long>(table[t0 / bt + b]) * p.rows_per_block +
-                                 (static_cast<long long>(which) * p.Hkv + g) * bt;
-            tma_load_2d(dst + b * bt * 128, &kv_map, full, 0, static_cast<int>(r0));
-            tma_load_2d(dst + kFaPanelBytes + b * bt * 128, &kv_map, full, 64, static_cast<int>(r0));
+            const int blk = table[t0 / bt + b];
+            for (int h = 0; h < panels; ++h)               // columns past the row's end arrive as zeros
+              tma_load_3d(dst + h * kFaPanelBytes + b * bt * 128, which ? &v_map : &k_map, full, h * 64, g * bt, blk);
           }
         }
       }
@@ -131,7 +142,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     // ------------------------------------------------------------------ MMA issuer
     if (lane == 0) {
       constexpr uint32_t idesc_qk = make_idesc(128, 128, 1, 1);
-      constexpr uint32_t idesc_pv = make_idesc(128, 128, 1, 1) | (1u << 16);     // B (= V) is MN-major
+      const uint32_t idesc_pv = make_idesc(128, vpanels * 64, 1, 1) | (1u << 16);     // B (= V) is MN-major
+      const int ksteps = (p.D + 15) >> 4;
       bool ok = mbar_wait(q_full, 0, abort_flag);
       for (int j = 0; j < ntiles && ok; ++j) {
         const uint32_t par = j & 1;
@@ -139,6 +151,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
         tc_fence_after();
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
+          if (k >= ksteps) break;
           const uint32_t off = (k >> 2) * kFaPanelBytes;
           const uint64_t adesc = make_smem_desc_sw128(smem_u32(q_s) + off) + 2 * (k & 3);
           const uint64_t bdesc = make_smem_desc_sw128(smem_u32(k_s) + off) + 2 * (k & 3);
@@ -168,15 +181,19 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     const bool active = vr < q_len * G;
     const int tok = vr / G, head = g * G + vr % G;
     const int limit = active ? past + tok : -1;            // last visible KV position
+    const int lo = WIN ? limit - p.window + 1 : 0;            // first position inside the window
+    const int keep = WIN ? p.keep : 0;
+    auto sees = [&](int pos) { return pos <= limit && (!WIN || pos >= lo || pos < keep); };
     const float slope2 = (p.alibi && active) ? p.alibi[head] * 1.44269504f : 0.f;
     float m_used = -CUDART_INF_F, l = 0.f;
     bool ok = true;
     for (int j = 0; j < ntiles; ++j) {
       const uint32_t par = j & 1;
-      const int t0 = j * kFaTile;
+      const int t0 = tile_start(j);
       if (!mbar_wait(s_full, par, abort_flag)) { ok = false; break; }
       tc_fence_after();
-      const bool need_mask = (t0 + kFaTile - 1 > limit) || slope2 != 0.f || p.scale_log2 <= 0.f;
+      const bool need_mask = (t0 + kFaTile - 1 > limit) || slope2 != 0.f || p.scale_log2 <= 0.f ||
+                             (WIN && t0 < lo && t0 + kFaTile > keep);
       // lazy rescale of O: keep the old reference maximum unless the row's maximum grew by more than 2^8
       auto update_reference = [&](float mx) {
         float m_new = m_used;
@@ -232,7 +249,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
           for (int i = 0; i < 32; ++i) {
             const int pos = t0 + c * 32 + i;
             const float v = __uint_as_float(r[i]) * p.scale_log2 + slope2 * static_cast<float>(pos - limit);
-            mx = fmaxf(mx, pos <= limit ? v : -CUDART_INF_F);
+            mx = fmaxf(mx, sees(pos) ? v : -CUDART_INF_F);
           }
         }
         const float mref = update_reference(mx);
@@ -247,8 +264,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
             const int pos = t0 + c * 32 + i;
             const float v0 = __uint_as_float(r[i]) * p.scale_log2 + slope2 * static_cast<float>(pos - limit) - mref;
             const float v1 = __uint_as_float(r[i + 1]) * p.scale_log2 + slope2 * static_cast<float>(pos + 1 - limit) - mref;
-            const float p0 = pos <= limit ? fast_exp2(v0) : 0.f;
-            const float p1 = pos + 1 <= limit ? fast_exp2(v1) : 0.f;
+            const float p0 = sees(pos) ? fast_exp2(v0) : 0.f;
+            const float p1 = sees(pos + 1) ? fast_exp2(v1) : 0.f;
             l += p0 + p1;
             __nv_bfloat162 pb = __floats2bfloat162_rn(p0, p1);
             pk[i >> 1] = *reinterpret_cast<uint32_t*>(&pb);
@@ -276,16 +293,19 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     }
     if (ok && mbar_wait(o_full, 0, abort_flag)) {
       tc_fence_after();
+      if (p.sinks && active) l += exp2f(p.sinks[head] * 1.44269504f - m_used);
       const float inv = l > 0.f ? 1.f / l : 0.f;
-      bf16* dst = p.out + static_cast<size_t>(q0 + tok) * p.out_stride + head * kFaD;
+      bf16* dst = p.out + static_cast<size_t>(q0 + tok) * p.out_stride + head * p.Dv;
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
+        if (c * 32 >= p.Dv) break;
         uint32_t r[32];
         tmem_ld32(tmem_o + lane_off + c * 32, r);
         tmem_ld_wait();
         if (active) {
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
+            if (c * 32 + i >= p.Dv) break;
             uint4 ov;
             __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&ov);
 #pragma unroll
@@ -329,24 +349,25 @@ using namespace ksana;
 
 // Returns 0 when launched, -100 when this kernel does not cover the configuration (the caller then uses the
 // general kernel of attention.cu), other negatives on setup errors.
-// q: [T, q_stride] bf16 with head h at column h*128 (T = rows addressable from q); cache: layer base of
-// [block][2][Hkv][block_tokens][128] bf16, blocks block_stride elements apart, cache_rows rows of 128 elements
-// addressable.
+// q: [T, q_stride] bf16 with head h at column h*D (T = rows addressable from q); kc / vc: the layer's K and V panels of
+// block 0, [Hkv][block_tokens][D] and [Hkv][block_tokens][Dv] bf16, blocks block_stride elements apart, num_blocks of them.
+// window 0: no sliding window. sinks: [Hq] fp32 or null.
 extern "C" int ksana_paged_prefill_tc(const void* q, long long q_stride, long long q_rows, void* out, long long out_stride,
-                                      const void* cache, long long block_stride, int block_tokens,
+                                      const void* kc, const void* vc, long long block_stride, int block_tokens,
                                       const int* block_table, int table_stride, const int* cu_q, const int* kv_lens,
-                                      const float* alibi, int B, int max_q_len, int Hq, int Hkv, int D, float scale,
-                                      long long cache_rows, int* err, cudaStream_t st) {
+                                      const float* alibi, const float* sinks, int B, int max_q_len, int Hq, int Hkv, int D,
+                                      int Dv, int window, int keep, float scale, int num_blocks, int* err, cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0) return 0;
-  if (D != kFaD || Hkv <= 0 || Hq % Hkv) return -100;
+  if (D <= 0 || Dv <= 0 || D > kFaD || Dv > kFaD || D % 8 || Dv % 8 || Hkv <= 0 || Hq % Hkv) return -100;
   const int G = Hq / Hkv;
   const int bt = block_tokens;
-  if (kFaTile % G || G > 128 || !(bt == 8 || bt == 16 || bt == 32 || bt == 64 || bt == 128)) return -100;
-  if (block_stride % D || block_stride < 2LL * Hkv * bt * D || cache_rows <= 0 || q_rows <= 0) return -100;
-  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache)) & 15 || (q_stride % 8)) return -100;
+  if (G > 128 || kFaTile % G || !(bt == 8 || bt == 16 || bt == 32 || bt == 64 || bt == 128)) return -100;
+  if (block_stride % 8 || num_blocks <= 0 || q_rows <= 0 || (out_stride % 8)) return -100;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kc) | reinterpret_cast<uintptr_t>(vc) |
+       reinterpret_cast<uintptr_t>(out)) & 15 || (q_stride % 8)) return -100;
   FaEncodeFn enc = fa_encode_fn();
   if (!enc) return -100;
-  CUtensorMap q_map, kv_map;
+  CUtensorMap q_map, k_map, v_map;
   {
     cuuint64_t dims[3] = {static_cast<cuuint64_t>(D), static_cast<cuuint64_t>(Hq), static_cast<cuuint64_t>(q_rows)};
     cuuint64_t strides[2] = {static_cast<cuuint64_t>(D) * 2, static_cast<cuuint64_t>(q_stride) * 2};
@@ -356,29 +377,32 @@ extern "C" int ksana_paged_prefill_tc(const void* q, long long q_stride, long lo
             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS) return -100;
   }
-  {
-    cuuint64_t dims[2] = {static_cast<cuuint64_t>(D), static_cast<cuuint64_t>(cache_rows)};
-    cuuint64_t strides[1] = {static_cast<cuuint64_t>(D) * 2};
-    cuuint32_t box[2] = {64, static_cast<cuuint32_t>(bt)};
-    cuuint32_t estr[2] = {1, 1};
-    if (enc(&kv_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(cache), dims, strides, box, estr,
-            CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+  for (int which = 0; which < 2; ++which) {
+    const int d = which ? Dv : D;
+    cuuint64_t dims[3] = {static_cast<cuuint64_t>(d), static_cast<cuuint64_t>(Hkv) * bt, static_cast<cuuint64_t>(num_blocks)};
+    cuuint64_t strides[2] = {static_cast<cuuint64_t>(d) * 2, static_cast<cuuint64_t>(block_stride) * 2};
+    cuuint32_t box[3] = {64, static_cast<cuuint32_t>(bt), 1};
+    cuuint32_t estr[3] = {1, 1, 1};
+    if (enc(which ? &v_map : &k_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(which ? vc : kc), dims, strides, box,
+            estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS) return -100;
   }
   static bool set = false;
   if (!set) {
-    if (cudaFuncSetAttribute(prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kFaSmemBytes) != cudaSuccess)
+    if (cudaFuncSetAttribute(prefill_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kFaSmemBytes) != cudaSuccess ||
+        cudaFuncSetAttribute(prefill_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kFaSmemBytes) != cudaSuccess)
       return -3;
     set = true;
   }
   FaParams p{};
   p.out = static_cast<bf16*>(out); p.out_stride = out_stride;
   p.block_table = block_table; p.table_stride = table_stride; p.cu_q = cu_q; p.kv_lens = kv_lens; p.alibi = alibi;
+  p.sinks = sinks; p.D = D; p.Dv = Dv; p.window = window; p.keep = window > 0 ? keep : 0;
   p.Hq = Hq; p.Hkv = Hkv; p.G = G; p.block_tokens = bt;
-  p.rows_per_block = block_stride / D;        // a block of one layer may sit inside a larger per-block record
   p.scale_log2 = scale * 1.44269504f;
   p.err = err;
   dim3 grid((max_q_len * G + kFaTile - 1) / kFaTile, Hkv, B);
-  prefill_tc_kernel<<<grid, kFaThreads, kFaSmemBytes, st>>>(q_map, kv_map, p);
+  if (window > 0) prefill_tc_kernel<true><<<grid, kFaThreads, kFaSmemBytes, st>>>(q_map, k_map, v_map, p);
+  else prefill_tc_kernel<false><<<grid, kFaThreads, kFaSmemBytes, st>>>(q_map, k_map, v_map, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

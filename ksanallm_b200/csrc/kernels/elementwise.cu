@@ -481,7 +481,7 @@ template <> __device__ __forceinline__ uint8_t kv_from_float<uint8_t>(float v) {
 template <typename T>
 __global__ void rerotate_blocks_kernel(T* __restrict__ cache, const int* __restrict__ triples, const float* __restrict__ cos_sin,
                                        int max_pos, int layers, int hkv, int bt, int D, int rot_dim, int neox,
-                                       int num_blocks, int* err) {
+                                       int num_blocks, long long rec_stride, int* err) {
   const int db = triples[3 * blockIdx.x + 1], delta = triples[3 * blockIdx.x + 2];
   if (delta == 0) return;
   const int ad = delta < 0 ? -delta : delta;
@@ -494,7 +494,7 @@ __global__ void rerotate_blocks_kernel(T* __restrict__ cache, const int* __restr
   const float* cs = cos_sin + static_cast<size_t>(ad) * rot_dim;
   const float sgn = delta > 0 ? 1.f : -1.f;
   const long long panel = static_cast<long long>(bt) * D;                 // one head's K panel
-  const long long layer_stride = 2LL * hkv * panel, block_stride = layers * layer_stride;
+  const long long layer_stride = 2LL * hkv * panel, block_stride = rec_stride > 0 ? rec_stride : layers * layer_stride;
   T* blk = cache + static_cast<size_t>(db) * block_stride;
   const long long pairs = static_cast<long long>(layers) * hkv * bt * half;
   for (long long i = blockIdx.y * static_cast<long long>(blockDim.x) + threadIdx.x; i < pairs;
@@ -754,18 +754,19 @@ extern "C" int ksana_swap_blocks(void* cache, void* pool, const int* pairs, int 
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
-// kv_bytes: 2 (bf16 cache) or 1 (e4m3 cache).
+// kv_bytes: 2 (bf16 cache) or 1 (e4m3 cache). rec_stride: elements between blocks, 0 = a dense
+// [blocks][layers][2][kv heads][block tokens][head dim] cache.
 extern "C" int ksana_rerotate_blocks(void* cache, const int* triples, int n, const float* cos_sin, int max_pos, int layers,
                                      int hkv, int bt, int D, int rot_dim, int neox, int kv_bytes, int num_blocks,
-                                     int* err, cudaStream_t st) {
+                                     long long rec_stride, int* err, cudaStream_t st) {
   if (n <= 0) return 0;
   if (rot_dim <= 0 || rot_dim > D || (rot_dim & 1) || (kv_bytes != 1 && kv_bytes != 2)) return -10;
   if (kv_bytes == 2)
     rerotate_blocks_kernel<bf16><<<dim3(n, 8), 256, 0, st>>>((bf16*)cache, triples, cos_sin, max_pos, layers, hkv, bt, D,
-                                                            rot_dim, neox, num_blocks, err);
+                                                            rot_dim, neox, num_blocks, rec_stride, err);
   else
     rerotate_blocks_kernel<uint8_t><<<dim3(n, 8), 256, 0, st>>>((uint8_t*)cache, triples, cos_sin, max_pos, layers, hkv,
-                                                                bt, D, rot_dim, neox, num_blocks, err);
+                                                                bt, D, rot_dim, neox, num_blocks, rec_stride, err);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

@@ -1,0 +1,68 @@
+// True 32-bit GEMM on the CUDA cores, for models served entirely in fp32 (no reduced-precision tensor-core mode):
+// D[M,N] = A[M,K] W[N,K]^T (+ bias[N]) (+ residual[M,N]). 64 x 64 tiles, 4 x 4 outputs per thread, K walked in steps of
+// 16 in ascending order for every shape, so that a row's result does not depend on the other rows of the call.
+#include "pdl.cuh"
+#include <cuda_runtime.h>
+
+namespace ksana {
+
+constexpr int kSgTile = 64, kSgK = 16, kSgThreads = 256;
+
+__global__ void __launch_bounds__(kSgThreads)
+gemm_f32_kernel(const float* __restrict__ A, int lda, const float* __restrict__ W, int ldw, float* __restrict__ D, int ldd,
+                const float* __restrict__ bias, const float* __restrict__ residual, int ldr, int M, int N, int K) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float as[kSgK][kSgTile + 4], ws[kSgK][kSgTile + 4];
+  const int m0 = blockIdx.y * kSgTile, n0 = blockIdx.x * kSgTile;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;          // staging: one row, four consecutive k per thread
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += kSgK) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int k = k0 + lk + e;
+      as[lk + e][lr] = (m0 + lr < M && k < K) ? A[static_cast<size_t>(m0 + lr) * lda + k] : 0.f;
+      ws[lk + e][lr] = (n0 + lr < N && k < K) ? W[static_cast<size_t>(n0 + lr) * ldw + k] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kSgK; ++k) {
+      float a[4], b[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { a[e] = as[k][ty * 4 + e]; b[e] = ws[k][tx * 4 + e]; }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = m0 + ty * 4 + i;
+    if (m >= M) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx * 4 + j;
+      if (n >= N) continue;
+      float v = acc[i][j];
+      if (bias) v += bias[n];
+      if (residual) v += residual[static_cast<size_t>(m) * ldr + n];
+      D[static_cast<size_t>(m) * ldd + n] = v;
+    }
+  }
+}
+
+}  // namespace ksana
+
+using namespace ksana;
+
+extern "C" int ksana_gemm_f32(const float* A, int lda, const float* W, int ldw, float* D, int ldd, const float* bias,
+                              const float* residual, int ldr, int M, int N, int K, cudaStream_t st) {
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  const dim3 grid((N + kSgTile - 1) / kSgTile, (M + kSgTile - 1) / kSgTile);
+  if (grid.y > 65535u) return -10;
+  return launch_pdl(gemm_f32_kernel, grid, dim3(kSgThreads), 0, st, A, lda, W, ldw, D, ldd, bias, residual, ldr, M, N, K) ==
+                 cudaSuccess ? 0 : -4;
+}

@@ -50,6 +50,7 @@ class StepInput:
     decode_workspace: Optional[tuple] = None
     sample_k: int = 0                    # > 0: tensor-parallel ranks return merged per-shard top-k candidates, not logits
     want_hidden: bool = False            # keep final hidden states / post-norm states for /forward
+    prev_ids: Optional[torch.Tensor] = None   # the token before each row's (-1: none); models with ``needs_prev_ids`` only
 
 
 @dataclass
@@ -88,7 +89,29 @@ def alibi_slopes(num_heads: int) -> torch.Tensor:
     return torch.tensor(s, dtype=torch.float32)
 
 
+class PanelLayout:
+    """Layout of a cache block whose layers differ in head counts or head sizes: one record per block that holds the K
+    panel [kv heads, block tokens, key size] and the V panel [kv heads, block tokens, value size] of every cache layer,
+    one after the other. Sizes are multiples of 8 elements, so every panel starts on a 16-byte boundary."""
+
+    def __init__(self, shapes, block_tokens: int):
+        self.entries, self.record = [], 0
+        for hkv, d, dv in shapes:
+            if d % 8 or dv % 8:
+                raise ValueError(f"head sizes {d}, {dv} are not multiples of 8")
+            k0, v0 = self.record, self.record + hkv * block_tokens * d
+            self.record = v0 + hkv * block_tokens * dv
+            self.entries.append((k0, (hkv, block_tokens, d), v0, (hkv, block_tokens, dv)))
+
+    def views(self, cache: torch.Tensor, i: int):
+        """(K, V) of cache layer ``i``: [blocks, kv heads, block tokens, size] views of the records."""
+        k0, ks, v0, vs = self.entries[i]
+        return cache[:, k0:v0].unflatten(1, ks), cache[:, v0:v0 + vs[0] * vs[1] * vs[2]].unflatten(1, vs)
+
+
 class CommonModel:
+    needs_prev_ids = False               # the step carries the token before each row's (StepInput.prev_ids)
+
     def __init__(self, cfg: ModelConfig, tp_rank: int = 0, tp_size: int = 1, comm=None, device="cpu",
                  dtype=torch.bfloat16, layer_range: Optional[tuple] = None, kv_cache_dtype=None,
                  max_positions: Optional[int] = None):
@@ -229,6 +252,8 @@ class CommonModel:
 
     def compute_logits(self, normed: torch.Tensor) -> torch.Tensor:
         """Vocab-sharded lm_head GEMM with fp32 output, shards gathered across the TP group."""
+        if normed.shape[0] == 0:
+            return torch.empty(0, self.cfg.vocab_size, dtype=torch.float32, device=normed.device)
         logits = ops.linear(normed, self.lm_head, out_f32=True)
         if self.tp_size > 1:
             logits = self.comm.all_gather_last_dim(logits, valid=self.vocab_shard)

@@ -160,6 +160,8 @@ def linear(x, W: LinearWeight, residual=None, out=None, out_f32: bool = False):
                 o = torch.empty(x.q.shape[0], W.out_features, dtype=torch.float32, device=x.q.device)
                 return native.gemm_fp8(x.q, x.s, W.wq, W.ws, bias=W.bias, residual=residual, out_f32=o, hw_scale=W.ue8m0)
             return native.gemm_fp8(x.q, x.s, W.wq, W.ws, out=out, bias=W.bias, residual=residual, hw_scale=W.ue8m0)
+        if W.w.dtype == torch.float32:
+            return native.gemm_f32(x, W.w, out=out, bias=W.bias, residual=residual)
         if out_f32:
             o = torch.empty(x.shape[0], W.out_features, dtype=torch.float32, device=x.device)
             return native.gemm_bf16(x, W.w, bias=W.bias, residual=residual, out_f32=o)
@@ -237,6 +239,119 @@ def rope_kv_append(qkv, positions, slots, cos_sin, cache_layer, block_tokens, Hq
     else:
         ref.rope_kv_append(qkv, positions, slots, cos_sin, cache_layer, block_tokens, Hq, Hkv, D, rot_dim, neox,
                            mrope_sections, k_scale, v_scale, apply_rope)
+
+
+# ------------------------------------------------------------------------------- 32-bit residual stream
+@dataclass
+class NormParams:
+    """Weight and optional bias of a norm over ``size`` real columns (stored padded with zeros to a multiple of 8)."""
+    w: torch.Tensor
+    b: Optional[torch.Tensor]
+    size: int
+    eps: float
+    rms: bool = False
+
+
+def embed_pair(ids, prev, table, pair, scale, buckets=0, mul_prev=0, mul_cur=0, copy=None, vocab=None):
+    """fp32 rows: scaled token embedding plus, with a ``pair`` table, the row (prev * mul_prev + id * mul_cur) mod buckets
+    of it (row ``buckets`` where prev < 0: the first token of a sequence). ``copy`` receives the rows in the table's type."""
+    if table.is_cuda:
+        return native.embed_pair(ids, prev, table, pair, scale, buckets, mul_prev, mul_cur, copy, vocab)
+    x = ref.embed_pair(ids, prev, table, pair, scale, buckets, mul_prev, mul_cur)
+    if copy is not None:
+        copy.copy_(x)
+    return x
+
+
+def stream_norm(x, norm: NormParams, dtype, rows=None):
+    """norm of the fp32 residual stream (of its ``rows``) as the next linear's operand."""
+    if x.is_cuda:
+        z = torch.empty(rows.numel() if rows is not None else x.shape[0], x.shape[1], dtype=dtype, device=x.device)
+        native.residual_norm(x, norm.size, norm.eps, w2=norm.w, b2=norm.b, z=z, rows=rows, rms=norm.rms)
+        return z
+    return ref.stream_norm(x[rows.long()] if rows is not None else x, norm).to(dtype)
+
+
+def stream_copy(x, out):
+    """The fp32 stream's rows in the type of ``out`` (a strided view is fine)."""
+    if x.is_cuda:
+        native.residual_norm(x, x.shape[1], 0.0, z=out)
+    else:
+        out.copy_(x)
+
+
+def stream_add(x, y, post: Optional[NormParams], scale, then: Optional[NormParams] = None, copy=None, inplace=True):
+    """x + scale * norm(y; post) on the fp32 residual stream, fused with what reads the sum next: ``then`` (the following
+    norm, returned in y's type) or ``copy`` (a buffer that receives the sum in its own type). Returns (x, normed or None);
+    ``inplace`` updates x."""
+    if x.is_cuda:
+        z = torch.empty_like(y) if then is not None else copy
+        out = x if inplace else torch.empty_like(x)
+        size, eps, rms = (post.size, post.eps, post.rms) if post is not None else (
+            (then.size, then.eps, then.rms) if then is not None else (x.shape[1], 0.0, False))
+        native.residual_norm(x, size, eps, y=y, w1=post.w if post else None, b1=post.b if post else None, ls=scale, x_out=out,
+                             w2=then.w if then else None, b2=then.b if then else None, z=z, rms=rms)
+        return out, (z if then is not None else None)
+    a = ref.stream_norm(y, post) if post is not None else y.float()
+    if scale is not None:
+        a = a * scale.float()
+    out = x.add_(a) if inplace else x + a
+    if copy is not None:
+        copy.copy_(out)
+    return out, (ref.stream_norm(out, then).to(y.dtype) if then is not None else None)
+
+
+def glu_clamp(x, limit, alpha=1.702, offset=1.0):
+    """min(gate, limit) * sigmoid(alpha * gate) * (clamp(up, -limit, limit) + offset) of packed gate | up columns."""
+    if x.is_cuda:
+        return native.glu_clamp(x, limit, alpha, offset)
+    return ref.glu_clamp(x, limit, alpha, offset)
+
+
+def qkv_rope_append(qkv, positions, slots, cos_sin, k_cache, v_cache, block_tokens, Hq, Hkv, rot_dim):
+    """Partial rotation of q and k and append of k, v to separate paged panels (key and value sizes may differ)."""
+    fn = native.qkv_rope_append if qkv.is_cuda else ref.qkv_rope_append
+    fn(qkv, positions, slots, cos_sin, k_cache, v_cache, block_tokens, Hq, Hkv, rot_dim)
+
+
+def refit_stream_rows(x, pos, emb):
+    """Rows of the residual stream replaced by given embeddings (real columns only)."""
+    if x.is_cuda:
+        native.refit_rows_f32(x, pos, emb.contiguous())
+    else:
+        x[pos.long(), :emb.shape[1]] = emb.float()
+
+
+def panel_attention(qkv, k_cache, v_cache, block_tokens, step, Hq, Hkv, scale, window=0, keep=0, sinks=None):
+    """Attention of a step's new rows (multi-token sequences first, then single-token ones) against separate K and V
+    panels, with an optional sliding window (``keep`` first tokens stay visible) and per-head sink logits."""
+    D, Dv = k_cache.shape[-1], v_cache.shape[-1]
+    T = qkv.shape[0]
+    out = torch.empty(T, Hq * Dv, dtype=qkv.dtype, device=qkv.device)
+    if not qkv.is_cuda:
+        out.copy_(ref.panel_attention(qkv[:, :Hq * D], k_cache, v_cache, step.block_table, step.cu_q, step.kv_lens, Hq, Hkv, scale,
+                                      window, keep, sinks))
+        return out
+    if qkv.dtype == torch.float32:
+        native.attention_f32(qkv, qkv.stride(0), out, k_cache, v_cache, block_tokens, step.block_table, step.cu_q, step.kv_lens,
+                             step.num_multi + step.num_single, max(step.max_q_len, 1), Hq, Hkv, scale, window, keep, sinks)
+        return out
+    nm, ns, tm = step.num_multi, step.num_single, step.num_multi_tokens
+    if nm:
+        native.paged_prefill(qkv, qkv.stride(0), out, k_cache, k_cache.stride(0), block_tokens, step.block_table, step.cu_q,
+                             step.kv_lens, nm, step.max_q_len, Hq, Hkv, D, scale, v_cache=v_cache, window=window, keep=keep,
+                             sinks=sinks)
+    if ns:
+        seen = min(step.max_kv_len, window + keep + 128) if window > 0 else step.max_kv_len
+        n = decode_splits(ns, Hkv * ((Hq // Hkv + 15) // 16), seen)
+        po = pml = None
+        if n > 1:
+            po = torch.empty(ns * Hq * n * Dv, dtype=torch.float32, device=qkv.device)
+            pml = torch.empty(ns * Hq * n * 2, dtype=torch.float32, device=qkv.device)
+        native.paged_decode(qkv[tm:], qkv.stride(0), out[tm:], k_cache, k_cache.stride(0), block_tokens, step.block_table[nm:],
+                            step.kv_lens[nm:], ns, Hq, Hkv, D, scale, num_splits=n, part_o=po, part_ml=pml, v_cache=v_cache,
+                            window=window, keep=keep, sinks=sinks)
+    return out
 
 
 def decode_splits(batch: int, hkv: int, max_kv_len: int, sms: int = 148, ctas_per_sm: int = 2) -> int:

@@ -64,14 +64,22 @@ _SIGS = {
     "ksana_patch_ids": [vp, vp, vp, vp, i32, i32, i32, vp, vp],
     "ksana_smallm_estimate": [i32, i32, i32, i32, vp],
     "ksana_absmax_scale": [vp, i32, i32, i64, f32, f32, vp, vp, vp],
-    "ksana_rerotate_blocks": [vp, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp],
+    "ksana_rerotate_blocks": [vp, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, i64, vp, vp],
+    "ksana_embed_pair": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i64, i64, i64, f32, i32, vp, vp],
+    "ksana_residual_norm": [vp, i32, vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, f32, i32, i32, vp, vp],
+    "ksana_glu_clamp": [vp, vp, i32, i32, i32, f32, f32, f32, i32, vp],
+    "ksana_qkv_rope_append": [vp, vp, vp, vp, i32, vp, vp, i64, i32, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp],
+    "ksana_refit_rows_f32": [vp, i32, vp, vp, i32, i32, i32, vp, vp],
+    "ksana_gemm_f32": [vp, i32, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, vp],
+    "ksana_attention_f32": [vp, i64, vp, i64, vp, vp, i64, i32, i32, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32,
+                            f32, vp, vp],
     "ksana_cast_f32": [vp, vp, i64, vp],
-    "ksana_paged_prefill_tc": [vp, i64, i64, vp, i64, vp, i64, i32, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, f32, i64,
-                               vp, vp],
-    "ksana_paged_prefill": [vp, i64, vp, i64, vp, i64, i32, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32,
-                            f32, f32, i64, vp, vp],
-    "ksana_paged_decode": [vp, i64, vp, i64, vp, i64, i32, vp, i32, vp, vp, i32, i32, i32, i32, f32, i32, f32, f32,
-                           i32, vp, vp, i64, vp, vp, i32, vp, vp],
+    "ksana_paged_prefill_tc": [vp, i64, i64, vp, i64, vp, vp, i64, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32,
+                               i32, i32, f32, i32, vp, vp],
+    "ksana_paged_prefill": [vp, i64, vp, i64, vp, vp, i64, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32,
+                            f32, i32, f32, f32, i32, vp, vp],
+    "ksana_paged_decode": [vp, i64, vp, i64, vp, vp, i64, i32, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, i32,
+                           f32, f32, i32, vp, vp, i32, vp, vp, i32, vp, vp],
     "ksana_mla_attention": [vp, i64, vp, i64, vp, i64, i32, vp, i32, vp, vp, i32, i32, i32, f32, i64, i32, vp, vp, vp, vp],
     "ksana_mla_rope_append": [vp, i64, i32, vp, i64, vp, f32, vp, vp, vp, vp, vp, i64, i32, i32, i32, i32, i64, vp, vp],
     "ksana_gemm_smallm_w4": [vp, i32, vp, vp, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, vp, i64, vp, i32, vp, vp],
@@ -623,8 +631,17 @@ def rerotate_blocks(cache, triples, cos_sin, rot_dim, neox):
     block tokens, head dim], bf16 or e4m3; ``cos_sin``: [max_pos, rot_dim] fp32."""
     nb, layers, _, hkv, bt, D = cache.shape
     _check(lib().ksana_rerotate_blocks(_p(cache), _p(triples), triples.shape[0], _p(cos_sin), cos_sin.shape[0], layers,
-                                       hkv, bt, D, rot_dim, int(bool(neox)), cache.element_size(), nb,
+                                       hkv, bt, D, rot_dim, int(bool(neox)), cache.element_size(), nb, 0,
                                        _p(err_flag(cache.device)), _st()), "ksana_rerotate_blocks")
+
+
+def rerotate_panel(k_panel, triples, cos_sin, rot_dim, neox=True):
+    """:func:`rerotate_blocks` for one layer whose K panels [blocks, kv heads, block tokens, head dim] (bf16) sit inside
+    larger block records."""
+    nb, hkv, bt, D = k_panel.shape
+    _check(lib().ksana_rerotate_blocks(_p(k_panel), _p(triples), triples.shape[0], _p(cos_sin), cos_sin.shape[0], 1, hkv, bt, D,
+                                       rot_dim, int(bool(neox)), k_panel.element_size(), nb, int(k_panel.stride(0)),
+                                       _p(err_flag(k_panel.device)), _st()), "ksana_rerotate_blocks")
 
 
 def add(a, b=None, bias=None, out=None):
@@ -640,6 +657,55 @@ def cast_f32(x, out=None):
         out = torch.empty(x.shape, dtype=torch.float32, device=x.device)
     _check(lib().ksana_cast_f32(_p(x), _p(out), x.numel(), _st()), "ksana_cast_f32")
     return out
+
+
+# -------------------------------------------------------------------------- 32-bit residual stream
+def gemm_f32(x, w, out=None, bias=None, residual=None):
+    """out[M,N] = x[M,K] @ w[N,K]^T (+bias)(+residual), everything fp32 on the CUDA cores."""
+    M, K = x.shape
+    N = w.shape[0]
+    assert x.dtype == w.dtype == torch.float32 and x.stride(1) == 1 and w.stride(1) == 1 and w.shape[1] == K
+    if out is None:
+        out = torch.empty(M, N, dtype=torch.float32, device=x.device)
+    _check(lib().ksana_gemm_f32(_p(x), x.stride(0), _p(w), w.stride(0), _p(out), out.stride(0), _p(bias), _p(residual),
+                                residual.stride(0) if residual is not None else 0, M, N, K, _st()), "ksana_gemm_f32")
+    return out
+
+
+def embed_pair(ids, prev, table, pair, scale, buckets=0, mul_prev=0, mul_cur=0, copy=None, vocab=None):
+    """fp32 rows table[id] * scale (+ the pair table's row of (previous id, id)); ``copy``: the same rows in the table's
+    type (a strided view is fine)."""
+    T, H = ids.numel(), table.shape[1]
+    x = torch.empty(T, H, dtype=torch.float32, device=table.device)
+    _check(lib().ksana_embed_pair(_p(ids), _p(prev), _p(table), _p(pair), _p(x), _p(copy), copy.stride(0) if copy is not None else 0,
+                                  T, H, vocab or table.shape[0], buckets, mul_prev, mul_cur, float(scale),
+                                  int(table.dtype == torch.float32), _p(err_flag(table.device)), _st()), "ksana_embed_pair")
+    return x
+
+
+def residual_norm(x, H, eps, y=None, w1=None, b1=None, ls=None, x_out=None, w2=None, b2=None, z=None, rows=None, rms=False):
+    """One pass over rows of the fp32 stream ``x`` (``H`` real columns, padded to a multiple of 8):
+    x' = x + ls * norm(y; w1, b1), stored to ``x_out``; z = norm(x'; w2, b2), or a copy of x' without ``w2``. Parts whose
+    arguments are None are left out; ``rows`` gathers stream rows."""
+    M = rows.numel() if rows is not None else x.shape[0]
+    t = z if z is not None else y
+    _check(lib().ksana_residual_norm(_p(x), x.stride(0), _p(rows), x.shape[0], _p(y), y.stride(0) if y is not None else 0, _p(w1),
+                                     _p(b1), _p(ls), _p(x_out), _p(w2), _p(b2), _p(z), z.stride(0) if z is not None else 0, M, H,
+                                     float(eps), int(rms), int(t.dtype == torch.float32), _p(err_flag(x.device)), _st()),
+           "ksana_residual_norm")
+
+
+def glu_clamp(x, limit, alpha, offset):
+    M, I = x.shape[0], x.shape[1] // 2
+    out = torch.empty(M, I, dtype=x.dtype, device=x.device)
+    _check(lib().ksana_glu_clamp(_p(x), _p(out), M, I, x.stride(0), float(limit), float(alpha), float(offset),
+                                 int(x.dtype == torch.float32), _st()), "ksana_glu_clamp")
+    return out
+
+
+def refit_rows_f32(x, pos, emb):
+    _check(lib().ksana_refit_rows_f32(_p(x), x.stride(0), _p(pos), _p(emb), pos.numel(), emb.shape[1], x.shape[0],
+                                      _p(err_flag(x.device)), _st()), "ksana_refit_rows_f32")
 
 
 # ---------------------------------------------------------------------------- attention path
@@ -666,38 +732,73 @@ def _cache_rows(cache_layer, block_stride, D):
 PREFILL_TC = True                  # prefill attention on tcgen05 where the kernel covers the configuration
 
 
+def _panels(cache_layer, v_cache, D):
+    """(K panel of block 0, V panel of block 0, V head size) as addresses: from one interleaved layer tensor
+    [blocks, 2, kv heads, block tokens, D], or from separate K and V panel views [blocks, kv heads, block tokens, size]."""
+    if v_cache is not None:
+        return cache_layer.data_ptr(), v_cache.data_ptr(), int(v_cache.shape[-1])
+    return cache_layer.data_ptr(), cache_layer.data_ptr() + cache_layer.stride(1) * cache_layer.element_size(), D
+
+
 def paged_prefill(q, q_stride, out, cache_layer, block_stride, block_tokens, block_table, cu_q, kv_lens, B, max_q_len,
-                  Hq, Hkv, D, scale, alibi=None, k_scale=1.0, v_scale=1.0):
+                  Hq, Hkv, D, scale, alibi=None, k_scale=1.0, v_scale=1.0, v_cache=None, window=0, keep=0, sinks=None):
+    """``v_cache``: V panels of their own (``cache_layer`` then holds the K panels). ``window`` > 0: position i sees j <= i
+    with i - j < window or j < keep. ``sinks``: fp32 [Hq] logits in the softmax denominator."""
     fp8 = cache_layer.dtype != torch.bfloat16
-    if PREFILL_TC and not fp8 and D == 128:
-        # tcgen05 kernel (head dim 128, bf16 cache, group size dividing 128); -100 = configuration not covered
-        rc = lib().ksana_paged_prefill_tc(_p(q), q_stride, q.shape[0], _p(out), out.stride(0), _p(cache_layer),
-                                          block_stride, block_tokens, _p(block_table), block_table.stride(0),
-                                          _p(cu_q), _p(kv_lens), _p(alibi), B, max_q_len, Hq, Hkv, D, float(scale),
-                                          _cache_rows(cache_layer, block_stride, D), _p(err_flag(q.device)), _st())
+    kc, vc, Dv = _panels(cache_layer, v_cache, D)
+    nblocks = int(cache_layer.shape[0])
+    if PREFILL_TC and not fp8 and max(D, Dv) <= 128:
+        # tcgen05 kernel (head sizes up to 128, bf16 cache, group size dividing 128); -100 = configuration not covered
+        rc = lib().ksana_paged_prefill_tc(_p(q), q_stride, q.shape[0], _p(out), out.stride(0), kc, vc, block_stride,
+                                          block_tokens, _p(block_table), block_table.stride(0), _p(cu_q), _p(kv_lens),
+                                          _p(alibi), _p(sinks), B, max_q_len, Hq, Hkv, D, Dv, window, keep, float(scale),
+                                          nblocks, _p(err_flag(q.device)), _st())
         if rc != -100:
             _check(rc, "ksana_paged_prefill_tc")
             return
-    rc = lib().ksana_paged_prefill(_p(q), q_stride, _p(out), out.stride(0), _p(cache_layer), block_stride,
-                                   block_tokens, _p(block_table), block_table.stride(0), _p(cu_q), _p(kv_lens),
-                                   _p(alibi), B, max_q_len, Hq, Hkv, D, float(scale), int(fp8), float(k_scale),
-                                   float(v_scale), _cache_rows(cache_layer, block_stride, D), _p(err_flag(q.device)), _st())
+    rc = lib().ksana_paged_prefill(_p(q), q_stride, _p(out), out.stride(0), kc, vc, block_stride, block_tokens,
+                                   _p(block_table), block_table.stride(0), _p(cu_q), _p(kv_lens), _p(alibi), _p(sinks), B,
+                                   max_q_len, Hq, Hkv, D, Dv, window, keep, float(scale), int(fp8), float(k_scale),
+                                   float(v_scale), nblocks, _p(err_flag(q.device)), _st())
     _check(rc, "ksana_paged_prefill")
 
 
 def paged_decode(q, q_stride, out, cache_layer, block_stride, block_tokens, block_table, kv_lens, B, Hq, Hkv, D, scale,
                  alibi=None, k_scale=1.0, v_scale=1.0, num_splits=1, part_o=None, part_ml=None, out_q=None,
-                 out_scale=None):
+                 out_scale=None, v_cache=None, window=0, keep=0, sinks=None):
     """``out_q`` / ``out_scale`` (head dim 128): the output also (or, with ``out`` None, only) as the FP8 operand of the
-    next GEMM: e4m3 [B, Hq * D] and scales [Hq, ld]."""
+    next GEMM: e4m3 [B, Hq * D] and scales [Hq, ld]. ``v_cache`` / ``window`` / ``keep`` / ``sinks``: see
+    :func:`paged_prefill`."""
     fp8 = cache_layer.dtype != torch.bfloat16
-    rc = lib().ksana_paged_decode(_p(q), q_stride, _p(out), out.stride(0) if out is not None else Hq * D, _p(cache_layer),
-                                  block_stride, block_tokens,
-                                  _p(block_table), block_table.stride(0), _p(kv_lens), _p(alibi), B, Hq, Hkv, D,
-                                  float(scale), int(fp8), float(k_scale), float(v_scale), num_splits, _p(part_o),
-                                  _p(part_ml), _cache_rows(cache_layer, block_stride, D), _p(out_q), _p(out_scale),
-                                  out_scale.stride(0) if out_scale is not None else 0, _p(err_flag(q.device)), _st())
+    kc, vc, Dv = _panels(cache_layer, v_cache, D)
+    rc = lib().ksana_paged_decode(_p(q), q_stride, _p(out), out.stride(0) if out is not None else Hq * Dv, kc, vc,
+                                  block_stride, block_tokens, _p(block_table), block_table.stride(0), _p(kv_lens), _p(alibi),
+                                  _p(sinks), B, Hq, Hkv, D, Dv, window, keep, float(scale), int(fp8), float(k_scale),
+                                  float(v_scale), num_splits, _p(part_o), _p(part_ml), int(cache_layer.shape[0]), _p(out_q),
+                                  _p(out_scale), out_scale.stride(0) if out_scale is not None else 0,
+                                  _p(err_flag(q.device)), _st())
     _check(rc, "ksana_paged_decode")
+
+
+def attention_f32(q, q_stride, out, k_cache, v_cache, block_tokens, block_table, cu_q, kv_lens, B, max_q_len, Hq, Hkv, scale,
+                  window=0, keep=0, sinks=None):
+    """All of a step's new rows (any lengths) against fp32 K and V panels, in 32-bit arithmetic throughout."""
+    rc = lib().ksana_attention_f32(_p(q), q_stride, _p(out), out.stride(0), _p(k_cache), _p(v_cache), k_cache.stride(0),
+                                   block_tokens, k_cache.shape[0], _p(block_table), block_table.stride(0), _p(cu_q),
+                                   _p(kv_lens), _p(sinks), B, max_q_len, Hq, Hkv, k_cache.shape[-1], v_cache.shape[-1], window,
+                                   keep, float(scale), _p(err_flag(q.device)), _st())
+    _check(rc, "ksana_attention_f32")
+
+
+def qkv_rope_append(qkv, positions, slots, cos_sin, k_cache, v_cache, block_tokens, Hq, Hkv, rot_dim):
+    """Rotation (halves) of the first ``rot_dim`` dimensions of q (in place) and k, and append of k and v to their paged
+    panels [blocks, kv heads, block tokens, size]."""
+    T = qkv.shape[0]
+    rc = lib().ksana_qkv_rope_append(_p(qkv), _p(positions), _p(slots), _p(cos_sin), cos_sin.shape[0] if cos_sin is not None else 0,
+                                     _p(k_cache), _p(v_cache), k_cache.stride(0), block_tokens, k_cache.shape[0], T, Hq, Hkv,
+                                     k_cache.shape[-1], v_cache.shape[-1], rot_dim, int(qkv.dtype == torch.float32),
+                                     _p(err_flag(qkv.device)), _st())
+    _check(rc, "ksana_qkv_rope_append")
 
 
 def mla_rope_append(q, nope, kv, norm_w, eps, positions, slots, cos_sin, qfull, cache_layer, block_stride, block_tokens, G):

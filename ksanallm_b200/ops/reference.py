@@ -261,6 +261,77 @@ def paged_attention(q, cache_layer, block_table, cu_q, kv_lens, Hq, Hkv, D, scal
     return out
 
 
+# ------------------------------------------------------------------------------- 32-bit residual stream
+def embed_pair(ids, prev, table, pair, scale, buckets=0, mul_prev=0, mul_cur=0):
+    x = table[ids.long()].float() * scale
+    if pair is not None:
+        a = prev.long()
+        row = torch.where(a < 0, torch.full_like(a, buckets), (a * mul_prev + ids.long() * mul_cur) % buckets)
+        x = x + pair[row].float()
+    return x
+
+
+def stream_norm(x, norm):
+    """fp32 norm over the first ``norm.size`` columns; pad columns come out as zeros."""
+    h = x[:, :norm.size].float()
+    if norm.rms:
+        y = h * torch.rsqrt(h.pow(2).mean(-1, keepdim=True) + norm.eps)
+    else:
+        d = h - h.mean(-1, keepdim=True)
+        y = d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + norm.eps)
+    y = y * norm.w[:norm.size].float()
+    if norm.b is not None:
+        y = y + norm.b[:norm.size].float()
+    return F.pad(y, (0, x.shape[1] - norm.size))
+
+
+def glu_clamp(x, limit, alpha, offset):
+    g, u = x.float().chunk(2, dim=-1)
+    g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+    return (g * torch.sigmoid(alpha * g) * (u + offset)).to(x.dtype)
+
+
+def qkv_rope_append(qkv, positions, slots, cos_sin, k_cache, v_cache, block_tokens, Hq, Hkv, rot_dim):
+    """In place on q of qkv [T, Hq*D + Hkv*D + Hkv*Dv]; rotated k and v into panels [blocks, Hkv, block_tokens, size]."""
+    T, D, Dv = qkv.shape[0], k_cache.shape[-1], v_cache.shape[-1]
+    q, k = qkv[:, :Hq * D].reshape(T, Hq, D), qkv[:, Hq * D:(Hq + Hkv) * D].reshape(T, Hkv, D)
+    v = qkv[:, (Hq + Hkv) * D:].reshape(T, Hkv, Dv)
+    if rot_dim:
+        qkv[:, :Hq * D] = apply_rope(q, positions, cos_sin, rot_dim).reshape(T, Hq * D)
+        k = apply_rope(k, positions, cos_sin, rot_dim)
+    ok = slots >= 0
+    blk, off = slots[ok].long() // block_tokens, slots[ok].long() % block_tokens
+    k_cache[blk, :, off] = k[ok].to(k_cache.dtype)
+    v_cache[blk, :, off] = v[ok].to(v_cache.dtype)
+
+
+def panel_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, Hq, Hkv, scale, window=0, keep=0, sinks=None):
+    """q [T, Hq*D] (new tokens only) -> [T, Hq*Dv]; see the sliding window and sink in dispatch.panel_attention."""
+    T, G, D, Dv, bt = q.shape[0], Hq // Hkv, k_cache.shape[-1], v_cache.shape[-1], k_cache.shape[2]
+    out = torch.zeros(T, Hq * Dv, dtype=q.dtype, device=q.device)
+    for s in range(kv_lens.numel()):
+        q0, q1 = int(cu_q[s]), int(cu_q[s + 1])
+        ql, kl = q1 - q0, int(kv_lens[s])
+        if ql == 0:
+            continue
+        blocks = block_table[s, :(kl + bt - 1) // bt].long()
+        k = k_cache[blocks].float().permute(1, 0, 2, 3).reshape(Hkv, -1, D)[:, :kl]
+        v = v_cache[blocks].float().permute(1, 0, 2, 3).reshape(Hkv, -1, Dv)[:, :kl]
+        qs = q[q0:q1].float().reshape(ql, Hkv, G, D).permute(1, 2, 0, 3)
+        att = torch.einsum("hgqd,hkd->hgqk", qs, k) * scale
+        qpos = torch.arange(kl - ql, kl, device=q.device).unsqueeze(1)
+        kpos = torch.arange(kl, device=q.device).unsqueeze(0)
+        hide = kpos > qpos
+        if window > 0:
+            hide = hide | ((qpos - kpos >= window) & (kpos >= keep))
+        att = att.masked_fill(hide, float("-inf"))
+        if sinks is not None:
+            att = torch.cat([att, sinks.float().reshape(Hkv, G, 1, 1).expand(-1, -1, ql, 1)], dim=-1)
+        p = torch.softmax(att, dim=-1)[..., :kl]
+        out[q0:q1] = torch.einsum("hgqk,hkd->hgqd", p, v).permute(2, 0, 1, 3).reshape(ql, Hq * Dv).to(q.dtype)
+    return out
+
+
 def sample(logits, temperature, top_k, top_p, uniforms, num_logprobs=0):
     """Row-wise reference of the fused sampler; ``uniforms`` [B] in [0,1) replaces the device RNG."""
     B, V = logits.shape

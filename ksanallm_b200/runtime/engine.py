@@ -108,6 +108,7 @@ class ModelRunner:
         self._swap_stream = None
         self.exchange_candidates = os.environ.get("KSANA_SHARD_SAMPLING", "1") != "0"
         self.pipeline = None             # parallel.pipeline.PipelineRunner when the job has several stages
+        self.needs_prev_ids = bool(getattr(model, "needs_prev_ids", False))
         self.h2d_bytes = 0
         self.d2h_bytes = 0
 
@@ -203,15 +204,18 @@ class ModelRunner:
     def _stage_plan(self, plan) -> torch.Tensor:
         """The step's device metadata (ids, positions, slots, sequence offsets, lengths, block table, sample rows) in
         one upload. A scheduler plan writes its image straight into the pinned staging buffer."""
+        prev = np.asarray(plan.prev_ids, dtype=np.int32) if self.needs_prev_ids else np.zeros(0, np.int32)
         if self.cuda and hasattr(plan, "write_step_image"):
-            n = int(plan.step_image_words())
+            n = int(plan.step_image_words()) + prev.size
             slot = self._stage_buffer(n)
             plan.write_step_image(slot[0].data_ptr(), slot[1])
+            if prev.size:
+                slot[0].numpy()[n - prev.size:n] = prev
             self.h2d_bytes += n * 4
             dev = slot[0][:n].to(self.device, non_blocking=True)
             slot[2].record()
             return dev
-        parts = [plan.input_ids, plan.positions, plan.slots, plan.cu_q, plan.kv_lens, plan.block_table, plan.sample_rows]
+        parts = [plan.input_ids, plan.positions, plan.slots, plan.cu_q, plan.kv_lens, plan.block_table, plan.sample_rows, prev]
         return self._stage(np.concatenate([np.asarray(p, dtype=np.int32).reshape(-1) for p in parts]))
 
     def _patch_ids(self, ids: torch.Tensor, patch) -> None:
@@ -246,6 +250,8 @@ class ModelRunner:
         rows = take(nsamp)
         step = StepInput(input_ids, positions, slots, cu_q, kv_lens, table, plan.num_multi, plan.num_single, T,
                          plan.num_multi_tokens, plan.max_q_len, logits_rows=rows)
+        if self.needs_prev_ids:
+            step.prev_ids = take(T)
         kv_lens = np.asarray(plan.kv_lens)
         step.max_kv_len = int(kv_lens.max()) if nseq else 0
         step.sample_k = self.candidate_k(plan, extra)
@@ -299,15 +305,17 @@ class ModelRunner:
             return g
         mb = self.graph_max_blocks
         n = 4 * bs + bs * mb
-        img = torch.zeros(n, dtype=torch.int32, device=self.device)
+        img = torch.zeros(n + (bs if self.needs_prev_ids else 0), dtype=torch.int32, device=self.device)
         ids, pos, slots, kvl = img[0:bs], img[bs:2 * bs], img[2 * bs:3 * bs], img[3 * bs:4 * bs]
-        table = img[4 * bs:].view(bs, mb)
+        table = img[4 * bs:n].view(bs, mb)
         slots.fill_(-1)
         cu_q = torch.arange(bs + 1, dtype=torch.int32, device=self.device)
         step = StepInput(ids, pos, slots, cu_q, kvl, table, 0, bs, bs, 0, 1, logits_rows=None)
         step.decode_splits = ops.decode_splits(bs, self.model.Hkv, self.graph_max_kv)
         step.max_kv_len = self.graph_max_kv
         step.sample_k = kx
+        if self.needs_prev_ids:
+            step.prev_ids = img[n:]
         side = torch.cuda.Stream(device=self.device)
         side.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(side):
@@ -327,14 +335,19 @@ class ModelRunner:
         nseq = len(plan.seq_ids)
         if getattr(self, "graphs", None) is None or plan.num_multi or nseq == 0 or nseq > self.graph_max_batch:
             return None
-        if plan.sample_rows.size != nseq or plan.max_blocks > self.graph_max_blocks:
-            return None
+        if plan.max_blocks > self.graph_max_blocks or not np.array_equal(plan.sample_rows, np.arange(nseq)):
+            return None                  # the graph returns one logits row per sequence, in order
         bs = next(b for b in self.GRAPH_SIZES if b >= nseq)
         graph, img, logits, mb, _step = self._graph_for(bs, self.candidate_k(plan, None))
-        n = 4 * bs + bs * mb
+        n0 = n = 4 * bs + bs * mb
+        prev = np.full(bs if self.needs_prev_ids else 0, -1, dtype=np.int32)
+        if prev.size:
+            prev[:nseq] = plan.prev_ids
+            n += bs
         if hasattr(plan, "write_decode_image"):
             slot = self._stage_buffer(n)                  # the plan writes the padded image into pinned memory itself
             plan.write_decode_image(slot[0].data_ptr(), slot[1], bs, mb)
+            slot[0].numpy()[n0:n] = prev
             self.h2d_bytes += n * 4
             img.copy_(slot[0][:n], non_blocking=True)
             slot[2].record()
@@ -345,7 +358,8 @@ class ModelRunner:
             host[2 * bs:3 * bs] = -1
             host[2 * bs:2 * bs + nseq] = plan.slots
             host[3 * bs:3 * bs + nseq] = plan.kv_lens
-            tbl = host[4 * bs:].reshape(bs, mb)
+            host[n0:] = prev
+            tbl = host[4 * bs:n0].reshape(bs, mb)
             tbl[:nseq, :plan.max_blocks] = np.asarray(plan.block_table).reshape(nseq, plan.max_blocks)
             self._stage(host, out=img)
         if patch is not None:
@@ -905,6 +919,35 @@ class LLMEngine:
         tm["steps"] = tm.get("steps", 0) + 1
         self._phase_wall(phase, t0)
         return True
+
+    # ------------------------------------------------------------------ given-token stepping
+    # Replaying a trace or scoring given text: the caller names every step's sequences and tokens and the rows whose
+    # logits it wants. Blocks, step metadata and the forward are those of generation; nothing is sampled.
+    def open_given(self) -> int:
+        """A new sequence whose tokens the caller will supply."""
+        with self._lock:
+            req_id = self._next_req
+            self._next_req += 1
+        return int(self.scheduler.open_given(req_id))
+
+    def step_given(self, entries) -> torch.Tensor:
+        """One step over ``entries`` (sequence id, next tokens, wanted places among them), all in one batch. Returns the
+        logits [wanted rows, vocab] in the order of the entries and their places."""
+        if self.world_size > 1:
+            raise RuntimeError("given-token steps run on a single rank")
+        code, message, plan, order = self.scheduler.plan_given([(int(s), list(t), list(w)) for s, t, w in entries])
+        if code != 0:
+            raise RuntimeError(message)
+        logits, _ = self.run_with_extras(plan, None)
+        self.scheduler.advance(plan)
+        self.steps += 1
+        out = torch.empty_like(logits)
+        out[torch.from_numpy(order.astype(np.int64)).to(logits.device)] = logits
+        return out
+
+    def close_given(self, seq_id: int) -> None:
+        """The sequence is finished: its blocks go back to the pool."""
+        self.scheduler.finish_sequence(int(seq_id), -1, 0, "")
 
     def _sample(self, plan, logits):
         sample_seq_ids = plan.sample_seq_ids.tolist()

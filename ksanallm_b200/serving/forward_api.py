@@ -86,5 +86,5 @@ def extract_targets(engine, plan, logits) -> None:
                     else:
                         sel = pos
                     idx = torch.tensor([row0 + i for i in sel], dtype=torch.long, device=src.device)
-                    req.response[name] = src[idx].float().cpu()
+                    req.response[name] = src[idx][:, :model.cfg.hidden_size].float().cpu()     # (rows may be padded)
         row0 += ql
