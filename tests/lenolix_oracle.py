@@ -1,5 +1,6 @@
 """Plain, slow statement of the Lenolix decoder: whole sequences, no cache, one function per mechanism. Shares no code
 with the package; every function works in the dtype of its inputs (float32 or float64)."""
+import functools
 import math
 
 import torch
@@ -47,13 +48,10 @@ def rope_frequencies(dims, base, scaling):
 def rotate(x, position, freqs):
     """x [..., dim] of one position: dimension i turns with dimension i + n (n = number of frequencies)."""
     n = len(freqs)
-    y = x.clone()
-    for i, f in enumerate(freqs):
-        c, s = math.cos(position * f), math.sin(position * f)
-        u, v = x[..., i], x[..., i + n]
-        y[..., i] = u * c - v * s
-        y[..., i + n] = v * c + u * s
-    return y
+    c = torch.tensor([math.cos(position * f) for f in freqs], dtype=x.dtype)
+    s = torch.tensor([math.sin(position * f) for f in freqs], dtype=x.dtype)
+    u, v = x[..., :n], x[..., n:2 * n]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * n:]], dim=-1)
 
 
 def visible(i, j, mask):
@@ -62,11 +60,17 @@ def visible(i, j, mask):
     return mask is None or i - j < mask["size"] or j < mask["keep_first"]
 
 
+@functools.lru_cache(maxsize=None)
+def _visibility(T, size, keep_first):
+    mask = None if size is None else {"size": size, "keep_first": keep_first}
+    return torch.tensor([[visible(i, j, mask) for j in range(T)] for i in range(T)])
+
+
 def attend(q, k, v, sink, scale, mask):
     """One head: q [T, dim], k [T, dim], v [T, vdim]; ``sink``: extra logit in the denominator (or None)."""
     T = q.shape[0]
     out = torch.zeros(T, v.shape[1], dtype=q.dtype)
-    see = torch.tensor([[visible(i, j, mask) for j in range(T)] for i in range(T)])
+    see = _visibility(T, None if mask is None else mask["size"], None if mask is None else mask["keep_first"])
     s = (q @ k.t()) * scale
     for i in range(T):
         si = s[i][see[i]]
