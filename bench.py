@@ -187,7 +187,23 @@ def main():
     ap.add_argument("--breakdown", action="store_true",
                     help="instead of the benchmark: device time of one decode step and one prefill step of this model by "
                          "kernel class (benchmarks/step_breakdown.py; --layers limits the depth, --comm picks the path)")
+    ap.add_argument("--design", default=None, choices=["lenolix"],
+                    help="instead of the benchmark: prefill and decode throughput of this model family beside the dense "
+                         "model at equal sizes, kernel by kernel (benchmarks/lenolix_bench.py)")
+    ap.add_argument("--sizes", default="1b,3b,8b", help="--design: sizes to run")
+    ap.add_argument("--window", type=int, default=512, help="--design: sliding window")
+    ap.add_argument("--keep-first", type=int, default=64, help="--design: first tokens that stay visible")
+    ap.add_argument("--prefill-batch", type=int, default=4, help="--design: sequences of the prefill step")
+    ap.add_argument("--prefill-len", type=int, default=2048, help="--design: tokens per sequence of the prefill step")
+    ap.add_argument("--decode-batch", type=int, default=64, help="--design: sequences of the decode step")
+    ap.add_argument("--decode-ctx", type=int, default=2048, help="--design: context of the decode step")
+    ap.add_argument("--reps", type=int, default=20, help="--design: timed replays")
     args = ap.parse_args()
+
+    if args.design is not None:
+        from benchmarks import lenolix_bench
+        args.layers = args.layers or 8
+        return lenolix_bench.main(args)
 
     if args.breakdown:
         from benchmarks import step_breakdown

@@ -85,15 +85,18 @@ def build_step(torch, model, phase, batch, ctx, q_len, block_tokens):
     rows = None if phase == "decode" else (cu_q[1:] - 1).to(torch.int32)
     step = StepInput(ids, pos, slots, cu_q, kv_lens, table, logits_rows=rows, **step_kw)
     step.max_kv_len = kv
+    if model.needs_prev_ids:
+        step.prev_ids = torch.roll(ids, 1)
     if phase == "decode":
         step.decode_splits = ops.decode_splits(batch, model.Hkv, kv)
     return step, batch * bps
 
 
 def run_breakdown(model, phase="decode", batch=64, ctx=2176, q_len=2048, reps=10, block_tokens=16, sync_all=None,
-                  classes=True):
+                  classes=True, cost=None):
     """``classes=False`` times the whole step only: needed when a kernel of one class waits for a flag that a kernel of
-    another class raises (a graph of one class alone would wait until its limit)."""
+    another class raises (a graph of one class alone would wait until its limit). ``cost(entry point, arguments)`` ->
+    (job, bytes, operations) adds these to every class."""
     import torch
     from ksanallm_b200.ops import native
     step, nblocks = build_step(torch, model, phase, batch, ctx, q_len, block_tokens)
@@ -112,9 +115,11 @@ def run_breakdown(model, phase="decode", batch=64, ctx=2176, q_len=2048, reps=10
             with torch.cuda.graph(full):
                 keep = model.forward(step)
         t_full = _time_graph(torch, full, reps, sync_all)
-        groups = OrderedDict()
+        groups, costs = OrderedDict(), {}
         for name, fn, args in calls:
             groups.setdefault(_class_key(name, args), []).append((fn, args))
+            if cost is not None:
+                costs.setdefault(_class_key(name, args), cost(name, args))
         rows = []
         for key, lst in (groups.items() if classes else ()):
             g = torch.cuda.CUDAGraph()
@@ -124,6 +129,8 @@ def run_breakdown(model, phase="decode", batch=64, ctx=2176, q_len=2048, reps=10
                     fn(*args[:-1], st)                   # the stream is every entry point's last argument
             t = _time_graph(torch, g, reps, sync_all)
             rows.append({"class": key, "launches": len(lst), "us_total": round(t, 1), "us_each": round(t / len(lst), 2)})
+            if key in costs:
+                rows[-1].update(zip(("job", "bytes", "flops"), costs[key]))
             del g
         native.check_err_flag(model.device)
     s = sum(r["us_total"] for r in rows)

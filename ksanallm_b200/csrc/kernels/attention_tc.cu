@@ -192,7 +192,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       const int t0 = tile_start(j);
       if (!mbar_wait(s_full, par, abort_flag)) { ok = false; break; }
       tc_fence_after();
-      const bool need_mask = (t0 + kFaTile - 1 > limit) || slope2 != 0.f || p.scale_log2 <= 0.f ||
+      const bool biased = slope2 != 0.f || p.scale_log2 <= 0.f;
+      const bool need_mask = (t0 + kFaTile - 1 > limit) ||
                              (WIN && t0 < lo && t0 + kFaTile > keep);
       // lazy rescale of O: keep the old reference maximum unless the row's maximum grew by more than 2^8
       auto update_reference = [&](float mx) {
@@ -215,12 +216,18 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
         m_used = m_new;
         return (m_used == -CUDART_INF_F) ? 0.f : m_used;
       };
-      if (!__any_sync(0xffffffffu, need_mask)) {
-        // interior tile: the whole row in registers with a single TMEM round trip
+      if (!__any_sync(0xffffffffu, biased)) {
+        // the whole row in registers with a single TMEM round trip; hidden keys (window, diagonal) become -inf there
         uint32_t r[128];
 #pragma unroll
         for (int c = 0; c < 4; ++c) tmem_ld32(tmem_s + lane_off + c * 32, *reinterpret_cast<uint32_t(*)[32]>(&r[c * 32]));
         tmem_ld_wait();
+        if (__any_sync(0xffffffffu, need_mask)) {
+          const int last = limit - t0, first = lo - t0, kept = keep - t0;       // column bounds of this row
+#pragma unroll
+          for (int i = 0; i < 128; ++i)
+            if (i > last || (WIN && i < first && i >= kept)) r[i] = 0xff800000u;
+        }
         float mx4[4] = {-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F};
 #pragma unroll
         for (int i = 0; i < 128; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(r[i]));
@@ -238,7 +245,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
 #pragma unroll
         for (int c = 0; c < 4; ++c) tmem_st16(tmem_s + lane_off + c * 16, *reinterpret_cast<uint32_t(*)[16]>(&r[c * 16]));
       } else {
-        // diagonal / last / ALiBi tile: masked two-pass form
+        // ALiBi (or a scale that is not positive): masked two-pass form
         float mx = -CUDART_INF_F;
 #pragma unroll
         for (int c = 0; c < 4; ++c) {

@@ -309,55 +309,48 @@ __global__ void qkv_rope_append_kernel(T* __restrict__ qkv, const int* __restric
   T* vdst = vc + static_cast<size_t>(blk) * block_stride + static_cast<size_t>(off) * Dv;
   const size_t kh = static_cast<size_t>(block_tokens) * D, vh = static_cast<size_t>(block_tokens) * Dv;   // per-head panels
   const float* cs = cos_sin + static_cast<size_t>(pos) * rot;
-  if ((half & 7) == 0) {
-    const int hv = half >> 3, pv = (D - rot) >> 3, per = hv + pv;      // items per head: rotated pairs, then plain vectors
-    for (int i = threadIdx.x; i < (Hq + Hkv) * per; i += blockDim.x) {
-      const int h = i / per, j = i - h * per;
+  // one item list per token, so that all of a token's loads are in flight at once: rotated vectors of q and k, then
+  // the rest of k, then v (the rest of q stays where it is)
+  const bool vec = (half & 7) == 0;
+  const int unit = vec ? 8 : 1;
+  const int hv = half / unit, pv = (D - rot) / unit, dv8 = Dv >> 3;
+  const int n_rot = (Hq + (slot >= 0 ? Hkv : 0)) * hv, n_rest = slot >= 0 ? Hkv * pv : 0, n_v = slot >= 0 ? Hkv * dv8 : 0;
+  for (int i = threadIdx.x; i < n_rot + n_rest + n_v; i += blockDim.x) {
+    if (i < n_rot) {
+      const int h = i / hv, j = (i - h * hv) * unit;
       T* src = row + static_cast<size_t>(h) * D;
-      const bool key = h >= Hq;
-      if (key && slot < 0) continue;
-      T* dst = key ? kdst + (h - Hq) * kh : src;
-      if (j < hv) {
+      T* dst = h >= Hq ? kdst + (h - Hq) * kh : src;
+      if (vec) {
         float a[8], b[8], c[8], s[8], ra[8], rb[8];
-        load8(src + j * 8, a);
-        load8(src + half + j * 8, b);
-        load8(cs + j * 8, c);
-        load8(cs + half + j * 8, s);
+        load8(src + j, a);
+        load8(src + half + j, b);
+        load8(cs + j, c);
+        load8(cs + half + j, s);
 #pragma unroll
         for (int e = 0; e < 8; ++e) { ra[e] = a[e] * c[e] - b[e] * s[e]; rb[e] = b[e] * c[e] + a[e] * s[e]; }
-        store8(dst + j * 8, ra);
-        store8(dst + half + j * 8, rb);
-      } else if (key) {
-        float a[8];
-        load8(src + rot + (j - hv) * 8, a);
-        store8(dst + rot + (j - hv) * 8, a);
-      }
-    }
-  } else {
-    const int pl = D - rot, per = half + pl;
-    for (int i = threadIdx.x; i < (Hq + Hkv) * per; i += blockDim.x) {
-      const int h = i / per, j = i - h * per;
-      T* src = row + static_cast<size_t>(h) * D;
-      const bool key = h >= Hq;
-      if (key && slot < 0) continue;
-      T* dst = key ? kdst + (h - Hq) * kh : src;
-      if (j < half) {
+        store8(dst + j, ra);
+        store8(dst + half + j, rb);
+      } else {
         const float a = to_f(src[j]), b = to_f(src[half + j]), c = cs[j], s = cs[half + j];
         dst[j] = from_f<T>(a * c - b * s);
         dst[half + j] = from_f<T>(b * c + a * s);
-      } else if (key) {
-        dst[rot + j - half] = src[rot + j - half];
       }
+    } else if (i < n_rot + n_rest) {
+      const int k = i - n_rot, h = k / pv, j = rot + (k - h * pv) * unit;
+      const T* src = row + static_cast<size_t>(Hq + h) * D;
+      if (vec) {
+        float a[8];
+        load8(src + j, a);
+        store8(kdst + h * kh + j, a);
+      } else {
+        kdst[h * kh + j] = src[j];
+      }
+    } else {
+      const int k = i - n_rot - n_rest, h = k / dv8, j = (k - h * dv8) * 8;
+      float a[8];
+      load8(row + static_cast<size_t>(Hq + Hkv) * D + h * Dv + j, a);
+      store8(vdst + h * vh + j, a);
     }
-  }
-  if (slot < 0) return;
-  const T* vsrc = row + static_cast<size_t>(Hq + Hkv) * D;
-  const int dv8 = Dv >> 3;
-  for (int i = threadIdx.x; i < Hkv * dv8; i += blockDim.x) {
-    const int h = i / dv8, j = i - h * dv8;
-    float a[8];
-    load8(vsrc + h * Dv + j * 8, a);
-    store8(vdst + h * vh + j * 8, a);
   }
 }
 
@@ -440,8 +433,8 @@ extern "C" int ksana_qkv_rope_append(void* qkv, const int* positions, const int*
   if (T <= 0) return 0;
   if (D % 8 || Dv % 8 || rot < 0 || rot > D || (rot & 1) || block_tokens <= 0 || block_stride % 8 || (rot && !cos_sin)) return -10;
   if (!aligned16(qkv) || !aligned16(kc) || !aligned16(vc) || !aligned16(cos_sin)) return -11;
-  const int items = (Hq + Hkv) * (D / 8);
-  const int threads = items >= 256 ? 256 : (items + 31) / 32 * 32;
+  const int items = (rot % 16 ? (Hq + Hkv) * (rot / 2) : (Hq + Hkv) * (rot / 16) + Hkv * ((D - rot) / 8)) + Hkv * (Dv / 8);
+  const int threads = items >= 512 ? 512 : (items + 31) / 32 * 32;
   cudaError_t e;
   if (f32)
     e = launch_pdl(qkv_rope_append_kernel<float>, dim3(T), dim3(threads), 0, st, (float*)qkv, positions, slots, cos_sin, max_pos,

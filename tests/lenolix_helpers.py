@@ -60,6 +60,14 @@ CONFIGS = {
 }
 
 
+# layouts that split evenly over ranks, with sizes that do not
+SPLIT = {
+    "wide2": config(70, 151, [entry(mixer(4, 2, 20, 12, {"size": 9, "keep_first": 2}, _rot(10)), 51)], None, (31, 5, 2)),
+    "unequal4": config(72, 90, [entry(mixer(4, 2, 24, 16, {"size": 13, "keep_first": 3}, ROTATION), 50),
+                                entry(mixer(8, 4, 8, 8, None, _rot(8)))], (0, 1, 2)),
+}
+
+
 def shapes(c):
     W, out = c["width"], {}
     out["embed"] = (c["vocab"], W)

@@ -410,3 +410,29 @@ def test_these_tests_would_notice():
         assert planted(lambda cc: cc["layers"][0]["mixer"]["rot"].update(scaling=None)) > bar
         assert planted(None, {k: v for k, v in w.items() if not k.endswith("sink")}) > bar
         assert planted(None, {**w, "loop.step": w["loop.step"].flip(0)}) > bar
+
+
+# ------------------------------------------------------------------------------------------------ several ranks
+@pytest.mark.parametrize("name,world", [("grouped", 2), ("wide2", 2), ("unequal4", 4)])
+def test_tensor_parallel_shards(tmp_path, name, world):
+    """Heads, feed-forward columns and the vocabulary split over ranks (key/value heads shared where there are fewer)."""
+    import socket
+    with socket.socket() as s:
+        s.bind(("127.0.0.1", 0))
+        port = s.getsockname()[1]
+    out = str(tmp_path / "logits.pt")
+    r = subprocess.run([sys.executable, "-m", "torch.distributed.run", "--nnodes=1", f"--nproc-per-node={world}", "--master-addr",
+                        "127.0.0.1", "--master-port", str(port), os.path.join(ROOT, "tests", "lenolix_tp_worker.py"), out, name],
+                       env=dict(os.environ, CUDA_VISIBLE_DEVICES="", OMP_NUM_THREADS="2"), capture_output=True, text=True, timeout=300)
+    assert r.returncode == 0, r.stderr[-3000:]
+    c = hlp.SPLIT.get(name) or CONFIGS[name]
+    check(torch.load(out), oracle.forward(hlp.tokens(c, 60), c, hlp.weights(c, 3)), torch.float32, "cpu")
+
+
+def test_layouts_that_cannot_be_split_are_refused():
+    from ksanallm_b200.models.weights import DictSource, build_model
+    cfg = model_config_from_hf(copy.deepcopy(CONFIGS["odd"]))
+    with pytest.raises(ValueError):
+        build_model(cfg, DictSource(weights_of("odd"), "lenolix"), 0, 2)
+    with pytest.raises(ValueError):
+        build_model(cfg, DictSource(weights_of("odd"), "lenolix"), layer_range=(0, 0))
