@@ -84,6 +84,14 @@ def prepare_config(args):
             args.model_type = "qwen_vl"
 
 
+def has_tokenizer(folder) -> bool:
+    """Whether a folder holds anything a tokenizer could be made of (a checkpoint without one is served by token ids)."""
+    if not folder or not os.path.isdir(folder):
+        return False
+    return any(n.startswith(("tokeniz", "vocab", "merges", "spiece", "sentencepiece", "preprocessor_config")) or
+               n.endswith((".tiktoken", ".model")) for n in os.listdir(folder))
+
+
 def load_tokenizer(tokenizer_dir: str):
     """Tokenizer of a checkpoint directory, by the reference server's rules (src/ksana_llm/python/serving_server.py:381-390):
     a directory whose tokenizer_config.json names ``LlamaTokenizer`` gets that class itself (the automatic choice may
@@ -378,7 +386,7 @@ def main(argv=None):
     args = args_config(argv)
     logger.install_logging_handler()          # uvicorn / serving records go to the engine's log sink (KLLM_LOG_FILE)
     logger.info(f"serving_server starting: config {args.config_file}, endpoint {args.endpoint} on {args.host}:{args.port}")
-    tokenizer = load_tokenizer(args.tokenizer_dir) if args.tokenizer_dir and os.path.isdir(args.tokenizer_dir) else None
+    tokenizer = load_tokenizer(args.tokenizer_dir) if has_tokenizer(args.tokenizer_dir) else None
     model = ServingModel(args.config_file, tokenizer=tokenizer)
     plugin_config = PluginConfig(model_dir=args.model_dir, config_file=args.config_file, plugin_name=args.model_type,
                                  enable_trt=args.plugin_enable_trt, thread_pool_size=args.plugin_thread_pool_size)

@@ -355,6 +355,41 @@ def test_trace_replay_refuses_what_has_no_32_bit_path(tmp_path):
     assert p.returncode == 3
 
 
+def test_served_over_http_by_token_ids(tmp_path):
+    """The server's entry point from a YAML file, for a checkpoint without a tokenizer."""
+    import time
+    import urllib.error
+    import urllib.request
+    import socket
+    name = "grouped"
+    hlp.save_checkpoint(str(tmp_path / "model"), CONFIGS[name], weights_of(name))
+    (tmp_path / "serve.yaml").write_text(
+        "setting:\n  batch_scheduler: {max_token_len: 128, max_batch_size: 4}\n"
+        "  block_manager: {device_blocks_num: 40, host_blocks_num: 4}\n"
+        "model_spec:\n  base_model: {model_dir: model}\n")
+    with socket.socket() as s:
+        s.bind(("127.0.0.1", 0))
+        port = s.getsockname()[1]
+    p = subprocess.Popen([sys.executable, os.path.join(ROOT, "serving_server.py"), "--config_file", str(tmp_path / "serve.yaml"),
+                          "--host", "127.0.0.1", "--port", str(port)], env=dict(os.environ, CUDA_VISIBLE_DEVICES=""),
+                         stdout=subprocess.DEVNULL, stderr=subprocess.DEVNULL, cwd=str(tmp_path))
+    try:
+        prompt = hlp.tokens(CONFIGS[name], 20, 80)
+        body = json.dumps({"input_tokens": prompt, "sampling_config": {"max_new_tokens": 8, "ignore_eos": True}}).encode()
+        for _ in range(120):
+            try:
+                r = urllib.request.urlopen(urllib.request.Request(f"http://127.0.0.1:{port}/generate", body,
+                                                                  {"Content-Type": "application/json"}), timeout=60)
+                break
+            except (urllib.error.URLError, ConnectionError):
+                assert p.poll() is None
+                time.sleep(0.5)
+        assert_greedy(name, prompt, json.loads(r.read().split(b"\0")[0])["output_token_ids"][0], torch.bfloat16)
+    finally:
+        p.terminate()
+        p.wait(30)
+
+
 # ------------------------------------------------------------------------------------------------ configuration, loading
 def test_configuration_is_read():
     c = model_config_from_hf(copy.deepcopy(CONFIGS["unequal"]))
