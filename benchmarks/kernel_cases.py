@@ -167,7 +167,7 @@ def _mla(B, q_len, kv_len, G, nsplit):
     out = torch.empty(B * q_len, G, 512, device=DEV, dtype=torch.bfloat16)
 
     def run():
-        native.mla_attention(q, out, layer, layer.stride(0), bt, table, cu, kvl, B, q_len, G, 1 / math.sqrt(192), nsplit)
+        native.mla_attention(q, out, layer, bt, table, cu, kvl, B, q_len, 1 / math.sqrt(192), nsplit)
     # work per launch: causal pairs x heads x (576 + 512) x 2 flops; cache bytes read once
     pairs = B * (q_len * (kv_len - q_len) + q_len * (q_len + 1) // 2)
     run.flops = pairs * G * (576 + 512) * 2

@@ -57,9 +57,9 @@ def engine_lib_path() -> Path:
     return LIB / f"_ksana_engine{suffix}"
 
 
-# what a dense decoder in bf16 or fp32 calls (no FP8 / FP4 / 4-bit weights, experts, latent attention or peer memory)
+# what a dense decoder in bf16 or fp32 calls (no FP8 / FP4 / 4-bit weights, experts or peer memory)
 DENSE_KERNELS = ("attention", "attention_f32", "attention_tc", "elementwise", "gemm_f32", "gemm_smallm", "gemm_tcgen05",
-                 "residual_stream", "sampler")
+                 "mla_attention", "recurrence", "residual_stream", "sampler")
 
 
 def build_kernels(force: bool = False, verbose: bool = False, only=None) -> Path:

@@ -11,9 +11,10 @@ from __future__ import annotations
 
 import json
 import logging
+import math
 import os
 from dataclasses import dataclass, field, fields
-from typing import Any, Dict, List, Optional
+from typing import Any, Dict, List, Optional, Union
 
 import yaml
 
@@ -221,9 +222,36 @@ class MlpSpec:
 
 
 @dataclass
+class LatentAttentionSpec:
+    """Attention over cached latents: per head ``dim`` plain and ``rot_dim`` rotated (pairs 2i, 2i + 1) query and key
+    dimensions and ``vdim`` value dimensions, a sigmoid gate on the output."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int                          # latent size
+    scale: float
+    rotary: RotarySpec
+    window: int = 0                       # sliding window in tokens, 0: full causal attention
+    kv_from: Optional[int] = None         # layer whose cached latents are read; None: the layer's own
+
+
+@dataclass
+class GatedRecurrenceSpec:
+    """Element-wise recurrence whose gates read the current token only."""
+    width: int
+
+
+@dataclass
+class PlainMlpSpec:
+    """up, piecewise unit, down."""
+    size: int
+
+
+@dataclass
 class LayerSpec:
-    mixer: AttentionSpec
-    mlp: Optional[MlpSpec]
+    mixer: Union[AttentionSpec, LatentAttentionSpec, GatedRecurrenceSpec]
+    mlp: Optional[Union[MlpSpec, PlainMlpSpec]]
 
 
 @dataclass
@@ -309,6 +337,8 @@ class ModelConfig:
     layer_specs: Optional[List[LayerSpec]] = None
     loop: Optional[LoopSpec] = None
     pair_embedding: Optional[PairEmbeddingSpec] = None
+    norm_groups: int = 1                  # equal parts of a row that the norms treat one by one
+    residual_mult: float = 1.0            # factor of every sublayer's result
 
     @property
     def is_moe(self) -> bool:
@@ -323,9 +353,9 @@ _ARCH_ALIASES = {
     "llama": "llama", "mistral": "llama", "qwen2": "qwen", "qwen": "qwen", "qwen2_vl": "qwen2_vl", "baichuan": "baichuan",
     "chatglm": "chatglm", "glm": "chatglm", "gpt2": "gpt", "openai-gpt": "gpt", "fairseq-transformer": "gpt", "mixtral": "mixtral",
     "qwen2_moe": "qwen2_moe", "deepseek_v3": "deepseek_v3", "deepseek_v2": "deepseek_v3", "internlm2": "llama",
-    "yi": "llama", "lenolix": "lenolix",
+    "yi": "llama", "lenolix": "lenolix", "rasizen": "rasizen",
 }
-# No position limit is part of the Lenolix design: the serving configuration's max_token_len decides
+# No position limit is part of the Lenolix and Rasizen designs: the serving configuration's max_token_len decides
 _UNBOUNDED_POSITIONS = 1 << 20
 
 
@@ -405,6 +435,8 @@ def model_config_from_hf(hf: dict, generation: Optional[dict] = None, model_dir:
     arch = resolve_architecture(mt, model_dir)
     if arch == "lenolix":
         return lenolix_config(hf, generation)
+    if arch == "rasizen":
+        return rasizen_config(hf, generation)
     c = ModelConfig(model_type=arch, hf_model_type=mt)
     if arch == "gpt":
         c.hidden_size = hf.get("n_embd", hf.get("hidden_size", hf.get("decoder_embed_dim", 768)))
@@ -498,14 +530,17 @@ def model_config_from_hf(hf: dict, generation: Optional[dict] = None, model_dir:
             c.weight_block_size = q.get("weight_block_size")
     td = hf.get("torch_dtype") or hf.get("dtype") or "bfloat16"          # newer exports write "dtype"
     c.dtype = {"float16": "float16", "bfloat16": "bfloat16", "float32": "float32"}.get(str(td).replace("torch.", ""), "bfloat16")
-    eos = (generation or {}).get("eos_token_id", hf.get("eos_token_id"))
-    if eos is not None:
-        c.eos_token_ids = [int(e) for e in (eos if isinstance(eos, (list, tuple)) else [eos])]
+    c.eos_token_ids = _eos_ids(hf, generation)
     pad = hf.get("pad_token_id")
     c.pad_token_id = int(pad) if pad is not None else (1 if mt == "fairseq-transformer" else 0)   # fairseq dictionaries put <pad> at 1
     if c.num_heads % max(c.num_kv_heads, 1):
         raise ValueError("num_attention_heads must be a multiple of num_key_value_heads")
     return c
+
+
+def _eos_ids(hf: dict, generation: Optional[dict]) -> List[int]:
+    eos = (generation or {}).get("eos_token_id", hf.get("eos_token_id"))
+    return [] if eos is None else [int(e) for e in (eos if isinstance(eos, (list, tuple)) else [eos])]
 
 
 def _positive(d: dict, key: str, where: str) -> int:
@@ -567,9 +602,59 @@ def lenolix_config(hf: dict, generation: Optional[dict] = None) -> ModelConfig:
         c.loop = LoopSpec(int(loop["start"]), int(loop["stop"]), _positive(loop, "times", "loop"))
         if not 0 <= c.loop.start < c.loop.stop <= len(layers):
             raise ValueError("loop must cover at least one of the layers")
-    eos = (generation or {}).get("eos_token_id", hf.get("eos_token_id"))
-    if eos is not None:
-        c.eos_token_ids = [int(e) for e in (eos if isinstance(eos, (list, tuple)) else [eos])]
+    c.eos_token_ids = _eos_ids(hf, generation)
+    return c
+
+
+def _latent_attention(m: dict, where: str) -> LatentAttentionSpec:
+    rot = m["rot"]
+    a = LatentAttentionSpec(*(_positive(m, k, where) for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank")), float(m["scale"]),
+                            RotarySpec(_positive(rot, "dims", where + ".rot"), float(rot["base"])))
+    if a.rotary.dims != a.rot_dim or a.rot_dim % 2:
+        raise ValueError(f"{where}: rot.dims must equal rot_dim and be even")
+    if m.get("mask"):
+        a.window = _positive(m["mask"], "size", where + ".mask")
+    if m.get("kv_from") is not None:
+        a.kv_from = int(m["kv_from"])
+    return a
+
+
+def rasizen_config(hf: dict, generation: Optional[dict] = None) -> ModelConfig:
+    """config.json of a Rasizen model: ``vocab``, ``width``, ``norm`` (``eps``, ``groups``), ``residual_mult`` and ``layers``
+    (``type``, ``mixer``, ``mlp``)."""
+    layers = []
+    for i, e in enumerate(hf["layers"]):
+        where = f"layers[{i}]"
+        mlp = e.get("mlp")
+        if mlp and mlp.get("kind", "dense") != "dense":
+            raise ValueError(f"{where}: unknown feed-forward kind {mlp['kind']!r}")
+        if e["type"] == "mingru":
+            mixer = GatedRecurrenceSpec(_positive(e["mixer"], "width", where + ".mixer"))
+        elif e["type"] == "latent_attention":
+            mixer = _latent_attention(e["mixer"], where + ".mixer")
+            if mixer.kv_from is not None:
+                src = layers[mixer.kv_from].mixer if 0 <= mixer.kv_from < i else None
+                if not isinstance(src, LatentAttentionSpec) or src.kv_from is not None:
+                    raise ValueError(f"{where}.mixer.kv_from must name an earlier layer with latents of its own")
+                if (src.kv_rank, src.rot_dim, src.rotary) != (mixer.kv_rank, mixer.rot_dim, mixer.rotary):
+                    raise ValueError(f"{where}.mixer: kv_rank, rot_dim and rot must equal those of layer {mixer.kv_from}")
+        else:
+            raise ValueError(f"{where}: unknown mixer type {e['type']!r}")
+        layers.append(LayerSpec(mixer, PlainMlpSpec(_positive(mlp, "ff", where + ".mlp")) if mlp else None))
+    if not layers:
+        raise ValueError("layers is empty")
+    attn = [s.mixer for s in layers if isinstance(s.mixer, LatentAttentionSpec)]
+    heads = math.gcd(*(a.heads for a in attn)) if attn else math.gcd(*(s.mixer.width for s in layers))   # what tensor parallelism splits
+    c = ModelConfig(model_type="rasizen", hf_model_type="rasizen", hidden_size=_positive(hf, "width", "config"), num_layers=len(layers),
+                    num_heads=heads, num_kv_heads=heads, head_dim=attn[0].dim + attn[0].rot_dim if attn else 1,
+                    v_head_dim=attn[0].vdim if attn else 0, intermediate_size=max([s.mlp.size for s in layers if s.mlp] or [0]),
+                    vocab_size=_positive(hf, "vocab", "config"), rms_norm_eps=float(hf["norm"]["eps"]), tie_word_embeddings=True,
+                    position_embedding="per_layer", gated_mlp=False, activation="xielu", layer_specs=layers,
+                    norm_groups=int(hf["norm"].get("groups", 1)), residual_mult=float(hf.get("residual_mult", 1.0)))
+    if c.norm_groups < 1 or c.hidden_size % c.norm_groups:
+        raise ValueError(f"width {c.hidden_size} does not divide into {c.norm_groups} norm groups")
+    c.max_position_embeddings = c.max_token_len = int(hf.get("max_position_embeddings", _UNBOUNDED_POSITIONS))
+    c.eos_token_ids = _eos_ids(hf, generation)
     return c
 
 

@@ -176,6 +176,7 @@ PYBIND11_MODULE(_ksana_engine, m) {
       .def_readwrite("split_fuse_token_num", &SchedulerConfig::split_fuse_token_num)
       .def_readwrite("min_flexible_cache_num", &SchedulerConfig::min_flexible_cache_num)
       .def_readwrite("enable_prefix_cache", &SchedulerConfig::enable_prefix_cache)
+.def_readwrite("resume_at_block_ends", &SchedulerConfig::resume_at_block_ends)
       .def_readwrite("block_token_num", &SchedulerConfig::block_token_num)
       .def_readwrite("auto_batch_wait_ms", &SchedulerConfig::auto_batch_wait_ms)
       .def_readwrite("eos_token_ids", &SchedulerConfig::eos_token_ids);

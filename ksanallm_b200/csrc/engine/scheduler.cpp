@@ -530,8 +530,13 @@ bool Scheduler::Schedule(StepPlan* plan) {
     std::vector<int> pre_blocks;
     std::vector<BlockCopy> flex_copies;
     int matched = cache.AcquirePrefix(s->tokens, &pre_blocks);
+    if (cfg_.resume_at_block_ends && matched == len && matched > 0) {
+      cache.Release({pre_blocks.back()});      // the last block is computed again, into a block of the sequence's own
+      pre_blocks.pop_back();
+      matched -= B;
+    }
     int flex = 0;
-    if (cfg_.min_flexible_cache_num > 0)
+    if (cfg_.min_flexible_cache_num > 0 && !cfg_.resume_at_block_ends)
       flex = cache.AcquireFlexible(s->tokens, matched, cfg_.min_flexible_cache_num, &pre_blocks, &flex_copies);
     const int cached = std::min(matched + flex, len - 1);    // at least the last token is computed
     const int remaining = len - cached;
@@ -647,7 +652,8 @@ void Scheduler::PostStep(const StepPlan& plan, const std::vector<SampledToken>& 
       if (lit != by_id_.end() && lit->second->state == SeqState::RUNNING) {
         SeqPtr l = lit->second;
         // leader appended its own token already when it precedes us; share only the prompt part
-        const int shared_tokens = std::min(l->kv_cached, s->prompt_len);
+        int shared_tokens = std::min(l->kv_cached, s->prompt_len);
+        if (cfg_.resume_at_block_ends && shared_tokens != l->kv_cached) shared_tokens = shared_tokens / cfg_.block_token_num * cfg_.block_token_num;
         std::vector<BlockCopy> cps;
         if (RankOf(*l) == RankOf(*s) && CacheOf(*l).Fork(l->blocks, shared_tokens, &s->blocks, &cps)) {
           for (auto& c : cps) { c.src += PoolBase(*l); c.dst += PoolBase(*l); }

@@ -37,6 +37,9 @@ struct SchedulerConfig {
   int split_fuse_token_num = 0;
   int min_flexible_cache_num = 0;
   bool enable_prefix_cache = false;
+  // Blocks hold recurrent state as of their last computed token: a sequence resumes at the end of a cached block only
+  // (never inside one, as a fully cached prompt otherwise does to compute its last token again)
+  bool resume_at_block_ends = false;
   int block_token_num = 16;
   int auto_batch_wait_ms = 100;
   // attention data parallelism: sequence s lives on rank s % dp_size and only that rank holds its KV blocks, so

@@ -1,12 +1,16 @@
-// Multi-head latent attention (DeepSeek-V2/V3 "absorbed" form) on the tcgen05 tensor cores, prefill and decode,
-// over the paged latent cache. The reference has no MLA (its attention layers are flash-attention + vLLM paged
+// Multi-head latent attention ("absorbed" form) on the tcgen05 tensor cores, prefill and decode, over the paged latent
+// cache, with an optional sliding window. The reference has no MLA (its attention layers are flash-attention + vLLM paged
 // attention over per-head K/V: src/ksana_llm/layers/nvidia/flash_attention_layer.cpp, paged_attention_layer.cpp);
-// this file is new work for the DeepSeek family.
+// this file is new work.
 //
-// Cache row (one per token and layer): 512 latent values c_kv followed by the 64 rotary key values k_pe, bf16.
-// Query row (one per token and head): q_lat = q_nope W_uk (512) followed by the rotated q_pe (64).
-//   S = Q K^T over all 576 columns, softmax, O = P V with V = the first 512 columns of the same cache rows,
-// i.e. multi-query attention with one shared 576/512-wide "KV head".
+// Cache row (one per token and layer): the latent values c_kv followed by the rotary key values k_pe, bf16, DV and DK - DV
+// of them (DeepSeek-V2/V3: 512 and 64). Query row (one per token and head): q_lat = q_nope W_uk, then the rotated q_pe.
+//   S = Q K^T over all DK columns, softmax, O = P V with V = the first DV columns of the same cache rows,
+// i.e. multi-query attention with one shared "KV head". DK up to 576 and DV up to 512, both multiples of 8: rows are
+// staged as 64-column panels, TMA fills the columns past DK with zeros, and output columns past DV are not stored (those
+// of the last value panel that are key columns are computed and dropped).
+//
+// The sizes in the rest of this comment are those of DK = 576, DV = 512.
 //
 // One CTA owns 128 packed query rows (row = (token, head), all G heads of this rank share every staged tile) and
 // one half (256 columns) of the output. TMEM (512 columns): the O accumulator of the half (256), a double-buffered
@@ -28,17 +32,17 @@
 // Every wait is bounded; a timeout sets the error word and leaves the output untouched.
 #include "sm100_ptx.cuh"
 #include "guards.cuh"
-#include <cuda_bf16.h>
+#include "pdl.cuh"
+#include "vec8.cuh"
 #include <math_constants.h>
 
 namespace ksana {
 
-typedef __nv_bfloat16 bf16;
 constexpr int kMlaThreads = 192;
 constexpr int kMlaM = 128;                    // packed query rows per CTA
 constexpr int kMlaTok = 64;                   // KV tokens per tile
-constexpr int kMlaLora = 512, kMlaDk = 576;
-constexpr int kMlaPanels = 9;                 // 64-column panels of a 576-wide row
+constexpr int kMlaMaxDv = 512, kMlaMaxDk = 576;
+constexpr int kMlaPanels = 9;                 // 64-column panels of the widest row
 constexpr int kMlaQPanelBytes = kMlaM * 128;
 constexpr int kMlaQTmemPanels = 4;            // Q columns [0, 256) live in TMEM (128 columns of bf16 pairs)
 constexpr int kMlaQSmemPanels = kMlaPanels - kMlaQTmemPanels;   // columns [384, 576) stay in shared memory
@@ -53,12 +57,13 @@ static_assert(kMlaQTmemPanels * kMlaQPanelBytes <= kMlaStages * kMlaKvBytes, "Q 
 constexpr float kMlaRescaleLog2 = 8.f;
 
 struct MlaParams {
-  bf16* out; long long out_tok_stride;        // [T, G, 512] bf16, elements between tokens
-  float* part_o; float* part_ml;              // [nsplit, T, G, 512] / [nsplit, T, G, 2] when nsplit > 1
+  bf16* out; long long out_tok_stride;        // [T, G, dv] bf16, elements between tokens
+  float* part_o; float* part_ml;              // [nsplit, T, G, dv] / [nsplit, T, G, 2] when nsplit > 1
   const int* block_table; int table_stride;
   const int* cu_q; const int* kv_lens;
   int G, block_tokens, box_rows, nsplit, T;
-  long long rows_per_block;                   // cache rows (576 elements each) between consecutive blocks
+  int panels, kmmas, dv;                      // 64-column panels of a row, K = 16 steps over its columns, value columns
+  int window;                                 // keys a query sees, itself included; 0: all earlier ones
   int num_blocks;                             // blocks addressable from the layer base (block-table entries are checked)
   float scale_log2;
   int* err;
@@ -107,10 +112,14 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
   const int past = kv_len - q_len;
   const int last_row = min(row0 + kMlaM - 1, q_len * G - 1);
   const int kv_end = min(kv_len, past + last_row / G + 1);
-  const int nt_all = (kv_end + kMlaTok - 1) / kMlaTok;
-  const int per = (nt_all + p.nsplit - 1) / p.nsplit;
-  const int tile_lo = split * per;
-  const int ntiles = max(min(nt_all, tile_lo + per) - tile_lo, 0);
+  // tiles from the first key that the first row sees to the last one that the last row sees
+  const int tile_first = p.window > 0 ? max(0, past + row0 / G - p.window + 1) / kMlaTok : 0;
+  const int tile_end = (kv_end + kMlaTok - 1) / kMlaTok;
+  const int per = (tile_end - tile_first + p.nsplit - 1) / p.nsplit;
+  const int tile_lo = tile_first + split * per;
+  const int ntiles = max(min(tile_end, tile_lo + per) - tile_lo, 0);
+  const int panels = p.panels, q_tmem = min(panels, kMlaQTmemPanels);
+  const int cols = min(256, p.dv - half * 256);             // output columns of this half
   const int* table = p.block_table + static_cast<size_t>(s) * p.table_stride;
 
   if (ntiles == 0) {
@@ -128,8 +137,8 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
           }
         } else {
           uint4* dst = reinterpret_cast<uint4*>(p.out + static_cast<size_t>(q0 + vr / G) * p.out_tok_stride +
-                                                (vr % G) * kMlaLora + half * 256);
-          for (int i = 0; i < 32; ++i) dst[i] = make_uint4(0, 0, 0, 0);
+                                                (vr % G) * p.dv + half * 256);
+          for (int i = 0; i < cols / 8; ++i) dst[i] = make_uint4(0, 0, 0, 0);
         }
       }
     }
@@ -156,13 +165,12 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
     if (lane == 0) {
       tma_prefetch_desc(&q_map);
       tma_prefetch_desc(&kv_map);
-      // Q: panels 0..5 into the (still unused) KV stages as a staging area for their copy to TMEM, 6..8 to their home
-      mbar_expect_tx(q_full, kMlaPanels * kMlaQPanelBytes);
-      const int tok0 = q0 + row0 / G;
-#pragma unroll
-      for (int pn = 0; pn < kMlaPanels; ++pn) {
+      // Q: the first panels into the (still unused) KV stages as a staging area for their copy to TMEM, the rest to
+      // their home. Rows of a tile are consecutive (token, head) pairs; those past the sequence are computed and dropped
+      mbar_expect_tx(q_full, panels * kMlaQPanelBytes);
+      for (int pn = 0; pn < panels; ++pn) {
         uint8_t* dst = pn < kMlaQTmemPanels ? kv_s + pn * kMlaQPanelBytes : q_s + (pn - kMlaQTmemPanels) * kMlaQPanelBytes;
-        tma_load_3d(dst, &q_map, q_full, pn * 64, 0, tok0);
+        tma_load_2d(dst, &q_map, q_full, pn * 64, q0 * G + row0);
       }
     }
     __syncwarp();
@@ -195,16 +203,15 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
         if (j + 1 < ntiles) fetch(j + 1, blk_next);
         ok = ok && mbar_wait(kv_empty + b, ((j / kMlaStages) & 1) ^ 1, abort_flag);
         if (!__all_sync(0xffffffffu, ok)) break;
-        if (lane == 0) mbar_expect_tx(kv_full + b, static_cast<uint32_t>(nbox) * br * 128 * kMlaPanels);
+        if (lane == 0) mbar_expect_tx(kv_full + b, static_cast<uint32_t>(nbox) * br * 128 * panels);
         __syncwarp();
-        if (lane < kMlaPanels) {
+        if (lane < panels) {
           uint8_t* dst = kv_s + b * kMlaKvBytes + lane * kMlaKvPanelBytes;
 #pragma unroll
           for (int bx = 0; bx < kMlaMaxBoxes; ++bx) {
             if (bx < nbox) {
               const int t = t0 + bx * br;
-              const long long r0 = static_cast<long long>(blk[bx]) * p.rows_per_block + (t % bt);
-              tma_load_2d(dst + bx * br * 128, &kv_map, kv_full + b, lane * 64, static_cast<int>(r0));
+              tma_load_3d(dst + bx * br * 128, &kv_map, kv_full + b, lane * 64, t % bt, blk[bx]);
             }
           }
         }
@@ -215,7 +222,7 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
     // ------------------------------------------------------------------ MMA issuer
     if (lane == 0) {
       constexpr uint32_t idesc_qk = make_idesc(128, kMlaTok, 1, 1);
-      constexpr uint32_t idesc_pv = make_idesc(128, 256, 1, 1) | (1u << 16);     // B (= V) is MN-major
+      const uint32_t idesc_pv = make_idesc(128, (cols + 63) / 64 * 64, 1, 1) | (1u << 16);     // B (= V) is MN-major
       bool ok = mbar_wait(q_full, 0, abort_flag) && mbar_wait(q_moved, 0, abort_flag);
       tc_fence_after();
       const uint32_t qb = smem_u32(q_s);
@@ -248,8 +255,8 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
           const int bb = s_next & 1;
           tc_fence_after();
           const uint32_t kb = smem_u32(kv_s + (s_next % kMlaStages) * kMlaKvBytes);
-#pragma unroll
-          for (int k = 0; k < 4 * kMlaPanels; ++k) {
+#pragma unroll 4
+          for (int k = 0; k < p.kmmas; ++k) {
             const int pn = k >> 2;
             const uint64_t bdesc = make_smem_desc_sw128(kb + pn * kMlaKvPanelBytes) + 2 * (k & 3);
             if (pn < kMlaQTmemPanels) {
@@ -281,6 +288,7 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
     const bool active = vr < q_len * G;
     const int tok = vr / G, head = vr % G;
     const int limit = active ? past + tok : -1;            // last visible KV position
+    const int lowest = p.window > 0 ? limit - p.window + 1 : 0;              // first visible one
     float m_used = -CUDART_INF_F, l = 0.f;
     bool ok = mbar_wait(q_full, 0, abort_flag);
     if (ok) {
@@ -288,7 +296,7 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
       // layout the MMA reads an A operand from TMEM (row = lane, two consecutive bf16 per 32-bit column)
       const int rr = qd * 32 + lane;
 #pragma unroll 1
-      for (int pn = 0; pn < kMlaQTmemPanels; ++pn) {
+      for (int pn = 0; pn < q_tmem; ++pn) {
         const uint8_t* src = kv_s + pn * kMlaQPanelBytes + rr * 128;
         uint32_t v[32];
 #pragma unroll
@@ -316,7 +324,7 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
       float mx = -CUDART_INF_F;
 #pragma unroll
       for (int i = 0; i < kMlaTok; ++i) {
-        const float v = (t0 + i <= limit) ? __uint_as_float(r[i]) * p.scale_log2 : -CUDART_INF_F;
+        const float v = (t0 + i <= limit && t0 + i >= lowest) ? __uint_as_float(r[i]) * p.scale_log2 : -CUDART_INF_F;
         r[i] = __float_as_uint(v);
         mx = fmaxf(mx, v);
       }
@@ -331,7 +339,7 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
         const float f = grow ? exp2f(m_used - m_new) : 1.f;
         l *= f;
 #pragma unroll 1
-        for (int c = 0; c < 8; ++c) {
+        for (int c = 0; c * 32 < cols; ++c) {
           uint32_t o[32];
           tmem_ld32(tmem_o + lane_off + c * 32, o);
           tmem_ld_wait();
@@ -358,10 +366,10 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
         // last tile of the sequence: rows past the sequence end hold stale shared memory or whatever the cache has
         // there; their probabilities are 0, but 0 x NaN would poison O. Zero them before the P V MMA reads them.
         const int first_bad = kv_len - t0;
-        const int nchunks = (kMlaTok - first_bad) * (kMlaPanels * 8);      // 16-byte chunks
+        const int nchunks = (kMlaTok - first_bad) * (panels * 8);          // 16-byte chunks
         uint8_t* buf = kv_s + (j % kMlaStages) * kMlaKvBytes;
         for (int i = threadIdx.x - 64; i < nchunks; i += 128) {
-          const int rr = first_bad + i / (kMlaPanels * 8), c = i % (kMlaPanels * 8);
+          const int rr = first_bad + i / (panels * 8), c = i % (panels * 8);
           *reinterpret_cast<uint4*>(buf + (c >> 3) * kMlaKvPanelBytes + rr * 128 + ((c & 7) << 4)) = make_uint4(0, 0, 0, 0);
         }
         fence_async_smem();
@@ -374,15 +382,16 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
       tc_fence_after();
       if (p.nsplit == 1) {
         const float inv = l > 0.f ? 1.f / l : 0.f;
-        bf16* dst = p.out + static_cast<size_t>(q0 + tok) * p.out_tok_stride + head * kMlaLora + half * 256;
+        bf16* dst = p.out + static_cast<size_t>(q0 + tok) * p.out_tok_stride + head * p.dv + half * 256;
 #pragma unroll 1
-        for (int c = 0; c < 8; ++c) {
+        for (int c = 0; c * 32 < cols; ++c) {
           uint32_t o[32];
           tmem_ld32(tmem_o + lane_off + c * 32, o);
           tmem_ld_wait();
           if (active) {
 #pragma unroll
             for (int i = 0; i < 32; i += 8) {
+              if (c * 32 + i >= cols) break;
               uint4 ov;
               __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&ov);
 #pragma unroll
@@ -394,16 +403,16 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
         }
       } else {
         const size_t prow = (static_cast<size_t>(split) * p.T + q0 + tok) * G + head;
-        float* dst = p.part_o + prow * kMlaLora + half * 256;
+        float* dst = p.part_o + prow * p.dv + half * 256;
 #pragma unroll 1
-        for (int c = 0; c < 8; ++c) {
+        for (int c = 0; c * 32 < cols; ++c) {
           uint32_t o[32];
           tmem_ld32(tmem_o + lane_off + c * 32, o);
           tmem_ld_wait();
           if (active) {
 #pragma unroll
             for (int i = 0; i < 32; i += 4)
-              *reinterpret_cast<uint4*>(dst + c * 32 + i) = make_uint4(o[i], o[i + 1], o[i + 2], o[i + 3]);
+              if (c * 32 + i < cols) *reinterpret_cast<uint4*>(dst + c * 32 + i) = make_uint4(o[i], o[i + 1], o[i + 2], o[i + 3]);
           }
         }
         if (active && half == 0) {
@@ -426,7 +435,8 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
 
 // Merge of split-KV partials: out[row] = sum_s 2^(m_s - m) O_s / sum_s 2^(m_s - m) l_s. One CTA per (token, head).
 __global__ void mla_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, bf16* __restrict__ out,
-                                 long long out_tok_stride, int T, int G, int nsplit) {
+                                 long long out_tok_stride, int T, int G, int nsplit, int dv) {
+  if (threadIdx.x * 4 >= dv) return;
   const int row = blockIdx.x, tok = row / G, head = row % G;
   const size_t rows = static_cast<size_t>(T) * G;
   float m = -CUDART_INF_F;
@@ -441,7 +451,7 @@ __global__ void mla_merge_kernel(const float* __restrict__ part_o, const float* 
     if (!(ml[1] > 0.f)) continue;
     const float w = exp2f(ml[0] - m);
     denom += w * ml[1];
-    const float4 o = *reinterpret_cast<const float4*>(part_o + (s * rows + row) * kMlaLora + threadIdx.x * 4);
+    const float4 o = *reinterpret_cast<const float4*>(part_o + (s * rows + row) * dv + threadIdx.x * 4);
     acc.x += w * o.x; acc.y += w * o.y; acc.z += w * o.z; acc.w += w * o.w;
   }
   const float inv = denom > 0.f ? 1.f / denom : 0.f;
@@ -449,60 +459,106 @@ __global__ void mla_merge_kernel(const float* __restrict__ part_o, const float* 
   uint2 v;
   v.x = *reinterpret_cast<uint32_t*>(&lo);
   v.y = *reinterpret_cast<uint32_t*>(&hi);
-  *reinterpret_cast<uint2*>(out + static_cast<size_t>(tok) * out_tok_stride + head * kMlaLora + threadIdx.x * 4) = v;
+  *reinterpret_cast<uint2*>(out + static_cast<size_t>(tok) * out_tok_stride + head * dv + threadIdx.x * 4) = v;
 }
 
-// Per token: RMSNorm of the 512 latent values, rotation of the shared rotary key, append of both to the paged
-// latent cache (slot < 0 skips the write), and rotation of every head's q_pe into the packed query rows.
-//   q      [T, G, nope + 64] bf16 (q_b projection), q_stride elements between tokens
-//   kv     [T, 576] bf16 (kv_a projection: raw latent | raw rotary key), kv_stride elements between tokens
-//   qfull  [T, G, 576] bf16: columns [512, 576) are written here, [0, 512) by the q_nope W_uk product
-// Rotation pairs are (2i, 2i+1) ("interleaved"); cos_sin: [max_pos][64] = cos(32) | sin(32).
-__global__ void mla_rope_append_kernel(const bf16* __restrict__ q, long long q_stride, int nope, const bf16* __restrict__ kv,
-                                       long long kv_stride, const bf16* __restrict__ norm_w, float eps,
-                                       const int* __restrict__ positions, const int* __restrict__ slots,
-                                       const float* __restrict__ cos_sin, bf16* __restrict__ qfull, bf16* __restrict__ cache,
-                                       long long rows_per_block, int block_tokens, int G, int max_pos, long long num_slots,
-                                       int* err) {
-  __shared__ float red[4];
-  const int t = blockIdx.x, tid = threadIdx.x;                 // 128 threads
-  const bf16* row = kv + static_cast<size_t>(t) * kv_stride;
-  int pos = positions[t];
-  if (pos < 0 || pos >= max_pos) { if (tid == 0) guard_report(err, kGuardPosition, pos); pos = 0; }
-  const float* cs = cos_sin + static_cast<size_t>(pos) * 64;
-  int slot = slots[t];
-  if (slot >= num_slots) { if (tid == 0) guard_report(err, kGuardSlot, slot); slot = -1; }
-  bf16* crow = nullptr;
-  if (slot >= 0 && cache != nullptr)
-    crow = cache + (static_cast<size_t>(slot / block_tokens) * rows_per_block + slot % block_tokens) * kMlaDk;
-  float v[4];
-  float ss = 0.f;
+// Per token: RMS norm of the latent values, rotation of the shared rotary key, append of both to the paged latent cache
+// (slot < 0 or no kv: skipped), and rotation of every head's q_pe into the packed query rows.
+//   q      [T, G, nope + rot_p] (query projection), q_stride elements between tokens
+//   kv     [T, rank_p + rot_p] (latent projection: raw latent | raw rotary key), kv_stride elements between tokens
+//   qfull  [T, G, rank_p + rot_p]: columns from rank_p on are written here, the first rank_p by the q_nope W_uk product
+// rank_p and rot_p are the sizes rounded up to multiples of 8; the pad columns of q and kv are zero and stay so. Rotation
+// pairs are (2i, 2i+1) ("interleaved"); cos_sin: [max_pos][rot] = cos(rot/2) | sin(rot/2).
+template <typename T>
+struct LatentParams {
+  const T* q; long long q_stride; int nope;
+  const T* kv; long long kv_stride;
+  const T* norm_w; float eps;
+  const int* positions; const int* slots;
+  const float* cos_sin;
+  T* qfull; T* cache; long long block_stride;            // elements between blocks
+  int block_tokens, G, rank, rank_p, rot, rot_p, max_pos;
+  long long num_slots;
+  int* err;
+};
+
+constexpr int kLatentThreads = 128;
+
+// four pairs of a rotary vector, starting with pair j
+template <typename T>
+__device__ __forceinline__ void rotate8(const T* src, T* dst, const float* cs, int j, int half) {
+  float x[8], y[8];
+  load8(src, x);
 #pragma unroll
-  for (int i = 0; i < 4; ++i) { v[i] = __bfloat162float(row[tid * 4 + i]); ss += v[i] * v[i]; }
+  for (int e = 0; e < 4; ++e) {
+    const bool on = j + e < half;
+    const float c = on ? cs[j + e] : 1.f, s = on ? cs[half + j + e] : 0.f;
+    y[2 * e] = x[2 * e] * c - x[2 * e + 1] * s;
+    y[2 * e + 1] = x[2 * e + 1] * c + x[2 * e] * s;
+  }
+  store8(dst, y);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kLatentThreads) mla_rope_append_kernel(const LatentParams<T> p) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float red[kLatentThreads / 32];
+  const int t = blockIdx.x, tid = threadIdx.x;
+  int pos = p.positions[t];
+  if (pos < 0 || pos >= p.max_pos) { if (tid == 0) guard_report(p.err, kGuardPosition, pos); pos = 0; }
+  const float* cs = p.cos_sin + static_cast<size_t>(pos) * p.rot;
+  const int half = p.rot >> 1, rv = p.rot_p >> 3, dk = p.rank_p + p.rot_p;
+  int slot = p.kv ? p.slots[t] : -1;
+  if (slot >= p.num_slots) { if (tid == 0) guard_report(p.err, kGuardSlot, slot); slot = -1; }
+  if (slot >= 0) {                                           // the same for the whole block
+    const T* row = p.kv + static_cast<size_t>(t) * p.kv_stride;
+    T* crow = p.cache + static_cast<size_t>(slot / p.block_tokens) * p.block_stride + static_cast<size_t>(slot % p.block_tokens) * dk;
+    float ss = 0.f;
+    for (int i = tid * 8; i < p.rank_p; i += kLatentThreads * 8) {
+      float v[8];
+      load8(row + i, v);
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  if ((tid & 31) == 0) red[tid >> 5] = ss;
-  __syncthreads();
-  const float inv = rsqrtf((red[0] + red[1] + red[2] + red[3]) * (1.f / kMlaLora) + eps);
-  if (crow) {
-#pragma unroll
-    for (int i = 0; i < 4; ++i) crow[tid * 4 + i] = __float2bfloat16(v[i] * inv * __bfloat162float(norm_w[tid * 4 + i]));
-    if (tid < 32) {
-      const float x0 = __bfloat162float(row[kMlaLora + 2 * tid]), x1 = __bfloat162float(row[kMlaLora + 2 * tid + 1]);
-      const float c = cs[tid], s = cs[32 + tid];
-      crow[kMlaLora + 2 * tid] = __float2bfloat16(x0 * c - x1 * s);
-      crow[kMlaLora + 2 * tid + 1] = __float2bfloat16(x1 * c + x0 * s);
+      for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
     }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if ((tid & 31) == 0) red[tid >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int w = 0; w < kLatentThreads / 32; ++w) ss += red[w];
+    const float inv = rsqrtf(ss / static_cast<float>(p.rank) + p.eps);
+    for (int i = tid * 8; i < p.rank_p; i += kLatentThreads * 8) {
+      float v[8], w[8];
+      load8(row + i, v);
+      load8(p.norm_w + i, w);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] *= inv * w[e];
+      store8(crow + i, v);
+    }
+    for (int i = tid; i < rv; i += kLatentThreads) rotate8(row + p.rank_p + i * 8, crow + p.rank_p + i * 8, cs, i * 4, half);
   }
-  for (int i = tid; i < G * 32; i += 128) {
-    const int h = i >> 5, j = i & 31;
-    const bf16* qp = q + static_cast<size_t>(t) * q_stride + static_cast<size_t>(h) * (nope + 64) + nope;
-    const float x0 = __bfloat162float(qp[2 * j]), x1 = __bfloat162float(qp[2 * j + 1]);
-    const float c = cs[j], s = cs[32 + j];
-    bf16* dst = qfull + (static_cast<size_t>(t) * G + h) * kMlaDk + kMlaLora;
-    dst[2 * j] = __float2bfloat16(x0 * c - x1 * s);
-    dst[2 * j + 1] = __float2bfloat16(x1 * c + x0 * s);
+  for (int i = tid; i < p.G * rv; i += kLatentThreads) {
+    const int h = i / rv, j = i - h * rv;
+    rotate8(p.q + static_cast<size_t>(t) * p.q_stride + static_cast<size_t>(h) * (p.nope + p.rot_p) + p.nope + j * 8,
+            p.qfull + (static_cast<size_t>(t) * p.G + h) * dk + p.rank_p + j * 8, cs, j * 4, half);
   }
+}
+
+template <typename T>
+static cudaError_t launch_rope_append(const void* q, long long q_stride, int nope, const void* kv, long long kv_stride,
+                                      const void* norm_w, float eps, const int* positions, const int* slots, const float* cos_sin,
+                                      void* qfull, void* cache, long long block_stride, int block_tokens, int T_, int G, int rank,
+                                      int rot, int max_pos, long long num_slots, int* err, cudaStream_t st) {
+  LatentParams<T> p{};
+  p.q = static_cast<const T*>(q); p.q_stride = q_stride; p.nope = nope;
+  p.kv = static_cast<const T*>(kv); p.kv_stride = kv_stride; p.norm_w = static_cast<const T*>(norm_w); p.eps = eps;
+  p.positions = positions; p.slots = slots; p.cos_sin = cos_sin;
+  p.qfull = static_cast<T*>(qfull); p.cache = static_cast<T*>(cache); p.block_stride = block_stride;
+  p.block_tokens = block_tokens; p.G = G; p.rank = rank; p.rank_p = (rank + 7) / 8 * 8; p.rot = rot; p.rot_p = (rot + 7) / 8 * 8;
+  p.max_pos = max_pos; p.num_slots = num_slots; p.err = err;
+  return launch_pdl(mla_rope_append_kernel<T>, dim3(T_), dim3(kLatentThreads), 0, st, p);
 }
 
 typedef CUresult (*MlaEncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
@@ -524,24 +580,25 @@ static MlaEncodeFn mla_encode_fn() {
 
 using namespace ksana;
 
-// Absorbed MLA attention of this step's query rows against the paged latent cache.
-//   q      [T, G, 576] bf16 contiguous (q_lat | rotated q_pe), T = rows addressable from q
-//   out    [T, G, 512] bf16, out_tok_stride elements between tokens
-//   cache  layer base of [block][block_tokens][576] bf16, blocks block_stride elements apart, cache_rows rows addressable
+// Absorbed latent attention of this step's query rows against the paged latent cache.
+//   q      [T, G, dk] bf16 contiguous (q_lat | rotated q_pe), T = rows addressable from q
+//   out    [T, G, dv] bf16, out_tok_stride elements between tokens
+//   cache  layer base of [block][block_tokens][dk] bf16, blocks block_stride elements apart, num_blocks of them
 // Sequences: cu_q [B+1], kv_lens [B] (KV length including this step's rows), block_table [B][table_stride].
-// nsplit > 1 needs part_o [nsplit*T*G*512] and part_ml [nsplit*T*G*2] fp32.
+// window > 0: a query sees itself and the window - 1 tokens before it.
+// nsplit > 1 needs part_o [nsplit*T*G*dv] and part_ml [nsplit*T*G*2] fp32.
 // Returns 0 when launched, -100 when the configuration is not covered (the caller uses its own fallback).
 extern "C" int ksana_mla_attention(const void* q, long long T, void* out, long long out_tok_stride, const void* cache,
                                    long long block_stride, int block_tokens, const int* block_table, int table_stride,
-                                   const int* cu_q, const int* kv_lens, int B, int max_q_len, int G, float scale,
-                                   long long cache_rows, int nsplit, float* part_o, float* part_ml, int* err,
+                                   const int* cu_q, const int* kv_lens, int B, int max_q_len, int G, int dk, int dv, int window,
+                                   float scale, int num_blocks, int nsplit, float* part_o, float* part_ml, int* err,
                                    cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0) return 0;
   const int bt = block_tokens;
-  if (G <= 0 || G > 128 || (G & (G - 1))) return -100;
-  if (bt < 8 || (bt & (bt - 1)) || bt > 256) return -100;
-  if (block_stride % kMlaDk || block_stride < static_cast<long long>(bt) * kMlaDk) return -100;
-  if (cache_rows <= 0 || cache_rows >= (1LL << 31) || T <= 0 || T >= (1LL << 31)) return -100;
+  if (G <= 0 || dk <= 0 || dv <= 0 || dk % 8 || dv % 8 || dv > dk || dk > kMlaMaxDk || dv > kMlaMaxDv || window < 0) return -100;
+  if (bt < 8 || (bt & (bt - 1)) || bt > 256 || B > 65535) return -100;
+  if (block_stride % 8 || block_stride < static_cast<long long>(bt) * dk) return -100;
+  if (num_blocks <= 0 || T <= 0 || T * G >= (1LL << 31)) return -100;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(out)) & 15) return -100;
   if (out_tok_stride % 8) return -100;
   if (nsplit < 1) nsplit = 1;
@@ -551,20 +608,20 @@ extern "C" int ksana_mla_attention(const void* q, long long T, void* out, long l
   const int box_rows = bt < kMlaTok ? bt : kMlaTok;
   CUtensorMap q_map, kv_map;
   {
-    cuuint64_t dims[3] = {static_cast<cuuint64_t>(kMlaDk), static_cast<cuuint64_t>(G), static_cast<cuuint64_t>(T)};
-    cuuint64_t strides[2] = {static_cast<cuuint64_t>(kMlaDk) * 2, static_cast<cuuint64_t>(G) * kMlaDk * 2};
-    cuuint32_t box[3] = {64, static_cast<cuuint32_t>(G), static_cast<cuuint32_t>(kMlaM / G)};
-    cuuint32_t estr[3] = {1, 1, 1};
-    if (enc(&q_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(q), dims, strides, box, estr,
+    cuuint64_t dims[2] = {static_cast<cuuint64_t>(dk), static_cast<cuuint64_t>(T) * G};
+    cuuint64_t strides[1] = {static_cast<cuuint64_t>(dk) * 2};
+    cuuint32_t box[2] = {64, kMlaM};
+    cuuint32_t estr[2] = {1, 1};
+    if (enc(&q_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(q), dims, strides, box, estr,
             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS) return -100;
   }
   {
-    cuuint64_t dims[2] = {static_cast<cuuint64_t>(kMlaDk), static_cast<cuuint64_t>(cache_rows)};
-    cuuint64_t strides[1] = {static_cast<cuuint64_t>(kMlaDk) * 2};
-    cuuint32_t box[2] = {64, static_cast<cuuint32_t>(box_rows)};
-    cuuint32_t estr[2] = {1, 1};
-    if (enc(&kv_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(cache), dims, strides, box, estr,
+    cuuint64_t dims[3] = {static_cast<cuuint64_t>(dk), static_cast<cuuint64_t>(bt), static_cast<cuuint64_t>(num_blocks)};
+    cuuint64_t strides[2] = {static_cast<cuuint64_t>(dk) * 2, static_cast<cuuint64_t>(block_stride) * 2};
+    cuuint32_t box[3] = {64, static_cast<cuuint32_t>(box_rows), 1};
+    cuuint32_t estr[3] = {1, 1, 1};
+    if (enc(&kv_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(cache), dims, strides, box, estr,
             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS) return -100;
   }
@@ -579,32 +636,37 @@ extern "C" int ksana_mla_attention(const void* q, long long T, void* out, long l
   p.part_o = part_o; p.part_ml = part_ml;
   p.block_table = block_table; p.table_stride = table_stride; p.cu_q = cu_q; p.kv_lens = kv_lens;
   p.G = G; p.block_tokens = bt; p.box_rows = box_rows; p.nsplit = nsplit; p.T = static_cast<int>(T);
-  p.rows_per_block = block_stride / kMlaDk;
-  p.num_blocks = static_cast<int>(cache_rows / p.rows_per_block);
+  p.panels = (dk + 63) / 64; p.kmmas = (dk + 15) / 16; p.dv = dv; p.window = window;
+  p.num_blocks = num_blocks;
   p.scale_log2 = scale * 1.44269504f;
   p.err = err;
   const int nqt = (max_q_len * G + kMlaM - 1) / kMlaM;
-  dim3 grid(nqt * nsplit, 2, B);
+  dim3 grid(nqt * nsplit, (dv + 255) / 256, B);
   mla_tc_kernel<<<grid, kMlaThreads, kMlaSmemBytes, st>>>(q_map, kv_map, p);
   if (cudaGetLastError() != cudaSuccess) return -4;
   if (nsplit > 1) {
-    mla_merge_kernel<<<static_cast<unsigned>(T) * G, 128, 0, st>>>(part_o, part_ml, static_cast<bf16*>(out), out_tok_stride,
-                                                                 static_cast<int>(T), G, nsplit);
+    mla_merge_kernel<<<static_cast<unsigned>(T) * G, (dv / 4 + 31) / 32 * 32, 0, st>>>(
+        part_o, part_ml, static_cast<bf16*>(out), out_tok_stride, static_cast<int>(T), G, nsplit, dv);
     if (cudaGetLastError() != cudaSuccess) return -4;
   }
   return 0;
 }
 
+// kv null: only the queries are rotated (the latents are another layer's). f32: fp32 rows and cache instead of bf16.
 extern "C" int ksana_mla_rope_append(const void* q, long long q_stride, int nope, const void* kv, long long kv_stride,
                                      const void* norm_w, float eps, const int* positions, const int* slots,
                                      const float* cos_sin, void* qfull, void* cache, long long block_stride,
-                                     int block_tokens, int T, int G, int max_pos, long long num_slots, int* err,
-                                     cudaStream_t st) {
+                                     int block_tokens, int T, int G, int rank, int rot, int max_pos, long long num_slots,
+                                     int f32, int* err, cudaStream_t st) {
   if (T <= 0) return 0;
-  if (block_stride % kMlaDk) return -10;
-  mla_rope_append_kernel<<<T, 128, 0, st>>>(static_cast<const bf16*>(q), q_stride, nope, static_cast<const bf16*>(kv),
-                                            kv_stride, static_cast<const bf16*>(norm_w), eps, positions, slots, cos_sin,
-                                            static_cast<bf16*>(qfull), static_cast<bf16*>(cache), block_stride / kMlaDk,
-                                            block_tokens, G, max_pos, num_slots, err);
-  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+  if (nope < 0 || nope % 8 || q_stride % 8 || rank <= 0 || rot <= 0 || rot % 2 || G <= 0 || max_pos <= 0) return -10;
+  if (!aligned16(q) || !aligned16(qfull)) return -11;
+  if (kv && (kv_stride % 8 || block_stride % 8 || block_tokens <= 0 || !cache || !norm_w || !aligned16(kv) || !aligned16(cache) ||
+             !aligned16(norm_w))) return -12;
+  const cudaError_t e =
+      f32 ? launch_rope_append<float>(q, q_stride, nope, kv, kv_stride, norm_w, eps, positions, slots, cos_sin, qfull, cache,
+                                      block_stride, block_tokens, T, G, rank, rot, max_pos, num_slots, err, st)
+          : launch_rope_append<bf16>(q, q_stride, nope, kv, kv_stride, norm_w, eps, positions, slots, cos_sin, qfull, cache,
+                                     block_stride, block_tokens, T, G, rank, rot, max_pos, num_slots, err, st);
+  return e == cudaSuccess ? 0 : -4;
 }

@@ -1,51 +1,24 @@
 // Ops around a 32-bit residual stream, for decoders that keep the sum of their sublayers in fp32 and normalise before
-// and after every sublayer. Activations (GEMM operands and results) are bf16, or fp32 in the all-32-bit mode
+// (and some after) every sublayer. Activations (GEMM operands and results) are bf16, or fp32 in the all-32-bit mode
 // (template parameter T); parameters have the activations' type.
 //
 //   embed_pair        x = table[id] * scale (+ pair[hash(previous id, id)]), fp32, plus an optional copy in T
 //   residual_norm     x += scale * norm(y) ; z = norm(x)  - one pass for "norm after the sublayer, layer scale, residual
 //                     add, norm before the next sublayer"; every part is optional (a plain norm, a cast, a row gather)
+//                     The addend may have a scalar factor, and the stream's norm may be taken per part of a row
 //   glu_clamp         min(g, limit) * sigmoid(alpha * g) * (clamp(u, -limit, limit) + offset)
+//   xielu             pos z^2 + lin z (z > 0), neg (exp(z) - 1 - z) + lin z (z <= 0)
+//   sigmoid_gate      a * sigmoid(gate)
 //   qkv_rope_append   rotary embedding on the first rot dims of q and k, k and v into the paged cache; k and v may have
 //                     different head sizes and live in separate panels
 //   refit_rows_f32    rows of x overwritten with given embeddings
 #include "guards.cuh"
 #include "pdl.cuh"
-#include <cuda_bf16.h>
+#include "vec8.cuh"
 #include <cuda_runtime.h>
 #include <stdint.h>
 
 namespace ksana {
-
-typedef __nv_bfloat16 bf16;
-
-// 8 consecutive elements as floats
-__device__ __forceinline__ void load8(const bf16* p, float (&f)[8]) {
-  const uint4 v = *reinterpret_cast<const uint4*>(p);
-  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&v);
-#pragma unroll
-  for (int i = 0; i < 4; ++i) { const float2 t = __bfloat1622float2(h[i]); f[2 * i] = t.x; f[2 * i + 1] = t.y; }
-}
-__device__ __forceinline__ void load8(const float* p, float (&f)[8]) {
-  *reinterpret_cast<float4*>(&f[0]) = *reinterpret_cast<const float4*>(p);
-  *reinterpret_cast<float4*>(&f[4]) = *reinterpret_cast<const float4*>(p + 4);
-}
-__device__ __forceinline__ void store8(bf16* p, const float (&f)[8]) {
-  uint4 v;
-  __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&v);
-#pragma unroll
-  for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
-  *reinterpret_cast<uint4*>(p) = v;
-}
-__device__ __forceinline__ void store8(float* p, const float (&f)[8]) {
-  *reinterpret_cast<float4*>(p) = *reinterpret_cast<const float4*>(&f[0]);
-  *reinterpret_cast<float4*>(p + 4) = *reinterpret_cast<const float4*>(&f[4]);
-}
-__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
-__device__ __forceinline__ float to_f(float v) { return v; }
-template <typename T> __device__ __forceinline__ T from_f(float v);
-template <> __device__ __forceinline__ bf16 from_f<bf16>(float v) { return __float2bfloat16(v); }
-template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
 
 // ------------------------------------------------------------------------------------------------ embedding
 // One CTA per token. H is the padded row width (a multiple of 8; pad columns of the tables are zero). The pair row of
@@ -132,8 +105,60 @@ struct ResNormParams {
   int H;                                // real row width; buffers are padded to a multiple of 8, pads are kept zero
   float eps;
   int rms;                              // 1: root-mean-square norms (no mean, no bias needed)
+  float alpha;                          // factor of the addend, all columns
+  int groups;                           // > 1: the stream's norm takes its mean square per consecutive part of H / groups columns
   int* err;
 };
+
+// z = the row v scaled by the reciprocal root mean square of each of its equal consecutive parts, times w2. Squares are
+// summed per unit (a vector of 8, or a single element where a part is not a multiple of 8) in dynamic shared memory, one
+// warp per part. `part` holds H / unit sums, then one reciprocal per part.
+template <typename T, int VPT>
+__device__ __forceinline__ void grouped_norm(const ResNormParams<T>& p, int m, float (&v)[VPT][8], int nvec) {
+  extern __shared__ float part[];
+  const int size = p.H / p.groups, unit = size % 8 == 0 ? 8 : 1, per = size / unit;
+  float* rstd = part + p.H / unit;
+#pragma unroll
+  for (int j = 0; j < VPT; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i < nvec) {
+      if (unit == 8) {
+        float s = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) s = fmaf(v[j][e], v[j][e], s);
+        part[i] = s;
+      } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) if (i * 8 + e < p.H) part[i * 8 + e] = v[j][e] * v[j][e];
+      }
+    }
+  }
+  __syncthreads();
+  const int lane = threadIdx.x & 31;
+  for (int g = threadIdx.x >> 5; g < p.groups; g += blockDim.x >> 5) {
+    float s = 0.f;
+    for (int k = lane; k < per; k += 32) s += part[g * per + k];
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+    if (lane == 0) rstd[g] = rsqrtf(s / static_cast<float>(size) + p.eps);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int j = 0; j < VPT; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i < nvec) {
+      float wf[8], r0 = unit == 8 ? rstd[i / per] : 0.f;
+      load8(p.w2 + i * 8, wf);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const int c = i * 8 + e;
+        if (unit != 8) r0 = c < p.H ? rstd[c / size] : 0.f;
+        v[j][e] = c < p.H ? v[j][e] * r0 * wf[e] : 0.f;
+      }
+      store8(p.z + static_cast<size_t>(m) * p.ldz + i * 8, v[j]);
+    }
+  }
+}
 
 // One CTA per row, VPT vectors of 8 elements per thread.
 template <typename T, int VPT>
@@ -215,7 +240,7 @@ __global__ void residual_norm_kernel(const ResNormParams<T> p) {
         }
         const int k = min(8, p.H - i * 8);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[j][e] = e < k ? v[j][e] + y[j][e] : 0.f;
+        for (int e = 0; e < 8; ++e) v[j][e] = e < k ? fmaf(p.alpha, y[j][e], v[j][e]) : 0.f;
       }
     }
   }
@@ -227,6 +252,10 @@ __global__ void residual_norm_kernel(const ResNormParams<T> p) {
     }
   }
   if (!p.z) return;
+  if (p.groups > 1) {                   // same for every thread of the launch
+    grouped_norm<T, VPT>(p, m, v, nvec);
+    return;
+  }
   float mean = 0.f, rstd = 1.f;
   if (p.w2) {
     const Moments s = moments_of(v, red[1]);
@@ -252,10 +281,16 @@ template <typename T>
 static int launch_residual_norm(const ResNormParams<T>& p, int M, cudaStream_t st) {
   const int nvec = (p.H + 7) >> 3;
   auto threads = [&](int vpt) { return ((nvec + vpt - 1) / vpt + 31) / 32 * 32; };
+  size_t smem = 0;
+  if (p.groups > 1) {
+    const int size = p.H / p.groups;
+    smem = (static_cast<size_t>(p.H) / (size % 8 == 0 ? 8 : 1) + p.groups) * sizeof(float);
+    if (smem > 46 * 1024) return -10;
+  }
   cudaError_t e;
-  if (nvec <= 256) e = launch_pdl(residual_norm_kernel<T, 1>, dim3(M), dim3(threads(1)), 0, st, p);
-  else if (nvec <= 1024) e = launch_pdl(residual_norm_kernel<T, 2>, dim3(M), dim3(threads(2)), 0, st, p);
-  else if (nvec <= 4096) e = launch_pdl(residual_norm_kernel<T, 4>, dim3(M), dim3(threads(4)), 0, st, p);
+  if (nvec <= 256) e = launch_pdl(residual_norm_kernel<T, 1>, dim3(M), dim3(threads(1)), smem, st, p);
+  else if (nvec <= 1024) e = launch_pdl(residual_norm_kernel<T, 2>, dim3(M), dim3(threads(2)), smem, st, p);
+  else if (nvec <= 4096) e = launch_pdl(residual_norm_kernel<T, 4>, dim3(M), dim3(threads(4)), smem, st, p);
   else return -10;
   return e == cudaSuccess ? 0 : -4;
 }
@@ -282,6 +317,53 @@ __global__ void glu_clamp_kernel(const T* __restrict__ in, T* __restrict__ out, 
     }
     store8(out + static_cast<size_t>(m) * I + i * 8, g);
   }
+}
+
+// ------------------------------------------------------------------------------------------------ elementwise units
+// Piecewise unit of a plain feed-forward: pos z^2 + lin z above zero, neg (exp(z) - 1 - z) + lin z below.
+struct XieluOp {
+  float pos, neg, lin;
+  __device__ __forceinline__ float operator()(float z, float) const {
+    return (z > 0.f ? pos * z * z : neg * (expm1f(z) - z)) + lin * z;
+  }
+};
+// a sigmoid(b)
+struct SigmoidGateOp {
+  __device__ __forceinline__ float operator()(float a, float b) const { return a * sigmoid_f(b); }
+};
+
+// out[m, i] = op(a[m, i], b[m, i]) over rows of I elements (b null: op reads a only); out may alias a.
+template <typename T, typename Op>
+__global__ void rowwise_kernel(const T* a, int lda, const T* b, int ldb, T* out, int ldo, int M, int I, Op op) {
+  pdl_trigger();
+  pdl_wait();
+  const int nvec = I >> 3;
+  const long long total = static_cast<long long>(M) * nvec;
+  for (long long idx = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; idx < total;
+       idx += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const int m = static_cast<int>(idx / nvec), i = static_cast<int>(idx - static_cast<long long>(m) * nvec);
+    float f[8], g[8] = {};
+    load8(a + static_cast<size_t>(m) * lda + i * 8, f);
+    if (b) load8(b + static_cast<size_t>(m) * ldb + i * 8, g);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) f[e] = op(f[e], g[e]);
+    store8(out + static_cast<size_t>(m) * ldo + i * 8, f);
+  }
+}
+
+template <typename Op>
+static int launch_rowwise(const void* a, int lda, const void* b, int ldb, void* out, int ldo, int M, int I, Op op, int f32,
+                          cudaStream_t st) {
+  if (M <= 0) return 0;
+  if (I <= 0 || I % 8 || lda % 8 || lda < I || (b && (ldb % 8 || ldb < I)) || ldo % 8 || ldo < I) return -10;
+  if (!aligned16(a) || !aligned16(b) || !aligned16(out)) return -11;
+  long long g = (static_cast<long long>(M) * (I >> 3) + 255) / 256;
+  if (g > 148 * 8) g = 148 * 8;
+  const dim3 grid(static_cast<unsigned>(g)), block(256);
+  const cudaError_t e =
+      f32 ? launch_pdl(rowwise_kernel<float, Op>, grid, block, 0, st, (const float*)a, lda, (const float*)b, ldb, (float*)out, ldo, M, I, op)
+          : launch_pdl(rowwise_kernel<bf16, Op>, grid, block, 0, st, (const bf16*)a, lda, (const bf16*)b, ldb, (bf16*)out, ldo, M, I, op);
+  return e == cudaSuccess ? 0 : -4;
 }
 
 // ------------------------------------------------------------------------------------------------ rotary + append
@@ -367,8 +449,6 @@ __global__ void refit_rows_f32_kernel(float* __restrict__ x, int ldx, const int*
 
 using namespace ksana;
 
-static inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
-
 // f32: activations and tables are fp32 instead of bf16 (all entry points below)
 extern "C" int ksana_embed_pair(const int* ids, const int* prev, const void* table, const void* pair, float* x, void* copy,
                                 int ldc, int T, int H, int vocab, long long buckets, long long mul_prev, long long mul_cur,
@@ -389,23 +469,24 @@ extern "C" int ksana_embed_pair(const int* ids, const int* prev, const void* tab
 
 extern "C" int ksana_residual_norm(const float* x, int ldx, const int* rows, int in_rows, const void* y, int ldy,
                                    const void* w1, const void* b1, const void* ls, float* x_out, const void* w2,
-                                   const void* b2, void* z, int ldz, int M, int H, float eps, int rms, int f32, int* err,
-                                   cudaStream_t st) {
+                                   const void* b2, void* z, int ldz, int M, int H, float eps, int rms, int f32,
+                                   float alpha, int groups, int* err, cudaStream_t st) {
   if (M <= 0) return 0;
   const int hp = (H + 7) / 8 * 8;
   if (H <= 0 || ldx % 8 || ldx < hp || (y && (ldy % 8 || ldy < hp)) || (z && (ldz % 8 || ldz < hp))) return -10;
   for (const void* q : {(const void*)x, y, w1, b1, ls, (const void*)x_out, w2, b2, (const void*)z})
     if (!aligned16(q)) return -11;
   if (rows && x_out == x) return -12;
+  if (groups > 1 && (!rms || H % groups || w1 || b2 || !w2)) return -13;
   if (f32) {
     typedef float T;
     const ResNormParams<T> p{x, ldx, rows, in_rows, (const T*)y, ldy, (const T*)w1, (const T*)b1, (const T*)ls, x_out,
-                             (const T*)w2, (const T*)b2, (T*)z, ldz, H, eps, rms, err};
+                             (const T*)w2, (const T*)b2, (T*)z, ldz, H, eps, rms, alpha, groups, err};
     return launch_residual_norm(p, M, st);
   }
   typedef bf16 T;
   const ResNormParams<T> p{x, ldx, rows, in_rows, (const T*)y, ldy, (const T*)w1, (const T*)b1, (const T*)ls, x_out,
-                           (const T*)w2, (const T*)b2, (T*)z, ldz, H, eps, rms, err};
+                           (const T*)w2, (const T*)b2, (T*)z, ldz, H, eps, rms, alpha, groups, err};
   return launch_residual_norm(p, M, st);
 }
 
@@ -425,6 +506,17 @@ extern "C" int ksana_glu_clamp(const void* in, void* out, int M, int I, int in_l
     e = launch_pdl(glu_clamp_kernel<bf16>, dim3((unsigned)g), dim3(256), 0, st, (const bf16*)in, (bf16*)out, M, I, in_ld, limit,
                    alpha, offset);
   return e == cudaSuccess ? 0 : -4;
+}
+
+extern "C" int ksana_xielu(const void* in, int ldi, void* out, int ldo, int M, int I, float pos, float neg, float lin, int f32,
+                           cudaStream_t st) {
+  return launch_rowwise(in, ldi, nullptr, 0, out, ldo, M, I, XieluOp{pos, neg, lin}, f32, st);
+}
+
+// out = a * sigmoid(gate); out may be a itself
+extern "C" int ksana_sigmoid_gate(const void* a, int lda, const void* gate, int ldg, void* out, int ldo, int M, int I, int f32,
+                                  cudaStream_t st) {
+  return launch_rowwise(a, lda, gate, ldg, out, ldo, M, I, SigmoidGateOp{}, f32, st);
 }
 
 extern "C" int ksana_qkv_rope_append(void* qkv, const int* positions, const int* slots, const float* cos_sin, int max_pos,

@@ -89,6 +89,28 @@ def alibi_slopes(num_heads: int) -> torch.Tensor:
     return torch.tensor(s, dtype=torch.float32)
 
 
+class RecordLayout:
+    """Layout of a cache block as one record of panels of any shapes: ``add`` appends a panel, ``view`` gives it for every
+    block. Panels start on 16-byte boundaries; a panel may have another element type than the cache tensor."""
+
+    def __init__(self, dtype: torch.dtype):
+        self.dtype, self.record, self.entries = dtype, 0, []
+
+    def add(self, shape, dtype: Optional[torch.dtype] = None) -> int:
+        dt, unit = dtype or self.dtype, self.dtype.itemsize
+        n = math.prod(shape) * dt.itemsize
+        self.entries.append((self.record, n // unit, tuple(shape), dt))
+        if n % unit:
+            raise ValueError(f"a panel of {n} bytes in a cache of {unit}-byte elements")
+        self.record += (n + 15) // 16 * 16 // unit
+        return len(self.entries) - 1
+
+    def view(self, cache: torch.Tensor, i: int) -> torch.Tensor:
+        """[blocks, *shape] view of panel ``i`` of a cache tensor [blocks, record]."""
+        at, n, shape, dt = self.entries[i]
+        return cache[:, at:at + n].view(dt).unflatten(1, shape)
+
+
 class PanelLayout:
     """Layout of a cache block whose layers differ in head counts or head sizes: one record per block that holds the K
     panel [kv heads, block tokens, key size] and the V panel [kv heads, block tokens, value size] of every cache layer,
@@ -111,6 +133,11 @@ class PanelLayout:
 
 class CommonModel:
     needs_prev_ids = False               # the step carries the token before each row's (StepInput.prev_ids)
+    # A cache block holds recurrent state as of its last computed token: a sequence can only go on from the end of what
+    # its last block has seen (whole cached blocks, or its own partly filled one), and a block's content is tied to its
+    # position
+    carries_state = False
+    moves_blocks = True                  # copies of a block may be used at another position (flexible cache)
 
     def __init__(self, cfg: ModelConfig, tp_rank: int = 0, tp_size: int = 1, comm=None, device="cpu",
                  dtype=torch.bfloat16, layer_range: Optional[tuple] = None, kv_cache_dtype=None,

@@ -11,7 +11,7 @@ Absorbed attention (per head h):   q_lat[h] = q_nope[h] @ W_uk[h]            (12
                                    o_lat[h] = softmax(s) @ c_kv                (512)
                                    o[h] = o_lat[h] @ W_uv[h]^T                 (512 -> 128)
 so attention is multi-query over a single 576/512-wide latent "head" shared by all query heads.
-The projections run on the tcgen05 GEMMs. On a GPU with the DeepSeek-V2/V3 dimensions (latent 512, rotary 64)
+The projections run on the tcgen05 GEMMs. On a GPU (latent up to 512, 576 with the rotary part, multiples of 8)
 the attention core is the tcgen05 latent-attention kernel (csrc/kernels/mla_attention.cu); other dimensions
 and the CPU use batched PyTorch matmuls over the gathered latent rows of each sequence.
 """
@@ -115,8 +115,8 @@ class DeepseekModel(CommonModel):
 
     # ------------------------------------------------------------------ tcgen05 latent attention (GPU)
     def _mla_native_ok(self, q) -> bool:
-        Hq = self.Hq
-        return (self.lora == 512 and self.rope == 64 and q.dtype == torch.bfloat16 and Hq <= 128 and Hq & (Hq - 1) == 0
+        return (self.lora <= 512 and self.lora + self.rope <= 576 and all(n % 8 == 0 for n in (self.lora, self.rope, self.nope, self.vdim))
+                and q.dtype == torch.bfloat16 and self.block_tokens in (8, 16, 32, 64, 128, 256)
                 and self.kv_cache is not None and self.kv_cache.dtype == torch.bfloat16)
 
     def _attention_native(self, li, mw, q, kv, step):
@@ -127,7 +127,7 @@ class DeepseekModel(CommonModel):
         cache = self.kv_cache[:, li - self.layer_lo]                # [blocks, bt, 576]
         qfull = torch.empty(T, Hq, self.lora + self.rope, dtype=q.dtype, device=q.device)
         native.mla_rope_append(q, self.nope, kv, mw.kv_a_norm, self.cfg.rms_norm_eps, step.positions, step.slots,
-                               self.cos_sin, qfull, cache, cache.stride(0), self.block_tokens, Hq)
+                               self.cos_sin, qfull, cache, self.block_tokens, Hq, self.lora)
         # absorbed query: per head q_nope W_uk straight into the packed query rows (one batched tcgen05 GEMM whose
         # operand and result views are head-interleaved: no transposes, no copy)
         q_nope = q.view(T, Hq, self.nope + self.rope)[..., : self.nope].transpose(0, 1)          # [Hq, T, nope]
@@ -137,8 +137,8 @@ class DeepseekModel(CommonModel):
         o_lat = torch.empty(T, Hq, self.lora, dtype=q.dtype, device=q.device)
         B = step.num_multi + step.num_single
         nsplit = native.mla_splits(B, step.max_q_len, step.max_kv_len) if step.num_multi == 0 else 1
-        if not native.mla_attention(qfull, o_lat, cache, cache.stride(0), self.block_tokens, step.block_table, step.cu_q,
-                                    step.kv_lens, B, max(step.max_q_len, 1), Hq, self.scale, nsplit):
+        if not native.mla_attention(qfull, o_lat, cache, self.block_tokens, step.block_table, step.cu_q, step.kv_lens, B,
+                                    max(step.max_q_len, 1), self.scale, nsplit):
             raise RuntimeError("latent-attention kernel rejected a configuration that _mla_native_ok accepted")
         o = torch.empty(T, Hq, self.vdim, dtype=q.dtype, device=q.device)
         native.gemm_bf16_batched(o_lat.transpose(0, 1), mw.w_uv, o.transpose(0, 1))              # per head o_lat W_uv^T

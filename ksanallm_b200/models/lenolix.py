@@ -9,10 +9,9 @@ describes the layers in terms of the shared ops. Per sublayer:
   norm (fused into the previous sublayer's add) -> QKV GEMM -> rotation + paged append -> attention -> output GEMM
   -> [norm, layer scale, residual add, next norm] in one kernel -> gate|up GEMM -> clamped unit -> down GEMM -> same kernel
 
-Sizes that are not multiples of 8 are padded with zeros when the weights are loaded (rows of the residual stream, head
-sizes, feed-forward widths, vocabulary), so the kernels always see 16-byte vectors; norms count the real columns only.
-Tensor parallelism: query and key/value heads, feed-forward columns and the vocabulary are split; the partial sums of
-the output and down projections are added across ranks before the norm that follows them.
+The residual stream, the padding of odd sizes and the loading helpers are those of models/stream.py. Tensor parallelism:
+query and key/value heads, feed-forward columns and the vocabulary are split; the partial sums of the output and down
+projections are added across ranks before the norm that follows them.
 """
 from __future__ import annotations
 
@@ -20,21 +19,16 @@ from dataclasses import dataclass
 from typing import List, Optional
 
 import torch
-import torch.nn.functional as F
 
 from ..config import AttentionSpec, LayerSpec, ModelConfig
 from ..ops import dispatch as ops
 from ..ops import native
-from ..ops import reference as ref
 from ..ops.dispatch import LinearWeight, NormParams
 from ..utils import nvtx
-from .common import CommonModel, PanelLayout, StepInput
+from .common import PanelLayout, StepInput
+from .stream import StreamLoader, StreamModel, pad8, pad_to
 
 MAX_HEAD = 256                    # largest head size of the attention kernels
-
-
-def pad8(n: int) -> int:
-    return (n + 7) // 8 * 8
 
 
 @dataclass
@@ -75,31 +69,19 @@ def layer_runs(cfg: ModelConfig) -> List[LayerRun]:
     return [LayerRun(i, c, enter) for c, (i, enter) in enumerate(order)]
 
 
-class LenolixModel(CommonModel):
-    def __init__(self, cfg: ModelConfig, tp_rank=0, tp_size=1, comm=None, device="cpu", dtype=torch.bfloat16, max_positions=None):
-        super().__init__(cfg, tp_rank, tp_size, comm, device, dtype)
-        self.width = pad8(cfg.hidden_size)
+class LenolixModel(StreamModel):
+    def __init__(self, cfg: ModelConfig, *a, **kw):
+        super().__init__(cfg, *a, **kw)
         self.needs_prev_ids = cfg.pair_embedding is not None
         self.runs = layer_runs(cfg)
         self.pair: Optional[torch.Tensor] = None
-        self.final: Optional[NormParams] = None
         self.loop_in: List[LinearWeight] = []            # one per pass: shared weight, the pass's step vector as bias
-        n = max_positions or min(cfg.max_token_len, 1 << 15)
-        self.rotary = {}                                 # layer -> cos|sin table, shared by layers with equal rotations
-        tables = {}
-        for i, s in enumerate(cfg.layer_specs):
-            r = s.mixer.rotary
-            if r is not None:
-                key = (r.dims, r.base, tuple(sorted((r.scaling or {}).items())))
-                if key not in tables:
-                    tables[key] = ref.build_cos_sin_cache(r.dims, n, r.base, r.scaling, self.device)
-                self.rotary[i] = tables[key]
+        self.rotary = {i: self.rotation_table(s.mixer.rotary) for i, s in enumerate(cfg.layer_specs) if s.mixer.rotary is not None}
 
     # ------------------------------------------------------------------ KV cache
     def allocate_kv_cache(self, num_blocks: int, block_tokens: int, dtype=None):
         """[blocks, record]: the K and V panels of every layer run, one after the other (sizes differ by layer)."""
-        if dtype is not None and dtype != self.dtype:
-            raise ValueError(f"{self.cfg.model_type}: the KV cache has the activations' type ({self.dtype}), not {dtype}")
+        self.check_cache_dtype(dtype)
         self.block_tokens = block_tokens
         shapes = []
         for run in self.runs:
@@ -131,17 +113,8 @@ class LenolixModel(CommonModel):
 
     # ------------------------------------------------------------------ blocks
     def embed_tokens(self, step: StepInput, copy=None) -> torch.Tensor:
-        """The fp32 embedding output; ``copy`` receives it in the activations' type."""
         p = self.cfg.pair_embedding
-        refit = step.refit_positions is not None and step.refit_positions.numel() > 0
-        hashed = (p.buckets, p.mul_prev, p.mul_cur) if p is not None else (0, 0, 0)
-        x = ops.embed_pair(step.input_ids, step.prev_ids, self.embed, self.pair, self.cfg.emb_scale, *hashed,
-                           copy=None if refit else copy, vocab=self.cfg.vocab_size)
-        if refit:
-            ops.refit_stream_rows(x, step.refit_positions, step.refit_embeddings)
-            if copy is not None:
-                ops.stream_copy(x, copy)
-        return x
+        return super().embed_tokens(step, copy, self.pair, (p.buckets, p.mul_prev, p.mul_cur) if p is not None else (0, 0, 0))
 
     def attention(self, run: LayerRun, lw: SandwichLayer, xn: torch.Tensor, step: StepInput) -> torch.Tensor:
         m: AttentionSpec = lw.spec.mixer
@@ -156,11 +129,6 @@ class LenolixModel(CommonModel):
     def mlp(self, lw: SandwichLayer, xn: torch.Tensor) -> torch.Tensor:
         s = lw.spec.mlp
         return ops.glu_clamp(ops.linear(xn, lw.gate_up), s.limit, s.alpha, s.offset)
-
-    def project(self, a: torch.Tensor, w: LinearWeight) -> torch.Tensor:
-        """Row-parallel output projection: the sublayer's full result, before its norm."""
-        y = ops.linear(a, w)
-        return self.comm.all_reduce(y) if self.tp_size > 1 else y
 
     def forward_layers(self, step: StepInput, hidden_in: Optional[torch.Tensor] = None) -> torch.Tensor:
         T, W = step.input_ids.shape[0], self.width
@@ -193,33 +161,15 @@ class LenolixModel(CommonModel):
                 self.stream_hook(r, x)
         return x
 
-    stream_hook = None                                   # debugging: called with (run, stream) after every layer run
-
-    def forward(self, step: StepInput, hidden_in: Optional[torch.Tensor] = None):
-        return self.lm_head_forward(self.forward_layers(step), step)
-
-    def lm_head_forward(self, x: torch.Tensor, step: StepInput):
-        if step.want_hidden:
-            self.step_hidden, self.step_normed = x, ops.stream_norm(x, self.final, self.dtype)
-        return self.logits_or_candidates(ops.stream_norm(x, self.final, self.dtype, rows=step.logits_rows), step)
-
     def weight_bytes(self) -> int:
         extra = [t for t in (self.pair, self.loop_in[0].w if self.loop_in else None) if t is not None]
         return super().weight_bytes() + sum(t.numel() * t.element_size() for t in extra)
 
 
 # ------------------------------------------------------------------------------------- loading
-def _pad(t: torch.Tensor, *sizes: int) -> torch.Tensor:
-    """Zero-pads every dimension of ``t`` to ``sizes``."""
-    spec = []
-    for have, want in zip(reversed(t.shape), reversed(sizes)):
-        spec += [0, want - have]
-    return F.pad(t, spec) if any(spec) else t
-
-
 def build_lenolix(cfg: ModelConfig, source, tp_rank=0, tp_size=1, comm=None, device="cpu", dtype=torch.bfloat16, quant=None,
                   layer_range=None, max_positions=None) -> LenolixModel:
-    from .weights import RandomSource, _cols, _make_linear, _rows
+    from .weights import _rows
     if layer_range is not None and tuple(layer_range) != (0, cfg.num_layers - 1):
         raise ValueError("lenolix: repeated layers need the embedding output, pipeline stages are not supported")
     for s in cfg.layer_specs:
@@ -228,29 +178,18 @@ def build_lenolix(cfg: ModelConfig, source, tp_rank=0, tp_size=1, comm=None, dev
         if torch.device(device).type == "cuda" and max(s.mixer.dim, s.mixer.vdim) > MAX_HEAD:
             raise ValueError(f"lenolix: head sizes above {MAX_HEAD} are not supported")
     m = LenolixModel(cfg, tp_rank, tp_size, comm, device, dtype, max_positions)
+    ld = StreamLoader(m, source, quant)
+    get, param, linear, rows, cols = ld.get, ld.param, ld.linear, ld.rows, ld.cols
     W, WP = cfg.hidden_size, m.width
-
-    def get(name, shape, kind="normal"):
-        t = source.get(name, shape, device=device, kind=kind)
-        if tuple(t.shape) != tuple(shape):
-            raise ValueError(f"{name}: shape {tuple(t.shape)} in the checkpoint, {tuple(shape)} by the configuration")
-        return t
-
-    def param(t, *sizes):
-        return _pad(t, *sizes).to(device=device, dtype=dtype).contiguous()
 
     def norm(name):
         return NormParams(param(get(name, (W,), "ones"), WP), param(get(name + ".b", (W,), "zeros"), WP), W, cfg.rms_norm_eps)
 
-    def linear(t):
-        return _make_linear(t.contiguous(), None, device, dtype, quant)
-
-    table = get("embed", (cfg.vocab_size, W))
-    m.embed = param(table, pad8(cfg.vocab_size), WP)
+    ld.vocabulary()
     if cfg.pair_embedding is not None:
         m.pair = param(get("bigram", (cfg.pair_embedding.buckets + 1, W)), cfg.pair_embedding.buckets + 1, WP)
     if cfg.loop is not None:
-        w_in = param(_pad(get("loop.in", (W, 2 * W)).reshape(W, 2, W), WP, 2, WP).reshape(WP, 2 * WP))
+        w_in = param(pad_to(get("loop.in", (W, 2 * W)).reshape(W, 2, W), WP, 2, WP).reshape(WP, 2 * WP))
         steps = param(get("loop.step", (cfg.loop.times, W)), cfg.loop.times, WP)
         m.loop_in = [LinearWeight(w=w_in, bias=steps[t]) for t in range(cfg.loop.times)]
     for i, spec in enumerate(cfg.layer_specs):
@@ -258,10 +197,10 @@ def build_lenolix(cfg: ModelConfig, source, tp_rank=0, tp_size=1, comm=None, dev
         D, DV = pad8(a.dim), pad8(a.vdim)
         rep = max(1, tp_size // a.kv_heads)              # ranks sharing one key/value head
         kv_rank, kv_size = tp_rank // rep, tp_size // rep
-        q = _rows(_pad(get(p + "mix.q", (a.heads * a.dim, W)).reshape(a.heads, a.dim, W), a.heads, D, WP), tp_rank, tp_size)
-        k = _rows(_pad(get(p + "mix.k", (a.kv_heads * a.dim, W)).reshape(a.kv_heads, a.dim, W), a.kv_heads, D, WP), kv_rank, kv_size)
-        v = _rows(_pad(get(p + "mix.v", (a.kv_heads * a.vdim, W)).reshape(a.kv_heads, a.vdim, W), a.kv_heads, DV, WP), kv_rank, kv_size)
-        o = _cols(_pad(get(p + "mix.o", (W, a.heads * a.vdim)).reshape(W, a.heads, a.vdim), WP, a.heads, DV), tp_rank, tp_size)
+        q = rows(pad_to(get(p + "mix.q", (a.heads * a.dim, W)).reshape(a.heads, a.dim, W), a.heads, D, WP))
+        k = _rows(pad_to(get(p + "mix.k", (a.kv_heads * a.dim, W)).reshape(a.kv_heads, a.dim, W), a.kv_heads, D, WP), kv_rank, kv_size)
+        v = _rows(pad_to(get(p + "mix.v", (a.kv_heads * a.vdim, W)).reshape(a.kv_heads, a.vdim, W), a.kv_heads, DV, WP), kv_rank, kv_size)
+        o = cols(pad_to(get(p + "mix.o", (W, a.heads * a.vdim)).reshape(W, a.heads, a.vdim), WP, a.heads, DV))
         sinks = get(p + "mix.sink", (a.heads,))[tp_rank * q.shape[0]:(tp_rank + 1) * q.shape[0]] if a.sink else None
         lw = SandwichLayer(spec, q.shape[0], k.shape[0], norm(p + "norm1"), norm(p + "norm1b"),
                            linear(torch.cat([t.reshape(-1, WP) for t in (q, k, v)], 0)), linear(o.reshape(WP, -1)),
@@ -269,15 +208,11 @@ def build_lenolix(cfg: ModelConfig, source, tp_rank=0, tp_size=1, comm=None, dev
                            param(get(p + "ls1", (W,), "ones"), WP))
         if spec.mlp is not None:
             ff = spec.mlp.size
-            n = pad8((ff + tp_size - 1) // tp_size)      # columns of a rank
-            gate, up = (_rows(_pad(get(p + "mlp." + s, (ff, W)), n * tp_size, WP), tp_rank, tp_size) for s in ("gate", "up"))
-            down = _cols(_pad(get(p + "mlp.down", (W, ff)), WP, n * tp_size), tp_rank, tp_size)
+            n = ld.shard(ff)                             # columns of a rank
+            gate, up = (rows(pad_to(get(p + "mlp." + s, (ff, W)), n * tp_size, WP)) for s in ("gate", "up"))
+            down = cols(pad_to(get(p + "mlp.down", (W, ff)), WP, n * tp_size))
             lw.norm2, lw.norm2b, lw.ls2 = norm(p + "norm2"), norm(p + "norm2b"), param(get(p + "ls2", (W,), "ones"), WP)
             lw.gate_up, lw.down = linear(torch.cat([gate, up], 0)), linear(down)
         m.layers.append(lw)
     m.final = norm("final.norm")
-    vs = (cfg.vocab_size + tp_size - 1) // tp_size
-    shard = m.embed if tp_size == 1 else param(_rows(m.embed[:cfg.vocab_size], tp_rank, tp_size), pad8(vs), WP)
-    m.lm_head = LinearWeight(w=shard)                    # the table itself, without the embedding's scale
-    m.vocab_shard = vs
     return m

@@ -335,7 +335,9 @@ def build_model(cfg: ModelConfig, source, tp_rank: int = 0, tp_size: int = 1, co
     embeddings, router and lm_head stay in ``dtype``)."""
     if cfg.layer_specs is not None:
         from .lenolix import build_lenolix
-        return build_lenolix(cfg, source, tp_rank, tp_size, comm, device, dtype, quant, layer_range, max_positions)
+        from .rasizen import build_rasizen
+        build = {"lenolix": build_lenolix, "rasizen": build_rasizen}[cfg.model_type]
+        return build(cfg, source, tp_rank, tp_size, comm, device, dtype, quant, layer_range, max_positions)
     if cfg.is_mla:
         from .deepseek import build_deepseek
         return build_deepseek(cfg, source, tp_rank, tp_size, comm, device, dtype, quant, layer_range, max_positions)

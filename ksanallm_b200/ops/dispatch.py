@@ -244,12 +244,14 @@ def rope_kv_append(qkv, positions, slots, cos_sin, cache_layer, block_tokens, Hq
 # ------------------------------------------------------------------------------- 32-bit residual stream
 @dataclass
 class NormParams:
-    """Weight and optional bias of a norm over ``size`` real columns (stored padded with zeros to a multiple of 8)."""
+    """Weight and optional bias of a norm over ``size`` real columns (stored padded with zeros to a multiple of 8).
+    ``groups`` > 1: root-mean-square norm of each of that many equal consecutive parts."""
     w: torch.Tensor
     b: Optional[torch.Tensor]
     size: int
     eps: float
     rms: bool = False
+    groups: int = 1
 
 
 def embed_pair(ids, prev, table, pair, scale, buckets=0, mul_prev=0, mul_cur=0, copy=None, vocab=None):
@@ -267,7 +269,8 @@ def stream_norm(x, norm: NormParams, dtype, rows=None):
     """norm of the fp32 residual stream (of its ``rows``) as the next linear's operand."""
     if x.is_cuda:
         z = torch.empty(rows.numel() if rows is not None else x.shape[0], x.shape[1], dtype=dtype, device=x.device)
-        native.residual_norm(x, norm.size, norm.eps, w2=norm.w, b2=norm.b, z=z, rows=rows, rms=norm.rms)
+        native.residual_norm(x, norm.size, norm.eps, w2=norm.w, b2=norm.b, z=z, rows=rows, rms=norm.rms,
+                             groups=norm.groups)
         return z
     return ref.stream_norm(x[rows.long()] if rows is not None else x, norm).to(dtype)
 
@@ -280,8 +283,8 @@ def stream_copy(x, out):
         out.copy_(x)
 
 
-def stream_add(x, y, post: Optional[NormParams], scale, then: Optional[NormParams] = None, copy=None, inplace=True):
-    """x + scale * norm(y; post) on the fp32 residual stream, fused with what reads the sum next: ``then`` (the following
+def stream_add(x, y, post: Optional[NormParams], scale, then: Optional[NormParams] = None, copy=None, inplace=True, alpha=1.0):
+    """x + alpha * scale * norm(y; post) (``scale``: per column, ``alpha``: one number) on the fp32 residual stream, fused with what reads the sum next: ``then`` (the following
     norm, returned in y's type) or ``copy`` (a buffer that receives the sum in its own type). Returns (x, normed or None);
     ``inplace`` updates x."""
     if x.is_cuda:
@@ -290,11 +293,14 @@ def stream_add(x, y, post: Optional[NormParams], scale, then: Optional[NormParam
         size, eps, rms = (post.size, post.eps, post.rms) if post is not None else (
             (then.size, then.eps, then.rms) if then is not None else (x.shape[1], 0.0, False))
         native.residual_norm(x, size, eps, y=y, w1=post.w if post else None, b1=post.b if post else None, ls=scale, x_out=out,
-                             w2=then.w if then else None, b2=then.b if then else None, z=z, rms=rms)
+                             w2=then.w if then else None, b2=then.b if then else None, z=z, rms=rms, alpha=alpha,
+                             groups=then.groups if then else 1)
         return out, (z if then is not None else None)
     a = ref.stream_norm(y, post) if post is not None else y.float()
     if scale is not None:
         a = a * scale.float()
+    if alpha != 1.0:
+        a = a * alpha
     out = x.add_(a) if inplace else x + a
     if copy is not None:
         copy.copy_(out)
@@ -306,6 +312,78 @@ def glu_clamp(x, limit, alpha=1.702, offset=1.0):
     if x.is_cuda:
         return native.glu_clamp(x, limit, alpha, offset)
     return ref.glu_clamp(x, limit, alpha, offset)
+
+
+def xielu(x, pos, neg, lin=0.5):
+    """pos x^2 + lin x above zero, neg (exp(x) - 1 - x) + lin x below."""
+    return native.xielu(x, pos, neg, lin) if x.is_cuda else ref.xielu(x, pos, neg, lin)
+
+
+def sigmoid_gate(a, gate):
+    """a * sigmoid(gate), in place on ``a``; ``gate`` may be a column range of wider rows."""
+    if a.is_cuda:
+        return native.sigmoid_gate(a, gate, out=a)
+    return a.copy_(ref.sigmoid_gate(a, gate))
+
+
+def gated_recurrence(y, W, state, block_tokens, step, offset=0.5):
+    """S_t = (1 - gate) S_(t-1) + gate * cand with gate = sigmoid(z) and cand = u + offset (u >= 0) or sigmoid(u), out =
+    S_t * silu(g), over a step's new rows; y [T, 3 W] holds z | u | g. ``state`` [blocks, W] (fp32, part of the cache's
+    block records): a block's row is the state after the last of its tokens computed so far."""
+    z, u, g = y[:, :W], y[:, W:2 * W], y[:, 2 * W:]
+    if not y.is_cuda:
+        return ref.gated_recurrence(z, u, g, state, block_tokens, step.block_table, step.cu_q, step.kv_lens, offset)
+    out = torch.empty(y.shape[0], W, dtype=y.dtype, device=y.device)
+    nm, ns, tm = step.num_multi, step.num_single, step.num_multi_tokens
+    if nm:
+        native.gated_recurrence(z, u, g, out, state, block_tokens, step.block_table, step.cu_q, step.kv_lens[:nm], offset)
+    if ns:
+        native.gated_recurrence(z[tm:], u[tm:], g[tm:], out[tm:], state, block_tokens, step.block_table[nm:], None,
+                                step.kv_lens[nm:], offset)
+    return out
+
+
+# ------------------------------------------------------------------------------- latent attention
+def bmm(a, w, out):
+    """out[b] = a[b] w[b]^T over (strided) views a [B, M, K], w [B, N, K], out [B, M, N]."""
+    if not a.is_cuda:
+        return out.copy_(torch.matmul(a.float(), w.float().transpose(1, 2)))
+    return (native.gemm_f32_batched if a.dtype == torch.float32 else native.gemm_bf16_batched)(a, w, out)
+
+
+def latent_append(q, nope, kv, norm: Optional[NormParams], step, cos_sin, cache, block_tokens):
+    """Packed query rows [T, G, DK] whose rotary columns (the last ones) are filled with the rotated queries' (q: [T, G, nope
+    + rotary], rows may be part of wider ones), and the append of the normed latents and the rotated key of ``kv`` [T, DK]
+    to the panel ``cache`` [blocks, block tokens, DK]. ``kv`` None: the latents are another layer's, nothing is appended."""
+    T, G = q.shape[:2]
+    qfull = torch.empty(T, G, cache.shape[2], dtype=q.dtype, device=q.device)
+    if q.is_cuda:
+        native.mla_rope_append(q, nope, kv, norm.w if kv is not None else None, norm.eps if kv is not None else 0.0, step.positions,
+                               step.slots, cos_sin, qfull, cache, block_tokens, G, norm.size if kv is not None else 1)
+    else:
+        ref.latent_append(q, nope, kv, norm.w if kv is not None else None, norm.eps if kv is not None else 0.0,
+                          norm.size if kv is not None else 1, step.positions, step.slots, cos_sin, qfull, cache, block_tokens)
+    return qfull
+
+
+def latent_attention(qfull, cache, dv, block_tokens, step, scale, window=0):
+    """Absorbed attention of packed query rows [T, G, DK] against the latent panel [blocks, block tokens, DK], values = the
+    first ``dv`` columns of its rows: [T, G, dv]. The tensor-core kernel serves bf16 rows up to 576 / 512 columns over
+    blocks of 8 to 256 (a power of two) tokens, the 32-bit one the rest."""
+    T, G, dk = qfull.shape
+    if not qfull.is_cuda:
+        return ref.mla_attention(qfull, cache, step.block_table, step.cu_q, step.kv_lens, scale, dv, window).to(qfull.dtype)
+    out = torch.empty(T, G, dv, dtype=qfull.dtype, device=qfull.device)
+    B, mq = step.num_multi + step.num_single, max(step.max_q_len, 1)
+    if qfull.dtype == torch.bfloat16:
+        seen = min(step.max_kv_len, window + 64) if window > 0 else step.max_kv_len
+        n = native.mla_splits(B, mq, seen, halves=(dv + 255) // 256) if step.num_multi == 0 else 1
+        if native.mla_attention(qfull, out, cache, block_tokens, step.block_table, step.cu_q, step.kv_lens, B, mq, scale, n, window):
+            return out
+    panel = cache.unsqueeze(1)                           # one key/value head shared by all query heads
+    native.attention_f32(qfull, G * dk, out.view(T, G * dv), panel, panel[..., :dv], block_tokens, step.block_table, step.cu_q,
+                         step.kv_lens, B, mq, G, 1, scale, window)
+    return out
 
 
 def qkv_rope_append(qkv, positions, slots, cos_sin, k_cache, v_cache, block_tokens, Hq, Hkv, rot_dim):

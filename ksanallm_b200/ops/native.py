@@ -66,8 +66,12 @@ _SIGS = {
     "ksana_absmax_scale": [vp, i32, i32, i64, f32, f32, vp, vp, vp],
     "ksana_rerotate_blocks": [vp, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, i64, vp, vp],
     "ksana_embed_pair": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i64, i64, i64, f32, i32, vp, vp],
-    "ksana_residual_norm": [vp, i32, vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, f32, i32, i32, vp, vp],
+    "ksana_residual_norm": [vp, i32, vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, f32, i32, i32, f32, i32, vp, vp],
     "ksana_glu_clamp": [vp, vp, i32, i32, i32, f32, f32, f32, i32, vp],
+    "ksana_xielu": [vp, i32, vp, i32, i32, i32, f32, f32, f32, i32, vp],
+    "ksana_sigmoid_gate": [vp, i32, vp, i32, vp, i32, i32, i32, i32, vp],
+    "ksana_gated_recurrence": [vp, vp, vp, i64, vp, i64, vp, i64, i32, i32, vp, i32, vp, vp, i32, i32, f32, i32, vp, vp],
+    "ksana_gemm_f32_batched": [vp, i32, i64, vp, i32, i64, vp, i32, i64, i32, i32, i32, i32, vp],
     "ksana_qkv_rope_append": [vp, vp, vp, vp, i32, vp, vp, i64, i32, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp],
     "ksana_refit_rows_f32": [vp, i32, vp, vp, i32, i32, i32, vp, vp],
     "ksana_gemm_f32": [vp, i32, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, vp],
@@ -80,8 +84,8 @@ _SIGS = {
                             f32, i32, f32, f32, i32, vp, vp],
     "ksana_paged_decode": [vp, i64, vp, i64, vp, vp, i64, i32, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, i32,
                            f32, f32, i32, vp, vp, i32, vp, vp, i32, vp, vp],
-    "ksana_mla_attention": [vp, i64, vp, i64, vp, i64, i32, vp, i32, vp, vp, i32, i32, i32, f32, i64, i32, vp, vp, vp, vp],
-    "ksana_mla_rope_append": [vp, i64, i32, vp, i64, vp, f32, vp, vp, vp, vp, vp, i64, i32, i32, i32, i32, i64, vp, vp],
+    "ksana_mla_attention": [vp, i64, vp, i64, vp, i64, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, f32, i32, i32, vp, vp, vp, vp],
+    "ksana_mla_rope_append": [vp, i64, i32, vp, i64, vp, f32, vp, vp, vp, vp, vp, i64, i32, i32, i32, i32, i32, i32, i64, i32, vp, vp],
     "ksana_gemm_smallm_w4": [vp, i32, vp, vp, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, vp, i64, vp, i32, vp, vp],
     "ksana_w4_gemv": [vp, i64, vp, vp, vp, vp, vp, i64, vp, i64, i32, i32, i32, i32, vp],
     "ksana_w4_dequant": [vp, vp, vp, vp, i64, i32, i32, i32, vp],
@@ -683,16 +687,18 @@ def embed_pair(ids, prev, table, pair, scale, buckets=0, mul_prev=0, mul_cur=0, 
     return x
 
 
-def residual_norm(x, H, eps, y=None, w1=None, b1=None, ls=None, x_out=None, w2=None, b2=None, z=None, rows=None, rms=False):
+def residual_norm(x, H, eps, y=None, w1=None, b1=None, ls=None, x_out=None, w2=None, b2=None, z=None, rows=None, rms=False,
+                  alpha=1.0, groups=1):
     """One pass over rows of the fp32 stream ``x`` (``H`` real columns, padded to a multiple of 8):
-    x' = x + ls * norm(y; w1, b1), stored to ``x_out``; z = norm(x'; w2, b2), or a copy of x' without ``w2``. Parts whose
-    arguments are None are left out; ``rows`` gathers stream rows."""
+    x' = x + alpha * ls * norm(y; w1, b1), stored to ``x_out``; z = norm(x'; w2, b2), or a copy of x' without ``w2``. Parts
+    whose arguments are None are left out; ``rows`` gathers stream rows. ``groups`` > 1: the stream's norm (RMS, without
+    ``w1``) is taken for each of that many equal parts of a row."""
     M = rows.numel() if rows is not None else x.shape[0]
     t = z if z is not None else y
     _check(lib().ksana_residual_norm(_p(x), x.stride(0), _p(rows), x.shape[0], _p(y), y.stride(0) if y is not None else 0, _p(w1),
                                      _p(b1), _p(ls), _p(x_out), _p(w2), _p(b2), _p(z), z.stride(0) if z is not None else 0, M, H,
-                                     float(eps), int(rms), int(t.dtype == torch.float32), _p(err_flag(x.device)), _st()),
-           "ksana_residual_norm")
+                                     float(eps), int(rms), int(t.dtype == torch.float32), float(alpha), int(groups),
+                                     _p(err_flag(x.device)), _st()), "ksana_residual_norm")
 
 
 def glu_clamp(x, limit, alpha, offset):
@@ -700,6 +706,48 @@ def glu_clamp(x, limit, alpha, offset):
     out = torch.empty(M, I, dtype=x.dtype, device=x.device)
     _check(lib().ksana_glu_clamp(_p(x), _p(out), M, I, x.stride(0), float(limit), float(alpha), float(offset),
                                  int(x.dtype == torch.float32), _st()), "ksana_glu_clamp")
+    return out
+
+
+def xielu(x, pos, neg, lin, out=None):
+    M, I = x.shape
+    if out is None:
+        out = torch.empty(M, I, dtype=x.dtype, device=x.device)
+    _check(lib().ksana_xielu(_p(x), x.stride(0), _p(out), out.stride(0), M, I, float(pos), float(neg), float(lin),
+                             int(x.dtype == torch.float32), _st()), "ksana_xielu")
+    return out
+
+
+def sigmoid_gate(a, gate, out=None):
+    """a * sigmoid(gate) row by row; ``gate`` may be a column range of wider rows, ``out`` may be ``a``."""
+    M, I = a.shape
+    if out is None:
+        out = torch.empty(M, I, dtype=a.dtype, device=a.device)
+    assert gate.shape == a.shape and gate.dtype == a.dtype and gate.stride(1) == a.stride(1) == 1
+    _check(lib().ksana_sigmoid_gate(_p(a), a.stride(0), _p(gate), gate.stride(0), _p(out), out.stride(0), M, I,
+                                    int(a.dtype == torch.float32), _st()), "ksana_sigmoid_gate")
+    return out
+
+
+def gated_recurrence(z, u, g, out, state, block_tokens, block_table, cu_q, kv_lens, offset):
+    """Recurrence over the new tokens of ``kv_lens.numel()`` sequences; z, u, g: column ranges [T, W] of one projection's
+    rows, ``state``: [blocks, W] fp32 rows inside the cache's block records. ``cu_q`` None: one row per sequence."""
+    assert z.stride() == u.stride() == g.stride() and z.dtype == u.dtype == g.dtype == out.dtype and z.stride(1) == 1
+    assert state.dtype == torch.float32 and state.stride(1) == 1
+    _check(lib().ksana_gated_recurrence(_p(z), _p(u), _p(g), z.stride(0), _p(out), out.stride(0), _p(state), state.stride(0),
+                                        block_tokens, state.shape[0], _p(block_table), block_table.stride(0), _p(cu_q), _p(kv_lens),
+                                        kv_lens.numel(), z.shape[1], float(offset), int(z.dtype == torch.float32),
+                                        _p(err_flag(z.device)), _st()), "ksana_gated_recurrence")
+
+
+def gemm_f32_batched(a, w, out):
+    """:func:`gemm_bf16_batched` in fp32 on the CUDA cores."""
+    B, M, K = a.shape
+    N = w.shape[1]
+    assert w.shape[0] == B and w.shape[2] == K and tuple(out.shape) == (B, M, N)
+    assert a.stride(2) == 1 and w.stride(2) == 1 and out.stride(2) == 1
+    _check(lib().ksana_gemm_f32_batched(_p(a), a.stride(1), a.stride(0), _p(w), w.stride(1), w.stride(0), _p(out), out.stride(1),
+                                        out.stride(0), B, M, N, K, _st()), "ksana_gemm_f32_batched")
     return out
 
 
@@ -722,14 +770,6 @@ def rope_kv_append(qkv, positions, slots, cos_sin, cache_layer, block_stride, bl
                                     block_stride, block_tokens, T, Hq, Hkv, D, rot_dim, int(neox), s0, s1, int(fp8),
                                     float(k_scale), float(v_scale), int(apply_rope), _st())
     _check(rc, "ksana_rope_kv_append")
-
-
-def _cache_rows(cache_layer, block_stride, D):
-    """Rows of D elements addressable from the layer's base pointer (bounds of the TMA tensor map)."""
-    return int(cache_layer.shape[0]) * int(block_stride) // int(D)
-
-
-PREFILL_TC = True                  # prefill attention on tcgen05 where the kernel covers the configuration
 
 
 def _panels(cache_layer, v_cache, D):
@@ -782,11 +822,12 @@ def paged_decode(q, q_stride, out, cache_layer, block_stride, block_tokens, bloc
 
 def attention_f32(q, q_stride, out, k_cache, v_cache, block_tokens, block_table, cu_q, kv_lens, B, max_q_len, Hq, Hkv, scale,
                   window=0, keep=0, sinks=None):
-    """All of a step's new rows (any lengths) against fp32 K and V panels, in 32-bit arithmetic throughout."""
-    rc = lib().ksana_attention_f32(_p(q), q_stride, _p(out), out.stride(0), _p(k_cache), _p(v_cache), k_cache.stride(0),
-                                   block_tokens, k_cache.shape[0], _p(block_table), block_table.stride(0), _p(cu_q),
-                                   _p(kv_lens), _p(sinks), B, max_q_len, Hq, Hkv, k_cache.shape[-1], v_cache.shape[-1], window,
-                                   keep, float(scale), _p(err_flag(q.device)), _st())
+    """All of a step's new rows (any lengths) against K and V panels, in 32-bit arithmetic throughout (bf16 storage is fine).
+    ``v_cache`` may be a column range of ``k_cache``."""
+    rc = lib().ksana_attention_f32(_p(q), q_stride, _p(out), out.stride(0), _p(k_cache), _p(v_cache), v_cache.stride(-2),
+                                   k_cache.stride(0), block_tokens, k_cache.shape[0], _p(block_table), block_table.stride(0),
+                                   _p(cu_q), _p(kv_lens), _p(sinks), B, max_q_len, Hq, Hkv, k_cache.shape[-1], v_cache.shape[-1],
+                                   window, keep, float(scale), int(q.dtype == torch.float32), _p(err_flag(q.device)), _st())
     _check(rc, "ksana_attention_f32")
 
 
@@ -801,18 +842,19 @@ def qkv_rope_append(qkv, positions, slots, cos_sin, k_cache, v_cache, block_toke
     _check(rc, "ksana_qkv_rope_append")
 
 
-def mla_rope_append(q, nope, kv, norm_w, eps, positions, slots, cos_sin, qfull, cache_layer, block_stride, block_tokens, G):
-    """Latent RMSNorm + rotary key rotation + append to the paged latent cache, and q_pe rotation into ``qfull``
-    ([T, G, 576]; its first 512 columns are filled by the caller). q: [T, G*(nope+64)], kv: [T, 576]."""
+def mla_rope_append(q, nope, kv, norm_w, eps, positions, slots, cos_sin, qfull, cache, block_tokens, G, rank):
+    """Latent RMS norm + rotary key rotation + append to the paged latent panel ``cache`` [blocks, block tokens, DK], and
+    rotation of the queries' rotary parts into ``qfull`` [T, G, DK] (its leading columns are filled by the caller). q: [T,
+    G * (nope + rotary)], kv: [T, DK] or None (queries only: the latents are another layer's). ``rank``: real latent
+    size; latent and rotary columns are padded to multiples of 8 with zeros."""
     T = q.shape[0]
-    rc = lib().ksana_mla_rope_append(_p(q), q.stride(0), nope, _p(kv), kv.stride(0), _p(norm_w), float(eps), _p(positions),
-                                     _p(slots), _p(cos_sin), _p(qfull), _p(cache_layer), block_stride, block_tokens, T, G,
-                                     int(cos_sin.shape[0]), int(cache_layer.shape[0]) * block_tokens,
-                                     _p(err_flag(q.device)), _st())
-    _check(rc, "ksana_mla_rope_append")
+    _check(lib().ksana_mla_rope_append(
+        _p(q), q.stride(0), nope, _p(kv), kv.stride(0) if kv is not None else 0, _p(norm_w), float(eps), _p(positions), _p(slots),
+        _p(cos_sin), _p(qfull), _p(cache), cache.stride(0), block_tokens, T, G, rank, int(cos_sin.shape[1]), int(cos_sin.shape[0]),
+        int(cache.shape[0]) * block_tokens, int(q.dtype == torch.float32), _p(err_flag(q.device)), _st()), "ksana_mla_rope_append")
 
 
-def mla_splits(num_seqs: int, max_q_len: int, max_kv: int, sms: int = 148) -> int:
+def mla_splits(num_seqs: int, max_q_len: int, max_kv: int, sms: int = 148, halves: int = 2) -> int:
     """KV splits for the latent-attention kernel: only pure decode steps split; the count minimises the number of
     CTA waves times the tiles per CTA, and a split never holds fewer than 4 tiles of 64 tokens."""
     if max_q_len != 1 or num_seqs <= 0:
@@ -821,26 +863,27 @@ def mla_splits(num_seqs: int, max_q_len: int, max_kv: int, sms: int = 148) -> in
     most = max(1, min(32, tiles // 4))
     best, best_cost = 1, None
     for n in range(1, most + 1):
-        waves = (2 * num_seqs * n + sms - 1) // sms            # one CTA per SM, two output halves per sequence
+        waves = (halves * num_seqs * n + sms - 1) // sms       # one CTA per SM and output half of a sequence
         cost = waves * ((tiles + n - 1) // n + 2)              # tile times of the longest CTA chain (+ set-up)
         if best_cost is None or cost < best_cost:
             best, best_cost = n, cost
     return best
 
 
-def mla_attention(qfull, out, cache_layer, block_stride, block_tokens, block_table, cu_q, kv_lens, B, max_q_len, G, scale,
-                  nsplit=1) -> bool:
-    """Absorbed multi-head latent attention on tcgen05 (see csrc/kernels/mla_attention.cu). qfull [T, G, 576],
-    out [T, G, 512]. Returns False when the kernel does not cover the configuration."""
-    T = qfull.shape[0]
+def mla_attention(qfull, out, cache, block_tokens, block_table, cu_q, kv_lens, B, max_q_len, scale, nsplit=1, window=0) -> bool:
+    """Absorbed multi-head latent attention on tcgen05 (see csrc/kernels/mla_attention.cu). qfull [T, G, DK], cache: latent
+    panel [blocks, block tokens, DK], out [T, G, DV] (values are the leading DV columns of the cache rows). Returns False
+    when the kernel does not cover the configuration."""
+    T, G, dk = qfull.shape
+    dv = out.shape[2]
+    assert qfull.is_contiguous() and out.stride(2) == 1 and out.stride(1) == dv and cache.stride(1) == dk == cache.shape[2]
     po = pml = None
     if nsplit > 1:
-        po = torch.empty(nsplit * T * G * 512, dtype=torch.float32, device=qfull.device)
+        po = torch.empty(nsplit * T * G * dv, dtype=torch.float32, device=qfull.device)
         pml = torch.empty(nsplit * T * G * 2, dtype=torch.float32, device=qfull.device)
-    rc = lib().ksana_mla_attention(_p(qfull), T, _p(out), out.stride(0), _p(cache_layer), block_stride, block_tokens,
-                                   _p(block_table), block_table.stride(0), _p(cu_q), _p(kv_lens), B, max_q_len, G,
-                                   float(scale), _cache_rows(cache_layer, block_stride, 576), nsplit, _p(po), _p(pml),
-                                   _p(err_flag(qfull.device)), _st())
+    rc = lib().ksana_mla_attention(_p(qfull), T, _p(out), out.stride(0), _p(cache), cache.stride(0), block_tokens, _p(block_table),
+                                   block_table.stride(0), _p(cu_q), _p(kv_lens), B, max_q_len, G, dk, dv, window, float(scale),
+                                   int(cache.shape[0]), nsplit, _p(po), _p(pml), _p(err_flag(qfull.device)), _st())
     if rc == -100:
         return False
     _check(rc, "ksana_mla_attention")

@@ -272,10 +272,12 @@ def embed_pair(ids, prev, table, pair, scale, buckets=0, mul_prev=0, mul_cur=0):
 
 
 def stream_norm(x, norm):
-    """fp32 norm over the first ``norm.size`` columns; pad columns come out as zeros."""
+    """fp32 norm over the first ``norm.size`` columns (of each of ``norm.groups`` equal parts of them); pad columns come
+    out as zeros."""
     h = x[:, :norm.size].float()
     if norm.rms:
-        y = h * torch.rsqrt(h.pow(2).mean(-1, keepdim=True) + norm.eps)
+        p = h.unflatten(-1, (norm.groups, -1))
+        y = (p * torch.rsqrt(p.pow(2).mean(-1, keepdim=True) + norm.eps)).flatten(-2)
     else:
         d = h - h.mean(-1, keepdim=True)
         y = d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + norm.eps)
@@ -289,6 +291,52 @@ def glu_clamp(x, limit, alpha, offset):
     g, u = x.float().chunk(2, dim=-1)
     g, u = g.clamp(max=limit), u.clamp(-limit, limit)
     return (g * torch.sigmoid(alpha * g) * (u + offset)).to(x.dtype)
+
+
+def xielu(x, pos, neg, lin):
+    z = x.float()
+    low = z.clamp(max=0)
+    return (torch.where(z > 0, pos * z * z, neg * (torch.expm1(low) - low)) + lin * z).to(x.dtype)
+
+
+def sigmoid_gate(a, gate):
+    return (a.float() * torch.sigmoid(gate.float())).to(a.dtype)
+
+
+def gated_recurrence(z, u, g, state, block_tokens, block_table, cu_q, kv_lens, offset):
+    """See dispatch.gated_recurrence; ``state`` [blocks, W] is updated in place."""
+    out = torch.zeros(z.shape, dtype=z.dtype, device=z.device)
+    for s in range(kv_lens.numel()):
+        q0, q1 = int(cu_q[s]), int(cu_q[s + 1])
+        pos = int(kv_lens[s]) - (q1 - q0)
+        if q1 == q0 or pos < 0:
+            continue
+        S = state[int(block_table[s, (pos - 1) // block_tokens])].clone() if pos > 0 else torch.zeros_like(state[0])
+        gate = torch.sigmoid(z[q0:q1].float())
+        uf = u[q0:q1].float()
+        inc = gate * torch.where(uf >= 0, uf + offset, torch.sigmoid(uf))
+        for i in range(q1 - q0):
+            S = (1 - gate[i]) * S + inc[i]
+            out[q0 + i] = (S * F.silu(g[q0 + i].float())).to(out.dtype)
+            if i == q1 - q0 - 1 or (pos + i + 1) % block_tokens == 0:
+                state[int(block_table[s, (pos + i) // block_tokens])] = S
+    return out
+
+
+def latent_append(q, nope, kv, norm_w, eps, rank, positions, slots, cos_sin, qfull, cache, block_tokens):
+    """q [T, G, nope + rotary] -> rotary columns of qfull [T, G, DK]; normed latents | rotated key of kv [T, DK] into the
+    panel [blocks, block tokens, DK]."""
+    R, rot = q.shape[2] - nope, cos_sin.shape[1]
+    rank_p = qfull.shape[2] - R
+    qfull[..., rank_p:] = apply_rope(q[..., nope:], positions, cos_sin, rot, neox=False).to(qfull.dtype)
+    if kv is None:
+        return
+    c = kv[:, :rank_p].float()
+    c = c * torch.rsqrt(c.pow(2).sum(-1, keepdim=True) / rank + eps) * norm_w.float()
+    r = apply_rope(kv[:, None, rank_p:], positions, cos_sin, rot, neox=False)[:, 0]
+    ok = slots >= 0
+    sl = slots[ok].long()
+    cache[sl // block_tokens, sl % block_tokens] = torch.cat([c.to(cache.dtype), r.to(cache.dtype)], -1)[ok]
 
 
 def qkv_rope_append(qkv, positions, slots, cos_sin, k_cache, v_cache, block_tokens, Hq, Hkv, rot_dim):
@@ -410,7 +458,7 @@ def gemm_nvfp4(aq, a_bs, a_ts, wq, w_bs, w_ts, bias=None, residual=None, out_dty
     return y.to(out_dtype)
 
 
-def mla_attention(qfull, cache_layer, block_table, cu_q, kv_lens, scale, lora=512):
+def mla_attention(qfull, cache_layer, block_table, cu_q, kv_lens, scale, lora=512, window=0):
     """Absorbed multi-head latent attention, plain fp32 statement. qfull [T, G, lora+rope] (q_lat | q_pe),
     cache_layer [blocks, block_tokens, lora+rope] (c_kv | k_pe). Returns [T, G, lora] fp32."""
     T, G, _ = qfull.shape
@@ -426,8 +474,8 @@ def mla_attention(qfull, cache_layer, block_table, cu_q, kv_lens, scale, lora=51
         sc = torch.einsum("qhd,kd->hqk", qfull[q0:q1].float(), rows) * scale
         qpos = torch.arange(kl - (q1 - q0), kl, device=qfull.device).unsqueeze(1)
         kpos = torch.arange(kl, device=qfull.device).unsqueeze(0)
-        sc = sc.masked_fill(kpos > qpos, float("-inf"))
-        out[q0:q1] = torch.einsum("hqk,kl->qhl", torch.softmax(sc, -1), rows[:, :lora])
+        hide = (kpos > qpos) | (qpos - kpos >= window) if window > 0 else kpos > qpos
+        out[q0:q1] = torch.einsum("hqk,kl->qhl", torch.softmax(sc.masked_fill(hide, float("-inf")), -1), rows[:, :lora])
     return out
 
 

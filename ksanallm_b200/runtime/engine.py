@@ -415,6 +415,9 @@ class LLMEngine:
             setattr(sc, k, getattr(bs, k))
         sc.max_token_len = min(bs.max_token_len, model_cfg.max_token_len) if model_cfg.max_token_len else bs.max_token_len
         sc.enable_prefix_cache = bool(bs.enable_auto_prefix_cache)
+        sc.resume_at_block_ends = bool(getattr(model, "carries_state", False))
+        if bs.min_flexible_cache_num > 0 and not getattr(model, "moves_blocks", True):
+            raise ValueError(f"{model_cfg.model_type}: cached blocks cannot be moved to another position (min_flexible_cache_num)")
         sc.block_token_num = cfg.block_manager.block_token_num
         sc.eos_token_ids = list(model_cfg.eos_token_ids)
         dp = getattr(model, "dp", None)

@@ -42,7 +42,7 @@ def test_mla_attention_matches_reference(G, bt, q_lens, kv_lens, nsplit):
     T = q.shape[0]
     out = torch.zeros(T, G, 512, dtype=torch.bfloat16, device=DEV)
     scale = 1.0 / math.sqrt(192)
-    ok = native.mla_attention(q, out, layer, layer.stride(0), bt, table, cu, kvl, len(q_lens), max(q_lens), G, scale, nsplit)
+    ok = native.mla_attention(q, out, layer, bt, table, cu, kvl, len(q_lens), max(q_lens), scale, nsplit)
     assert ok
     torch.cuda.synchronize()
     native.check_err_flag(q.device)
@@ -66,7 +66,7 @@ def test_mla_rope_append_matches_reference():
     cache = torch.zeros(10, 3, bt, 576, dtype=torch.bfloat16, device=DEV)
     layer = cache[:, 2]
     qfull = torch.zeros(T, G, 576, dtype=torch.bfloat16, device=DEV)
-    native.mla_rope_append(q, nope, kv, w, 1e-6, pos, slots, cos_sin, qfull, layer, layer.stride(0), bt, G)
+    native.mla_rope_append(q, nope, kv, w, 1e-6, pos, slots, cos_sin, qfull, layer, bt, G, 512)
     torch.cuda.synchronize()
     c = ref.norm(kv[:, :512].float(), w.float(), 1e-6)[0]
     kpe = ref.apply_rope(kv[:, 512:].float().reshape(T, 1, 64), pos, cos_sin, 64, neox=False).reshape(T, 64)
