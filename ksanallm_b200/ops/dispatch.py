@@ -357,12 +357,11 @@ def latent_append(q, nope, kv, norm: Optional[NormParams], step, cos_sin, cache,
     to the panel ``cache`` [blocks, block tokens, DK]. ``kv`` None: the latents are another layer's, nothing is appended."""
     T, G = q.shape[:2]
     qfull = torch.empty(T, G, cache.shape[2], dtype=q.dtype, device=q.device)
+    w, eps, rank = (norm.w, norm.eps, norm.size) if kv is not None else (None, 0.0, cache.shape[2] - (q.shape[2] - nope))
     if q.is_cuda:
-        native.mla_rope_append(q, nope, kv, norm.w if kv is not None else None, norm.eps if kv is not None else 0.0, step.positions,
-                               step.slots, cos_sin, qfull, cache, block_tokens, G, norm.size if kv is not None else 1)
+        native.mla_rope_append(q, nope, kv, w, eps, step.positions, step.slots, cos_sin, qfull, cache, block_tokens, G, rank)
     else:
-        ref.latent_append(q, nope, kv, norm.w if kv is not None else None, norm.eps if kv is not None else 0.0,
-                          norm.size if kv is not None else 1, step.positions, step.slots, cos_sin, qfull, cache, block_tokens)
+        ref.latent_append(q, nope, kv, w, eps, rank, step.positions, step.slots, cos_sin, qfull, cache, block_tokens)
     return qfull
 
 

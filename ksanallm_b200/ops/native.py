@@ -75,8 +75,8 @@ _SIGS = {
     "ksana_qkv_rope_append": [vp, vp, vp, vp, i32, vp, vp, i64, i32, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp],
     "ksana_refit_rows_f32": [vp, i32, vp, vp, i32, i32, i32, vp, vp],
     "ksana_gemm_f32": [vp, i32, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, vp],
-    "ksana_attention_f32": [vp, i64, vp, i64, vp, vp, i64, i32, i32, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32,
-                            f32, vp, vp],
+    "ksana_attention_f32": [vp, i64, vp, i64, vp, vp, i32, i64, i32, i32, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32,
+                            i32, f32, i32, vp, vp],
     "ksana_cast_f32": [vp, vp, i64, vp],
     "ksana_paged_prefill_tc": [vp, i64, i64, vp, i64, vp, vp, i64, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32,
                                i32, i32, f32, i32, vp, vp],
@@ -770,6 +770,9 @@ def rope_kv_append(qkv, positions, slots, cos_sin, cache_layer, block_stride, bl
                                     block_stride, block_tokens, T, Hq, Hkv, D, rot_dim, int(neox), s0, s1, int(fp8),
                                     float(k_scale), float(v_scale), int(apply_rope), _st())
     _check(rc, "ksana_rope_kv_append")
+
+
+PREFILL_TC = True                  # prefill attention on tcgen05 where the kernel covers the configuration
 
 
 def _panels(cache_layer, v_cache, D):
