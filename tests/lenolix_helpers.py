@@ -1,20 +1,7 @@
-"""Small Lenolix models for the tests: configurations, seeded weights that make attention sharp, and a driver that runs
-given tokens through the engine in arbitrary portions."""
-import copy
-import json
-import os
-
-import pytest
+"""Small Lenolix models for the tests: configurations and seeded weights that make attention sharp."""
 import torch
 
-from ksanallm_b200.config import EngineConfig, model_config_from_hf
-from ksanallm_b200.models.weights import DictSource, build_model
-from ksanallm_b200.runtime.engine import LLMEngine
-
-gpu = pytest.mark.gpu
-# where the same test runs: the plain statements of the ops, and the kernels in both precisions
-PLACES = [pytest.param("cpu", torch.float32, id="cpu-f32"), pytest.param("cuda", torch.float32, id="gpu-f32", marks=gpu),
-          pytest.param("cuda", torch.bfloat16, id="gpu-bf16", marks=gpu)]
+from decoder_helpers import PLACES, build, engine, error, run_portions, save_checkpoint, tokens  # noqa: F401
 ROTATION = {"base": 5000.0, "dims": 8, "scaling": {"factor": 3.0, "low": 1.5, "high": 6.0, "original": 120}}
 
 
@@ -116,55 +103,3 @@ def weights(c, seed=0):
             t = 0.8 + 0.3 * t
         w[name] = t.bfloat16().float()
     return w
-
-
-def save_checkpoint(path, c, w):
-    from safetensors.torch import save_file
-    os.makedirs(path, exist_ok=True)
-    with open(os.path.join(path, "config.json"), "w") as f:
-        json.dump(c, f)
-    save_file({k: v.bfloat16().contiguous() for k, v in w.items()}, os.path.join(path, "model.safetensors"))
-
-
-def build(c, w, device, dtype, max_positions=512):
-    return build_model(model_config_from_hf(copy.deepcopy(c)), DictSource(w, "lenolix"), device=device, dtype=dtype,
-                       max_positions=max_positions)
-
-
-def engine(c, w, device, dtype, blocks=64, max_len=None, host_blocks=0, block_tokens=16, graphs=False, **sched):
-    model = build(c, w, device, dtype)
-    ec = EngineConfig()
-    ec.block_manager.block_token_num = block_tokens
-    ec.batch_scheduler.max_batch_size = 8
-    ec.batch_scheduler.max_token_len = max_len or min(blocks * block_tokens, 512)
-    ec.global_.enable_cuda_graph = graphs
-    for k, v in sched.items():
-        setattr(ec.batch_scheduler, k, v)
-    return LLMEngine(model, model.cfg, ec, num_blocks=blocks, num_host_blocks=host_blocks)
-
-
-def tokens(c, n, seed=0):
-    return torch.randint(0, c["vocab"], (n,), generator=torch.Generator().manual_seed(1000 + seed)).tolist()
-
-
-@torch.inference_mode()
-def run_portions(eng, toks, sizes):
-    """Logits of every position of one request that arrives in portions of the given sizes (the last one repeats)."""
-    sid, out, at, k = eng.open_given(), [], 0, 0
-    while at < len(toks):
-        n = min(sizes[min(k, len(sizes) - 1)], len(toks) - at)
-        out.append(eng.step_given([(sid, toks[at:at + n], list(range(n)))]).float().cpu())
-        at, k = at + n, k + 1
-    eng.close_given(sid)
-    return torch.cat(out)
-
-
-def error(got, want):
-    """Largest error of a row: root mean square over the vocabulary, means taken off, relative to the rows' spread."""
-    d = got - want
-    d = d - d.mean(-1, keepdim=True)
-    scale = (want - want.mean(-1, keepdim=True)).pow(2).mean().sqrt()
-    return float(d.pow(2).mean(-1).sqrt().max() / scale)
-
-
-LIMIT = {torch.float32: 3e-5, torch.bfloat16: 0.1}

@@ -1,5 +1,7 @@
-"""Rank of the tensor-parallel test of the Lenolix family (launched by torchrun, gloo on the CPU): its shard of a seeded
-model runs a prompt in two portions; rank 0 writes the logits. argv: out_path config_name"""
+"""Rank of the tensor-parallel tests of the families whose layers are configured one by one (launched by torchrun, gloo
+on the CPU): its shard of a seeded model runs a prompt in two portions; rank 0 writes the logits. argv: out_path family
+config_name"""
+import importlib
 import os
 import sys
 
@@ -9,7 +11,6 @@ import torch.distributed as dist
 sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
 sys.path.insert(0, os.path.dirname(os.path.abspath(__file__)))
 
-import lenolix_helpers as hlp  # noqa: E402
 from ksanallm_b200.config import model_config_from_hf  # noqa: E402
 from ksanallm_b200.models.common import StepInput  # noqa: E402
 from ksanallm_b200.models.weights import DictSource, build_model  # noqa: E402
@@ -17,12 +18,13 @@ from ksanallm_b200.parallel.comm import TPComm  # noqa: E402
 
 
 def main():
-    out, name = sys.argv[1], sys.argv[2]
+    out, family, name = sys.argv[1:4]
+    hlp = importlib.import_module(family + "_helpers")
     os.environ.setdefault("MASTER_ADDR", "127.0.0.1")
     dist.init_process_group("gloo")
     rank, world = dist.get_rank(), dist.get_world_size()
     c = hlp.SPLIT.get(name) or hlp.CONFIGS[name]
-    model = build_model(model_config_from_hf(c), DictSource(hlp.weights(c, 3), "lenolix"), rank, world,
+    model = build_model(model_config_from_hf(c), DictSource(hlp.weights(c, 3), family), rank, world,
                         TPComm(dist.group.WORLD, rank, world, "nccl", "cpu"), device="cpu", dtype=torch.float32, max_positions=256)
     model.allocate_kv_cache(8, 16)
     t, parts, at = hlp.tokens(c, 60), [], 0

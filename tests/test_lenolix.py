@@ -13,7 +13,8 @@ import torch
 
 import lenolix_helpers as hlp
 import lenolix_oracle as oracle
-from lenolix_helpers import CONFIGS, LIMIT, PLACES, gpu
+from decoder_helpers import LIMIT, PLACES, check, greedy, greedy_within_rounding, run_batch
+from lenolix_helpers import CONFIGS
 from ksanallm_b200.config import EngineConfig, model_config_from_hf
 from ksanallm_b200.llm import LLM
 from ksanallm_b200.ops import native
@@ -37,14 +38,6 @@ def truth(name, n, seed=0):
 
 def engine(name, device, dtype, **kw):
     return hlp.engine(CONFIGS[name], weights_of(name), device, dtype, **kw)
-
-
-def check(got, want, dtype, device):
-    if device == "cuda":
-        native.check_err_flag("cuda")
-    assert torch.isfinite(got).all()
-    e = hlp.error(got, want)
-    assert e < LIMIT[dtype], e
 
 
 # ------------------------------------------------------------------------------------------------ one request
@@ -91,36 +84,6 @@ def test_other_block_sizes(block_tokens, device, dtype):
 
 
 # ------------------------------------------------------------------------------------------------ batches
-@torch.inference_mode()
-def run_batch(eng, requests, seed, slots=4):
-    """Feeds requests (token lists) in random portions, up to ``slots`` live at a time; a request may pause. Returns the
-    logits of every position per request."""
-    rng = np.random.default_rng(seed)
-    waiting, live, out = list(range(len(requests))), {}, {i: [] for i in range(len(requests))}
-    at = {i: 0 for i in out}
-    while waiting or live:
-        while waiting and len(live) < slots:
-            i = waiting.pop(0)
-            live[i] = eng.open_given()
-        entries, who = [], []
-        for i in rng.permutation(sorted(live)).tolist():
-            if len(live) > 1 and rng.random() < 0.2:
-                continue
-            left = len(requests[i]) - at[i]
-            n = min(left, 1 if rng.random() < 0.5 else int(rng.integers(2, 40)))
-            entries.append((live[i], requests[i][at[i]:at[i] + n], list(range(n))))
-            who.append((i, n))
-        if not entries:
-            continue
-        logits, k = eng.step_given(entries).float().cpu(), 0
-        for i, n in who:
-            out[i].append(logits[k:k + n])
-            k, at[i] = k + n, at[i] + n
-            if at[i] == len(requests[i]):
-                eng.close_given(live.pop(i))
-    return [torch.cat(out[i]) for i in range(len(requests))]
-
-
 @pytest.mark.parametrize("device,dtype", PLACES)
 @pytest.mark.parametrize("name", NAMES)
 def test_mixed_batches_and_reused_blocks(name, device, dtype):
@@ -174,18 +137,8 @@ def test_plans_carry_the_previous_tokens():
 
 
 # ------------------------------------------------------------------------------------------------ generation
-def greedy(n):
-    s = ne.SamplingConfig()
-    s.max_new_tokens, s.ignore_eos, s.topk = n, True, 1
-    return s
-
-
 def assert_greedy(name, prompt, out, dtype):
-    """Every generated token is the oracle's best one at its place (within rounding)."""
-    lg = oracle.forward(prompt + out[:-1], CONFIGS[name], weights_of(name))[len(prompt) - 1:]
-    spread = float(lg.std())
-    for row, tok in zip(lg, out):
-        assert float(row.max() - row[tok]) <= (1e-3 if dtype == torch.float32 else 0.12) * spread
+    greedy_within_rounding(oracle.forward(prompt + out[:-1], CONFIGS[name], weights_of(name))[len(prompt) - 1:], out, dtype)
 
 
 PROMPTS = (70, 1, 33, 18, 96, 2)
@@ -457,7 +410,7 @@ def test_tensor_parallel_shards(tmp_path, name, world):
         port = s.getsockname()[1]
     out = str(tmp_path / "logits.pt")
     r = subprocess.run([sys.executable, "-m", "torch.distributed.run", "--nnodes=1", f"--nproc-per-node={world}", "--master-addr",
-                        "127.0.0.1", "--master-port", str(port), os.path.join(ROOT, "tests", "lenolix_tp_worker.py"), out, name],
+                        "127.0.0.1", "--master-port", str(port), os.path.join(ROOT, "tests", "stream_tp_worker.py"), out, "lenolix", name],
                        env=dict(os.environ, CUDA_VISIBLE_DEVICES="", OMP_NUM_THREADS="2"), capture_output=True, text=True, timeout=300)
     assert r.returncode == 0, r.stderr[-3000:]
     c = hlp.SPLIT.get(name) or CONFIGS[name]
