@@ -187,9 +187,9 @@ def main():
     ap.add_argument("--breakdown", action="store_true",
                     help="instead of the benchmark: device time of one decode step and one prefill step of this model by "
                          "kernel class (benchmarks/step_breakdown.py; --layers limits the depth, --comm picks the path)")
-    ap.add_argument("--design", default=None, choices=["lenolix"],
-                    help="instead of the benchmark: prefill and decode throughput of this model family beside the dense "
-                         "model at equal sizes, kernel by kernel (benchmarks/lenolix_bench.py)")
+    ap.add_argument("--design", default=None, choices=["lenolix", "rasizen"],
+                    help="instead of the benchmark: prefill and decode throughput of this model family beside the "
+                         "closest other model at equal sizes, kernel by kernel (benchmarks/<design>_bench.py)")
     ap.add_argument("--sizes", default="1b,3b,8b", help="--design: sizes to run")
     ap.add_argument("--window", type=int, default=512, help="--design: sliding window")
     ap.add_argument("--keep-first", type=int, default=64, help="--design: first tokens that stay visible")
@@ -201,9 +201,9 @@ def main():
     args = ap.parse_args()
 
     if args.design is not None:
-        from benchmarks import lenolix_bench
+        import importlib
         args.layers = args.layers or 8
-        return lenolix_bench.main(args)
+        return importlib.import_module(f"benchmarks.{args.design}_bench").main(args)
 
     if args.breakdown:
         from benchmarks import step_breakdown

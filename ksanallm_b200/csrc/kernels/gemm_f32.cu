@@ -11,12 +11,13 @@ constexpr int kSgTile = 64, kSgK = 16, kSgThreads = 256;
 __global__ void __launch_bounds__(kSgThreads)
 gemm_f32_kernel(const float* __restrict__ A, int lda, const float* __restrict__ W, int ldw, float* __restrict__ D, int ldd,
                 const float* __restrict__ bias, const float* __restrict__ residual, int ldr, int M, int N, int K,
-                long long a_batch, long long w_batch, long long d_batch) {
+                long long a_batch, long long w_batch, long long d_batch, const float* __restrict__ gate, int ldg, long long g_batch) {
   pdl_trigger();
   pdl_wait();
   A += blockIdx.z * a_batch;
   W += blockIdx.z * w_batch;
   D += blockIdx.z * d_batch;
+  if (gate) gate += blockIdx.z * g_batch;
   __shared__ float as[kSgK][kSgTile + 4], ws[kSgK][kSgTile + 4];
   const int m0 = blockIdx.y * kSgTile, n0 = blockIdx.x * kSgTile;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
@@ -53,6 +54,7 @@ gemm_f32_kernel(const float* __restrict__ A, int lda, const float* __restrict__ 
       float v = acc[i][j];
       if (bias) v += bias[n];
       if (residual) v += residual[static_cast<size_t>(m) * ldr + n];
+      if (gate) v /= 1.f + __expf(-gate[static_cast<size_t>(m) * ldg + n]);
       D[static_cast<size_t>(m) * ldd + n] = v;
     }
   }
@@ -68,16 +70,17 @@ extern "C" int ksana_gemm_f32(const float* A, int lda, const float* W, int ldw, 
   const dim3 grid((N + kSgTile - 1) / kSgTile, (M + kSgTile - 1) / kSgTile);
   if (grid.y > 65535u) return -10;
   return launch_pdl(gemm_f32_kernel, grid, dim3(kSgThreads), 0, st, A, lda, W, ldw, D, ldd, bias, residual, ldr, M, N, K,
-                    0LL, 0LL, 0LL) == cudaSuccess ? 0 : -4;
+                    0LL, 0LL, 0LL, static_cast<const float*>(nullptr), 0, 0LL) == cudaSuccess ? 0 : -4;
 }
 
-// D[b] = A[b] W[b]^T for every b; a_batch / w_batch / d_batch: elements between batch entries.
+// D[b] = A[b] W[b]^T for every b, with a gate times sigmoid(gate[b]) element by element; a_batch / w_batch / d_batch: elements between batch entries.
 extern "C" int ksana_gemm_f32_batched(const float* A, int lda, long long a_batch, const float* W, int ldw, long long w_batch,
-                                      float* D, int ldd, long long d_batch, int batch, int M, int N, int K, cudaStream_t st) {
+                                      float* D, int ldd, long long d_batch, int batch, int M, int N, int K, const float* gate,
+                                      int ldg, long long g_batch, cudaStream_t st) {
   if (M <= 0 || N <= 0 || K <= 0 || batch <= 0) return 0;
   const dim3 grid((N + kSgTile - 1) / kSgTile, (M + kSgTile - 1) / kSgTile, batch);
   if (grid.y > 65535u || batch > 65535) return -10;
   const float* none = nullptr;
   return launch_pdl(gemm_f32_kernel, grid, dim3(kSgThreads), 0, st, A, lda, W, ldw, D, ldd, none, none, 0, M, N, K, a_batch, w_batch,
-                    d_batch) == cudaSuccess ? 0 : -4;
+                    d_batch, gate, ldg, g_batch) == cudaSuccess ? 0 : -4;
 }

@@ -61,6 +61,9 @@ struct GemmParams {
   // after D_{b-1} (any layout in which a row of D_b is contiguous: e.g. head-interleaved [rows, batch, N])
   int batch;
   long long d_batch_stride;
+  // output gate (batched mode): D_b is multiplied element by element with sigmoid(gate_b); null: none
+  const __nv_bfloat16* gate;
+  long long gate_ld, gate_batch_stride;
 };
 
 template <int BN, int KIND>
@@ -95,7 +98,8 @@ __device__ __forceinline__ void tile_coords(int tile, int m_tiles, int n_tiles, 
   n_blk = in_group / gsz;
 }
 
-template <int BN, int KIND>
+// GATED: batched bf16 products with an output gate in the epilogue (an instance of its own, the plain epilogue stays lean)
+template <int BN, int KIND, bool GATED>
 __global__ void __launch_bounds__(GemmCfg<BN, KIND>::kThreads, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant__ CUtensorMap tma_b,
                     const GemmParams p) {
@@ -239,7 +243,14 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_cons
       const int row = m0 + q * 32 + lane;
       const bool row_ok = row < p.M;
 
-      auto store_chunk = [&](int c0, const float (&v)[32]) {
+      // the gate's columns of one 32-column chunk of this row, fetched a chunk ahead of their use
+      auto fetch_gate = [&](int c0, uint4 (&g)[4]) {
+        const __nv_bfloat16* src = p.gate + static_cast<size_t>(b) * p.gate_batch_stride + static_cast<size_t>(row) * p.gate_ld;
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          if (row_ok && n0 + c0 + i * 8 < p.N) g[i] = __ldg(reinterpret_cast<const uint4*>(src + n0 + c0 + i * 8));
+      };
+      auto store_chunk = [&](int c0, const float (&v)[32], const uint4* gv = nullptr) {
         if (!row_ok) return;
         const int col0 = n0 + c0;
 #pragma unroll
@@ -261,6 +272,15 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_cons
 #pragma unroll
             for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(r2[i]); o[2 * i] += f.x; o[2 * i + 1] += f.y; }
           }
+          if (GATED) {
+            const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gv[g]);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              const float2 f = __bfloat1622float2(g2[i]);
+              o[2 * i] = o[2 * i] / (1.f + __expf(-f.x));
+              o[2 * i + 1] = o[2 * i + 1] / (1.f + __expf(-f.y));
+            }
+          }
           if (p.out_f32) {
             float4* dst = reinterpret_cast<float4*>(p.out_f32 + static_cast<size_t>(row) * p.ldd + col);
             dst[0] = make_float4(o[0], o[1], o[2], o[3]);
@@ -281,17 +301,21 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_cons
       };
 
       if (KIND == kBf16) {
+        uint4 gate_next[4] = {};
+        if (GATED) fetch_gate(0, gate_next);
         if (!mbar_wait(&tfull_bar[acc], acc_phase, abort_flag)) { ok = false; break; }
         tc_fence_after();
 #pragma unroll
         for (int c0 = 0; c0 < BN; c0 += 32) {
+          const uint4 gate_now[4] = {gate_next[0], gate_next[1], gate_next[2], gate_next[3]};
+          if (GATED && c0 + 32 < BN) fetch_gate(c0 + 32, gate_next);
           uint32_t r[32];
           tmem_ld32(tmem_base + lane_base + acc * BN + c0, r);
           tmem_ld_wait();
           float v[32];
 #pragma unroll
           for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
-          store_chunk(c0, v);
+          store_chunk(c0, v, gate_now);
         }
         tc_fence_before();
         mbar_arrive(&tempty_bar[acc]);
@@ -391,13 +415,13 @@ static int num_sms() {
   return g_num_sms;
 }
 
-template <int BN, int KIND>
+template <int BN, int KIND, bool GATED = false>
 static int launch_gemm(const CUtensorMap& ma, const CUtensorMap& mb, const GemmParams& p, int max_ctas,
                        cudaStream_t stream) {
   using Cfg = GemmCfg<BN, KIND>;
   static bool attr_set = false;
   if (!attr_set) {
-    cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_kernel<BN, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_kernel<BN, KIND, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          Cfg::kSmemBytes);
     if (e != cudaSuccess) return -3;
     attr_set = true;
@@ -405,7 +429,7 @@ static int launch_gemm(const CUtensorMap& ma, const CUtensorMap& mb, const GemmP
   const int tiles = ((p.M + kBM - 1) / kBM) * ((p.N + BN - 1) / BN) * (p.batch > 0 ? p.batch : 1);
   int grid = tiles < num_sms() ? tiles : num_sms();
   if (max_ctas > 0 && grid > max_ctas) grid = max_ctas;
-  gemm_tcgen05_kernel<BN, KIND><<<grid, Cfg::kThreads, Cfg::kSmemBytes, stream>>>(ma, mb, p);
+  gemm_tcgen05_kernel<BN, KIND, GATED><<<grid, Cfg::kThreads, Cfg::kSmemBytes, stream>>>(ma, mb, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
@@ -484,7 +508,8 @@ static int make_batched_map(CUtensorMap* map, const void* base, int rows, int co
 
 extern "C" int ksana_gemm_bf16_batched(const void* A, long long lda, long long a_batch, const void* W, long long ldw,
                                        long long w_batch, void* D, long long ldd, long long d_batch, int batch, int M,
-                                       int N, int K, int* err_flag, cudaStream_t stream) {
+                                       int N, int K, const void* gate, long long ldg, long long g_batch, int* err_flag,
+                                       cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0 || batch <= 0) return 0;
   if ((N % 8) || (K % 8) || (lda % 8) || (ldw % 8) || (ldd % 8) || (a_batch % 8) || (w_batch % 8) || (d_batch % 8) ||
       ldd > 0x7fffffffLL) return -10;
@@ -503,6 +528,16 @@ extern "C" int ksana_gemm_bf16_batched(const void* A, long long lda, long long a
   p.err = err_flag;
   p.batch = batch;
   p.d_batch_stride = d_batch;
+  if (gate && ((ldg % 8) || (g_batch % 8) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -11;
+  p.gate = static_cast<const __nv_bfloat16*>(gate); p.gate_ld = ldg; p.gate_batch_stride = g_batch;
+  if (gate) {
+    switch (bn) {
+      case 256: return launch_gemm<256, kBf16, true>(ma, mb, p, 0, stream);
+      case 128: return launch_gemm<128, kBf16, true>(ma, mb, p, 0, stream);
+      case 64: return launch_gemm<64, kBf16, true>(ma, mb, p, 0, stream);
+      default: return launch_gemm<32, kBf16, true>(ma, mb, p, 0, stream);
+    }
+  }
   switch (bn) {
     case 256: return launch_gemm<256, kBf16>(ma, mb, p, 0, stream);
     case 128: return launch_gemm<128, kBf16>(ma, mb, p, 0, stream);

@@ -62,7 +62,8 @@ struct MlaParams {
   const int* block_table; int table_stride;
   const int* cu_q; const int* kv_lens;
   int G, block_tokens, box_rows, nsplit, T;
-  int panels, kmmas, dv;                      // 64-column panels of a row, K = 16 steps over its columns, value columns
+  int dv;                                     // value columns
+  int rows_per_block;                         // cache rows between consecutive blocks (a 2-D map); 0: not whole rows, 3-D map
   int window;                                 // keys a query sees, itself included; 0: all earlier ones
   int num_blocks;                             // blocks addressable from the layer base (block-table entries are checked)
   float scale_log2;
@@ -75,6 +76,10 @@ __device__ __forceinline__ float mla_exp2(float x) {
   return y;
 }
 
+// PANELS: 64-column panels of a row. FLAT: the cache blocks are whole rows apart (a 2-D map serves them). WINDOW: with a
+// sliding window. All three are compile-time: the issue loops of the MMA and TMA threads and the softmax are the critical
+// path, and run-time forms of them cost a plain decode step 5 to 15 % each.
+template <int PANELS, bool FLAT, bool WINDOW>
 __global__ void __launch_bounds__(kMlaThreads, 1)
 mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap kv_map, const MlaParams p) {
   extern __shared__ uint8_t mla_smem_raw[];
@@ -113,12 +118,12 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
   const int last_row = min(row0 + kMlaM - 1, q_len * G - 1);
   const int kv_end = min(kv_len, past + last_row / G + 1);
   // tiles from the first key that the first row sees to the last one that the last row sees
-  const int tile_first = p.window > 0 ? max(0, past + row0 / G - p.window + 1) / kMlaTok : 0;
+  const int tile_first = WINDOW ? max(0, past + row0 / G - p.window + 1) / kMlaTok : 0;
   const int tile_end = (kv_end + kMlaTok - 1) / kMlaTok;
   const int per = (tile_end - tile_first + p.nsplit - 1) / p.nsplit;
   const int tile_lo = tile_first + split * per;
   const int ntiles = max(min(tile_end, tile_lo + per) - tile_lo, 0);
-  const int panels = p.panels, q_tmem = min(panels, kMlaQTmemPanels);
+  constexpr int panels = PANELS, q_tmem = PANELS < kMlaQTmemPanels ? PANELS : kMlaQTmemPanels;
   const int cols = min(256, p.dv - half * 256);             // output columns of this half
   const int* table = p.block_table + static_cast<size_t>(s) * p.table_stride;
 
@@ -168,6 +173,7 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
       // Q: the first panels into the (still unused) KV stages as a staging area for their copy to TMEM, the rest to
       // their home. Rows of a tile are consecutive (token, head) pairs; those past the sequence are computed and dropped
       mbar_expect_tx(q_full, panels * kMlaQPanelBytes);
+#pragma unroll
       for (int pn = 0; pn < panels; ++pn) {
         uint8_t* dst = pn < kMlaQTmemPanels ? kv_s + pn * kMlaQPanelBytes : q_s + (pn - kMlaQTmemPanels) * kMlaQPanelBytes;
         tma_load_2d(dst, &q_map, q_full, pn * 64, q0 * G + row0);
@@ -211,7 +217,10 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
           for (int bx = 0; bx < kMlaMaxBoxes; ++bx) {
             if (bx < nbox) {
               const int t = t0 + bx * br;
-              tma_load_3d(dst + bx * br * 128, &kv_map, kv_full + b, lane * 64, t % bt, blk[bx]);
+              if (FLAT)
+                tma_load_2d(dst + bx * br * 128, &kv_map, kv_full + b, lane * 64, blk[bx] * p.rows_per_block + t % bt);
+              else
+                tma_load_3d(dst + bx * br * 128, &kv_map, kv_full + b, lane * 64, t % bt, blk[bx]);
             }
           }
         }
@@ -255,8 +264,8 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
           const int bb = s_next & 1;
           tc_fence_after();
           const uint32_t kb = smem_u32(kv_s + (s_next % kMlaStages) * kMlaKvBytes);
-#pragma unroll 4
-          for (int k = 0; k < p.kmmas; ++k) {
+#pragma unroll
+          for (int k = 0; k < 4 * PANELS; ++k) {
             const int pn = k >> 2;
             const uint64_t bdesc = make_smem_desc_sw128(kb + pn * kMlaKvPanelBytes) + 2 * (k & 3);
             if (pn < kMlaQTmemPanels) {
@@ -288,7 +297,7 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
     const bool active = vr < q_len * G;
     const int tok = vr / G, head = vr % G;
     const int limit = active ? past + tok : -1;            // last visible KV position
-    const int lowest = p.window > 0 ? limit - p.window + 1 : 0;              // first visible one
+    const int lowest = WINDOW ? limit - p.window + 1 : 0;              // first visible one
     float m_used = -CUDART_INF_F, l = 0.f;
     bool ok = mbar_wait(q_full, 0, abort_flag);
     if (ok) {
@@ -324,7 +333,7 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
       float mx = -CUDART_INF_F;
 #pragma unroll
       for (int i = 0; i < kMlaTok; ++i) {
-        const float v = (t0 + i <= limit && t0 + i >= lowest) ? __uint_as_float(r[i]) * p.scale_log2 : -CUDART_INF_F;
+        const float v = (t0 + i <= limit && (!WINDOW || t0 + i >= lowest)) ? __uint_as_float(r[i]) * p.scale_log2 : -CUDART_INF_F;
         r[i] = __float_as_uint(v);
         mx = fmaxf(mx, v);
       }
@@ -561,6 +570,18 @@ static cudaError_t launch_rope_append(const void* q, long long q_stride, int nop
   return launch_pdl(mla_rope_append_kernel<T>, dim3(T_), dim3(kLatentThreads), 0, st, p);
 }
 
+template <int PANELS, bool FLAT, bool WINDOW>
+static int launch_mla(dim3 grid, const CUtensorMap& q_map, const CUtensorMap& kv_map, const MlaParams& p, cudaStream_t st) {
+  static bool set = false;
+  if (!set) {
+    if (cudaFuncSetAttribute(mla_tc_kernel<PANELS, FLAT, WINDOW>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMlaSmemBytes) != cudaSuccess)
+      return -3;
+    set = true;
+  }
+  mla_tc_kernel<PANELS, FLAT, WINDOW><<<grid, kMlaThreads, kMlaSmemBytes, st>>>(q_map, kv_map, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
 typedef CUresult (*MlaEncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
                                 const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
                                 CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
@@ -616,7 +637,17 @@ extern "C" int ksana_mla_attention(const void* q, long long T, void* out, long l
             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS) return -100;
   }
-  {
+  const long long span = (num_blocks - 1LL) * (block_stride / dk) + bt;               // rows from the base to the last block's end
+  const bool flat = block_stride % dk == 0 && span < (1LL << 31) && window == 0 && (dk + 63) / 64 == 9;
+  if (flat) {
+    cuuint64_t dims[2] = {static_cast<cuuint64_t>(dk), static_cast<cuuint64_t>(span)};
+    cuuint64_t strides[1] = {static_cast<cuuint64_t>(dk) * 2};
+    cuuint32_t box[2] = {64, static_cast<cuuint32_t>(box_rows)};
+    cuuint32_t estr[2] = {1, 1};
+    if (enc(&kv_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(cache), dims, strides, box, estr,
+            CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+            CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS) return -100;
+  } else {
     cuuint64_t dims[3] = {static_cast<cuuint64_t>(dk), static_cast<cuuint64_t>(bt), static_cast<cuuint64_t>(num_blocks)};
     cuuint64_t strides[2] = {static_cast<cuuint64_t>(dk) * 2, static_cast<cuuint64_t>(block_stride) * 2};
     cuuint32_t box[3] = {64, static_cast<cuuint32_t>(box_rows), 1};
@@ -625,25 +656,35 @@ extern "C" int ksana_mla_attention(const void* q, long long T, void* out, long l
             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS) return -100;
   }
-  static bool set = false;
-  if (!set) {
-    if (cudaFuncSetAttribute(mla_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kMlaSmemBytes) != cudaSuccess)
-      return -3;
-    set = true;
-  }
   MlaParams p{};
   p.out = static_cast<bf16*>(out); p.out_tok_stride = out_tok_stride;
   p.part_o = part_o; p.part_ml = part_ml;
   p.block_table = block_table; p.table_stride = table_stride; p.cu_q = cu_q; p.kv_lens = kv_lens;
   p.G = G; p.block_tokens = bt; p.box_rows = box_rows; p.nsplit = nsplit; p.T = static_cast<int>(T);
-  p.panels = (dk + 63) / 64; p.kmmas = (dk + 15) / 16; p.dv = dv; p.window = window;
+  p.dv = dv; p.window = window > 0 ? window : 1 << 30; p.rows_per_block = flat ? static_cast<int>(block_stride / dk) : 0;
   p.num_blocks = num_blocks;
   p.scale_log2 = scale * 1.44269504f;
   p.err = err;
   const int nqt = (max_q_len * G + kMlaM - 1) / kMlaM;
   dim3 grid(nqt * nsplit, (dv + 255) / 256, B);
-  mla_tc_kernel<<<grid, kMlaThreads, kMlaSmemBytes, st>>>(q_map, kv_map, p);
-  if (cudaGetLastError() != cudaSuccess) return -4;
+  const int panels = (dk + 63) / 64;
+  int rc = -100;
+  if (flat) {
+    rc = launch_mla<9, true, false>(grid, q_map, kv_map, p, st);
+  } else {
+    switch (panels) {
+      case 1: rc = launch_mla<1, false, true>(grid, q_map, kv_map, p, st); break;
+      case 2: rc = launch_mla<2, false, true>(grid, q_map, kv_map, p, st); break;
+      case 3: rc = launch_mla<3, false, true>(grid, q_map, kv_map, p, st); break;
+      case 4: rc = launch_mla<4, false, true>(grid, q_map, kv_map, p, st); break;
+      case 5: rc = launch_mla<5, false, true>(grid, q_map, kv_map, p, st); break;
+      case 6: rc = launch_mla<6, false, true>(grid, q_map, kv_map, p, st); break;
+      case 7: rc = launch_mla<7, false, true>(grid, q_map, kv_map, p, st); break;
+      case 8: rc = launch_mla<8, false, true>(grid, q_map, kv_map, p, st); break;
+      case 9: rc = launch_mla<9, false, true>(grid, q_map, kv_map, p, st); break;
+    }
+  }
+  if (rc) return rc;
   if (nsplit > 1) {
     mla_merge_kernel<<<static_cast<unsigned>(T) * G, (dv / 4 + 31) / 32 * 32, 0, st>>>(
         part_o, part_ml, static_cast<bf16*>(out), out_tok_stride, static_cast<int>(T), G, nsplit, dv);

@@ -9,7 +9,7 @@ state after the last of the block's tokens that has been computed. Blocks are th
 forks, swaps and recomputation act on them as on a pure attention model's. Per sublayer:
 
   attention    [q | latent, rotary key | gate] GEMM -> latent norm + rotations + append -> q W_uk -> attention over the
-               latent rows -> W_uv -> gate -> output GEMM -> [scaled residual add, next norm] in one kernel
+               latent rows -> W_uv with the output gate in its epilogue -> output GEMM -> [scaled residual add, next norm] in one kernel
   recurrence   [z | x | g] GEMM -> scan with gates, states and output gate in one kernel -> output GEMM -> same kernel
   feed-forward up GEMM -> unit -> down GEMM -> same kernel
 
@@ -92,8 +92,8 @@ class RasizenModel(StreamModel):
         ops.bmm(q[..., :dim].transpose(0, 1), lw.uk_t, qfull[..., :rank].transpose(0, 1))
         o_lat = ops.latent_attention(qfull, cache, rank, self.block_tokens, step, m.scale, m.window)
         o = torch.empty(T, H, pad8(m.vdim), dtype=y.dtype, device=y.device)
-        ops.bmm(o_lat.transpose(0, 1), lw.uv, o.transpose(0, 1))
-        return ops.sigmoid_gate(o.view(T, ng), g)
+        ops.bmm(o_lat.transpose(0, 1), lw.uv, o.transpose(0, 1), gate=g.unflatten(1, (H, -1)).transpose(0, 1))
+        return o.view(T, ng)
 
     def recurrence(self, i: int, lw: HybridLayer, xn: torch.Tensor, step: StepInput) -> torch.Tensor:
         return ops.gated_recurrence(ops.linear(xn, lw.w_in), lw.channels, self.panels[i], self.block_tokens, step, CANDIDATE_OFFSET)

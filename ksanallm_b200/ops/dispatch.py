@@ -319,13 +319,6 @@ def xielu(x, pos, neg, lin=0.5):
     return native.xielu(x, pos, neg, lin) if x.is_cuda else ref.xielu(x, pos, neg, lin)
 
 
-def sigmoid_gate(a, gate):
-    """a * sigmoid(gate), in place on ``a``; ``gate`` may be a column range of wider rows."""
-    if a.is_cuda:
-        return native.sigmoid_gate(a, gate, out=a)
-    return a.copy_(ref.sigmoid_gate(a, gate))
-
-
 def gated_recurrence(y, W, state, block_tokens, step, offset=0.5):
     """S_t = (1 - gate) S_(t-1) + gate * cand with gate = sigmoid(z) and cand = u + offset (u >= 0) or sigmoid(u), out =
     S_t * silu(g), over a step's new rows; y [T, 3 W] holds z | u | g. ``state`` [blocks, W] (fp32, part of the cache's
@@ -339,16 +332,17 @@ def gated_recurrence(y, W, state, block_tokens, step, offset=0.5):
         native.gated_recurrence(z, u, g, out, state, block_tokens, step.block_table, step.cu_q, step.kv_lens[:nm], offset)
     if ns:
         native.gated_recurrence(z[tm:], u[tm:], g[tm:], out[tm:], state, block_tokens, step.block_table[nm:], None,
-                                step.kv_lens[nm:], offset)
+                                step.kv_lens[nm:], offset, slots=step.slots[tm:])
     return out
 
 
 # ------------------------------------------------------------------------------- latent attention
-def bmm(a, w, out):
-    """out[b] = a[b] w[b]^T over (strided) views a [B, M, K], w [B, N, K], out [B, M, N]."""
+def bmm(a, w, out, gate=None):
+    """out[b] = a[b] w[b]^T (times sigmoid(gate[b])) over (strided) views a [B, M, K], w [B, N, K], out and gate [B, M, N]."""
     if not a.is_cuda:
-        return out.copy_(torch.matmul(a.float(), w.float().transpose(1, 2)))
-    return (native.gemm_f32_batched if a.dtype == torch.float32 else native.gemm_bf16_batched)(a, w, out)
+        y = torch.matmul(a.float(), w.float().transpose(1, 2))
+        return out.copy_(y if gate is None else y * torch.sigmoid(gate.float()))
+    return (native.gemm_f32_batched if a.dtype == torch.float32 else native.gemm_bf16_batched)(a, w, out, gate)
 
 
 def latent_append(q, nope, kv, norm: Optional[NormParams], step, cos_sin, cache, block_tokens):

@@ -22,7 +22,7 @@ _SIGS = {
     "ksana_gemm_bf16": [vp, i32, vp, i32, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp],
     "ksana_gemm_pair": [i32, vp, i32, vp, i32, vp, i32, vp, vp, i32, vp, vp, i32, i32, i32, i32, vp, i32, i32, vp, vp],
     "ksana_gemm_nvfp4": [vp, i32, vp, i32, vp, vp, i32, vp, i32, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp],
-    "ksana_gemm_bf16_batched": [vp, i64, i64, vp, i64, i64, vp, i64, i64, i32, i32, i32, i32, vp, vp],
+    "ksana_gemm_bf16_batched": [vp, i64, i64, vp, i64, i64, vp, i64, i64, i32, i32, i32, i32, vp, i64, i64, vp, vp],
     "ksana_gemm_grouped_nvfp4": [vp, i32, vp, i32, vp, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, vp, i32, vp, vp],
     "ksana_quant_nvfp4": [vp, i32, vp, i32, vp, i32, vp, i32, i32, vp],
     "ksana_gemm_mxfp8": [vp, i32, vp, i32, vp, i32, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, vp, i32, i32, vp,
@@ -69,9 +69,8 @@ _SIGS = {
     "ksana_residual_norm": [vp, i32, vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, f32, i32, i32, f32, i32, vp, vp],
     "ksana_glu_clamp": [vp, vp, i32, i32, i32, f32, f32, f32, i32, vp],
     "ksana_xielu": [vp, i32, vp, i32, i32, i32, f32, f32, f32, i32, vp],
-    "ksana_sigmoid_gate": [vp, i32, vp, i32, vp, i32, i32, i32, i32, vp],
-    "ksana_gated_recurrence": [vp, vp, vp, i64, vp, i64, vp, i64, i32, i32, vp, i32, vp, vp, i32, i32, f32, i32, vp, vp],
-    "ksana_gemm_f32_batched": [vp, i32, i64, vp, i32, i64, vp, i32, i64, i32, i32, i32, i32, vp],
+    "ksana_gated_recurrence": [vp, vp, vp, i64, vp, i64, vp, i64, i32, i32, vp, i32, vp, vp, vp, i32, i32, f32, i32, vp, vp],
+    "ksana_gemm_f32_batched": [vp, i32, i64, vp, i32, i64, vp, i32, i64, i32, i32, i32, i32, vp, i32, i64, vp],
     "ksana_qkv_rope_append": [vp, vp, vp, vp, i32, vp, vp, i64, i32, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp],
     "ksana_refit_rows_f32": [vp, i32, vp, vp, i32, i32, i32, vp, vp],
     "ksana_gemm_f32": [vp, i32, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, vp],
@@ -484,16 +483,24 @@ def gemm_nvfp4(aq, a_bs, a_ts, wq, w_bs, w_ts, out=None, bias=None, residual=Non
     return dst
 
 
-def gemm_bf16_batched(a, w, out):
+def _gate_args(gate, out):
+    if gate is None:
+        return None, 0, 0
+    assert gate.shape == out.shape and gate.dtype == out.dtype and gate.stride(2) == 1
+    return _p(gate), gate.stride(1), gate.stride(0)
+
+
+def gemm_bf16_batched(a, w, out, gate=None):
     """out[b] = a[b] @ w[b]^T for every b: a [B, M, K], w [B, N, K], out [B, M, N], bf16 views with unit stride in the
     last dimension and any (16-byte aligned) strides in the others, e.g. head-interleaved activations
-    ``x.view(T, H, D).transpose(0, 1)``. One launch of the tcgen05 GEMM over all batch entries' tiles."""
+    ``x.view(T, H, D).transpose(0, 1)``. One launch of the tcgen05 GEMM over all batch entries' tiles. ``gate`` [B, M, N]:
+    the result is multiplied with sigmoid(gate) before it is stored."""
     B, M, K = a.shape
     N = w.shape[1]
     assert w.shape[0] == B and w.shape[2] == K and tuple(out.shape) == (B, M, N)
     assert a.stride(2) == 1 and w.stride(2) == 1 and out.stride(2) == 1
     rc = lib().ksana_gemm_bf16_batched(_p(a), a.stride(1), a.stride(0), _p(w), w.stride(1), w.stride(0), _p(out),
-                                       out.stride(1), out.stride(0), B, M, N, K, _p(err_flag(a.device)), _st())
+                                       out.stride(1), out.stride(0), B, M, N, K, *_gate_args(gate, out), _p(err_flag(a.device)), _st())
     _check(rc, "ksana_gemm_bf16_batched")
     return out
 
@@ -718,36 +725,26 @@ def xielu(x, pos, neg, lin, out=None):
     return out
 
 
-def sigmoid_gate(a, gate, out=None):
-    """a * sigmoid(gate) row by row; ``gate`` may be a column range of wider rows, ``out`` may be ``a``."""
-    M, I = a.shape
-    if out is None:
-        out = torch.empty(M, I, dtype=a.dtype, device=a.device)
-    assert gate.shape == a.shape and gate.dtype == a.dtype and gate.stride(1) == a.stride(1) == 1
-    _check(lib().ksana_sigmoid_gate(_p(a), a.stride(0), _p(gate), gate.stride(0), _p(out), out.stride(0), M, I,
-                                    int(a.dtype == torch.float32), _st()), "ksana_sigmoid_gate")
-    return out
-
-
-def gated_recurrence(z, u, g, out, state, block_tokens, block_table, cu_q, kv_lens, offset):
+def gated_recurrence(z, u, g, out, state, block_tokens, block_table, cu_q, kv_lens, offset, slots=None):
     """Recurrence over the new tokens of ``kv_lens.numel()`` sequences; z, u, g: column ranges [T, W] of one projection's
-    rows, ``state``: [blocks, W] fp32 rows inside the cache's block records. ``cu_q`` None: one row per sequence."""
+    rows, ``state``: [blocks, W] fp32 rows inside the cache's block records. ``slots``: every sequence has one row, with
+    this cache slot."""
     assert z.stride() == u.stride() == g.stride() and z.dtype == u.dtype == g.dtype == out.dtype and z.stride(1) == 1
     assert state.dtype == torch.float32 and state.stride(1) == 1
     _check(lib().ksana_gated_recurrence(_p(z), _p(u), _p(g), z.stride(0), _p(out), out.stride(0), _p(state), state.stride(0),
                                         block_tokens, state.shape[0], _p(block_table), block_table.stride(0), _p(cu_q), _p(kv_lens),
-                                        kv_lens.numel(), z.shape[1], float(offset), int(z.dtype == torch.float32),
+                                        _p(slots), kv_lens.numel(), z.shape[1], float(offset), int(z.dtype == torch.float32),
                                         _p(err_flag(z.device)), _st()), "ksana_gated_recurrence")
 
 
-def gemm_f32_batched(a, w, out):
+def gemm_f32_batched(a, w, out, gate=None):
     """:func:`gemm_bf16_batched` in fp32 on the CUDA cores."""
     B, M, K = a.shape
     N = w.shape[1]
     assert w.shape[0] == B and w.shape[2] == K and tuple(out.shape) == (B, M, N)
     assert a.stride(2) == 1 and w.stride(2) == 1 and out.stride(2) == 1
     _check(lib().ksana_gemm_f32_batched(_p(a), a.stride(1), a.stride(0), _p(w), w.stride(1), w.stride(0), _p(out), out.stride(1),
-                                        out.stride(0), B, M, N, K, _st()), "ksana_gemm_f32_batched")
+                                        out.stride(0), B, M, N, K, *_gate_args(gate, out), _st()), "ksana_gemm_f32_batched")
     return out
 
 

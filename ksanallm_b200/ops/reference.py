@@ -299,10 +299,6 @@ def xielu(x, pos, neg, lin):
     return (torch.where(z > 0, pos * z * z, neg * (torch.expm1(low) - low)) + lin * z).to(x.dtype)
 
 
-def sigmoid_gate(a, gate):
-    return (a.float() * torch.sigmoid(gate.float())).to(a.dtype)
-
-
 def gated_recurrence(z, u, g, state, block_tokens, block_table, cu_q, kv_lens, offset):
     """See dispatch.gated_recurrence; ``state`` [blocks, W] is updated in place."""
     out = torch.zeros(z.shape, dtype=z.dtype, device=z.device)

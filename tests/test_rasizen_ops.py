@@ -26,15 +26,16 @@ def close(got, want, dtype, scale=None):
     assert float((got - want).abs().max()) <= TOL[dtype] * s, float((got - want).abs().max()) / s
 
 
-def make_step(lens, tables, device):
-    """Step of sequences (cached, new), multi-token ones first; ``tables``: block ids per sequence."""
+def make_step(lens, tables, bt, device):
+    """Step of sequences (cached, new), multi-token ones first; ``tables``: block ids (of bt tokens) per sequence."""
     news = [n for _, n in lens]
     cu = torch.tensor([0] + news).cumsum(0).to(torch.int32)
     multi = sum(n > 1 for n in news)
     width = max(len(t) for t in tables) + 1
     table = torch.tensor([list(t) + [0] * (width - len(t)) for t in tables], dtype=torch.int32)
     kv = torch.tensor([p + n for p, n in lens], dtype=torch.int32)
-    return SimpleNamespace(block_table=table.to(device), cu_q=cu.to(device), kv_lens=kv.to(device), num_multi=multi,
+    slots = torch.tensor([tables[s][t // bt] * bt + t % bt for s, (p, n) in enumerate(lens) for t in range(p, p + n)], dtype=torch.int32)
+    return SimpleNamespace(slots=slots.to(device), block_table=table.to(device), cu_q=cu.to(device), kv_lens=kv.to(device), num_multi=multi,
                            num_single=len(news) - multi, num_multi_tokens=int(cu[multi]), max_q_len=max(news), max_kv_len=int(kv.max()))
 
 
@@ -69,14 +70,6 @@ def test_piecewise_unit(device, dtype, p, q):
     got = ops.xielu(x.to(device), oracle.softplus(p), 0.5 + oracle.softplus(q))
     # the two parts of the lower branch may cancel: errors are relative to the larger of them
     assert float(((got.double().cpu() - want).abs() / (want.abs() + x.double().abs() + 1e-3)).max()) < TOL[dtype]
-
-
-@pytest.mark.parametrize("device,dtype", PLACES)
-def test_output_gate(device, dtype):
-    a, wide = rand(0, 33, 40), rand(1, 33, 64) * 5
-    g = wide.to(device, dtype)[:, 16:56]
-    got = ops.sigmoid_gate(a.clone().to(device, dtype), g)
-    close(got, a * oracle.sigmoid(g.float().cpu()), dtype)
 
 
 # ------------------------------------------------------------------------------------------------ recurrence
@@ -118,7 +111,7 @@ def run_recurrence(W, lens, bt, device, dtype, portions=None, seed=0):
                 todo.append((s, min(p[min(turn, len(p) - 1)], n - done[s])))
         todo.sort(key=lambda e: e[1] == 1)
         y = torch.cat([torch.cat([t[done[s]:done[s] + n] for t in data[s]], 1) for s, n in todo]).to(device, dtype)
-        step = make_step([(done[s], n) for s, n in todo], [tables[s] for s, _ in todo], device)
+        step = make_step([(done[s], n) for s, n in todo], [tables[s] for s, _ in todo], bt, device)
         out, r = ops.gated_recurrence(y, W, state, bt, step).float().cpu(), 0
         for s, n in todo:
             outs[s].append(out[r:r + n])
@@ -169,12 +162,12 @@ def test_recurrence_padding_rows_and_bad_blocks():
     cache = torch.zeros(4, layout.record, dtype=torch.bfloat16, device="cuda")
     state = layout.view(cache, at)
     y = rand(0, 3, 3 * W).cuda().bfloat16()
-    step = make_step([(0, 1), (0, 1), (0, 1)], [[2], [0], [1]], "cuda")
-    step.kv_lens[1] = 0                                  # a padding row of a captured decode step
+    step = make_step([(0, 1), (0, 1), (0, 1)], [[2], [0], [1]], bt, "cuda")
+    step.kv_lens[1], step.slots[1] = 0, -1                                  # a padding row of a captured decode step
     out = ops.gated_recurrence(y, W, state, bt, step)
     assert not out[1].any() and not state[0].any() and out[0].any() and state[2].any()
     native.clear_err_flag("cuda")
-    bad = make_step([(0, 1)], [[4]], "cuda")             # a block id outside the cache: recorded and skipped
+    bad = make_step([(0, 1)], [[4]], bt, "cuda")             # a block id outside the cache: recorded and skipped
     ops.gated_recurrence(y[:1], W, state, bt, bad)
     with pytest.raises(RuntimeError):
         native.check_err_flag("cuda")
@@ -230,6 +223,11 @@ def test_batched_product(device, dtype, B, M, N, K):
     want = torch.einsum("mbk,bnk->mbn", a[..., :K].double(), w.double())
     close(out[..., 8:8 + N], want, dtype, scale=float(want.abs().max()))
     assert not out[..., :8].any() and not out[..., 8 + N:].any()
+    wide = (rand(2, M, 16 + B * N) * 4).to(device, dtype)              # the gate is a column range of wider rows
+    gate = wide[:, 16:].unflatten(1, (B, N))
+    ops.bmm(a.to(device, dtype)[..., :K].transpose(0, 1), w.to(device, dtype), out[..., 8:8 + N].transpose(0, 1), gate.transpose(0, 1))
+    want = want * oracle.sigmoid(gate.double().cpu())
+    close(out[..., 8:8 + N], want, dtype, scale=float(want.abs().max()))
 
 
 def latent_case(G, rank, rot, window, lens, bt, device, dtype, seed=0):
@@ -267,7 +265,7 @@ def latent_case(G, rank, rot, window, lens, bt, device, dtype, seed=0):
         for t in range(T):
             panel[blk[t // bt], t % bt] = kv[t].to(device, dtype)
         qs.append(q[past:])
-    got = ops.latent_attention(torch.cat(qs).to(device, dtype).contiguous(), panel, rank, bt, make_step(lens, tables, device), scale, window)
+    got = ops.latent_attention(torch.cat(qs).to(device, dtype).contiguous(), panel, rank, bt, make_step(lens, tables, bt, device), scale, window)
     return got, torch.cat(want)
 
 
