@@ -57,9 +57,10 @@ def engine_lib_path() -> Path:
     return LIB / f"_ksana_engine{suffix}"
 
 
-# what a dense decoder in bf16 or fp32 calls (no FP8 / FP4 / 4-bit weights, experts or peer memory)
-DENSE_KERNELS = ("attention", "attention_f32", "attention_tc", "elementwise", "gemm_f32", "gemm_smallm", "gemm_tcgen05",
-                 "mla_attention", "recurrence", "residual_stream", "sampler")
+# kernel sources that a family needs in bf16 or fp32 on one GPU (no FP8 / FP4 / 4-bit weights, experts or peer memory)
+_STREAM_KERNELS = ("attention_f32", "elementwise", "gemm_f32", "gemm_smallm", "gemm_tcgen05", "residual_stream", "sampler")
+FAMILY_KERNELS = {"lenolix": _STREAM_KERNELS + ("attention", "attention_tc"),
+                  "rasizen": _STREAM_KERNELS + ("mla_attention", "recurrence")}
 
 
 def build_kernels(force: bool = False, verbose: bool = False, only=None) -> Path:

@@ -332,8 +332,11 @@ static int launch_gated(const void* z, const void* u, const void* g, long long l
     const int vec = W / 8, threads = vec >= 128 ? 128 : (vec + 31) / 32 * 32;
     e = launch_pdl(gated_step_kernel<T>, dim3((vec + threads - 1) / threads, B), dim3(threads), 0, st, p);
   } else {
-    // 32 channels per CTA where that fills the GPU two and a half times over, else 16
-    return static_cast<long long>(B) * ((W + 31) / 32) >= 370 ? launch_tile<T, 4, 128>(p, B, st) : launch_tile<T, 2, 128>(p, B, st);
+    // 32 channels per CTA where that fills the GPU two and a half times over, else 16, with few sequences over more threads
+    const long long fill = 370, n = B;
+    if (n * ((W + 31) / 32) >= fill) return launch_tile<T, 4, 128>(p, B, st);
+    if (n * ((W + 15) / 16) >= fill) return launch_tile<T, 2, 128>(p, B, st);
+    return launch_tile<T, 2, 256>(p, B, st);
   }
   return e == cudaSuccess ? 0 : -4;
 }

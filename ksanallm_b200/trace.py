@@ -85,7 +85,7 @@ def main(argv=None) -> int:
     if a.dtype == "float32" and a.device == "cuda" and cfg.layer_specs is None:
         print(f"model type {cfg.model_type} is not served in float32", file=sys.stderr)
         return 3
-    build.ensure_built(only=build.DENSE_KERNELS if cfg.layer_specs is not None else None)
+    build.ensure_built(only=build.FAMILY_KERNELS.get(cfg.model_type))
     import torch
     with torch.inference_mode():
         llm = make_llm(a.model, a.dtype, a.max_tokens, a.device)
