@@ -238,7 +238,7 @@ class LatentAttentionSpec:
 
 @dataclass
 class GatedRecurrenceSpec:
-    """Element-wise recurrence whose gates read the current token only."""
+    """Element-wise recurrence that is linear in its state: the gates do not see the state."""
     width: int
 
 

@@ -1,4 +1,4 @@
-// Gated linear recurrence over the new tokens of a step, for recurrent layers whose gates read the current token only:
+// Gated linear recurrence over the new tokens of a step, for recurrent layers whose gates do not depend on the state:
 //
 //   gate_t = sigmoid(z_t),  cand_t = u_t + offset where u_t >= 0, sigmoid(u_t) elsewhere
 //   S_t = (1 - gate_t) S_(t-1) + gate_t cand_t,   out_t = S_t silu(g_t)        element by element

@@ -109,7 +109,7 @@ struct ResNormParams {
   int* err;
 };
 
-// z = the row v scaled by the reciprocal root mean square of each of its equal consecutive parts, times w2. Squares are
+// z = the row v scaled by the reciprocal root mean square of each of its `groups` parts of equal size, times w2. Squares are
 // summed per unit (a vector of 8, or a single element where a part is not a multiple of 8) in dynamic shared memory, one
 // warp per part. `part` holds H / unit sums, then one reciprocal per part.
 template <typename T, int VPT>

@@ -1,6 +1,6 @@
 """Rasizen: a pre-norm decoder with a 32-bit residual stream that mixes two kinds of layers: latent attention (absorbed
 form) with a sliding window and an output gate, where a layer may read another layer's latents, and a gated recurrence
-whose gates read the current token only. Norms take the root mean square of each of several equal parts of a row, the
+that is linear in its state (the gates do not see it). Norms take the root mean square of each of several equal parts of a row, the
 residual additions have a common factor, the feed-forwards are plain with a piecewise unit, any layer may lack one.
 
 The step functions, the block pool, the scheduler and the sampler are the ones of every other family. A cache block is one

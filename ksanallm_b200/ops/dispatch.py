@@ -245,7 +245,7 @@ def rope_kv_append(qkv, positions, slots, cos_sin, cache_layer, block_tokens, Hq
 @dataclass
 class NormParams:
     """Weight and optional bias of a norm over ``size`` real columns (stored padded with zeros to a multiple of 8).
-    ``groups`` > 1: root-mean-square norm of each of that many equal consecutive parts."""
+    ``groups`` > 1: root-mean-square norm of each of that many parts of equal size."""
     w: torch.Tensor
     b: Optional[torch.Tensor]
     size: int

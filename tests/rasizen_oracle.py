@@ -6,7 +6,7 @@ import torch
 
 
 def group_norm(x, w, groups, eps):
-    """Every one of the equal consecutive parts of a row divided by its own root mean square, then the weight."""
+    """RMS norm part by part (``groups`` parts of equal size), then the weight over the whole row."""
     size = x.shape[-1] // groups
     parts = []
     for g in range(groups):
