@@ -57,9 +57,10 @@ def engine_lib_path() -> Path:
     return LIB / f"_ksana_engine{suffix}"
 
 
-# kernel sources that a family needs in bf16 or fp32 on one GPU (no FP8 / FP4 / 4-bit weights, experts or peer memory)
+# kernel sources that a family needs in bf16 or fp32 on one GPU (no FP8 / FP4 / 4-bit weights or peer memory)
 _STREAM_KERNELS = ("attention_f32", "elementwise", "gemm_f32", "gemm_smallm", "gemm_tcgen05", "residual_stream", "sampler")
-FAMILY_KERNELS = {"lenolix": _STREAM_KERNELS + ("attention", "attention_tc"),
+FAMILY_KERNELS = {"fidevik": _STREAM_KERNELS + ("attention", "attention_tc", "mla_attention", "moe"),
+                  "lenolix": _STREAM_KERNELS + ("attention", "attention_tc"),
                   "rasizen": _STREAM_KERNELS + ("mla_attention", "recurrence")}
 
 

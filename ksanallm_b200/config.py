@@ -195,9 +195,10 @@ def load_yaml_config(path_or_dict) -> EngineConfig:
 # Descriptions of layers that are configured one by one (families whose config.json lists its layers)
 @dataclass
 class RotarySpec:
-    dims: int                             # leading dimensions of a head that rotate (halves: i with i + dims/2)
+    dims: int                             # leading dimensions of a head that rotate
     base: float
     scaling: Optional[dict] = None        # Hugging Face style rope_scaling dict
+    interleaved: bool = False             # pairs (2i, 2i + 1) instead of halves (i, i + dims/2)
 
 
 @dataclass
@@ -211,6 +212,7 @@ class AttentionSpec:
     keep_first: int = 0                   # first tokens that stay visible behind the window
     sink: bool = False                    # learned per-head logit in the softmax denominator
     rotary: Optional[RotarySpec] = None
+    qk_norm: bool = False                 # root-mean-square norm of all of q (and of k) at once, before the rotation
 
 
 @dataclass
@@ -227,13 +229,16 @@ class LatentAttentionSpec:
     dimensions and ``vdim`` value dimensions, a sigmoid gate on the output."""
     heads: int
     dim: int
-    rot_dim: int
+    rot_dim: int                          # 0: no rotated part
     vdim: int
     kv_rank: int                          # latent size
     scale: float
-    rotary: RotarySpec
+    rotary: Optional[RotarySpec] = None
     window: int = 0                       # sliding window in tokens, 0: full causal attention
     kv_from: Optional[int] = None         # layer whose cached latents are read; None: the layer's own
+    q_rank: int = 0                       # size of the normed latent that the queries go through; 0: straight from the input
+    sink: bool = False                    # learned per-head logit in the softmax denominator
+    head_gate: bool = False               # one gate per head instead of one per output element
 
 
 @dataclass
@@ -249,9 +254,36 @@ class PlainMlpSpec:
 
 
 @dataclass
+class GatedMlpSpec:
+    """down(act(gate) * up)."""
+    size: int
+    act: str = "silu"                     # silu | gelu (tanh form)
+
+
+@dataclass
+class RouterSpec:
+    experts: int
+    top: int
+    scoring: str = "softmax"              # softmax | sigmoid
+    renorm: bool = False                  # the chosen weights are divided by their sum
+    scale: float = 1.0
+    correction: bool = False              # learned per-expert offset that enters the choice, not the weights
+    groups: int = 1                       # equal groups of neighbouring experts ...
+    keep_groups: int = 1                  # ... of which the best by the sum of their two largest choice scores stay
+
+
+@dataclass
+class MoeSpec:
+    """Mixture of gated feed-forwards, and optionally one (``shared``) that every token goes through, with a gate."""
+    router: RouterSpec
+    expert: GatedMlpSpec
+    shared: Optional[GatedMlpSpec] = None
+
+
+@dataclass
 class LayerSpec:
     mixer: Union[AttentionSpec, LatentAttentionSpec, GatedRecurrenceSpec]
-    mlp: Optional[Union[MlpSpec, PlainMlpSpec]]
+    mlp: Optional[Union[MlpSpec, PlainMlpSpec, GatedMlpSpec, MoeSpec]]
 
 
 @dataclass
@@ -339,6 +371,7 @@ class ModelConfig:
     pair_embedding: Optional[PairEmbeddingSpec] = None
     norm_groups: int = 1                  # equal parts of a row that the norms treat one by one
     residual_mult: float = 1.0            # factor of every sublayer's result
+    logit_scale: float = 1.0
 
     @property
     def is_moe(self) -> bool:
@@ -353,9 +386,9 @@ _ARCH_ALIASES = {
     "llama": "llama", "mistral": "llama", "qwen2": "qwen", "qwen": "qwen", "qwen2_vl": "qwen2_vl", "baichuan": "baichuan",
     "chatglm": "chatglm", "glm": "chatglm", "gpt2": "gpt", "openai-gpt": "gpt", "fairseq-transformer": "gpt", "mixtral": "mixtral",
     "qwen2_moe": "qwen2_moe", "deepseek_v3": "deepseek_v3", "deepseek_v2": "deepseek_v3", "internlm2": "llama",
-    "yi": "llama", "lenolix": "lenolix", "rasizen": "rasizen",
+    "yi": "llama", "lenolix": "lenolix", "rasizen": "rasizen", "fidevik": "fidevik",
 }
-# No position limit is part of the Lenolix and Rasizen designs: the serving configuration's max_token_len decides
+# No position limit is part of the Lenolix, Rasizen and Fidevik designs: the serving configuration's max_token_len decides
 _UNBOUNDED_POSITIONS = 1 << 20
 
 
@@ -437,6 +470,8 @@ def model_config_from_hf(hf: dict, generation: Optional[dict] = None, model_dir:
         return lenolix_config(hf, generation)
     if arch == "rasizen":
         return rasizen_config(hf, generation)
+    if arch == "fidevik":
+        return fidevik_config(hf, generation)
     c = ModelConfig(model_type=arch, hf_model_type=mt)
     if arch == "gpt":
         c.hidden_size = hf.get("n_embd", hf.get("hidden_size", hf.get("decoder_embed_dim", 768)))
@@ -558,15 +593,7 @@ def _lenolix_attention(m: dict, where: str) -> AttentionSpec:
     mask = m.get("mask")
     if mask:
         a.window, a.keep_first = _positive(mask, "size", where + ".mask"), int(mask.get("keep_first", 0))
-    rot = m.get("rot")
-    if rot and int(rot["dims"]) > 0:
-        dims = int(rot["dims"])
-        if dims % 2 or dims > a.dim:
-            raise ValueError(f"{where}.rot.dims must be even and at most dim")
-        sc = rot.get("scaling")
-        a.rotary = RotarySpec(dims, float(rot["base"]), {
-            "rope_type": "llama3", "factor": float(sc["factor"]), "low_freq_factor": float(sc["low"]),
-            "high_freq_factor": float(sc["high"]), "original_max_position_embeddings": float(sc["original"])} if sc else None)
+    a.rotary = _rotary(m, where)
     return a
 
 
@@ -597,13 +624,32 @@ def lenolix_config(hf: dict, generation: Optional[dict] = None) -> ModelConfig:
     if emb.get("bigram"):
         b = emb["bigram"]
         c.pair_embedding = PairEmbeddingSpec(_positive(b, "buckets", "embedding.bigram"), int(b["mul_prev"]), int(b["mul_cur"]))
-    loop = hf.get("loop")
-    if loop:
-        c.loop = LoopSpec(int(loop["start"]), int(loop["stop"]), _positive(loop, "times", "loop"))
-        if not 0 <= c.loop.start < c.loop.stop <= len(layers):
-            raise ValueError("loop must cover at least one of the layers")
+    c.loop = _loop(hf, len(layers))
     c.eos_token_ids = _eos_ids(hf, generation)
     return c
+
+
+def _loop(hf: dict, layers: int) -> Optional[LoopSpec]:
+    d = hf.get("loop")
+    if not d:
+        return None
+    loop = LoopSpec(int(d["start"]), int(d["stop"]), _positive(d, "times", "loop"))
+    if not 0 <= loop.start < loop.stop <= layers:
+        raise ValueError("loop must cover at least one of the layers")
+    return loop
+
+
+def _rotary(m: dict, where: str, interleaved: bool = False) -> Optional[RotarySpec]:
+    rot = m.get("rot")
+    if not rot or int(rot["dims"]) <= 0:
+        return None
+    dims = int(rot["dims"])
+    if dims % 2 or dims > int(m["dim"]):
+        raise ValueError(f"{where}.rot.dims must be even and at most dim")
+    sc = rot.get("scaling")
+    return RotarySpec(dims, float(rot["base"]), {
+        "rope_type": "llama3", "factor": float(sc["factor"]), "low_freq_factor": float(sc["low"]),
+        "high_freq_factor": float(sc["high"]), "original_max_position_embeddings": float(sc["original"])} if sc else None, interleaved)
 
 
 def _latent_attention(m: dict, where: str) -> LatentAttentionSpec:
@@ -653,6 +699,63 @@ def rasizen_config(hf: dict, generation: Optional[dict] = None) -> ModelConfig:
                     norm_groups=int(hf["norm"].get("groups", 1)), residual_mult=float(hf.get("residual_mult", 1.0)))
     if c.norm_groups < 1 or c.hidden_size % c.norm_groups:
         raise ValueError(f"width {c.hidden_size} does not divide into {c.norm_groups} norm groups")
+    c.max_position_embeddings = c.max_token_len = int(hf.get("max_position_embeddings", _UNBOUNDED_POSITIONS))
+    c.eos_token_ids = _eos_ids(hf, generation)
+    return c
+
+
+def _gated_mlp(m: dict, where: str, act: str) -> GatedMlpSpec:
+    return GatedMlpSpec(_positive(m, "ff", where), act)
+
+
+def _moe(m: dict, where: str) -> MoeSpec:
+    r, at = m["router"], where + ".router"
+    groups = r.get("groups") or {"count": 1, "keep": 1}
+    router = RouterSpec(_positive(r, "experts", at), _positive(r, "top", at), scoring="sigmoid", correction=True,
+                        groups=_positive(groups, "count", at + ".groups"), keep_groups=_positive(groups, "keep", at + ".groups"))
+    if router.experts % router.groups or router.keep_groups > router.groups:
+        raise ValueError(f"{at}: {router.experts} experts, {router.keep_groups} of {router.groups} groups")
+    if router.top > router.experts // router.groups * router.keep_groups:
+        raise ValueError(f"{at}: {router.top} of the kept groups' experts cannot be chosen")
+    return MoeSpec(router, _gated_mlp(m["expert"], where + ".expert", "silu"),
+                   _gated_mlp(m["shared"], where + ".shared", "silu") if m.get("shared") else None)
+
+
+def fidevik_config(hf: dict, generation: Optional[dict] = None) -> ModelConfig:
+    """config.json of a Fidevik model: ``vocab``, ``width``, ``norm.eps``, ``logit_scale``, ``layers`` (``type``, ``mixer``,
+    ``mlp``) and ``loop``."""
+    layers = []
+    for i, e in enumerate(hf["layers"]):
+        where = f"layers[{i}]"
+        m, mlp, at = e["mixer"], e.get("mlp"), where + ".mixer"
+        if e["type"] == "attention":
+            mixer = AttentionSpec(*(_positive(m, k, at) for k in ("heads", "kv_heads", "dim", "vdim")), float(m["scale"]),
+                                  rotary=_rotary(m, at, interleaved=True), qk_norm=True)
+            if mixer.heads % mixer.kv_heads:
+                raise ValueError(f"{at}: heads must be a multiple of kv_heads")
+        elif e["type"] == "latent_attention":
+            mixer = LatentAttentionSpec(_positive(m, "heads", at), _positive(m, "dim", at), 0, _positive(m, "vdim", at),
+                                        _positive(m, "kv_rank", at), float(m["scale"]), q_rank=_positive(m, "q_rank", at), sink=True,
+                                        head_gate=True)
+        else:
+            raise ValueError(f"{where}: unknown mixer type {e['type']!r}")
+        if mlp and mlp.get("kind", "dense") not in ("dense", "moe"):
+            raise ValueError(f"{where}: unknown feed-forward kind {mlp['kind']!r}")
+        ff = None
+        if mlp:
+            ff = _moe(mlp, where + ".mlp") if mlp.get("kind") == "moe" else _gated_mlp(mlp, where + ".mlp", "gelu")
+        layers.append(LayerSpec(mixer, ff))
+    if not layers:
+        raise ValueError("layers is empty")
+    mixers = [s.mixer for s in layers]
+    heads = math.gcd(*(a.heads for a in mixers))             # what tensor parallelism splits
+    kv = math.gcd(*(a.kv_heads if isinstance(a, AttentionSpec) else a.heads for a in mixers))
+    c = ModelConfig(model_type="fidevik", hf_model_type="fidevik", hidden_size=_positive(hf, "width", "config"), num_layers=len(layers),
+                    num_heads=heads, num_kv_heads=math.gcd(heads, kv), head_dim=mixers[0].dim, v_head_dim=mixers[0].vdim,
+                    intermediate_size=max([s.mlp.size for s in layers if isinstance(s.mlp, GatedMlpSpec)] or [0]),
+                    vocab_size=_positive(hf, "vocab", "config"), rms_norm_eps=float(hf["norm"]["eps"]), norm_type="layernorm",
+                    position_embedding="per_layer", layer_specs=layers, logit_scale=float(hf.get("logit_scale", 1.0)))
+    c.loop = _loop(hf, len(layers))
     c.max_position_embeddings = c.max_token_len = int(hf.get("max_position_embeddings", _UNBOUNDED_POSITIONS))
     c.eos_token_ids = _eos_ids(hf, generation)
     return c

@@ -176,12 +176,16 @@ __device__ __forceinline__ float tanh_fast(float x) {
   asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// 0.5 x (1 + tanh(c)) = x / (1 + exp(-2 c)) with c = sqrt(2 / pi) (x + 0.044715 x^3): no cancellation where tanh is near -1
+__device__ __forceinline__ float gelu_tanh(float x) {
+  return x / (1.f + __expf(-1.5957691216f * (x + 0.044715f * x * x * x)));
+}
 __device__ __forceinline__ float act_fn(float x, int act) {
   // silu(x) = x * sigmoid(x) = 0.5 x (1 + tanh(x / 2)): one special-function op per element instead of an
   // exponential and a division (the special-function unit, not memory, paced this kernel); the approximation's
   // error (about 2^-11) is below the bf16 rounding of the result
   if (act == 0) { const float hx = 0.5f * x; return fmaf(hx, tanh_fast(hx), hx); }
-  if (act == 1) return 0.5f * x * (1.f + tanhf(0.7978845608f * (x + 0.044715f * x * x * x)));
+  if (act == 1) return gelu_tanh(x);
   return fmaxf(x, 0.f);
 }
 
@@ -227,6 +231,21 @@ __global__ void act_mul_kernel(const bf16* __restrict__ in, bf16* __restrict__ o
         if ((i & 15) == 0) oscale[static_cast<size_t>(i >> 4) * scale_ld + m] = scale;
       }
     }
+  }
+}
+
+// The same on fp32 rows, with the exponential instead of the approximate tanh.
+__global__ void act_mul_f32_kernel(const float* __restrict__ in, float* __restrict__ out, int M, int I, int in_ld, int act, int gated) {
+  pdl_trigger();
+  pdl_wait();
+  const long long total = static_cast<long long>(M) * I;
+  for (long long idx = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; idx < total;
+       idx += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long m = idx / I, i = idx - m * I;
+    const float* row = in + m * in_ld;
+    const float g = row[i];
+    const float a = act == 0 ? g / (1.f + __expf(-g)) : act == 1 ? gelu_tanh(g) : fmaxf(g, 0.f);
+    out[idx] = gated ? a * row[I + i] : a;
   }
 }
 
@@ -663,6 +682,13 @@ extern "C" int ksana_act_mul(const void* in, void* out, void* outq, float* oscal
   launch_pdl(act_mul_kernel, dim3(grid_for(total, 256)), dim3(256), 0, st, (const bf16*)in, (bf16*)out, (uint8_t*)outq, oscale, scale_ld, M,
                                                        I, in_ld, act, gated);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+extern "C" int ksana_act_mul_f32(const float* in, float* out, int M, int I, int in_ld, int act, int gated, cudaStream_t st) {
+  if (M <= 0 || I <= 0) return 0;
+  if (in_ld < I * (gated ? 2 : 1) || act < 0 || act > 2) return -10;
+  return launch_pdl(act_mul_f32_kernel, dim3(grid_for(static_cast<long long>(M) * I, 256)), dim3(256), 0, st, in, out, M, I, in_ld, act,
+                    gated) == cudaSuccess ? 0 : -4;
 }
 
 extern "C" int ksana_quant_fp8(const void* x, void* q, float* scale, int scale_ld, int M, int K, int x_ld,

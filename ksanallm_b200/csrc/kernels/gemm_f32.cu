@@ -11,9 +11,15 @@ constexpr int kSgTile = 64, kSgK = 16, kSgThreads = 256;
 __global__ void __launch_bounds__(kSgThreads)
 gemm_f32_kernel(const float* __restrict__ A, int lda, const float* __restrict__ W, int ldw, float* __restrict__ D, int ldd,
                 const float* __restrict__ bias, const float* __restrict__ residual, int ldr, int M, int N, int K,
-                long long a_batch, long long w_batch, long long d_batch, const float* __restrict__ gate, int ldg, long long g_batch) {
+                long long a_batch, long long w_batch, long long d_batch, const float* __restrict__ gate, int ldg, long long g_batch,
+                const int* __restrict__ tile_expert, int num_experts) {
   pdl_trigger();
   pdl_wait();
+  if (tile_expert) {                    // rows of one expert per 128-row tile; W stacks the experts' N rows
+    const int e = tile_expert[blockIdx.y * kSgTile / 128];
+    if (e < 0 || e >= num_experts) return;
+    W += static_cast<size_t>(e) * N * ldw;
+  }
   A += blockIdx.z * a_batch;
   W += blockIdx.z * w_batch;
   D += blockIdx.z * d_batch;
@@ -70,7 +76,7 @@ extern "C" int ksana_gemm_f32(const float* A, int lda, const float* W, int ldw, 
   const dim3 grid((N + kSgTile - 1) / kSgTile, (M + kSgTile - 1) / kSgTile);
   if (grid.y > 65535u) return -10;
   return launch_pdl(gemm_f32_kernel, grid, dim3(kSgThreads), 0, st, A, lda, W, ldw, D, ldd, bias, residual, ldr, M, N, K,
-                    0LL, 0LL, 0LL, static_cast<const float*>(nullptr), 0, 0LL) == cudaSuccess ? 0 : -4;
+                    0LL, 0LL, 0LL, static_cast<const float*>(nullptr), 0, 0LL, static_cast<const int*>(nullptr), 0) == cudaSuccess ? 0 : -4;
 }
 
 // D[b] = A[b] W[b]^T for every b, with a gate times sigmoid(gate[b]) element by element; a_batch / w_batch / d_batch: elements between batch entries.
@@ -82,5 +88,16 @@ extern "C" int ksana_gemm_f32_batched(const float* A, int lda, long long a_batch
   if (grid.y > 65535u || batch > 65535) return -10;
   const float* none = nullptr;
   return launch_pdl(gemm_f32_kernel, grid, dim3(kSgThreads), 0, st, A, lda, W, ldw, D, ldd, none, none, 0, M, N, K, a_batch, w_batch,
-                    d_batch, gate, ldg, g_batch) == cudaSuccess ? 0 : -4;
+                    d_batch, gate, ldg, g_batch, static_cast<const int*>(nullptr), 0) == cudaSuccess ? 0 : -4;
+}
+
+// Mixture of experts: 128-row tiles of A, tile i times W[tile_expert[i]] (W [E * N, K]; a negative entry: an unused tile).
+extern "C" int ksana_gemm_grouped_f32(const float* A, int lda, const float* W, int ldw, float* D, int ldd, int M_cap, int N, int K,
+                                      int E, const int* tile_expert, cudaStream_t st) {
+  if (M_cap <= 0 || N <= 0 || K <= 0 || E <= 0) return 0;
+  if (M_cap % 128 || !tile_expert || M_cap / kSgTile > 65535) return -10;
+  const dim3 grid((N + kSgTile - 1) / kSgTile, M_cap / kSgTile);
+  const float* none = nullptr;
+  return launch_pdl(gemm_f32_kernel, grid, dim3(kSgThreads), 0, st, A, lda, W, ldw, D, ldd, none, none, 0, M_cap, N, K, 0LL, 0LL, 0LL,
+                    none, 0, 0LL, tile_expert, E) == cudaSuccess ? 0 : -4;
 }

@@ -1,5 +1,6 @@
 // Multi-head latent attention ("absorbed" form) on the tcgen05 tensor cores, prefill and decode, over the paged latent
-// cache, with an optional sliding window. The reference has no MLA (its attention layers are flash-attention + vLLM paged
+// cache, with an optional sliding window, per-head sink logits (a share of the softmax denominator without a key) and a gate
+// per query row and head. The reference has no MLA (its attention layers are flash-attention + vLLM paged
 // attention over per-head K/V: src/ksana_llm/layers/nvidia/flash_attention_layer.cpp, paged_attention_layer.cpp);
 // this file is new work.
 //
@@ -35,6 +36,7 @@
 #include "pdl.cuh"
 #include "vec8.cuh"
 #include <math_constants.h>
+#include <type_traits>
 
 namespace ksana {
 
@@ -66,6 +68,8 @@ struct MlaParams {
   int rows_per_block;                         // cache rows between consecutive blocks (a 2-D map); 0: not whole rows, 3-D map
   int window;                                 // keys a query sees, itself included; 0: all earlier ones
   int num_blocks;                             // blocks addressable from the layer base (block-table entries are checked)
+  const float* sinks;                         // [G], null: none
+  const bf16* gate; long long gate_ld;        // [T][gate_ld], null: none; a head's output is multiplied by sigmoid(gate)
   float scale_log2;
   int* err;
 };
@@ -74,6 +78,16 @@ __device__ __forceinline__ float mla_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+
+// Factor of a row's unnormalised output: 1 / (sum of weights + the sink's), times the gate. m: the running maximum that the
+// weights refer to (base 2).
+__device__ __forceinline__ float mla_out_factor(float l, float m, const float* sinks, const bf16* gate, long long gate_ld, int row,
+                                                int head) {
+  if (sinks) l += exp2f(sinks[head] * 1.44269504f - m);
+  float f = l > 0.f ? 1.f / l : 0.f;
+  if (gate) f *= sigmoid_f(to_f(gate[static_cast<size_t>(row) * gate_ld + head]));
+  return f;
 }
 
 // PANELS: 64-column panels of a row. FLAT: the cache blocks are whole rows apart (a 2-D map serves them). WINDOW: with a
@@ -390,7 +404,7 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
     if (ok && mbar_wait(o_full, 0, abort_flag)) {
       tc_fence_after();
       if (p.nsplit == 1) {
-        const float inv = l > 0.f ? 1.f / l : 0.f;
+        const float inv = active ? mla_out_factor(l, m_used, p.sinks, p.gate, p.gate_ld, q0 + tok, head) : 0.f;
         bf16* dst = p.out + static_cast<size_t>(q0 + tok) * p.out_tok_stride + head * p.dv + half * 256;
 #pragma unroll 1
         for (int c = 0; c * 32 < cols; ++c) {
@@ -442,9 +456,11 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
   if (warp == 1) { tc_fence_after(); tmem_dealloc(tmem_base, kMlaTmemCols); }
 }
 
-// Merge of split-KV partials: out[row] = sum_s 2^(m_s - m) O_s / sum_s 2^(m_s - m) l_s. One CTA per (token, head).
+// Merge of split-KV partials: out[row] = sum_s 2^(m_s - m) O_s / sum_s 2^(m_s - m) l_s, with the sink in the denominator and
+// the gate. One CTA per (token, head).
 __global__ void mla_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, bf16* __restrict__ out,
-                                 long long out_tok_stride, int T, int G, int nsplit, int dv) {
+                                 long long out_tok_stride, int T, int G, int nsplit, int dv, const float* __restrict__ sinks,
+                                 const bf16* __restrict__ gate, long long gate_ld) {
   if (threadIdx.x * 4 >= dv) return;
   const int row = blockIdx.x, tok = row / G, head = row % G;
   const size_t rows = static_cast<size_t>(T) * G;
@@ -463,7 +479,7 @@ __global__ void mla_merge_kernel(const float* __restrict__ part_o, const float* 
     const float4 o = *reinterpret_cast<const float4*>(part_o + (s * rows + row) * dv + threadIdx.x * 4);
     acc.x += w * o.x; acc.y += w * o.y; acc.z += w * o.z; acc.w += w * o.w;
   }
-  const float inv = denom > 0.f ? 1.f / denom : 0.f;
+  const float inv = denom > 0.f ? mla_out_factor(denom, m, sinks, gate, gate_ld, tok, head) : 0.f;
   __nv_bfloat162 lo = __floats2bfloat162_rn(acc.x * inv, acc.y * inv), hi = __floats2bfloat162_rn(acc.z * inv, acc.w * inv);
   uint2 v;
   v.x = *reinterpret_cast<uint32_t*>(&lo);
@@ -606,14 +622,14 @@ using namespace ksana;
 //   out    [T, G, dv] bf16, out_tok_stride elements between tokens
 //   cache  layer base of [block][block_tokens][dk] bf16, blocks block_stride elements apart, num_blocks of them
 // Sequences: cu_q [B+1], kv_lens [B] (KV length including this step's rows), block_table [B][table_stride].
-// window > 0: a query sees itself and the window - 1 tokens before it.
+// window > 0: a query sees itself and the window - 1 tokens before it. sinks [G] fp32 and gate [T][gate_ld] bf16 may be null.
 // nsplit > 1 needs part_o [nsplit*T*G*dv] and part_ml [nsplit*T*G*2] fp32.
 // Returns 0 when launched, -100 when the configuration is not covered (the caller uses its own fallback).
 extern "C" int ksana_mla_attention(const void* q, long long T, void* out, long long out_tok_stride, const void* cache,
                                    long long block_stride, int block_tokens, const int* block_table, int table_stride,
                                    const int* cu_q, const int* kv_lens, int B, int max_q_len, int G, int dk, int dv, int window,
-                                   float scale, int num_blocks, int nsplit, float* part_o, float* part_ml, int* err,
-                                   cudaStream_t st) {
+                                   const float* sinks, const void* gate, long long gate_ld, float scale, int num_blocks,
+                                   int nsplit, float* part_o, float* part_ml, int* err, cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0) return 0;
   const int bt = block_tokens;
   if (G <= 0 || dk <= 0 || dv <= 0 || dk % 8 || dv % 8 || dv > dk || dk > kMlaMaxDk || dv > kMlaMaxDv || window < 0) return -100;
@@ -661,8 +677,9 @@ extern "C" int ksana_mla_attention(const void* q, long long T, void* out, long l
   p.part_o = part_o; p.part_ml = part_ml;
   p.block_table = block_table; p.table_stride = table_stride; p.cu_q = cu_q; p.kv_lens = kv_lens;
   p.G = G; p.block_tokens = bt; p.box_rows = box_rows; p.nsplit = nsplit; p.T = static_cast<int>(T);
-  p.dv = dv; p.window = window > 0 ? window : 1 << 30; p.rows_per_block = flat ? static_cast<int>(block_stride / dk) : 0;
+  p.dv = dv; p.window = window; p.rows_per_block = flat ? static_cast<int>(block_stride / dk) : 0;
   p.num_blocks = num_blocks;
+  p.sinks = sinks; p.gate = static_cast<const bf16*>(gate); p.gate_ld = gate_ld;
   p.scale_log2 = scale * 1.44269504f;
   p.err = err;
   const int nqt = (max_q_len * G + kMlaM - 1) / kMlaM;
@@ -672,22 +689,28 @@ extern "C" int ksana_mla_attention(const void* q, long long T, void* out, long l
   if (flat) {
     rc = launch_mla<9, true, false>(grid, q_map, kv_map, p, st);
   } else {
+    auto go = [&](auto n) {
+      constexpr int kPanels = decltype(n)::value;
+      return window > 0 ? launch_mla<kPanels, false, true>(grid, q_map, kv_map, p, st)
+                        : launch_mla<kPanels, false, false>(grid, q_map, kv_map, p, st);
+    };
     switch (panels) {
-      case 1: rc = launch_mla<1, false, true>(grid, q_map, kv_map, p, st); break;
-      case 2: rc = launch_mla<2, false, true>(grid, q_map, kv_map, p, st); break;
-      case 3: rc = launch_mla<3, false, true>(grid, q_map, kv_map, p, st); break;
-      case 4: rc = launch_mla<4, false, true>(grid, q_map, kv_map, p, st); break;
-      case 5: rc = launch_mla<5, false, true>(grid, q_map, kv_map, p, st); break;
-      case 6: rc = launch_mla<6, false, true>(grid, q_map, kv_map, p, st); break;
-      case 7: rc = launch_mla<7, false, true>(grid, q_map, kv_map, p, st); break;
-      case 8: rc = launch_mla<8, false, true>(grid, q_map, kv_map, p, st); break;
-      case 9: rc = launch_mla<9, false, true>(grid, q_map, kv_map, p, st); break;
+      case 1: rc = go(std::integral_constant<int, 1>()); break;
+      case 2: rc = go(std::integral_constant<int, 2>()); break;
+      case 3: rc = go(std::integral_constant<int, 3>()); break;
+      case 4: rc = go(std::integral_constant<int, 4>()); break;
+      case 5: rc = go(std::integral_constant<int, 5>()); break;
+      case 6: rc = go(std::integral_constant<int, 6>()); break;
+      case 7: rc = go(std::integral_constant<int, 7>()); break;
+      case 8: rc = go(std::integral_constant<int, 8>()); break;
+      case 9: rc = go(std::integral_constant<int, 9>()); break;
     }
   }
   if (rc) return rc;
   if (nsplit > 1) {
     mla_merge_kernel<<<static_cast<unsigned>(T) * G, (dv / 4 + 31) / 32 * 32, 0, st>>>(
-        part_o, part_ml, static_cast<bf16*>(out), out_tok_stride, static_cast<int>(T), G, nsplit, dv);
+        part_o, part_ml, static_cast<bf16*>(out), out_tok_stride, static_cast<int>(T), G, nsplit, dv, sinks,
+        static_cast<const bf16*>(gate), gate_ld);
     if (cudaGetLastError() != cudaSuccess) return -4;
   }
   return 0;

@@ -22,14 +22,15 @@ namespace ksana {
 
 typedef __nv_bfloat16 bf16;
 constexpr int kMaxExperts = 512;
-constexpr int kMaxTopK = 16;
+constexpr int kMaxTopK = 64;
 
 // One warp per token. scoring 0 = softmax over all experts, 1 = sigmoid. `bias` (may be null) is added
 // for SELECTION only (DeepSeek-V3 e_score_correction_bias). n_group/topk_group: keep only the best
-// topk_group groups (group score = sum of its two largest biased scores).
-__global__ void moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias,
-                                 int* __restrict__ topk_ids, float* __restrict__ topk_w, int T, int E, int K,
-                                 int scoring, int renorm, float scale, int n_group, int topk_group) {
+// topk_group groups (group score = sum of its two largest biased scores). Logit rows are ldl apart, weight rows
+// ldw; with `gate_col` >= 0 the sigmoid of that logit column (a shared expert's gate) is a row's weight number K.
+__global__ void moe_route_kernel(const float* __restrict__ logits, int ldl, const float* __restrict__ bias,
+                                 int* __restrict__ topk_ids, float* __restrict__ topk_w, int ldw, int T, int E, int K,
+                                 int scoring, int renorm, float scale, int n_group, int topk_group, int gate_col) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
   if (warp >= T) return;
@@ -37,7 +38,8 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
   __shared__ float s_sel[8][kMaxExperts];
   float* score = s_score[(threadIdx.x >> 5)];
   float* sel = s_sel[(threadIdx.x >> 5)];
-  const float* row = logits + static_cast<size_t>(warp) * E;
+  const float* row = logits + static_cast<size_t>(warp) * ldl;
+  topk_w += static_cast<size_t>(warp) * ldw;
   float mx = -INFINITY;
   for (int e = lane; e < E; e += 32) mx = fmaxf(mx, row[e]);
   for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -56,26 +58,26 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
   __syncwarp();
   if (n_group > 1 && topk_group < n_group) {
     const int gs = E / n_group;
-    // lane g (< n_group <= 32) scores its group
-    float gscore = -INFINITY;
-    if (lane < n_group) {
+    // lane l owns the groups l, l + 32, ...; a group's score goes to where its members' are hidden afterwards
+    __shared__ float s_group[8][kMaxExperts];
+    float* gsc = s_group[threadIdx.x >> 5];
+    for (int g = lane; g < n_group; g += 32) {
       float a = -INFINITY, b = -INFINITY;
       for (int i = 0; i < gs; ++i) {
-        const float v = sel[lane * gs + i];
+        const float v = sel[g * gs + i];
         if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
       }
-      gscore = a + b;
+      gsc[g] = gs > 1 ? a + b : a;
     }
-    // keep the topk_group best groups: a group survives if fewer than topk_group groups beat it
-    int better = 0;
-    for (int g = 0; g < n_group; ++g) {
-      const float og = __shfl_sync(0xffffffffu, gscore, g);
-      if (og > gscore || (og == gscore && g < lane)) ++better;
+    __syncwarp();
+    // a group survives if fewer than topk_group groups beat it (of equal ones the first)
+    for (int g = lane; g < n_group; g += 32) {
+      const float mine = gsc[g];
+      int better = 0;
+      for (int o = 0; o < n_group; ++o) better += gsc[o] > mine || (gsc[o] == mine && o < g);
+      if (better >= topk_group)
+        for (int i = 0; i < gs; ++i) sel[g * gs + i] = -INFINITY;
     }
-    const bool keep = lane < n_group && better < topk_group;
-    const unsigned mask = __ballot_sync(0xffffffffu, keep);
-    for (int e = lane; e < E; e += 32)
-      if (!((mask >> (e / gs)) & 1u)) sel[e] = -INFINITY;
     __syncwarp();
   }
   float wsum = 0.f;
@@ -94,7 +96,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
     const float w = score[bi];
     if (lane == 0) {
       topk_ids[static_cast<size_t>(warp) * K + k] = bi;
-      topk_w[static_cast<size_t>(warp) * K + k] = w;
+      topk_w[k] = w;
       sel[bi] = -INFINITY;
     }
     wsum += w;
@@ -102,7 +104,9 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
   }
   if (lane == 0) {
     const float f = (renorm ? 1.f / fmaxf(wsum, 1e-20f) : 1.f) * scale;
-    for (int k = 0; k < K; ++k) topk_w[static_cast<size_t>(warp) * K + k] *= f;
+    if (f != 1.f)
+      for (int k = 0; k < K; ++k) topk_w[k] *= f;
+    if (gate_col >= 0) topk_w[K] = 1.f / (1.f + __expf(-row[gate_col]));
   }
 }
 
@@ -207,12 +211,14 @@ __global__ void moe_combine_kernel(const bf16* __restrict__ y, const int* __rest
 
 using namespace ksana;
 
-extern "C" int ksana_moe_route(const float* logits, const float* bias, int* topk_ids, float* topk_w, int T, int E, int K,
-                               int scoring, int renorm, float scale, int n_group, int topk_group, cudaStream_t st) {
+extern "C" int ksana_moe_route(const float* logits, int ldl, const float* bias, int* topk_ids, float* topk_w, int ldw, int T,
+                               int E, int K, int scoring, int renorm, float scale, int n_group, int topk_group, int gate_col,
+                               cudaStream_t st) {
   if (T <= 0) return 0;
-  if (E > kMaxExperts || K > kMaxTopK || n_group > 32 || (n_group > 1 && E % n_group)) return -10;
-  moe_route_kernel<<<(T + 7) / 8, 256, 0, st>>>(logits, bias, topk_ids, topk_w, T, E, K, scoring, renorm, scale,
-                                                n_group, topk_group);
+  if (E > kMaxExperts || K > kMaxTopK || K > E || n_group > E || (n_group > 1 && E % n_group)) return -10;
+  if (ldl < E || gate_col >= ldl || ldw < K + (gate_col >= 0)) return -11;
+  moe_route_kernel<<<(T + 7) / 8, 256, 0, st>>>(logits, ldl, bias, topk_ids, topk_w, ldw, T, E, K, scoring, renorm, scale,
+                                                n_group, topk_group, gate_col);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

@@ -5,11 +5,15 @@
 //   embed_pair        x = table[id] * scale (+ pair[hash(previous id, id)]), fp32, plus an optional copy in T
 //   residual_norm     x += scale * norm(y) ; z = norm(x)  - one pass for "norm after the sublayer, layer scale, residual
 //                     add, norm before the next sublayer"; every part is optional (a plain norm, a cast, a row gather)
-//                     The addend may have a scalar factor, and the stream's norm may be taken per part of a row
+//                     The addend may have a scalar factor, and the stream's norm may be taken per part of a row. It may be
+//                     the weighted sum of a token's expert outputs, gathered here; other stream rows (the embedding output,
+//                     say) and a vector may be added as well
 //   glu_clamp         min(g, limit) * sigmoid(alpha * g) * (clamp(u, -limit, limit) + offset)
 //   xielu             pos z^2 + lin z (z > 0), neg (exp(z) - 1 - z) + lin z (z <= 0)
 //   qkv_rope_append   rotary embedding on the first rot dims of q and k, k and v into the paged cache; k and v may have
 //                     different head sizes and live in separate panels
+//   qkv_norm_rope_append   the same with a norm over all of q and over all of k first, and rotated pairs (2i, 2i + 1)
+//   latent_norms      the norms of a row's query latent (to a buffer) and key/value latent (to the paged cache)
 //   refit_rows_f32    rows of x overwritten with given embeddings
 #include "guards.cuh"
 #include "pdl.cuh"
@@ -106,8 +110,15 @@ struct ResNormParams {
   int rms;                              // 1: root-mean-square norms (no mean, no bias needed)
   float alpha;                          // factor of the addend, all columns
   int groups;                           // > 1: the stream's norm takes its mean square per consecutive part of H / groups columns
+  const float* add; const T* vec;       // optional: stream rows (ldx apart) and a vector that are added too
+  float z_scale;                        // factor of the normed row
+  // addend = sum over k < top of w[row][k] * y[dst_row[row][k]] (+ w[row][top] * shared[row]); rows of `ldw` weights. A
+  // negative dst_row is an expert that lives elsewhere
+  const int* dst_row; const float* w; int ldw, top, cap;
+  const T* shared; int lds;
   int* err;
 };
+constexpr int kMaxTop = 64;
 
 // z = the row v scaled by the reciprocal root mean square of each of its `groups` parts of equal size, times w2. Squares are
 // summed per unit (a vector of 8, or a single element where a part is not a multiple of 8) in dynamic shared memory, one
@@ -159,13 +170,25 @@ __device__ __forceinline__ void grouped_norm(const ResNormParams<T>& p, int m, f
   }
 }
 
-// One CTA per row, VPT vectors of 8 elements per thread.
-template <typename T, int VPT>
+// One CTA per row, VPT vectors of 8 elements per thread. EXPERTS: the addend is gathered from expert outputs.
+template <typename T, int VPT, bool EXPERTS>
 __global__ void residual_norm_kernel(const ResNormParams<T> p) {
   pdl_trigger();
   pdl_wait();
   __shared__ Moments red[2][32];
+  __shared__ int src_row[EXPERTS ? kMaxTop : 1];
+  __shared__ float src_w[EXPERTS ? kMaxTop + 1 : 1];
   const int m = blockIdx.x;
+  if (EXPERTS) {
+    for (int k = threadIdx.x; k < p.top; k += blockDim.x) {
+      int d = p.dst_row[static_cast<size_t>(m) * p.top + k];
+      if (d >= p.cap) { guard_report(p.err, kGuardDstRow, d); d = -1; }
+      src_row[k] = d;
+      src_w[k] = p.w[static_cast<size_t>(m) * p.ldw + k];
+    }
+    if (threadIdx.x == 0 && p.shared) src_w[p.top] = p.w[static_cast<size_t>(m) * p.ldw + p.top];
+    __syncthreads();
+  }
   int r = m;
   if (p.rows) {
     r = p.rows[m];
@@ -178,7 +201,25 @@ __global__ void residual_norm_kernel(const ResNormParams<T> p) {
     const int i = threadIdx.x + j * blockDim.x;
     if (i < nvec) {
       load8(p.x + static_cast<size_t>(r) * p.ldx + i * 8, v[j]);
-      if (p.y) load8(p.y + static_cast<size_t>(r) * p.ldy + i * 8, y[j]);
+      if (EXPERTS) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[j][e] = 0.f;
+        if (p.shared) {
+          load8(p.shared + static_cast<size_t>(r) * p.lds + i * 8, y[j]);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) y[j][e] *= src_w[p.top];
+        }
+#pragma unroll 4
+        for (int k = 0; k < p.top; ++k) {
+          if (src_row[k] < 0) continue;
+          float f[8];
+          load8(p.y + static_cast<size_t>(src_row[k]) * p.ldy + i * 8, f);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) y[j][e] = fmaf(src_w[k], f[e], y[j][e]);
+        }
+      } else if (p.y) {
+        load8(p.y + static_cast<size_t>(r) * p.ldy + i * 8, y[j]);
+      }
     }
   }
   // statistics of the valid elements of f: (n, mean, m2), or for RMS (n, 0, sum of squares)
@@ -243,6 +284,25 @@ __global__ void residual_norm_kernel(const ResNormParams<T> p) {
       }
     }
   }
+  if (p.add || p.vec) {                 // pad columns of both are zero
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+      const int i = threadIdx.x + j * blockDim.x;
+      if (i < nvec) {
+        float f[8];
+        if (p.add) {
+          load8(p.add + static_cast<size_t>(r) * p.ldx + i * 8, f);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) v[j][e] += f[e];
+        }
+        if (p.vec) {
+          load8(p.vec + i * 8, f);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) v[j][e] += f[e];
+        }
+      }
+    }
+  }
   if (p.x_out) {
 #pragma unroll
     for (int j = 0; j < VPT; ++j) {
@@ -271,6 +331,8 @@ __global__ void residual_norm_kernel(const ResNormParams<T> p) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) v[j][e] = e < k ? v[j][e] : 0.f;
       }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[j][e] *= p.z_scale;
       store8(p.z + static_cast<size_t>(m) * p.ldz + i * 8, v[j]);
     }
   }
@@ -287,9 +349,12 @@ static int launch_residual_norm(const ResNormParams<T>& p, int M, cudaStream_t s
     if (smem > 46 * 1024) return -10;
   }
   cudaError_t e;
-  if (nvec <= 256) e = launch_pdl(residual_norm_kernel<T, 1>, dim3(M), dim3(threads(1)), smem, st, p);
-  else if (nvec <= 1024) e = launch_pdl(residual_norm_kernel<T, 2>, dim3(M), dim3(threads(2)), smem, st, p);
-  else if (nvec <= 4096) e = launch_pdl(residual_norm_kernel<T, 4>, dim3(M), dim3(threads(4)), smem, st, p);
+  auto launch = [&](auto* plain, auto* experts, int vpt) {
+    return launch_pdl(p.dst_row ? experts : plain, dim3(M), dim3(threads(vpt)), smem, st, p);
+  };
+  if (nvec <= 256) e = launch(residual_norm_kernel<T, 1, false>, residual_norm_kernel<T, 1, true>, 1);
+  else if (nvec <= 1024) e = launch(residual_norm_kernel<T, 2, false>, residual_norm_kernel<T, 2, true>, 2);
+  else if (nvec <= 4096) e = launch(residual_norm_kernel<T, 4, false>, residual_norm_kernel<T, 4, true>, 4);
   else return -10;
   return e == cudaSuccess ? 0 : -4;
 }
@@ -416,6 +481,189 @@ __global__ void qkv_rope_append_kernel(T* __restrict__ qkv, const int* __restric
   }
 }
 
+// q and k normed by the root mean square of all of q's (k's) columns at once, pairs (2i, 2i + 1) of the first `rot` dimensions
+// of a head rotated, k and v into the paged cache (layout as above), q in place. One CTA per token, VPT vectors of q | k per
+// thread in registers between the reduction and the rotation. Pad columns (head sizes that are not multiples of 8) are zero
+// and have zero weights. sums: optional [T, 2] sums of squares of the whole q and k rows where this rank holds a part of them.
+template <typename T>
+struct NormRopeParams {
+  T* qkv;
+  const int* positions; const int* slots;
+  const float* cos_sin; int max_pos;
+  const T* qw; const T* kw; float eps;
+  int nq, nk;                           // real columns of the whole q and k
+  const float* sums;
+  T* kc; T* vc; long long block_stride;
+  int block_tokens, num_blocks, Hq, Hkv, D, Dv, rot;
+  int* err;
+};
+
+template <typename T, int VPT>
+__global__ void qkv_norm_rope_append_kernel(const NormRopeParams<T> p) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float red[2][32];
+  const int t = blockIdx.x, D = p.D, Dv = p.Dv;
+  T* row = p.qkv + static_cast<size_t>(t) * ((p.Hq + p.Hkv) * D + p.Hkv * Dv);
+  int pos = p.rot ? p.positions[t] : 0;
+  if (pos < 0 || (p.rot && pos >= p.max_pos)) { if (threadIdx.x == 0) guard_report(p.err, kGuardPosition, pos); pos = 0; }
+  int slot = p.slots[t];
+  if (slot >= 0 && slot / p.block_tokens >= p.num_blocks) { if (threadIdx.x == 0) guard_report(p.err, kGuardSlot, slot); slot = -1; }
+  const int blk = slot < 0 ? 0 : slot / p.block_tokens, off = slot < 0 ? 0 : slot - blk * p.block_tokens;
+  T* kdst = p.kc + static_cast<size_t>(blk) * p.block_stride + static_cast<size_t>(off) * D;
+  T* vdst = p.vc + static_cast<size_t>(blk) * p.block_stride + static_cast<size_t>(off) * Dv;
+  const size_t kh = static_cast<size_t>(p.block_tokens) * D, vh = static_cast<size_t>(p.block_tokens) * Dv;
+  const int half = p.rot >> 1, d8 = D >> 3, dv8 = Dv >> 3;
+  const int nqv = p.Hq * d8, nv = nqv + p.Hkv * d8;
+  float f[VPT][8], sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int j = 0; j < VPT; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i < nv) {
+      load8(row + static_cast<size_t>(i) * 8, f[j]);
+      float s = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) s = fmaf(f[j][e], f[j][e], s);
+      if (i < nqv) sq += s; else sk += s;
+    }
+  }
+  // v needs neither: its copies are in flight during the reduction
+  if (slot >= 0) {
+    for (int i = threadIdx.x; i < p.Hkv * dv8; i += blockDim.x) {
+      const int h = i / dv8, j = (i - h * dv8) * 8;
+      float a[8];
+      load8(row + static_cast<size_t>(p.Hq + p.Hkv) * D + h * Dv + j, a);
+      store8(vdst + h * vh + j, a);
+    }
+  }
+  if (p.sums) {
+    sq = p.sums[2 * t];
+    sk = p.sums[2 * t + 1];
+  } else {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      sq += __shfl_xor_sync(0xffffffffu, sq, o);
+      sk += __shfl_xor_sync(0xffffffffu, sk, o);
+    }
+    if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = sq; red[1][threadIdx.x >> 5] = sk; }
+    __syncthreads();
+    sq = sk = 0.f;
+    for (int w = 0; w < static_cast<int>(blockDim.x >> 5); ++w) { sq += red[0][w]; sk += red[1][w]; }
+  }
+  const float rq = rsqrtf(sq / static_cast<float>(p.nq) + p.eps), rk = rsqrtf(sk / static_cast<float>(p.nk) + p.eps);
+  const float* cs = p.cos_sin + static_cast<size_t>(pos) * p.rot;
+#pragma unroll
+  for (int j = 0; j < VPT; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i < nv && (i < nqv || slot >= 0)) {
+      float w[8];
+      load8(i < nqv ? p.qw + static_cast<size_t>(i) * 8 : p.kw + static_cast<size_t>(i - nqv) * 8, w);
+      const float r = i < nqv ? rq : rk;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[j][e] *= r * w[e];
+      const int h = i / d8, c = (i - h * d8) * 8;
+      if (c < p.rot) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int pr = (c >> 1) + e;
+          if (pr < half) {
+            const float co = cs[pr], si = cs[half + pr], u = f[j][2 * e], v = f[j][2 * e + 1];
+            f[j][2 * e] = u * co - v * si;
+            f[j][2 * e + 1] = v * co + u * si;
+          }
+        }
+      }
+      store8(i < nqv ? row + static_cast<size_t>(i) * 8 : kdst + (h - p.Hq) * kh + c, f[j]);
+    }
+  }
+}
+
+template <typename T>
+static cudaError_t launch_norm_rope(const NormRopeParams<T>& p, int T_, cudaStream_t st) {
+  const int nv = (p.Hq + p.Hkv) * (p.D >> 3);
+  auto threads = [&](int vpt) { return dim3(((nv + vpt - 1) / vpt + 31) / 32 * 32); };
+  if (nv <= 256) return launch_pdl(qkv_norm_rope_append_kernel<T, 1>, dim3(T_), threads(1), 0, st, p);
+  if (nv <= 1024) return launch_pdl(qkv_norm_rope_append_kernel<T, 2>, dim3(T_), threads(2), 0, st, p);
+  if (nv <= 4096) return launch_pdl(qkv_norm_rope_append_kernel<T, 4>, dim3(T_), threads(4), 0, st, p);
+  return cudaErrorInvalidValue;
+}
+
+// Root-mean-square norms of two column ranges of a row: the query latent (blockIdx.y 0) to q_out, the key/value latent
+// (blockIdx.y 1) to its place in the paged panel (slot < 0: a padding row, skipped). Sizes are rounded up to multiples of 8
+// in storage; pad columns and their weights are zero.
+template <typename T>
+struct LatentNormsParams {
+  const T* q; const T* kv; long long ld;
+  const T* qw; const T* kvw; float eps;
+  T* q_out; int q_rank, kv_rank;
+  const int* slots; T* cache; long long block_stride; int block_tokens; long long num_slots;
+  int* err;
+};
+constexpr int kLnThreads = 128;
+
+template <typename T>
+__global__ void __launch_bounds__(kLnThreads) latent_norms_kernel(const LatentNormsParams<T> p) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float red[kLnThreads / 32];
+  const int t = blockIdx.x;
+  const bool is_q = blockIdx.y == 0;
+  const int n = is_q ? p.q_rank : p.kv_rank, np = (n + 7) / 8 * 8;
+  const T* src = (is_q ? p.q : p.kv) + static_cast<size_t>(t) * p.ld;
+  const T* w = is_q ? p.qw : p.kvw;
+  T* dst;
+  if (is_q) {
+    dst = p.q_out + static_cast<size_t>(t) * np;
+  } else {
+    const int slot = p.slots[t];
+    if (slot < 0) return;
+    if (slot >= p.num_slots) { if (threadIdx.x == 0) guard_report(p.err, kGuardSlot, slot); return; }
+    dst = p.cache + static_cast<size_t>(slot / p.block_tokens) * p.block_stride + static_cast<size_t>(slot % p.block_tokens) * np;
+  }
+  constexpr int kKeep = 2;              // vectors per thread that stay in registers between the two passes
+  float keep[kKeep][8], ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < kKeep; ++j) {
+    const int i = (threadIdx.x + j * kLnThreads) * 8;
+    if (i < np) {
+      load8(src + i, keep[j]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss = fmaf(keep[j][e], keep[j][e], ss);
+    }
+  }
+  for (int i = (threadIdx.x + kKeep * kLnThreads) * 8; i < np; i += kLnThreads * 8) {
+    float f[8];
+    load8(src + i, f);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss = fmaf(f[e], f[e], ss);
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < kLnThreads / 32; ++k) ss += red[k];
+  const float r = rsqrtf(ss / static_cast<float>(n) + p.eps);
+  auto put = [&](int i, float (&f)[8]) {
+    float g[8];
+    load8(w + i, g);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) f[e] *= r * g[e];
+    store8(dst + i, f);
+  };
+#pragma unroll
+  for (int j = 0; j < kKeep; ++j) {
+    const int i = (threadIdx.x + j * kLnThreads) * 8;
+    if (i < np) put(i, keep[j]);
+  }
+  for (int i = (threadIdx.x + kKeep * kLnThreads) * 8; i < np; i += kLnThreads * 8) {
+    float f[8];
+    load8(src + i, f);
+    put(i, f);
+  }
+}
+
 // x[pos[r], :] = emb[r, :] (fp32 rows of H real columns, stream rows ldx apart)
 __global__ void refit_rows_f32_kernel(float* __restrict__ x, int ldx, const int* __restrict__ pos, const float* __restrict__ emb,
                                       int H, int rows, int* err) {
@@ -447,27 +695,36 @@ extern "C" int ksana_embed_pair(const int* ids, const int* prev, const void* tab
   return e == cudaSuccess ? 0 : -4;
 }
 
+template <typename T>
+static int residual_norm_entry(const float* x, int ldx, const int* rows, int in_rows, const void* y, int ldy, const void* w1,
+                               const void* b1, const void* ls, float* x_out, const void* w2, const void* b2, void* z, int ldz,
+                               int M, int H, float eps, int rms, float alpha, int groups, const float* add, const void* vec,
+                               float z_scale, const int* dst_row, const float* w, int ldw, int top, int cap, const void* shared,
+                               int lds, int* err, cudaStream_t st) {
+  const ResNormParams<T> p{x, ldx, rows, in_rows, (const T*)y, ldy, (const T*)w1, (const T*)b1, (const T*)ls, x_out, (const T*)w2,
+                           (const T*)b2, (T*)z, ldz, H, eps, rms, alpha, groups, add, (const T*)vec, z_scale, dst_row, w, ldw, top,
+                           cap, (const T*)shared, lds, err};
+  return launch_residual_norm(p, M, st);
+}
+
+// dst_row [M, top] / w [M, ldw] / shared: the addend is gathered from the expert outputs y [cap, ldy] (see ResNormParams)
 extern "C" int ksana_residual_norm(const float* x, int ldx, const int* rows, int in_rows, const void* y, int ldy,
                                    const void* w1, const void* b1, const void* ls, float* x_out, const void* w2,
                                    const void* b2, void* z, int ldz, int M, int H, float eps, int rms, int f32,
-                                   float alpha, int groups, int* err, cudaStream_t st) {
+                                   float alpha, int groups, const float* add, const void* vec, float z_scale, const int* dst_row,
+                                   const float* w, int ldw, int top, int cap, const void* shared, int lds, int* err, cudaStream_t st) {
   if (M <= 0) return 0;
   const int hp = (H + 7) / 8 * 8;
   if (H <= 0 || ldx % 8 || ldx < hp || (y && (ldy % 8 || ldy < hp)) || (z && (ldz % 8 || ldz < hp))) return -10;
-  for (const void* q : {(const void*)x, y, w1, b1, ls, (const void*)x_out, w2, b2, (const void*)z})
+  for (const void* q : {(const void*)x, y, w1, b1, ls, (const void*)x_out, w2, b2, (const void*)z, (const void*)add, vec, shared})
     if (!aligned16(q)) return -11;
   if (rows && x_out == x) return -12;
-  if (groups > 1 && (!rms || H % groups || w1 || b2 || !w2)) return -13;
-  if (f32) {
-    typedef float T;
-    const ResNormParams<T> p{x, ldx, rows, in_rows, (const T*)y, ldy, (const T*)w1, (const T*)b1, (const T*)ls, x_out,
-                             (const T*)w2, (const T*)b2, (T*)z, ldz, H, eps, rms, alpha, groups, err};
-    return launch_residual_norm(p, M, st);
-  }
-  typedef bf16 T;
-  const ResNormParams<T> p{x, ldx, rows, in_rows, (const T*)y, ldy, (const T*)w1, (const T*)b1, (const T*)ls, x_out,
-                           (const T*)w2, (const T*)b2, (T*)z, ldz, H, eps, rms, alpha, groups, err};
-  return launch_residual_norm(p, M, st);
+  if (groups > 1 && (!rms || H % groups || w1 || b2 || !w2 || z_scale != 1.f)) return -13;
+  if (dst_row && (!y || !w || rows || top <= 0 || top > kMaxTop || ldw < top + (shared ? 1 : 0) || cap <= 0)) return -14;
+  if (shared && (!dst_row || lds % 8 || lds < hp)) return -15;
+  auto entry = f32 ? residual_norm_entry<float> : residual_norm_entry<bf16>;
+  return entry(x, ldx, rows, in_rows, y, ldy, w1, b1, ls, x_out, w2, b2, z, ldz, M, H, eps, rms, alpha, groups, add, vec, z_scale,
+               dst_row, w, ldw, top, cap, shared, lds, err, st);
 }
 
 // in [M, in_ld]: gate columns [0, I), up columns [I, 2I); out [M, I]. I a multiple of 8.
@@ -519,6 +776,51 @@ extern "C" int ksana_qkv_rope_append(void* qkv, const int* positions, const int*
     e = launch_pdl(qkv_rope_append_kernel<bf16>, dim3(T), dim3(threads), 0, st, (bf16*)qkv, positions, slots, cos_sin, max_pos,
                    (bf16*)kc, (bf16*)vc, block_stride, block_tokens, num_blocks, Hq, Hkv, D, Dv, rot, err);
   return e == cudaSuccess ? 0 : -4;
+}
+
+template <typename T>
+static cudaError_t norm_rope_entry(void* qkv, const int* positions, const int* slots, const float* cos_sin, int max_pos,
+                                   const void* qw, const void* kw, float eps, int nq, int nk, const float* sums, void* kc, void* vc,
+                                   long long block_stride, int block_tokens, int num_blocks, int T_, int Hq, int Hkv, int D, int Dv,
+                                   int rot, int* err, cudaStream_t st) {
+  const NormRopeParams<T> p{(T*)qkv, positions, slots, cos_sin, max_pos, (const T*)qw, (const T*)kw, eps, nq, nk, sums, (T*)kc, (T*)vc,
+                            block_stride, block_tokens, num_blocks, Hq, Hkv, D, Dv, rot, err};
+  return launch_norm_rope(p, T_, st);
+}
+
+extern "C" int ksana_qkv_norm_rope_append(void* qkv, const int* positions, const int* slots, const float* cos_sin, int max_pos,
+                                          const void* qw, const void* kw, float eps, int nq, int nk, const float* sums, void* kc,
+                                          void* vc, long long block_stride, int block_tokens, int num_blocks, int T, int Hq, int Hkv,
+                                          int D, int Dv, int rot, int f32, int* err, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (Hq <= 0 || Hkv <= 0 || D <= 0 || Dv <= 0 || D % 8 || Dv % 8 || rot < 0 || rot > D || (rot & 1) || block_tokens <= 0 ||
+      block_stride % 8 || (rot && !cos_sin) || !qw || !kw || nq <= 0 || nk <= 0 || (Hq + Hkv) * (D / 8) > 4096) return -10;
+  if (!aligned16(qkv) || !aligned16(kc) || !aligned16(vc) || !aligned16(qw) || !aligned16(kw)) return -11;
+  auto entry = f32 ? norm_rope_entry<float> : norm_rope_entry<bf16>;
+  return entry(qkv, positions, slots, cos_sin, max_pos, qw, kw, eps, nq, nk, sums, kc, vc, block_stride, block_tokens, num_blocks, T, Hq,
+               Hkv, D, Dv, rot, err, st) == cudaSuccess ? 0 : -4;
+}
+
+template <typename T>
+static cudaError_t latent_norms_entry(const void* q, const void* kv, long long ld, const void* qw, const void* kvw, float eps,
+                                      void* q_out, int q_rank, int kv_rank, const int* slots, void* cache, long long block_stride,
+                                      int block_tokens, long long num_slots, int T_, int* err, cudaStream_t st) {
+  const LatentNormsParams<T> p{(const T*)q, (const T*)kv, ld, (const T*)qw, (const T*)kvw, eps, (T*)q_out, q_rank, kv_rank, slots,
+                               (T*)cache, block_stride, block_tokens, num_slots, err};
+  return launch_pdl(latent_norms_kernel<T>, dim3(T_, 2), dim3(kLnThreads), 0, st, p);
+}
+
+// q, kv: column ranges of the same projection's rows, ld elements apart; q_out [T, q_rank rounded up to 8]
+extern "C" int ksana_latent_norms(const void* q, const void* kv, long long ld, const void* qw, const void* kvw, float eps,
+                                  void* q_out, int q_rank, int kv_rank, const int* slots, void* cache, long long block_stride,
+                                  int block_tokens, long long num_slots, int T, int f32, int* err, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (q_rank <= 0 || kv_rank <= 0 || ld % 8 || block_stride % 8 || block_tokens <= 0) return -10;
+  for (const void* a : {q, kv, qw, kvw, (const void*)q_out, (const void*)cache})
+    if (!a || !aligned16(a)) return -11;
+  auto entry = f32 ? latent_norms_entry<float> : latent_norms_entry<bf16>;
+  return entry(q, kv, ld, qw, kvw, eps, q_out, q_rank, kv_rank, slots, cache, block_stride, block_tokens, num_slots, T, err, st) ==
+                 cudaSuccess ? 0 : -4;
 }
 
 extern "C" int ksana_refit_rows_f32(float* x, int ldx, const int* pos, const float* emb, int R, int H, int rows, int* err,

@@ -22,11 +22,10 @@ import torch
 
 from ..config import AttentionSpec, LayerSpec, ModelConfig
 from ..ops import dispatch as ops
-from ..ops import native
 from ..ops.dispatch import LinearWeight, NormParams
 from ..utils import nvtx
 from .common import PanelLayout, StepInput
-from .stream import StreamLoader, StreamModel, pad8, pad_to
+from .stream import LayerRun, StreamLoader, StreamModel, layer_runs, pad8, pad_to, rerotate_panel
 
 MAX_HEAD = 256                    # largest head size of the attention kernels
 
@@ -48,25 +47,6 @@ class SandwichLayer:
     gate_up: Optional[LinearWeight] = None
     down: Optional[LinearWeight] = None
     moe: Optional[object] = None
-
-
-@dataclass
-class LayerRun:
-    layer: int
-    cache: int                    # cache layer of this run
-    enter: Optional[int] = None   # number of the loop pass that starts right before this run
-
-
-def layer_runs(cfg: ModelConfig) -> List[LayerRun]:
-    order, n, loop = [], len(cfg.layer_specs), cfg.loop
-    if loop is None:
-        order = [(i, None) for i in range(n)]
-    else:
-        order = [(i, None) for i in range(loop.start)]
-        for t in range(loop.times):
-            order += [(i, t if i == loop.start else None) for i in range(loop.start, loop.stop)]
-        order += [(i, None) for i in range(loop.stop, n)]
-    return [LayerRun(i, c, enter) for c, (i, enter) in enumerate(order)]
 
 
 class LenolixModel(StreamModel):
@@ -96,20 +76,8 @@ class LenolixModel(StreamModel):
         """Copies that landed at another position (flexible cache): every run's keys are turned by the position delta."""
         for run, (k, _) in zip(self.runs, self.panels):
             table = self.rotary.get(run.layer)
-            if table is None:
-                continue
-            dims = table.shape[1]
-            if k.is_cuda and k.dtype == torch.bfloat16:
-                t3 = torch.as_tensor(triples, dtype=torch.int32).contiguous().to(k.device)
-                native.rerotate_panel(k, t3, table, dims)
-                continue
-            for _, dst, delta in triples:
-                delta = int(delta)
-                if delta:
-                    cos, sin = table[abs(delta)].chunk(2)
-                    sin = sin if delta > 0 else -sin
-                    u, v = k[int(dst), ..., :dims].float().chunk(2, dim=-1)
-                    k[int(dst), ..., :dims] = torch.cat([u * cos - v * sin, v * cos + u * sin], -1).to(k.dtype)
+            if table is not None:
+                rerotate_panel(k, triples, table)
 
     # ------------------------------------------------------------------ blocks
     def embed_tokens(self, step: StepInput, copy=None) -> torch.Tensor:
@@ -169,7 +137,6 @@ class LenolixModel(StreamModel):
 # ------------------------------------------------------------------------------------- loading
 def build_lenolix(cfg: ModelConfig, source, tp_rank=0, tp_size=1, comm=None, device="cpu", dtype=torch.bfloat16, quant=None,
                   layer_range=None, max_positions=None) -> LenolixModel:
-    from .weights import _rows
     if layer_range is not None and tuple(layer_range) != (0, cfg.num_layers - 1):
         raise ValueError("lenolix: repeated layers need the embedding output, pipeline stages are not supported")
     for s in cfg.layer_specs:
@@ -195,11 +162,9 @@ def build_lenolix(cfg: ModelConfig, source, tp_rank=0, tp_size=1, comm=None, dev
     for i, spec in enumerate(cfg.layer_specs):
         p, a = f"l{i}.", spec.mixer
         D, DV = pad8(a.dim), pad8(a.vdim)
-        rep = max(1, tp_size // a.kv_heads)              # ranks sharing one key/value head
-        kv_rank, kv_size = tp_rank // rep, tp_size // rep
         q = rows(pad_to(get(p + "mix.q", (a.heads * a.dim, W)).reshape(a.heads, a.dim, W), a.heads, D, WP))
-        k = _rows(pad_to(get(p + "mix.k", (a.kv_heads * a.dim, W)).reshape(a.kv_heads, a.dim, W), a.kv_heads, D, WP), kv_rank, kv_size)
-        v = _rows(pad_to(get(p + "mix.v", (a.kv_heads * a.vdim, W)).reshape(a.kv_heads, a.vdim, W), a.kv_heads, DV, WP), kv_rank, kv_size)
+        k = ld.kv_heads(pad_to(get(p + "mix.k", (a.kv_heads * a.dim, W)).reshape(a.kv_heads, a.dim, W), a.kv_heads, D, WP))
+        v = ld.kv_heads(pad_to(get(p + "mix.v", (a.kv_heads * a.vdim, W)).reshape(a.kv_heads, a.vdim, W), a.kv_heads, DV, WP))
         o = cols(pad_to(get(p + "mix.o", (W, a.heads * a.vdim)).reshape(W, a.heads, a.vdim), WP, a.heads, DV))
         sinks = get(p + "mix.sink", (a.heads,))[tp_rank * q.shape[0]:(tp_rank + 1) * q.shape[0]] if a.sink else None
         lw = SandwichLayer(spec, q.shape[0], k.shape[0], norm(p + "norm1"), norm(p + "norm1b"),
@@ -207,10 +172,8 @@ def build_lenolix(cfg: ModelConfig, source, tp_rank=0, tp_size=1, comm=None, dev
                            sinks.to(device=device, dtype=torch.float32).contiguous() if sinks is not None else None,
                            param(get(p + "ls1", (W,), "ones"), WP))
         if spec.mlp is not None:
-            ff = spec.mlp.size
-            n = ld.shard(ff)                             # columns of a rank
-            gate, up = (rows(pad_to(get(p + "mlp." + s, (ff, W)), n * tp_size, WP)) for s in ("gate", "up"))
-            down = cols(pad_to(get(p + "mlp.down", (W, ff)), WP, n * tp_size))
+            gate, up = (ld.split_rows(p + "mlp." + s, spec.mlp.size) for s in ("gate", "up"))
+            down = ld.split_cols(p + "mlp.down", spec.mlp.size)
             lw.norm2, lw.norm2b, lw.ls2 = norm(p + "norm2"), norm(p + "norm2b"), param(get(p + "ls2", (W,), "ones"), WP)
             lw.gate_up, lw.down = linear(torch.cat([gate, up], 0)), linear(down)
         m.layers.append(lw)

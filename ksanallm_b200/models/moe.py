@@ -157,24 +157,30 @@ def load_moe(cfg: ModelConfig, source, prefix: str, tp_rank, tp_size, device, dt
 
 def route_reference(logits, cfg: ModelConfig, bias=None):
     """Plain statement of the routing rules; returns (ids [T,K] int64, weights [T,K] fp32)."""
-    K = cfg.num_experts_per_tok
-    if cfg.moe_scoring == "sigmoid":
-        score = torch.sigmoid(logits.float())
-    else:
-        score = torch.softmax(logits.float(), dim=-1)
-    sel = score + (bias.float() if bias is not None else 0.0)
-    if cfg.n_group > 1 and cfg.topk_group < cfg.n_group:
-        T, E = sel.shape
-        grp = sel.view(T, cfg.n_group, E // cfg.n_group)
-        gscore = grp.topk(2, dim=-1).values.sum(-1)
-        keep = gscore.topk(cfg.topk_group, dim=-1).indices
-        mask = torch.zeros(T, cfg.n_group, dtype=torch.bool, device=sel.device).scatter_(1, keep, True)
-        sel = sel.masked_fill(~mask.unsqueeze(-1).expand_as(grp).reshape(T, E), float("-inf"))
-    ids = sel.topk(K, dim=-1).indices
-    w = score.gather(1, ids)
-    if cfg.norm_topk_prob:
-        w = w / w.sum(-1, keepdim=True).clamp_min(1e-20)
-    return ids, w * cfg.routed_scaling_factor
+    return ref.moe_route(logits, cfg.num_experts_per_tok, cfg.moe_scoring, cfg.norm_topk_prob, cfg.routed_scaling_factor, bias,
+                         cfg.n_group, cfg.topk_group)
+
+
+def dense_experts(perm, w13, w2, tile_expert, n_local, inter, act):
+    """Expert-major rows through their experts' gate|up and down matrices (stacked [E * 2I, H] and [E * H, I], bf16 or fp32)."""
+    g = native.gemm_grouped(perm, w13, tile_expert, n_local, 2 * inter)
+    return native.gemm_grouped(native.act_mul(g, act, True), w2, tile_expert, n_local, perm.shape[1])
+
+
+def expert_outputs(x, ids, w13, w2, inter, act="silu"):
+    """Outputs of the chosen experts before they are weighted and summed: (rows, row of every (token, choice) [T, K])."""
+    T, K = ids.shape
+    E = w2.shape[0] // x.shape[1]
+    if x.is_cuda:
+        dst_row, tile_expert, _, _, cap = native.moe_align(ids, E)
+        return dense_experts(native.moe_permute(x, dst_row, K, cap), w13, w2, tile_expert, E, inter, act), dst_row.view(T, K)
+    y = torch.zeros(T * K, x.shape[1], dtype=x.dtype)
+    for e in range(E):
+        tok, slot = (ids == e).nonzero(as_tuple=True)
+        if tok.numel():
+            gu = ref.gemm(x[tok], w13[e * 2 * inter:(e + 1) * 2 * inter])
+            y[tok * K + slot] = ref.gemm(ref.act_mul(gu, act, True), w2[e * x.shape[1]:(e + 1) * x.shape[1]])
+    return y, torch.arange(T * K, dtype=torch.int32).view(T, K)
 
 
 def moe_forward(model, mw: MoEWeights, x: torch.Tensor, h: torch.Tensor) -> torch.Tensor:
@@ -254,9 +260,7 @@ def moe_partial(model, mw: MoEWeights, x: torch.Tensor, into: Optional[torch.Ten
             _, aq, as_ = native.act_mul(g, cfg.activation, True, quant=True, want_out=False)
             y = native.gemm_grouped(aq, mw.w2, tile_expert, n_local, H, a_scale=as_, w_scale=mw.w2_scale)
         else:
-            g = native.gemm_grouped(perm, mw.w13, tile_expert, n_local, 2 * mw.inter)
-            a = native.act_mul(g, cfg.activation, True)
-            y = native.gemm_grouped(a, mw.w2, tile_expert, n_local, H)
+            y = dense_experts(perm, mw.w13, mw.w2, tile_expert, n_local, mw.inter, cfg.activation)
         out = into if into is not None else torch.empty(T, H, dtype=x.dtype, device=x.device)
         have_shared = shared and mw.shared_gate_up is not None
         if have_shared:

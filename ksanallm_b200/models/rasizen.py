@@ -146,13 +146,6 @@ def build_rasizen(cfg: ModelConfig, source, tp_rank=0, tp_size=1, comm=None, dev
     def norm(name, n=W, groups=cfg.norm_groups):
         return NormParams(ld.param(ld.get(name, (n,), "ones"), pad8(n)), None, n, cfg.rms_norm_eps, rms=True, groups=groups)
 
-    def split_rows(name, n):
-        """Rows of a projection to channels that are split over the ranks, padded."""
-        return ld.rows(pad_to(ld.get(name, (n, W)), ld.shard(n) * tp_size, WP))
-
-    def split_cols(name, n):
-        return ld.cols(pad_to(ld.get(name, (W, n)), WP, ld.shard(n) * tp_size))
-
     ld.vocabulary()
     for i, spec in enumerate(cfg.layer_specs):
         p, a = f"l{i}.", spec.mixer
@@ -160,10 +153,10 @@ def build_rasizen(cfg: ModelConfig, source, tp_rank=0, tp_size=1, comm=None, dev
         n1 = norm(p + "norm1")
         if isinstance(a, GatedRecurrenceSpec):
             n = ld.shard(a.width)
-            z, u, g = (split_rows(x + s, a.width) for s in ("z", "x", "g"))
+            z, u, g = (ld.split_rows(x + s, a.width) for s in ("z", "x", "g"))
             bz, bu = (ld.rows(pad_to(ld.get(x + s, (a.width,), "zeros"), n * tp_size)) for s in ("z.b", "x.b"))
             lw = HybridLayer(spec, n1, ld.linear(torch.cat([z, u, g], 0), torch.cat([bz, bu, torch.zeros_like(bz)], 0)),
-                             ld.linear(split_cols(x + "o", a.width)), channels=n)
+                             ld.linear(ld.split_cols(x + "o", a.width)), channels=n)
         else:
             H, d, r, v, k = a.heads, pad8(a.dim), pad8(a.rot_dim), pad8(a.vdim), pad8(a.kv_rank)
             q = ld.get(x + "q", (H * (a.dim + a.rot_dim), W)).reshape(H, a.dim + a.rot_dim, W)
@@ -184,7 +177,7 @@ def build_rasizen(cfg: ModelConfig, source, tp_rank=0, tp_size=1, comm=None, dev
         if spec.mlp is not None:
             ff = spec.mlp.size
             lw.norm2 = norm(p + "norm2")
-            lw.up, lw.down = ld.linear(split_rows(p + "mlp.up", ff)), ld.linear(split_cols(p + "mlp.down", ff))
+            lw.up, lw.down = ld.linear(ld.split_rows(p + "mlp.up", ff)), ld.linear(ld.split_cols(p + "mlp.down", ff))
             above, below = (float(t) for t in ld.get(p + "mlp.act", (2,)).float().cpu())
             lw.unit = (_softplus(above), UNIT_LINEAR + _softplus(below))
         m.layers.append(lw)

@@ -1,19 +1,21 @@
 """Base of the families with a 32-bit residual stream whose layers are configured one by one (``ModelConfig.layer_specs``):
-padded stream rows, per-layer rotation tables, row-parallel projections, the final norm over the rows that need logits,
-and the loading helpers.
+padded stream rows, per-layer rotation tables, layers that run several times, row-parallel projections, the final norm over
+the rows that need logits, and the loading helpers.
 
 Sizes that are not multiples of 8 are padded with zeros when the weights are loaded (rows of the residual stream, head
 sizes, feed-forward widths, vocabulary), so the kernels always see 16-byte vectors; norms count the real columns only.
 """
 from __future__ import annotations
 
-from typing import Optional
+from dataclasses import dataclass
+from typing import List, Optional
 
 import torch
 import torch.nn.functional as F
 
 from ..config import ModelConfig, RotarySpec
 from ..ops import dispatch as ops
+from ..ops import native
 from ..ops import reference as ref
 from ..ops.dispatch import LinearWeight, NormParams
 from .common import CommonModel, StepInput
@@ -29,6 +31,44 @@ def pad_to(t: torch.Tensor, *sizes: int) -> torch.Tensor:
     for have, want in zip(reversed(t.shape), reversed(sizes)):
         spec += [0, want - have]
     return F.pad(t, spec) if any(spec) else t
+
+
+@dataclass
+class LayerRun:
+    layer: int
+    cache: int                    # cache layer of this run
+    enter: Optional[int] = None   # number of the loop pass that starts right before this run
+
+
+def layer_runs(cfg: ModelConfig) -> List[LayerRun]:
+    order, n, loop = [], len(cfg.layer_specs), cfg.loop
+    if loop is None:
+        order = [(i, None) for i in range(n)]
+    else:
+        order = [(i, None) for i in range(loop.start)]
+        for t in range(loop.times):
+            order += [(i, t if i == loop.start else None) for i in range(loop.start, loop.stop)]
+        order += [(i, None) for i in range(loop.stop, n)]
+    return [LayerRun(i, c, enter) for c, (i, enter) in enumerate(order)]
+
+
+def rerotate_panel(k: torch.Tensor, triples, table: torch.Tensor, interleaved: bool = False) -> None:
+    """Turns the keys of copied blocks (``triples``: source, destination, position delta) of a panel [blocks, heads, block
+    tokens, size] by the position delta."""
+    dims = table.shape[1]
+    if k.is_cuda and k.dtype == torch.bfloat16:
+        t3 = torch.as_tensor(triples, dtype=torch.int32).contiguous().to(k.device)
+        native.rerotate_panel(k, t3, table, dims, neox=not interleaved)
+        return
+    for _, dst, delta in triples:
+        delta = int(delta)
+        if delta:
+            cos, sin = table[abs(delta)].chunk(2)
+            sin = sin if delta > 0 else -sin
+            r = k[int(dst), ..., :dims].float()
+            u, v = (r[..., 0::2], r[..., 1::2]) if interleaved else r.chunk(2, dim=-1)
+            turned = (u * cos - v * sin, v * cos + u * sin)
+            k[int(dst), ..., :dims] = (torch.stack(turned, -1).flatten(-2) if interleaved else torch.cat(turned, -1)).to(k.dtype)
 
 
 class StreamModel(CommonModel):
@@ -74,7 +114,8 @@ class StreamModel(CommonModel):
     def lm_head_forward(self, x: torch.Tensor, step: StepInput):
         if step.want_hidden:
             self.step_hidden, self.step_normed = x, ops.stream_norm(x, self.final, self.dtype)
-        return self.logits_or_candidates(ops.stream_norm(x, self.final, self.dtype, rows=step.logits_rows), step)
+        # the factor of the logits goes into their GEMM's operand
+        return self.logits_or_candidates(ops.stream_norm(x, self.final, self.dtype, rows=step.logits_rows, scale=self.cfg.logit_scale), step)
 
 
 class StreamLoader:
@@ -109,10 +150,27 @@ class StreamLoader:
         """Padded share of ``n`` columns or channels that are split over the ranks."""
         return pad8((n + self.m.tp_size - 1) // self.m.tp_size)
 
+    def split_rows(self, name, n: int) -> torch.Tensor:
+        """This rank's rows of a projection of the stream to ``n`` columns that are split over the ranks, padded."""
+        return self.rows(pad_to(self.get(name, (n, self.m.cfg.hidden_size)), self.shard(n) * self.m.tp_size, self.m.width))
+
+    def split_cols(self, name, n: int) -> torch.Tensor:
+        """This rank's columns of a projection of ``n`` split columns to the stream, padded."""
+        return self.cols(pad_to(self.get(name, (self.m.cfg.hidden_size, n)), self.m.width, self.shard(n) * self.m.tp_size))
+
+    def kv_heads(self, t: torch.Tensor) -> torch.Tensor:
+        """This rank's key/value heads of ``t`` [heads, ...]: its share of them, or the one that it shares with other ranks."""
+        from .weights import _rows
+        rep = max(1, self.m.tp_size // t.shape[0])
+        return _rows(t, self.m.tp_rank // rep, self.m.tp_size // rep)
+
     def vocabulary(self) -> None:
-        """Embedding table, and the same table (this rank's rows of it) as the output projection."""
+        """Embedding table, and the output projection (this rank's rows): the tensor ``head``, or the table again."""
         m, cfg = self.m, self.m.cfg
-        m.embed = self.param(self.get("embed", (cfg.vocab_size, cfg.hidden_size)), pad8(cfg.vocab_size), m.width)
+        full = (cfg.vocab_size, cfg.hidden_size)
+        m.embed = self.param(self.get("embed", full), pad8(cfg.vocab_size), m.width)
         vs = (cfg.vocab_size + m.tp_size - 1) // m.tp_size
-        m.lm_head = LinearWeight(w=m.embed if m.tp_size == 1 else self.param(self.rows(m.embed[:cfg.vocab_size]), pad8(vs), m.width))
+        head = m.embed if cfg.tie_word_embeddings else self.get("head", full)
+        tied = cfg.tie_word_embeddings and m.tp_size == 1
+        m.lm_head = LinearWeight(w=head if tied else self.param(self.rows(head[:cfg.vocab_size]), pad8(vs), m.width))
         m.vocab_shard = vs

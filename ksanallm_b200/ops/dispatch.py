@@ -265,14 +265,42 @@ def embed_pair(ids, prev, table, pair, scale, buckets=0, mul_prev=0, mul_cur=0, 
     return x
 
 
-def stream_norm(x, norm: NormParams, dtype, rows=None):
-    """norm of the fp32 residual stream (of its ``rows``) as the next linear's operand."""
+@dataclass
+class ExpertSum:
+    """A sublayer's result that is still spread over expert outputs: row t is the sum over k of w[t, k] * y[dst_row[t, k]]
+    (negative rows: left out), plus w[t, K] * shared[t]."""
+    y: torch.Tensor
+    dst_row: torch.Tensor                 # [T, K] int32
+    w: torch.Tensor                       # [T, K] or [T, K + 1] fp32
+    shared: Optional[torch.Tensor] = None
+
+    @property
+    def dtype(self):
+        return self.y.dtype
+
+
+def stream_norm(x, norm: NormParams, dtype, rows=None, scale=1.0):
+    """norm of the fp32 residual stream (of its ``rows``) times ``scale`` as the next linear's operand."""
     if x.is_cuda:
         z = torch.empty(rows.numel() if rows is not None else x.shape[0], x.shape[1], dtype=dtype, device=x.device)
         native.residual_norm(x, norm.size, norm.eps, w2=norm.w, b2=norm.b, z=z, rows=rows, rms=norm.rms,
-                             groups=norm.groups)
+                             groups=norm.groups, z_scale=scale)
         return z
-    return ref.stream_norm(x[rows.long()] if rows is not None else x, norm).to(dtype)
+    return (ref.stream_norm(x[rows.long()] if rows is not None else x, norm) * scale).to(dtype)
+
+
+def stream_enter(x, add, vec, then: NormParams, dtype, inplace=True):
+    """x + add + vec (fp32 rows or None, one row) and the following norm of the sum: (x, normed)."""
+    if x.is_cuda:
+        z = torch.empty(x.shape, dtype=dtype, device=x.device)
+        out = x if inplace else torch.empty_like(x)
+        native.residual_norm(x, then.size, then.eps, x_out=out, w2=then.w, b2=then.b, z=z, rms=then.rms, groups=then.groups, add=add,
+                             vec=vec)
+        return out, z
+    out = x + vec.float() if add is None else x + add + vec.float()
+    if inplace:
+        out = x.copy_(out)
+    return out, ref.stream_norm(out, then).to(dtype)
 
 
 def stream_copy(x, out):
@@ -283,28 +311,38 @@ def stream_copy(x, out):
         out.copy_(x)
 
 
-def stream_add(x, y, post: Optional[NormParams], scale, then: Optional[NormParams] = None, copy=None, inplace=True, alpha=1.0):
-    """x + alpha * scale * norm(y; post) (``scale``: per column, ``alpha``: one number) on the fp32 residual stream, fused with what reads the sum next: ``then`` (the following
-    norm, returned in y's type) or ``copy`` (a buffer that receives the sum in its own type). Returns (x, normed or None);
+def stream_add(x, y, post: Optional[NormParams], scale, then: Optional[NormParams] = None, copy=None, inplace=True, alpha=1.0,
+               add=None, vec=None):
+    """x + alpha * scale * norm(y; post) + add + vec (``scale``: per column, ``alpha``: one number, ``add``: fp32 rows, ``vec``: one
+    row) on the fp32 residual stream, fused with what reads the sum next: ``then`` (the following norm, returned in y's type) or
+    ``copy`` (a buffer that receives the sum in its own type). ``y`` may be an :class:`ExpertSum`. Returns (x, normed or None);
     ``inplace`` updates x."""
     if x.is_cuda:
-        z = torch.empty_like(y) if then is not None else copy
+        experts = (y.dst_row, y.w, y.shared) if isinstance(y, ExpertSum) else None
+        z = torch.empty(x.shape, dtype=y.dtype, device=x.device) if then is not None else copy
         out = x if inplace else torch.empty_like(x)
         size, eps, rms = (post.size, post.eps, post.rms) if post is not None else (
             (then.size, then.eps, then.rms) if then is not None else (x.shape[1], 0.0, False))
-        native.residual_norm(x, size, eps, y=y, w1=post.w if post else None, b1=post.b if post else None, ls=scale, x_out=out,
-                             w2=then.w if then else None, b2=then.b if then else None, z=z, rms=rms, alpha=alpha,
-                             groups=then.groups if then else 1)
+        native.residual_norm(x, size, eps, y=y.y if experts else y, w1=post.w if post else None, b1=post.b if post else None, ls=scale,
+                             x_out=out, w2=then.w if then else None, b2=then.b if then else None, z=z, rms=rms, alpha=alpha,
+                             groups=then.groups if then else 1, add=add, vec=vec, experts=experts)
         return out, (z if then is not None else None)
+    dtype = y.dtype
+    if isinstance(y, ExpertSum):
+        y = ref.expert_sum(y.y, y.dst_row, y.w, y.shared)
     a = ref.stream_norm(y, post) if post is not None else y.float()
     if scale is not None:
         a = a * scale.float()
     if alpha != 1.0:
         a = a * alpha
+    if add is not None:
+        a = a + add
+    if vec is not None:
+        a = a + vec.float()
     out = x.add_(a) if inplace else x + a
     if copy is not None:
         copy.copy_(out)
-    return out, (ref.stream_norm(out, then).to(y.dtype) if then is not None else None)
+    return out, (ref.stream_norm(out, then).to(dtype) if then is not None else None)
 
 
 def glu_clamp(x, limit, alpha=1.702, offset=1.0):
@@ -359,23 +397,32 @@ def latent_append(q, nope, kv, norm: Optional[NormParams], step, cos_sin, cache,
     return qfull
 
 
-def latent_attention(qfull, cache, dv, block_tokens, step, scale, window=0):
+def latent_norms(q, kv, q_norm: NormParams, kv_norm: NormParams, step, cache, block_tokens):
+    """Normed query latents, and the append of the normed key/value latents to the panel ``cache`` [blocks, block tokens, rank];
+    q, kv: column ranges of one projection's rows."""
+    fn = native.latent_norms if q.is_cuda else ref.latent_norms
+    return fn(q, kv, q_norm.w, kv_norm.w, q_norm.eps, q_norm.size, kv_norm.size, step.slots, cache, block_tokens)
+
+
+def latent_attention(qfull, cache, dv, block_tokens, step, scale, window=0, sinks=None, gate=None):
     """Absorbed attention of packed query rows [T, G, DK] against the latent panel [blocks, block tokens, DK], values = the
-    first ``dv`` columns of its rows: [T, G, dv]. The tensor-core kernel serves bf16 rows up to 576 / 512 columns over
+    first ``dv`` columns of its rows: [T, G, dv]. ``sinks`` [G]: logits in the denominator only, ``gate`` [T, G]: a head's output
+    is multiplied by its sigmoid. The tensor-core kernel serves bf16 rows up to 576 / 512 columns over
     blocks of 8 to 256 (a power of two) tokens, the 32-bit one the rest."""
     T, G, dk = qfull.shape
     if not qfull.is_cuda:
-        return ref.mla_attention(qfull, cache, step.block_table, step.cu_q, step.kv_lens, scale, dv, window).to(qfull.dtype)
+        return ref.mla_attention(qfull, cache, step.block_table, step.cu_q, step.kv_lens, scale, dv, window, sinks, gate).to(qfull.dtype)
     out = torch.empty(T, G, dv, dtype=qfull.dtype, device=qfull.device)
     B, mq = step.num_multi + step.num_single, max(step.max_q_len, 1)
     if qfull.dtype == torch.bfloat16:
         seen = min(step.max_kv_len, window + 64) if window > 0 else step.max_kv_len
         n = native.mla_splits(B, mq, seen, halves=(dv + 255) // 256) if step.num_multi == 0 else 1
-        if native.mla_attention(qfull, out, cache, block_tokens, step.block_table, step.cu_q, step.kv_lens, B, mq, scale, n, window):
+        if native.mla_attention(qfull, out, cache, block_tokens, step.block_table, step.cu_q, step.kv_lens, B, mq, scale, n, window,
+                                sinks, gate):
             return out
     panel = cache.unsqueeze(1)                           # one key/value head shared by all query heads
     native.attention_f32(qfull, G * dk, out.view(T, G * dv), panel, panel[..., :dv], block_tokens, step.block_table, step.cu_q,
-                         step.kv_lens, B, mq, G, 1, scale, window)
+                         step.kv_lens, B, mq, G, 1, scale, window, sinks=sinks, gate=gate)
     return out
 
 
@@ -383,6 +430,23 @@ def qkv_rope_append(qkv, positions, slots, cos_sin, k_cache, v_cache, block_toke
     """Partial rotation of q and k and append of k, v to separate paged panels (key and value sizes may differ)."""
     fn = native.qkv_rope_append if qkv.is_cuda else ref.qkv_rope_append
     fn(qkv, positions, slots, cos_sin, k_cache, v_cache, block_tokens, Hq, Hkv, rot_dim)
+
+
+def qkv_norm_rope_append(qkv, step, cos_sin, q_norm: NormParams, k_norm: NormParams, k_cache, v_cache, block_tokens, Hq, Hkv, rot_dim,
+                         sums=None):
+    """Norms over all of q and all of k, partial rotation of neighbouring pairs, append of k and v to paged panels. ``sums`` [T, 2]:
+    sums of squares of the whole rows where ``qkv`` holds this rank's heads only (the norms' sizes are those of the whole)."""
+    fn = native.qkv_norm_rope_append if qkv.is_cuda else ref.qkv_norm_rope_append
+    fn(qkv, step.positions, step.slots, cos_sin, q_norm.w, k_norm.w, q_norm.eps, q_norm.size, k_norm.size, k_cache, v_cache, block_tokens,
+       Hq, Hkv, rot_dim, sums)
+
+
+def moe_route(logits, K, **kw):
+    """(ids [T, K] int32, weights fp32) by rows of router logits; options as in native.moe_route."""
+    if logits.is_cuda:
+        return native.moe_route(logits, K, **kw)
+    ids, w = ref.moe_route(logits, K, **kw)
+    return ids.to(torch.int32), w
 
 
 def refit_stream_rows(x, pos, emb):

@@ -35,7 +35,7 @@ _SIGS = {
     "ksana_gemm_smallm": [i32, vp, i32, vp, i32, vp, i32, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32, vp, i64, vp, i32,
                           vp, vp],
     "ksana_gemm_grouped": [i32, vp, i32, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, vp, i32, vp, vp],
-    "ksana_moe_route": [vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, i32, vp],
+    "ksana_moe_route": [vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32, f32, i32, i32, i32, vp],
     "ksana_moe_align": [vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
     "ksana_moe_permute": [vp, vp, vp, i32, i32, i32, i32, vp, vp],
     "ksana_moe_combine": [vp, vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
@@ -52,6 +52,7 @@ _SIGS = {
     "ksana_allgather_pull": [vp, vp, i32, i32, vp, i64, vp, i32, i32, i32, i32, vp, vp],
     "ksana_norm": [vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, f32, i32, vp],
     "ksana_act_mul": [vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
+    "ksana_act_mul_f32": [vp, vp, i32, i32, i32, i32, i32, vp],
     "ksana_quant_fp8": [vp, vp, vp, i32, i32, i32, i32, vp],
     "ksana_embedding": [vp, vp, vp, vp, vp, i32, i32, i32, i32, f32, vp],
     "ksana_gather_rows": [vp, vp, vp, i32, i32, i32, vp, vp],
@@ -66,15 +67,20 @@ _SIGS = {
     "ksana_absmax_scale": [vp, i32, i32, i64, f32, f32, vp, vp, vp],
     "ksana_rerotate_blocks": [vp, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, i64, vp, vp],
     "ksana_embed_pair": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i64, i64, i64, f32, i32, vp, vp],
-    "ksana_residual_norm": [vp, i32, vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, f32, i32, i32, f32, i32, vp, vp],
+    "ksana_residual_norm": [vp, i32, vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, f32, i32, i32, f32, i32, vp, vp, f32,
+                            vp, vp, i32, i32, i32, vp, i32, vp, vp],
     "ksana_glu_clamp": [vp, vp, i32, i32, i32, f32, f32, f32, i32, vp],
     "ksana_xielu": [vp, i32, vp, i32, i32, i32, f32, f32, f32, i32, vp],
     "ksana_gated_recurrence": [vp, vp, vp, i64, vp, i64, vp, i64, i32, i32, vp, i32, vp, vp, vp, i32, i32, f32, i32, vp, vp],
     "ksana_gemm_f32_batched": [vp, i32, i64, vp, i32, i64, vp, i32, i64, i32, i32, i32, i32, vp, i32, i64, vp],
     "ksana_qkv_rope_append": [vp, vp, vp, vp, i32, vp, vp, i64, i32, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp],
+    "ksana_qkv_norm_rope_append": [vp, vp, vp, vp, i32, vp, vp, f32, i32, i32, vp, vp, vp, i64, i32, i32, i32, i32, i32, i32, i32, i32,
+                                   i32, vp, vp],
+    "ksana_latent_norms": [vp, vp, i64, vp, vp, f32, vp, i32, i32, vp, vp, i64, i32, i64, i32, i32, vp, vp],
+    "ksana_gemm_grouped_f32": [vp, i32, vp, i32, vp, i32, i32, i32, i32, i32, vp, vp],
     "ksana_refit_rows_f32": [vp, i32, vp, vp, i32, i32, i32, vp, vp],
     "ksana_gemm_f32": [vp, i32, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, vp],
-    "ksana_attention_f32": [vp, i64, vp, i64, vp, vp, i32, i64, i32, i32, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32,
+    "ksana_attention_f32": [vp, i64, vp, i64, vp, vp, i32, i64, i32, i32, vp, i32, vp, vp, vp, vp, i64, i32, i32, i32, i32, i32, i32, i32,
                             i32, f32, i32, vp, vp],
     "ksana_cast_f32": [vp, vp, i64, vp],
     "ksana_paged_prefill_tc": [vp, i64, i64, vp, i64, vp, vp, i64, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32,
@@ -83,7 +89,8 @@ _SIGS = {
                             f32, i32, f32, f32, i32, vp, vp],
     "ksana_paged_decode": [vp, i64, vp, i64, vp, vp, i64, i32, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, i32,
                            f32, f32, i32, vp, vp, i32, vp, vp, i32, vp, vp],
-    "ksana_mla_attention": [vp, i64, vp, i64, vp, i64, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, f32, i32, i32, vp, vp, vp, vp],
+    "ksana_mla_attention": [vp, i64, vp, i64, vp, i64, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp, i64, f32, i32, i32, vp,
+                            vp, vp, vp],
     "ksana_mla_rope_append": [vp, i64, i32, vp, i64, vp, f32, vp, vp, vp, vp, vp, i64, i32, i32, i32, i32, i32, i32, i64, i32, vp, vp],
     "ksana_gemm_smallm_w4": [vp, i32, vp, vp, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, vp, i64, vp, i32, vp, vp],
     "ksana_w4_gemv": [vp, i64, vp, vp, vp, vp, vp, i64, vp, i64, i32, i32, i32, i32, vp],
@@ -592,6 +599,10 @@ _ACTS = {"silu": 0, "swiglu": 0, "gelu": 1, "gelu_new": 1, "gelu_pytorch_tanh": 
 def act_mul(x, act="silu", gated=True, out=None, quant=False, q=None, s=None, want_out=True):
     M = x.shape[0]
     inter = x.shape[1] // 2 if gated else x.shape[1]
+    if x.dtype == torch.float32:
+        out = torch.empty(M, inter, dtype=x.dtype, device=x.device)
+        _check(lib().ksana_act_mul_f32(_p(x), _p(out), M, inter, x.stride(0), _ACTS[act], int(gated), _st()), "ksana_act_mul_f32")
+        return out
     if want_out and out is None:
         out = torch.empty(M, inter, dtype=torch.bfloat16, device=x.device)
     if quant:
@@ -695,17 +706,25 @@ def embed_pair(ids, prev, table, pair, scale, buckets=0, mul_prev=0, mul_cur=0, 
 
 
 def residual_norm(x, H, eps, y=None, w1=None, b1=None, ls=None, x_out=None, w2=None, b2=None, z=None, rows=None, rms=False,
-                  alpha=1.0, groups=1):
+                  alpha=1.0, groups=1, add=None, vec=None, z_scale=1.0, experts=None):
     """One pass over rows of the fp32 stream ``x`` (``H`` real columns, padded to a multiple of 8):
-    x' = x + alpha * ls * norm(y; w1, b1), stored to ``x_out``; z = norm(x'; w2, b2), or a copy of x' without ``w2``. Parts
-    whose arguments are None are left out; ``rows`` gathers stream rows. ``groups`` > 1: the stream's norm (RMS, without
-    ``w1``) is taken for each of that many equal parts of a row."""
+    x' = x + alpha * ls * norm(y; w1, b1) + add + vec, stored to ``x_out``; z = z_scale * norm(x'; w2, b2), or a copy of x'
+    without ``w2``. Parts whose arguments are None are left out; ``rows`` gathers stream rows. ``groups`` > 1: the stream's
+    norm (RMS, without ``w1``) is taken for each of that many equal parts of a row. ``add``: fp32 rows like x, ``vec``: one
+    row of the activations' type. ``experts`` = (dst_row [M, K], weights [M, K or K + 1], shared or None): y are expert outputs
+    and a row's addend is the sum of weights[k] * y[dst_row[k]] (+ weights[K] * shared)."""
     M = rows.numel() if rows is not None else x.shape[0]
-    t = z if z is not None else y
+    t = z if z is not None else y if y is not None else vec
+    dst_row, w, shared = experts if experts is not None else (None, None, None)
+    top = dst_row.numel() // max(M, 1) if dst_row is not None else 0
+    assert add is None or (add.dtype == torch.float32 and add.stride(0) == x.stride(0))
     _check(lib().ksana_residual_norm(_p(x), x.stride(0), _p(rows), x.shape[0], _p(y), y.stride(0) if y is not None else 0, _p(w1),
                                      _p(b1), _p(ls), _p(x_out), _p(w2), _p(b2), _p(z), z.stride(0) if z is not None else 0, M, H,
-                                     float(eps), int(rms), int(t.dtype == torch.float32), float(alpha), int(groups),
-                                     _p(err_flag(x.device)), _st()), "ksana_residual_norm")
+                                     float(eps), int(rms), int(t is None or t.dtype == torch.float32), float(alpha), int(groups),
+                                     _p(add), _p(vec), float(z_scale), _p(dst_row), _p(w), w.stride(0) if w is not None else 0, top,
+                                     y.shape[0] if dst_row is not None else 0, _p(shared),
+                                     shared.stride(0) if shared is not None else 0, _p(err_flag(x.device)), _st()),
+           "ksana_residual_norm")
 
 
 def glu_clamp(x, limit, alpha, offset):
@@ -821,13 +840,14 @@ def paged_decode(q, q_stride, out, cache_layer, block_stride, block_tokens, bloc
 
 
 def attention_f32(q, q_stride, out, k_cache, v_cache, block_tokens, block_table, cu_q, kv_lens, B, max_q_len, Hq, Hkv, scale,
-                  window=0, keep=0, sinks=None):
+                  window=0, keep=0, sinks=None, gate=None):
     """All of a step's new rows (any lengths) against K and V panels, in 32-bit arithmetic throughout (bf16 storage is fine).
-    ``v_cache`` may be a column range of ``k_cache``."""
+    ``v_cache`` may be a column range of ``k_cache``. ``gate`` [rows, heads]: outputs are multiplied by its sigmoid."""
+    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1)
     rc = lib().ksana_attention_f32(_p(q), q_stride, _p(out), out.stride(0), _p(k_cache), _p(v_cache), v_cache.stride(-2),
                                    k_cache.stride(0), block_tokens, k_cache.shape[0], _p(block_table), block_table.stride(0),
-                                   _p(cu_q), _p(kv_lens), _p(sinks), B, max_q_len, Hq, Hkv, k_cache.shape[-1], v_cache.shape[-1],
-                                   window, keep, float(scale), int(q.dtype == torch.float32), _p(err_flag(q.device)), _st())
+                                   _p(cu_q), _p(kv_lens), _p(sinks), _p(gate), gate.stride(0) if gate is not None else 0, B, max_q_len,
+                                   Hq, Hkv, k_cache.shape[-1], v_cache.shape[-1], window, keep, float(scale), int(q.dtype == torch.float32), _p(err_flag(q.device)), _st())
     _check(rc, "ksana_attention_f32")
 
 
@@ -840,6 +860,33 @@ def qkv_rope_append(qkv, positions, slots, cos_sin, k_cache, v_cache, block_toke
                                      k_cache.shape[-1], v_cache.shape[-1], rot_dim, int(qkv.dtype == torch.float32),
                                      _p(err_flag(qkv.device)), _st())
     _check(rc, "ksana_qkv_rope_append")
+
+
+def qkv_norm_rope_append(qkv, positions, slots, cos_sin, qw, kw, eps, nq, nk, k_cache, v_cache, block_tokens, Hq, Hkv, rot_dim,
+                         sums=None):
+    """Root-mean-square norms over all of q (``nq`` real columns) and all of k (``nk``) of a row, rotation of the pairs (2i,
+    2i + 1) of the first ``rot_dim`` dimensions of every head, q in place, k and v to their paged panels. ``sums`` [T, 2]: sums of
+    squares of the whole rows where ``qkv`` holds a part of them."""
+    T = qkv.shape[0]
+    assert sums is None or (sums.dtype == torch.float32 and sums.is_contiguous())
+    rc = lib().ksana_qkv_norm_rope_append(
+        _p(qkv), _p(positions), _p(slots), _p(cos_sin), cos_sin.shape[0] if cos_sin is not None else 0, _p(qw), _p(kw), float(eps), nq, nk,
+        _p(sums), _p(k_cache), _p(v_cache), k_cache.stride(0), block_tokens, k_cache.shape[0], T, Hq, Hkv, k_cache.shape[-1],
+        v_cache.shape[-1], rot_dim, int(qkv.dtype == torch.float32), _p(err_flag(qkv.device)), _st())
+    _check(rc, "ksana_qkv_norm_rope_append")
+
+
+def latent_norms(q, kv, q_w, kv_w, eps, q_rank, kv_rank, slots, cache, block_tokens):
+    """Root-mean-square norms of the query latents ``q`` [T, q_rank padded] (returned) and of the key/value latents ``kv`` [T,
+    kv_rank padded] (into the paged panel ``cache`` [blocks, block tokens, kv_rank padded]); both are column ranges of the same
+    rows."""
+    T = q.shape[0]
+    assert q.stride() == kv.stride() and q.stride(1) == 1 and cache.stride(1) == cache.shape[2] == kv.shape[1]
+    out = torch.empty(T, q.shape[1], dtype=q.dtype, device=q.device)
+    _check(lib().ksana_latent_norms(_p(q), _p(kv), q.stride(0), _p(q_w), _p(kv_w), float(eps), _p(out), q_rank, kv_rank, _p(slots),
+                                    _p(cache), cache.stride(0), block_tokens, int(cache.shape[0]) * block_tokens, T,
+                                    int(q.dtype == torch.float32), _p(err_flag(q.device)), _st()), "ksana_latent_norms")
+    return out
 
 
 def mla_rope_append(q, nope, kv, norm_w, eps, positions, slots, cos_sin, qfull, cache, block_tokens, G, rank):
@@ -870,10 +917,14 @@ def mla_splits(num_seqs: int, max_q_len: int, max_kv: int, sms: int = 148, halve
     return best
 
 
-def mla_attention(qfull, out, cache, block_tokens, block_table, cu_q, kv_lens, B, max_q_len, scale, nsplit=1, window=0) -> bool:
+def mla_attention(qfull, out, cache, block_tokens, block_table, cu_q, kv_lens, B, max_q_len, scale, nsplit=1, window=0,
+                  sinks=None, gate=None) -> bool:
     """Absorbed multi-head latent attention on tcgen05 (see csrc/kernels/mla_attention.cu). qfull [T, G, DK], cache: latent
-    panel [blocks, block tokens, DK], out [T, G, DV] (values are the leading DV columns of the cache rows). Returns False
-    when the kernel does not cover the configuration."""
+    panel [blocks, block tokens, DK], out [T, G, DV] (values are the leading DV columns of the cache rows). ``sinks`` [G]: logits
+    that only enter the denominator, ``gate`` [T, G]: outputs are multiplied by its sigmoid. Returns False when the kernel does
+    not cover the configuration."""
+    assert gate is None or (gate.dtype == torch.bfloat16 and gate.stride(1) == 1)
+    assert sinks is None or sinks.dtype == torch.float32
     T, G, dk = qfull.shape
     dv = out.shape[2]
     assert qfull.is_contiguous() and out.stride(2) == 1 and out.stride(1) == dv and cache.stride(1) == dk == cache.shape[2]
@@ -882,8 +933,8 @@ def mla_attention(qfull, out, cache, block_tokens, block_table, cu_q, kv_lens, B
         po = torch.empty(nsplit * T * G * dv, dtype=torch.float32, device=qfull.device)
         pml = torch.empty(nsplit * T * G * 2, dtype=torch.float32, device=qfull.device)
     rc = lib().ksana_mla_attention(_p(qfull), T, _p(out), out.stride(0), _p(cache), cache.stride(0), block_tokens, _p(block_table),
-                                   block_table.stride(0), _p(cu_q), _p(kv_lens), B, max_q_len, G, dk, dv, window, float(scale),
-                                   int(cache.shape[0]), nsplit, _p(po), _p(pml), _p(err_flag(qfull.device)), _st())
+                                   block_table.stride(0), _p(cu_q), _p(kv_lens), B, max_q_len, G, dk, dv, window, _p(sinks), _p(gate),
+                                   gate.stride(0) if gate is not None else 0, float(scale), int(cache.shape[0]), nsplit, _p(po), _p(pml), _p(err_flag(qfull.device)), _st())
     if rc == -100:
         return False
     _check(rc, "ksana_mla_attention")
@@ -954,6 +1005,11 @@ def ban_tokens(logits, offsets, ids, row_idx=None):
 def gemm_grouped(a, w, tile_expert, E, N, out=None, a_scale=None, w_scale=None, bn=0):
     """Expert-major rows of ``a`` [cap, K] (128-row tiles, one expert each) times stacked W [E*N, K]."""
     cap, K = a.shape
+    if a.dtype == torch.float32:
+        out = torch.empty(cap, N, dtype=a.dtype, device=a.device)
+        _check(lib().ksana_gemm_grouped_f32(_p(a), a.stride(0), _p(w), w.stride(0), _p(out), out.stride(0), cap, N, K, E,
+                                            _p(tile_expert), _st()), "ksana_gemm_grouped_f32")
+        return out
     kind = 0 if a_scale is None else 1
     if out is None:
         out = torch.empty(cap, N, dtype=torch.bfloat16, device=a.device)
@@ -964,12 +1020,14 @@ def gemm_grouped(a, w, tile_expert, E, N, out=None, a_scale=None, w_scale=None, 
     return out
 
 
-def moe_route(logits, K, scoring="softmax", renorm=True, scale=1.0, bias=None, n_group=1, topk_group=1):
-    T, E = logits.shape
+def moe_route(logits, K, scoring="softmax", renorm=True, scale=1.0, bias=None, n_group=1, topk_group=1, E=None, gate_col=-1):
+    """Expert choice by rows of router logits (the first ``E`` columns of fp32 rows): (ids [T, K] int32, weights fp32 [T, K], or
+    [T, K + 1] with ``gate_col``: the sigmoid of that column comes last)."""
+    T, E = logits.shape[0], logits.shape[1] if E is None else E
     ids = torch.empty(T, K, dtype=torch.int32, device=logits.device)
-    w = torch.empty(T, K, dtype=torch.float32, device=logits.device)
-    rc = lib().ksana_moe_route(_p(logits), _p(bias), _p(ids), _p(w), T, E, K, 0 if scoring == "softmax" else 1,
-                               int(renorm), float(scale), n_group, topk_group, _st())
+    w = torch.empty(T, K + (gate_col >= 0), dtype=torch.float32, device=logits.device)
+    rc = lib().ksana_moe_route(_p(logits), logits.stride(0), _p(bias), _p(ids), _p(w), w.stride(0), T, E, K,
+                               0 if scoring == "softmax" else 1, int(renorm), float(scale), n_group, topk_group, gate_col, _st())
     _check(rc, "ksana_moe_route")
     return ids, w
 
@@ -992,8 +1050,9 @@ def moe_align(topk_ids, E, expert_lo=0, expert_hi=None):
 def moe_permute(x, dst_row, K, cap, zero=False):
     """``zero``: padding rows are zero instead of undefined (for consumers that reduce over the whole tensor)."""
     T, H = x.shape
-    perm = (torch.zeros if zero else torch.empty)(cap, H, dtype=torch.bfloat16, device=x.device)
-    _check(lib().ksana_moe_permute(_p(x), _p(dst_row), _p(perm), T, K, H, cap, _p(err_flag(x.device)), _st()),
+    perm = (torch.zeros if zero else torch.empty)(cap, H, dtype=x.dtype, device=x.device)
+    units = H * x.element_size() // 2                                        # the kernel moves 16-bit units
+    _check(lib().ksana_moe_permute(_p(x), _p(dst_row), _p(perm), T, K, units, cap, _p(err_flag(x.device)), _st()),
            "ksana_moe_permute")
     return perm
 

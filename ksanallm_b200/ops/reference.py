@@ -349,6 +349,61 @@ def qkv_rope_append(qkv, positions, slots, cos_sin, k_cache, v_cache, block_toke
     v_cache[blk, :, off] = v[ok].to(v_cache.dtype)
 
 
+def qkv_norm_rope_append(qkv, positions, slots, cos_sin, qw, kw, eps, nq, nk, k_cache, v_cache, block_tokens, Hq, Hkv, rot_dim,
+                         sums=None):
+    """In place on q of qkv [T, Hq*D + Hkv*D + Hkv*Dv], k and v into panels; see native.qkv_norm_rope_append."""
+    T, D, Dv = qkv.shape[0], k_cache.shape[-1], v_cache.shape[-1]
+    q, k = qkv[:, :Hq * D].float(), qkv[:, Hq * D:(Hq + Hkv) * D].float()
+    sq, sk = (q.pow(2).sum(-1), k.pow(2).sum(-1)) if sums is None else sums.unbind(1)
+    q = (q * torch.rsqrt(sq / nq + eps).unsqueeze(1) * qw.float()).view(T, Hq, D)
+    k = (k * torch.rsqrt(sk / nk + eps).unsqueeze(1) * kw.float()).view(T, Hkv, D)
+    if rot_dim:
+        q = apply_rope(q, positions, cos_sin, rot_dim, neox=False)
+        k = apply_rope(k, positions, cos_sin, rot_dim, neox=False)
+    qkv[:, :Hq * D] = q.reshape(T, Hq * D).to(qkv.dtype)
+    ok = slots >= 0
+    blk, off = slots[ok].long() // block_tokens, slots[ok].long() % block_tokens
+    k_cache[blk, :, off] = k[ok].to(k_cache.dtype)
+    v_cache[blk, :, off] = qkv[:, (Hq + Hkv) * D:].reshape(T, Hkv, Dv)[ok].to(v_cache.dtype)
+
+
+def latent_norms(q, kv, q_w, kv_w, eps, q_rank, kv_rank, slots, cache, block_tokens):
+    def normed(x, w, n):
+        f = x.float()
+        return f * torch.rsqrt(f.pow(2).sum(-1, keepdim=True) / n + eps) * w.float()
+    ok = slots >= 0
+    sl = slots[ok].long()
+    cache[sl // block_tokens, sl % block_tokens] = normed(kv, kv_w, kv_rank)[ok].to(cache.dtype)
+    return normed(q, q_w, q_rank).to(q.dtype)
+
+
+def moe_route(logits, K, scoring="softmax", renorm=True, scale=1.0, bias=None, n_group=1, topk_group=1, E=None, gate_col=-1):
+    """(ids [T, K] int64, weights fp32 [T, K (+ 1)]); see native.moe_route."""
+    z = logits[:, :logits.shape[1] if E is None else E].float()
+    score = torch.sigmoid(z) if scoring == "sigmoid" else torch.softmax(z, dim=-1)
+    sel = score + (bias.float() if bias is not None else 0.0)
+    if n_group > 1 and topk_group < n_group:
+        grp = sel.unflatten(-1, (n_group, -1))
+        gscore = grp.topk(min(2, grp.shape[-1]), dim=-1).values.sum(-1)
+        keep = torch.zeros_like(gscore, dtype=torch.bool).scatter_(1, gscore.topk(topk_group, dim=-1).indices, True)
+        sel = grp.masked_fill(~keep.unsqueeze(-1), float("-inf")).flatten(-2)
+    ids = sel.topk(K, dim=-1).indices
+    w = score.gather(1, ids)
+    if renorm:
+        w = w / w.sum(-1, keepdim=True).clamp_min(1e-20)
+    w = w * scale
+    if gate_col >= 0:
+        w = torch.cat([w, torch.sigmoid(logits[:, gate_col:gate_col + 1].float())], 1)
+    return ids, w
+
+
+def expert_sum(y, dst_row, w, shared=None):
+    """fp32 rows: sum over k of w[t, k] * y[dst_row[t, k]] (negative: left out), plus w[t, K] * shared[t]."""
+    rows = y.float()[dst_row.clamp_min(0).long()] * (dst_row >= 0).unsqueeze(-1)
+    out = (rows * w[:, :dst_row.shape[1], None]).sum(1)
+    return out if shared is None else out + shared.float() * w[:, dst_row.shape[1], None]
+
+
 def panel_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, Hq, Hkv, scale, window=0, keep=0, sinks=None):
     """q [T, Hq*D] (new tokens only) -> [T, Hq*Dv]; see the sliding window and sink in dispatch.panel_attention."""
     T, G, D, Dv, bt = q.shape[0], Hq // Hkv, k_cache.shape[-1], v_cache.shape[-1], k_cache.shape[2]
@@ -454,9 +509,10 @@ def gemm_nvfp4(aq, a_bs, a_ts, wq, w_bs, w_ts, bias=None, residual=None, out_dty
     return y.to(out_dtype)
 
 
-def mla_attention(qfull, cache_layer, block_table, cu_q, kv_lens, scale, lora=512, window=0):
+def mla_attention(qfull, cache_layer, block_table, cu_q, kv_lens, scale, lora=512, window=0, sinks=None, gate=None):
     """Absorbed multi-head latent attention, plain fp32 statement. qfull [T, G, lora+rope] (q_lat | q_pe),
-    cache_layer [blocks, block_tokens, lora+rope] (c_kv | k_pe). Returns [T, G, lora] fp32."""
+    cache_layer [blocks, block_tokens, lora+rope] (c_kv | k_pe). Returns [T, G, lora] fp32. ``sinks`` [G]: logits in the
+    denominator only, ``gate`` [T, G]: outputs are multiplied by its sigmoid."""
     T, G, _ = qfull.shape
     bt = cache_layer.shape[1]
     out = torch.zeros(T, G, lora, dtype=torch.float32, device=qfull.device)
@@ -471,8 +527,11 @@ def mla_attention(qfull, cache_layer, block_table, cu_q, kv_lens, scale, lora=51
         qpos = torch.arange(kl - (q1 - q0), kl, device=qfull.device).unsqueeze(1)
         kpos = torch.arange(kl, device=qfull.device).unsqueeze(0)
         hide = (kpos > qpos) | (qpos - kpos >= window) if window > 0 else kpos > qpos
-        out[q0:q1] = torch.einsum("hqk,kl->qhl", torch.softmax(sc.masked_fill(hide, float("-inf")), -1), rows[:, :lora])
-    return out
+        sc = sc.masked_fill(hide, float("-inf"))
+        if sinks is not None:
+            sc = torch.cat([sc, sinks.float().view(G, 1, 1).expand(-1, q1 - q0, 1)], dim=-1)
+        out[q0:q1] = torch.einsum("hqk,kl->qhl", torch.softmax(sc, -1)[..., :kl], rows[:, :lora])
+    return out if gate is None else out * torch.sigmoid(gate.float()).unsqueeze(-1)
 
 
 # ----------------------------------------------------------------------------- 4-bit weight-only groups (W4A16)
