@@ -112,10 +112,11 @@ class StreamModel(CommonModel):
         return self.lm_head_forward(self.forward_layers(step), step)
 
     def lm_head_forward(self, x: torch.Tensor, step: StepInput):
-        if step.want_hidden:
-            self.step_hidden, self.step_normed = x, ops.stream_norm(x, self.final, self.dtype)
         # the factor of the logits goes into their GEMM's operand
-        return self.logits_or_candidates(ops.stream_norm(x, self.final, self.dtype, rows=step.logits_rows, scale=self.cfg.logit_scale), step)
+        scale = self.cfg.logit_scale
+        if step.want_hidden:
+            self.step_hidden, self.step_normed = x, ops.stream_norm(x, self.final, self.dtype, scale=scale)
+        return self.logits_or_candidates(ops.stream_norm(x, self.final, self.dtype, rows=step.logits_rows, scale=scale), step)
 
 
 class StreamLoader:

@@ -399,7 +399,7 @@ def moe_route(logits, K, scoring="softmax", renorm=True, scale=1.0, bias=None, n
 
 def expert_sum(y, dst_row, w, shared=None):
     """fp32 rows: sum over k of w[t, k] * y[dst_row[t, k]] (negative: left out), plus w[t, K] * shared[t]."""
-    rows = y.float()[dst_row.clamp_min(0).long()] * (dst_row >= 0).unsqueeze(-1)
+    rows = y.float()[dst_row.clamp_min(0).long()].masked_fill((dst_row < 0).unsqueeze(-1), 0.0)
     out = (rows * w[:, :dst_row.shape[1], None]).sum(1)
     return out if shared is None else out + shared.float() * w[:, dst_row.shape[1], None]
 

@@ -41,14 +41,16 @@ def rotate(x, position, dims, base):
 def attend(q, k, v, scale, sink=None):
     """One head: q, k [T, d], v [T, dv]; a row sees itself and all earlier ones. ``sink``: a logit that takes its share of
     the weights and gives nothing."""
-    out = []
-    for i in range(q.shape[0]):
-        s = (k[:i + 1] @ q[i]) * scale
-        top = s.max() if sink is None else torch.maximum(s.max(), sink)
-        p = torch.exp(s - top)
-        total = p.sum() if sink is None else p.sum() + torch.exp(sink - top)
-        out.append((p / total) @ v[:i + 1])
-    return torch.stack(out)
+    s = (q @ k.t()) * scale
+    s = s.masked_fill(torch.ones(s.shape, dtype=torch.bool).triu(1), float("-inf"))
+    top = s.max(-1, keepdim=True).values
+    if sink is not None:
+        top = torch.clamp(top, min=float(sink))
+    p = torch.exp(s - top)
+    total = p.sum(-1, keepdim=True)
+    if sink is not None:
+        total = total + torch.exp(sink - top)
+    return (p / total) @ v
 
 
 def attention(h, m, w, pre, eps):

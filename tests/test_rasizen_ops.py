@@ -7,37 +7,11 @@ import pytest
 import torch
 
 import rasizen_oracle as oracle
-from decoder_helpers import PLACES
+from decoder_helpers import PLACES, close, make_step, pad, rand, TOL, up8
 from ksanallm_b200.models.common import RecordLayout
 from ksanallm_b200.ops import dispatch as ops
 from ksanallm_b200.ops import native
 from ksanallm_b200.ops import reference as ref
-
-TOL = {torch.float32: 2e-5, torch.bfloat16: 2e-2}
-rand = lambda seed, *s: torch.randn(*s, generator=torch.Generator().manual_seed(seed)).bfloat16().float()  # noqa: E731
-pad = lambda t, n: torch.nn.functional.pad(t, (0, n - t.shape[-1]))  # noqa: E731
-up8 = lambda n: (n + 7) // 8 * 8  # noqa: E731
-
-
-def close(got, want, dtype, scale=None):
-    got, want = got.float().cpu(), want.float()
-    s = scale if scale is not None else max(1.0, float(want.abs().max()))
-    assert torch.isfinite(got).all()
-    assert float((got - want).abs().max()) <= TOL[dtype] * s, float((got - want).abs().max()) / s
-
-
-def make_step(lens, tables, bt, device):
-    """Step of sequences (cached, new), multi-token ones first; ``tables``: block ids (of bt tokens) per sequence."""
-    news = [n for _, n in lens]
-    cu = torch.tensor([0] + news).cumsum(0).to(torch.int32)
-    multi = sum(n > 1 for n in news)
-    width = max(len(t) for t in tables) + 1
-    table = torch.tensor([list(t) + [0] * (width - len(t)) for t in tables], dtype=torch.int32)
-    kv = torch.tensor([p + n for p, n in lens], dtype=torch.int32)
-    slots = torch.tensor([tables[s][t // bt] * bt + t % bt for s, (p, n) in enumerate(lens) for t in range(p, p + n)], dtype=torch.int32)
-    return SimpleNamespace(slots=slots.to(device), block_table=table.to(device), cu_q=cu.to(device), kv_lens=kv.to(device), num_multi=multi,
-                           num_single=len(news) - multi, num_multi_tokens=int(cu[multi]), max_q_len=max(news), max_kv_len=int(kv.max()))
-
 
 # ------------------------------------------------------------------------------------------------ norms and units
 @pytest.mark.parametrize("device,dtype", PLACES)
