@@ -1,5 +1,5 @@
 """Throughput of a design whose layers are configured one by one beside the framework's closest existing model at equal
-sizes, kernel by kernel: the loop that benchmarks/lenolix_bench.py and benchmarks/rasizen_bench.py share.
+sizes, kernel by kernel: the loop that the benchmarks/<design>_bench.py files share.
 
 Per size, one JSON line: device time and tokens/s of one prefill step and one decode step of every variant (CUDA graphs,
 CUDA events, median of several replays; the weights of the layers are larger than L2), and every kernel class with its
@@ -65,9 +65,9 @@ def common_cost(n, a):
 
 def run(args, design, sizes, describe, variants, cost, base, mine, timed_only=(), match=None):
     """``variants(size)``: name -> function giving the variant's ModelConfig; ``base`` and ``mine``: the variants whose kernels
-    are compared; ``timed_only``: variants without a kernel table; ``match``: job of the design -> job of the base model
-    where the names differ. A GEMM without a counterpart of its own shape is compared with the base model's GEMMs
-    together."""
+    are compared (``base`` may be several names: a job is compared with the first that has it); ``timed_only``: variants
+    without a kernel table; ``match``: job of the design -> job of the base model where the names differ. A GEMM without a
+    counterpart of its own shape is compared with the base models' GEMMs together."""
     import torch
 
     from benchmarks.step_breakdown import run_breakdown
@@ -118,10 +118,12 @@ def run(args, design, sizes, describe, variants, cost, base, mine, timed_only=()
             return sum(map(total, rows)) / sum(total(c) / c["distance"] for c in rows)
 
         for phase, _, _ in phases:
-            a, b, like = tables[(mine, phase)], tables[(base, phase)], {}
+            bases = [tables[(name, phase)] for name in ([base] if isinstance(base, str) else base)]
+            a, like = tables[(mine, phase)], {}
             for job in dict.fromkeys(c["job"] for c in a):
                 x = distance(a, job)
-                y = distance(b, (match or {}).get(job, job)) or (gemms(b) if job.startswith("gemm ") else None)
+                y = next((d for b in bases if (d := distance(b, (match or {}).get(job, job)))), None)
+                y = y or (gemms([c for b in bases for c in b]) if job.startswith("gemm ") else None)
                 if x and y:
                     like[job] = round(x / y, 2)
             out["results"][phase]["like"] = like

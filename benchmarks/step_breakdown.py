@@ -5,7 +5,8 @@ arguments). The whole graph is then replayed and timed with CUDA events, and so 
 (entry point + its integer arguments, which separates the four GEMM shapes of a layer) holding only that class's
 launches in their original order. Because a class graph replays the launches of all layers back to back, each
 layer reading its own weights and cache, its time per launch includes the launch-to-launch cost inside a graph and
-sees a cold L2, like the real step. The sum over classes against the time of the full graph shows what the
+sees a cold L2, like the real step. Integer arguments (block tables, expert rows) keep their memory to themselves, so they
+still hold the step's values when a class is replayed alone. The sum over classes against the time of the full graph shows what the
 dependency chain itself costs.
 
   python benchmarks/step_breakdown.py --phase decode --batch 64 --ctx 2176                  (one GPU, TP1 shapes)

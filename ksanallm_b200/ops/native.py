@@ -115,6 +115,7 @@ def available() -> bool:
 
 
 _recorder = None
+_recorded_tensors: list = []              # integer arguments seen while recording: their memory is not given to anyone else
 
 
 class _RecordingLib:
@@ -144,6 +145,7 @@ class recording:
     def __enter__(self):
         global _recorder
         _recorder = self.calls
+        _recorded_tensors.clear()
         return self.calls
 
     def __exit__(self, *exc):
@@ -175,7 +177,11 @@ def _load():
 
 
 def _p(t: Optional[torch.Tensor]):
-    return None if t is None else t.data_ptr()
+    if t is None:
+        return None
+    if _recorder is not None and t.dtype == torch.int32:
+        _recorded_tensors.append(t)
+    return t.data_ptr()
 
 
 def _st():

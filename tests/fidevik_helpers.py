@@ -109,7 +109,7 @@ def weights(c, seed=0):
         elif name.endswith(("q.norm", "k.norm")) and "d" not in name.split(".")[-2]:
             t = 1.5 + 0.4 * t
         elif last == "down" and ".e" in name:
-            t = t * 0.12 / s[-1] ** 0.5
+            t = t * 0.05 / s[-1] ** 0.5
         elif len(s) == 2 and last != "embed":
             t = t * 1.2 / s[-1] ** 0.5
         elif len(s) == 1:                          # norm weights
