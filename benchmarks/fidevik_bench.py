@@ -112,6 +112,13 @@ def main(args):
         return {"width": W, "heads": H, "kv_heads": G, "dim": DIM, "q_rank": QR, "kv_rank": RANK, "ff": ff, "experts": EXPERTS, "top": TOP,
                 "expert_ff": xff, "shared_ff": sff}
 
+    def match():
+        """GEMMs of latent attention whose counterparts have other row counts: no rotated part, several projections in one."""
+        out = {}
+        for W, H, _, QR, _, _, _ in SIZES.values():
+            out.update({f"gemm {H * DIM}x{QR}": f"gemm {H * (DIM + 64)}x{QR}", f"gemm {QR + RANK + (H + 7) // 8 * 8}x{W}": f"gemm {QR}x{W}"})
+        return out
+
     batch = {"prefill": args.prefill_batch, "decode": args.decode_batch}
     return run(args, "fidevik", SIZES, describe, variants, cost(batch), ("deepseek", "qwen2_moe"), "fidevik", timed_only=("fidevik_loop",),
-               match={"norms, rotation": "rotation", "norm with expert sum": "combine", "norm alone": "norm"})
+               match={**match(), "norms, rotation": "rotation", "norm with expert sum": "combine", "norm alone": "norm"})

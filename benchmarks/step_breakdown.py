@@ -5,8 +5,8 @@ arguments). The whole graph is then replayed and timed with CUDA events, and so 
 (entry point + its integer arguments, which separates the four GEMM shapes of a layer) holding only that class's
 launches in their original order. Because a class graph replays the launches of all layers back to back, each
 layer reading its own weights and cache, its time per launch includes the launch-to-launch cost inside a graph and
-sees a cold L2, like the real step. Integer arguments (block tables, expert rows) keep their memory to themselves, so they
-still hold the step's values when a class is replayed alone. The sum over classes against the time of the full graph shows what the
+sees a cold L2, like the real step. No two tensors of the captured step share memory, so every argument (the
+experts' row numbers, for one) still holds the step's values when a class is replayed alone. The sum over classes against the time of the full graph shows what the
 dependency chain itself costs.
 
   python benchmarks/step_breakdown.py --phase decode --batch 64 --ctx 2176                  (one GPU, TP1 shapes)
@@ -112,7 +112,8 @@ def run_breakdown(model, phase="decode", batch=64, ctx=2176, q_len=2048, reps=10
         torch.cuda.synchronize()
         calls = []
         full = torch.cuda.CUDAGraph()
-        with native.recording(calls):
+        rec = native.recording(calls)                # holds the step's tensors
+        with rec:
             with torch.cuda.graph(full):
                 keep = model.forward(step)
         t_full = _time_graph(torch, full, reps, sync_all)
@@ -134,6 +135,7 @@ def run_breakdown(model, phase="decode", batch=64, ctx=2176, q_len=2048, reps=10
                 rows[-1].update(zip(("job", "bytes", "flops"), costs[key]))
             del g
         native.check_err_flag(model.device)
+        del rec
     s = sum(r["us_total"] for r in rows)
     return {"phase": phase, "batch": batch, "ctx": ctx if phase == "decode" else q_len, "native_launches": len(calls),
             "full_graph_us": round(t_full, 1), "sum_of_classes_us": round(s, 1), "classes": rows, "_keep": keep is not None}

@@ -170,7 +170,8 @@ __global__ void norm_kernel(const bf16* __restrict__ x, bf16* __restrict__ resid
 
 // ----------------------------------------------------------------------------
 // out[m, i] = act(gate_up[m, i]) * gate_up[m, I + i] ; optional fp8 copy. act: 0 silu 1 gelu(tanh) 2 relu
-// When `gated` is 0 the input is [M, I] and out = act(in).
+// When `gated` is 0 the input is [M, I] and out = act(in). tile_rows (may be null): of every 128 rows only so many hold
+// anything, the others are skipped.
 __device__ __forceinline__ float tanh_fast(float x) {
   float y;
   asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -190,16 +191,18 @@ __device__ __forceinline__ float act_fn(float x, int act) {
 }
 
 __global__ void act_mul_kernel(const bf16* __restrict__ in, bf16* __restrict__ out, uint8_t* __restrict__ outq,
-                               float* __restrict__ oscale, int scale_ld, int M, int I, int in_ld, int act, int gated) {
+                               float* __restrict__ oscale, int scale_ld, int M, int I, int in_ld, int act, int gated,
+                               const int* __restrict__ tile_rows) {
   pdl_trigger();
   pdl_wait();
   const int nvec = I >> 3;
   const long long total = static_cast<long long>(M) * nvec;
   for (long long idx = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x;
        idx < ((total + 31) / 32) * 32; idx += static_cast<long long>(gridDim.x) * blockDim.x) {
-    const bool on = idx < total;
+    bool on = idx < total;
     const int m = on ? static_cast<int>(idx / nvec) : 0;
     const int i = on ? static_cast<int>(idx % nvec) : 0;
+    if (tile_rows) on = on && (m & 127) < tile_rows[m >> 7];
     float o[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e) o[e] = 0.f;
@@ -674,13 +677,13 @@ extern "C" int ksana_norm(const void* x, void* residual, const void* w, const vo
 }
 
 extern "C" int ksana_act_mul(const void* in, void* out, void* outq, float* oscale, int scale_ld, int M, int I,
-                             int in_ld, int act, int gated, cudaStream_t st) {
+                             int in_ld, int act, int gated, const int* tile_rows, cudaStream_t st) {
   if (M <= 0) return 0;
   if (I % 8 || in_ld % 8) return -10;
   if (outq && (I % 128)) return -11;
   const long long total = static_cast<long long>(M) * (I >> 3);
   launch_pdl(act_mul_kernel, dim3(grid_for(total, 256)), dim3(256), 0, st, (const bf16*)in, (bf16*)out, (uint8_t*)outq, oscale, scale_ld, M,
-                                                       I, in_ld, act, gated);
+                                                       I, in_ld, act, gated, tile_rows);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

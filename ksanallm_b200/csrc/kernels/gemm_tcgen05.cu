@@ -49,6 +49,7 @@ struct GemmParams {
   // grouped (mixture-of-experts) mode: row tile i multiplies with expert tile_expert[i] (< 0: tile unused);
   // W stacks the experts as [E * expert_rows, K] and w_scale as [E * scale_rows_per_expert][K/128].
   const int* tile_expert;
+  const int* tile_rows;   // rows of each row tile that hold anything (null: all); the others are not stored
   int expert_rows;
   int scale_rows_per_expert;
   // push mode (tensor-parallel row-parallel linear): rows [r*push_rows, (r+1)*push_rows) of the partial
@@ -241,7 +242,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_cons
         if (expert < 0) continue;
       }
       const int row = m0 + q * 32 + lane;
-      const bool row_ok = row < p.M;
+      const bool row_ok = row < p.M && (!p.tile_rows || q * 32 + lane < p.tile_rows[m_blk]);
 
       // the gate's columns of one 32-column chunk of this row, fetched a chunk ahead of their use
       auto fetch_gate = [&](int c0, uint4 (&g)[4]) {
@@ -440,7 +441,18 @@ static int pick_bn(int M, int N, int kind, int bn_hint) {
   const int cands_bf16[4] = {256, 128, 64, 32};
   const int* c = cands_bf16;
   const int nc = 4;
-  (void)kind;
+  if (kind == kBf16) {
+    // a wave costs about the same for every width (operand latency; measured: 9.7 us at 32 columns, 15 us at 256 with
+    // K = 2048), so the fewest waves win, and among equal numbers the narrower tile
+    int best = c[0];
+    long long best_cost = -1;
+    for (int i = 0; i < nc; ++i) {
+      const long long tiles = static_cast<long long>(m_tiles) * ((N + c[i] - 1) / c[i]);
+      const long long cost = (tiles + sms - 1) / sms * (400 + c[i]);
+      if (best_cost < 0 || cost < best_cost) { best = c[i]; best_cost = cost; }
+    }
+    return best;
+  }
   for (int i = 0; i < nc; ++i) {
     const int tiles = m_tiles * ((N + c[i] - 1) / c[i]);
     if (tiles >= sms) return c[i];   // at least one full wave with the widest tile that allows it
@@ -603,11 +615,13 @@ extern "C" int ksana_gemm_fp8_block_push(const void* Aq, int lda, const float* a
 }
 
 // Grouped GEMM for mixture-of-experts: rows of A are expert-major (each expert's segment padded to a
-// multiple of 128 rows), tile_expert[m_tile] names the expert of every 128-row tile (-1 = unused).
+// multiple of 128 rows), tile_expert[m_tile] names the expert of every 128-row tile (-1 = unused), tile_rows[m_tile]
+// (may be null) how many of its rows are stored.
 // W: [E*N, K]; w_scale (fp8): [E * ceil(N/128)][K/128]. kind 0 = bf16, 1 = block-scaled fp8.
 extern "C" int ksana_gemm_grouped(int kind, const void* A, int lda, const float* a_scale, int a_scale_ld, const void* W,
                                   int ldw, const float* w_scale, void* D, int ldd, int M_cap, int N, int K, int E,
-                                  const int* tile_expert, int bn_hint, int* err_flag, cudaStream_t stream) {
+                                  const int* tile_expert, const int* tile_rows, int bn_hint, int* err_flag,
+                                  cudaStream_t stream) {
   if (M_cap <= 0 || N <= 0 || K <= 0 || E <= 0) return 0;
   const int esz = kind == kBf16 ? 2 : 1;
   if ((N % 8) || (K % (kind == kBf16 ? 8 : 128)) || (lda % (16 / esz)) || (ldw % (16 / esz)) || (ldd % 8) || (M_cap % 128)) return -10;
@@ -621,7 +635,7 @@ extern "C" int ksana_gemm_grouped(int kind, const void* A, int lda, const float*
   p.D = static_cast<__nv_bfloat16*>(D); p.ldd = ldd;
   p.a_scale = a_scale; p.a_scale_ld = a_scale_ld; p.w_scale = w_scale;
   p.err = err_flag;
-  p.tile_expert = tile_expert; p.expert_rows = N; p.scale_rows_per_expert = (N + 127) / 128;
+  p.tile_expert = tile_expert; p.tile_rows = tile_rows; p.expert_rows = N; p.scale_rows_per_expert = (N + 127) / 128;
   if (kind == kBf16) {
     switch (bn) {
       case 256: return launch_gemm<256, kBf16>(ma, mb, p, 0, stream);

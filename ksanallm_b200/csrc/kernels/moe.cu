@@ -110,11 +110,11 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ldl, cons
   }
 }
 
-// Single CTA. counts -> padded offsets (multiples of 128) -> tile_expert[] (-1 for unused tiles) and
-// dst_row[T*K]. `total_rows[0]` receives the padded row count.
+// Single CTA. counts -> padded offsets (multiples of 128) -> tile_expert[] (-1 for unused tiles), tile_rows[] (rows of
+// a tile that hold a token) and dst_row[T*K]. `total_rows[0]` receives the padded row count.
 __global__ void moe_align_kernel(const int* __restrict__ topk_ids, int* __restrict__ dst_row,
-                                 int* __restrict__ tile_expert, int* __restrict__ expert_offsets,
-                                 int* __restrict__ total_rows, int TK, int E, int max_tiles, int expert_lo,
+                                 int* __restrict__ tile_expert, int* __restrict__ tile_rows,
+                                 int* __restrict__ expert_offsets, int* __restrict__ total_rows, int TK, int E, int max_tiles, int expert_lo,
                                  int expert_hi, int* err) {
   __shared__ int cnt[kMaxExperts];
   __shared__ int off[kMaxExperts + 1];
@@ -149,6 +149,7 @@ __global__ void moe_align_kernel(const int* __restrict__ topk_ids, int* __restri
       if (r >= off[e] + ((cnt[e] + 127) / 128) * 128) e = -1;
     }
     tile_expert[t] = e;
+    tile_rows[t] = e < 0 ? 0 : min(128, off[e] + cnt[e] - r);
   }
   __syncthreads();
   for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
@@ -222,11 +223,11 @@ extern "C" int ksana_moe_route(const float* logits, int ldl, const float* bias, 
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
-extern "C" int ksana_moe_align(const int* topk_ids, int* dst_row, int* tile_expert, int* expert_offsets,
+extern "C" int ksana_moe_align(const int* topk_ids, int* dst_row, int* tile_expert, int* tile_rows, int* expert_offsets,
                                int* total_rows, int TK, int E, int max_tiles, int expert_lo, int expert_hi, int* err,
                                cudaStream_t st) {
   if (E > kMaxExperts) return -10;
-  moe_align_kernel<<<1, 1024, 0, st>>>(topk_ids, dst_row, tile_expert, expert_offsets, total_rows, TK, E, max_tiles,
+  moe_align_kernel<<<1, 1024, 0, st>>>(topk_ids, dst_row, tile_expert, tile_rows, expert_offsets, total_rows, TK, E, max_tiles,
                                        expert_lo, expert_hi, err);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

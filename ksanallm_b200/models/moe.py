@@ -161,10 +161,11 @@ def route_reference(logits, cfg: ModelConfig, bias=None):
                          cfg.n_group, cfg.topk_group)
 
 
-def dense_experts(perm, w13, w2, tile_expert, n_local, inter, act):
+def dense_experts(perm, w13, w2, tile_expert, tile_rows, n_local, inter, act):
     """Expert-major rows through their experts' gate|up and down matrices (stacked [E * 2I, H] and [E * H, I], bf16 or fp32)."""
-    g = native.gemm_grouped(perm, w13, tile_expert, n_local, 2 * inter)
-    return native.gemm_grouped(native.act_mul(g, act, True), w2, tile_expert, n_local, perm.shape[1])
+    g = native.gemm_grouped(perm, w13, tile_expert, n_local, 2 * inter, tile_rows=tile_rows)
+    a = native.act_mul(g, act, True, tile_rows=tile_rows)
+    return native.gemm_grouped(a, w2, tile_expert, n_local, perm.shape[1], tile_rows=tile_rows)
 
 
 def expert_outputs(x, ids, w13, w2, inter, act="silu"):
@@ -172,8 +173,8 @@ def expert_outputs(x, ids, w13, w2, inter, act="silu"):
     T, K = ids.shape
     E = w2.shape[0] // x.shape[1]
     if x.is_cuda:
-        dst_row, tile_expert, _, _, cap = native.moe_align(ids, E)
-        return dense_experts(native.moe_permute(x, dst_row, K, cap), w13, w2, tile_expert, E, inter, act), dst_row.view(T, K)
+        dst_row, tile_expert, _, _, cap, tile_rows = native.moe_align(ids, E)
+        return dense_experts(native.moe_permute(x, dst_row, K, cap), w13, w2, tile_expert, tile_rows, E, inter, act), dst_row.view(T, K)
     y = torch.zeros(T * K, x.shape[1], dtype=x.dtype)
     for e in range(E):
         tok, slot = (ids == e).nonzero(as_tuple=True)
@@ -240,7 +241,7 @@ def moe_partial(model, mw: MoEWeights, x: torch.Tensor, into: Optional[torch.Ten
     n_local = mw.expert_hi - mw.expert_lo
     if x.is_cuda:
         ids, w = routing if routing is not None else route(model, mw, x)
-        dst_row, tile_expert, _, _, cap = native.moe_align(ids, E, mw.expert_lo, mw.expert_hi)
+        dst_row, tile_expert, _, _, cap, tile_rows = native.moe_align(ids, E, mw.expert_lo, mw.expert_hi)
         if mw.expert_lo:
             tile_expert = torch.where(tile_expert >= 0, tile_expert - mw.expert_lo, tile_expert)
         perm = native.moe_permute(x, dst_row, K, cap, zero=mw.nvfp4)
@@ -256,11 +257,12 @@ def moe_partial(model, mw: MoEWeights, x: torch.Tensor, into: Optional[torch.Ten
             y = native.gemm_grouped_nvfp4(aq, abs_, a_ts2, mw.w2, mw.w2_bs, mw.w2_ts, tile_expert, n_local, H)
         elif mw.w13_scale is not None:
             pq, ps = native.quant_fp8(perm)
-            g = native.gemm_grouped(pq, mw.w13, tile_expert, n_local, 2 * mw.inter, a_scale=ps, w_scale=mw.w13_scale)
+            g = native.gemm_grouped(pq, mw.w13, tile_expert, n_local, 2 * mw.inter, a_scale=ps, w_scale=mw.w13_scale,
+                                    tile_rows=tile_rows)
             _, aq, as_ = native.act_mul(g, cfg.activation, True, quant=True, want_out=False)
-            y = native.gemm_grouped(aq, mw.w2, tile_expert, n_local, H, a_scale=as_, w_scale=mw.w2_scale)
+            y = native.gemm_grouped(aq, mw.w2, tile_expert, n_local, H, a_scale=as_, w_scale=mw.w2_scale, tile_rows=tile_rows)
         else:
-            y = dense_experts(perm, mw.w13, mw.w2, tile_expert, n_local, mw.inter, cfg.activation)
+            y = dense_experts(perm, mw.w13, mw.w2, tile_expert, tile_rows, n_local, mw.inter, cfg.activation)
         out = into if into is not None else torch.empty(T, H, dtype=x.dtype, device=x.device)
         have_shared = shared and mw.shared_gate_up is not None
         if have_shared:

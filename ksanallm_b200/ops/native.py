@@ -34,9 +34,9 @@ _SIGS = {
     "ksana_gemm_fp8_block": [vp, i32, vp, i32, vp, i32, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp],
     "ksana_gemm_smallm": [i32, vp, i32, vp, i32, vp, i32, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32, vp, i64, vp, i32,
                           vp, vp],
-    "ksana_gemm_grouped": [i32, vp, i32, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, vp, i32, vp, vp],
+    "ksana_gemm_grouped": [i32, vp, i32, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, vp, vp, i32, vp, vp],
     "ksana_moe_route": [vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32, f32, i32, i32, i32, vp],
-    "ksana_moe_align": [vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
+    "ksana_moe_align": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
     "ksana_moe_permute": [vp, vp, vp, i32, i32, i32, i32, vp, vp],
     "ksana_moe_combine": [vp, vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
     "ksana_gemm_smallm_push": [i32, vp, i32, vp, i32, vp, i32, vp, i32, vp, i32, i32, i32, vp, i64, vp, i32, vp, i32, vp, vp],
@@ -51,7 +51,7 @@ _SIGS = {
     "ksana_allreduce_nvls": [vp, vp, i32, i32, vp, C.c_ulonglong, i64, vp, vp, i64, vp, vp],
     "ksana_allgather_pull": [vp, vp, i32, i32, vp, i64, vp, i32, i32, i32, i32, vp, vp],
     "ksana_norm": [vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, f32, i32, vp],
-    "ksana_act_mul": [vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
+    "ksana_act_mul": [vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp],
     "ksana_act_mul_f32": [vp, vp, i32, i32, i32, i32, i32, vp],
     "ksana_quant_fp8": [vp, vp, vp, i32, i32, i32, i32, vp],
     "ksana_embedding": [vp, vp, vp, vp, vp, i32, i32, i32, i32, f32, vp],
@@ -115,7 +115,7 @@ def available() -> bool:
 
 
 _recorder = None
-_recorded_tensors: list = []              # integer arguments seen while recording: their memory is not given to anyone else
+_recorded_tensors: list = []              # arguments seen while recording: their memory is not given to anyone else
 
 
 class _RecordingLib:
@@ -151,6 +151,8 @@ class recording:
     def __exit__(self, *exc):
         global _recorder
         _recorder = None
+        self.tensors = list(_recorded_tensors)
+        _recorded_tensors.clear()
         return False
 
 
@@ -179,7 +181,7 @@ def _load():
 def _p(t: Optional[torch.Tensor]):
     if t is None:
         return None
-    if _recorder is not None and t.dtype == torch.int32:
+    if _recorder is not None:
         _recorded_tensors.append(t)
     return t.data_ptr()
 
@@ -602,7 +604,8 @@ def norm(x, w, eps, residual=None, beta=None, out=None, layernorm=False, quant=F
 _ACTS = {"silu": 0, "swiglu": 0, "gelu": 1, "gelu_new": 1, "gelu_pytorch_tanh": 1, "relu": 2}
 
 
-def act_mul(x, act="silu", gated=True, out=None, quant=False, q=None, s=None, want_out=True):
+def act_mul(x, act="silu", gated=True, out=None, quant=False, q=None, s=None, want_out=True, tile_rows=None):
+    """``tile_rows``: of every 128 rows only so many hold anything (expert-major rows); the others are skipped."""
     M = x.shape[0]
     inter = x.shape[1] // 2 if gated else x.shape[1]
     if x.dtype == torch.float32:
@@ -617,7 +620,7 @@ def act_mul(x, act="silu", gated=True, out=None, quant=False, q=None, s=None, wa
         if s is None:
             s = torch.empty(inter // 128, max(4, (M + 3) // 4 * 4), dtype=torch.float32, device=x.device)
     rc = lib().ksana_act_mul(_p(x), _p(out) if want_out else None, _p(q) if quant else None, _p(s) if quant else None,
-                             s.stride(0) if quant else 0, M, inter, x.stride(0), _ACTS[act], int(gated), _st())
+                             s.stride(0) if quant else 0, M, inter, x.stride(0), _ACTS[act], int(gated), _p(tile_rows), _st())
     _check(rc, "ksana_act_mul")
     return (out, q, s) if quant else out
 
@@ -1008,9 +1011,13 @@ def ban_tokens(logits, offsets, ids, row_idx=None):
 
 
 # --------------------------------------------------------------------------- mixture of experts
-def gemm_grouped(a, w, tile_expert, E, N, out=None, a_scale=None, w_scale=None, bn=0):
-    """Expert-major rows of ``a`` [cap, K] (128-row tiles, one expert each) times stacked W [E*N, K]."""
+def gemm_grouped(a, w, tile_expert, E, N, out=None, a_scale=None, w_scale=None, bn=0, tile_rows=None):
+    """Expert-major rows of ``a`` [cap, K] (128-row tiles, one expert each) times stacked W [E*N, K]. ``tile_rows``: rows of every
+    tile that hold anything; the others need not be stored (worth it where tiles are mostly empty; with full ones, reading the counts
+    only sets the CTAs apart that share operand tiles in L2, up to twice the time)."""
     cap, K = a.shape
+    if cap > 191 * E:                  # more than 64 rows per expert on average
+        tile_rows = None
     if a.dtype == torch.float32:
         out = torch.empty(cap, N, dtype=a.dtype, device=a.device)
         _check(lib().ksana_gemm_grouped_f32(_p(a), a.stride(0), _p(w), w.stride(0), _p(out), out.stride(0), cap, N, K, E,
@@ -1021,7 +1028,7 @@ def gemm_grouped(a, w, tile_expert, E, N, out=None, a_scale=None, w_scale=None, 
         out = torch.empty(cap, N, dtype=torch.bfloat16, device=a.device)
     rc = lib().ksana_gemm_grouped(kind, _p(a), a.stride(0), _p(a_scale), a_scale.stride(0) if a_scale is not None else 0,
                                   _p(w), w.stride(0), _p(w_scale), _p(out), out.stride(0), cap, N, K, E,
-                                  _p(tile_expert), bn, _p(err_flag(a.device)), _st())
+                                  _p(tile_expert), _p(tile_rows), bn, _p(err_flag(a.device)), _st())
     _check(rc, "ksana_gemm_grouped")
     return out
 
@@ -1039,18 +1046,21 @@ def moe_route(logits, K, scoring="softmax", renorm=True, scale=1.0, bias=None, n
 
 
 def moe_align(topk_ids, E, expert_lo=0, expert_hi=None):
+    """(destination row of every (token, choice), expert of every 128-row tile, row offsets of the experts, padded row count,
+    capacity in rows, rows of every tile that hold a token)."""
     TK = topk_ids.numel()
     hi = E if expert_hi is None else expert_hi
     max_tiles = (TK + (hi - expert_lo) * 127 + 127) // 128
     dev = topk_ids.device
     dst_row = torch.empty(TK, dtype=torch.int32, device=dev)
     tile_expert = torch.empty(max_tiles, dtype=torch.int32, device=dev)
+    tile_rows = torch.empty_like(tile_expert)
     offsets = torch.empty(E + 1, dtype=torch.int32, device=dev)
     total = torch.empty(1, dtype=torch.int32, device=dev)
-    rc = lib().ksana_moe_align(_p(topk_ids), _p(dst_row), _p(tile_expert), _p(offsets), _p(total), TK, E, max_tiles,
+    rc = lib().ksana_moe_align(_p(topk_ids), _p(dst_row), _p(tile_expert), _p(tile_rows), _p(offsets), _p(total), TK, E, max_tiles,
                                expert_lo, hi, _p(err_flag(dev)), _st())
     _check(rc, "ksana_moe_align")
-    return dst_row, tile_expert, offsets, total, max_tiles * 128
+    return dst_row, tile_expert, offsets, total, max_tiles * 128, tile_rows
 
 
 def moe_permute(x, dst_row, K, cap, zero=False):

@@ -33,21 +33,26 @@ def test_route(E, K, scoring, groups):
 
 
 @pytest.mark.parametrize("quant", [False, True])
-def test_grouped_moe_pipeline(quant):
+@pytest.mark.parametrize("T", [300, 150])
+def test_grouped_moe_pipeline(T, quant):
     torch.manual_seed(1)
-    T, H, I, E, K = 300, 512, 256, 8, 2
+    H, I, E, K = 512, 256, 8, 2
     x = torch.randn(T, H, device=DEV, dtype=torch.bfloat16)
     w13 = torch.randn(E * 2 * I, H, device=DEV) * 0.05
     w2 = torch.randn(E * H, I, device=DEV) * 0.05
     logits = torch.randn(T, E, device=DEV)
     ids, w = native.moe_route(logits, K, "softmax", True, 1.0)
-    dst_row, tile_expert, offsets, total, cap = native.moe_align(ids, E)
+    dst_row, tile_expert, offsets, total, cap, tile_rows = native.moe_align(ids, E)
     # every (token,k) row is unique, lands in its expert's segment
     rows = dst_row.long()
     assert rows.unique().numel() == T * K
     off = offsets.long()
     e_of_row = torch.bucketize(rows, off[1:], right=True)
     assert torch.equal(e_of_row, ids.long().reshape(-1))
+    assert int(tile_rows.sum()) == T * K and bool((tile_rows[tile_expert < 0] == 0).all())
+    tile_of = torch.zeros(tile_rows.numel(), 128, dtype=torch.bool, device=DEV)
+    tile_of.view(-1)[rows] = True                  # tokens fill the rows of a tile from its start
+    assert torch.equal(tile_of, torch.arange(128, device=DEV) < tile_rows.unsqueeze(1))
     perm = native.moe_permute(x, dst_row, K, cap)
     assert torch.equal(perm[rows], x.repeat_interleave(K, 0))
     if quant:
@@ -61,9 +66,13 @@ def test_grouped_moe_pipeline(quant):
         w13d, w2d = ref.dequant_weight_fp8_block(w13q, w13s), ref.dequant_weight_fp8_block(w2q, w2s)
         tol = 6e-2
     else:
-        g = native.gemm_grouped(perm, w13.to(torch.bfloat16), tile_expert, E, 2 * I)
-        a = native.act_mul(g, "silu", True)
-        y = native.gemm_grouped(a, w2.to(torch.bfloat16), tile_expert, E, H)
+        g, y = (torch.full((cap, n), 7.0, dtype=torch.bfloat16, device=DEV) for n in (2 * I, H))
+        native.gemm_grouped(perm, w13.to(torch.bfloat16), tile_expert, E, 2 * I, out=g, tile_rows=tile_rows)
+        a = native.act_mul(g, "silu", True, tile_rows=tile_rows)
+        native.gemm_grouped(a, w2.to(torch.bfloat16), tile_expert, E, H, out=y, tile_rows=tile_rows)
+        if T == 150:                               # mostly empty tiles: rows without a token are not written
+            empty = ~tile_of.view(-1)
+            assert bool((g[empty] == 7).all()) and bool((y[empty] == 7).all())
         w13d, w2d = w13.to(torch.bfloat16).float(), w2.to(torch.bfloat16).float()
         tol = 2e-2
     out = torch.zeros(T, H, device=DEV, dtype=torch.bfloat16)
