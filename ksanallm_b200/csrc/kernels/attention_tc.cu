@@ -2,8 +2,8 @@
 // against the paged KV cache, head sizes up to 128 (query/key and value sizes may differ; both padded with zeros in shared
 // memory only), bf16 cache, optionally a sliding window with kept first tokens and a per-head sink logit.
 //
-// One CTA owns 128 packed query rows of one KV head group: row = (token, head inside the group), so the G query
-// heads that share a KV head reuse every staged K/V tile (G must divide 128). Per 128-token KV tile:
+// One CTA owns up to 128 packed query rows of one KV head group: row = (token, head inside the group), so the G query
+// heads that share a KV head reuse every staged K/V tile (whole tokens only: 128 / G of them, the rows behind stay idle). Per 128-token KV tile:
 //   S = Q K^T      tcgen05.mma, both operands K-major in shared memory (TMA, 128-byte swizzle), S in TMEM
 //   softmax        4 warps, one thread per row (TMEM lane): no cross-thread reductions; online max with a
 //                  lazy rescale of O (only when a row's maximum grew by more than 2^8)
@@ -40,6 +40,7 @@ struct FaParams {
   const int* cu_q; const int* kv_lens; const float* alibi;
   const float* sinks;                        // [Hq] logits added to the softmax denominator, or null
   int Hq, Hkv, G, block_tokens;
+  int rows;                                  // query rows of a CTA: the largest multiple of G up to 128
   int D, Dv;                                 // real head sizes
   int window, keep;                          // sliding window in tokens (0: none), first tokens every row sees
   float scale_log2;
@@ -80,10 +81,10 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
   const int q0 = p.cu_q[s], q_len = p.cu_q[s + 1] - q0;
   const int kv_len = p.kv_lens[s];
   const int qtile = static_cast<int>(gridDim.x) - 1 - static_cast<int>(blockIdx.x);   // longest rows first
-  const int row0 = qtile * kFaTile;
+  const int row0 = qtile * p.rows;
   if (row0 >= q_len * G) return;
   const int past = kv_len - q_len;
-  const int last_row = min(row0 + kFaTile - 1, q_len * G - 1);
+  const int last_row = min(row0 + p.rows - 1, q_len * G - 1);
   const int kv_end = min(kv_len, past + last_row / G + 1);
   // tiles visited: those with kept first tokens, then from the first position in the window of this CTA's first row on
   const int first_lo = WIN ? past + row0 / G - p.window + 1 : 0;
@@ -113,7 +114,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       tma_prefetch_desc(&q_map);
       tma_prefetch_desc(&k_map);
       tma_prefetch_desc(&v_map);
-      mbar_expect_tx(q_full, kpanels * kFaPanelBytes);
+      mbar_expect_tx(q_full, kpanels * p.rows * 128);
       const int tok0 = q0 + row0 / G;
       for (int h = 0; h < kpanels; ++h) tma_load_3d(q_s + h * kFaPanelBytes, &q_map, q_full, h * 64, g * G, tok0);
       const int bt = p.block_tokens;
@@ -178,7 +179,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     const int qd = warp & 3;
     const uint32_t lane_off = static_cast<uint32_t>(qd * 32) << 16;
     const int vr = row0 + qd * 32 + lane;                  // packed row index inside the sequence
-    const bool active = vr < q_len * G;
+    const bool active = qd * 32 + lane < p.rows && vr < q_len * G;
     const int tok = vr / G, head = g * G + vr % G;
     const int limit = active ? past + tok : -1;            // last visible KV position
     const int lo = WIN ? limit - p.window + 1 : 0;            // first position inside the window
@@ -368,7 +369,7 @@ extern "C" int ksana_paged_prefill_tc(const void* q, long long q_stride, long lo
   if (D <= 0 || Dv <= 0 || D > kFaD || Dv > kFaD || D % 8 || Dv % 8 || Hkv <= 0 || Hq % Hkv) return -100;
   const int G = Hq / Hkv;
   const int bt = block_tokens;
-  if (G > 128 || kFaTile % G || !(bt == 8 || bt == 16 || bt == 32 || bt == 64 || bt == 128)) return -100;
+  if (G > kFaTile || !(bt == 8 || bt == 16 || bt == 32 || bt == 64 || bt == 128)) return -100;
   if (block_stride % 8 || num_blocks <= 0 || q_rows <= 0 || (out_stride % 8)) return -100;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kc) | reinterpret_cast<uintptr_t>(vc) |
        reinterpret_cast<uintptr_t>(out)) & 15 || (q_stride % 8)) return -100;
@@ -405,10 +406,10 @@ extern "C" int ksana_paged_prefill_tc(const void* q, long long q_stride, long lo
   p.out = static_cast<bf16*>(out); p.out_stride = out_stride;
   p.block_table = block_table; p.table_stride = table_stride; p.cu_q = cu_q; p.kv_lens = kv_lens; p.alibi = alibi;
   p.sinks = sinks; p.D = D; p.Dv = Dv; p.window = window; p.keep = window > 0 ? keep : 0;
-  p.Hq = Hq; p.Hkv = Hkv; p.G = G; p.block_tokens = bt;
+  p.Hq = Hq; p.Hkv = Hkv; p.G = G; p.block_tokens = bt; p.rows = kFaTile / G * G;
   p.scale_log2 = scale * 1.44269504f;
   p.err = err;
-  dim3 grid((max_q_len * G + kFaTile - 1) / kFaTile, Hkv, B);
+  dim3 grid((max_q_len * G + p.rows - 1) / p.rows, Hkv, B);
   if (window > 0) prefill_tc_kernel<true><<<grid, kFaThreads, kFaSmemBytes, st>>>(q_map, k_map, v_map, p);
   else prefill_tc_kernel<false><<<grid, kFaThreads, kFaSmemBytes, st>>>(q_map, k_map, v_map, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;

@@ -816,7 +816,7 @@ def paged_prefill(q, q_stride, out, cache_layer, block_stride, block_tokens, blo
     kc, vc, Dv = _panels(cache_layer, v_cache, D)
     nblocks = int(cache_layer.shape[0])
     if PREFILL_TC and not fp8 and max(D, Dv) <= 128:
-        # tcgen05 kernel (head sizes up to 128, bf16 cache, group size dividing 128); -100 = configuration not covered
+        # tcgen05 kernel (head sizes up to 128, bf16 cache, groups of up to 128 heads); -100 = configuration not covered
         rc = lib().ksana_paged_prefill_tc(_p(q), q_stride, q.shape[0], _p(out), out.stride(0), kc, vc, block_stride,
                                           block_tokens, _p(block_table), block_table.stride(0), _p(cu_q), _p(kv_lens),
                                           _p(alibi), _p(sinks), B, max_q_len, Hq, Hkv, D, Dv, window, keep, float(scale),
