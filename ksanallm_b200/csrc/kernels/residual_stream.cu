@@ -62,37 +62,19 @@ __global__ void embed_pair_kernel(const int* __restrict__ ids, const int* __rest
 }
 
 // ------------------------------------------------------------------------------------------------ norms
-// Running mean and sum of squared deviations of a set of values; two sets merge exactly (pairwise update), so a row's
-// statistics need one pass over the registers and one block reduction instead of two.
-struct Moments { float n, mean, m2; };
-__device__ __forceinline__ Moments merge(const Moments& a, const Moments& b) {
-  Moments r;
-  r.n = a.n + b.n;
-  if (r.n <= 0.f) return Moments{0.f, 0.f, 0.f};
-  const float inv = 1.f / r.n, d = b.mean - a.mean;
-  r.mean = (a.n * a.mean + b.n * b.mean) * inv;
-  r.m2 = a.m2 + b.m2 + d * d * (a.n * b.n * inv);
-  return r;
-}
-__device__ __forceinline__ Moments warp_moments(Moments v) {
+// Sum of v over the CTA, in every thread. `red`: 32 floats of shared memory, other ones for every sum of a kernel
+__device__ __forceinline__ float block_sum(float v, float* red) {
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    const Moments w{__shfl_xor_sync(0xffffffffu, v.n, o), __shfl_xor_sync(0xffffffffu, v.mean, o),
-                    __shfl_xor_sync(0xffffffffu, v.m2, o)};
-    v = merge(v, w);
-  }
-  return v;
-}
-// `red`: 32 entries of shared memory, different for the two reductions of a row
-__device__ __forceinline__ Moments block_moments(Moments v, Moments* red) {
-  v = warp_moments(v);
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
   const int nw = blockDim.x >> 5;
   if (nw == 1) return v;
   const int w = threadIdx.x >> 5, l = threadIdx.x & 31;
   if (l == 0) red[w] = v;
   __syncthreads();
-  v = l < nw ? red[l] : Moments{0.f, 0.f, 0.f};
-  return warp_moments(v);
+  v = l < nw ? red[l] : 0.f;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
 }
 
 template <typename T>
@@ -175,18 +157,30 @@ template <typename T, int VPT, bool EXPERTS>
 __global__ void residual_norm_kernel(const ResNormParams<T> p) {
   pdl_trigger();
   pdl_wait();
-  __shared__ Moments red[2][32];
-  __shared__ int src_row[EXPERTS ? kMaxTop : 1];
-  __shared__ float src_w[EXPERTS ? kMaxTop + 1 : 1];
+  __shared__ float red[4][32];
+  __shared__ int src_row[EXPERTS ? kMaxTop : 1], src_n;
+  __shared__ float src_w[EXPERTS ? kMaxTop : 1], shared_w;
   const int m = blockIdx.x;
   if (EXPERTS) {
-    for (int k = threadIdx.x; k < p.top; k += blockDim.x) {
-      int d = p.dst_row[static_cast<size_t>(m) * p.top + k];
-      if (d >= p.cap) { guard_report(p.err, kGuardDstRow, d); d = -1; }
-      src_row[k] = d;
-      src_w[k] = p.w[static_cast<size_t>(m) * p.ldw + k];
+    if (threadIdx.x < 32) {             // the rows that are here, in order, so that the loop over them has no branch
+      int n = 0;
+      for (int k0 = 0; k0 < p.top; k0 += 32) {
+        const int k = k0 + threadIdx.x;
+        int d = k < p.top ? p.dst_row[static_cast<size_t>(m) * p.top + k] : -1;
+        if (d >= p.cap) { guard_report(p.err, kGuardDstRow, d); d = -1; }
+        const unsigned here = __ballot_sync(0xffffffffu, d >= 0);
+        if (d >= 0) {
+          const int at = n + __popc(here & ((1u << threadIdx.x) - 1u));
+          src_row[at] = d;
+          src_w[at] = p.w[static_cast<size_t>(m) * p.ldw + k];
+        }
+        n += __popc(here);
+      }
+      if (threadIdx.x == 0) {
+        src_n = n;
+        if (p.shared) shared_w = p.w[static_cast<size_t>(m) * p.ldw + p.top];
+      }
     }
-    if (threadIdx.x == 0 && p.shared) src_w[p.top] = p.w[static_cast<size_t>(m) * p.ldw + p.top];
     __syncthreads();
   }
   int r = m;
@@ -207,11 +201,11 @@ __global__ void residual_norm_kernel(const ResNormParams<T> p) {
         if (p.shared) {
           load8(p.shared + static_cast<size_t>(r) * p.lds + i * 8, y[j]);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) y[j][e] *= src_w[p.top];
+          for (int e = 0; e < 8; ++e) y[j][e] *= shared_w;
         }
+        const int n = src_n;
 #pragma unroll 4
-        for (int k = 0; k < p.top; ++k) {
-          if (src_row[k] < 0) continue;
+        for (int k = 0; k < n; ++k) {
           float f[8];
           load8(p.y + static_cast<size_t>(src_row[k]) * p.ldy + i * 8, f);
 #pragma unroll
@@ -222,31 +216,34 @@ __global__ void residual_norm_kernel(const ResNormParams<T> p) {
       }
     }
   }
-  // statistics of the valid elements of f: (n, mean, m2), or for RMS (n, 0, sum of squares)
-  auto moments_of = [&](float (&f)[VPT][8], Moments* rd) {
-    Moments t{0.f, 0.f, 0.f};
+  // mean of the valid elements of f (RMS: 0) and reciprocal root of their mean squared distance from it; two sums, the
+  // second over the distances, so nothing cancels
+  auto statistics = [&](float (&f)[VPT][8], float (&rd)[4][32], int first, float& mean, float& rstd) {
+    mean = 0.f;
+    if (!p.rms) {
+      float s = 0.f;
+#pragma unroll
+      for (int j = 0; j < VPT; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        if (i < nvec) {
+          const int k = min(8, p.H - i * 8);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) s += e < k ? f[j][e] : 0.f;
+        }
+      }
+      mean = block_sum(s, rd[first]) / static_cast<float>(p.H);
+    }
     float s = 0.f;
 #pragma unroll
     for (int j = 0; j < VPT; ++j) {
       const int i = threadIdx.x + j * blockDim.x;
       if (i < nvec) {
         const int k = min(8, p.H - i * 8);
-        t.n += static_cast<float>(k);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) s += e < k ? f[j][e] : 0.f;
+        for (int e = 0; e < 8; ++e) { const float d = f[j][e] - mean; s += e < k ? d * d : 0.f; }
       }
     }
-    if (!p.rms && t.n > 0.f) t.mean = s / t.n;
-#pragma unroll
-    for (int j = 0; j < VPT; ++j) {
-      const int i = threadIdx.x + j * blockDim.x;
-      if (i < nvec) {
-        const int k = min(8, p.H - i * 8);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) { const float d = f[j][e] - t.mean; t.m2 += e < k ? d * d : 0.f; }
-      }
-    }
-    return block_moments(t, rd);
+    rstd = rsqrtf(block_sum(s, rd[first + 1]) / static_cast<float>(p.H) + p.eps);
   };
   auto affine = [&](float (&f)[8], int i, float mean, float rstd, const T* w, const T* b) {
     float wf[8];
@@ -262,11 +259,7 @@ __global__ void residual_norm_kernel(const ResNormParams<T> p) {
   };
   if (p.y) {
     float mean = 0.f, rstd = 1.f;
-    if (p.w1) {
-      const Moments s = moments_of(y, red[0]);
-      mean = s.mean;
-      rstd = rsqrtf(s.m2 / static_cast<float>(p.H) + p.eps);
-    }
+    if (p.w1) statistics(y, red, 0, mean, rstd);
 #pragma unroll
     for (int j = 0; j < VPT; ++j) {
       const int i = threadIdx.x + j * blockDim.x;
@@ -316,11 +309,7 @@ __global__ void residual_norm_kernel(const ResNormParams<T> p) {
     return;
   }
   float mean = 0.f, rstd = 1.f;
-  if (p.w2) {
-    const Moments s = moments_of(v, red[1]);
-    mean = s.mean;
-    rstd = rsqrtf(s.m2 / static_cast<float>(p.H) + p.eps);
-  }
+  if (p.w2) statistics(v, red, 2, mean, rstd);
 #pragma unroll
   for (int j = 0; j < VPT; ++j) {
     const int i = threadIdx.x + j * blockDim.x;
@@ -561,16 +550,25 @@ __global__ void qkv_norm_rope_append_kernel(const NormRopeParams<T> p) {
       const float r = i < nqv ? rq : rk;
 #pragma unroll
       for (int e = 0; e < 8; ++e) f[j][e] *= r * w[e];
-      const int h = i / d8, c = (i - h * d8) * 8;
+      const int h = i / d8, c = (i - h * d8) * 8, pr = c >> 1;
       if (c < p.rot) {
+        float co[4], si[4];
+        if ((p.rot & 7) == 0) {         // the same for all; table rows and their halves start on 16-byte boundaries
+          *reinterpret_cast<float4*>(co) = *reinterpret_cast<const float4*>(cs + pr);
+          *reinterpret_cast<float4*>(si) = *reinterpret_cast<const float4*>(cs + half + pr);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const bool on = pr + e < half;
+            co[e] = on ? cs[pr + e] : 1.f;
+            si[e] = on ? cs[half + pr + e] : 0.f;
+          }
+        }
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int pr = (c >> 1) + e;
-          if (pr < half) {
-            const float co = cs[pr], si = cs[half + pr], u = f[j][2 * e], v = f[j][2 * e + 1];
-            f[j][2 * e] = u * co - v * si;
-            f[j][2 * e + 1] = v * co + u * si;
-          }
+          const float u = f[j][2 * e], v = f[j][2 * e + 1];
+          f[j][2 * e] = u * co[e] - v * si[e];
+          f[j][2 * e + 1] = v * co[e] + u * si[e];
         }
       }
       store8(i < nqv ? row + static_cast<size_t>(i) * 8 : kdst + (h - p.Hq) * kh + c, f[j]);
@@ -588,26 +586,27 @@ static cudaError_t launch_norm_rope(const NormRopeParams<T>& p, int T_, cudaStre
   return cudaErrorInvalidValue;
 }
 
-// Root-mean-square norms of two column ranges of a row: the query latent (blockIdx.y 0) to q_out, the key/value latent
-// (blockIdx.y 1) to its place in the paged panel (slot < 0: a padding row, skipped). Sizes are rounded up to multiples of 8
-// in storage; pad columns and their weights are zero.
+// Root-mean-square norms of two column ranges of a row: the query latent to q_out, the key/value latent to its place in the
+// paged panel (slot < 0: a padding row, skipped). One warp per row and range. Sizes are rounded up to multiples of 8 in
+// storage; pad columns and their weights are zero.
 template <typename T>
 struct LatentNormsParams {
   const T* q; const T* kv; long long ld;
   const T* qw; const T* kvw; float eps;
   T* q_out; int q_rank, kv_rank;
   const int* slots; T* cache; long long block_stride; int block_tokens; long long num_slots;
+  int rows;
   int* err;
 };
-constexpr int kLnThreads = 128;
+constexpr int kLnWarps = 4;
 
 template <typename T>
-__global__ void __launch_bounds__(kLnThreads) latent_norms_kernel(const LatentNormsParams<T> p) {
+__global__ void __launch_bounds__(32 * kLnWarps) latent_norms_kernel(const LatentNormsParams<T> p) {
   pdl_trigger();
   pdl_wait();
-  __shared__ float red[kLnThreads / 32];
-  const int t = blockIdx.x;
-  const bool is_q = blockIdx.y == 0;
+  const int lane = threadIdx.x & 31, unit = blockIdx.x * kLnWarps + (threadIdx.x >> 5), t = unit >> 1;
+  if (t >= p.rows) return;
+  const bool is_q = (unit & 1) == 0;
   const int n = is_q ? p.q_rank : p.kv_rank, np = (n + 7) / 8 * 8;
   const T* src = (is_q ? p.q : p.kv) + static_cast<size_t>(t) * p.ld;
   const T* w = is_q ? p.qw : p.kvw;
@@ -617,21 +616,21 @@ __global__ void __launch_bounds__(kLnThreads) latent_norms_kernel(const LatentNo
   } else {
     const int slot = p.slots[t];
     if (slot < 0) return;
-    if (slot >= p.num_slots) { if (threadIdx.x == 0) guard_report(p.err, kGuardSlot, slot); return; }
+    if (slot >= p.num_slots) { if (lane == 0) guard_report(p.err, kGuardSlot, slot); return; }
     dst = p.cache + static_cast<size_t>(slot / p.block_tokens) * p.block_stride + static_cast<size_t>(slot % p.block_tokens) * np;
   }
-  constexpr int kKeep = 2;              // vectors per thread that stay in registers between the two passes
+  constexpr int kKeep = 6;              // vectors per lane that stay in registers between the two passes
   float keep[kKeep][8], ss = 0.f;
 #pragma unroll
   for (int j = 0; j < kKeep; ++j) {
-    const int i = (threadIdx.x + j * kLnThreads) * 8;
+    const int i = (lane + j * 32) * 8;
     if (i < np) {
       load8(src + i, keep[j]);
 #pragma unroll
       for (int e = 0; e < 8; ++e) ss = fmaf(keep[j][e], keep[j][e], ss);
     }
   }
-  for (int i = (threadIdx.x + kKeep * kLnThreads) * 8; i < np; i += kLnThreads * 8) {
+  for (int i = (lane + kKeep * 32) * 8; i < np; i += 32 * 8) {
     float f[8];
     load8(src + i, f);
 #pragma unroll
@@ -639,11 +638,6 @@ __global__ void __launch_bounds__(kLnThreads) latent_norms_kernel(const LatentNo
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
-  __syncthreads();
-  ss = 0.f;
-#pragma unroll
-  for (int k = 0; k < kLnThreads / 32; ++k) ss += red[k];
   const float r = rsqrtf(ss / static_cast<float>(n) + p.eps);
   auto put = [&](int i, float (&f)[8]) {
     float g[8];
@@ -654,10 +648,10 @@ __global__ void __launch_bounds__(kLnThreads) latent_norms_kernel(const LatentNo
   };
 #pragma unroll
   for (int j = 0; j < kKeep; ++j) {
-    const int i = (threadIdx.x + j * kLnThreads) * 8;
+    const int i = (lane + j * 32) * 8;
     if (i < np) put(i, keep[j]);
   }
-  for (int i = (threadIdx.x + kKeep * kLnThreads) * 8; i < np; i += kLnThreads * 8) {
+  for (int i = (lane + kKeep * 32) * 8; i < np; i += 32 * 8) {
     float f[8];
     load8(src + i, f);
     put(i, f);
@@ -795,7 +789,7 @@ extern "C" int ksana_qkv_norm_rope_append(void* qkv, const int* positions, const
   if (T <= 0) return 0;
   if (Hq <= 0 || Hkv <= 0 || D <= 0 || Dv <= 0 || D % 8 || Dv % 8 || rot < 0 || rot > D || (rot & 1) || block_tokens <= 0 ||
       block_stride % 8 || (rot && !cos_sin) || !qw || !kw || nq <= 0 || nk <= 0 || (Hq + Hkv) * (D / 8) > 4096) return -10;
-  if (!aligned16(qkv) || !aligned16(kc) || !aligned16(vc) || !aligned16(qw) || !aligned16(kw)) return -11;
+  if (!aligned16(qkv) || !aligned16(kc) || !aligned16(vc) || !aligned16(qw) || !aligned16(kw) || !aligned16(cos_sin)) return -11;
   auto entry = f32 ? norm_rope_entry<float> : norm_rope_entry<bf16>;
   return entry(qkv, positions, slots, cos_sin, max_pos, qw, kw, eps, nq, nk, sums, kc, vc, block_stride, block_tokens, num_blocks, T, Hq,
                Hkv, D, Dv, rot, err, st) == cudaSuccess ? 0 : -4;
@@ -806,8 +800,8 @@ static cudaError_t latent_norms_entry(const void* q, const void* kv, long long l
                                       void* q_out, int q_rank, int kv_rank, const int* slots, void* cache, long long block_stride,
                                       int block_tokens, long long num_slots, int T_, int* err, cudaStream_t st) {
   const LatentNormsParams<T> p{(const T*)q, (const T*)kv, ld, (const T*)qw, (const T*)kvw, eps, (T*)q_out, q_rank, kv_rank, slots,
-                               (T*)cache, block_stride, block_tokens, num_slots, err};
-  return launch_pdl(latent_norms_kernel<T>, dim3(T_, 2), dim3(kLnThreads), 0, st, p);
+                               (T*)cache, block_stride, block_tokens, num_slots, T_, err};
+  return launch_pdl(latent_norms_kernel<T>, dim3((2 * T_ + kLnWarps - 1) / kLnWarps), dim3(32 * kLnWarps), 0, st, p);
 }
 
 // q, kv: column ranges of the same projection's rows, ld elements apart; q_out [T, q_rank rounded up to 8]
