@@ -6,8 +6,8 @@ weights:
 One JSON line per size (see benchmarks/design_bench.py). Every other layer is latent attention, the rest grouped-query
 attention; the first layer's feed-forward is dense, the others are mixtures of experts with a shared expert. Latent attention
 and the experts are compared with a DeepSeek model (same latent sizes, router and experts, latent attention in every layer),
-grouped-query attention with a Qwen2-MoE model (same heads, experts and shared expert's gate). A third variant repeats the
-middle third of the layers twice (the family's loop).
+grouped-query attention with a Qwen2-MoE model (same heads, experts and shared expert's gate). A further variant repeats the
+middle layers (half of eight) twice (the family's loop).
 """
 from __future__ import annotations
 
