@@ -13,6 +13,7 @@ from ksanallm_b200.ops import dispatch as ops
 from ksanallm_b200.ops import native
 from ksanallm_b200.ops import reference as ref
 
+
 # ------------------------------------------------------------------------------------------------ norms and units
 @pytest.mark.parametrize("device,dtype", PLACES)
 @pytest.mark.parametrize("H,groups", [(64, 1), (64, 2), (72, 3), (70, 5), (70, 70), (66, 2), (2048, 4), (2304, 9), (8192, 2), (9000, 1000)])
