@@ -59,7 +59,8 @@ def engine_lib_path() -> Path:
 
 # kernel sources that a family needs in bf16 or fp32 on one GPU (no FP8 / FP4 / 4-bit weights or peer memory)
 _STREAM_KERNELS = ("attention_f32", "elementwise", "gemm_f32", "gemm_smallm", "gemm_tcgen05", "residual_stream", "sampler")
-FAMILY_KERNELS = {"fidevik": _STREAM_KERNELS + ("attention", "attention_tc", "mla_attention", "moe"),
+FAMILY_KERNELS = {"fapudra": _STREAM_KERNELS + ("attention", "attention_tc", "moe", "state_scan", "stream_ops"),
+                  "fidevik": _STREAM_KERNELS + ("attention", "attention_tc", "mla_attention", "moe"),
                   "lenolix": _STREAM_KERNELS + ("attention", "attention_tc"),
                   "rasizen": _STREAM_KERNELS + ("mla_attention", "recurrence")}
 

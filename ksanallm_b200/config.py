@@ -213,6 +213,39 @@ class AttentionSpec:
     sink: bool = False                    # learned per-head logit in the softmax denominator
     rotary: Optional[RotarySpec] = None
     qk_norm: bool = False                 # root-mean-square norm of all of q (and of k) at once, before the rotation
+    sigmoid: bool = False                 # a key's weight is the sigmoid of its score; weights are not normalised over keys
+    bias_far: int = 0                     # > 0: learned biases by distance, logarithmic buckets that end at this distance
+
+
+@dataclass
+class StateSpaceSpec:
+    """Selective state space: per head a state of ``state`` x ``vdim`` with one decay, ``groups`` of heads share input and output
+    vectors; a short convolution in front, a gated norm of ``norm_groups`` parts behind."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    taps: int                             # of the short convolution
+    norm_groups: int = 1
+
+
+@dataclass
+class DeltaRuleSpec:
+    """Gated delta rule: per head a state of ``dim`` x ``vdim`` with a decay per key channel."""
+    heads: int
+    kv_heads: int                         # heads of q and k
+    dim: int
+    vdim: int
+    taps: int
+
+
+@dataclass
+class ParallelSpec:
+    """Attention and a recurrence that read the same input; their results are added with a factor each."""
+    attention: AttentionSpec
+    recurrence: DeltaRuleSpec
+    attention_scale: float
+    recurrence_scale: float
 
 
 @dataclass
@@ -269,20 +302,21 @@ class RouterSpec:
     scale: float = 1.0
     correction: bool = False              # learned per-expert offset that enters the choice, not the weights
     groups: int = 1                       # equal groups of neighbouring experts ...
-    keep_groups: int = 1                  # ... of which the best by the sum of their two largest choice scores stay
+    keep_groups: int = 1                  # ... of which the best by the sum of their largest choice scores stay:
+    group_top: int = 2                    # ... of how many
 
 
 @dataclass
 class MoeSpec:
     """Mixture of gated feed-forwards, and optionally one (``shared``) that every token goes through, with a gate."""
     router: RouterSpec
-    expert: GatedMlpSpec
+    expert: Union[GatedMlpSpec, MlpSpec]
     shared: Optional[GatedMlpSpec] = None
 
 
 @dataclass
 class LayerSpec:
-    mixer: Union[AttentionSpec, LatentAttentionSpec, GatedRecurrenceSpec]
+    mixer: Union[AttentionSpec, LatentAttentionSpec, GatedRecurrenceSpec, StateSpaceSpec, ParallelSpec]
     mlp: Optional[Union[MlpSpec, PlainMlpSpec, GatedMlpSpec, MoeSpec]]
 
 
@@ -372,6 +406,7 @@ class ModelConfig:
     norm_groups: int = 1                  # equal parts of a row that the norms treat one by one
     residual_mult: float = 1.0            # factor of every sublayer's result
     logit_scale: float = 1.0
+    logit_softcap: float = 0.0            # > 0: logits are cap * tanh(logits / cap)
 
     @property
     def is_moe(self) -> bool:
@@ -386,7 +421,7 @@ _ARCH_ALIASES = {
     "llama": "llama", "mistral": "llama", "qwen2": "qwen", "qwen": "qwen", "qwen2_vl": "qwen2_vl", "baichuan": "baichuan",
     "chatglm": "chatglm", "glm": "chatglm", "gpt2": "gpt", "openai-gpt": "gpt", "fairseq-transformer": "gpt", "mixtral": "mixtral",
     "qwen2_moe": "qwen2_moe", "deepseek_v3": "deepseek_v3", "deepseek_v2": "deepseek_v3", "internlm2": "llama",
-    "yi": "llama", "lenolix": "lenolix", "rasizen": "rasizen", "fidevik": "fidevik",
+    "yi": "llama", "lenolix": "lenolix", "rasizen": "rasizen", "fidevik": "fidevik", "fapudra": "fapudra",
 }
 # No position limit is part of the Lenolix, Rasizen and Fidevik designs: the serving configuration's max_token_len decides
 _UNBOUNDED_POSITIONS = 1 << 20
@@ -472,6 +507,8 @@ def model_config_from_hf(hf: dict, generation: Optional[dict] = None, model_dir:
         return rasizen_config(hf, generation)
     if arch == "fidevik":
         return fidevik_config(hf, generation)
+    if arch == "fapudra":
+        return fapudra_config(hf, generation)
     c = ModelConfig(model_type=arch, hf_model_type=mt)
     if arch == "gpt":
         c.hidden_size = hf.get("n_embd", hf.get("hidden_size", hf.get("decoder_embed_dim", 768)))
@@ -708,15 +745,19 @@ def _gated_mlp(m: dict, where: str, act: str) -> GatedMlpSpec:
     return GatedMlpSpec(_positive(m, "ff", where), act)
 
 
-def _moe(m: dict, where: str) -> MoeSpec:
-    r, at = m["router"], where + ".router"
+def _router(r: dict, at: str, **fixed) -> RouterSpec:
     groups = r.get("groups") or {"count": 1, "keep": 1}
-    router = RouterSpec(_positive(r, "experts", at), _positive(r, "top", at), scoring="sigmoid", correction=True,
-                        groups=_positive(groups, "count", at + ".groups"), keep_groups=_positive(groups, "keep", at + ".groups"))
+    router = RouterSpec(_positive(r, "experts", at), _positive(r, "top", at), groups=_positive(groups, "count", at + ".groups"),
+                        keep_groups=_positive(groups, "keep", at + ".groups"), **fixed)
     if router.experts % router.groups or router.keep_groups > router.groups:
         raise ValueError(f"{at}: {router.experts} experts, {router.keep_groups} of {router.groups} groups")
     if router.top > router.experts // router.groups * router.keep_groups:
         raise ValueError(f"{at}: {router.top} of the kept groups' experts cannot be chosen")
+    return router
+
+
+def _moe(m: dict, where: str) -> MoeSpec:
+    router = _router(m["router"], where + ".router", scoring="sigmoid", correction=True)
     return MoeSpec(router, _gated_mlp(m["expert"], where + ".expert", "silu"),
                    _gated_mlp(m["shared"], where + ".shared", "silu") if m.get("shared") else None)
 
@@ -757,6 +798,66 @@ def fidevik_config(hf: dict, generation: Optional[dict] = None) -> ModelConfig:
                     position_embedding="per_layer", layer_specs=layers, logit_scale=float(hf.get("logit_scale", 1.0)))
     c.loop = _loop(hf, len(layers))
     c.max_position_embeddings = c.max_token_len = int(hf.get("max_position_embeddings", _UNBOUNDED_POSITIONS))
+    c.eos_token_ids = _eos_ids(hf, generation)
+    return c
+
+
+def _divides(n: int, k: int, where: str, names: str) -> None:
+    if n % k:
+        raise ValueError(f"{where}: {names}: {n} does not divide by {k}")
+
+
+def _state_space(m: dict, where: str) -> StateSpaceSpec:
+    a = StateSpaceSpec(*(_positive(m, k, where) for k in ("heads", "vdim", "state", "groups", "conv")), int(m.get("norm_groups") or 1))
+    _divides(a.heads, a.groups, where, "heads and groups")
+    _divides(a.heads * a.vdim, a.norm_groups, where, "heads * vdim and norm_groups")
+    return a
+
+
+def _parallel(m: dict, where: str) -> ParallelSpec:
+    left, right, at = m["left"], m["right"], where + ".left"
+    a = AttentionSpec(*(_positive(left, k, at) for k in ("heads", "kv_heads", "dim", "vdim")), float(left["scale"]), sigmoid=True,
+                      bias_far=_positive(left, "bias_max", at))
+    _divides(a.heads, a.kv_heads, at, "heads and kv_heads")
+    if a.dim != a.vdim:
+        raise ValueError(f"{at}: the values are the keys, dim {a.dim} and vdim {a.vdim} must be equal")
+    mask = left.get("mask")
+    if mask:
+        a.window, a.keep_first = _positive(mask, "size", at + ".mask"), int(mask.get("keep_first") or 0)
+    at = where + ".right"
+    r = DeltaRuleSpec(*(_positive(right, k, at) for k in ("heads", "kv_heads", "dim", "vdim", "conv")))
+    _divides(r.heads, r.kv_heads, at, "heads and kv_heads")
+    return ParallelSpec(a, r, float(m["left_scale"]), float(m["right_scale"]))
+
+
+def fapudra_config(hf: dict, generation: Optional[dict] = None) -> ModelConfig:
+    """config.json of a Fapudra model: ``vocab``, ``width``, ``max_positions``, ``norm.eps``, ``embedding.scale``, ``logit_softcap``
+    and ``layers`` (``type``, ``mixer``, ``mlp``)."""
+    layers = []
+    for i, e in enumerate(hf["layers"]):
+        where = f"layers[{i}]"
+        parse = {"mamba2": _state_space, "parallel": _parallel}.get(e["type"])
+        if parse is None:
+            raise ValueError(f"{where}: unknown mixer type {e['type']!r}")
+        mixer, mlp, ff = parse(e["mixer"], where + ".mixer"), e.get("mlp"), None
+        if mlp:
+            if mlp.get("kind", "moe") != "moe":
+                raise ValueError(f"{where}: unknown feed-forward kind {mlp['kind']!r}")
+            at = where + ".mlp"
+            ff = MoeSpec(_router(mlp["router"], at + ".router", renorm=True, group_top=1),
+                         MlpSpec(_positive(mlp["expert"], "ff", at + ".expert"), float(mlp["expert"]["limit"])))
+        layers.append(LayerSpec(mixer, ff))
+    if not layers:
+        raise ValueError("layers is empty")
+    attn = [s.mixer.attention for s in layers if isinstance(s.mixer, ParallelSpec)]
+    first = attn[0] if attn else None
+    c = ModelConfig(model_type="fapudra", hf_model_type="fapudra", hidden_size=_positive(hf, "width", "config"), num_layers=len(layers),
+                    num_heads=first.heads if first else 1, num_kv_heads=first.kv_heads if first else 1,
+                    head_dim=first.dim if first else 1, v_head_dim=first.vdim if first else 0, intermediate_size=0,
+                    vocab_size=_positive(hf, "vocab", "config"), rms_norm_eps=float(hf["norm"]["eps"]), position_embedding="per_layer",
+                    emb_scale=float((hf.get("embedding") or {}).get("scale", 1.0)), layer_specs=layers,
+                    logit_softcap=float(hf.get("logit_softcap") or 0.0))
+    c.max_position_embeddings = c.max_token_len = _positive(hf, "max_positions", "config")
     c.eos_token_ids = _eos_ids(hf, generation)
     return c
 

@@ -175,8 +175,10 @@ PYBIND11_MODULE(_ksana_engine, m) {
       .def_readwrite("preempt_mode", &SchedulerConfig::preempt_mode)
       .def_readwrite("split_fuse_token_num", &SchedulerConfig::split_fuse_token_num)
       .def_readwrite("min_flexible_cache_num", &SchedulerConfig::min_flexible_cache_num)
+      .def_readwrite("num_state_slots", &SchedulerConfig::num_state_slots)
+      .def_readwrite("num_host_state_slots", &SchedulerConfig::num_host_state_slots)
       .def_readwrite("enable_prefix_cache", &SchedulerConfig::enable_prefix_cache)
-.def_readwrite("resume_at_block_ends", &SchedulerConfig::resume_at_block_ends)
+      .def_readwrite("resume_at_block_ends", &SchedulerConfig::resume_at_block_ends)
       .def_readwrite("block_token_num", &SchedulerConfig::block_token_num)
       .def_readwrite("auto_batch_wait_ms", &SchedulerConfig::auto_batch_wait_ms)
       .def_readwrite("eos_token_ids", &SchedulerConfig::eos_token_ids);
@@ -189,6 +191,16 @@ PYBIND11_MODULE(_ksana_engine, m) {
       .def_property_readonly("input_ids", [](const StepPlan& p) { return ToArray(p.input_ids); })
       .def_property_readonly("prev_ids", [](const StepPlan& p) { return ToArray(p.prev_ids); })
       .def_property_readonly("positions", [](const StepPlan& p) { return ToArray(p.positions); })
+      .def_property_readonly("state_slots", [](const StepPlan& p) { return ToArray(p.state_slots); })
+      .def_property_readonly("state_copies", [](const StepPlan& p) {
+        std::vector<int> v; for (auto& s : p.state_copies) { v.push_back(s.device_block); v.push_back(s.host_block); }
+        return ToArray(v); })
+      .def_property_readonly("state_out", [](const StepPlan& p) {
+        std::vector<int> v; for (auto& s : p.state_out) { v.push_back(s.device_block); v.push_back(s.host_block); }
+        return ToArray(v); })
+      .def_property_readonly("state_in", [](const StepPlan& p) {
+        std::vector<int> v; for (auto& s : p.state_in) { v.push_back(s.device_block); v.push_back(s.host_block); }
+        return ToArray(v); })
       .def_property_readonly("slots", [](const StepPlan& p) { return ToArray(p.slots); })
       .def_property_readonly("cu_q", [](const StepPlan& p) { return ToArray(p.cu_q); })
       .def_property_readonly("block_table", [](const StepPlan& p) { return ToArray(p.block_table); })

@@ -293,4 +293,15 @@ bool CacheManager::CheckInvariants(std::string* why) const {
   return true;
 }
 
+bool StateSlots::CheckInvariants(std::string* why) const {
+  std::vector<int> seen(in_use_.begin(), in_use_.end());
+  for (int id : free_) ++seen[id];
+  for (int id : released_) ++seen[id];
+  std::vector<int> host(host_in_use_.begin(), host_in_use_.end());
+  for (int id : host_free_) ++host[id];
+  for (int n : seen) if (n != 1) { *why = "a state slot is lost or held twice"; return false; }
+  for (int n : host) if (n != 1) { *why = "a host state slot is lost or held twice"; return false; }
+  return true;
+}
+
 }  // namespace ksana

@@ -40,6 +40,43 @@ struct CacheStats {
   }
 };
 
+// Pool of ids for state that a sequence holds as a whole beside its blocks (recurrent layers): one device slot per live
+// sequence, one host slot per swapped one. A slot that is given back is handed out again only after Settle(): copies
+// decided in between may still read it, and they run before anything that Settle's caller plans.
+class StateSlots {
+ public:
+  StateSlots(int device, int host) : in_use_(device, 0), host_in_use_(host, 0) {
+    for (int i = device - 1; i >= 0; --i) free_.push_back(i);
+    for (int i = host - 1; i >= 0; --i) host_free_.push_back(i);
+  }
+  int available() const { return static_cast<int>(free_.size()); }
+  int device_slots() const { return static_cast<int>(in_use_.size()); }
+  int Acquire() { return Take(&free_, &in_use_); }          // -1: none left
+  int AcquireHost() { return Take(&host_free_, &host_in_use_); }
+  void Release(int* slot) {
+    if (*slot >= 0) { in_use_[*slot] = 0; released_.push_back(*slot); *slot = -1; }
+  }
+  void ReleaseHost(int* slot) {
+    if (*slot >= 0) { host_in_use_[*slot] = 0; host_free_.push_back(*slot); *slot = -1; }
+  }
+  void Settle() {
+    free_.insert(free_.end(), released_.rbegin(), released_.rend());
+    released_.clear();
+  }
+  bool CheckInvariants(std::string* why) const;
+
+ private:
+  static int Take(std::vector<int>* from, std::vector<char>* used) {
+    if (from->empty()) return -1;
+    const int id = from->back();
+    from->pop_back();
+    (*used)[id] = 1;
+    return id;
+  }
+  std::vector<int> free_, released_, host_free_;
+  std::vector<char> in_use_, host_in_use_;
+};
+
 class CacheManager {
  public:
   CacheManager(int num_device_blocks, int num_host_blocks, int block_tokens, bool enable_prefix_cache);

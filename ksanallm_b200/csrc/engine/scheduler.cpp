@@ -10,16 +10,18 @@ namespace ksana {
 
 namespace {
 constexpr int32_t kPlanMagic = 0x4B53504C;   // "KSPL"
+constexpr size_t kPlanHeader = 20;
 inline int CeilMul(int bs, float thr) { return static_cast<int>(std::ceil(static_cast<double>(bs) * thr)); }
 }  // namespace
 
 // ---------------------------------------------------------------------------------- StepPlan
 std::vector<int32_t> StepPlan::Pack() const {
   // header: magic, nseq, ntok, num_multi, num_single, num_multi_tokens, max_q_len, max_blocks,
-  //         nsample, nswap_out, nswap_in, ncopies, npre_copies, sample_k, sample_full, has_prev_ids
+  //         nsample, nswap_out, nswap_in, ncopies, npre_copies, sample_k, sample_full, has_prev_ids, nstate_slots,
+  //         nstate_copies, nstate_out, nstate_in
   std::vector<int32_t> out;
   const int nseq = static_cast<int>(seq_ids.size());
-  out.reserve(16 + nseq * (4 + max_blocks) + num_tokens * 3 + 64);
+  out.reserve(kPlanHeader + nseq * (5 + max_blocks) + num_tokens * 3 + 64);
   out.push_back(kPlanMagic);
   out.push_back(nseq);
   out.push_back(num_tokens);
@@ -37,6 +39,10 @@ std::vector<int32_t> StepPlan::Pack() const {
   out.push_back(sample_full ? 1 : 0);
   const bool has_prev = static_cast<int>(prev_ids.size()) == num_tokens;
   out.push_back(has_prev ? 1 : 0);
+  out.push_back(static_cast<int>(state_slots.size()));
+  out.push_back(static_cast<int>(state_copies.size()));
+  out.push_back(static_cast<int>(state_out.size()));
+  out.push_back(static_cast<int>(state_in.size()));
   auto put = [&](const std::vector<int>& v) { out.insert(out.end(), v.begin(), v.end()); };
   auto put64 = [&](const std::vector<int64_t>& v) {
     for (int64_t x : v) { out.push_back(static_cast<int32_t>(x & 0xffffffff)); out.push_back(static_cast<int32_t>(x >> 32)); }
@@ -49,11 +55,14 @@ std::vector<int32_t> StepPlan::Pack() const {
   for (auto& c : copies) { out.push_back(c.src); out.push_back(c.dst); out.push_back(c.pos_delta); }
   for (auto& c : pre_copies) { out.push_back(c.src); out.push_back(c.dst); out.push_back(c.pos_delta); }
   if (has_prev) put(prev_ids);
+  put(state_slots);
+  for (auto* list : {&state_copies, &state_out, &state_in})
+    for (auto& s : *list) { out.push_back(s.device_block); out.push_back(s.host_block); }
   return out;
 }
 
 bool StepPlan::Unpack(const int32_t* d, size_t n, StepPlan* p) {
-  if (n < 16 || d[0] != kPlanMagic) return false;
+  if (n < kPlanHeader || d[0] != kPlanMagic) return false;
   p->Clear();
   const int nseq = d[1];
   p->num_tokens = d[2]; p->num_multi = d[3]; p->num_single = d[4]; p->num_multi_tokens = d[5];
@@ -63,11 +72,14 @@ bool StepPlan::Unpack(const int32_t* d, size_t n, StepPlan* p) {
   p->sample_full = d[14] != 0;
   if (nseq < 0 || p->num_tokens < 0 || p->max_blocks < 0 || nsample < 0 || nso < 0 || nsi < 0 || ncp < 0 || npre < 0)
     return false;
-  size_t need = 16 + static_cast<size_t>(p->num_tokens) * 3 + (nseq + 1) + nseq * 2 +
+  for (int i = 16; i < 20; ++i)
+    if (d[i] < 0) return false;
+  size_t need = kPlanHeader + d[16] + 2 * (static_cast<size_t>(d[17]) + d[18] + d[19]) +
+                static_cast<size_t>(p->num_tokens) * 3 + (nseq + 1) + nseq * 2 +
                 static_cast<size_t>(nseq) * p->max_blocks + nsample + 2 * nseq + 2 * nsample + 2 * nso + 2 * nsi +
                 3 * ncp + 3 * npre + (d[15] ? static_cast<size_t>(p->num_tokens) : 0);
   if (n < need) return false;
-  const int32_t* c = d + 16;
+  const int32_t* c = d + kPlanHeader;
   auto get = [&](std::vector<int>* v, size_t cnt) { v->assign(c, c + cnt); c += cnt; };
   auto get64 = [&](std::vector<int64_t>* v, size_t cnt) {
     v->resize(cnt);
@@ -86,6 +98,10 @@ bool StepPlan::Unpack(const int32_t* d, size_t n, StepPlan* p) {
   for (int i = 0; i < ncp; ++i) { p->copies.push_back({c[0], c[1], c[2]}); c += 3; }
   for (int i = 0; i < npre; ++i) { p->pre_copies.push_back({c[0], c[1], c[2]}); c += 3; }
   if (d[15]) get(&p->prev_ids, p->num_tokens);
+  get(&p->state_slots, d[16]);
+  int at = 17;
+  for (auto* list : {&p->state_copies, &p->state_out, &p->state_in})
+    for (int i = d[at++]; i > 0; --i) { list->push_back({c[0], c[1]}); c += 2; }
   return true;
 }
 
@@ -118,9 +134,13 @@ size_t StepPlan::WriteDecodeImage(int32_t* dst, int bs, int mb) const {
 
 // --------------------------------------------------------------------------------- Scheduler
 Scheduler::Scheduler(const SchedulerConfig& cfg, int num_device_blocks, int num_host_blocks)
-    : cfg_(cfg), split_fuse_on_(cfg.split_fuse_token_num > 0) {
+    : cfg_(cfg), split_fuse_on_(cfg.split_fuse_token_num > 0), states_(cfg.num_state_slots, cfg.num_host_state_slots) {
+  if (HasState()) {
+    cfg_.enable_prefix_cache = false;
+    cfg_.min_flexible_cache_num = 0;
+  }
   for (int r = 0; r < std::max(1, cfg.dp_size); ++r)
-    caches_.emplace_back(new CacheManager(num_device_blocks, num_host_blocks, cfg.block_token_num, cfg.enable_prefix_cache));
+    caches_.emplace_back(new CacheManager(num_device_blocks, num_host_blocks, cfg.block_token_num, cfg_.enable_prefix_cache));
   if (cfg_.max_step_tokens < cfg_.max_batch_size) cfg_.max_step_tokens = cfg_.max_batch_size;
 }
 
@@ -194,6 +214,8 @@ void Scheduler::FinishLocked(const SeqPtr& s, int code, const std::string& msg, 
   s->blocks.clear();
   CacheOf(*s).ReleaseHost(s->host_blocks);
   s->host_blocks.clear();
+  states_.Release(&s->state_slot);
+  states_.ReleaseHost(&s->host_state);
   s->state = SeqState::FINISHED;
   s->finish_status = Status(static_cast<RetCode>(code), msg);
   ++stats_.finished;
@@ -257,15 +279,22 @@ void Scheduler::PreemptLocked(const SeqPtr& v, StepPlan* plan) {
   KLLM_LOG_DEBUG << "preempt seq " << v->seq_id << " (req " << v->req_id << ", " << v->blocks.size() << " blocks, mode "
                  << (cfg_.preempt_mode == 0 ? "swap" : "recompute") << ")";
   const size_t so0 = plan->swap_out.size();
-  if (cfg_.preempt_mode == 0 && CacheOf(*v).SwapOut(&v->blocks, &v->host_blocks, &plan->swap_out)) {
+  const bool state_fits = !HasState() || (cfg_.preempt_mode == 0 && (v->host_state = states_.AcquireHost()) >= 0);
+  if (cfg_.preempt_mode == 0 && state_fits && CacheOf(*v).SwapOut(&v->blocks, &v->host_blocks, &plan->swap_out)) {
     for (size_t i = so0; i < plan->swap_out.size(); ++i) plan->swap_out[i].device_block += PoolBase(*v);
     v->promoted = std::min(v->promoted, static_cast<int>(v->blocks.size()));
+    if (HasState()) {
+      plan->state_out.push_back({v->state_slot, v->host_state});
+      states_.Release(&v->state_slot);
+    }
     v->state = SeqState::SWAPPED;
     swapped_.push_back(v);
     ++stats_.preempt_swap;
     return;
   }
   // recompute: everything generated so far becomes the prompt of a fresh prefill
+  states_.ReleaseHost(&v->host_state);
+  states_.Release(&v->state_slot);
   CacheOf(*v).Release(v->blocks);
   v->blocks.clear();
   v->kv_cached = 0;
@@ -281,6 +310,7 @@ void Scheduler::EmitRows(const Sequence& s, StepPlan* plan) {
   plan->seq_ids.push_back(s.seq_id);
   plan->q_lens.push_back(s.chunk);
   plan->kv_lens.push_back(s.kv_cached + s.chunk);
+  if (HasState()) plan->state_slots.push_back(s.state_slot);
   for (int i = 0; i < s.chunk; ++i) {
     const int pos = s.kv_cached + i;
     plan->input_ids.push_back(s.tokens[pos]);
@@ -327,6 +357,8 @@ Status Scheduler::PlanGiven(const std::vector<GivenEntry>& entries, StepPlan* pl
   const int B = cfg_.block_token_num;
   std::vector<SeqPtr> seqs;
   std::vector<int> need(caches_.size(), 0);
+  int need_states = 0;
+  states_.Settle();
   for (auto& e : entries) {
     auto it = by_id_.find(e.seq_id);
     if (it == by_id_.end() || it->second->state != SeqState::RUNNING)
@@ -342,11 +374,13 @@ Status Scheduler::PlanGiven(const std::vector<GivenEntry>& entries, StepPlan* pl
     if (total > cfg_.max_token_len)
       return Status(RET_EXCEED_LENGTH, "sequence longer than max_token_len " + std::to_string(cfg_.max_token_len));
     need[RankOf(s)] += std::max(0, CeilDiv(total, B) - static_cast<int>(s.blocks.size()));
+    need_states += HasState() && s.state_slot < 0;
     seqs.push_back(it->second);
   }
   for (size_t r = 0; r < caches_.size(); ++r)
     if (need[r] > caches_[r]->usable_blocks())
       return Status(RET_OUT_OF_MEMORY, "not enough KV cache blocks for this step");
+  if (need_states > states_.available()) return Status(RET_OUT_OF_MEMORY, "not enough state slots for this step");
   std::vector<SeqPtr> multi, single;
   std::vector<size_t> at;                                        // plan order -> entry
   std::vector<int> first(entries.size() + 1, 0);                 // where an entry's wanted rows start, entries' order
@@ -356,6 +390,7 @@ Status Scheduler::PlanGiven(const std::vector<GivenEntry>& entries, StepPlan* pl
     s.prompt_len = static_cast<int>(s.tokens.size());
     s.chunk = static_cast<int>(entries[i].tokens.size());
     CacheOf(s).Allocate(BlocksNeeded(s), &s.blocks);
+    if (HasState() && s.state_slot < 0) s.state_slot = states_.Acquire();
     first[i + 1] = first[i] + static_cast<int>(entries[i].want.size());
   }
   for (int pass = 0; pass < 2; ++pass)
@@ -407,6 +442,48 @@ void Scheduler::EmitSequence(const SeqPtr& s, StepPlan* plan) {
   }
 }
 
+int Scheduler::PendingSiblings(const Sequence& leader) const {
+  int n = 0;
+  auto git = groups_.find(leader.req_id);
+  if (git != groups_.end())
+    for (auto& m : git->second) n += m->forked_pending && m->leader == leader.seq_id && m->state != SeqState::FINISHED;
+  return n;
+}
+
+int Scheduler::ReservedSlots() const {
+  int n = 0;
+  for (auto& s : running_) n += PendingSiblings(*s);
+  return n;
+}
+
+// Every moved sequence continues from its parent's state. A parent that has moved on itself leaves its slot to its first
+// child; the other children are copied into the slots of moved sequences that nobody continues from. There are exactly
+// as many of these, and no slot is both read and written.
+void Scheduler::MoveStates(const std::vector<StateMove>& moves) {
+  auto moved = [&](const Sequence* s) {
+    return std::any_of(moves.begin(), moves.end(), [&](const StateMove& m) { return m.dst == s; });
+  };
+  auto is_parent = [&](const Sequence* s) {
+    return std::any_of(moves.begin(), moves.end(), [&](const StateMove& m) { return m.parent == s; });
+  };
+  std::vector<int> unused, slots;
+  std::vector<const Sequence*> taken;
+  for (auto& m : moves)
+    if (m.dst->state_slot >= 0 && !is_parent(m.dst)) unused.push_back(m.dst->state_slot);
+  for (auto& m : moves) {
+    if (moved(m.parent) && std::find(taken.begin(), taken.end(), m.parent) == taken.end()) {
+      taken.push_back(m.parent);
+      slots.push_back(m.parent->state_slot);
+      continue;
+    }
+    int to = -1;
+    if (!unused.empty()) { to = unused.back(); unused.pop_back(); } else { to = states_.Acquire(); }
+    pending_state_copies_.push_back({m.parent->state_slot, to});
+    slots.push_back(to);
+  }
+  for (size_t i = 0; i < moves.size(); ++i) moves[i].dst->state_slot = slots[i];
+}
+
 bool Scheduler::SwapInQualified(CacheManager& cache, const SeqPtr& s, StepPlan* plan) {
   const size_t n0 = plan->swap_in.size();
   if (!cache.SwapIn(&s->blocks, &s->host_blocks, &plan->swap_in)) return false;
@@ -418,6 +495,7 @@ bool Scheduler::Schedule(StepPlan* plan) {
   std::lock_guard<std::mutex> g(mu_);
   MergeWaitingBuffer();
   plan->Clear();
+  states_.Settle();
   const int64_t now = NowMs();
   const int B = cfg_.block_token_num;
   ExpireAndAbort(now, &plan->events);
@@ -489,9 +567,15 @@ bool Scheduler::Schedule(StepPlan* plan) {
                        std::max(0, CeilDiv(s->kv_cached + s->chunk, B) -
                                        static_cast<int>(s->blocks.size() + s->host_blocks.size()));
       if (bs + 1 <= cfg_.max_batch_size && step_tokens + s->chunk <= cap &&
+          (!HasState() || 1 + PendingSiblings(*s) + ReservedSlots() <= states_.available()) &&
           need + CeilMul(bs_rank, cfg_.swapin_block_threshold) <= cache.usable_blocks() &&
           SwapInQualified(cache, s, plan)) {
         cache.Allocate(BlocksNeeded(*s), &s->blocks);
+        if (HasState()) {
+          s->state_slot = states_.Acquire();
+          plan->state_in.push_back({s->state_slot, s->host_state});
+          states_.ReleaseHost(&s->host_state);
+        }
         s->promoted = cache.Promote(s->tokens, &s->blocks, s->kv_cached, s->promoted);
         s->state = SeqState::RUNNING;
         running_.push_back(s);
@@ -517,12 +601,10 @@ bool Scheduler::Schedule(StepPlan* plan) {
   while (admit && !waiting_.empty()) {
     SeqPtr s = waiting_.front();
     const int len = static_cast<int>(s->tokens.size());
-    int siblings = 0;
-    auto git = groups_.find(s->req_id);
-    if (git != groups_.end())
-      for (auto& m : git->second) siblings += (m->forked_pending && m->leader == s->seq_id);
+    const int siblings = PendingSiblings(*s);
     const int bs = static_cast<int>(running_.size());
     if (bs + 1 + siblings > cfg_.max_batch_size) break;
+    if (HasState() && 1 + siblings + ReservedSlots() > states_.available()) break;
     int bs_rank = 0;
     for (auto& o : running_) bs_rank += (RankOf(*o) == RankOf(*s));
     CacheManager& cache = CacheOf(*s);
@@ -554,6 +636,7 @@ bool Scheduler::Schedule(StepPlan* plan) {
     s->promoted = matched / B;
     s->chunk = chunk;
     cache.Allocate(unique, &s->blocks);
+    if (HasState()) s->state_slot = states_.Acquire();
     for (auto& c : flex_copies) plan->copies.push_back({c.src + PoolBase(*s), c.dst + PoolBase(*s), c.pos_delta});
     s->state = SeqState::RUNNING;
     running_.push_back(s);
@@ -582,6 +665,8 @@ bool Scheduler::Schedule(StepPlan* plan) {
     plan->pre_copies.swap(pending_copies_);
     pending_copies_.clear();
   }
+  plan->state_copies.swap(pending_state_copies_);
+  pending_state_copies_.clear();
   ++stats_.steps;
   stats_.step_tokens += plan->num_tokens;
   return !plan->empty() || plan->has_block_ops();
@@ -616,6 +701,7 @@ void Scheduler::PostStep(const StepPlan& plan, const std::vector<SampledToken>& 
   // 2. beam re-parenting uses the parents' state before any token of this step is appended
   struct Reparent { SeqPtr dst; std::vector<int> tokens; std::vector<int> blocks; int kv; int promoted; };
   std::vector<Reparent> moves;
+  std::vector<StateMove> state_moves;
   std::vector<BlockCopy> fork_copies;
   for (size_t i = 0; i < plan.sample_seq_ids.size() && i < sampled.size(); ++i) {
     const int64_t pid = sampled[i].parent_seq;
@@ -630,7 +716,9 @@ void Scheduler::PostStep(const StepPlan& plan, const std::vector<SampledToken>& 
     for (size_t k = fc0; k < fork_copies.size(); ++k) { fork_copies[k].src += PoolBase(*pit->second); fork_copies[k].dst += PoolBase(*pit->second); }
     mv.promoted = std::min(pit->second->promoted, pit->second->kv_cached / cfg_.block_token_num);
     moves.push_back(std::move(mv));
+    state_moves.push_back({dit->second.get(), pit->second.get()});
   }
+  if (HasState()) MoveStates(state_moves);
   for (auto& mv : moves) {
     CacheOf(*mv.dst).Release(mv.dst->blocks);
     mv.dst->blocks = std::move(mv.blocks);
@@ -654,14 +742,20 @@ void Scheduler::PostStep(const StepPlan& plan, const std::vector<SampledToken>& 
         // leader appended its own token already when it precedes us; share only the prompt part
         int shared_tokens = std::min(l->kv_cached, s->prompt_len);
         if (cfg_.resume_at_block_ends && shared_tokens != l->kv_cached) shared_tokens = shared_tokens / cfg_.block_token_num * cfg_.block_token_num;
+        if (HasState() && shared_tokens != l->kv_cached) shared_tokens = 0;
         std::vector<BlockCopy> cps;
-        if (RankOf(*l) == RankOf(*s) && CacheOf(*l).Fork(l->blocks, shared_tokens, &s->blocks, &cps)) {
+        if (RankOf(*l) == RankOf(*s) && shared_tokens > 0 && CacheOf(*l).Fork(l->blocks, shared_tokens, &s->blocks, &cps)) {
           for (auto& c : cps) { c.src += PoolBase(*l); c.dst += PoolBase(*l); }
           pending_copies_.insert(pending_copies_.end(), cps.begin(), cps.end());
           s->kv_cached = shared_tokens;
           s->promoted = std::min(l->promoted, shared_tokens / cfg_.block_token_num);
+          if (HasState()) {
+            s->state_slot = states_.Acquire();
+            pending_state_copies_.push_back({l->state_slot, s->state_slot});
+          }
         }
       }
+      if (HasState() && s->state_slot < 0) s->state_slot = states_.Acquire();      // computed from its first token on
       s->forked_pending = false;
       s->state = SeqState::RUNNING;
       running_.push_back(s);
@@ -767,7 +861,7 @@ bool Scheduler::ReplaceGenerated(int64_t seq_id, const std::vector<int>& generat
   if (new_cached < s->kv_cached) {
     // blocks past the divergence point may be shared through the tree: give them back and let the
     // next step allocate private ones
-    const int keep_blocks = new_cached / B;   // whole blocks that stay valid
+    const int keep_blocks = HasState() ? 0 : new_cached / B;   // whole blocks that stay valid
     if (keep_blocks < static_cast<int>(s->blocks.size())) {
       std::vector<int> drop(s->blocks.begin() + keep_blocks, s->blocks.end());
       CacheOf(*s).Release(drop);
@@ -817,6 +911,9 @@ bool Scheduler::CheckInvariants(std::string* why) {
   std::lock_guard<std::mutex> g(mu_);
   for (auto& c : caches_)
     if (!c->CheckInvariants(why)) return false;
+  if (!states_.CheckInvariants(why)) return false;
+  for (auto& s : running_)
+    if (HasState() && s->state_slot < 0) { *why = "a running sequence without a state slot"; return false; }
   return true;
 }
 

@@ -40,6 +40,11 @@ struct SchedulerConfig {
   // Blocks hold recurrent state as of their last computed token: a sequence resumes at the end of a cached block only
   // (never inside one, as a fully cached prompt otherwise does to compute its last token again)
   bool resume_at_block_ends = false;
+  // State beside the blocks: device slots (one per live sequence; 0: the model has no such state) and host slots for
+  // swapped sequences. Such state exists for the end of a sequence only: no prefix is shared, and a sequence that loses
+  // tokens is computed again
+  int num_state_slots = 0;
+  int num_host_state_slots = 0;
   int block_token_num = 16;
   int auto_batch_wait_ms = 100;
   // attention data parallelism: sequence s lives on rank s % dp_size and only that rank holds its KV blocks, so
@@ -64,6 +69,8 @@ struct Sequence {
   int sampled = 0;               // tokens sampled so far (RNG counter)
   std::vector<int> blocks;
   std::vector<int> host_blocks;
+  int state_slot = -1;           // device slot of its state, while it runs
+  int host_state = -1;           // host slot of its state, while it is swapped
   std::shared_ptr<SamplingConfig> cfg;
   int64_t arrive_ms = 0;
   int64_t first_token_ms = 0;
@@ -98,6 +105,9 @@ struct StepPlan {
                                            // first, before this step's swap-outs can touch their destinations
   std::vector<SwapCopy> swap_out, swap_in;
   std::vector<BlockCopy> copies;
+  std::vector<int> state_slots;            // per sequence, where the model has state beside the blocks
+  std::vector<SwapCopy> state_copies;      // (source slot, destination slot) of forks: they run together with pre_copies
+  std::vector<SwapCopy> state_out, state_in;   // (device slot, host slot): together with swap_out and swap_in
   int num_multi = 0, num_single = 0, num_tokens = 0, num_multi_tokens = 0, max_q_len = 0;
   // What this step's sampling needs from the logits: the largest candidate count of any sampling row
   // (max(topk, logprobs_num)), and whether a row edits the whole logits row first (repetition penalty, n-gram
@@ -106,7 +116,10 @@ struct StepPlan {
   bool sample_full = false;
   std::vector<SeqEvent> events;            // timeouts / aborts / rejections decided while planning
   bool empty() const { return seq_ids.empty(); }
-  bool has_block_ops() const { return !pre_copies.empty() || !swap_out.empty() || !swap_in.empty() || !copies.empty(); }
+  bool has_block_ops() const {
+    return !pre_copies.empty() || !swap_out.empty() || !swap_in.empty() || !copies.empty() || !state_copies.empty() ||
+           !state_out.empty() || !state_in.empty();
+  }
   void Clear() { *this = StepPlan(); }
   // Flat int32 image (header + arrays) used for the single host->device upload and for
   // broadcasting the step to the other ranks / nodes.
@@ -203,6 +216,11 @@ class Scheduler {
   // Copy and swap lists are executed by the ranks, and block ids are per rank: a device block in those lists is
   // written as rank * blocks_per_rank + block, so that each rank picks out (and un-offsets) its own entries.
   int PoolBase(const Sequence& s) const { return RankOf(s) * caches_[0]->num_device_blocks(); }
+  bool HasState() const { return cfg_.num_state_slots > 0; }
+  int PendingSiblings(const Sequence& leader) const;
+  int ReservedSlots() const;             // slots that siblings of running sequences will need when they fork
+  struct StateMove { Sequence* dst; Sequence* parent; };
+  void MoveStates(const std::vector<StateMove>& moves);
   bool SwapInQualified(CacheManager& cache, const SeqPtr& s, StepPlan* plan);
   int RankOf(const Sequence& s) const { return static_cast<int>(s.seq_id % static_cast<int64_t>(caches_.size())); }
 
@@ -216,6 +234,8 @@ class Scheduler {
   std::unordered_map<int64_t, std::vector<SeqPtr>> groups_;
   int64_t next_seq_id_ = 1;
   bool split_fuse_on_;
+  StateSlots states_;
+  std::vector<SwapCopy> pending_state_copies_;
   std::vector<BlockCopy> pending_copies_;   // fork copies decided in PostStep, executed by the next step
   SchedulerStats stats_;
 };

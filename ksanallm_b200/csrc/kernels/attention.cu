@@ -23,6 +23,8 @@
 // columns past the row's end). K and V lie in panels of their own: [block][Hkv][block_tokens][D] and [...][Dv].
 // Sliding window: position i sees j <= i with i - j < window or j < keep; tiles between the kept tokens and the
 // window are not visited. Sink: an extra logit per head in the softmax denominator, without a value.
+// Sigmoid weights (SIG): every visible key has the weight sigmoid(score + bias[head][distance]), nothing is normalised over
+// keys. Gate: outputs are multiplied by the sigmoid of a gate element and by one factor.
 //
 // Functional counterpart of the reference's decode kernels
 // (3rdparty/LLM_kernels/csrc/kernels/nvidia/paged_attention/paged_attention.cu:81-640)
@@ -61,6 +63,9 @@ struct AttnParams {
   const int* cu_q;                       // [B+1] query row offsets (prefill) or null (decode: row = s)
   const int* kv_lens;                    // [B]
   const float* alibi;                    // [Hq] slopes or null
+  const float* bias; int bias_len;       // sigmoid weights: [Hq][bias_len] added by distance (the last entry holds beyond)
+  const bf16* gate; long long gate_stride;   // optional, same layout as out
+  float out_factor;                      // of gated outputs
   int Hq, Hkv;
   float scale_log2;                      // softmax scale * log2(e)
   float k_scale, v_scale;                // fp8 cache dequant scales
@@ -299,13 +304,35 @@ __device__ __forceinline__ void softmax_update(float (&s)[NT][4], float (&o)[D /
   }
 }
 
+// Independent weights for one warp's 16 x (NT*8) score tile; bias[i]: the bias row of row i's head.
+template <int NT>
+__device__ __forceinline__ void sigmoid_weights(float (&s)[NT][4], const int (&limit)[2], const int (&lo)[2], int keep,
+                                                const float* const (&bias)[2], int bias_last, int tok0, int lane, float scale_log2) {
+#pragma unroll
+  for (int j = 0; j < NT; ++j) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int i = e >> 1;
+      const int tok = tok0 + j * 8 + (lane & 3) * 2 + (e & 1);
+      const bool seen = tok <= limit[i] && (tok >= lo[i] || tok < keep);
+      const float b = seen ? __ldg(bias[i] + min(limit[i] - tok, bias_last)) : 0.f;
+      s[j][e] = seen ? 1.f / (1.f + exp2f(-fmaf(s[j][e], scale_log2, b * 1.44269504f))) : 0.f;
+    }
+  }
+}
+
+// factor of an output element: sigmoid of its gate
+__device__ __forceinline__ float gate_of(const AttnParams& p, long long row, int col) {
+  return p.gate ? p.out_factor / (1.f + exp2f(-1.44269504f * __bfloat162float(p.gate[row * p.gate_stride + col]))) : 1.f;
+}
+
 // exp(sink - m) of the softmax denominator; m is the row's reference maximum in the log2 domain
 __device__ __forceinline__ float sink_term(const AttnParams& p, int head, float m) {
   return (p.sinks && m != -INFINITY) ? exp2f(p.sinks[head] * 1.44269504f - m) : 0.f;
 }
 
 // ----------------------------------------------------------------------------- prefill
-template <int D, int MODE>
+template <int D, int MODE, bool SIG>
 __global__ void __launch_bounds__(kAttnThreads)
 paged_prefill_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, const AttnParams p) {
   constexpr bool FP8 = MODE == kKvFp8;
@@ -378,12 +405,14 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_con
     ldsm_x4(qf[kk], smem_addr(tile_ptr<D, 64>(qs, r, c)));
   }
   int limit[2], lo[2]; float slope[2];
+  const float* bias[2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int vr = row0 + warp * 16 + (lane >> 2) + i * 8;
     limit[i] = vr < q_len * G ? past + vr / G : -1;
     lo[i] = p.window > 0 ? limit[i] - p.window + 1 : 0;
     slope[i] = (p.alibi && vr < q_len * G) ? p.alibi[g * G + vr % G] : 0.f;
+    bias[i] = SIG ? p.bias + static_cast<size_t>(g * G + vr % G) * p.bias_len : nullptr;
   }
   float o[D / 8][4];
 #pragma unroll
@@ -403,7 +432,8 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_con
     issue(t + kKvStages - 1);     // refill the stage tile t-1 used
     float sc[8][4];
     warp_qk<D, 8>(sc, qf, ks + buf * kTileTok * D, 0, lane);
-    softmax_update<D, 8>(sc, o, m, l, limit, lo, p.keep, slope, tok0, lane, p.scale_log2);
+    if constexpr (SIG) sigmoid_weights<8>(sc, limit, lo, p.keep, bias, p.bias_len - 1, tok0, lane, p.scale_log2);
+    else softmax_update<D, 8>(sc, o, m, l, limit, lo, p.keep, slope, tok0, lane, p.scale_log2);
     warp_pv<D, 8>(o, sc, vs + buf * kTileTok * D, 0, lane);
   }
   if (!ok) {                      // a bounded wait gave up: leave the output untouched, report through the error word
@@ -421,18 +451,26 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_con
     if (vr >= q_len * G) continue;
     const int tok = vr / G, head = g * G + vr % G;
     l[i] += sink_term(p, head, m[i]);
-    const float inv = l[i] > 0.f ? 1.f / l[i] : 0.f;
+    const float inv = SIG ? 1.f : l[i] > 0.f ? 1.f / l[i] : 0.f;
     bf16* dst = p.out + static_cast<size_t>(q0 + tok) * p.out_stride + head * p.Dv + (lane & 3) * 2;
 #pragma unroll
     for (int n = 0; n < D / 8; ++n) {
-      if (n * 8 < p.Dv) *reinterpret_cast<uint32_t*>(dst + n * 8) = pack_bf16(o[n][2 * i] * inv, o[n][2 * i + 1] * inv);
+      if (n * 8 < p.Dv) {
+        float a = o[n][2 * i] * inv, b = o[n][2 * i + 1] * inv;
+        if (SIG && p.gate) {
+          const int col = head * p.Dv + (lane & 3) * 2 + n * 8;
+          a *= gate_of(p, q0 + tok, col);
+          b *= gate_of(p, q0 + tok, col + 1);
+        }
+        *reinterpret_cast<uint32_t*>(dst + n * 8) = pack_bf16(a, b);
+      }
     }
   }
 }
 
 // ------------------------------------------------------------------------------ decode
 // grid (Hkv x row groups, B, splits). Rows = up to 16 of the G query heads of kv head g, one new token each.
-template <int D, int MODE>
+template <int D, int MODE, bool SIG>
 __global__ void __launch_bounds__(kAttnThreads)
 paged_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, const AttnParams p) {
   constexpr bool FP8 = MODE == kKvFp8;
@@ -500,17 +538,20 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
     ldsm_x4(qf[kk], smem_addr(tile_ptr<D, 16>(qs, r, c)));
   }
   int limit[2], lo[2]; float slope[2];
+  const float* bias[2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int r = (lane >> 2) + i * 8;
     limit[i] = r < G ? kv_len - 1 : -1;
     lo[i] = win_lo;
     slope[i] = (p.alibi && r < G) ? p.alibi[head0 + r] : 0.f;
+    bias[i] = SIG ? p.bias + static_cast<size_t>(head0 + (r < G ? r : 0)) * p.bias_len : nullptr;
   }
   float o[D / 8][4];
 #pragma unroll
   for (int n = 0; n < D / 8; ++n) { o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f; }
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  if (SIG) { m[0] = m[1] = 0.f; }            // nothing is rescaled when partial sums are merged
 
   bool ok = true;
   for (int t = t_begin; t < t_end; ++t) {
@@ -525,7 +566,8 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
     issue(t + kKvStages - 1);
     float sc[2][4];
     warp_qk<D, 2>(sc, qf, ks + buf * kTileTok * D, warp * 16, lane);
-    softmax_update<D, 2>(sc, o, m, l, limit, lo, p.keep, slope, tok0 + warp * 16, lane, p.scale_log2);
+    if constexpr (SIG) sigmoid_weights<2>(sc, limit, lo, p.keep, bias, p.bias_len - 1, tok0 + warp * 16, lane, p.scale_log2);
+    else softmax_update<D, 2>(sc, o, m, l, limit, lo, p.keep, slope, tok0 + warp * 16, lane, p.scale_log2);
     warp_pv<D, 2>(o, sc, vs + buf * kTileTok * D, warp * 16, lane);
   }
   cp_wait<0>();
@@ -570,7 +612,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
     const int head = head0 + r;
     if (p.num_splits == 1) {
       ll += sink_term(p, head, mm);
-      const float v = ll > 0.f ? acc / ll : 0.f;
+      const float v = SIG ? acc * gate_of(p, s, head * Dv + d) : ll > 0.f ? acc / ll : 0.f;
       if constexpr (D == 128) {
         if (p.outq) { store_head_row_q(p, s, head, d, v, red4); continue; }   // (Dv == blockDim: r is uniform per pass)
       }
@@ -604,7 +646,7 @@ __global__ void decode_reduce_kernel(const AttnParams p) {
       ll += p.part_ml[(base + k) * 2 + 1] * f;
     }
     ll += sink;
-    const float v = ll > 0.f ? acc / ll : 0.f;
+    const float v = p.bias ? acc * gate_of(p, s, head * Dv + d) : ll > 0.f ? acc / ll : 0.f;
     if constexpr (D == 128) {
       if (p.outq) { store_head_row_q(p, s, head, d, v, red4); continue; }     // 128 threads: one pass, every thread in it
     }
@@ -650,33 +692,33 @@ static bool tma_maps(const AttnParams& p, int num_blocks, CUtensorMap* km, CUten
          make_kv_map(vm, p.vc, p.block_stride, num_blocks, p.Hkv, p.Dv, bt);
 }
 
-template <int D, int MODE>
+template <int D, int MODE, bool SIG = false>
 static int launch_prefill(const AttnParams& p, const CUtensorMap& km, const CUtensorMap& vm, int B, int max_q_len, cudaStream_t st) {
   const int smem = (64 + 2 * kv_stages(D) * kTileTok) * D * 2 + 1024;
   static bool set = false;
   if (!set) {
-    if (cudaFuncSetAttribute(paged_prefill_kernel<D, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) !=
+    if (cudaFuncSetAttribute(paged_prefill_kernel<D, MODE, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) !=
         cudaSuccess) return -3;
     set = true;
   }
   const int G = p.Hq / p.Hkv;
   dim3 grid((max_q_len * G + 63) / 64, p.Hkv, B);
-  paged_prefill_kernel<D, MODE><<<grid, kAttnThreads, smem, st>>>(km, vm, p);
+  paged_prefill_kernel<D, MODE, SIG><<<grid, kAttnThreads, smem, st>>>(km, vm, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
-template <int D, int MODE>
+template <int D, int MODE, bool SIG = false>
 static int launch_decode(const AttnParams& p, const CUtensorMap& km, const CUtensorMap& vm, int B, cudaStream_t st) {
   const int smem = (16 + 2 * kv_stages(D) * kTileTok) * D * 2 + 1024;   // the fp32 merge area fits inside the K and V rings
   static_assert(4 * 16 * (D + 2) * 4 <= 2 * kv_stages(D) * kTileTok * D * 2, "merge area");
   static bool set = false;
   if (!set) {
-    if (cudaFuncSetAttribute(paged_decode_kernel<D, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) !=
+    if (cudaFuncSetAttribute(paged_decode_kernel<D, MODE, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) !=
         cudaSuccess) return -3;
     set = true;
   }
   dim3 grid(p.Hkv * ((p.Hq / p.Hkv + 15) / 16), B, p.num_splits);
-  if (launch_pdl(paged_decode_kernel<D, MODE>, grid, dim3(kAttnThreads), smem, st, km, vm, p) != cudaSuccess)
+  if (launch_pdl(paged_decode_kernel<D, MODE, SIG>, grid, dim3(kAttnThreads), smem, st, km, vm, p) != cudaSuccess)
     return -4;
   if (p.num_splits > 1) {
     if (launch_pdl(decode_reduce_kernel<D>, dim3(p.Hq, B), dim3(D < 128 ? 64 : 128), 0, st, p) != cudaSuccess) return -5;
@@ -687,6 +729,11 @@ static int launch_decode(const AttnParams& p, const CUtensorMap& km, const CUten
 template <int D>
 static int dispatch_prefill(const AttnParams& p, int cache_fp8, int num_blocks, int B, int max_q_len, cudaStream_t st) {
   CUtensorMap km{}, vm{};
+  if (p.bias) {
+    if (cache_fp8) return -11;
+    if (tma_maps(p, num_blocks, &km, &vm)) return launch_prefill<D, kKvTma, true>(p, km, vm, B, max_q_len, st);
+    return launch_prefill<D, kKvCpAsync, true>(p, km, vm, B, max_q_len, st);
+  }
   if constexpr (D <= 128) {
     if (cache_fp8) return launch_prefill<D, kKvFp8>(p, km, vm, B, max_q_len, st);
   } else if (cache_fp8) {
@@ -699,6 +746,11 @@ static int dispatch_prefill(const AttnParams& p, int cache_fp8, int num_blocks, 
 template <int D>
 static int dispatch_decode(const AttnParams& p, int cache_fp8, int num_blocks, int B, cudaStream_t st) {
   CUtensorMap km{}, vm{};
+  if (p.bias) {
+    if (cache_fp8) return -11;
+    if (tma_maps(p, num_blocks, &km, &vm)) return launch_decode<D, kKvTma, true>(p, km, vm, B, st);
+    return launch_decode<D, kKvCpAsync, true>(p, km, vm, B, st);
+  }
   if constexpr (D <= 128) {
     if (cache_fp8) return launch_decode<D, kKvFp8>(p, km, vm, B, st);
   } else if (cache_fp8) {
@@ -722,13 +774,17 @@ using namespace ksana;
 // Causal attention of new query rows against the paged cache (which already holds their K/V). kc / vc: the layer's K and
 // V panels of block 0; block_stride: elements between blocks; num_blocks: blocks addressable (0 disables the TMA path).
 // window 0: no sliding window. sinks: [Hq] fp32 or null. D, Dv: query/key and value head size (out rows: Hq * Dv).
+// bias [Hq][bias_len] fp32 switches to sigmoid weights; gate: optional rows like out's, with a common factor (sigmoid weights
+// only).
 extern "C" int ksana_paged_prefill(const void* q, long long q_stride, void* out, long long out_stride,
                                    const void* kc, const void* vc, long long block_stride, int block_tokens,
                                    const int* block_table, int table_stride, const int* cu_q, const int* kv_lens,
                                    const float* alibi, const float* sinks, int B, int max_q_len, int Hq, int Hkv, int D, int Dv,
                                    int window, int keep, float scale, int cache_fp8, float k_scale, float v_scale,
-                                   int num_blocks, int* err, cudaStream_t st) {
+                                   int num_blocks, const float* bias, int bias_len, const void* gate, long long gate_stride,
+                                   float out_factor, int* err, cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0) return 0;
+  if (bias ? (bias_len <= 0 || sinks || alibi) : gate != nullptr) return -14;
   if (Hkv <= 0 || Hq % Hkv || q_stride % 8 || (reinterpret_cast<uintptr_t>(q) & 15)) return -10;
   AttnParams p{};
   p.q = (const bf16*)q; p.q_stride = q_stride; p.out = (bf16*)out; p.out_stride = out_stride;
@@ -737,6 +793,7 @@ extern "C" int ksana_paged_prefill(const void* q, long long q_stride, void* out,
   p.block_table = block_table; p.table_stride = table_stride; p.cu_q = cu_q; p.kv_lens = kv_lens; p.alibi = alibi;
   p.Hq = Hq; p.Hkv = Hkv; p.scale_log2 = scale * 1.44269504f; p.k_scale = k_scale; p.v_scale = v_scale;
   p.num_splits = 1; p.err = err;
+  p.bias = bias; p.bias_len = bias_len; p.gate = (const bf16*)gate; p.gate_stride = gate_stride; p.out_factor = out_factor;
   switch (padded_head(D, Dv)) {
     case 64: return dispatch_prefill<64>(p, cache_fp8, num_blocks, B, max_q_len, st);
     case 128: return dispatch_prefill<128>(p, cache_fp8, num_blocks, B, max_q_len, st);
@@ -752,8 +809,10 @@ extern "C" int ksana_paged_decode(const void* q, long long q_stride, void* out, 
                                   const int* block_table, int table_stride, const int* kv_lens, const float* alibi,
                                   const float* sinks, int B, int Hq, int Hkv, int D, int Dv, int window, int keep, float scale,
                                   int cache_fp8, float k_scale, float v_scale, int num_splits, float* part_o, float* part_ml,
-                                  int num_blocks, void* outq, float* oscale, int oscale_ld, int* err, cudaStream_t st) {
+                                  int num_blocks, void* outq, float* oscale, int oscale_ld, const float* bias, int bias_len,
+                                  const void* gate, long long gate_stride, float out_factor, int* err, cudaStream_t st) {
   if (B <= 0) return 0;
+  if (bias ? (bias_len <= 0 || sinks || alibi || outq) : gate != nullptr) return -14;
   if (outq && (D != 128 || Dv != 128 || !oscale)) return -13;
   if (Hkv <= 0 || Hq % Hkv || q_stride % 8 || (reinterpret_cast<uintptr_t>(q) & 15)) return -10;
   if (num_splits < 1) num_splits = 1;
@@ -766,6 +825,7 @@ extern "C" int ksana_paged_decode(const void* q, long long q_stride, void* out, 
   p.Hq = Hq; p.Hkv = Hkv; p.scale_log2 = scale * 1.44269504f; p.k_scale = k_scale; p.v_scale = v_scale;
   p.num_splits = num_splits; p.part_o = part_o; p.part_ml = part_ml; p.err = err;
   p.outq = static_cast<uint8_t*>(outq); p.oscale = oscale; p.oscale_ld = oscale_ld;
+  p.bias = bias; p.bias_len = bias_len; p.gate = (const bf16*)gate; p.gate_stride = gate_stride; p.out_factor = out_factor;
   switch (padded_head(D, Dv)) {
     case 64: return dispatch_decode<64>(p, cache_fp8, num_blocks, B, st);
     case 128: return dispatch_decode<128>(p, cache_fp8, num_blocks, B, st);

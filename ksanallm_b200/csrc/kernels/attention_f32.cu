@@ -3,7 +3,8 @@
 // kernel does not cover. Keys are walked in chunks of 128 (one key per thread for the scores, one output
 // column per thread for the sum) with an online softmax. Sliding window with kept first tokens, grouped query heads,
 // different key and value sizes (values may be the leading columns of the key rows), an optional per-head sink logit in the
-// denominator and an optional gate per query row and head.
+// denominator and an optional gate per query row and head, or per output element (with a common factor). With a bias table
+// [heads][distances] the weights are sigmoid(score + bias) instead, without normalisation.
 #include "guards.cuh"
 #include "pdl.cuh"
 #include "vec8.cuh"
@@ -28,6 +29,8 @@ struct AttnF32Params {
   const int* cu_q; const int* kv_lens;
   const float* sinks;
   const T* gate; long long gate_ld;          // optional [rows][gate_ld]: a head's output is multiplied by sigmoid(gate)
+  int gate_wide; float out_factor;           // gate_wide: a gate per output element (columns like out's)
+  const float* bias; int bias_len;           // sigmoid weights: [Hq][bias_len] by distance (the last entry holds beyond)
   int Hq, Hkv, D, Dv, window, keep;
   float scale;
   int* err;
@@ -94,6 +97,23 @@ __global__ void __launch_bounds__(kAfThreads) attention_f32_kernel(const AttnF32
         vo = static_cast<long long>(blk) * p.block_stride + (static_cast<long long>(g) * p.block_tokens + off) * p.ldv;
       }
     }
+    if (p.bias) {                             // same for every thread of the launch
+      const int tok = i < nkeep ? i : lo + i - nkeep;
+      const float b = vo >= 0 ? p.bias[static_cast<size_t>(head) * p.bias_len + min(pos - tok, p.bias_len - 1)] : 0.f;
+      ps[threadIdx.x] = vo >= 0 ? 1.f / (1.f + expf(-(sc + b))) : 0.f;
+      voff[threadIdx.x] = vo;
+      l = 1.f;
+      __syncthreads();
+      const int n = min(kAfThreads, nvis - c0);
+#pragma unroll
+      for (int c = 0; c < MAXD / kAfThreads; ++c) {
+        const int d = threadIdx.x + c * kAfThreads;
+        if (d < p.Dv)
+          for (int k = 0; k < n; ++k) if (voff[k] >= 0) o[c] = fmaf(ps[k], to_f(p.vc[voff[k] + d]), o[c]);
+      }
+      __syncthreads();
+      continue;
+    }
     const float mx = fmaxf(m, block_reduce(sc, red, true));
     const float corr = (m == -CUDART_INF_F) ? 0.f : expf(m - mx);
     const float pr = (sc == -CUDART_INF_F) ? 0.f : expf(sc - mx);
@@ -113,7 +133,13 @@ __global__ void __launch_bounds__(kAfThreads) attention_f32_kernel(const AttnF32
     }
     __syncthreads();
   }
-  if (p.gate) {
+  if (p.gate && p.gate_wide) {
+#pragma unroll
+    for (int c = 0; c < MAXD / kAfThreads; ++c) {
+      const int d = threadIdx.x + c * kAfThreads;
+      if (d < p.Dv) o[c] *= p.out_factor * sigmoid_f(to_f(p.gate[static_cast<size_t>(q0 + qi) * p.gate_ld + static_cast<size_t>(head) * p.Dv + d]));
+    }
+  } else if (p.gate) {
     const float f = sigmoid_f(to_f(p.gate[static_cast<size_t>(q0 + qi) * p.gate_ld + head]));
 #pragma unroll
     for (int c = 0; c < MAXD / kAfThreads; ++c) o[c] *= f;
@@ -129,13 +155,15 @@ template <typename T>
 static int launch_attention_f32(const void* q, long long q_stride, void* out, long long out_stride, const void* kc, const void* vc,
                                 int ldv, long long block_stride, int block_tokens, int num_blocks, const int* block_table,
                                 int table_stride, const int* cu_q, const int* kv_lens, const float* sinks, const void* gate,
-                                long long gate_ld, int B, int max_q_len, int Hq, int Hkv, int D, int Dv, int window, int keep, float scale, int* err, cudaStream_t st) {
+                                long long gate_ld, int gate_wide, float out_factor, const float* bias, int bias_len, int B, int max_q_len,
+                                int Hq, int Hkv, int D, int Dv, int window, int keep, float scale, int* err, cudaStream_t st) {
   AttnF32Params<T> p{};
   p.q = static_cast<const T*>(q); p.q_stride = q_stride; p.out = static_cast<T*>(out); p.out_stride = out_stride;
   p.kc = static_cast<const T*>(kc); p.vc = static_cast<const T*>(vc); p.ldv = ldv;
   p.block_stride = block_stride; p.block_tokens = block_tokens; p.num_blocks = num_blocks;
   p.block_table = block_table; p.table_stride = table_stride; p.cu_q = cu_q; p.kv_lens = kv_lens; p.sinks = sinks;
-  p.gate = static_cast<const T*>(gate); p.gate_ld = gate_ld;
+  p.gate = static_cast<const T*>(gate); p.gate_ld = gate_ld; p.gate_wide = gate_wide; p.out_factor = out_factor;
+  p.bias = bias; p.bias_len = bias_len;
   p.Hq = Hq; p.Hkv = Hkv; p.D = D; p.Dv = Dv; p.window = window; p.keep = window > 0 ? keep : 0; p.scale = scale; p.err = err;
   const dim3 grid(max_q_len, Hq, B), block(kAfThreads);
   const cudaError_t e = (D > kAfMaxD || Dv > kAfMaxD)
@@ -148,18 +176,21 @@ static int launch_attention_f32(const void* q, long long q_stride, void* out, lo
 
 using namespace ksana;
 
-// window 0: full causal attention. D and Dv multiples of 8, at most 1024. ldv: elements between value rows. f32: q, out and
+// window 0: full causal attention. bias: sigmoid weights. D and Dv multiples of 8, at most 1024. ldv: elements between value rows. f32: q, out and
 // the panels are fp32 instead of bf16.
 extern "C" int ksana_attention_f32(const void* q, long long q_stride, void* out, long long out_stride, const void* kc,
                                    const void* vc, int ldv, long long block_stride, int block_tokens, int num_blocks,
                                    const int* block_table, int table_stride, const int* cu_q, const int* kv_lens,
-                                   const float* sinks, const void* gate, long long gate_ld, int B, int max_q_len, int Hq,
-                                   int Hkv, int D, int Dv, int window, int keep, float scale, int f32, int* err, cudaStream_t st) {
+                                   const float* sinks, const void* gate, long long gate_ld, int gate_wide, float out_factor,
+                                   const float* bias, int bias_len, int B, int max_q_len, int Hq, int Hkv, int D, int Dv, int window, int keep, float scale, int f32, int* err, cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0) return 0;
+  if (bias && bias_len <= 0) return -14;
   if (Hkv <= 0 || Hq % Hkv || D <= 0 || Dv <= 0 || D > kAfMaxWide || Dv > kAfMaxWide || D % 8 || Dv % 8 || ldv < Dv || Hq > 65535 ||
       B > 65535 || block_tokens <= 0 || block_stride % 8 || !aligned16(kc)) return -10;
   return f32 ? launch_attention_f32<float>(q, q_stride, out, out_stride, kc, vc, ldv, block_stride, block_tokens, num_blocks, block_table,
-                                           table_stride, cu_q, kv_lens, sinks, gate, gate_ld, B, max_q_len, Hq, Hkv, D, Dv, window, keep, scale, err, st)
+                                           table_stride, cu_q, kv_lens, sinks, gate, gate_ld, gate_wide, out_factor, bias, bias_len, B, max_q_len, Hq,
+                                           Hkv, D, Dv, window, keep, scale, err, st)
              : launch_attention_f32<bf16>(q, q_stride, out, out_stride, kc, vc, ldv, block_stride, block_tokens, num_blocks, block_table,
-                                          table_stride, cu_q, kv_lens, sinks, gate, gate_ld, B, max_q_len, Hq, Hkv, D, Dv, window, keep, scale, err, st);
+                                          table_stride, cu_q, kv_lens, sinks, gate, gate_ld, gate_wide, out_factor, bias, bias_len, B, max_q_len, Hq,
+                                          Hkv, D, Dv, window, keep, scale, err, st);
 }

@@ -12,6 +12,8 @@
 // Warp roles: warp 0 TMA producer (Q once; K and V tiles through the block table, one box per cache block and
 // 64-column panel), warp 1 MMA issuer + TMEM owner, warps 2..5 softmax + epilogue. Two CTAs share an SM
 // (96 KB of shared memory, 256 TMEM columns each), so one CTA's softmax overlaps the other's MMAs.
+// With sigmoid weights (SIG) a key's weight is sigmoid(score + bias[head][distance]): no maximum, no sum, no rescale; the
+// heads' bias rows are staged in shared memory where they fit. Outputs may be multiplied by the sigmoid of a gate.
 // Every wait is bounded; a timeout sets the error word and leaves the output untouched.
 //
 // Same operator as the reference's flash-attention prefill call plus its separate prefix-cache gather
@@ -31,6 +33,7 @@ constexpr int kFaD = 128;                    // padded head size
 constexpr int kFaPanelBytes = kFaTile * 128; // one 64-column panel of a 128-row tile
 constexpr int kFaTileBytes = 2 * kFaPanelBytes;
 constexpr int kFaSmemBytes = 3 * kFaTileBytes + 1024 + 256;
+constexpr int kFaBiasBytes = 14 * 1024;      // distance biases of a head group that still let two CTAs share an SM
 constexpr uint32_t kFaTmemCols = 256;        // S / P at columns [0,128), O at [128,256)
 constexpr float kFaRescaleLog2 = 8.f;        // O is rescaled only when a row maximum grew by more than this
 
@@ -43,6 +46,9 @@ struct FaParams {
   int rows;                                  // query rows of a CTA: the largest multiple of G up to 128
   int D, Dv;                                 // real head sizes
   int window, keep;                          // sliding window in tokens (0: none), first tokens every row sees
+  const float* bias; int bias_len;           // sigmoid weights: [Hq][bias_len] by distance (the last entry holds beyond)
+  int bias_ld;                               // floats between the heads' rows in shared memory; 0: read from global memory
+  const bf16* gate; long long gate_stride; float out_factor;     // sigmoid weights: optional gate rows like out's, and a factor
   float scale_log2;
   int* err;
 };
@@ -53,8 +59,14 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
+__device__ __forceinline__ float fast_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 // WIN: sliding window (p.window > 0); without it the window's tests are not compiled in
-template <bool WIN>
+template <bool WIN, bool SIG>
 __global__ void __launch_bounds__(kFaThreads, 2)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
                   const __grid_constant__ CUtensorMap v_map, const FaParams p) {
@@ -74,6 +86,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
   uint64_t* o_full = bars + 7;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 8);
   volatile uint32_t* abort_flag = tmem_slot + 1;
+  float* bias_s = reinterpret_cast<float*>(smem + 3 * kFaTileBytes + 256);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int s = blockIdx.z, g = blockIdx.y;
@@ -102,6 +115,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     mbar_fence_init();
   }
   if (warp == 1) { tmem_alloc(tmem_slot, kFaTmemCols); tmem_relinquish(); }
+  if (SIG && p.bias_ld > 0)
+    for (int i = threadIdx.x; i < G * p.bias_len; i += kFaThreads)
+      bias_s[i / p.bias_len * p.bias_ld + i % p.bias_len] = p.bias[static_cast<size_t>(g) * G * p.bias_len + i];
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -186,6 +202,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     const int keep = WIN ? p.keep : 0;
     auto sees = [&](int pos) { return pos <= limit && (!WIN || pos >= lo || pos < keep); };
     const float slope2 = (p.alibi && active) ? p.alibi[head] * 1.44269504f : 0.f;
+    const float* tab = !SIG ? nullptr : p.bias_ld > 0 ? bias_s + (vr % G) * p.bias_ld : p.bias + static_cast<size_t>(head) * p.bias_len;
+    const int bias_last = SIG ? p.bias_len - 1 : 0;
     float m_used = -CUDART_INF_F, l = 0.f;
     bool ok = true;
     for (int j = 0; j < ntiles; ++j) {
@@ -217,7 +235,38 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
         m_used = m_new;
         return (m_used == -CUDART_INF_F) ? 0.f : m_used;
       };
-      if (!__any_sync(0xffffffffu, biased)) {
+      if constexpr (SIG) {
+        uint32_t r[128];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) tmem_ld32(tmem_s + lane_off + c * 32, *reinterpret_cast<uint32_t(*)[32]>(&r[c * 32]));
+        tmem_ld_wait();
+        const int from = limit - t0;                       // distance of the tile's first key
+        auto weigh = [&](auto bias_at, auto hidden) {
+#pragma unroll
+          for (int i = 0; i < 128; i += 2) {
+            float w2[2];
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              const float b = bias_at(i + e) * -1.44269504f;
+              const float v = fast_rcp(1.f + fast_exp2(fmaf(__uint_as_float(r[i + e]), -p.scale_log2, b)));
+              w2[e] = hidden(i + e) ? 0.f : v;
+            }
+            __nv_bfloat162 pb = __floats2bfloat162_rn(w2[0], w2[1]);
+            r[i >> 1] = *reinterpret_cast<uint32_t*>(&pb);
+          }
+        };
+        const bool far = from - (kFaTile - 1) >= bias_last;      // every distance of the row has the last bias
+        if (__all_sync(0xffffffffu, far && !need_mask)) {
+          const float b = tab[bias_last];
+          weigh([&](int) { return b; }, [](int) { return false; });
+        } else {
+          const int last = from, first = lo - t0, kept = keep - t0;
+          weigh([&](int i) { return tab[min(max(from - i, 0), bias_last)]; },
+                [&](int i) { return i > last || (WIN && i < first && i >= kept); });
+        }
+#pragma unroll
+        for (int c = 0; c < 4; ++c) tmem_st16(tmem_s + lane_off + c * 16, *reinterpret_cast<uint32_t(*)[16]>(&r[c * 16]));
+      } else if (!__any_sync(0xffffffffu, biased)) {
         // the whole row in registers with a single TMEM round trip; hidden keys (window, diagonal) become -inf there
         uint32_t r[128];
 #pragma unroll
@@ -302,8 +351,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     if (ok && mbar_wait(o_full, 0, abort_flag)) {
       tc_fence_after();
       if (p.sinks && active) l += exp2f(p.sinks[head] * 1.44269504f - m_used);
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      const float inv = SIG ? 1.f : l > 0.f ? 1.f / l : 0.f;
       bf16* dst = p.out + static_cast<size_t>(q0 + tok) * p.out_stride + head * p.Dv;
+      const bf16* gate = SIG && p.gate ? p.gate + static_cast<size_t>(q0 + tok) * p.gate_stride + head * p.Dv : nullptr;
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         if (c * 32 >= p.Dv) break;
@@ -314,6 +364,16 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
             if (c * 32 + i >= p.Dv) break;
+            if (SIG && gate) {
+              const uint4 gv = *reinterpret_cast<const uint4*>(gate + c * 32 + i);
+              const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gv);
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                const float2 z = __bfloat1622float2(g2[e]);
+                r[i + 2 * e] = __float_as_uint(__uint_as_float(r[i + 2 * e]) * p.out_factor / (1.f + fast_exp2(z.x * -1.44269504f)));
+                r[i + 2 * e + 1] = __float_as_uint(__uint_as_float(r[i + 2 * e + 1]) * p.out_factor / (1.f + fast_exp2(z.y * -1.44269504f)));
+              }
+            }
             uint4 ov;
             __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&ov);
 #pragma unroll
@@ -359,13 +419,17 @@ using namespace ksana;
 // general kernel of attention.cu), other negatives on setup errors.
 // q: [T, q_stride] bf16 with head h at column h*D (T = rows addressable from q); kc / vc: the layer's K and V panels of
 // block 0, [Hkv][block_tokens][D] and [Hkv][block_tokens][Dv] bf16, blocks block_stride elements apart, num_blocks of them.
-// window 0: no sliding window. sinks: [Hq] fp32 or null.
+// window 0: no sliding window. sinks: [Hq] fp32 or null. bias [Hq][bias_len] fp32 switches to sigmoid weights; gate: optional
+// rows like out's (16-byte aligned), with a common factor.
 extern "C" int ksana_paged_prefill_tc(const void* q, long long q_stride, long long q_rows, void* out, long long out_stride,
                                       const void* kc, const void* vc, long long block_stride, int block_tokens,
                                       const int* block_table, int table_stride, const int* cu_q, const int* kv_lens,
                                       const float* alibi, const float* sinks, int B, int max_q_len, int Hq, int Hkv, int D,
-                                      int Dv, int window, int keep, float scale, int num_blocks, int* err, cudaStream_t st) {
+                                      int Dv, int window, int keep, float scale, int num_blocks, const float* bias, int bias_len,
+                                      const void* gate, long long gate_stride, float out_factor, int* err, cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0) return 0;
+  if (bias ? (bias_len <= 0 || sinks || alibi) : gate != nullptr) return -14;
+  if (gate && ((reinterpret_cast<uintptr_t>(gate) & 15) || gate_stride % 8)) return -100;
   if (D <= 0 || Dv <= 0 || D > kFaD || Dv > kFaD || D % 8 || Dv % 8 || Hkv <= 0 || Hq % Hkv) return -100;
   const int G = Hq / Hkv;
   const int bt = block_tokens;
@@ -397,9 +461,8 @@ extern "C" int ksana_paged_prefill_tc(const void* q, long long q_stride, long lo
   }
   static bool set = false;
   if (!set) {
-    if (cudaFuncSetAttribute(prefill_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kFaSmemBytes) != cudaSuccess ||
-        cudaFuncSetAttribute(prefill_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kFaSmemBytes) != cudaSuccess)
-      return -3;
+    for (auto* k : {prefill_tc_kernel<false, false>, prefill_tc_kernel<true, false>, prefill_tc_kernel<false, true>, prefill_tc_kernel<true, true>})
+      if (cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, kFaSmemBytes + kFaBiasBytes) != cudaSuccess) return -3;
     set = true;
   }
   FaParams p{};
@@ -409,8 +472,13 @@ extern "C" int ksana_paged_prefill_tc(const void* q, long long q_stride, long lo
   p.Hq = Hq; p.Hkv = Hkv; p.G = G; p.block_tokens = bt; p.rows = kFaTile / G * G;
   p.scale_log2 = scale * 1.44269504f;
   p.err = err;
+  p.bias = bias; p.bias_len = bias_len; p.gate = static_cast<const bf16*>(gate); p.gate_stride = gate_stride; p.out_factor = out_factor;
+  const long long table = bias ? static_cast<long long>(G) * (bias_len | 1) * 4 : 0;       // odd row pitch: heads in different banks
+  p.bias_ld = table > 0 && table <= kFaBiasBytes ? bias_len | 1 : 0;
+  const int smem = kFaSmemBytes + (p.bias_ld ? static_cast<int>(table) : 0);
   dim3 grid((max_q_len * G + p.rows - 1) / p.rows, Hkv, B);
-  if (window > 0) prefill_tc_kernel<true><<<grid, kFaThreads, kFaSmemBytes, st>>>(q_map, k_map, v_map, p);
-  else prefill_tc_kernel<false><<<grid, kFaThreads, kFaSmemBytes, st>>>(q_map, k_map, v_map, p);
+  auto* kernel = bias ? (window > 0 ? prefill_tc_kernel<true, true> : prefill_tc_kernel<false, true>)
+                      : (window > 0 ? prefill_tc_kernel<true, false> : prefill_tc_kernel<false, false>);
+  kernel<<<grid, kFaThreads, smem, st>>>(q_map, k_map, v_map, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

@@ -26,11 +26,11 @@ constexpr int kMaxTopK = 64;
 
 // One warp per token. scoring 0 = softmax over all experts, 1 = sigmoid. `bias` (may be null) is added
 // for SELECTION only (DeepSeek-V3 e_score_correction_bias). n_group/topk_group: keep only the best
-// topk_group groups (group score = sum of its two largest biased scores). Logit rows are ldl apart, weight rows
+// topk_group groups (group score = sum of its two largest biased scores, or with group_top 1 its largest). Logit rows are ldl apart, weight rows
 // ldw; with `gate_col` >= 0 the sigmoid of that logit column (a shared expert's gate) is a row's weight number K.
 __global__ void moe_route_kernel(const float* __restrict__ logits, int ldl, const float* __restrict__ bias,
                                  int* __restrict__ topk_ids, float* __restrict__ topk_w, int ldw, int T, int E, int K,
-                                 int scoring, int renorm, float scale, int n_group, int topk_group, int gate_col) {
+                                 int scoring, int renorm, float scale, int n_group, int topk_group, int group_top, int gate_col) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
   if (warp >= T) return;
@@ -67,7 +67,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ldl, cons
         const float v = sel[g * gs + i];
         if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
       }
-      gsc[g] = gs > 1 ? a + b : a;
+      gsc[g] = gs > 1 && group_top > 1 ? a + b : a;
     }
     __syncwarp();
     // a group survives if fewer than topk_group groups beat it (of equal ones the first)
@@ -213,13 +213,13 @@ __global__ void moe_combine_kernel(const bf16* __restrict__ y, const int* __rest
 using namespace ksana;
 
 extern "C" int ksana_moe_route(const float* logits, int ldl, const float* bias, int* topk_ids, float* topk_w, int ldw, int T,
-                               int E, int K, int scoring, int renorm, float scale, int n_group, int topk_group, int gate_col,
-                               cudaStream_t st) {
+                               int E, int K, int scoring, int renorm, float scale, int n_group, int topk_group, int group_top,
+                               int gate_col, cudaStream_t st) {
   if (T <= 0) return 0;
   if (E > kMaxExperts || K > kMaxTopK || K > E || n_group > E || (n_group > 1 && E % n_group)) return -10;
   if (ldl < E || gate_col >= ldl || ldw < K + (gate_col >= 0)) return -11;
   moe_route_kernel<<<(T + 7) / 8, 256, 0, st>>>(logits, ldl, bias, topk_ids, topk_w, ldw, T, E, K, scoring, renorm, scale,
-                                                n_group, topk_group, gate_col);
+                                                n_group, topk_group, group_top, gate_col);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

@@ -12,6 +12,7 @@
 //   gated_scan_kernel   sequences of any number of new tokens: one CTA per (sequence, channel tile), the time axis split
 //                       over the threads, prefixes combined in registers, shuffles and one exchange per chunk
 //   gated_step_kernel   sequences of one new token
+#include "f32x2.cuh"
 #include "guards.cuh"
 #include "pdl.cuh"
 #include "vec8.cuh"
@@ -39,18 +40,6 @@ struct ScanParams {
   int* err;
 };
 
-// Two floats in one 64-bit register: additions, products and fused products of pairs are single instructions here.
-struct F2 { unsigned long long v; };
-__device__ __forceinline__ F2 f2(float x, float y) { F2 r; asm("mov.b64 %0, {%1, %2};" : "=l"(r.v) : "f"(x), "f"(y)); return r; }
-__device__ __forceinline__ F2 f2(float x) { return f2(x, x); }
-__device__ __forceinline__ void split(F2 p, float& x, float& y) { asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(p.v)); }
-__device__ __forceinline__ F2 operator*(F2 a, F2 b) { F2 r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r.v) : "l"(a.v), "l"(b.v)); return r; }
-__device__ __forceinline__ F2 operator+(F2 a, F2 b) { F2 r; asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r.v) : "l"(a.v), "l"(b.v)); return r; }
-__device__ __forceinline__ F2 fma2(F2 a, F2 b, F2 c) {
-  F2 r;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r.v) : "l"(a.v), "l"(b.v), "l"(c.v));
-  return r;
-}
 // 1 + exp(-x) of a pair
 __device__ __forceinline__ F2 one_plus_exp_neg(F2 x) {
   float a, b;

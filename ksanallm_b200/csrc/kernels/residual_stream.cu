@@ -94,8 +94,8 @@ struct ResNormParams {
   int groups;                           // > 1: the stream's norm takes its mean square per consecutive part of H / groups columns
   const float* add; const T* vec;       // optional: stream rows (ldx apart) and a vector that are added too
   float z_scale;                        // factor of the normed row
-  // addend = sum over k < top of w[row][k] * y[dst_row[row][k]] (+ w[row][top] * shared[row]); rows of `ldw` weights. A
-  // negative dst_row is an expert that lives elsewhere
+  // addend = sum over k < top of w[row][k] * y[dst_row[row][k]] (+ w[row][top] * shared[row], or + shared[row] where a row has
+  // no weight for it); rows of `ldw` weights. A negative dst_row is an expert that lives elsewhere
   const int* dst_row; const float* w; int ldw, top, cap;
   const T* shared; int lds;
   int* err;
@@ -178,7 +178,7 @@ __global__ void residual_norm_kernel(const ResNormParams<T> p) {
       }
       if (threadIdx.x == 0) {
         src_n = n;
-        if (p.shared) shared_w = p.w[static_cast<size_t>(m) * p.ldw + p.top];
+        if (p.shared) shared_w = p.ldw > p.top ? p.w[static_cast<size_t>(m) * p.ldw + p.top] : 1.f;
       }
     }
     __syncthreads();
@@ -351,7 +351,7 @@ static int launch_residual_norm(const ResNormParams<T>& p, int M, cudaStream_t s
 // ------------------------------------------------------------------------------------------------ gated unit
 template <typename T>
 __global__ void glu_clamp_kernel(const T* __restrict__ in, T* __restrict__ out, int M, int I, int in_ld, float limit,
-                                 float alpha, float offset) {
+                                 float alpha, float offset, const int* __restrict__ tile_rows) {
   pdl_trigger();
   pdl_wait();
   const int nvec = I >> 3;
@@ -359,6 +359,7 @@ __global__ void glu_clamp_kernel(const T* __restrict__ in, T* __restrict__ out, 
   for (long long idx = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; idx < total;
        idx += static_cast<long long>(gridDim.x) * blockDim.x) {
     const int m = static_cast<int>(idx / nvec), i = static_cast<int>(idx - static_cast<long long>(m) * nvec);
+    if (tile_rows && (m & 127) >= tile_rows[m >> 7]) continue;       // of every 128 rows only so many hold anything
     const T* row = in + static_cast<size_t>(m) * in_ld;
     float g[8], u[8];
     load8(row + i * 8, g);
@@ -714,7 +715,7 @@ extern "C" int ksana_residual_norm(const float* x, int ldx, const int* rows, int
     if (!aligned16(q)) return -11;
   if (rows && x_out == x) return -12;
   if (groups > 1 && (!rms || H % groups || w1 || b2 || !w2 || z_scale != 1.f)) return -13;
-  if (dst_row && (!y || !w || rows || top <= 0 || top > kMaxTop || ldw < top + (shared ? 1 : 0) || cap <= 0)) return -14;
+  if (dst_row && (!y || !w || rows || top <= 0 || top > kMaxTop || ldw < top || cap <= 0)) return -14;
   if (shared && (!dst_row || lds % 8 || lds < hp)) return -15;
   auto entry = f32 ? residual_norm_entry<float> : residual_norm_entry<bf16>;
   return entry(x, ldx, rows, in_rows, y, ldy, w1, b1, ls, x_out, w2, b2, z, ldz, M, H, eps, rms, alpha, groups, add, vec, z_scale,
@@ -723,7 +724,7 @@ extern "C" int ksana_residual_norm(const float* x, int ldx, const int* rows, int
 
 // in [M, in_ld]: gate columns [0, I), up columns [I, 2I); out [M, I]. I a multiple of 8.
 extern "C" int ksana_glu_clamp(const void* in, void* out, int M, int I, int in_ld, float limit, float alpha, float offset,
-                               int f32, cudaStream_t st) {
+                               const int* tile_rows, int f32, cudaStream_t st) {
   if (M <= 0) return 0;
   if (I % 8 || in_ld % 8 || in_ld < 2 * I || !aligned16(in) || !aligned16(out)) return -10;
   const long long total = static_cast<long long>(M) * (I >> 3);
@@ -732,10 +733,10 @@ extern "C" int ksana_glu_clamp(const void* in, void* out, int M, int I, int in_l
   cudaError_t e;
   if (f32)
     e = launch_pdl(glu_clamp_kernel<float>, dim3((unsigned)g), dim3(256), 0, st, (const float*)in, (float*)out, M, I, in_ld, limit,
-                   alpha, offset);
+                   alpha, offset, tile_rows);
   else
     e = launch_pdl(glu_clamp_kernel<bf16>, dim3((unsigned)g), dim3(256), 0, st, (const bf16*)in, (bf16*)out, M, I, in_ld, limit,
-                   alpha, offset);
+                   alpha, offset, tile_rows);
   return e == cudaSuccess ? 0 : -4;
 }
 

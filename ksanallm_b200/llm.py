@@ -67,8 +67,8 @@ def kv_dtype_from(cfg: EngineConfig, default):
     return default
 
 
-def auto_num_blocks(cfg: EngineConfig, block_bytes: int, device) -> int:
-    """Device blocks from free memory: (free - reserved share) / block bytes, or the explicit ratio
+def auto_num_blocks(cfg: EngineConfig, block_bytes: int, device, set_aside: int = 0) -> int:
+    """Device blocks from free memory: (free - reserved share - bytes set aside) / block bytes, or the explicit ratio
     (src/ksana_llm/block_manager/block_manager.cpp:102-163)."""
     bm = cfg.block_manager
     if bm.device_blocks_num > 0:
@@ -79,7 +79,7 @@ def auto_num_blocks(cfg: EngineConfig, block_bytes: int, device) -> int:
     if bm.block_device_memory_ratio >= 0:
         budget = int(total * bm.block_device_memory_ratio)
     else:
-        budget = free - int(total * bm.reserved_device_memory_ratio)
+        budget = free - int(total * bm.reserved_device_memory_ratio) - set_aside
     return max(int(budget // block_bytes), 0)
 
 
@@ -192,7 +192,8 @@ class LLM:
         probe = self.model.allocate_kv_cache(1, bt, kv_dtype)
         block_bytes = probe[0].numel() * probe.element_size()
         self.model.kv_cache = None
-        nblocks = auto_num_blocks(self.engine_cfg, block_bytes, self.device)
+        nblocks = auto_num_blocks(self.engine_cfg, block_bytes, self.device,
+                                  self.model.state_bytes() * self.engine_cfg.batch_scheduler.max_batch_size)
         nhost = auto_host_blocks(self.engine_cfg, nblocks, block_bytes)
         if self.world > 1:
             import torch.distributed as dist

@@ -51,6 +51,7 @@ class StepInput:
     sample_k: int = 0                    # > 0: tensor-parallel ranks return merged per-shard top-k candidates, not logits
     want_hidden: bool = False            # keep final hidden states / post-norm states for /forward
     prev_ids: Optional[torch.Tensor] = None   # the token before each row's (-1: none); models with ``needs_prev_ids`` only
+    state_slots: Optional[torch.Tensor] = None   # per sequence (-1: padding); models with ``needs_state_slots`` only
 
 
 @dataclass
@@ -137,6 +138,10 @@ class CommonModel:
     # its last block has seen (whole cached blocks, or its own partly filled one), and a block's content is tied to its
     # position
     carries_state = False
+    # A sequence holds state as a whole beside its blocks, in a slot of ``state`` [slots, record]: it exists for the end of
+    # the sequence only, so no prefix of it can be shared. A slot's content counts from position 1 on (no clearing)
+    needs_state_slots = False
+    state: Optional[torch.Tensor] = None
     moves_blocks = True                  # copies of a block may be used at another position (flexible cache)
 
     def __init__(self, cfg: ModelConfig, tp_rank: int = 0, tp_size: int = 1, comm=None, device="cpu",
@@ -185,6 +190,13 @@ class CommonModel:
 
     def block_bytes(self) -> int:
         return self.kv_cache[0].numel() * self.kv_cache.element_size()
+
+    def state_bytes(self) -> int:
+        """Bytes of one state slot (a multiple of 16)."""
+        return 0
+
+    def allocate_state(self, num_slots: int) -> None:
+        """Fills ``state`` (models with ``needs_state_slots``)."""
 
     def _kv_scale(self, layer: int):
         if self.kv_scales is None or self.kv_cache is None or self.kv_cache.dtype in (torch.bfloat16, torch.float16, torch.float32):
@@ -282,6 +294,8 @@ class CommonModel:
         if normed.shape[0] == 0:
             return torch.empty(0, self.cfg.vocab_size, dtype=torch.float32, device=normed.device)
         logits = ops.linear(normed, self.lm_head, out_f32=True)
+        if self.cfg.logit_softcap:
+            logits = ops.softcap(logits, self.cfg.logit_softcap)
         if self.tp_size > 1:
             logits = self.comm.all_gather_last_dim(logits, valid=self.vocab_shard)
         return logits[:, : self.cfg.vocab_size] if logits.shape[1] != self.cfg.vocab_size else logits
@@ -299,6 +313,8 @@ class CommonModel:
         if stage is None:
             return None
         logits = ops.linear(normed, self.lm_head, out_f32=True)
+        if self.cfg.logit_softcap:
+            logits = ops.softcap(logits, self.cfg.logit_softcap)
         lo = self.tp_rank * self.vocab_shard
         valid = max(0, min(self.vocab_shard, self.cfg.vocab_size - lo))
         ops.native.shard_topk(logits, valid, k, lo, stage[0], stage[1])

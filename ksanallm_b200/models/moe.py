@@ -18,7 +18,7 @@ from typing import Optional
 
 import torch
 
-from ..config import ModelConfig
+from ..config import MlpSpec, ModelConfig
 from ..ops import dispatch as ops
 from ..ops import native, reference as ref
 from ..ops.dispatch import LinearWeight
@@ -162,9 +162,13 @@ def route_reference(logits, cfg: ModelConfig, bias=None):
 
 
 def dense_experts(perm, w13, w2, tile_expert, tile_rows, n_local, inter, act):
-    """Expert-major rows through their experts' gate|up and down matrices (stacked [E * 2I, H] and [E * H, I], bf16 or fp32)."""
+    """Expert-major rows through their experts' gate|up and down matrices (stacked [E * 2I, H] and [E * H, I], bf16 or fp32).
+    ``act``: name of the gate's activation, or the :class:`MlpSpec` of a clamped unit."""
     g = native.gemm_grouped(perm, w13, tile_expert, n_local, 2 * inter, tile_rows=tile_rows)
-    a = native.act_mul(g, act, True, tile_rows=tile_rows)
+    if isinstance(act, MlpSpec):
+        a = native.glu_clamp(g, act.limit, act.alpha, act.offset, tile_rows=tile_rows)
+    else:
+        a = native.act_mul(g, act, True, tile_rows=tile_rows)
     return native.gemm_grouped(a, w2, tile_expert, n_local, perm.shape[1], tile_rows=tile_rows)
 
 
@@ -180,7 +184,8 @@ def expert_outputs(x, ids, w13, w2, inter, act="silu"):
         tok, slot = (ids == e).nonzero(as_tuple=True)
         if tok.numel():
             gu = ref.gemm(x[tok], w13[e * 2 * inter:(e + 1) * 2 * inter])
-            y[tok * K + slot] = ref.gemm(ref.act_mul(gu, act, True), w2[e * x.shape[1]:(e + 1) * x.shape[1]])
+            a = ref.glu_clamp(gu, act.limit, act.alpha, act.offset) if isinstance(act, MlpSpec) else ref.act_mul(gu, act, True)
+            y[tok * K + slot] = ref.gemm(a, w2[e * x.shape[1]:(e + 1) * x.shape[1]])
     return y, torch.arange(T * K, dtype=torch.int32).view(T, K)
 
 

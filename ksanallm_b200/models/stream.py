@@ -7,6 +7,7 @@ sizes, feed-forward widths, vocabulary), so the kernels always see 16-byte vecto
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 from typing import List, Optional
 
@@ -50,6 +51,23 @@ def layer_runs(cfg: ModelConfig) -> List[LayerRun]:
             order += [(i, t if i == loop.start else None) for i in range(loop.start, loop.stop)]
         order += [(i, None) for i in range(loop.stop, n)]
     return [LayerRun(i, c, enter) for c, (i, enter) in enumerate(order)]
+
+
+def distance_biases(rel: torch.Tensor, far: int) -> torch.Tensor:
+    """[heads, n] biases by distance from a table [buckets, heads]: the first half of the buckets are single distances, the
+    others grow logarithmically up to ``far``; distances from n - 1 on have the last one's bias."""
+    count = rel.shape[0]
+    half = count // 2
+
+    def bucket(n):
+        if n < half:
+            return n
+        if half == 0 or far <= half:
+            return count - 1
+        return min(count - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (count - half)))
+
+    index = torch.tensor([bucket(n) for n in range(max(far, half) + 1)], device=rel.device)
+    return rel.float()[index].t().contiguous()
 
 
 def rerotate_panel(k: torch.Tensor, triples, table: torch.Tensor, interleaved: bool = False) -> None:
@@ -130,6 +148,14 @@ class StreamLoader:
         if tuple(t.shape) != tuple(shape):
             raise ValueError(f"{name}: shape {tuple(t.shape)} in the checkpoint, {tuple(shape)} by the configuration")
         return t
+
+    def shape(self, name, default):
+        """Shape of a tensor whose sizes the configuration does not give (``default``: where the source makes up its tensors)."""
+        from .weights import RandomSource
+        return tuple(default) if isinstance(self.source, RandomSource) else tuple(self.source.get(name, None, device="cpu").shape)
+
+    def f32(self, t):
+        return t.to(device=self.m.device, dtype=torch.float32).contiguous()
 
     def param(self, t, *sizes):
         return pad_to(t, *sizes).to(device=self.m.device, dtype=self.m.dtype).contiguous()

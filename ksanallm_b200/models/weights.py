@@ -334,10 +334,11 @@ def build_model(cfg: ModelConfig, source, tp_rank: int = 0, tp_size: int = 1, co
     """Instantiate and fill a model. ``quant``: None | "fp8_block" (projection weights only; norms,
     embeddings, router and lm_head stay in ``dtype``)."""
     if cfg.layer_specs is not None:
+        from .fapudra import build_fapudra
         from .fidevik import build_fidevik
         from .lenolix import build_lenolix
         from .rasizen import build_rasizen
-        build = {"fidevik": build_fidevik, "lenolix": build_lenolix, "rasizen": build_rasizen}[cfg.model_type]
+        build = {"fapudra": build_fapudra, "fidevik": build_fidevik, "lenolix": build_lenolix, "rasizen": build_rasizen}[cfg.model_type]
         return build(cfg, source, tp_rank, tp_size, comm, device, dtype, quant, layer_range, max_positions)
     if cfg.is_mla:
         from .deepseek import build_deepseek

@@ -11,6 +11,7 @@ from typing import Optional
 import torch
 
 from . import native, reference as ref
+from .native import SigmoidWeights  # noqa: F401
 
 
 @dataclass
@@ -268,7 +269,7 @@ def embed_pair(ids, prev, table, pair, scale, buckets=0, mul_prev=0, mul_cur=0, 
 @dataclass
 class ExpertSum:
     """A sublayer's result that is still spread over expert outputs: row t is the sum over k of w[t, k] * y[dst_row[t, k]]
-    (negative rows: left out), plus w[t, K] * shared[t]."""
+    (negative rows: left out), plus w[t, K] * shared[t], or plus shared[t] where w has K columns."""
     y: torch.Tensor
     dst_row: torch.Tensor                 # [T, K] int32
     w: torch.Tensor                       # [T, K] or [T, K + 1] fp32
@@ -343,6 +344,90 @@ def stream_add(x, y, post: Optional[NormParams], scale, then: Optional[NormParam
     if copy is not None:
         copy.copy_(out)
     return out, (ref.stream_norm(out, then).to(dtype) if then is not None else None)
+
+
+def embed_normed(ids, positions, table, pos_table, scale, norm: NormParams, vocab):
+    """fp32 rows norm(table[id] * scale + pos_table[position]) (root mean square)."""
+    if table.is_cuda:
+        return native.embed_normed(ids, positions, table, pos_table, norm.w, norm.size, scale, norm.eps, vocab)
+    return ref.stream_norm(table[ids.long()].float() * scale + pos_table[positions.long()].float(), norm)
+
+
+def token_shift(h, mu, ring, step):
+    """h_t + (h_(t-1) - h_t) * mu over a step's rows; ``ring`` [slots, 2, W]: the last rows of earlier steps (position p in row p
+    mod 2)."""
+    if h.is_cuda:
+        return native.token_shift(h, mu, ring, step.cu_q, step.kv_lens, step.state_slots, max(step.max_q_len, 1))
+    return ref.token_shift(h, mu, ring, step.cu_q, step.kv_lens, step.state_slots)
+
+
+def gated_norm(y, w, eps, heads, real, parts, z=None, g=None, factor=1.0, out=None):
+    """factor * norm(y * silu(z)) * w * sigmoid(g), the root mean square taken over each of ``parts`` equal parts of a row of
+    ``heads`` heads of ``real`` columns (padded to y's width)."""
+    if y.is_cuda:
+        return native.gated_norm(y, w, y.shape[1] // heads, real, parts, eps, z, g, factor, out)
+    v = ref.gated_norm(y, w, y.shape[1] // heads, real, parts, eps, z, g, factor)
+    return v if out is None else out.copy_(v)
+
+
+def panel_append(k, step, cache, block_tokens):
+    """Columns k [T, heads * size] of a projection into the paged panel ``cache`` [blocks, heads, block tokens, size]."""
+    if k.is_cuda:
+        return native.panel_append(k, step.slots, cache, block_tokens)
+    on = step.slots >= 0
+    slots = step.slots[on].long()
+    cache[slots // block_tokens, :, slots % block_tokens] = k[on].unflatten(1, (cache.shape[1], -1))
+
+
+def softcap(z, cap):
+    """cap * tanh(z / cap); fp32 rows are overwritten on the GPU."""
+    return native.softcap(z, cap) if z.is_cuda else cap * torch.tanh(z / cap)
+
+
+@dataclass
+class ShortConv:
+    """Causal convolution per channel with the inputs that earlier steps left: ``w`` [taps, C] (the last row is the current
+    token's), ``ring`` [slots, taps, C] inside the state records (the input of position p in row p mod taps)."""
+    w: torch.Tensor
+    bias: Optional[torch.Tensor]
+    ring: torch.Tensor
+
+
+def _recurrence(x, conv: ShortConv, step, run):
+    """Several-token sequences of a step (convolution, then scan), then its single-token ones (one fused step): ``run`` gets the
+    rows' range, the convolved rows or None, and cu_q, kv_lens and state slots of its sequences."""
+    nm, tm = step.num_multi, step.num_multi_tokens
+    if nm:
+        cu, kv, slots = step.cu_q[:nm + 1], step.kv_lens[:nm], step.state_slots[:nm]
+        run(slice(0, tm), native.causal_conv(x[:tm], conv, cu, kv, slots, step.max_q_len), cu, kv, slots)
+    if step.num_single:
+        run(slice(tm, None), None, None, step.kv_lens[nm:], step.state_slots[nm:])
+
+
+def state_space(x, conv: ShortConv, dt, dt_bias, A, D, state, groups, step):
+    """y_t = S_t^T C_t + D x_t with S_t = exp(-A dt_t) S_(t-1) + dt_t B_t x_t^T per head, dt = softplus(dt + dt_bias), over a
+    step's rows. x [T, heads * P + 2 * groups * N]: raw x | B | C, which pass the short convolution and silu first. ``state``
+    [slots, heads, P, N] (fp32)."""
+    n, H, P, N = state.shape
+    y = torch.empty(x.shape[0], H * P, dtype=x.dtype, device=x.device)
+    if not x.is_cuda:
+        return y.copy_(ref.state_space(x, conv, dt, dt_bias, A, D, state, groups, step))
+    _recurrence(x, conv, step, lambda r, c, cu, kv, slots: native.state_space(
+        x[r], conv, c, dt[r], dt_bias, A, D, y[r], state, groups, cu, kv, slots))
+    return y
+
+
+def delta_rule(x, conv: ShortConv, beta, decay, decay_bias, A, state, groups, q_scale, step):
+    """Gated delta rule over a step's rows: per head S' = diag(g) S, u = beta (v - S'^T k), S = S' + k u^T, o = S^T q, with q and k
+    unit vectors (q times ``q_scale``), beta = sigmoid(beta) and g = exp(-A softplus(decay + decay_bias)) per key channel. x [T,
+    2 * groups * K + heads * V]: raw q | k | v, which pass the short convolution and silu first. ``state`` [slots, heads, V, K]."""
+    n, H, V, _ = state.shape
+    o = torch.empty(x.shape[0], H * V, dtype=x.dtype, device=x.device)
+    if not x.is_cuda:
+        return o.copy_(ref.delta_rule(x, conv, beta, decay, decay_bias, A, state, groups, q_scale, step))
+    _recurrence(x, conv, step, lambda r, c, cu, kv, slots: native.delta_rule(
+        x[r], conv, c, beta[r], decay[r], decay_bias, A, o[r], state, groups, q_scale, cu, kv, slots))
+    return o
 
 
 def glu_clamp(x, limit, alpha=1.702, offset=1.0):
@@ -457,25 +542,27 @@ def refit_stream_rows(x, pos, emb):
         x[pos.long(), :emb.shape[1]] = emb.float()
 
 
-def panel_attention(qkv, k_cache, v_cache, block_tokens, step, Hq, Hkv, scale, window=0, keep=0, sinks=None):
-    """Attention of a step's new rows (multi-token sequences first, then single-token ones) against separate K and V
-    panels, with an optional sliding window (``keep`` first tokens stay visible) and per-head sink logits."""
+def panel_attention(qkv, k_cache, v_cache, block_tokens, step, Hq, Hkv, scale, window=0, keep=0, sinks=None, weights=None, out=None):
+    """Attention of a step's new rows (multi-token sequences first, then single-token ones; the queries are the leading columns of
+    ``qkv``) against separate K and V panels, with an optional sliding window (``keep`` first tokens stay visible) and per-head
+    sink logits, or with the unnormalised ``weights`` of a :class:`SigmoidWeights`."""
     D, Dv = k_cache.shape[-1], v_cache.shape[-1]
     T = qkv.shape[0]
-    out = torch.empty(T, Hq * Dv, dtype=qkv.dtype, device=qkv.device)
+    if out is None:
+        out = torch.empty(T, Hq * Dv, dtype=qkv.dtype, device=qkv.device)
     if not qkv.is_cuda:
         out.copy_(ref.panel_attention(qkv[:, :Hq * D], k_cache, v_cache, step.block_table, step.cu_q, step.kv_lens, Hq, Hkv, scale,
-                                      window, keep, sinks))
+                                      window, keep, sinks, weights))
         return out
     if qkv.dtype == torch.float32:
         native.attention_f32(qkv, qkv.stride(0), out, k_cache, v_cache, block_tokens, step.block_table, step.cu_q, step.kv_lens,
-                             step.num_multi + step.num_single, max(step.max_q_len, 1), Hq, Hkv, scale, window, keep, sinks)
+                             step.num_multi + step.num_single, max(step.max_q_len, 1), Hq, Hkv, scale, window, keep, sinks, weights=weights)
         return out
     nm, ns, tm = step.num_multi, step.num_single, step.num_multi_tokens
     if nm:
         native.paged_prefill(qkv, qkv.stride(0), out, k_cache, k_cache.stride(0), block_tokens, step.block_table, step.cu_q,
                              step.kv_lens, nm, step.max_q_len, Hq, Hkv, D, scale, v_cache=v_cache, window=window, keep=keep,
-                             sinks=sinks)
+                             sinks=sinks, weights=weights)
     if ns:
         seen = min(step.max_kv_len, window + keep + 128) if window > 0 else step.max_kv_len
         n = decode_splits(ns, Hkv * ((Hq // Hkv + 15) // 16), seen)
@@ -485,7 +572,7 @@ def panel_attention(qkv, k_cache, v_cache, block_tokens, step, Hq, Hkv, scale, w
             pml = torch.empty(ns * Hq * n * 2, dtype=torch.float32, device=qkv.device)
         native.paged_decode(qkv[tm:], qkv.stride(0), out[tm:], k_cache, k_cache.stride(0), block_tokens, step.block_table[nm:],
                             step.kv_lens[nm:], ns, Hq, Hkv, D, scale, num_splits=n, part_o=po, part_ml=pml, v_cache=v_cache,
-                            window=window, keep=keep, sinks=sinks)
+                            window=window, keep=keep, sinks=sinks, weights=weights.rows(tm) if weights is not None else None)
     return out
 
 

@@ -8,6 +8,7 @@ from __future__ import annotations
 
 import ctypes as C
 import math
+from dataclasses import dataclass
 from pathlib import Path
 from typing import Optional
 
@@ -35,7 +36,7 @@ _SIGS = {
     "ksana_gemm_smallm": [i32, vp, i32, vp, i32, vp, i32, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32, vp, i64, vp, i32,
                           vp, vp],
     "ksana_gemm_grouped": [i32, vp, i32, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, vp, vp, i32, vp, vp],
-    "ksana_moe_route": [vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32, f32, i32, i32, i32, vp],
+    "ksana_moe_route": [vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32, f32, i32, i32, i32, i32, vp],
     "ksana_moe_align": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
     "ksana_moe_permute": [vp, vp, vp, i32, i32, i32, i32, vp, vp],
     "ksana_moe_combine": [vp, vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
@@ -69,7 +70,17 @@ _SIGS = {
     "ksana_embed_pair": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i64, i64, i64, f32, i32, vp, vp],
     "ksana_residual_norm": [vp, i32, vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, f32, i32, i32, f32, i32, vp, vp, f32,
                             vp, vp, i32, i32, i32, vp, i32, vp, vp],
-    "ksana_glu_clamp": [vp, vp, i32, i32, i32, f32, f32, f32, i32, vp],
+    "ksana_glu_clamp": [vp, vp, i32, i32, i32, f32, f32, f32, vp, i32, vp],
+    "ksana_embed_normed": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, f32, i32, vp, vp],
+    "ksana_token_shift": [vp, i64, vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
+    "ksana_gated_norm": [vp, i64, vp, i64, vp, i64, vp, vp, i64, i32, i32, i32, i32, i32, f32, f32, i32, vp],
+    "ksana_panel_append": [vp, i64, vp, vp, i64, i32, i32, i32, i32, i32, i32, vp, vp],
+    "ksana_softcap": [vp, i64, i32, i32, f32, vp],
+    "ksana_causal_conv": [vp, i64, vp, vp, vp, i64, i32, i32, vp, i64, vp, vp, vp, i32, i32, i32, i32, vp, vp],
+    "ksana_state_space": [vp, i64, vp, vp, vp, i64, i32, vp, i64, vp, i64, vp, vp, vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32,
+                          i32, i32, i32, vp, vp],
+    "ksana_delta_rule": [vp, i64, vp, vp, i64, i32, vp, i64, vp, i64, vp, i64, vp, vp, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32,
+                         i32, i32, f32, i32, vp, vp],
     "ksana_xielu": [vp, i32, vp, i32, i32, i32, f32, f32, f32, i32, vp],
     "ksana_gated_recurrence": [vp, vp, vp, i64, vp, i64, vp, i64, i32, i32, vp, i32, vp, vp, vp, i32, i32, f32, i32, vp, vp],
     "ksana_gemm_f32_batched": [vp, i32, i64, vp, i32, i64, vp, i32, i64, i32, i32, i32, i32, vp, i32, i64, vp],
@@ -80,15 +91,15 @@ _SIGS = {
     "ksana_gemm_grouped_f32": [vp, i32, vp, i32, vp, i32, i32, i32, i32, i32, vp, vp],
     "ksana_refit_rows_f32": [vp, i32, vp, vp, i32, i32, i32, vp, vp],
     "ksana_gemm_f32": [vp, i32, vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, vp],
-    "ksana_attention_f32": [vp, i64, vp, i64, vp, vp, i32, i64, i32, i32, vp, i32, vp, vp, vp, vp, i64, i32, i32, i32, i32, i32, i32, i32,
-                            i32, f32, i32, vp, vp],
+    "ksana_attention_f32": [vp, i64, vp, i64, vp, vp, i32, i64, i32, i32, vp, i32, vp, vp, vp, vp, i64, i32, f32, vp, i32, i32, i32, i32,
+                            i32, i32, i32, i32, i32, f32, i32, vp, vp],
     "ksana_cast_f32": [vp, vp, i64, vp],
     "ksana_paged_prefill_tc": [vp, i64, i64, vp, i64, vp, vp, i64, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32,
-                               i32, i32, f32, i32, vp, vp],
+                               i32, i32, f32, i32, vp, i32, vp, i64, f32, vp, vp],
     "ksana_paged_prefill": [vp, i64, vp, i64, vp, vp, i64, i32, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32,
-                            f32, i32, f32, f32, i32, vp, vp],
+                            f32, i32, f32, f32, i32, vp, i32, vp, i64, f32, vp, vp],
     "ksana_paged_decode": [vp, i64, vp, i64, vp, vp, i64, i32, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, i32,
-                           f32, f32, i32, vp, vp, i32, vp, vp, i32, vp, vp],
+                           f32, f32, i32, vp, vp, i32, vp, vp, i32, vp, i32, vp, i64, f32, vp, vp],
     "ksana_mla_attention": [vp, i64, vp, i64, vp, i64, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp, i64, f32, i32, i32, vp,
                             vp, vp, vp],
     "ksana_mla_rope_append": [vp, i64, i32, vp, i64, vp, f32, vp, vp, vp, vp, vp, i64, i32, i32, i32, i32, i32, i32, i64, i32, vp, vp],
@@ -736,11 +747,12 @@ def residual_norm(x, H, eps, y=None, w1=None, b1=None, ls=None, x_out=None, w2=N
            "ksana_residual_norm")
 
 
-def glu_clamp(x, limit, alpha, offset):
+def glu_clamp(x, limit, alpha, offset, tile_rows=None):
+    """``tile_rows``: of every 128 rows only so many hold anything; the others are skipped."""
     M, I = x.shape[0], x.shape[1] // 2
     out = torch.empty(M, I, dtype=x.dtype, device=x.device)
     _check(lib().ksana_glu_clamp(_p(x), _p(out), M, I, x.stride(0), float(limit), float(alpha), float(offset),
-                                 int(x.dtype == torch.float32), _st()), "ksana_glu_clamp")
+                                 _p(tile_rows), int(x.dtype == torch.float32), _st()), "ksana_glu_clamp")
     return out
 
 
@@ -763,6 +775,97 @@ def gated_recurrence(z, u, g, out, state, block_tokens, block_table, cu_q, kv_le
                                         block_tokens, state.shape[0], _p(block_table), block_table.stride(0), _p(cu_q), _p(kv_lens),
                                         _p(slots), kv_lens.numel(), z.shape[1], float(offset), int(z.dtype == torch.float32),
                                         _p(err_flag(z.device)), _st()), "ksana_gated_recurrence")
+
+
+def embed_normed(ids, positions, table, pos_table, norm_w, real, scale, eps, vocab):
+    """fp32 rows: root-mean-square norm (``real`` columns) of table[id] * scale + pos_table[position]."""
+    T, H = ids.numel(), table.shape[1]
+    x = torch.empty(T, H, dtype=torch.float32, device=table.device)
+    _check(lib().ksana_embed_normed(_p(ids), _p(positions), _p(table), _p(pos_table), _p(norm_w), _p(x), T, H, real, vocab,
+                                    pos_table.shape[0], float(scale), float(eps), int(table.dtype == torch.float32),
+                                    _p(err_flag(table.device)), _st()), "ksana_embed_normed")
+    return x
+
+
+def token_shift(h, mu, ring, cu_q, kv_lens, slots, max_q, out=None):
+    """h + (previous row - h) * mu; ``ring`` [slots, 2, W] (inside the state records) holds the rows of earlier steps."""
+    T, W = h.shape
+    if out is None:
+        out = torch.empty(T, W, dtype=h.dtype, device=h.device)
+    assert ring.dtype == mu.dtype == h.dtype and ring.stride(2) == 1 and ring.stride(1) == W and ring.shape[1] == 2
+    _check(lib().ksana_token_shift(_p(h), h.stride(0), _p(mu), _p(out), out.stride(0), _p(ring), ring.stride(0), _p(cu_q), _p(kv_lens),
+                                   _p(slots), ring.shape[0], kv_lens.numel(), max_q, W, int(h.dtype == torch.float32),
+                                   _p(err_flag(h.device)), _st()), "ksana_token_shift")
+    return out
+
+
+def gated_norm(y, w, pad, real, parts, eps, z=None, g=None, factor=1.0, out=None):
+    """factor * norm(y * silu(z)) * w * sigmoid(g) with the root mean square of each of ``parts`` equal parts of a row; the row is
+    heads of ``pad`` columns, of which ``real`` count."""
+    T, C = y.shape
+    if out is None:
+        out = torch.empty(T, C, dtype=y.dtype, device=y.device)
+    assert w.dtype == y.dtype and w.numel() == C
+    ld = lambda t: t.stride(0) if t is not None else 0  # noqa: E731
+    _check(lib().ksana_gated_norm(_p(y), y.stride(0), _p(z), ld(z), _p(g), ld(g), _p(w), _p(out), out.stride(0), T, C, pad, real, parts,
+                                  float(eps), float(factor), int(y.dtype == torch.float32), _st()), "ksana_gated_norm")
+    return out
+
+
+def panel_append(k, slots, cache, block_tokens):
+    """Columns k [T, heads * size] of a projection to the paged panel ``cache`` [blocks, heads, block tokens, size]."""
+    _check(lib().ksana_panel_append(_p(k), k.stride(0), _p(slots), _p(cache), cache.stride(0), block_tokens, cache.shape[0],
+                                    cache.shape[1], cache.shape[3], k.shape[0], int(k.dtype == torch.float32), _p(err_flag(k.device)),
+                                    _st()), "ksana_panel_append")
+
+
+def softcap(z, cap):
+    """cap * tanh(z / cap) of fp32 rows, in place."""
+    assert z.dtype == torch.float32 and z.stride(1) == 1
+    _check(lib().ksana_softcap(_p(z), z.stride(0), z.shape[0], z.shape[1], float(cap), _st()), "ksana_softcap")
+    return z
+
+
+def _conv_args(x, conv):
+    ring, w = conv.ring, conv.w
+    assert x.stride(1) == 1 and w.dtype == x.dtype == ring.dtype and w.is_contiguous() and ring.stride(2) == 1
+    assert ring.shape[1:] == w.shape and ring.stride(1) == w.shape[1] == x.shape[1]
+    return _p(x), x.stride(0), _p(w), conv.bias, _p(ring), ring.stride(0), w.shape[0]
+
+
+def causal_conv(x, conv, cu_q, kv_lens, slots, max_q):
+    """silu(conv(x) + bias) over the new rows x [T, C] of sequences of any number of new tokens; ``conv``: a
+    :class:`ksanallm_b200.ops.dispatch.ShortConv`."""
+    px, ld, w, bias, ring, rs, taps = _conv_args(x, conv)
+    out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
+    _check(lib().ksana_causal_conv(px, ld, w, _p(bias), ring, rs, taps, x.shape[1], _p(out), out.stride(0), _p(cu_q), _p(kv_lens),
+                                   _p(slots), conv.ring.shape[0], kv_lens.numel(), max_q, int(x.dtype == torch.float32),
+                                   _p(err_flag(x.device)), _st()), "ksana_causal_conv")
+    return out
+
+
+def state_space(x, conv, c, dt, dt_bias, A, D, y, state, G, cu_q, kv_lens, slots):
+    """State-space recurrence: a scan over convolved rows ``c`` (``cu_q`` given), or one token per sequence straight from the raw
+    rows ``x``. ``state`` [slots, heads, columns, keys] fp32 inside the state records; y [T, heads * columns] receives the result."""
+    px, ld, w, bias, ring, rs, taps = _conv_args(x, conv)
+    n, H, P, N = state.shape
+    assert state.dtype == torch.float32 and state[0].is_contiguous() and dt.stride(1) == y.stride(1) == 1
+    _check(lib().ksana_state_space(px, ld, w, _p(bias), ring, rs, taps, _p(c), c.stride(0) if c is not None else 0, _p(dt), dt.stride(0),
+                                   _p(dt_bias), _p(A), _p(D), _p(y), y.stride(0), _p(state), state.stride(0), _p(cu_q), _p(kv_lens),
+                                   _p(slots), n, kv_lens.numel(), H, G, P, N, int(x.dtype == torch.float32), _p(err_flag(x.device)),
+                                   _st()), "ksana_state_space")
+
+
+def delta_rule(x, conv, c, beta, decay, decay_bias, A, o, state, G, q_scale, cu_q, kv_lens, slots):
+    """Gated delta rule, forms as in :func:`state_space`; ``state`` [slots, heads, value size, key size]."""
+    px, ld, w, bias, ring, rs, taps = _conv_args(x, conv)
+    assert bias is None
+    n, H, V, Kd = state.shape
+    assert state.dtype == torch.float32 and state[0].is_contiguous() and beta.stride(1) == decay.stride(1) == o.stride(1) == 1
+    _check(lib().ksana_delta_rule(px, ld, w, ring, rs, taps, _p(c), c.stride(0) if c is not None else 0, _p(beta), beta.stride(0),
+                                  _p(decay), decay.stride(0), _p(decay_bias), _p(A), _p(o), o.stride(0), _p(state), state.stride(0),
+                                  _p(cu_q), _p(kv_lens), _p(slots), n, kv_lens.numel(), H, G, Kd, V, float(q_scale),
+                                  int(x.dtype == torch.float32), _p(err_flag(x.device)), _st()), "ksana_delta_rule")
 
 
 def gemm_f32_batched(a, w, out, gate=None):
@@ -808,10 +911,33 @@ def _panels(cache_layer, v_cache, D):
     return cache_layer.data_ptr(), cache_layer.data_ptr() + cache_layer.stride(1) * cache_layer.element_size(), D
 
 
+@dataclass
+class SigmoidWeights:
+    """Attention whose weights are sigmoid(score + bias[head, distance]), not normalised over keys. ``bias`` [heads, n] fp32:
+    distances from n - 1 on have the last value. ``gate`` [rows, heads * value size]: outputs are multiplied by its sigmoid and
+    by ``factor``."""
+    bias: torch.Tensor
+    gate: Optional[torch.Tensor] = None
+    factor: float = 1.0
+
+    def rows(self, first: int) -> "SigmoidWeights":
+        return SigmoidWeights(self.bias, self.gate[first:] if self.gate is not None else None, self.factor)
+
+
+def _sigmoid_args(weights: Optional[SigmoidWeights]):
+    if weights is None:
+        return None, 0, None, 0, 1.0
+    b, g = weights.bias, weights.gate
+    assert b.dtype == torch.float32 and b.is_contiguous() and (g is None or g.stride(1) == 1) and (g is not None or weights.factor == 1.0)
+    return _p(b), b.shape[1], _p(g), g.stride(0) if g is not None else 0, float(weights.factor)
+
+
 def paged_prefill(q, q_stride, out, cache_layer, block_stride, block_tokens, block_table, cu_q, kv_lens, B, max_q_len,
-                  Hq, Hkv, D, scale, alibi=None, k_scale=1.0, v_scale=1.0, v_cache=None, window=0, keep=0, sinks=None):
+                  Hq, Hkv, D, scale, alibi=None, k_scale=1.0, v_scale=1.0, v_cache=None, window=0, keep=0, sinks=None,
+                  weights=None):
     """``v_cache``: V panels of their own (``cache_layer`` then holds the K panels). ``window`` > 0: position i sees j <= i
-    with i - j < window or j < keep. ``sinks``: fp32 [Hq] logits in the softmax denominator."""
+    with i - j < window or j < keep. ``sinks``: fp32 [Hq] logits in the softmax denominator. ``weights``: see
+    :class:`SigmoidWeights`."""
     fp8 = cache_layer.dtype != torch.bfloat16
     kc, vc, Dv = _panels(cache_layer, v_cache, D)
     nblocks = int(cache_layer.shape[0])
@@ -820,22 +946,22 @@ def paged_prefill(q, q_stride, out, cache_layer, block_stride, block_tokens, blo
         rc = lib().ksana_paged_prefill_tc(_p(q), q_stride, q.shape[0], _p(out), out.stride(0), kc, vc, block_stride,
                                           block_tokens, _p(block_table), block_table.stride(0), _p(cu_q), _p(kv_lens),
                                           _p(alibi), _p(sinks), B, max_q_len, Hq, Hkv, D, Dv, window, keep, float(scale),
-                                          nblocks, _p(err_flag(q.device)), _st())
+                                          nblocks, *_sigmoid_args(weights), _p(err_flag(q.device)), _st())
         if rc != -100:
             _check(rc, "ksana_paged_prefill_tc")
             return
     rc = lib().ksana_paged_prefill(_p(q), q_stride, _p(out), out.stride(0), kc, vc, block_stride, block_tokens,
                                    _p(block_table), block_table.stride(0), _p(cu_q), _p(kv_lens), _p(alibi), _p(sinks), B,
                                    max_q_len, Hq, Hkv, D, Dv, window, keep, float(scale), int(fp8), float(k_scale),
-                                   float(v_scale), nblocks, _p(err_flag(q.device)), _st())
+                                   float(v_scale), nblocks, *_sigmoid_args(weights), _p(err_flag(q.device)), _st())
     _check(rc, "ksana_paged_prefill")
 
 
 def paged_decode(q, q_stride, out, cache_layer, block_stride, block_tokens, block_table, kv_lens, B, Hq, Hkv, D, scale,
                  alibi=None, k_scale=1.0, v_scale=1.0, num_splits=1, part_o=None, part_ml=None, out_q=None,
-                 out_scale=None, v_cache=None, window=0, keep=0, sinks=None):
+                 out_scale=None, v_cache=None, window=0, keep=0, sinks=None, weights=None):
     """``out_q`` / ``out_scale`` (head dim 128): the output also (or, with ``out`` None, only) as the FP8 operand of the
-    next GEMM: e4m3 [B, Hq * D] and scales [Hq, ld]. ``v_cache`` / ``window`` / ``keep`` / ``sinks``: see
+    next GEMM: e4m3 [B, Hq * D] and scales [Hq, ld]. ``v_cache`` / ``window`` / ``keep`` / ``sinks`` / ``weights``: see
     :func:`paged_prefill`."""
     fp8 = cache_layer.dtype != torch.bfloat16
     kc, vc, Dv = _panels(cache_layer, v_cache, D)
@@ -843,20 +969,24 @@ def paged_decode(q, q_stride, out, cache_layer, block_stride, block_tokens, bloc
                                   block_stride, block_tokens, _p(block_table), block_table.stride(0), _p(kv_lens), _p(alibi),
                                   _p(sinks), B, Hq, Hkv, D, Dv, window, keep, float(scale), int(fp8), float(k_scale),
                                   float(v_scale), num_splits, _p(part_o), _p(part_ml), int(cache_layer.shape[0]), _p(out_q),
-                                  _p(out_scale), out_scale.stride(0) if out_scale is not None else 0,
+                                  _p(out_scale), out_scale.stride(0) if out_scale is not None else 0, *_sigmoid_args(weights),
                                   _p(err_flag(q.device)), _st())
     _check(rc, "ksana_paged_decode")
 
 
 def attention_f32(q, q_stride, out, k_cache, v_cache, block_tokens, block_table, cu_q, kv_lens, B, max_q_len, Hq, Hkv, scale,
-                  window=0, keep=0, sinks=None, gate=None):
+                  window=0, keep=0, sinks=None, gate=None, weights=None):
     """All of a step's new rows (any lengths) against K and V panels, in 32-bit arithmetic throughout (bf16 storage is fine).
-    ``v_cache`` may be a column range of ``k_cache``. ``gate`` [rows, heads]: outputs are multiplied by its sigmoid."""
-    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1)
+    ``v_cache`` may be a column range of ``k_cache``. ``gate`` [rows, heads]: outputs are multiplied by its sigmoid.
+    ``weights``: see :class:`SigmoidWeights`."""
+    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and weights is None)
+    bias, bias_len, wide, wide_ld, factor = _sigmoid_args(weights)
     rc = lib().ksana_attention_f32(_p(q), q_stride, _p(out), out.stride(0), _p(k_cache), _p(v_cache), v_cache.stride(-2),
                                    k_cache.stride(0), block_tokens, k_cache.shape[0], _p(block_table), block_table.stride(0),
-                                   _p(cu_q), _p(kv_lens), _p(sinks), _p(gate), gate.stride(0) if gate is not None else 0, B, max_q_len,
-                                   Hq, Hkv, k_cache.shape[-1], v_cache.shape[-1], window, keep, float(scale), int(q.dtype == torch.float32), _p(err_flag(q.device)), _st())
+                                   _p(cu_q), _p(kv_lens), _p(sinks), _p(gate) if wide is None else wide,
+                                   gate.stride(0) if gate is not None else wide_ld, int(wide is not None), factor, bias, bias_len, B,
+                                   max_q_len, Hq, Hkv, k_cache.shape[-1], v_cache.shape[-1], window, keep, float(scale),
+                                   int(q.dtype == torch.float32), _p(err_flag(q.device)), _st())
     _check(rc, "ksana_attention_f32")
 
 
@@ -1033,14 +1163,16 @@ def gemm_grouped(a, w, tile_expert, E, N, out=None, a_scale=None, w_scale=None, 
     return out
 
 
-def moe_route(logits, K, scoring="softmax", renorm=True, scale=1.0, bias=None, n_group=1, topk_group=1, E=None, gate_col=-1):
+def moe_route(logits, K, scoring="softmax", renorm=True, scale=1.0, bias=None, n_group=1, topk_group=1, E=None, gate_col=-1,
+              group_top=2):
     """Expert choice by rows of router logits (the first ``E`` columns of fp32 rows): (ids [T, K] int32, weights fp32 [T, K], or
-    [T, K + 1] with ``gate_col``: the sigmoid of that column comes last)."""
+    [T, K + 1] with ``gate_col``: the sigmoid of that column comes last). A group's score is the sum of its two largest choice
+    scores, or with ``group_top`` 1 its largest."""
     T, E = logits.shape[0], logits.shape[1] if E is None else E
     ids = torch.empty(T, K, dtype=torch.int32, device=logits.device)
     w = torch.empty(T, K + (gate_col >= 0), dtype=torch.float32, device=logits.device)
     rc = lib().ksana_moe_route(_p(logits), logits.stride(0), _p(bias), _p(ids), _p(w), w.stride(0), T, E, K,
-                               0 if scoring == "softmax" else 1, int(renorm), float(scale), n_group, topk_group, gate_col, _st())
+                               0 if scoring == "softmax" else 1, int(renorm), float(scale), n_group, topk_group, group_top, gate_col, _st())
     _check(rc, "ksana_moe_route")
     return ids, w
 

@@ -319,6 +319,85 @@ def gated_recurrence(z, u, g, state, block_tokens, block_table, cu_q, kv_lens, o
     return out
 
 
+def _new_rows(cu_q, kv_lens, slots):
+    """(state slot, rows, position of the first new token) of every sequence with new rows."""
+    for s in range(kv_lens.numel()):
+        q0, q1 = int(cu_q[s]), int(cu_q[s + 1])
+        if q1 > q0 and int(slots[s]) >= 0:
+            yield int(slots[s]), slice(q0, q1), int(kv_lens[s]) - (q1 - q0)
+
+
+def _with_history(x, ring, slot, past):
+    """x with the ring's rows that come before it in front (zeros before the sequence); the ring takes x's last rows."""
+    n = ring.shape[1]
+    back = [ring[slot, (past - b) % n] if past - b >= 0 else torch.zeros_like(x[0]) for b in range(n - 1, 0, -1)]
+    out = torch.cat([torch.stack(back), x]) if back else x
+    for t in range(max(0, x.shape[0] - n), x.shape[0]):
+        ring[slot, (past + t) % n] = x[t]
+    return out
+
+
+def token_shift(h, mu, ring, cu_q, kv_lens, slots):
+    out = torch.empty_like(h)
+    for slot, r, past in _new_rows(cu_q, kv_lens, slots):
+        f = _with_history(h[r], ring, slot, past).float()
+        out[r] = (f[1:] + (f[:-1] - f[1:]) * mu.float()).to(h.dtype)
+    return out
+
+
+def gated_norm(y, w, pad, real, parts, eps, z=None, g=None, factor=1.0):
+    v = y.float() if z is None else y.float() * torch.nn.functional.silu(z.float())
+    v = v.unflatten(1, (-1, pad))
+    parts_ = v[..., :real].flatten(1).unflatten(1, (parts, -1))
+    rstd = torch.rsqrt(parts_.pow(2).mean(-1, keepdim=True) + eps)
+    n = torch.zeros_like(v)
+    n[..., :real] = (parts_ * rstd).flatten(1).unflatten(1, (-1, real))
+    n = n.flatten(1) * w.float() * factor
+    return (n if g is None else n * torch.sigmoid(g.float())).to(y.dtype)
+
+
+def _convolved(x, conv, slot, past):
+    f, taps = _with_history(x, conv.ring, slot, past).float(), conv.w.shape[0]
+    y = sum(f[j:j + x.shape[0]] * conv.w[j].float() for j in range(taps))
+    return torch.nn.functional.silu(y if conv.bias is None else y + conv.bias.float())
+
+
+def state_space(x, conv, dt, dt_bias, A, D, state, groups, step):
+    n, H, P, N = state.shape
+    out = torch.zeros(x.shape[0], H * P)
+    for slot, r, past in _new_rows(step.cu_q, step.kv_lens, step.state_slots):
+        c = _convolved(x[r], conv, slot, past).to(x.dtype).float()
+        xs = c[:, :H * P].unflatten(1, (H, P))
+        B, C = (t.unflatten(1, (groups, N)).repeat_interleave(H // groups, 1) for t in c[:, H * P:].chunk(2, 1))
+        d = torch.nn.functional.softplus(dt[r][:, :H].float() + dt_bias)
+        S = state[slot] if past > 0 else torch.zeros_like(state[slot])
+        for t in range(xs.shape[0]):
+            S = S * torch.exp(-A * d[t])[:, None, None] + (d[t][:, None] * xs[t])[:, :, None] * B[t][:, None, :]
+            out[r.start + t] = ((S * C[t][:, None, :]).sum(-1) + D[:, None] * xs[t]).flatten()
+        state[slot] = S
+    return out
+
+
+def delta_rule(x, conv, beta, decay, decay_bias, A, state, groups, q_scale, step):
+    n, H, V, K = state.shape
+    out = torch.zeros(x.shape[0], H * V)
+    for slot, r, past in _new_rows(step.cu_q, step.kv_lens, step.state_slots):
+        c = _convolved(x[r], conv, slot, past).to(x.dtype).float()
+        q, k = (t.unflatten(1, (groups, K)) for t in c[:, :2 * groups * K].chunk(2, 1))
+        q, k = ((t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) + 1e-6)).repeat_interleave(H // groups, 1) for t in (q, k))
+        q, v = q * q_scale, c[:, 2 * groups * K:].unflatten(1, (H, V))
+        b = torch.sigmoid(beta[r][:, :H].float())
+        g = torch.exp(-A[:, None] * torch.nn.functional.softplus(decay[r].float() + decay_bias).unflatten(1, (H, K)))
+        S = state[slot] if past > 0 else torch.zeros_like(state[slot])
+        for t in range(v.shape[0]):
+            S = S * g[t][:, None, :]
+            u = b[t][:, None] * (v[t] - (S * k[t][:, None, :]).sum(-1))
+            S = S + u[:, :, None] * k[t][:, None, :]
+            out[r.start + t] = (S * q[t][:, None, :]).sum(-1).flatten()
+        state[slot] = S
+    return out
+
+
 def latent_append(q, nope, kv, norm_w, eps, rank, positions, slots, cos_sin, qfull, cache, block_tokens):
     """q [T, G, nope + rotary] -> rotary columns of qfull [T, G, DK]; normed latents | rotated key of kv [T, DK] into the
     panel [blocks, block tokens, DK]."""
@@ -377,14 +456,14 @@ def latent_norms(q, kv, q_w, kv_w, eps, q_rank, kv_rank, slots, cache, block_tok
     return normed(q, q_w, q_rank).to(q.dtype)
 
 
-def moe_route(logits, K, scoring="softmax", renorm=True, scale=1.0, bias=None, n_group=1, topk_group=1, E=None, gate_col=-1):
+def moe_route(logits, K, scoring="softmax", renorm=True, scale=1.0, bias=None, n_group=1, topk_group=1, E=None, gate_col=-1, group_top=2):
     """(ids [T, K] int64, weights fp32 [T, K (+ 1)]); see native.moe_route."""
     z = logits[:, :logits.shape[1] if E is None else E].float()
     score = torch.sigmoid(z) if scoring == "sigmoid" else torch.softmax(z, dim=-1)
     sel = score + (bias.float() if bias is not None else 0.0)
     if n_group > 1 and topk_group < n_group:
         grp = sel.unflatten(-1, (n_group, -1))
-        gscore = grp.topk(min(2, grp.shape[-1]), dim=-1).values.sum(-1)
+        gscore = grp.topk(min(group_top, grp.shape[-1]), dim=-1).values.sum(-1)
         keep = torch.zeros_like(gscore, dtype=torch.bool).scatter_(1, gscore.topk(topk_group, dim=-1).indices, True)
         sel = grp.masked_fill(~keep.unsqueeze(-1), float("-inf")).flatten(-2)
     ids = sel.topk(K, dim=-1).indices
@@ -398,14 +477,18 @@ def moe_route(logits, K, scoring="softmax", renorm=True, scale=1.0, bias=None, n
 
 
 def expert_sum(y, dst_row, w, shared=None):
-    """fp32 rows: sum over k of w[t, k] * y[dst_row[t, k]] (negative: left out), plus w[t, K] * shared[t]."""
+    """fp32 rows: sum over k of w[t, k] * y[dst_row[t, k]] (negative: left out), plus w[t, K] * shared[t] (without such a
+    weight: plus shared[t])."""
     rows = y.float()[dst_row.clamp_min(0).long()].masked_fill((dst_row < 0).unsqueeze(-1), 0.0)
     out = (rows * w[:, :dst_row.shape[1], None]).sum(1)
-    return out if shared is None else out + shared.float() * w[:, dst_row.shape[1], None]
+    if shared is None:
+        return out
+    return out + (shared.float() * w[:, dst_row.shape[1], None] if w.shape[1] > dst_row.shape[1] else shared.float())
 
 
-def panel_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, Hq, Hkv, scale, window=0, keep=0, sinks=None):
-    """q [T, Hq*D] (new tokens only) -> [T, Hq*Dv]; see the sliding window and sink in dispatch.panel_attention."""
+def panel_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, Hq, Hkv, scale, window=0, keep=0, sinks=None, weights=None):
+    """q [T, Hq*D] (new tokens only) -> [T, Hq*Dv]; see the sliding window, the sink and the unnormalised weights in
+    dispatch.panel_attention."""
     T, G, D, Dv, bt = q.shape[0], Hq // Hkv, k_cache.shape[-1], v_cache.shape[-1], k_cache.shape[2]
     out = torch.zeros(T, Hq * Dv, dtype=q.dtype, device=q.device)
     for s in range(kv_lens.numel()):
@@ -423,6 +506,14 @@ def panel_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, Hq, Hkv, sc
         hide = kpos > qpos
         if window > 0:
             hide = hide | ((qpos - kpos >= window) & (kpos >= keep))
+        if weights is not None:
+            far = (qpos - kpos).clamp(0, weights.bias.shape[1] - 1)
+            att = torch.sigmoid(att + weights.bias[:, far].unflatten(0, (Hkv, G)))
+            o = torch.einsum("hgqk,hkd->hgqd", att.masked_fill(hide, 0.0), v).permute(2, 0, 1, 3).reshape(ql, Hq * Dv)
+            if weights.gate is not None:
+                o = o * torch.sigmoid(weights.gate[q0:q1].float()) * weights.factor
+            out[q0:q1] = o.to(q.dtype)
+            continue
         att = att.masked_fill(hide, float("-inf"))
         if sinks is not None:
             att = torch.cat([att, sinks.float().reshape(Hkv, G, 1, 1).expand(-1, -1, ql, 1)], dim=-1)

@@ -92,7 +92,8 @@ class Request:
 class ModelRunner:
     """Owns the model, its KV cache and the per-step device metadata."""
 
-    def __init__(self, model, block_tokens: int, num_blocks: int, num_host_blocks: int, kv_dtype=None):
+    def __init__(self, model, block_tokens: int, num_blocks: int, num_host_blocks: int, kv_dtype=None,
+                 num_state_slots: int = 0, num_host_state_slots: int = 0):
         self.model = model
         self.device = model.device
         self.cuda = self.device.type == "cuda"
@@ -103,12 +104,20 @@ class ModelRunner:
         if num_host_blocks > 0:
             self.host_cache = torch.zeros(num_host_blocks, self.block_bytes, dtype=torch.uint8,
                                           pin_memory=self.cuda)
+        self.host_state = None
+        if num_state_slots:
+            model.allocate_state(num_state_slots)
+            if num_host_state_slots:
+                self.host_state = torch.zeros(num_host_state_slots, model.state_bytes(), dtype=torch.uint8, pin_memory=self.cuda)
         self._ring: list = []
         self._ring_pos = 0
         self._swap_stream = None
         self.exchange_candidates = os.environ.get("KSANA_SHARD_SAMPLING", "1") != "0"
         self.pipeline = None             # parallel.pipeline.PipelineRunner when the job has several stages
-        self.needs_prev_ids = bool(getattr(model, "needs_prev_ids", False))
+        # what some models read beside the common step metadata, behind it in the uploads: (field of the plan and of the
+        # step, per row instead of per sequence, value in padding rows)
+        self.tail_fields = [f for f, on in ((("prev_ids", True, -1), "needs_prev_ids"), (("state_slots", False, -1), "needs_state_slots"))
+                            if getattr(model, on, False)]
         self.h2d_bytes = 0
         self.d2h_bytes = 0
 
@@ -148,11 +157,51 @@ class ModelRunner:
         slot[2].record()
         return out
 
+    def _apply_state_ops(self, plan) -> None:
+        """Copies of forked sequences' states, then states of preempted sequences to the host, then those of resumed ones
+        back, in stream order with the block operations of the same step."""
+        lists = [np.asarray(getattr(plan, k, ()), dtype=np.int32) for k in ("state_copies", "state_out", "state_in")]
+        if not any(a.size for a in lists):
+            return
+        state = self.model.state
+        if (lists[1].size or lists[2].size) and self.host_state is None:
+            raise RuntimeError("swap requested without a host state pool")
+        if self.cuda:
+            dev = self._stage(np.concatenate([a.reshape(-1) for a in lists]))
+            copies, out, back = dev.split([a.size for a in lists])
+            bytes_ = self.model.state_bytes()
+            if copies.numel():
+                native.copy_blocks(state, copies, bytes_)
+            if out.numel():
+                native.swap_blocks(state, self.host_state, out, bytes_, to_host=True)
+            if back.numel():
+                native.swap_blocks(state, self.host_state, back, bytes_, to_host=False)
+            return
+        raw = state.view(torch.uint8)
+        copies, out, back = (torch.from_numpy(a.reshape(-1, 2).astype(np.int64)) for a in lists)
+        raw[copies[:, 1]] = raw[copies[:, 0]]
+        if out.numel():
+            self.host_state[out[:, 1]] = raw[out[:, 0]]
+        if back.numel():
+            raw[back[:, 0]] = self.host_state[back[:, 1]]
+
+    def _tail(self, plan, rows=None, seqs=None) -> np.ndarray:
+        """The plan's values of ``tail_fields``, padded to ``rows`` rows and ``seqs`` sequences."""
+        parts = []
+        for name, per_row, fill in self.tail_fields:
+            v = np.asarray(getattr(plan, name), dtype=np.int32)
+            n = rows if per_row else seqs
+            if n is not None:
+                v = np.concatenate([v, np.full(n - v.size, fill, dtype=np.int32)])
+            parts.append(v)
+        return np.concatenate(parts) if parts else np.zeros(0, np.int32)
+
     def apply_block_ops(self, plan) -> None:
         """Block copies of forks decided after the previous step, then swap-outs, swap-ins and the copies decided by
         this plan, in that order. On a GPU the four lists travel in one staged upload; a swap is one kernel per
         direction that moves the blocks between the cache and the pinned host pool over PCIe (no staging copy, no
         host synchronisation), issued on a side stream that the compute stream joins before the forward."""
+        self._apply_state_ops(plan)
         pre = np.asarray(getattr(plan, "pre_copies", ()), dtype=np.int32)
         so, si, cp = np.asarray(plan.swap_out, dtype=np.int32), np.asarray(plan.swap_in, dtype=np.int32), \
             np.asarray(plan.copies, dtype=np.int32)
@@ -204,18 +253,18 @@ class ModelRunner:
     def _stage_plan(self, plan) -> torch.Tensor:
         """The step's device metadata (ids, positions, slots, sequence offsets, lengths, block table, sample rows) in
         one upload. A scheduler plan writes its image straight into the pinned staging buffer."""
-        prev = np.asarray(plan.prev_ids, dtype=np.int32) if self.needs_prev_ids else np.zeros(0, np.int32)
+        tail = self._tail(plan)
         if self.cuda and hasattr(plan, "write_step_image"):
-            n = int(plan.step_image_words()) + prev.size
+            n = int(plan.step_image_words()) + tail.size
             slot = self._stage_buffer(n)
             plan.write_step_image(slot[0].data_ptr(), slot[1])
-            if prev.size:
-                slot[0].numpy()[n - prev.size:n] = prev
+            if tail.size:
+                slot[0].numpy()[n - tail.size:n] = tail
             self.h2d_bytes += n * 4
             dev = slot[0][:n].to(self.device, non_blocking=True)
             slot[2].record()
             return dev
-        parts = [plan.input_ids, plan.positions, plan.slots, plan.cu_q, plan.kv_lens, plan.block_table, plan.sample_rows, prev]
+        parts = [plan.input_ids, plan.positions, plan.slots, plan.cu_q, plan.kv_lens, plan.block_table, plan.sample_rows, tail]
         return self._stage(np.concatenate([np.asarray(p, dtype=np.int32).reshape(-1) for p in parts]))
 
     def _patch_ids(self, ids: torch.Tensor, patch) -> None:
@@ -250,8 +299,8 @@ class ModelRunner:
         rows = take(nsamp)
         step = StepInput(input_ids, positions, slots, cu_q, kv_lens, table, plan.num_multi, plan.num_single, T,
                          plan.num_multi_tokens, plan.max_q_len, logits_rows=rows)
-        if self.needs_prev_ids:
-            step.prev_ids = take(T)
+        for name, per_row, _ in self.tail_fields:
+            setattr(step, name, take(T if per_row else nseq))
         kv_lens = np.asarray(plan.kv_lens)
         step.max_kv_len = int(kv_lens.max()) if nseq else 0
         step.sample_k = self.candidate_k(plan, extra)
@@ -305,7 +354,7 @@ class ModelRunner:
             return g
         mb = self.graph_max_blocks
         n = 4 * bs + bs * mb
-        img = torch.zeros(n + (bs if self.needs_prev_ids else 0), dtype=torch.int32, device=self.device)
+        img = torch.zeros(n + bs * len(self.tail_fields), dtype=torch.int32, device=self.device)
         ids, pos, slots, kvl = img[0:bs], img[bs:2 * bs], img[2 * bs:3 * bs], img[3 * bs:4 * bs]
         table = img[4 * bs:n].view(bs, mb)
         slots.fill_(-1)
@@ -314,8 +363,8 @@ class ModelRunner:
         step.decode_splits = ops.decode_splits(bs, self.model.Hkv, self.graph_max_kv)
         step.max_kv_len = self.graph_max_kv
         step.sample_k = kx
-        if self.needs_prev_ids:
-            step.prev_ids = img[n:]
+        for i, (name, _, fill) in enumerate(self.tail_fields):
+            setattr(step, name, img[n + i * bs:n + (i + 1) * bs].fill_(fill))
         side = torch.cuda.Stream(device=self.device)
         side.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(side):
@@ -340,14 +389,12 @@ class ModelRunner:
         bs = next(b for b in self.GRAPH_SIZES if b >= nseq)
         graph, img, logits, mb, _step = self._graph_for(bs, self.candidate_k(plan, None))
         n0 = n = 4 * bs + bs * mb
-        prev = np.full(bs if self.needs_prev_ids else 0, -1, dtype=np.int32)
-        if prev.size:
-            prev[:nseq] = plan.prev_ids
-            n += bs
+        tail = self._tail(plan, bs, bs)
+        n += tail.size
         if hasattr(plan, "write_decode_image"):
             slot = self._stage_buffer(n)                  # the plan writes the padded image into pinned memory itself
             plan.write_decode_image(slot[0].data_ptr(), slot[1], bs, mb)
-            slot[0].numpy()[n0:n] = prev
+            slot[0].numpy()[n0:n] = tail
             self.h2d_bytes += n * 4
             img.copy_(slot[0][:n], non_blocking=True)
             slot[2].record()
@@ -358,7 +405,7 @@ class ModelRunner:
             host[2 * bs:3 * bs] = -1
             host[2 * bs:2 * bs + nseq] = plan.slots
             host[3 * bs:3 * bs + nseq] = plan.kv_lens
-            host[n0:] = prev
+            host[n0:] = tail
             tbl = host[4 * bs:n0].reshape(bs, mb)
             tbl[:nseq, :plan.max_blocks] = np.asarray(plan.block_table).reshape(nseq, plan.max_blocks)
             self._stage(host, out=img)
@@ -418,6 +465,13 @@ class LLMEngine:
         sc.resume_at_block_ends = bool(getattr(model, "carries_state", False))
         if bs.min_flexible_cache_num > 0 and not getattr(model, "moves_blocks", True):
             raise ValueError(f"{model_cfg.model_type}: cached blocks cannot be moved to another position (min_flexible_cache_num)")
+        if getattr(model, "needs_state_slots", False):
+            sc.num_state_slots = bs.max_batch_size
+            sc.num_host_state_slots = bs.max_batch_size if num_host_blocks > 0 and bs.preempt_mode == 0 else 0
+            if sc.enable_prefix_cache:
+                logger.warning(f"{model_cfg.model_type}: state of recurrent layers exists for whole sequences only, "
+                               "the prefix cache is off")
+                sc.enable_prefix_cache = False
         sc.block_token_num = cfg.block_manager.block_token_num
         sc.eos_token_ids = list(model_cfg.eos_token_ids)
         dp = getattr(model, "dp", None)
@@ -429,7 +483,8 @@ class LLMEngine:
             raise ValueError(f"{num_blocks} KV blocks of {sc.block_token_num} tokens cannot hold max_token_len "
                              f"{sc.max_token_len}")
         self.scheduler = ne.Scheduler(sc, num_blocks, num_host_blocks) if rank == 0 else None
-        self.runner = ModelRunner(model, sc.block_token_num, num_blocks, num_host_blocks, kv_dtype)
+        self.runner = ModelRunner(model, sc.block_token_num, num_blocks, num_host_blocks, kv_dtype, sc.num_state_slots,
+                                  sc.num_host_state_slots)
         self.runner.pipeline = pipeline
         if cfg.global_.enable_cuda_graph:
             self.runner.enable_graphs(bs.max_batch_size, sc.max_token_len)
