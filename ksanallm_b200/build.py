@@ -23,6 +23,8 @@ NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "--use_fast_math", "-Xcompiler", "-fPIC", "-Xcompiler", "-Wno-unused-function",
 ]
+# sources whose exponentials, divisions and roots feed long recurrences: no approximations that they do not ask for by name
+PRECISE = {"state_scan", "stream_ops"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread", "-Wall", "-Wno-sign-compare"]
 
 
@@ -82,7 +84,8 @@ def build_kernels(force: bool = False, verbose: bool = False, only=None) -> Path
             continue
         objs.append(o)
         if stale:
-            cmd = [_nvcc(), *NVCC_FLAGS, "-I", str(kdir), "-c", str(s), "-o", str(o)]
+            flags = [f for f in NVCC_FLAGS if f != "--use_fast_math" or s.stem not in PRECISE]
+            cmd = [_nvcc(), *flags, "-I", str(kdir), "-c", str(s), "-o", str(o)]
             if verbose:
                 cmd.insert(1, "-Xptxas")
                 cmd.insert(2, "-v")

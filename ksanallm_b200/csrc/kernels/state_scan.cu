@@ -33,8 +33,11 @@ constexpr int kSlab = kScanThreads / kLanes * kCols;
 constexpr int kMaxTaps = 16;
 constexpr float kUnitEps = 1e-6f;
 
-__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(__expf(-fabsf(x))); }
-__device__ __forceinline__ float silu_f(float x) { return x * sigmoid_f(x); }
+__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// exp(-x), x >= 0, rounded to nearest near 1: a decay is applied once per token, a bias of its last bit would add up
+__device__ __forceinline__ float decay_f(float x) { return 1.f + expm1f(-x); }
+__device__ __forceinline__ float sigmoid_exact(float x) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
 
 struct StateRef {                            // where sequences keep their state
   const int* slots; int num_slots;           // per sequence; < 0: padding
@@ -274,7 +277,7 @@ __global__ void __launch_bounds__(kScanThreads) space_scan_kernel(const SpacePar
     if (threadIdx.x < m) {
       const float dt = softplus_f(to_f(p.dt[static_cast<long long>(q0 + t0 + threadIdx.x) * p.ld_dt + h]) + dtb);
       dts[threadIdx.x] = dt;
-      as[threadIdx.x] = __expf(-A * dt);
+      as[threadIdx.x] = decay_f(A * dt);
     }
     __syncthreads();
 #pragma unroll 2
@@ -342,7 +345,7 @@ __global__ void space_step_kernel(const SpaceParams<T> p) {
 #pragma unroll
     for (int e = 0; e < 8; ++e) dst[e] = f[e];
   }
-  const float dt = softplus_f(to_f(p.dt[static_cast<long long>(s) * p.ld_dt + h]) + p.dt_bias[h]), a = __expf(-p.A[h] * dt);
+  const float dt = softplus_f(to_f(p.dt[static_cast<long long>(s) * p.ld_dt + h]) + p.dt_bias[h]), a = decay_f(p.A[h] * dt);
   __syncthreads();
   F2 B[J][2], C[J][2];
   load_keys<J>(Bs, lane, B);
@@ -409,7 +412,7 @@ __device__ __forceinline__ void delta_operands(int K, float A, const float* deca
     float z = 0.f, b = 0.f;
     q[e] = k[e] = 0.f;
     if (i < K) { load(i, q[e], k[e], z); b = decay_bias[i]; }
-    gs[i] = __expf(-A * softplus_f(z + b));
+    gs[i] = decay_f(A * softplus_f(z + b));
     qq = fmaf(q[e], q[e], qq);
     kk = fmaf(k[e], k[e], kk);
     dot = fmaf(q[e], k[e], dot);
@@ -420,7 +423,7 @@ __device__ __forceinline__ void delta_operands(int K, float A, const float* deca
     kk += __shfl_xor_sync(0xffffffffu, kk, o);
     dot += __shfl_xor_sync(0xffffffffu, dot, o);
   }
-  const float fq = q_scale * rsqrtf(qq + kUnitEps), fk = rsqrtf(kk + kUnitEps);
+  const float fq = q_scale / sqrtf(qq + kUnitEps), fk = 1.f / sqrtf(kk + kUnitEps);
 #pragma unroll
   for (int e = 0; e < E; ++e) { qs[lane + e * 32] = q[e] * fq; ks[lane + e * 32] = k[e] * fk; }
   if (lane == 0) *qk = dot * fq * fk;
@@ -482,7 +485,7 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
 #pragma unroll
       for (int e = 0; e < 8; ++e) vs[t][k + e] = f[e];
     }
-    if (threadIdx.x < m) bs[threadIdx.x] = sigmoid_f(to_f(p.beta[static_cast<long long>(q0 + t0 + threadIdx.x) * p.ld_beta + h]));
+    if (threadIdx.x < m) bs[threadIdx.x] = sigmoid_exact(to_f(p.beta[static_cast<long long>(q0 + t0 + threadIdx.x) * p.ld_beta + h]));
     __syncthreads();
     for (int t = 0; t < m; ++t) {
       F2 q[J][2], k[J][2], d[J][2];
@@ -547,7 +550,7 @@ __global__ void delta_step_kernel(const DeltaParams<T> p) {
 #pragma unroll
     for (int e = 0; e < 8; ++e) dst[e] = f[e];
   }
-  const float beta = sigmoid_f(to_f(p.beta[static_cast<long long>(s) * p.ld_beta + h]));
+  const float beta = sigmoid_exact(to_f(p.beta[static_cast<long long>(s) * p.ld_beta + h]));
   __syncthreads();
   if (threadIdx.x < 32) {
     const T* z = p.decay + static_cast<long long>(s) * p.ld_decay + h * p.K;

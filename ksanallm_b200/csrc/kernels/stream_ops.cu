@@ -14,6 +14,8 @@
 
 namespace ksana {
 
+__device__ __forceinline__ float sigmoid_exact(float x) { return 1.f / (1.f + expf(-x)); }
+
 // Sum over the CTA, in every thread. `red`: 32 floats of shared memory
 __device__ __forceinline__ float cta_sum(float v, float* red) {
 #pragma unroll
@@ -55,7 +57,7 @@ __global__ void embed_normed_kernel(const int* __restrict__ ids, const int* __re
       }
     }
   }
-  const float rstd = rsqrtf(cta_sum(s, red) / static_cast<float>(real) + eps);
+  const float rstd = 1.f / sqrtf(cta_sum(s, red) / static_cast<float>(real) + eps);
 #pragma unroll
   for (int j = 0; j < VPT; ++j) {
     const int i = threadIdx.x + j * blockDim.x;
@@ -139,7 +141,7 @@ __global__ void gated_norm_kernel(const GatedNormParams<T> p) {
         float f[8];
         load8(p.z + static_cast<long long>(m) * p.ldz + i * 8, f);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[j][e] *= f[e] * sigmoid_f(f[e]);
+        for (int e = 0; e < 8; ++e) v[j][e] *= f[e] * sigmoid_exact(f[e]);
       }
       if (whole) {
         float s = 0.f;
@@ -162,7 +164,7 @@ __global__ void gated_norm_kernel(const GatedNormParams<T> p) {
     for (int k = lane; k < per; k += 32) s += sums[q * per + k];
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-    if (lane == 0) rstd[q] = rsqrtf(s / static_cast<float>(size) + p.eps) * p.factor;
+    if (lane == 0) rstd[q] = 1.f / sqrtf(s / static_cast<float>(size) + p.eps) * p.factor;
   }
   __syncthreads();
 #pragma unroll
@@ -186,7 +188,7 @@ __global__ void gated_norm_kernel(const GatedNormParams<T> p) {
         float f[8];
         load8(p.g + static_cast<long long>(m) * p.ldg + i * 8, f);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[j][e] *= sigmoid_f(f[e]);
+        for (int e = 0; e < 8; ++e) v[j][e] *= sigmoid_exact(f[e]);
       }
       store8(p.out + static_cast<long long>(m) * p.ldo + i * 8, v[j]);
     }
@@ -214,15 +216,13 @@ __global__ void panel_append_kernel(const T* __restrict__ k, long long ldk, cons
   }
 }
 
-// tanh from one exponential; its error is absolute (the result is multiplied by the cap)
 __global__ void softcap_kernel(float* __restrict__ z, long long ld, int M, int N, float cap) {
   pdl_trigger();
   pdl_wait();
-  const float f = 2.f / cap;
   for (int m = blockIdx.y; m < M; m += gridDim.y)
     for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < N; i += gridDim.x * blockDim.x) {
       float* at = z + m * ld + i;
-      *at = cap * (1.f - 2.f / (1.f + __expf(*at * f)));
+      *at = cap * tanhf(*at / cap);
     }
 }
 

@@ -63,6 +63,7 @@ class ParallelLayer:
 
 class FapudraModel(StreamModel):
     needs_state_slots = True
+    moves_blocks = False
 
     def __init__(self, cfg: ModelConfig, *a, **kw):
         super().__init__(cfg, *a, **kw)

@@ -167,11 +167,14 @@ def experts(h, m, w, pre):
 
 
 # ------------------------------------------------------------------------------------------------ model
-def forward(tokens, cfg, w, streams=None):
-    """Logits [T, vocab] of one sequence. ``streams`` (a list) receives the residual stream after every layer."""
+def forward(tokens, cfg, w, streams=None, splice=None):
+    """Logits [T, vocab] of one sequence. ``streams`` (a list) receives the residual stream after every layer; ``splice`` {row:
+    vector} replaces rows of the first stream."""
     eps = cfg["norm"]["eps"]
     x = w["embed"][torch.tensor(tokens)] * cfg["embedding"]["scale"] + w["pos"][:len(tokens)]
     x = rms(x, eps) * w["embed.norm"]
+    for row, vector in (splice or {}).items():
+        x[row] = vector
     for i, e in enumerate(cfg["layers"]):
         p = f"l{i}."
         h = rms(x, eps) * w[p + "norm1"]
