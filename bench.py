@@ -187,7 +187,7 @@ def main():
     ap.add_argument("--breakdown", action="store_true",
                     help="instead of the benchmark: device time of one decode step and one prefill step of this model by "
                          "kernel class (benchmarks/step_breakdown.py; --layers limits the depth, --comm picks the path)")
-    ap.add_argument("--design", default=None, choices=["lenolix", "rasizen", "fidevik"],
+    ap.add_argument("--design", default=None, choices=["lenolix", "rasizen", "fidevik", "fapudra"],
                     help="instead of the benchmark: prefill and decode throughput of this model family beside the "
                          "closest other model at equal sizes, kernel by kernel (benchmarks/<design>_bench.py)")
     ap.add_argument("--sizes", default="1b,3b,8b", help="--design: sizes to run")

@@ -102,7 +102,7 @@ def run(args, design, sizes, describe, variants, cost, base, mine, timed_only=()
                     res["kernels"] = rows
                     tables[(variant, phase)] = rows
                 out["results"].setdefault(phase, {})[variant] = res
-                model.kv_cache = None
+                model.kv_cache = model.state = None
             del model
             torch.cuda.empty_cache()
         out["clocks"] = sampler.stop()

@@ -88,6 +88,10 @@ def build_step(torch, model, phase, batch, ctx, q_len, block_tokens):
     step.max_kv_len = kv
     if model.needs_prev_ids:
         step.prev_ids = torch.roll(ids, 1)
+    if model.needs_state_slots:
+        step.state_slots = torch.arange(batch, dtype=torch.int32, device=dev)
+        if model.state is None or model.state.shape[0] < batch:
+            model.allocate_state(batch)
     if phase == "decode":
         step.decode_splits = ops.decode_splits(batch, model.Hkv, kv)
     return step, batch * bps

@@ -606,8 +606,9 @@ static ConvRef<T> conv_ref(const void* x, long long ld, const void* w, const voi
   return {static_cast<const T*>(x), ld, static_cast<const T*>(w), static_cast<const T*>(bias), static_cast<T*>(ring), ring_stride, taps, C};
 }
 
-static bool bad_conv(const void* x, long long ld, const void* w, const void* bias, const void* ring, long long ring_stride, int taps, int C) {
-  return taps < 1 || taps > kMaxTaps || C <= 0 || C % 8 || ld % 8 || ring_stride % 8 || !aligned16(x) || !aligned16(w) ||
+static bool bad_conv(const void* x, long long ld, const void* w, const void* bias, const void* ring, long long ring_stride, int taps, int C,
+                     int f32) {
+  return taps < 1 || taps > kMaxTaps || C <= 0 || C % 8 || ld % 8 || ring_stride % (f32 ? 4 : 8) || !aligned16(x) || !aligned16(w) ||
          !aligned16(bias) || !aligned16(ring);
 }
 
@@ -621,7 +622,7 @@ extern "C" int ksana_causal_conv(const void* x, long long ld, const void* w, con
                                  int C, void* out, long long ldo, const int* cu_q, const int* kv_lens, const int* slots, int num_slots,
                                  int B, int max_q, int f32, int* err, cudaStream_t st) {
   if (B <= 0 || max_q <= 0) return 0;
-  if (bad_conv(x, ld, w, bias, ring, ring_stride, taps, C) || ldo % 8 || !aligned16(out) || B > 65535 || !cu_q) return -10;
+  if (bad_conv(x, ld, w, bias, ring, ring_stride, taps, C, f32) || ldo % 8 || !aligned16(out) || B > 65535 || !cu_q) return -10;
   const StateRef r{slots, num_slots, kv_lens, err};
   return f32 ? launch_conv<float>(conv_ref<float>(x, ld, w, bias, ring, ring_stride, taps, C), r, static_cast<float*>(out), ldo, cu_q, B, max_q, st)
              : launch_conv<bf16>(conv_ref<bf16>(x, ld, w, bias, ring, ring_stride, taps, C), r, static_cast<bf16*>(out), ldo, cu_q, B, max_q, st);
@@ -636,7 +637,7 @@ extern "C" int ksana_state_space(const void* x, long long ld, const void* w, con
   if (B <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || P <= 0 || N <= 0 || P % 8 || N % 8 || H > 65535 || B > 65535 || slot_stride % 4 || ldy % 8 || !aligned16(y) ||
       !aligned16(state) || (cu_q && (!c || ldc % 8 || !aligned16(c))) ||
-      bad_conv(x, ld, w, bias, ring, ring_stride, taps, H * P + 2 * G * N))
+      bad_conv(x, ld, w, bias, ring, ring_stride, taps, H * P + 2 * G * N, f32))
     return -10;
   auto run = [&](auto tag) {
     typedef decltype(tag) T;
@@ -666,7 +667,7 @@ extern "C" int ksana_delta_rule(const void* x, long long ld, const void* w, void
   if (B <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || K <= 0 || V <= 0 || K % 8 || V % 8 || H > 65535 || B > 65535 || slot_stride % 4 || ldo % 8 || !aligned16(o) ||
       !aligned16(state) || (cu_q && (!c || ldc % 8 || !aligned16(c))) ||
-      bad_conv(x, ld, w, nullptr, ring, ring_stride, taps, 2 * G * K + H * V))
+      bad_conv(x, ld, w, nullptr, ring, ring_stride, taps, 2 * G * K + H * V, f32))
     return -10;
   auto run = [&](auto tag) {
     typedef decltype(tag) T;

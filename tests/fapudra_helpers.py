@@ -43,8 +43,10 @@ CONFIGS = {
     # sizes of the fast paths, more experts than a warp has lanes
     "long": config(128, 320, [(space(8, 64, 128, 2, 4, 8), moe(64, 6, (8, 3), 40)), (both((8, 2, 64), (64, 20), (4, 2, 64, 64, 4), bias_max=100), moe(40, 8, (40, 12), 24)),
                               (both((6, 3, 128), (100, 7), (2, 1, 128, 128, 3)), None)]),
-    # degenerate values: one head, one column, one tap, one expert, one bucket per distance
-    "ones": config(64, 90, [(space(1, 1, 1, 1, 1, 1), moe(1, 1, (1, 1), 1)), (both((1, 1, 1), (1, 1), (1, 1, 1, 1, 1), (1.0, 1.0), 9, 1.0), moe(2, 1, (2, 1), 8))]),
+    # degenerate values: one head, one column, one tap, one expert, one bucket per distance (a large eps: norms of single columns
+    # would be signs)
+    "ones": config(64, 90, [(space(1, 1, 1, 1, 1, 1), moe(1, 1, (1, 1), 1)), (both((1, 1, 1), (1, 1), (1, 1, 2, 1, 1), (1.0, 1.0), 9, 1.0), moe(2, 1, (2, 1), 8))],
+                   eps=0.1),
     # heads beyond the tensor-core prefill kernel, many heads per key/value head, long keys, many taps
     "wide": config(96, 150, [(both((2, 1, 136), (40, 9), (2, 1, 136, 40, 6)), None), (space(2, 72, 136, 2, 6, 4), None),
                              (both((40, 2, 8), (21, 4), (2, 2, 40, 136, 1), bias_max=700), None)]),
