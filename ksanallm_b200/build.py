@@ -24,7 +24,7 @@ NVCC_FLAGS = [
     "--use_fast_math", "-Xcompiler", "-fPIC", "-Xcompiler", "-Wno-unused-function",
 ]
 # sources whose exponentials, divisions and roots feed long recurrences: no approximations that they do not ask for by name
-PRECISE = {"state_scan", "stream_ops"}
+PRECISE = {"state_chunk", "state_scan", "stream_ops"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread", "-Wall", "-Wno-sign-compare"]
 
 
@@ -61,7 +61,7 @@ def engine_lib_path() -> Path:
 
 # kernel sources that a family needs in bf16 or fp32 on one GPU (no FP8 / FP4 / 4-bit weights or peer memory)
 _STREAM_KERNELS = ("attention_f32", "elementwise", "gemm_f32", "gemm_smallm", "gemm_tcgen05", "residual_stream", "sampler")
-FAMILY_KERNELS = {"fapudra": _STREAM_KERNELS + ("attention", "attention_tc", "moe", "state_scan", "stream_ops"),
+FAMILY_KERNELS = {"fapudra": _STREAM_KERNELS + ("attention", "attention_tc", "moe", "state_chunk", "state_scan", "stream_ops"),
                   "fidevik": _STREAM_KERNELS + ("attention", "attention_tc", "mla_attention", "moe"),
                   "lenolix": _STREAM_KERNELS + ("attention", "attention_tc"),
                   "rasizen": _STREAM_KERNELS + ("mla_attention", "recurrence")}

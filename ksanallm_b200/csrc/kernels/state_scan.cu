@@ -13,15 +13,12 @@
 //                   q (times dim^-1/2) and k per head, a decay g = exp(-A softplus(projection + bias)) per head and key channel
 //                   and beta = sigmoid(projection)
 //
-// Both recurrences have a scan (several tokens per sequence, convolved inputs) and a step (one token per sequence, the
-// convolution is part of it). Every column of a state is independent of the others: a CTA takes a slab of columns of one
+// Both recurrences have a scan (several tokens per sequence, convolved inputs; in bf16 the tensor-core form of state_chunk.cu
+// takes most sizes) and a step (one token per sequence, the convolution is part of it). Every column of a state is independent of the others: a CTA takes a slab of columns of one
 // head, eight neighbouring lanes share a column and split its keys. Head and key sizes are multiples of 8 (padded with
 // zeros). At position 0 the state is zero whatever the slot holds.
 #include "f32x2.cuh"
-#include "guards.cuh"
-#include "pdl.cuh"
-#include "vec8.cuh"
-#include <cuda_runtime.h>
+#include "state_scan.cuh"
 
 namespace ksana {
 
@@ -30,35 +27,6 @@ constexpr int kChunk = 16;                   // tokens staged at a time
 constexpr int kCols = 2;                     // columns per thread in scans
 constexpr int kScanThreads = 128;
 constexpr int kSlab = kScanThreads / kLanes * kCols;
-constexpr int kMaxTaps = 16;
-constexpr float kUnitEps = 1e-6f;
-
-__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
-// exp(-x), x >= 0, rounded to nearest near 1: a decay is applied once per token, a bias of its last bit would add up
-__device__ __forceinline__ float decay_f(float x) { return 1.f + expm1f(-x); }
-__device__ __forceinline__ float sigmoid_exact(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
-
-struct StateRef {                            // where sequences keep their state
-  const int* slots; int num_slots;           // per sequence; < 0: padding
-  const int* kv_lens;
-  int* err;
-};
-// The slot of sequence s, or -1 where it has none (padding, or an id outside the pool, which is recorded).
-__device__ __forceinline__ int slot_of(const StateRef& r, int s) {
-  const int slot = r.slots[s];
-  if (slot >= r.num_slots) { if (threadIdx.x == 0) guard_report(r.err, kGuardSlot, slot); return -1; }
-  return slot;
-}
-
-template <typename T>
-struct ConvRef {                             // a short convolution's inputs, weights and ring
-  const T* x; long long ld;                  // raw projection rows, first channel
-  const T* w; const T* bias;                 // [taps][C] (the last tap is the current token's), [C] or null
-  T* ring; long long slot_stride;            // ring of slot 0, elements between slots
-  int taps, C;
-};
-
 // silu(conv) of 8 channels of a single new token at position pos
 template <typename T>
 __device__ __forceinline__ void conv_one(const ConvRef<T>& v, const T* row, const T* ring, int pos, int c, float (&acc)[8]) {
@@ -76,18 +44,6 @@ __device__ __forceinline__ void conv_one(const ConvRef<T>& v, const T* row, cons
   }
 #pragma unroll
   for (int e = 0; e < 8; ++e) acc[e] = silu_f(acc[e]);
-}
-
-// Channels [c0, c0 + n) of the last inputs of a sequence's new tokens go to the ring.
-template <typename T>
-__device__ __forceinline__ void ring_store(const ConvRef<T>& v, const T* rows, T* ring, int past, int n, int c0, int count) {
-  const int vecs = count >> 3, keep = min(v.taps, n);
-  for (int i = threadIdx.x; i < vecs * keep; i += blockDim.x) {
-    const int t = n - 1 - i / vecs, c = c0 + (i % vecs) * 8;
-    float f[8];
-    load8(rows + static_cast<long long>(t) * v.ld + c, f);
-    store8(ring + static_cast<size_t>((past + t) % v.taps) * v.C + c, f);
-  }
 }
 
 // ------------------------------------------------------------------------------------------------ convolution
@@ -192,19 +148,6 @@ __device__ __forceinline__ float lanes_sum(float v) {
 }
 
 // ------------------------------------------------------------------------------------------------ state space
-template <typename T>
-struct SpaceParams {
-  ConvRef<T> conv;                           // channels: x [H][P] | B [G][N] | C [G][N]
-  const T* c; long long ldc;                 // convolved rows (scan)
-  const T* dt; long long ld_dt;              // raw step sizes, [rows][H]
-  const float* dt_bias; const float* A; const float* D;      // [H]
-  T* y; long long ldy;                       // [rows][H * P]
-  float* state; long long slot_stride;       // matrix state of slot 0 of the layer, floats between slots
-  StateRef ref;
-  const int* cu_q;
-  int H, G, P, N;
-};
-
 // One token for one column: decay, write, read-out (summed over this thread's keys)
 template <int J>
 __device__ __forceinline__ float space_token(F2 (&S)[J][2], const F2 (&B)[J][2], const F2 (&C)[J][2], F2 a, F2 dx) {
@@ -218,19 +161,6 @@ __device__ __forceinline__ float space_token(F2 (&S)[J][2], const F2 (&B)[J][2],
     }
   }
   return sum2(acc);
-}
-
-// Channels of the ring that the CTA of (head, slab of columns [p0, p0 + np)) stores: its own x, and B and C of the head's group
-// where it is the group's first.
-template <typename T>
-__device__ __forceinline__ void space_ring(const SpaceParams<T>& p, const T* rows, int slot, int past, int n, int h, int p0, int np) {
-  T* ring = p.conv.ring + static_cast<long long>(slot) * p.conv.slot_stride;
-  ring_store(p.conv, rows, ring, past, n, h * p.P + p0, np);
-  const int per = p.H / p.G, g = h / per;
-  if (h % per == 0 && p0 == 0) {
-    ring_store(p.conv, rows, ring, past, n, p.H * p.P + g * p.N, p.N);
-    ring_store(p.conv, rows, ring, past, n, p.H * p.P + (p.G + g) * p.N, p.N);
-  }
 }
 
 // grid (slabs, H, sequences)
@@ -308,7 +238,7 @@ __global__ void __launch_bounds__(kScanThreads) space_scan_kernel(const SpacePar
     const int col = tg + c * (kSlab / kCols);
     if (col < np) store_column<J>(state + static_cast<long long>(p0 + col) * p.N, p.N, lane, S[c]);
   }
-  space_ring(p, p.conv.x + static_cast<long long>(q0) * p.conv.ld, slot, past, n, h, p0, np);
+  space_ring(p, p.conv.x + static_cast<long long>(q0) * p.conv.ld, slot, past, n, h, p0, np, threadIdx.x, blockDim.x);
 }
 
 // One token per sequence: grid (slabs, H, sequences), blockDim = 8 lanes x columns of the slab (a multiple of 8).
@@ -356,25 +286,10 @@ __global__ void space_step_kernel(const SpaceParams<T> p) {
     store_column<J>(state, p.N, lane, S);
     if (lane == 0) y[col] = from_f<T>(fmaf(p.D[h], x, v));
   }
-  space_ring(p, row, slot, pos, 1, h, p0, np);
+  space_ring(p, row, slot, pos, 1, h, p0, np, threadIdx.x, blockDim.x);
 }
 
 // ------------------------------------------------------------------------------------------------ delta rule
-template <typename T>
-struct DeltaParams {
-  ConvRef<T> conv;                           // channels: q [G][K] | k [G][K] | v [H][V]
-  const T* c; long long ldc;                 // convolved rows (scan)
-  const T* beta; long long ld_beta;          // raw, [rows][H]
-  const T* decay; long long ld_decay;        // raw, [rows][H * K]
-  const float* decay_bias; const float* A;   // [H * K], [H]
-  T* o; long long ldo;                       // [rows][H * V]
-  float* state; long long slot_stride;
-  StateRef ref;
-  const int* cu_q;
-  int H, G, K, V;
-  float q_scale;
-};
-
 // One token for one column. qk = q . k
 template <int J>
 __device__ __forceinline__ float delta_token(F2 (&S)[J][2], const F2 (&q)[J][2], const F2 (&k)[J][2], const F2 (&g)[J][2], float qk,
@@ -427,17 +342,6 @@ __device__ __forceinline__ void delta_operands(int K, float A, const float* deca
 #pragma unroll
   for (int e = 0; e < E; ++e) { qs[lane + e * 32] = q[e] * fq; ks[lane + e * 32] = k[e] * fk; }
   if (lane == 0) *qk = dot * fq * fk;
-}
-
-template <typename T>
-__device__ __forceinline__ void delta_ring(const DeltaParams<T>& p, const T* rows, int slot, int past, int n, int h, int p0, int np) {
-  T* ring = p.conv.ring + static_cast<long long>(slot) * p.conv.slot_stride;
-  ring_store(p.conv, rows, ring, past, n, 2 * p.G * p.K + h * p.V + p0, np);
-  const int per = p.H / p.G, g = h / per;
-  if (h % per == 0 && p0 == 0) {
-    ring_store(p.conv, rows, ring, past, n, g * p.K, p.K);
-    ring_store(p.conv, rows, ring, past, n, (p.G + g) * p.K, p.K);
-  }
 }
 
 // grid (slabs, H, sequences)
@@ -513,7 +417,7 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
     const int col = tg + c * (kSlab / kCols);
     if (col < np) store_column<J>(state + static_cast<long long>(p0 + col) * p.K, p.K, lane, S[c]);
   }
-  delta_ring(p, p.conv.x + static_cast<long long>(q0) * p.conv.ld, slot, past, n, h, p0, np);
+  delta_ring(p, p.conv.x + static_cast<long long>(q0) * p.conv.ld, slot, past, n, h, p0, np, threadIdx.x, blockDim.x);
 }
 
 // One token per sequence: grid (slabs, H, sequences), blockDim = 8 lanes x columns of the slab (a multiple of 8).
@@ -567,7 +471,7 @@ __global__ void delta_step_kernel(const DeltaParams<T> p) {
     store_column<J>(state, p.K, lane, S);
     if (lane == 0) o[col] = from_f<T>(v);
   }
-  delta_ring(p, row, slot, pos, 1, h, p0, np);
+  delta_ring(p, row, slot, pos, 1, h, p0, np, threadIdx.x, blockDim.x);
 }
 
 // ------------------------------------------------------------------------------------------------ host
@@ -590,12 +494,20 @@ static int launch_conv(const ConvRef<T>& v, const StateRef& r, T* out, long long
 
 template <typename T, int J>
 static int launch_space(const SpaceParams<T>& p, int B, cudaStream_t st) {
+  if constexpr (sizeof(T) == 2) {
+    const int rc = p.cu_q ? space_chunks(p, B, st) : -100;
+    if (rc != -100) return rc;
+  }
   if (p.cu_q) return launched(launch_pdl(space_scan_kernel<T, J>, dim3((p.P + kSlab - 1) / kSlab, p.H, B), dim3(kScanThreads), 0, st, p));
   const int threads = step_threads(p.P), slab = threads / kLanes;
   return launched(launch_pdl(space_step_kernel<T, J>, dim3((p.P + slab - 1) / slab, p.H, B), dim3(threads), 0, st, p));
 }
 template <typename T, int J>
 static int launch_delta(const DeltaParams<T>& p, int B, cudaStream_t st) {
+  if constexpr (sizeof(T) == 2) {
+    const int rc = p.cu_q ? delta_chunks(p, B, st) : -100;
+    if (rc != -100) return rc;
+  }
   if (p.cu_q) return launched(launch_pdl(delta_scan_kernel<T, J>, dim3((p.V + kSlab - 1) / kSlab, p.H, B), dim3(kScanThreads), 0, st, p));
   const int threads = step_threads(p.V), slab = threads / kLanes;
   return launched(launch_pdl(delta_step_kernel<T, J>, dim3((p.V + slab - 1) / slab, p.H, B), dim3(threads), 0, st, p));
