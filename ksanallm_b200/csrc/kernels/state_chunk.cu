@@ -9,12 +9,12 @@
 // A warp owns 16 columns: its part of S stays in registers in the accumulator layout of the update (rows: columns of the state,
 // columns: keys), which is the operand layout of C S. The weights M are computed by rows, 16 per warp, and shared.
 //
-// delta_chunk_kernel: one CTA per (sequence, head, 64 columns), chunks of 16 tokens. With P_t = g_1 .. g_t per key channel:
+// delta_chunk_kernel: one CTA per (sequence, head, 64 or 128 columns), chunks of 16 tokens. With P_t = g_1 .. g_t per key channel:
 //   (I + A) U = beta (V - (k P) S),  A_ts = beta_t sum_c k_tc k_sc (g_(s+1) .. g_t)_c for s < t
 //   O = (q P) S + Q U,  Q_ts likewise with q_t, for s <= t;   S <- P_L S + sum_s (k_s g_(s+1) .. g_L) u_s^T
-// Decays enter as products of factors <= 1 only, never as quotients, so no decay is too strong. Four warps prepare the operands of
-// the next chunk (unit vectors, decays, A and its unit-triangular inverse, Q), four warps with 16 columns each apply them; U and the
-// state never leave their registers.
+// Decays enter as products of factors <= 1 only, never as quotients, so no decay is too strong. Three groups of four warps prepare the
+// operands of the chunks in turn (unit vectors, decays, A and the inverse of I + A, Q) in a ring of four buffers; four warps apply
+// them, each to 16 or 32 columns, whose state never leaves their registers.
 #include "state_scan.cuh"
 
 namespace ksana {
@@ -54,7 +54,7 @@ constexpr int kSpaceTokens = 64, kSpaceCols = 64, kSpaceThreads = 128;
 constexpr int kXPitch = (kSpaceCols + 8) * 2;            // bytes between rows of X and M: ldmatrix rows fall into different banks
 template <int NK> constexpr int kBPitch = (NK * 16 + 8) * 2;
 template <int NK> constexpr int kSpaceStage = kSpaceTokens * (2 * kBPitch<NK> + kXPitch);
-template <int NK> constexpr int kSpaceSmem = 2 * kSpaceStage<NK> + 2 * kSpaceTokens * kXPitch + 4 * kSpaceTokens * 4;
+template <int NK> constexpr int kSpaceSmem = 2 * kSpaceStage<NK> + 2 * kSpaceTokens * kXPitch + 8 * kSpaceTokens * 4;
 
 // NK: steps of 16 keys. grid (column slabs, H, sequences)
 template <int NK>
@@ -65,10 +65,7 @@ __global__ void __launch_bounds__(kSpaceThreads, 2) space_chunk_kernel(const Spa
   constexpr int PB = kBPitch<NK>, L = kSpaceTokens;
   uint8_t* mh = smem + 2 * kSpaceStage<NK>;
   uint8_t* ml = mh + L * kXPitch;
-  float* cum = reinterpret_cast<float*>(ml + L * kXPitch);      // G_t
-  float* dts = cum + L;
-  float* wend = dts + L;                                        // dt_s exp(G_L - G_s)
-  float* edec = wend + L;                                       // exp(G_t)
+  float* scalars = reinterpret_cast<float*>(ml + L * kXPitch);  // per stage: G_t, dt_t, dt_s exp(G_L - G_s), exp(G_t)
   const int s = blockIdx.z, h = blockIdx.y, p0 = blockIdx.x * kSpaceCols, np = min(kSpaceCols, p.P - p0);
   const int q0 = p.cu_q[s], n = p.cu_q[s + 1] - q0, past = p.ref.kv_lens[s] - n;
   if (n <= 0) return;
@@ -95,45 +92,66 @@ __global__ void __launch_bounds__(kSpaceThreads, 2) space_chunk_kernel(const Spa
   }
   auto stage = [&](int buf) { return smem + buf * kSpaceStage<NK>; };
   auto issue = [&](int t0, int buf) {
-    uint8_t* b = stage(buf);
-    constexpr int V = NK * 2, W = 2 * V + kSpaceCols / 8;       // 16-byte pieces of a row
-    for (int i = threadIdx.x; i < L * W; i += kSpaceThreads) {
-      const int t = i / W, k = i % W;
-      const bool is_x = k >= 2 * V, is_c = !is_x && k >= V;
-      const int v = is_x ? k - 2 * V : is_c ? k - V : k;
-      const bool there = t0 + t < n && (is_x ? v * 8 < np : v * 8 < p.N);
-      uint8_t* dst = is_x ? b + 2 * L * PB + t * kXPitch : b + (is_c ? L * PB : 0) + t * PB;
-      const bf16* src = rows + static_cast<long long>(there ? t0 + t : 0) * p.ldc + (there ? (is_x ? xoff : is_c ? coff : boff) + v * 8 : 0);
-      sc_copy16(sc_addr(dst + v * 16), src, there);
+    // a thread has one 16-byte piece of every STEP-th row of B and C, and one of every 16th row of X
+    constexpr int V = NK * 2, STEP = kSpaceThreads / V, XV = kSpaceCols / 8, XSTEP = kSpaceThreads / XV;
+    const uint32_t b = sc_addr(stage(buf));
+    {
+      const int v = threadIdx.x % V, t = threadIdx.x / V;
+      const bool in = v * 8 < p.N;
+      const bf16* src = rows + static_cast<long long>(t0 + t) * p.ldc + (in ? v * 8 : 0);
+      const uint32_t dst = b + t * PB + v * 16;
+#pragma unroll
+      for (int i = 0; i < (L + STEP - 1) / STEP; ++i) {
+        const bool there = in && t0 + t + i * STEP < n;
+        const bf16* at = there ? src + i * STEP * p.ldc : rows;
+        if (L % STEP == 0 || t + i * STEP < L) {
+          sc_copy16(dst + i * STEP * PB, at + (there ? boff : 0), there);
+          sc_copy16(dst + L * PB + i * STEP * PB, at + (there ? coff : 0), there);
+        }
+      }
+    }
+    {
+      const int v = threadIdx.x % XV, t = threadIdx.x / XV;
+      const bool in = v * 8 < np;
+      const bf16* src = rows + static_cast<long long>(t0 + t) * p.ldc + xoff + (in ? v * 8 : 0);
+      const uint32_t dst = b + 2 * L * PB + t * kXPitch + v * 16;
+#pragma unroll
+      for (int i = 0; i < L / XSTEP; ++i) {
+        const bool there = in && t0 + t + i * XSTEP < n;
+        sc_copy16(dst + i * XSTEP * kXPitch, there ? src + i * XSTEP * p.ldc : rows, there);
+      }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   auto raw_dt = [&](int t) { return t < n ? to_f(p.dt[static_cast<long long>(q0 + t) * p.ld_dt + h]) : 0.f; };
+  float d0 = 0.f, d1 = 0.f;
+  // step sizes of the chunk at t0 (raw ones in d0, d1), their running sums, decays; then the raw ones of the chunk behind it
+  auto decays = [&](int t0, float* out) {
+    const float a = t0 + 2 * lane < n ? softplus_f(d0 + dtb) : 0.f, b = t0 + 2 * lane + 1 < n ? softplus_f(d1 + dtb) : 0.f;
+    float sum = a + b;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float up = __shfl_up_sync(0xffffffffu, sum, o);
+      if (lane >= o) sum += up;
+    }
+    const float total = __shfl_sync(0xffffffffu, sum, 31), g1 = -A * sum, g0 = -A * (sum - b), gl = -A * total;
+    *reinterpret_cast<float2*>(out + 2 * lane) = make_float2(g0, g1);
+    *reinterpret_cast<float2*>(out + L + 2 * lane) = make_float2(a, b);
+    *reinterpret_cast<float2*>(out + 2 * L + 2 * lane) = make_float2(a * expf(gl - g0), b * expf(gl - g1));
+    *reinterpret_cast<float2*>(out + 3 * L + 2 * lane) = make_float2(expf(g0), expf(g1));
+    d0 = raw_dt(t0 + L + 2 * lane);
+    d1 = raw_dt(t0 + L + 2 * lane + 1);
+  };
   issue(0, 0);
-  float d0 = warp == 0 ? raw_dt(2 * lane) : 0.f, d1 = warp == 0 ? raw_dt(2 * lane + 1) : 0.f;
+  if (warp == 0) {
+    d0 = raw_dt(2 * lane);
+    d1 = raw_dt(2 * lane + 1);
+    decays(0, scalars);
+  }
   for (int t0 = 0, buf = 0; t0 < n; t0 += L, buf ^= 1) {
     if (t0 + L < n) issue(t0 + L, buf ^ 1);
     else asm volatile("cp.async.commit_group;" ::: "memory");
-    if (warp == 0) {                                     // step sizes, their running sums, decays
-      const float a = t0 + 2 * lane < n ? softplus_f(d0 + dtb) : 0.f, b = t0 + 2 * lane + 1 < n ? softplus_f(d1 + dtb) : 0.f;
-      float sum = a + b;
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float up = __shfl_up_sync(0xffffffffu, sum, o);
-        if (lane >= o) sum += up;
-      }
-      const float total = __shfl_sync(0xffffffffu, sum, 31), g1 = -A * sum, g0 = -A * (sum - b), gl = -A * total;
-      cum[2 * lane] = g0;
-      cum[2 * lane + 1] = g1;
-      dts[2 * lane] = a;
-      dts[2 * lane + 1] = b;
-      edec[2 * lane] = expf(g0);
-      edec[2 * lane + 1] = expf(g1);
-      wend[2 * lane] = a * expf(gl - g0);
-      wend[2 * lane + 1] = b * expf(gl - g1);
-      d0 = raw_dt(t0 + L + 2 * lane);
-      d1 = raw_dt(t0 + L + 2 * lane + 1);
-    }
+    const float *cum = scalars + buf * 4 * L, *dts = cum + L, *wend = dts + L, *edec = wend + L;
     asm volatile("cp.async.wait_group 1;" ::: "memory");
     __syncthreads();
     const uint32_t bs = sc_addr(stage(buf)), cs = bs + L * PB, xs = bs + 2 * L * PB;
@@ -176,6 +194,7 @@ __global__ void __launch_bounds__(kSpaceThreads, 2) space_chunk_kernel(const Spa
         }
       }
     }
+    if (warp == 0 && t0 + L < n) decays(t0 + L, scalars + (buf ^ 1) * 4 * L);      // this warp had the fewest weights
     // the state as an operand
     uint32_t sh[2 * NK][2], sl[2 * NK][2];
 #pragma unroll
@@ -287,24 +306,35 @@ int space_chunks(const SpaceParams<bf16>& p, int B, cudaStream_t st) {
 }
 
 // ------------------------------------------------------------------------------------------------ delta rule
-constexpr int kDeltaTokens = 16, kDeltaCols = 64, kDeltaThreads = 256, kMPitch = (kDeltaTokens + 8) * 2;
-template <int NK> struct DeltaSmem {
-  static constexpr int KP = NK * 16, pitch = (KP + 8) * 2, rows = kDeltaTokens * pitch, fpitch = KP + 4;
+constexpr int kDeltaTokens = 16, kDeltaGroups = 3, kDeltaBuffers = 4, kDeltaThreads = 128 * (1 + kDeltaGroups);
+constexpr int kMPitch = (kDeltaTokens + 8) * 2;
+// NK: steps of 16 keys, CT: 16-column tiles per warp that applies
+template <int NK, int CT> struct DeltaSmem {
+  static constexpr int KP = NK * 16, cols = 64 * CT, pitch = (KP + 8) * 2, rows = kDeltaTokens * pitch, vpitch = (cols + 8) * 2, fpitch = KP + 4;
   // operands of one chunk
   static constexpr int kt = 0, qt = 2 * rows, kh = 4 * rows, inv = 6 * rows, qk = inv + 2 * kDeltaTokens * kMPitch,
-                       v = qk + 2 * kDeltaTokens * kMPitch, beta = v + kDeltaTokens * kXPitch, total = beta + kDeltaTokens * 4,
+                       v = qk + 2 * kDeltaTokens * kMPitch, beta = v + kDeltaTokens * vpitch, total = beta + kDeltaTokens * 4,
                        operands = total + KP * 4;
-  // raw rows of one chunk: q, k, decay
-  static constexpr int raw = 3 * kDeltaTokens * KP * 2;
-  static constexpr int out = 2 * operands + 2 * raw, f32 = out + kDeltaTokens * kXPitch,
-                       bytes = f32 + (3 * kDeltaTokens * fpitch + kDeltaTokens * (kDeltaTokens + 4) + 2 * kDeltaTokens) * 4;
+  // what a preparing group works on: raw rows (q, k, decay), decays, A, reciprocal lengths
+  static constexpr int raw = 3 * kDeltaTokens * KP * 2, work = raw + (kDeltaTokens * fpitch + kDeltaTokens * (kDeltaTokens + 4) + 2 * kDeltaTokens) * 4;
+  static constexpr int out = kDeltaBuffers * operands + kDeltaGroups * work, bytes = out + kDeltaTokens * vpitch;
 };
 
 __device__ __forceinline__ void sc_stsm_t(uint32_t addr, const uint32_t (&r)[4]) {
   asm volatile("stmatrix.sync.aligned.m8n8.x4.trans.shared.b16 [%0], {%1,%2,%3,%4};" ::"r"(addr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3])
                : "memory");
 }
-__device__ __forceinline__ void half_barrier(int id) { asm volatile("bar.sync %0, 128;" ::"r"(id) : "memory"); }
+// barriers: 1 the applying warps, 2 .. the preparing groups, then per buffer "full" and "empty" (a group and the applying warps)
+constexpr int kBarGroup = 2, kBarFull = kBarGroup + kDeltaGroups, kBarEmpty = kBarFull + kDeltaBuffers;
+__device__ __forceinline__ void bar_wait(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
+__device__ __forceinline__ void bar_signal(int id, int threads) { asm volatile("bar.arrive %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
+template <int N> __device__ __forceinline__ void registers_up() { asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(N)); }
+template <int N> __device__ __forceinline__ void registers_down() { asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(N)); }
+template <int CT> constexpr int kApplyRegs = CT == 1 ? 200 : 248;       // 128 * these + 384 * the others = 512 * 128, the launch's
+template <int CT> constexpr int kPrepareRegs = CT == 1 ? 104 : 88;
+constexpr int kLaunchRegs = 128;
+static_assert(128 * kApplyRegs<1> + 384 * kPrepareRegs<1> <= kDeltaThreads * kLaunchRegs, "register split");
+static_assert(128 * kApplyRegs<2> + 384 * kPrepareRegs<2> <= kDeltaThreads * kLaunchRegs, "register split");
 __device__ __forceinline__ void put_split(uint8_t* hi, uint8_t* lo, float v) {
   const bf16 h = __float2bfloat16(v);
   *reinterpret_cast<bf16*>(hi) = h;
@@ -325,93 +355,91 @@ __device__ __forceinline__ void mma_split(float (&c)[4], const uint32_t (&ah)[4]
   sc_mma(c, ah, bl0, bl1);
 }
 
-// One chunk's operands from its raw rows, by 128 threads (tid 0 .. 127); m of its 16 tokens exist.
-template <int NK>
-__device__ __forceinline__ void delta_prepare(const DeltaParams<bf16>& p, uint8_t* op, const uint8_t* raw, float* f, int tid, int m, float A,
+// One chunk's operands from its raw rows, by a group of 128 threads (tid 0 .. 127); m of its 16 tokens exist.
+template <int NK, int CT>
+__device__ __forceinline__ void delta_prepare(const DeltaParams<bf16>& p, uint8_t* op, uint8_t* work, int tid, int group, int m, float A,
                                               float bias, const bf16* beta) {
-  typedef DeltaSmem<NK> Sm;
+  typedef DeltaSmem<NK, CT> Sm;
   constexpr int KP = Sm::KP, T = kDeltaTokens, FP = Sm::fpitch;
-  const int warp = tid >> 5, lane = tid & 31;
-  const bf16* rq = reinterpret_cast<const bf16*>(raw);
+  const int warp = tid >> 5, lane = tid & 31, bar = kBarGroup + group;
+  const bf16* rq = reinterpret_cast<const bf16*>(work);
   const bf16* rk = rq + T * KP;
   const bf16* rz = rk + T * KP;
-  float* kf = f;
-  float* qf = kf + T * FP;
-  float* gf = qf + T * FP;
+  float* gf = reinterpret_cast<float*>(work + Sm::raw);
   float* am = gf + T * FP;                       // A, [T][T + 4]
   float* iq = am + T * (T + 4);                  // reciprocal lengths
   float* ik = iq + T;
   float* bt = reinterpret_cast<float*>(op + Sm::beta);
-  // lengths: four tokens per warp
-#pragma unroll
-  for (int i = 0; i < T / 4; ++i) {
-    const int t = warp * (T / 4) + i;
+  // lengths: four tokens per warp, eight lanes per token
+  {
+    const int t = warp * 4 + (lane >> 3);
     float qq = 0.f, kk = 0.f;
-    for (int c = lane * 2; c < KP; c += 64) {
+#pragma unroll
+    for (int c = (lane & 7) * 2; c < KP; c += 16) {
       const float2 q = unpair(*reinterpret_cast<const uint32_t*>(rq + t * KP + c)), k = unpair(*reinterpret_cast<const uint32_t*>(rk + t * KP + c));
       qq = fmaf(q.x, q.x, fmaf(q.y, q.y, qq));
       kk = fmaf(k.x, k.x, fmaf(k.y, k.y, kk));
     }
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
+    for (int o = 4; o > 0; o >>= 1) {
       qq += __shfl_xor_sync(0xffffffffu, qq, o);
       kk += __shfl_xor_sync(0xffffffffu, kk, o);
     }
-    if (lane == 0) {
+    if ((lane & 7) == 0) {
       iq[t] = p.q_scale * rsqrtf(qq + kUnitEps);
       ik[t] = rsqrtf(kk + kUnitEps);
       bt[t] = t < m ? sigmoid_exact(to_f(beta[static_cast<long long>(t) * p.ld_beta])) : 0.f;
     }
   }
-  half_barrier(2);
+  bar_wait(bar, 128);
   if (tid < KP) {                                // one key channel per thread
     const int c = tid;
-    float k[T], g[T], P = 1.f;
+    float g[T], P = 1.f;
 #pragma unroll
     for (int t = 0; t < T; ++t) {
-      k[t] = to_f(rk[t * KP + c]) * ik[t];
-      const float q = to_f(rq[t * KP + c]) * iq[t], z = to_f(rz[t * KP + c]) + bias;
-      const float soft = fmaxf(z, 0.f) + __logf(1.f + __expf(-fabsf(z)));
+      const float z = to_f(rz[t * KP + c]) + bias, soft = fmaxf(z, 0.f) + __logf(1.f + __expf(-fabsf(z)));
       g[t] = t < m && c < p.K ? __expf(-A * soft) : 1.f;
-      P *= g[t];
-      kf[t * FP + c] = k[t];
-      qf[t * FP + c] = q;
       gf[t * FP + c] = g[t];
+    }
+#pragma unroll
+    for (int t = 0; t < T; ++t) {
+      P *= g[t];
       uint8_t* at = op + t * Sm::pitch + c * 2;
-      put_split(at + Sm::kt, at + Sm::kt + Sm::rows, k[t] * P);
-      put_split(at + Sm::qt, at + Sm::qt + Sm::rows, q * P);
+      put_split(at + Sm::kt, at + Sm::kt + Sm::rows, to_f(rk[t * KP + c]) * ik[t] * P);
+      put_split(at + Sm::qt, at + Sm::qt + Sm::rows, to_f(rq[t * KP + c]) * iq[t] * P);
     }
     reinterpret_cast<float*>(op + Sm::total)[c] = P;
     P = 1.f;
 #pragma unroll
     for (int t = T - 1; t >= 0; --t) {
       uint8_t* at = op + Sm::kh + t * Sm::pitch + c * 2;
-      put_split(at, at + Sm::rows, k[t] * P);
+      put_split(at, at + Sm::rows, to_f(rk[t * KP + c]) * ik[t] * P);
       P *= g[t];
     }
   }
-  half_barrier(2);
-  // A and Q by columns s, four per warp; a lane has four key channels
-#pragma unroll
+  bar_wait(bar, 128);
+  // A and Q by columns s, four per warp; a lane has four key channels, lengths enter at the end
+#pragma unroll 1
   for (int i = 0; i < T / 4; ++i) {
     const int s = i * 4 + (i & 1 ? 3 - warp : warp);
     float v[2 * T];
-    float4 d = make_float4(0.f, 0.f, 0.f, 0.f);
+    float2 d0 = make_float2(0.f, 0.f), d1 = d0;
     const bool on = lane * 4 < KP;
 #pragma unroll
     for (int t = 0; t < T; ++t) {
       v[t] = v[T + t] = 0.f;
-      if (t < s) continue;
-      if (!on) continue;
-      const float4 k = *reinterpret_cast<const float4*>(kf + t * FP + lane * 4), q = *reinterpret_cast<const float4*>(qf + t * FP + lane * 4);
+      if (t < s || !on) continue;
+      const uint2 kr = *reinterpret_cast<const uint2*>(rk + t * KP + lane * 4), qr = *reinterpret_cast<const uint2*>(rq + t * KP + lane * 4);
+      const float2 k0 = unpair(kr.x), k1 = unpair(kr.y), y0 = unpair(qr.x), y1 = unpair(qr.y);
       if (t == s) {
-        d = k;
+        d0 = k0;
+        d1 = k1;
       } else {
         const float4 g = *reinterpret_cast<const float4*>(gf + t * FP + lane * 4);
-        d.x *= g.x; d.y *= g.y; d.z *= g.z; d.w *= g.w;
-        v[t] = fmaf(d.x, k.x, fmaf(d.y, k.y, fmaf(d.z, k.z, d.w * k.w)));
+        d0.x *= g.x; d0.y *= g.y; d1.x *= g.z; d1.y *= g.w;
+        v[t] = fmaf(d0.x, k0.x, fmaf(d0.y, k0.y, fmaf(d1.x, k1.x, d1.y * k1.y)));
       }
-      v[T + t] = fmaf(d.x, q.x, fmaf(d.y, q.y, fmaf(d.z, q.z, d.w * q.w)));
+      v[T + t] = fmaf(d0.x, y0.x, fmaf(d0.y, y0.y, fmaf(d1.x, y1.x, d1.y * y1.y)));
     }
     // sums over the lanes; lane l keeps entry l
 #pragma unroll
@@ -424,22 +452,25 @@ __device__ __forceinline__ void delta_prepare(const DeltaParams<bf16>& p, uint8_
       }
     }
     const int t = lane & 15;
-    if (lane < T) am[t * (T + 4) + s] = t > s ? bt[t] * v[0] : 0.f;
+    if (lane < T) am[t * (T + 4) + s] = t > s ? bt[t] * ik[t] * ik[s] * v[0] : 0.f;
     else {
       uint8_t* at = op + Sm::qk + t * kMPitch + s * 2;
-      put_split(at, at + T * kMPitch, t >= s ? v[0] : 0.f);
+      put_split(at, at + T * kMPitch, t >= s ? iq[t] * ik[s] * v[0] : 0.f);
     }
   }
-  half_barrier(2);
+  bar_wait(bar, 128);
   if (tid < T) {                                 // column tid of the inverse of I + A
     float x[T];
 #pragma unroll
     for (int t = 0; t < T; ++t) {
       float a = t == tid ? 1.f : 0.f, b = 0.f;
 #pragma unroll
-      for (int s = 0; s < t; ++s) {
-        if (s & 1) b = fmaf(-am[t * (T + 4) + s], x[s], b);
-        else a = fmaf(-am[t * (T + 4) + s], x[s], a);
+      for (int s4 = 0; s4 < t; s4 += 4) {
+        const float4 r = *reinterpret_cast<const float4*>(am + t * (T + 4) + s4);
+        a = fmaf(-r.x, x[s4], a);
+        if (s4 + 1 < t) b = fmaf(-r.y, x[s4 + 1], b);
+        if (s4 + 2 < t) a = fmaf(-r.z, x[s4 + 2], a);
+        if (s4 + 3 < t) b = fmaf(-r.w, x[s4 + 3], b);
       }
       x[t] = a + b;
       uint8_t* at = op + Sm::inv + t * kMPitch + tid * 2;
@@ -448,15 +479,15 @@ __device__ __forceinline__ void delta_prepare(const DeltaParams<bf16>& p, uint8_
   }
 }
 
-// grid (column slabs, H, sequences); warps 0 - 3 apply, warps 4 - 7 prepare
-template <int NK>
+// grid (column slabs, H, sequences); warps 0 - 3 apply, the others prepare: group r the chunks r, r + 3, ..
+template <int NK, int CT>
 __global__ void __launch_bounds__(kDeltaThreads, 1) delta_chunk_kernel(const DeltaParams<bf16> p) {
   pdl_trigger();
   pdl_wait();
-  typedef DeltaSmem<NK> Sm;
+  typedef DeltaSmem<NK, CT> Sm;
   extern __shared__ __align__(128) uint8_t smem[];
-  constexpr int KP = Sm::KP, T = kDeltaTokens;
-  const int s = blockIdx.z, h = blockIdx.y, p0 = blockIdx.x * kDeltaCols, np = min(kDeltaCols, p.V - p0);
+  constexpr int KP = Sm::KP, T = kDeltaTokens, NB = kDeltaBuffers;
+  const int s = blockIdx.z, h = blockIdx.y, p0 = blockIdx.x * Sm::cols, np = min(Sm::cols, p.V - p0);
   const int q0 = p.cu_q[s], n = p.cu_q[s + 1] - q0, past = p.ref.kv_lens[s] - n;
   if (n <= 0) return;
   const int slot = slot_of(p.ref, s);
@@ -466,162 +497,203 @@ __global__ void __launch_bounds__(kDeltaThreads, 1) delta_chunk_kernel(const Del
   float* state = p.state + static_cast<long long>(slot) * p.slot_stride + (static_cast<long long>(h) * p.V + p0) * p.K;
   const bf16* rows = p.c + static_cast<long long>(q0) * p.ldc;
   if (warp >= 4) {
-    const int tid = threadIdx.x - 128;
+    registers_down<kPrepareRegs<CT>>();
+    const int group = (warp >> 2) - 1, tid = threadIdx.x & 127;
+    uint8_t* work = smem + NB * Sm::operands + group * Sm::work;
     const float A = p.A[h], bias = tid < p.K ? p.decay_bias[h * p.K + tid] : 0.f;
     const bf16* z = p.decay + static_cast<long long>(q0) * p.ld_decay + h * p.K;
     const bf16* beta = p.beta + static_cast<long long>(q0) * p.ld_beta + h;
+    // a thread copies one 16-byte piece of some rows
+    constexpr int V = KP / 8, STEP = 128 / V, VV = Sm::cols / 8, VSTEP = 128 / VV;
     auto fetch = [&](int i) {                    // raw rows of chunk i
-      uint8_t* dst = smem + 2 * Sm::operands + (i & 1) * Sm::raw;
-      for (int j = tid; j < 3 * T * (KP / 8); j += 128) {
-        const int what = j / (T * (KP / 8)), t = j / (KP / 8) % T, c = j % (KP / 8) * 8, row = i * T + t;
-        const bool there = row < n && c < p.K;
-        const bf16* src = what == 2 ? z + static_cast<long long>(there ? row : 0) * p.ld_decay
-                                    : rows + static_cast<long long>(there ? row : 0) * p.ldc + (what ? p.G + g : g) * p.K;
-        sc_copy16(sc_addr(dst + (what * T * KP + t * KP + c) * 2), src + (there ? c : 0), there);
+      const int c = tid % V * 8;
+      const bool in = c < p.K;
+#pragma unroll
+      for (int j = 0; j < (T + STEP - 1) / STEP; ++j) {
+        const int t = tid / V + j * STEP, row = i * T + t;
+        if (STEP > T && t >= T) break;
+        const bool there = in && row < n;
+        const long long r = there ? row : 0;
+        const uint32_t dst = sc_addr(work) + (t * KP + c) * 2;
+        const bf16* src = rows + r * p.ldc + (there ? g * p.K + c : 0);
+        sc_copy16(dst, src, there);
+        sc_copy16(dst + T * KP * 2, src + (there ? p.G * p.K : 0), there);
+        sc_copy16(dst + 2 * T * KP * 2, z + r * p.ld_decay + (there ? c : 0), there);
       }
     };
-    auto fetch_v = [&](int i) {
-      uint8_t* dst = smem + (i & 1) * Sm::operands + Sm::v;
-      const int t = tid >> 3, c = (tid & 7) * 8, row = i * T + t;                          // 16 rows of 8 pieces
-      const bool there = row < n && c < np;
-      sc_copy16(sc_addr(dst + t * kXPitch + c * 2),
-                rows + static_cast<long long>(there ? row : 0) * p.ldc + 2 * p.G * p.K + h * p.V + p0 + (there ? c : 0), there);
+    auto fetch_v = [&](int i, uint8_t* op) {
+      const int c = tid % VV * 8;
+#pragma unroll
+      for (int j = 0; j < T / VSTEP; ++j) {
+        const int t = tid / VV + j * VSTEP, row = i * T + t;
+        const bool there = row < n && c < np;
+        sc_copy16(sc_addr(op + Sm::v) + t * Sm::vpitch + c * 2,
+                  rows + static_cast<long long>(there ? row : 0) * p.ldc + (there ? 2 * p.G * p.K + h * p.V + p0 + c : 0), there);
+      }
     };
     auto landed = [&]() { asm volatile("cp.async.commit_group;\ncp.async.wait_group 0;" ::: "memory"); };
-    float* f = reinterpret_cast<float*>(smem + Sm::f32);
-    fetch(0);
-    fetch_v(0);
-    landed();
-    half_barrier(2);
-    if (chunks > 1) fetch(1);
-    delta_prepare<NK>(p, smem, smem + 2 * Sm::operands, f, tid, min(T, n), A, bias, beta);
-    landed();
-    __syncthreads();
-    for (int i = 0; i < chunks; ++i) {
-      if (i + 1 < chunks) {
-        fetch_v(i + 1);
-        if (i + 2 < chunks) fetch(i + 2);
-        delta_prepare<NK>(p, smem + ((i + 1) & 1) * Sm::operands, smem + 2 * Sm::operands + ((i + 1) & 1) * Sm::raw, f, tid,
-                          min(T, n - (i + 1) * T), A, bias, beta + static_cast<long long>((i + 1) * T) * p.ld_beta);
-        landed();
-      }
-      __syncthreads();
+    if (group < chunks) fetch(group);
+    for (int i = group; i < chunks; i += kDeltaGroups) {
+      uint8_t* op = smem + (i % NB) * Sm::operands;
+      landed();
+      if (i >= NB) bar_wait(kBarEmpty + i % NB, 256);
+      bar_wait(kBarGroup + group, 128);          // every thread's raw rows are here
+      fetch_v(i, op);
+      delta_prepare<NK, CT>(p, op, work, tid, group, min(T, n - i * T), A, bias, beta + static_cast<long long>(i * T) * p.ld_beta);
+      landed();
+      bar_signal(kBarFull + i % NB, 256);
+      // the group's last barrier inside lies behind the last read of its raw rows
+      if (i + kDeltaGroups < chunks) fetch(i + kDeltaGroups);
     }
-    delta_ring(p, p.conv.x + static_cast<long long>(q0) * p.conv.ld, slot, past, n, h, p0, np, tid, 128);
+    if (group == 0) delta_ring(p, p.conv.x + static_cast<long long>(q0) * p.conv.ld, slot, past, n, h, p0, np, tid, 128);
     return;
   }
-  float S[2 * NK][4];
+  registers_up<kApplyRegs<CT>>();
+  float S[CT][2 * NK][4];
 #pragma unroll
-  for (int j = 0; j < 2 * NK; ++j) {
+  for (int ct = 0; ct < CT; ++ct) {
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int col = warp * 16 + r4 + half * 8, key = j * 8 + c2;
-      const float2 v = past > 0 && col < np && key < p.K ? *reinterpret_cast<const float2*>(state + static_cast<long long>(col) * p.K + key)
-                                                         : make_float2(0.f, 0.f);
-      S[j][2 * half] = v.x;
-      S[j][2 * half + 1] = v.y;
+    for (int j = 0; j < 2 * NK; ++j) {
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int col = (warp * CT + ct) * 16 + r4 + half * 8, key = j * 8 + c2;
+        const float2 v = past > 0 && col < np && key < p.K ? *reinterpret_cast<const float2*>(state + static_cast<long long>(col) * p.K + key)
+                                                           : make_float2(0.f, 0.f);
+        S[ct][j][2 * half] = v.x;
+        S[ct][j][2 * half + 1] = v.y;
+      }
     }
   }
-  __syncthreads();
   const uint32_t out = sc_addr(smem + Sm::out);
   const uint32_t flat = ((lane & 7) + ((lane >> 4) << 3)), side = ((lane >> 3) & 1) * 16;        // 16 rows x 16 columns, rows as columns of B
   const uint32_t across = (lane & 7) + (((lane >> 3) & 1) << 3), part = lane >> 4;               // transposed reads
   for (int i = 0; i < chunks; ++i) {
-    const uint8_t* op = smem + (i & 1) * Sm::operands;
+    const uint8_t* op = smem + (i % NB) * Sm::operands;
     const uint32_t ob = sc_addr(op);
-    float w[2][4] = {}, o[2][4] = {};
+    bar_wait(kBarFull + i % NB, 256);
+    float w[CT][2][4] = {}, o[CT][2][4] = {};
 #pragma unroll
     for (int kk = 0; kk < NK; ++kk) {
-      uint32_t ah[4], al[4], bh[4], bl[4];
-      operand_split(S[2 * kk], S[2 * kk + 1], ah, al);
+      uint32_t bh[4], bl[4], dh[4], dl[4];
       const uint32_t at = ob + flat * Sm::pitch + kk * 32 + side;
       sc_ldsm(bh, at + Sm::kt);
       sc_ldsm(bl, at + Sm::kt + Sm::rows);
-      mma_split(w[0], ah, al, bh[0], bh[1], bl[0], bl[1]);
-      mma_split(w[1], ah, al, bh[2], bh[3], bl[2], bl[3]);
-      sc_ldsm(bh, at + Sm::qt);
-      sc_ldsm(bl, at + Sm::qt + Sm::rows);
-      mma_split(o[0], ah, al, bh[0], bh[1], bl[0], bl[1]);
-      mma_split(o[1], ah, al, bh[2], bh[3], bl[2], bl[3]);
-    }
-    uint32_t v[4];                               // (tokens 0-7, columns 0-7), (tokens 8-15, columns 0-7), then columns 8-15
-    sc_ldsm_t(v, ob + Sm::v + across * kXPitch + (warp * 2 + part) * 16);
-    const float* bt = reinterpret_cast<const float*>(op + Sm::beta);
+      sc_ldsm(dh, at + Sm::qt);
+      sc_ldsm(dl, at + Sm::qt + Sm::rows);
 #pragma unroll
-    for (int j = 0; j < 2; ++j) {
-      const float2 b = *reinterpret_cast<const float2*>(bt + j * 8 + c2), v0 = unpair(v[j]), v1 = unpair(v[2 + j]);
-      w[j][0] = b.x * (v0.x - w[j][0]);
-      w[j][1] = b.y * (v0.y - w[j][1]);
-      w[j][2] = b.x * (v1.x - w[j][2]);
-      w[j][3] = b.y * (v1.y - w[j][3]);
+      for (int ct = 0; ct < CT; ++ct) {
+        uint32_t ah[4], al[4];
+        operand_split(S[ct][2 * kk], S[ct][2 * kk + 1], ah, al);
+        mma_split(w[ct][0], ah, al, bh[0], bh[1], bl[0], bl[1]);
+        mma_split(w[ct][1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+        mma_split(o[ct][0], ah, al, dh[0], dh[1], dl[0], dl[1]);
+        mma_split(o[ct][1], ah, al, dh[2], dh[3], dl[2], dl[3]);
+      }
     }
-    uint32_t ah[4], al[4], bh[4], bl[4];
-    operand_split(w[0], w[1], ah, al);
-    float u[2][4] = {};
+    const float* bt = reinterpret_cast<const float*>(op + Sm::beta);
     const uint32_t mat = ob + flat * kMPitch + side;
-    sc_ldsm(bh, mat + Sm::inv);
-    sc_ldsm(bl, mat + Sm::inv + T * kMPitch);
-    mma_split(u[0], ah, al, bh[0], bh[1], bl[0], bl[1]);
-    mma_split(u[1], ah, al, bh[2], bh[3], bl[2], bl[3]);
-    operand_split(u[0], u[1], ah, al);
-    sc_ldsm(bh, mat + Sm::qk);
-    sc_ldsm(bl, mat + Sm::qk + T * kMPitch);
-    mma_split(o[0], ah, al, bh[0], bh[1], bl[0], bl[1]);
-    mma_split(o[1], ah, al, bh[2], bh[3], bl[2], bl[3]);
-    const uint32_t packed[4] = {pair(o[0][0], o[0][1]), pair(o[1][0], o[1][1]), pair(o[0][2], o[0][3]), pair(o[1][2], o[1][3])};
-    sc_stsm_t(out + across * kXPitch + (warp * 2 + part) * 16, packed);
+    uint32_t uh[CT][4], ul[CT][4];
+#pragma unroll
+    for (int ct = 0; ct < CT; ++ct) {
+      uint32_t v[4];                             // (tokens 0-7, columns 0-7), (tokens 8-15, columns 0-7), then columns 8-15
+      sc_ldsm_t(v, ob + Sm::v + across * Sm::vpitch + ((warp * CT + ct) * 2 + part) * 16);
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        const float2 b = *reinterpret_cast<const float2*>(bt + j * 8 + c2), v0 = unpair(v[j]), v1 = unpair(v[2 + j]);
+        w[ct][j][0] = b.x * (v0.x - w[ct][j][0]);
+        w[ct][j][1] = b.y * (v0.y - w[ct][j][1]);
+        w[ct][j][2] = b.x * (v1.x - w[ct][j][2]);
+        w[ct][j][3] = b.y * (v1.y - w[ct][j][3]);
+      }
+      uint32_t ah[4], al[4], bh[4], bl[4];
+      operand_split(w[ct][0], w[ct][1], ah, al);
+      float u[2][4] = {};
+      sc_ldsm(bh, mat + Sm::inv);
+      sc_ldsm(bl, mat + Sm::inv + T * kMPitch);
+      mma_split(u[0], ah, al, bh[0], bh[1], bl[0], bl[1]);
+      mma_split(u[1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+      operand_split(u[0], u[1], uh[ct], ul[ct]);
+    }
     const float* total = reinterpret_cast<const float*>(op + Sm::total);
 #pragma unroll
     for (int kk = 0; kk < NK; ++kk) {
+      uint32_t bh[4], bl[4];
       const uint32_t at = ob + Sm::kh + across * Sm::pitch + (kk * 2 + part) * 16;
       sc_ldsm_t(bh, at);
       sc_ldsm_t(bl, at + Sm::rows);
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const float2 d = *reinterpret_cast<const float2*>(total + kk * 16 + j * 8 + c2);
-        float (&t)[4] = S[2 * kk + j];
-        t[0] *= d.x; t[1] *= d.y; t[2] *= d.x; t[3] *= d.y;
-        mma_split(t, ah, al, bh[2 * j], bh[2 * j + 1], bl[2 * j], bl[2 * j + 1]);
+#pragma unroll
+        for (int ct = 0; ct < CT; ++ct) {
+          float (&t)[4] = S[ct][2 * kk + j];
+          t[0] *= d.x; t[1] *= d.y; t[2] *= d.x; t[3] *= d.y;
+          mma_split(t, uh[ct], ul[ct], bh[2 * j], bh[2 * j + 1], bl[2 * j], bl[2 * j + 1]);
+        }
       }
     }
-    half_barrier(1);                             // the chunk's output rows are complete
     {
-      const int t = threadIdx.x >> 3, c = (threadIdx.x & 7) * 8;
+      uint32_t bh[4], bl[4];
+      sc_ldsm(bh, mat + Sm::qk);
+      sc_ldsm(bl, mat + Sm::qk + T * kMPitch);
+      if (i > 0) bar_wait(1, 128);               // the rows of the chunk before have been stored
+#pragma unroll
+      for (int ct = 0; ct < CT; ++ct) {
+        mma_split(o[ct][0], uh[ct], ul[ct], bh[0], bh[1], bl[0], bl[1]);
+        mma_split(o[ct][1], uh[ct], ul[ct], bh[2], bh[3], bl[2], bl[3]);
+        const uint32_t packed[4] = {pair(o[ct][0][0], o[ct][0][1]), pair(o[ct][1][0], o[ct][1][1]), pair(o[ct][0][2], o[ct][0][3]),
+                                    pair(o[ct][1][2], o[ct][1][3])};
+        sc_stsm_t(out + across * Sm::vpitch + ((warp * CT + ct) * 2 + part) * 16, packed);
+      }
+    }
+    if (i + NB < chunks) bar_signal(kBarEmpty + i % NB, 256);
+    bar_wait(1, 128);                            // the chunk's output rows are complete
+#pragma unroll
+    for (int j = 0; j < CT; ++j) {
+      const int at = threadIdx.x + j * 128, t = at / (8 * CT), c = at % (8 * CT) * 8;
       if (i * T + t < n && c < np)
         *reinterpret_cast<uint4*>(p.o + static_cast<long long>(q0 + i * T + t) * p.ldo + h * p.V + p0 + c) =
-            *reinterpret_cast<const uint4*>(smem + Sm::out + t * kXPitch + c * 2);
+            *reinterpret_cast<const uint4*>(smem + Sm::out + t * Sm::vpitch + c * 2);
     }
-    __syncthreads();
   }
 #pragma unroll
-  for (int j = 0; j < 2 * NK; ++j) {
+  for (int ct = 0; ct < CT; ++ct) {
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int col = warp * 16 + r4 + half * 8, key = j * 8 + c2;
-      if (col < np && key < p.K)
-        *reinterpret_cast<float2*>(state + static_cast<long long>(col) * p.K + key) = make_float2(S[j][2 * half], S[j][2 * half + 1]);
+    for (int j = 0; j < 2 * NK; ++j) {
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int col = (warp * CT + ct) * 16 + r4 + half * 8, key = j * 8 + c2;
+        if (col < np && key < p.K)
+          *reinterpret_cast<float2*>(state + static_cast<long long>(col) * p.K + key) = make_float2(S[ct][j][2 * half], S[ct][j][2 * half + 1]);
+      }
     }
   }
 }
 
-template <int NK>
+template <int NK, int CT>
 static int launch_delta_chunks(const DeltaParams<bf16>& p, int B, cudaStream_t st) {
-  static bool set = false;
-  if (!set) {
-    if (cudaFuncSetAttribute(delta_chunk_kernel<NK>, cudaFuncAttributeMaxDynamicSharedMemorySize, DeltaSmem<NK>::bytes) != cudaSuccess) return -3;
-    set = true;
+  typedef DeltaSmem<NK, CT> Sm;
+  static int ok = 0;                             // 1: ready, -1: not with the registers that the kernel was compiled to
+  if (ok == 0) {
+    cudaFuncAttributes a;
+    if (cudaFuncGetAttributes(&a, delta_chunk_kernel<NK, CT>) != cudaSuccess ||
+        cudaFuncSetAttribute(delta_chunk_kernel<NK, CT>, cudaFuncAttributeMaxDynamicSharedMemorySize, Sm::bytes) != cudaSuccess) return -3;
+    ok = a.numRegs == kLaunchRegs ? 1 : -1;
   }
-  return launch_pdl(delta_chunk_kernel<NK>, dim3((p.V + kDeltaCols - 1) / kDeltaCols, p.H, B), dim3(kDeltaThreads), DeltaSmem<NK>::bytes, st,
-                    p) == cudaSuccess ? 0 : -4;
+  if (ok < 0) return -100;
+  return launch_pdl(delta_chunk_kernel<NK, CT>, dim3((p.V + Sm::cols - 1) / Sm::cols, p.H, B), dim3(kDeltaThreads), Sm::bytes, st, p) ==
+                 cudaSuccess ? 0 : -4;
 }
 
 int delta_chunks(const DeltaParams<bf16>& p, int B, cudaStream_t st) {
   const int steps = (p.K + 15) / 16;
   if (steps > 8 || p.ldc % 8 || p.ld_decay % 8 || !aligned16(p.c) || !aligned16(p.decay) || p.ldo % 8) return -100;
-  if (steps <= 1) return launch_delta_chunks<1>(p, B, st);
-  if (steps <= 2) return launch_delta_chunks<2>(p, B, st);
-  if (steps <= 4) return launch_delta_chunks<4>(p, B, st);
-  return launch_delta_chunks<8>(p, B, st);
+  // 64 columns per CTA while these fill at most one wave, else 128
+  const bool wide = p.V > 64 && static_cast<long long>((p.V + 63) / 64) * p.H * B > 148;
+  if (steps <= 1) return wide ? launch_delta_chunks<1, 2>(p, B, st) : launch_delta_chunks<1, 1>(p, B, st);
+  if (steps <= 2) return wide ? launch_delta_chunks<2, 2>(p, B, st) : launch_delta_chunks<2, 1>(p, B, st);
+  if (steps <= 4) return wide ? launch_delta_chunks<4, 2>(p, B, st) : launch_delta_chunks<4, 1>(p, B, st);
+  return wide ? launch_delta_chunks<8, 2>(p, B, st) : launch_delta_chunks<8, 1>(p, B, st);
 }
 
 }  // namespace ksana
