@@ -23,6 +23,7 @@
 // columns past the row's end). K and V lie in panels of their own: [block][Hkv][block_tokens][D] and [...][Dv].
 // Sliding window: position i sees j <= i with i - j < window or j < keep; tiles between the kept tokens and the
 // window are not visited. Sink: an extra logit per head in the softmax denominator, without a value.
+// Panels that coincide (the values are the keys) are staged once.
 // Sigmoid weights (SIG): every visible key has the weight sigmoid(score + bias[head][distance]), nothing is normalised over
 // keys. Gate: outputs are multiplied by the sigmoid of a gate element and by one factor.
 //
@@ -179,20 +180,21 @@ __device__ __forceinline__ void load_kv_tile(bf16* dst, const AttnParams& p, con
   }
 }
 
-// TMA staging of one K + V tile (one thread): a box of [block_tokens rows x 64 columns] per cache block and
+// TMA staging of one K + V tile (one thread; `shared`: the keys are the values, one tile): a box of [block_tokens rows x 64 columns] per cache block and
 // 64-column panel. Tokens past kv_len inside the last block are loaded as they are (finite cache contents)
 // and masked by the softmax; blocks past the sequence are not loaded at all.
 template <int D>
-__device__ __forceinline__ void tma_issue_kv(bf16* ks, bf16* vs, uint64_t* bar, const CUtensorMap* kmap, const CUtensorMap* vmap,
+__device__ __forceinline__ void tma_issue_kv(bf16* ks, bf16* vs, bool shared, uint64_t* bar, const CUtensorMap* kmap, const CUtensorMap* vmap,
                                              const AttnParams& p, const int* table, int g, int tok0, int kv_len) {
   const int bt = p.block_tokens;
   const int nblk = min(kTileTok / bt, (kv_len - tok0 + bt - 1) / bt);
   constexpr int PANELS = D / 64;
-  mbar_expect_tx(bar, static_cast<uint32_t>(nblk) * 2 * PANELS * bt * 128);
+  mbar_expect_tx(bar, static_cast<uint32_t>(nblk) * (shared ? 1 : 2) * PANELS * bt * 128);
   for (int b = 0; b < nblk; ++b) {
     const int blk = table[tok0 / bt + b];
 #pragma unroll
     for (int which = 0; which < 2; ++which) {
+      if (which && shared) break;
       bf16* dst = which ? vs : ks;
 #pragma unroll
       for (int h = 0; h < PANELS; ++h)      // columns past the row's end arrive as zeros
@@ -343,7 +345,8 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_con
   __shared__ uint32_t abort_word;
   bf16* qs = reinterpret_cast<bf16*>(smem_attn);            // 64 x D
   bf16* ks = qs + 64 * D;                                   // kKvStages x (64 x D)
-  bf16* vs = ks + kKvStages * kTileTok * D;                 // kKvStages x (64 x D)
+  const bool shared = p.kc == p.vc;
+  bf16* vs = shared ? ks : ks + kKvStages * kTileTok * D;   // kKvStages x (64 x D)
 
   const int s = blockIdx.z, g = blockIdx.y;
   const int G = p.Hq / p.Hkv;
@@ -384,12 +387,12 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_con
     const int st = t % kKvStages, tok0 = tile_at(tiles, t) * kTileTok;
     if (MODE == kKvTma) {
       if (threadIdx.x == 0 && t < ntiles)
-        tma_issue_kv<D>(ks + st * kTileTok * D, vs + st * kTileTok * D, &full_bar[st], &k_map, &v_map, p, table, g, tok0, kv_len);
+        tma_issue_kv<D>(ks + st * kTileTok * D, vs + st * kTileTok * D, shared, &full_bar[st], &k_map, &v_map, p, table, g, tok0, kv_len);
       return;
     }
     if (t < ntiles) {
       load_kv_tile<D, FP8>(ks + st * kTileTok * D, p, table, g, 0, tok0, kv_len, p.k_scale);
-      load_kv_tile<D, FP8>(vs + st * kTileTok * D, p, table, g, 1, tok0, kv_len, p.v_scale);
+      if (!shared) load_kv_tile<D, FP8>(vs + st * kTileTok * D, p, table, g, 1, tok0, kv_len, p.v_scale);
     }
     cp_commit();
   };
@@ -482,7 +485,8 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
   __shared__ float red4[4];
   bf16* qs = reinterpret_cast<bf16*>(smem_attn);            // 16 x D
   bf16* ks = qs + 16 * D;                                   // kKvStages x (64 x D)
-  bf16* vs = ks + kKvStages * kTileTok * D;
+  const bool shared = p.kc == p.vc;
+  bf16* vs = shared ? ks : ks + kKvStages * kTileTok * D;
   float* merge = reinterpret_cast<float*>(ks);              // 4 warps x 16 rows x (D + 2), reuses the K ring after the loop
 
   pdl_trigger();
@@ -518,12 +522,12 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
     const int st = (t - t_begin) % kKvStages, tok0 = tile_at(tiles, t) * kTileTok;
     if (MODE == kKvTma) {
       if (threadIdx.x == 0 && t < t_end)
-        tma_issue_kv<D>(ks + st * kTileTok * D, vs + st * kTileTok * D, &full_bar[st], &k_map, &v_map, p, table, g, tok0, kv_len);
+        tma_issue_kv<D>(ks + st * kTileTok * D, vs + st * kTileTok * D, shared, &full_bar[st], &k_map, &v_map, p, table, g, tok0, kv_len);
       return;
     }
     if (t < t_end) {
       load_kv_tile<D, FP8>(ks + st * kTileTok * D, p, table, g, 0, tok0, kv_len, p.k_scale);
-      load_kv_tile<D, FP8>(vs + st * kTileTok * D, p, table, g, 1, tok0, kv_len, p.v_scale);
+      if (!shared) load_kv_tile<D, FP8>(vs + st * kTileTok * D, p, table, g, 1, tok0, kv_len, p.v_scale);
     }
     cp_commit();
   };

@@ -43,6 +43,7 @@ struct FaParams {
   const int* cu_q; const int* kv_lens; const float* alibi;
   const float* sinks;                        // [Hq] logits added to the softmax denominator, or null
   int Hq, Hkv, G, block_tokens;
+  int shared;                                // the values are the keys: one tile per step, two in flight
   int rows;                                  // query rows of a CTA: the largest multiple of G up to 128
   int D, Dv;                                 // real head sizes
   int window, keep;                          // sliding window in tokens (0: none), first tokens every row sees
@@ -135,7 +136,18 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       for (int h = 0; h < kpanels; ++h) tma_load_3d(q_s + h * kFaPanelBytes, &q_map, q_full, h * 64, g * G, tok0);
       const int bt = p.block_tokens;
       bool ok = true;
-      for (int j = 0; j < ntiles && ok; ++j) {
+      for (int j = 0; p.shared && j < ntiles && ok; ++j) {       // key tiles alternate between the two places
+        const int t0 = tile_start(j), nblk = min(kFaTile / bt, (kv_len - t0 + bt - 1) / bt);
+        uint8_t* dst = j & 1 ? v_s : k_s;
+        uint64_t* full = j & 1 ? v_full : k_full;
+        if (!mbar_wait(j & 1 ? v_empty : k_empty, ((j >> 1) & 1) ^ 1, abort_flag)) { ok = false; break; }
+        mbar_expect_tx(full, static_cast<uint32_t>(nblk) * kpanels * bt * 128);
+        for (int b = 0; b < nblk; ++b) {
+          const int blk = table[t0 / bt + b];
+          for (int h = 0; h < kpanels; ++h) tma_load_3d(dst + h * kFaPanelBytes + b * bt * 128, &k_map, full, h * 64, g * bt, blk);
+        }
+      }
+      for (int j = 0; !p.shared && j < ntiles && ok; ++j) {
         const int t0 = tile_start(j);
         const int nblk = min(kFaTile / bt, (kv_len - t0 + bt - 1) / bt);
 #pragma unroll
@@ -164,28 +176,33 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       bool ok = mbar_wait(q_full, 0, abort_flag);
       for (int j = 0; j < ntiles && ok; ++j) {
         const uint32_t par = j & 1;
-        if (!mbar_wait(k_full, par, abort_flag)) { ok = false; break; }
+        const bool second = p.shared && (j & 1);
+        uint8_t* kt = second ? v_s : k_s;
+        uint8_t* vt = p.shared ? kt : v_s;
+        if (!mbar_wait(second ? v_full : k_full, p.shared ? (j >> 1) & 1 : par, abort_flag)) { ok = false; break; }
         tc_fence_after();
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
           if (k >= ksteps) break;
           const uint32_t off = (k >> 2) * kFaPanelBytes;
           const uint64_t adesc = make_smem_desc_sw128(smem_u32(q_s) + off) + 2 * (k & 3);
-          const uint64_t bdesc = make_smem_desc_sw128(smem_u32(k_s) + off) + 2 * (k & 3);
+          const uint64_t bdesc = make_smem_desc_sw128(smem_u32(kt) + off) + 2 * (k & 3);
           mma_f16(tmem_s, adesc, bdesc, idesc_qk, k != 0);
         }
         tc_commit(s_full);
-        tc_commit(k_empty);
-        if (!mbar_wait(v_full, par, abort_flag)) { ok = false; break; }
+        if (!p.shared) {
+          tc_commit(k_empty);
+          if (!mbar_wait(v_full, par, abort_flag)) { ok = false; break; }
+        }
         if (!mbar_wait(p_full, par, abort_flag)) { ok = false; break; }
         tc_fence_after();
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
           // 16 tokens per MMA: 8 TMEM columns of P (two bf16 each), 16 rows (2 KB) of the V tile
-          const uint64_t bdesc = make_smem_desc_mn_sw128(smem_u32(v_s) + k * 2048, kFaPanelBytes);
+          const uint64_t bdesc = make_smem_desc_mn_sw128(smem_u32(vt) + k * 2048, kFaPanelBytes);
           mma_f16_ts(tmem_o, tmem_s + 8 * k, bdesc, idesc_pv, (j | k) != 0);
         }
-        tc_commit(v_empty);
+        tc_commit(p.shared && !second ? k_empty : v_empty);
         if (j == ntiles - 1) tc_commit(o_full);
       }
     }
@@ -334,12 +351,14 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       if (t0 + kFaTile > kv_len) {
         // last tile of the sequence: V rows past the sequence end hold stale shared memory or whatever the cache
         // has there; their probabilities are 0, but 0 x NaN would poison O. Zero them before the PV MMA reads.
-        if (!mbar_wait(v_full, par, abort_flag)) { ok = false; break; }
+        // (the keys' product is complete here, so a shared tile is free to be changed)
+        if (!p.shared && !mbar_wait(v_full, par, abort_flag)) { ok = false; break; }
+        uint8_t* vt = p.shared && !(j & 1) ? k_s : v_s;
         const int first_bad = kv_len - t0;
         const int nchunks = (kFaTile - first_bad) * 16;       // 16-byte chunks per row: 2 panels x 8
         for (int i = threadIdx.x - 64; i < nchunks; i += 128) {
           const int r = first_bad + (i >> 4), ch = i & 15;
-          *reinterpret_cast<uint4*>(v_s + (ch >> 3) * kFaPanelBytes + r * 128 + (((ch & 7) ^ (r & 7)) << 4)) =
+          *reinterpret_cast<uint4*>(vt + (ch >> 3) * kFaPanelBytes + r * 128 + (((ch & 7) ^ (r & 7)) << 4)) =
               make_uint4(0, 0, 0, 0);
         }
         fence_async_smem();
@@ -468,6 +487,7 @@ extern "C" int ksana_paged_prefill_tc(const void* q, long long q_stride, long lo
   FaParams p{};
   p.out = static_cast<bf16*>(out); p.out_stride = out_stride;
   p.block_table = block_table; p.table_stride = table_stride; p.cu_q = cu_q; p.kv_lens = kv_lens; p.alibi = alibi;
+  p.shared = kc == vc && D == Dv;
   p.sinks = sinks; p.D = D; p.Dv = Dv; p.window = window; p.keep = window > 0 ? keep : 0;
   p.Hq = Hq; p.Hkv = Hkv; p.G = G; p.block_tokens = bt; p.rows = kFaTile / G * G;
   p.scale_log2 = scale * 1.44269504f;

@@ -43,7 +43,7 @@ __device__ __forceinline__ void conv_one(const ConvRef<T>& v, const T* row, cons
     for (int e = 0; e < 8; ++e) acc[e] = fmaf(f[e], w[e], acc[e]);
   }
 #pragma unroll
-  for (int e = 0; e < 8; ++e) acc[e] = silu_f(acc[e]);
+  for (int e = 0; e < 8; ++e) acc[e] *= sigmoid_as<T>(acc[e]);
 }
 
 // ------------------------------------------------------------------------------------------------ convolution
@@ -79,12 +79,13 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(const ConvRef<T> v, co
     for (int j = 0; j < TAPS - 1; ++j) input(row0 - (TAPS - 1) + j, hist[j]);
   }
   const int end = min(row0 + kConvRows, n);
+#pragma unroll 4
   for (int t = row0; t < end; ++t) {
     float acc[8], f[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e) acc[e] = b[e];
     if constexpr (TAPS > 0) {
-      input(t, f);
+      load8(x + t * v.ld, f);
 #pragma unroll
       for (int j = 0; j < TAPS - 1; ++j) {
 #pragma unroll
@@ -107,7 +108,7 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(const ConvRef<T> v, co
       }
     }
 #pragma unroll
-    for (int e = 0; e < 8; ++e) acc[e] = silu_f(acc[e]);
+    for (int e = 0; e < 8; ++e) acc[e] *= sigmoid_as<T>(acc[e]);
     store8(out + static_cast<long long>(q0 + t) * ldo + c, acc);
   }
 }
@@ -248,6 +249,7 @@ __global__ void space_step_kernel(const SpaceParams<T> p) {
   pdl_wait();
   constexpr int KP = J * kLanes * 4;
   __shared__ __align__(16) float Bs[KP], Cs[KP], xs[64];
+  __shared__ float step, decay;
   const int slab = blockDim.x / kLanes, s = blockIdx.z, h = blockIdx.y, p0 = blockIdx.x * slab, np = min(slab, p.P - p0);
   const int slot = slot_of(p.ref, s), pos = p.ref.kv_lens[s] - 1;
   const int lane = threadIdx.x & (kLanes - 1), col = threadIdx.x / kLanes, g = h / (p.H / p.G);
@@ -275,13 +277,16 @@ __global__ void space_step_kernel(const SpaceParams<T> p) {
 #pragma unroll
     for (int e = 0; e < 8; ++e) dst[e] = f[e];
   }
-  const float dt = softplus_f(to_f(p.dt[static_cast<long long>(s) * p.ld_dt + h]) + p.dt_bias[h]), a = decay_f(p.A[h] * dt);
+  if (threadIdx.x == blockDim.x - 1) {
+    step = softplus_f(to_f(p.dt[static_cast<long long>(s) * p.ld_dt + h]) + p.dt_bias[h]);
+    decay = decay_f(p.A[h] * step);
+  }
   __syncthreads();
   F2 B[J][2], C[J][2];
   load_keys<J>(Bs, lane, B);
   load_keys<J>(Cs, lane, C);
   const float x = col < np ? xs[col] : 0.f;
-  const float v = lanes_sum(space_token<J>(S, B, C, f2(a), f2(dt * x)));
+  const float v = lanes_sum(space_token<J>(S, B, C, f2(decay), f2(step * x)));
   if (col < np) {
     store_column<J>(state, p.N, lane, S);
     if (lane == 0) y[col] = from_f<T>(fmaf(p.D[h], x, v));
@@ -426,8 +431,7 @@ __global__ void delta_step_kernel(const DeltaParams<T> p) {
   pdl_trigger();
   pdl_wait();
   constexpr int KP = J * kLanes * 4;
-  __shared__ __align__(16) float qr[KP], kr[KP], qs[KP], ks[KP], gs[KP], vs[64];
-  __shared__ float qk;
+  __shared__ __align__(16) float qs[KP], ks[KP], gs[KP], vs[64];
   const int slab = blockDim.x / kLanes, s = blockIdx.z, h = blockIdx.y, p0 = blockIdx.x * slab, np = min(slab, p.V - p0);
   const int slot = slot_of(p.ref, s), pos = p.ref.kv_lens[s] - 1;
   const int lane = threadIdx.x & (kLanes - 1), col = threadIdx.x / kLanes, g = h / (p.H / p.G);
@@ -445,28 +449,61 @@ __global__ void delta_step_kernel(const DeltaParams<T> p) {
   }
   const T* row = p.conv.x + static_cast<long long>(s) * p.conv.ld;
   const T* ring = p.conv.ring + static_cast<long long>(slot) * p.conv.slot_stride;
-  const int kv = p.K >> 3, pv = np >> 3;
+  const int kv = KP >> 3, rv = p.K >> 3, pv = np >> 3;
   for (int i = threadIdx.x; i < 2 * kv + pv; i += blockDim.x) {
     const int k = i < kv ? i : i < 2 * kv ? i - kv : i - 2 * kv;
-    float f[8];
-    float* dst = i < kv ? qr + k * 8 : i < 2 * kv ? kr + k * 8 : vs + k * 8;
-    conv_one(p.conv, row, ring, pos, (i < kv ? g * p.K : i < 2 * kv ? (p.G + g) * p.K : 2 * p.G * p.K + h * p.V + p0) + k * 8, f);
+    float f[8] = {};
+    float* dst = i < kv ? qs + k * 8 : i < 2 * kv ? ks + k * 8 : vs + k * 8;
+    if (i >= 2 * kv || k < rv)
+      conv_one(p.conv, row, ring, pos, (i < kv ? g * p.K : i < 2 * kv ? (p.G + g) * p.K : 2 * p.G * p.K + h * p.V + p0) + k * 8, f);
 #pragma unroll
     for (int e = 0; e < 8; ++e) dst[e] = f[e];
   }
+  const float A = p.A[h];
+  for (int i = blockDim.x - 1 - threadIdx.x; i < KP; i += blockDim.x)        // the other end of the CTA meanwhile
+    gs[i] = i < p.K ? decay_f(A * softplus_f(to_f(p.decay[static_cast<long long>(s) * p.ld_decay + h * p.K + i]) + p.decay_bias[h * p.K + i])) : 1.f;
   const float beta = sigmoid_exact(to_f(p.beta[static_cast<long long>(s) * p.ld_beta + h]));
   __syncthreads();
-  if (threadIdx.x < 32) {
-    const T* z = p.decay + static_cast<long long>(s) * p.ld_decay + h * p.K;
-    delta_operands<KP>(p.K, p.A[h], p.decay_bias + h * p.K, p.q_scale,
-                       [&](int i, float& a, float& b, float& d) { a = qr[i]; b = kr[i]; d = to_f(z[i]); }, qs, ks, gs, &qk);
+  // lengths in every warp; the vectors stay as they are, their reciprocal lengths go into the sums
+  float qq = 0.f, kk = 0.f, qk = 0.f;
+  {
+    const int l = threadIdx.x & 31;
+#pragma unroll
+    for (int e = 0; e < KP / 32; ++e) {
+      const float a = qs[l + e * 32], b = ks[l + e * 32];
+      qq = fmaf(a, a, qq);
+      kk = fmaf(b, b, kk);
+      qk = fmaf(a, b, qk);
+    }
+#pragma unroll
+    for (int t = 16; t > 0; t >>= 1) {
+      qq += __shfl_xor_sync(0xffffffffu, qq, t);
+      kk += __shfl_xor_sync(0xffffffffu, kk, t);
+      qk += __shfl_xor_sync(0xffffffffu, qk, t);
+    }
   }
-  __syncthreads();
+  const float fq = p.q_scale / sqrtf(qq + kUnitEps), fk = 1.f / sqrtf(kk + kUnitEps);
   F2 q[J][2], k[J][2], d[J][2];
   load_keys<J>(qs, lane, q);
   load_keys<J>(ks, lane, k);
   load_keys<J>(gs, lane, d);
-  const float v = delta_token<J>(S, q, k, d, qk, col < np ? vs[col] : 0.f, beta);
+  F2 kept = f2(0.f), seen = f2(0.f);
+#pragma unroll
+  for (int j = 0; j < J; ++j) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      S[j][i] = S[j][i] * d[j][i];
+      kept = fma2(S[j][i], k[j][i], kept);
+      seen = fma2(S[j][i], q[j][i], seen);
+    }
+  }
+  const float u = beta * ((col < np ? vs[col] : 0.f) - fk * lanes_sum(sum2(kept))), v = fq * fmaf(qk * fk, u, lanes_sum(sum2(seen)));
+  const F2 u2 = f2(u * fk);
+#pragma unroll
+  for (int j = 0; j < J; ++j) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i) S[j][i] = fma2(k[j][i], u2, S[j][i]);
+  }
   if (col < np) {
     store_column<J>(state, p.K, lane, S);
     if (lane == 0) o[col] = from_f<T>(v);

@@ -15,7 +15,11 @@ __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + lo
 // exp(-x), x >= 0, rounded to nearest near 1: a decay is applied once per token, a bias of its last bit would add up
 __device__ __forceinline__ float decay_f(float x) { return 1.f + expm1f(-x); }
 __device__ __forceinline__ float sigmoid_exact(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+// in the activations' precision
+template <typename T> __device__ __forceinline__ float sigmoid_as(float x) {
+  if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-x));
+  else return sigmoid_exact(x);
+}
 
 struct StateRef {                            // where sequences keep their state
   const int* slots; int num_slots;           // per sequence; < 0: padding

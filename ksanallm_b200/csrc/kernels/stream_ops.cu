@@ -14,7 +14,10 @@
 
 namespace ksana {
 
-__device__ __forceinline__ float sigmoid_exact(float x) { return 1.f / (1.f + expf(-x)); }
+// in the activations' precision
+template <typename T> __device__ __forceinline__ float sigmoid_as(float x) {
+  return sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-x)) : 1.f / (1.f + expf(-x));
+}
 
 // Sum over the CTA, in every thread. `red`: 32 floats of shared memory
 __device__ __forceinline__ float cta_sum(float v, float* red) {
@@ -141,7 +144,7 @@ __global__ void gated_norm_kernel(const GatedNormParams<T> p) {
         float f[8];
         load8(p.z + static_cast<long long>(m) * p.ldz + i * 8, f);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[j][e] *= f[e] * sigmoid_exact(f[e]);
+        for (int e = 0; e < 8; ++e) v[j][e] *= f[e] * sigmoid_as<T>(f[e]);
       }
       if (whole) {
         float s = 0.f;
@@ -188,7 +191,7 @@ __global__ void gated_norm_kernel(const GatedNormParams<T> p) {
         float f[8];
         load8(p.g + static_cast<long long>(m) * p.ldg + i * 8, f);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[j][e] *= sigmoid_exact(f[e]);
+        for (int e = 0; e < 8; ++e) v[j][e] *= sigmoid_as<T>(f[e]);
       }
       store8(p.out + static_cast<long long>(m) * p.ldo + i * 8, v[j]);
     }
