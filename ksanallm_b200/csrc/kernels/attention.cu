@@ -49,6 +49,7 @@ enum KvMode { kKvCpAsync = 0, kKvFp8 = 1, kKvTma = 2 };
 typedef __nv_bfloat16 bf16;
 constexpr int kTileTok = 64;     // KV tokens per shared-memory tile
 constexpr int kAttnThreads = 128;
+constexpr int kBiasSmem = 2048;  // floats of bias rows that a decode CTA stages
 __host__ __device__ constexpr int kv_stages(int dp) { return dp <= 192 ? 3 : 2; }    // K/V tile ring: all but one tile in flight while one is consumed
 
 struct AttnParams {
@@ -65,6 +66,7 @@ struct AttnParams {
   const int* kv_lens;                    // [B]
   const float* alibi;                    // [Hq] slopes or null
   const float* bias; int bias_len;       // sigmoid weights: [Hq][bias_len] added by distance (the last entry holds beyond)
+  int bias_smem;                         // decode: the rows of a CTA's heads are staged in shared memory (floats; 0: not)
   const bf16* gate; long long gate_stride;   // optional, same layout as out
   float out_factor;                      // of gated outputs
   int Hq, Hkv;
@@ -317,7 +319,7 @@ __device__ __forceinline__ void sigmoid_weights(float (&s)[NT][4], const int (&l
       const int i = e >> 1;
       const int tok = tok0 + j * 8 + (lane & 3) * 2 + (e & 1);
       const bool seen = tok <= limit[i] && (tok >= lo[i] || tok < keep);
-      const float b = seen ? __ldg(bias[i] + min(limit[i] - tok, bias_last)) : 0.f;
+      const float b = seen ? bias[i][min(limit[i] - tok, bias_last)] : 0.f;
       s[j][e] = seen ? 1.f / (1.f + exp2f(-fmaf(s[j][e], scale_log2, b * 1.44269504f))) : 0.f;
     }
   }
@@ -512,6 +514,9 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
       v = *reinterpret_cast<const uint4*>(p.q + static_cast<size_t>(s) * p.q_stride + (head0 + r) * p.D + c * 8);
     *reinterpret_cast<uint4*>(tile_ptr<D, 16>(qs, r, c)) = v;
   }
+  float* bias_s = reinterpret_cast<float*>(ks + 2 * kKvStages * kTileTok * D);
+  if (SIG && p.bias_smem)
+    for (int i = threadIdx.x; i < G * p.bias_len; i += kAttnThreads) bias_s[i] = p.bias[static_cast<size_t>(head0) * p.bias_len + i];
   if (MODE == kKvTma && threadIdx.x == 0) {
     for (int i = 0; i < kKvStages; ++i) mbar_init(&full_bar[i], 1);
     abort_word = 0;
@@ -549,7 +554,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
     limit[i] = r < G ? kv_len - 1 : -1;
     lo[i] = win_lo;
     slope[i] = (p.alibi && r < G) ? p.alibi[head0 + r] : 0.f;
-    bias[i] = SIG ? p.bias + static_cast<size_t>(head0 + (r < G ? r : 0)) * p.bias_len : nullptr;
+    bias[i] = !SIG ? nullptr : (p.bias_smem ? bias_s : p.bias + static_cast<size_t>(head0) * p.bias_len) + (r < G ? r : 0) * p.bias_len;
   }
   float o[D / 8][4];
 #pragma unroll
@@ -713,11 +718,13 @@ static int launch_prefill(const AttnParams& p, const CUtensorMap& km, const CUte
 
 template <int D, int MODE, bool SIG = false>
 static int launch_decode(const AttnParams& p, const CUtensorMap& km, const CUtensorMap& vm, int B, cudaStream_t st) {
-  const int smem = (16 + 2 * kv_stages(D) * kTileTok) * D * 2 + 1024;   // the fp32 merge area fits inside the K and V rings
+  constexpr int ring = (16 + 2 * kv_stages(D) * kTileTok) * D * 2 + 1024;   // the fp32 merge area fits inside the K and V rings
+  const int smem = ring + (SIG ? p.bias_smem * 4 : 0);
   static_assert(4 * 16 * (D + 2) * 4 <= 2 * kv_stages(D) * kTileTok * D * 2, "merge area");
   static bool set = false;
   if (!set) {
-    if (cudaFuncSetAttribute(paged_decode_kernel<D, MODE, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) !=
+    if (cudaFuncSetAttribute(paged_decode_kernel<D, MODE, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             ring + (SIG ? kBiasSmem * 4 : 0)) !=
         cudaSuccess) return -3;
     set = true;
   }
@@ -830,6 +837,8 @@ extern "C" int ksana_paged_decode(const void* q, long long q_stride, void* out, 
   p.num_splits = num_splits; p.part_o = part_o; p.part_ml = part_ml; p.err = err;
   p.outq = static_cast<uint8_t*>(outq); p.oscale = oscale; p.oscale_ld = oscale_ld;
   p.bias = bias; p.bias_len = bias_len; p.gate = (const bf16*)gate; p.gate_stride = gate_stride; p.out_factor = out_factor;
+  const int table = bias ? (Hq / Hkv < 16 ? Hq / Hkv : 16) * bias_len : 0;
+  p.bias_smem = table <= kBiasSmem ? table : 0;
   switch (padded_head(D, Dv)) {
     case 64: return dispatch_decode<64>(p, cache_fp8, num_blocks, B, st);
     case 128: return dispatch_decode<128>(p, cache_fp8, num_blocks, B, st);

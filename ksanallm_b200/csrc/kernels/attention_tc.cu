@@ -48,7 +48,9 @@ struct FaParams {
   int D, Dv;                                 // real head sizes
   int window, keep;                          // sliding window in tokens (0: none), first tokens every row sees
   const float* bias; int bias_len;           // sigmoid weights: [Hq][bias_len] by distance (the last entry holds beyond)
-  int bias_ld;                               // floats between the heads' rows in shared memory; 0: read from global memory
+  // floats between the heads' rows in shared memory (there times -log2 e, with kFaTile entries in front for keys behind the
+  // row and kFaTile repetitions of the last entry behind, so that a tile's distances need no clamping); 0: read from global memory
+  int bias_ld;
   const bf16* gate; long long gate_stride; float out_factor;     // sigmoid weights: optional gate rows like out's, and a factor
   float scale_log2;
   int* err;
@@ -117,8 +119,10 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
   }
   if (warp == 1) { tmem_alloc(tmem_slot, kFaTmemCols); tmem_relinquish(); }
   if (SIG && p.bias_ld > 0)
-    for (int i = threadIdx.x; i < G * p.bias_len; i += kFaThreads)
-      bias_s[i / p.bias_len * p.bias_ld + i % p.bias_len] = p.bias[static_cast<size_t>(g) * G * p.bias_len + i];
+    for (int i = threadIdx.x; i < G * p.bias_ld; i += kFaThreads) {
+      const int at = min(max(i % p.bias_ld - kFaTile, 0), p.bias_len - 1);
+      bias_s[i] = -1.44269504f * p.bias[static_cast<size_t>(g * G + i / p.bias_ld) * p.bias_len + at];
+    }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -219,7 +223,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     const int keep = WIN ? p.keep : 0;
     auto sees = [&](int pos) { return pos <= limit && (!WIN || pos >= lo || pos < keep); };
     const float slope2 = (p.alibi && active) ? p.alibi[head] * 1.44269504f : 0.f;
-    const float* tab = !SIG ? nullptr : p.bias_ld > 0 ? bias_s + (vr % G) * p.bias_ld : p.bias + static_cast<size_t>(head) * p.bias_len;
+    const float* near = SIG ? bias_s + (vr % G) * p.bias_ld + kFaTile : nullptr;
+    const float* tab = SIG ? p.bias + static_cast<size_t>(head) * p.bias_len : nullptr;
     const int bias_last = SIG ? p.bias_len - 1 : 0;
     float m_used = -CUDART_INF_F, l = 0.f;
     bool ok = true;
@@ -258,28 +263,41 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
         for (int c = 0; c < 4; ++c) tmem_ld32(tmem_s + lane_off + c * 32, *reinterpret_cast<uint32_t(*)[32]>(&r[c * 32]));
         tmem_ld_wait();
         const int from = limit - t0;                       // distance of the tile's first key
-        auto weigh = [&](auto bias_at, auto hidden) {
+        // the row's visible keys as bits
+        uint32_t seen[4] = {~0u, ~0u, ~0u, ~0u};
+        const bool masked = __any_sync(0xffffffffu, need_mask);
+        if (masked) {
+          const int last = from, first = lo - t0, kept = keep - t0;
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            auto below = [&](int n) { return n - c * 32 >= 32 ? ~0u : n - c * 32 <= 0 ? 0u : (1u << (n - c * 32)) - 1u; };   // keys before n
+            seen[c] = below(last + 1);
+            if (WIN) seen[c] &= ~below(first) | below(kept);
+          }
+        }
+        auto weigh = [&](auto bias_at) {                   // -log2(e) times the bias of the tile's key i
 #pragma unroll
           for (int i = 0; i < 128; i += 2) {
             float w2[2];
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-              const float b = bias_at(i + e) * -1.44269504f;
-              const float v = fast_rcp(1.f + fast_exp2(fmaf(__uint_as_float(r[i + e]), -p.scale_log2, b)));
-              w2[e] = hidden(i + e) ? 0.f : v;
+              const float v = fast_rcp(1.f + fast_exp2(fmaf(__uint_as_float(r[i + e]), -p.scale_log2, bias_at(i + e))));
+              w2[e] = seen[(i + e) >> 5] >> ((i + e) & 31) & 1u ? v : 0.f;
             }
             __nv_bfloat162 pb = __floats2bfloat162_rn(w2[0], w2[1]);
             r[i >> 1] = *reinterpret_cast<uint32_t*>(&pb);
           }
         };
         const bool far = from - (kFaTile - 1) >= bias_last;      // every distance of the row has the last bias
-        if (__all_sync(0xffffffffu, far && !need_mask)) {
-          const float b = tab[bias_last];
-          weigh([&](int) { return b; }, [](int) { return false; });
+        if (__all_sync(0xffffffffu, far || !active)) {
+          const float b = tab[bias_last] * -1.44269504f;
+          weigh([&](int) { return b; });
+        } else if (p.bias_ld > 0) {
+          // (a row that is far, or that does not exist, in a warp that is not: any entry inside the table, then the last one)
+          const float* at = near + min(max(from, -1), bias_last + kFaTile - 1);
+          weigh([&](int i) { return at[-i]; });
         } else {
-          const int last = from, first = lo - t0, kept = keep - t0;
-          weigh([&](int i) { return tab[min(max(from - i, 0), bias_last)]; },
-                [&](int i) { return i > last || (WIN && i < first && i >= kept); });
+          weigh([&](int i) { return tab[min(max(from - i, 0), bias_last)] * -1.44269504f; });
         }
 #pragma unroll
         for (int c = 0; c < 4; ++c) tmem_st16(tmem_s + lane_off + c * 16, *reinterpret_cast<uint32_t(*)[16]>(&r[c * 16]));
@@ -493,8 +511,9 @@ extern "C" int ksana_paged_prefill_tc(const void* q, long long q_stride, long lo
   p.scale_log2 = scale * 1.44269504f;
   p.err = err;
   p.bias = bias; p.bias_len = bias_len; p.gate = static_cast<const bf16*>(gate); p.gate_stride = gate_stride; p.out_factor = out_factor;
-  const long long table = bias ? static_cast<long long>(G) * (bias_len | 1) * 4 : 0;       // odd row pitch: heads in different banks
-  p.bias_ld = table > 0 && table <= kFaBiasBytes ? bias_len | 1 : 0;
+  const int pitch = (bias_len + 2 * kFaTile) | 1;                                          // odd: heads in different banks
+  const long long table = bias ? static_cast<long long>(G) * pitch * 4 : 0;
+  p.bias_ld = table > 0 && table <= kFaBiasBytes ? pitch : 0;
   const int smem = kFaSmemBytes + (p.bias_ld ? static_cast<int>(table) : 0);
   dim3 grid((max_q_len * G + p.rows - 1) / p.rows, Hkv, B);
   auto* kernel = bias ? (window > 0 ? prefill_tc_kernel<true, true> : prefill_tc_kernel<false, true>)

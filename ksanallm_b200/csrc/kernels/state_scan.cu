@@ -49,7 +49,7 @@ __device__ __forceinline__ void conv_one(const ConvRef<T>& v, const T* row, cons
 // ------------------------------------------------------------------------------------------------ convolution
 // grid (channel tiles, row tiles, sequences); a thread walks the rows of its tile with 8 channels, the inputs before a row
 // in registers (TAPS 0: any number of taps, reloaded).
-constexpr int kConvRows = 16;
+constexpr int kConvRows = 32;
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128) causal_conv_kernel(const ConvRef<T> v, const StateRef r, T* out, long long ldo, const int* cu_q) {
   pdl_trigger();
