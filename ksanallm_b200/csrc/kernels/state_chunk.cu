@@ -15,6 +15,7 @@
 // Decays enter as products of factors <= 1 only, never as quotients, so no decay is too strong. Three groups of four warps prepare the
 // operands of the chunks in turn (unit vectors, decays, A and the inverse of I + A, Q) in a ring of four buffers; four warps apply
 // them, each to 16 or 32 columns, whose state never leaves their registers.
+#include "f32x2.cuh"
 #include "state_scan.cuh"
 
 namespace ksana {
@@ -42,6 +43,16 @@ __device__ __forceinline__ uint32_t pair(float a, float b) {
   return *reinterpret_cast<const uint32_t*>(&v);
 }
 __device__ __forceinline__ float2 unpair(uint32_t v) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v)); }
+__device__ __forceinline__ float exp2_fast(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float log2_fast(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 // a, b as the sum of two pairs of bf16
 __device__ __forceinline__ void pair_split(float a, float b, uint32_t& hi, uint32_t& lo) {
   hi = pair(a, b);
@@ -184,7 +195,7 @@ __global__ void __launch_bounds__(kSpaceThreads, 2) space_chunk_kernel(const Spa
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
             const int u = j * 8 + c2 + e;
-            v[e] = u <= t ? acc[j][2 * half + e] * __expf(gt - cum[u]) * dts[u] : 0.f;
+            v[e] = u <= t ? acc[j][2 * half + e] * exp2_fast((gt - cum[u]) * 1.44269504f) * dts[u] : 0.f;
             if (u == t) v[e] += D;
           }
           uint32_t hi, lo;
@@ -340,6 +351,7 @@ __device__ __forceinline__ void put_split(uint8_t* hi, uint8_t* lo, float v) {
   *reinterpret_cast<bf16*>(hi) = h;
   *reinterpret_cast<bf16*>(lo) = __float2bfloat16(v - __bfloat162float(h));
 }
+__device__ __forceinline__ F2 wide2(uint32_t v) { return f2(__uint_as_float(v << 16), __uint_as_float(v & 0xffff0000u)); }    // two bf16
 // accumulators of two 8-column tiles as a 16 x 16 operand
 __device__ __forceinline__ void operand_split(const float (&t0)[4], const float (&t1)[4], uint32_t (&hi)[4], uint32_t (&lo)[4]) {
   pair_split(t0[0], t0[1], hi[0], lo[0]);
@@ -397,9 +409,10 @@ __device__ __forceinline__ void delta_prepare(const DeltaParams<bf16>& p, uint8_
     float g[T], P = 1.f;
 #pragma unroll
     for (int t = 0; t < T; ++t) {
-      const float z = to_f(rz[t * KP + c]) + bias, soft = fmaxf(z, 0.f) + __logf(1.f + __expf(-fabsf(z)));
-      g[t] = t < m && c < p.K ? __expf(-A * soft) : 1.f;
-      gf[t * FP + c] = g[t];
+      // exp(-A softplus(z)) = 2^(-A log2(1 + e^z))
+      const float z = (to_f(rz[t * KP + c]) + bias) * 1.44269504f;
+      g[t] = t < m && c < p.K ? exp2_fast(-A * (z > 30.f ? z : log2_fast(1.f + exp2_fast(z)))) : 1.f;
+      gf[t * FP + ((c >> 2) & 1) * (KP / 2) + (c >> 3) * 4 + (c & 3)] = g[t];       // halves of the pieces of 8 apart
     }
 #pragma unroll
     for (int t = 0; t < T; ++t) {
@@ -418,52 +431,71 @@ __device__ __forceinline__ void delta_prepare(const DeltaParams<bf16>& p, uint8_
     }
   }
   bar_wait(bar, 128);
-  // A and Q by columns s, four per warp; a lane has four key channels, lengths enter at the end
-#pragma unroll 1
-  for (int i = 0; i < T / 4; ++i) {
-    const int s = i * 4 + (i & 1 ? 3 - warp : warp);
+  // A and Q by columns s, four per warp: eight lanes share a column, each with pieces of 8 key channels; lengths enter at the end.
+  // Columns with more rows go to another warp in every group
+  {
+    constexpr int PIECES = KP >= 64 ? KP / 64 : 1;
+    const int block = (warp + group) & 3, l = lane & 7, s = block * 4 + (lane >> 3);
     float v[2 * T];
-    float2 d0 = make_float2(0.f, 0.f), d1 = d0;
-    const bool on = lane * 4 < KP;
+    F2 d[PIECES][4];
+#pragma unroll
+    for (int i = 0; i < PIECES; ++i) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) d[i][e] = f2(0.f);
+    }
 #pragma unroll
     for (int t = 0; t < T; ++t) {
       v[t] = v[T + t] = 0.f;
-      if (t < s || !on) continue;
-      const uint2 kr = *reinterpret_cast<const uint2*>(rk + t * KP + lane * 4), qr = *reinterpret_cast<const uint2*>(rq + t * KP + lane * 4);
-      const float2 k0 = unpair(kr.x), k1 = unpair(kr.y), y0 = unpair(qr.x), y1 = unpair(qr.y);
-      if (t == s) {
-        d0 = k0;
-        d1 = k1;
-      } else {
-        const float4 g = *reinterpret_cast<const float4*>(gf + t * FP + lane * 4);
-        d0.x *= g.x; d0.y *= g.y; d1.x *= g.z; d1.y *= g.w;
-        v[t] = fmaf(d0.x, k0.x, fmaf(d0.y, k0.y, fmaf(d1.x, k1.x, d1.y * k1.y)));
+      if (t < block * 4) continue;
+      const F2 first = f2(t == s ? 1.f : 0.f);
+      F2 kk = f2(0.f), qk = f2(0.f);
+#pragma unroll
+      for (int i = 0; i < PIECES; ++i) {
+        const int piece = l + 8 * i;
+        if (KP < 64 && piece * 8 >= KP) break;
+        const uint4 kr = *reinterpret_cast<const uint4*>(rk + t * KP + piece * 8), qr = *reinterpret_cast<const uint4*>(rq + t * KP + piece * 8);
+        const ulonglong2 g0 = *reinterpret_cast<const ulonglong2*>(gf + t * FP + piece * 4),
+                         g1 = *reinterpret_cast<const ulonglong2*>(gf + t * FP + KP / 2 + piece * 4);
+        const uint32_t kw[4] = {kr.x, kr.y, kr.z, kr.w}, qw[4] = {qr.x, qr.y, qr.z, qr.w};
+        const unsigned long long gw[4] = {g0.x, g0.y, g1.x, g1.y};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const F2 k = wide2(kw[e]);
+          d[i][e] = fma2(k, first, d[i][e] * F2{gw[e]});
+          kk = fma2(d[i][e], k, kk);
+          qk = fma2(d[i][e], wide2(qw[e]), qk);
+        }
       }
-      v[T + t] = fmaf(d0.x, y0.x, fmaf(d0.y, y0.y, fmaf(d1.x, y1.x, d1.y * y1.y)));
+      v[t] = sum2(kk);
+      v[T + t] = sum2(qk);
     }
-    // sums over the lanes; lane l keeps entry l
+    // sums over the eight lanes; each keeps four entries
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
+    for (int o = 4; o > 0; o >>= 1) {
 #pragma unroll
-      for (int j = 0; j < o; ++j) {
-        const bool up = lane & o;
-        const float send = up ? v[j] : v[j + o], keep = up ? v[j + o] : v[j];
+      for (int j = 0; j < 4 * o; ++j) {
+        const bool up = l & o;
+        const float send = up ? v[j] : v[j + 4 * o], keep = up ? v[j + 4 * o] : v[j];
         v[j] = keep + __shfl_xor_sync(0xffffffffu, send, o);
       }
     }
-    const int t = lane & 15;
-    if (lane < T) am[t * (T + 4) + s] = t > s ? bt[t] * ik[t] * ik[s] * v[0] : 0.f;
-    else {
-      uint8_t* at = op + Sm::qk + t * kMPitch + s * 2;
-      put_split(at, at + T * kMPitch, t >= s ? iq[t] * ik[s] * v[0] : 0.f);
+    const float mine = ik[s];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int t = (l & 3) * 4 + j;
+      if (l < 4) am[t * (T + 4) + s] = t > s ? bt[t] * ik[t] * mine * v[j] : 0.f;
+      else {
+        uint8_t* at = op + Sm::qk + t * kMPitch + s * 2;
+        put_split(at, at + T * kMPitch, t >= s ? iq[t] * mine * v[j] : 0.f);
+      }
     }
   }
   bar_wait(bar, 128);
-  if (tid < T) {                                 // column tid of the inverse of I + A
+  if (warp == ((group + 1) & 3) && lane < T) {   // column `lane` of the inverse of I + A
     float x[T];
 #pragma unroll
     for (int t = 0; t < T; ++t) {
-      float a = t == tid ? 1.f : 0.f, b = 0.f;
+      float a = t == lane ? 1.f : 0.f, b = 0.f;
 #pragma unroll
       for (int s4 = 0; s4 < t; s4 += 4) {
         const float4 r = *reinterpret_cast<const float4*>(am + t * (T + 4) + s4);
@@ -473,7 +505,7 @@ __device__ __forceinline__ void delta_prepare(const DeltaParams<bf16>& p, uint8_
         if (s4 + 3 < t) b = fmaf(-r.w, x[s4 + 3], b);
       }
       x[t] = a + b;
-      uint8_t* at = op + Sm::inv + t * kMPitch + tid * 2;
+      uint8_t* at = op + Sm::inv + t * kMPitch + lane * 2;
       put_split(at, at + T * kMPitch, x[t]);
     }
   }

@@ -47,69 +47,85 @@ __device__ __forceinline__ void conv_one(const ConvRef<T>& v, const T* row, cons
 }
 
 // ------------------------------------------------------------------------------------------------ convolution
-// grid (channel tiles, row tiles, sequences); a thread walks the rows of its tile with 8 channels, the inputs before a row
+// 4 consecutive elements as floats
+__device__ __forceinline__ void load4(const bf16* p, float (&f)[4]) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+}
+__device__ __forceinline__ void load4(const float* p, float (&f)[4]) { *reinterpret_cast<float4*>(f) = *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ void store4(bf16* p, const float (&f)[4]) {
+  __nv_bfloat162 v[2] = {__floats2bfloat162_rn(f[0], f[1]), __floats2bfloat162_rn(f[2], f[3])};
+  *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(v);
+}
+__device__ __forceinline__ void store4(float* p, const float (&f)[4]) { *reinterpret_cast<float4*>(p) = *reinterpret_cast<const float4*>(f); }
+
+// grid (channel tiles, row tiles, sequences); a thread walks the rows of its tile with 4 channels, the inputs before a row
 // in registers (TAPS 0: any number of taps, reloaded).
-constexpr int kConvRows = 32;
+constexpr int kConvRows = 16, kConvAhead = 16;
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(128) causal_conv_kernel(const ConvRef<T> v, const StateRef r, T* out, long long ldo, const int* cu_q) {
+__global__ void __launch_bounds__(256) causal_conv_kernel(const ConvRef<T> v, const StateRef r, T* out, long long ldo, const int* cu_q) {
   pdl_trigger();
   pdl_wait();
-  const int s = blockIdx.z, c = (blockIdx.x * blockDim.x + threadIdx.x) * 8, row0 = blockIdx.y * kConvRows;
+  const int s = blockIdx.z, c = (blockIdx.x * blockDim.x + threadIdx.x) * 4, row0 = blockIdx.y * kConvRows;
   const int q0 = cu_q[s], n = cu_q[s + 1] - q0, past = r.kv_lens[s] - n;
   if (row0 >= n || c >= v.C) return;
   const int slot = slot_of(r, s);
   const T* ring = v.ring + static_cast<long long>(slot < 0 ? 0 : slot) * v.slot_stride + c;
   const T* x = v.x + static_cast<long long>(q0) * v.ld + c;
-  auto input = [&](int t, float (&f)[8]) {             // of the row t (negative: from the ring, zero before the sequence)
-    if (t >= 0) load8(x + t * v.ld, f);
-    else if (past + t >= 0 && slot >= 0) load8(ring + static_cast<size_t>((past + t) % v.taps) * v.C, f);
-    else {
-#pragma unroll
-      for (int e = 0; e < 8; ++e) f[e] = 0.f;
-    }
+  auto input = [&](int t, float (&f)[4]) {             // of the row t (negative: from the ring, zero before the sequence)
+    if (t >= 0) load4(x + t * v.ld, f);
+    else if (past + t >= 0 && slot >= 0) load4(ring + static_cast<size_t>((past + t) % v.taps) * v.C, f);
+    else f[0] = f[1] = f[2] = f[3] = 0.f;
   };
-  float b[8] = {};
-  if (v.bias) load8(v.bias + c, b);
-  constexpr int H = TAPS > 1 ? TAPS - 1 : 1;
-  float w[TAPS > 0 ? TAPS : 1][8], hist[H][8];
-  if constexpr (TAPS > 0) {
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) load8(v.w + static_cast<size_t>(j) * v.C + c, w[j]);
-#pragma unroll
-    for (int j = 0; j < TAPS - 1; ++j) input(row0 - (TAPS - 1) + j, hist[j]);
-  }
+  float b[4] = {};
+  if (v.bias) load4(v.bias + c, b);
+  T* dst = out + static_cast<long long>(q0 + row0) * ldo + c;
   const int end = min(row0 + kConvRows, n);
-#pragma unroll 4
-  for (int t = row0; t < end; ++t) {
-    float acc[8], f[8];
+  auto finish = [&](float (&acc)[4]) {
 #pragma unroll
-    for (int e = 0; e < 8; ++e) acc[e] = b[e];
-    if constexpr (TAPS > 0) {
-      load8(x + t * v.ld, f);
+    for (int e = 0; e < 4; ++e) acc[e] *= sigmoid_as<T>(acc[e]);
+    store4(dst, acc);
+    dst += ldo;
+  };
+  if constexpr (TAPS > 0) {
+    float w[TAPS][4], hist[TAPS][4];                     // hist: the last TAPS inputs, the row's own last
 #pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j) {
+    for (int j = 0; j < TAPS; ++j) load4(v.w + static_cast<size_t>(j) * v.C + c, w[j]);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) acc[e] = fmaf(hist[j][e], w[j][e], acc[e]);
-      }
+    for (int j = 1; j < TAPS; ++j) input(row0 - TAPS + j, hist[j]);
+    for (int t = row0; t < end; t += kConvAhead) {
+      float f[kConvAhead][4];                            // all loads of some rows before their stores
 #pragma unroll
-      for (int e = 0; e < 8; ++e) acc[e] = fmaf(f[e], w[TAPS - 1][e], acc[e]);
+      for (int u = 0; u < kConvAhead; ++u) load4(x + min(t + u, n - 1) * v.ld, f[u]);
 #pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j) {
+      for (int u = 0; u < kConvAhead; ++u) {
+        if (t + u >= end) break;
+        float acc[4];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) hist[j][e] = j + 1 < TAPS - 1 ? hist[j + 1 < H ? j + 1 : 0][e] : f[e];
-      }
-    } else {
-      for (int j = 0; j < v.taps; ++j) {
-        float wj[8];
-        input(t - (v.taps - 1) + j, f);
-        load8(v.w + static_cast<size_t>(j) * v.C + c, wj);
+        for (int e = 0; e < 4; ++e) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) acc[e] = fmaf(f[e], wj[e], acc[e]);
+          for (int j = 0; j + 1 < TAPS; ++j) hist[j][e] = hist[j + 1][e];
+          hist[TAPS - 1][e] = f[u][e];
+          acc[e] = b[e];
+#pragma unroll
+          for (int j = 0; j < TAPS; ++j) acc[e] = fmaf(hist[j][e], w[j][e], acc[e]);
+        }
+        finish(acc);
       }
     }
+  } else {
+    for (int t = row0; t < end; ++t) {
+      float acc[4] = {b[0], b[1], b[2], b[3]};
+      for (int j = 0; j < v.taps; ++j) {
+        float f[4], w[4];
+        input(t - (v.taps - 1) + j, f);
+        load4(v.w + static_cast<size_t>(j) * v.C + c, w);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) acc[e] *= sigmoid_as<T>(acc[e]);
-    store8(out + static_cast<long long>(q0 + t) * ldo + c, acc);
+        for (int e = 0; e < 4; ++e) acc[e] = fmaf(f[e], w[e], acc[e]);
+      }
+      finish(acc);
+    }
   }
 }
 
@@ -518,7 +534,7 @@ static int step_threads(int cols) { return (cols < 64 ? (cols + 7) / 8 * 8 : 64)
 
 template <typename T>
 static int launch_conv(const ConvRef<T>& v, const StateRef& r, T* out, long long ldo, const int* cu_q, int B, int max_q, cudaStream_t st) {
-  const int vec = v.C / 8, threads = vec < 128 ? (vec + 31) / 32 * 32 : 128;
+  const int vec = v.C / 4, threads = vec < 256 ? (vec + 31) / 32 * 32 : 256;
   const dim3 grid((vec + threads - 1) / threads, (max_q + kConvRows - 1) / kConvRows, B);
   switch (v.taps) {
     case 1: return launched(launch_pdl(causal_conv_kernel<T, 1>, grid, dim3(threads), 0, st, v, r, out, ldo, cu_q));
