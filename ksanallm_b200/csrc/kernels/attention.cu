@@ -52,6 +52,12 @@ constexpr int kAttnThreads = 128;
 constexpr int kBiasSmem = 2048;  // floats of bias rows that a decode CTA stages
 __host__ __device__ constexpr int kv_stages(int dp) { return dp <= 192 ? 3 : 2; }    // K/V tile ring: all but one tile in flight while one is consumed
 
+// elements of a decode CTA's K and V rings (one ring where they are the same); the fp32 merge area lies over them
+__host__ __device__ constexpr int decode_ring(int dp, bool shared) {
+  const int rings = (shared ? 1 : 2) * kv_stages(dp) * kTileTok * dp, merge = 4 * 16 * (dp + 2) * 2;
+  return rings > merge ? rings : merge;
+}
+
 struct AttnParams {
   const bf16* q; long long q_stride;     // [T, q_stride] ; head h at column h*D
   bf16* out; long long out_stride;       // [T, out_stride]
@@ -182,8 +188,8 @@ __device__ __forceinline__ void load_kv_tile(bf16* dst, const AttnParams& p, con
   }
 }
 
-// TMA staging of one K + V tile (one thread; `shared`: the keys are the values, one tile): a box of [block_tokens rows x 64 columns] per cache block and
-// 64-column panel. Tokens past kv_len inside the last block are loaded as they are (finite cache contents)
+// TMA staging of one K + V tile (one thread; `shared`: the keys are the values, one tile): a box of [block_tokens rows x 64
+// columns] per cache block and 64-column panel. Tokens past kv_len inside the last block are loaded as they are (finite cache contents)
 // and masked by the softmax; blocks past the sequence are not loaded at all.
 template <int D>
 __device__ __forceinline__ void tma_issue_kv(bf16* ks, bf16* vs, bool shared, uint64_t* bar, const CUtensorMap* kmap, const CUtensorMap* vmap,
@@ -514,7 +520,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
       v = *reinterpret_cast<const uint4*>(p.q + static_cast<size_t>(s) * p.q_stride + (head0 + r) * p.D + c * 8);
     *reinterpret_cast<uint4*>(tile_ptr<D, 16>(qs, r, c)) = v;
   }
-  float* bias_s = reinterpret_cast<float*>(ks + 2 * kKvStages * kTileTok * D);
+  float* bias_s = reinterpret_cast<float*>(ks + decode_ring(D, shared));
   if (SIG && p.bias_smem)
     for (int i = threadIdx.x; i < G * p.bias_len; i += kAttnThreads) bias_s[i] = p.bias[static_cast<size_t>(head0) * p.bias_len + i];
   if (MODE == kKvTma && threadIdx.x == 0) {
@@ -716,15 +722,13 @@ static int launch_prefill(const AttnParams& p, const CUtensorMap& km, const CUte
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
-template <int D, int MODE, bool SIG = false>
+template <int D, int MODE, bool SIG>
 static int launch_decode(const AttnParams& p, const CUtensorMap& km, const CUtensorMap& vm, int B, cudaStream_t st) {
-  constexpr int ring = (16 + 2 * kv_stages(D) * kTileTok) * D * 2 + 1024;   // the fp32 merge area fits inside the K and V rings
-  const int smem = ring + (SIG ? p.bias_smem * 4 : 0);
-  static_assert(4 * 16 * (D + 2) * 4 <= 2 * kv_stages(D) * kTileTok * D * 2, "merge area");
+  constexpr int most = (16 * D + decode_ring(D, false)) * 2 + 1024 + (SIG ? kBiasSmem * 4 : 0);
+  const int smem = (16 * D + decode_ring(D, p.kc == p.vc)) * 2 + 1024 + (SIG ? p.bias_smem * 4 : 0);
   static bool set = false;
   if (!set) {
-    if (cudaFuncSetAttribute(paged_decode_kernel<D, MODE, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                             ring + (SIG ? kBiasSmem * 4 : 0)) !=
+    if (cudaFuncSetAttribute(paged_decode_kernel<D, MODE, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, most) !=
         cudaSuccess) return -3;
     set = true;
   }
@@ -763,12 +767,12 @@ static int dispatch_decode(const AttnParams& p, int cache_fp8, int num_blocks, i
     return launch_decode<D, kKvCpAsync, true>(p, km, vm, B, st);
   }
   if constexpr (D <= 128) {
-    if (cache_fp8) return launch_decode<D, kKvFp8>(p, km, vm, B, st);
+    if (cache_fp8) return launch_decode<D, kKvFp8, false>(p, km, vm, B, st);
   } else if (cache_fp8) {
     return -11;
   }
-  if (tma_maps(p, num_blocks, &km, &vm)) return launch_decode<D, kKvTma>(p, km, vm, B, st);
-  return launch_decode<D, kKvCpAsync>(p, km, vm, B, st);
+  if (tma_maps(p, num_blocks, &km, &vm)) return launch_decode<D, kKvTma, false>(p, km, vm, B, st);
+  return launch_decode<D, kKvCpAsync, false>(p, km, vm, B, st);
 }
 
 // The padded head size that serves (D, Dv), 0 when none does.

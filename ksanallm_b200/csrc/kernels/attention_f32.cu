@@ -176,13 +176,14 @@ static int launch_attention_f32(const void* q, long long q_stride, void* out, lo
 
 using namespace ksana;
 
-// window 0: full causal attention. bias: sigmoid weights. D and Dv multiples of 8, at most 1024. ldv: elements between value rows. f32: q, out and
-// the panels are fp32 instead of bf16.
+// window 0: full causal attention. bias: sigmoid weights. D and Dv multiples of 8, at most 1024. ldv: elements between value
+// rows. f32: q, out and the panels are fp32 instead of bf16.
 extern "C" int ksana_attention_f32(const void* q, long long q_stride, void* out, long long out_stride, const void* kc,
                                    const void* vc, int ldv, long long block_stride, int block_tokens, int num_blocks,
                                    const int* block_table, int table_stride, const int* cu_q, const int* kv_lens,
                                    const float* sinks, const void* gate, long long gate_ld, int gate_wide, float out_factor,
-                                   const float* bias, int bias_len, int B, int max_q_len, int Hq, int Hkv, int D, int Dv, int window, int keep, float scale, int f32, int* err, cudaStream_t st) {
+                                   const float* bias, int bias_len, int B, int max_q_len, int Hq, int Hkv, int D, int Dv, int window,
+                                   int keep, float scale, int f32, int* err, cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0) return 0;
   if (bias && bias_len <= 0) return -14;
   if (Hkv <= 0 || Hq % Hkv || D <= 0 || Dv <= 0 || D > kAfMaxWide || Dv > kAfMaxWide || D % 8 || Dv % 8 || ldv < Dv || Hq > 65535 ||

@@ -327,7 +327,8 @@ template <int NK, int CT> struct DeltaSmem {
                        v = qk + 2 * kDeltaTokens * kMPitch, beta = v + kDeltaTokens * vpitch, total = beta + kDeltaTokens * 4,
                        operands = total + KP * 4;
   // what a preparing group works on: raw rows (q, k, decay), decays, A, reciprocal lengths
-  static constexpr int raw = 3 * kDeltaTokens * KP * 2, work = raw + (kDeltaTokens * fpitch + kDeltaTokens * (kDeltaTokens + 4) + 2 * kDeltaTokens) * 4;
+  static constexpr int raw = 3 * kDeltaTokens * KP * 2,
+                       work = raw + (kDeltaTokens * fpitch + kDeltaTokens * (kDeltaTokens + 4) + 2 * kDeltaTokens) * 4;
   static constexpr int out = kDeltaBuffers * operands + kDeltaGroups * work, bytes = out + kDeltaTokens * vpitch;
 };
 

@@ -14,9 +14,9 @@
 //                   and beta = sigmoid(projection)
 //
 // Both recurrences have a scan (several tokens per sequence, convolved inputs; in bf16 the tensor-core form of state_chunk.cu
-// takes most sizes) and a step (one token per sequence, the convolution is part of it). Every column of a state is independent of the others: a CTA takes a slab of columns of one
-// head, eight neighbouring lanes share a column and split its keys. Head and key sizes are multiples of 8 (padded with
-// zeros). At position 0 the state is zero whatever the slot holds.
+// takes most sizes) and a step (one token per sequence, the convolution is part of it). Every column of a state is independent of
+// the others: a CTA takes a slab of columns of one head, eight neighbouring lanes share a column and split its keys. Head and key
+// sizes are multiples of 8 (padded with zeros). At position 0 the state is zero whatever the slot holds.
 #include "f32x2.cuh"
 #include "state_scan.cuh"
 
@@ -50,7 +50,8 @@ __device__ __forceinline__ void conv_one(const ConvRef<T>& v, const T* row, cons
 // 4 consecutive elements as floats
 __device__ __forceinline__ void load4(const bf16* p, float (&f)[4]) {
   const uint2 v = *reinterpret_cast<const uint2*>(p);
-  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
   f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
 }
 __device__ __forceinline__ void load4(const float* p, float (&f)[4]) { *reinterpret_cast<float4*>(f) = *reinterpret_cast<const float4*>(p); }

@@ -69,7 +69,8 @@ struct SpaceParams {
 // Channels of the ring that the CTA of (head, slab of columns [p0, p0 + np)) stores: its own x, and B and C of the head's group
 // where it is the group's first.
 template <typename T>
-__device__ __forceinline__ void space_ring(const SpaceParams<T>& p, const T* rows, int slot, int past, int n, int h, int p0, int np, int tid, int threads) {
+__device__ __forceinline__ void space_ring(const SpaceParams<T>& p, const T* rows, int slot, int past, int n, int h, int p0, int np, int tid,
+                                           int threads) {
   T* ring = p.conv.ring + static_cast<long long>(slot) * p.conv.slot_stride;
   ring_store(p.conv, rows, ring, past, n, h * p.P + p0, np, tid, threads);
   const int per = p.H / p.G, g = h / per;
@@ -95,7 +96,8 @@ struct DeltaParams {
 };
 
 template <typename T>
-__device__ __forceinline__ void delta_ring(const DeltaParams<T>& p, const T* rows, int slot, int past, int n, int h, int p0, int np, int tid, int threads) {
+__device__ __forceinline__ void delta_ring(const DeltaParams<T>& p, const T* rows, int slot, int past, int n, int h, int p0, int np, int tid,
+                                           int threads) {
   T* ring = p.conv.ring + static_cast<long long>(slot) * p.conv.slot_stride;
   ring_store(p.conv, rows, ring, past, n, 2 * p.G * p.K + h * p.V + p0, np, tid, threads);
   const int per = p.H / p.G, g = h / per;

@@ -275,7 +275,9 @@ extern "C" int ksana_token_shift(const void* h, long long ldh, const void* mu, v
                                  const int* cu_q, const int* kv_lens, const int* slots, int num_slots, int B, int max_q, int W, int f32,
                                  int* err, cudaStream_t st) {
   if (B <= 0 || max_q <= 0) return 0;
-  if (W <= 0 || W % 8 || ldh % 8 || ldo % 8 || slot_stride % (f32 ? 4 : 8) || B > 65535 || !aligned16(h) || !aligned16(out) || !aligned16(ring)) return -10;
+  if (W <= 0 || W % 8 || ldh % 8 || ldo % 8 || slot_stride % (f32 ? 4 : 8) || B > 65535 || !aligned16(h) || !aligned16(out) ||
+      !aligned16(ring))
+    return -10;
   const int vec = W / 8, threads = vec < 256 ? (vec + 31) / 32 * 32 : 256;
   const dim3 grid((vec + threads - 1) / threads, (max_q + kShiftRows - 1) / kShiftRows, B);
   const cudaError_t e = f32 ? launch_pdl(token_shift_kernel<float>, grid, dim3(threads), 0, st, static_cast<const float*>(h), ldh,

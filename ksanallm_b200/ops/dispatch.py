@@ -565,7 +565,8 @@ def panel_attention(qkv, k_cache, v_cache, block_tokens, step, Hq, Hkv, scale, w
                              sinks=sinks, weights=weights)
     if ns:
         seen = min(step.max_kv_len, window + keep + 128) if window > 0 else step.max_kv_len
-        n = decode_splits(ns, Hkv * ((Hq // Hkv + 15) // 16), seen)
+        # keys that are the values take half of the shared memory
+        n = decode_splits(ns, Hkv * ((Hq // Hkv + 15) // 16), seen, ctas_per_sm=4 if k_cache.data_ptr() == v_cache.data_ptr() else 2)
         po = pml = None
         if n > 1:
             po = torch.empty(ns * Hq * n * Dv, dtype=torch.float32, device=qkv.device)

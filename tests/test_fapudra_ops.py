@@ -120,10 +120,10 @@ def padded_channels(parts):
     return torch.cat(out, -1)
 
 
-def space_case(H, P, N, G, taps, T, seed=0):
+def space_case(H, P, N, G, taps, T, seed=0, shift=0.0):
     x, B, C = rand(seed, T, H * P), rand(seed + 1, T, G * N), rand(seed + 2, T, G * N)
     dt, w, b = rand(seed + 3, T, H), rand(seed + 4, H * P + 2 * G * N, taps), rand(seed + 5, H * P + 2 * G * N) * 0.3
-    A_log, D, dt_bias = rand(seed + 6, H) - 1, rand(seed + 7, H), rand(seed + 8, H) - 3          # decays from slow to moderate
+    A_log, D, dt_bias = rand(seed + 6, H) - 1, rand(seed + 7, H), rand(seed + 8, H) - 3 + shift          # decays from slow to moderate
     c = oracle.silu(oracle.causal_conv(torch.cat([x, B, C], 1).double(), w.double(), b.double()))
     cx, cB, cC = c.split([H * P, G * N, G * N], 1)
     step = oracle.softplus(dt.double() + dt_bias.double())
@@ -135,7 +135,8 @@ def space_case(H, P, N, G, taps, T, seed=0):
                            b=padded_channels([(t, n) for t, n in zip(b.split([H * P, G * N, G * N]), (H, G, G))]))
 
 
-SPACES = [(1, 1, 1, 1, 1), (6, 16, 24, 2, 3), (3, 10, 13, 3, 2), (4, 24, 16, 4, 4), (8, 64, 128, 2, 4), (2, 72, 136, 2, 6), (5, 40, 64, 1, 3), (2, 33, 256, 1, 4)]
+SPACES = [(1, 1, 1, 1, 1), (6, 16, 24, 2, 3), (3, 10, 13, 3, 2), (4, 24, 16, 4, 4), (8, 64, 128, 2, 4), (2, 72, 136, 2, 6), (5, 40, 64, 1, 3),
+          (2, 33, 256, 1, 4), (2, 136, 48, 1, 4)]
 # bf16 rounds the convolved inputs; everything behind them is 32-bit
 LOOSE = {torch.float32: 1.0, torch.bfloat16: 2.0}
 
@@ -164,10 +165,10 @@ def test_state_space(device, dtype, H, P, N, G, taps):
     fault_free(device)
 
 
-def delta_case(H, G, K, V, taps, T, seed=0):
+def delta_case(H, G, K, V, taps, T, seed=0, shift=0.0):
     q, kk, v = rand(seed, T, G * K), rand(seed + 1, T, G * K), rand(seed + 2, T, H * V)
     w = rand(seed + 3, 2 * G * K + H * V, taps)
-    beta, decay, bias, A_log = rand(seed + 4, T, H), rand(seed + 5, T, H * K), rand(seed + 6, H * K) - 4, rand(seed + 7, H) - 1
+    beta, decay, bias, A_log = rand(seed + 4, T, H), rand(seed + 5, T, H * K), rand(seed + 6, H * K) - 4 + shift, rand(seed + 7, H) - 1
     c = oracle.silu(oracle.causal_conv(torch.cat([q, kk, v], 1).double(), w.double()))
     cq, ck, cv = c.split([G * K, G * K, H * V], 1)
     cq, ck = oracle.unit(cq.view(T, G, K)) * K ** -0.5, oracle.unit(ck.view(T, G, K))
@@ -181,8 +182,9 @@ def delta_case(H, G, K, V, taps, T, seed=0):
                            w=padded_channels([(t, n) for t, n in zip(w.t().split(parts, 1), (G, G, H))]))
 
 
-DELTAS = [(1, 1, 2, 1, 1), (4, 2, 16, 24, 4), (3, 3, 10, 6, 3), (2, 2, 24, 8, 2), (4, 2, 64, 64, 4), (2, 1, 128, 128, 3), (2, 1, 136, 40, 6), (6, 2, 40, 136, 4),
-          (1, 1, 256, 72, 4)]
+# the last ones: more columns of states than one wave of 64 each
+DELTAS = [(1, 1, 2, 1, 1), (4, 2, 16, 24, 4), (3, 3, 10, 6, 3), (2, 2, 24, 8, 2), (4, 2, 64, 64, 4), (2, 1, 128, 128, 3), (2, 1, 136, 40, 6),
+          (6, 2, 40, 136, 4), (1, 1, 256, 72, 4), (80, 2, 128, 72, 4), (80, 4, 24, 128, 3)]
 
 
 @pytest.mark.parametrize("device,dtype", PLACES)
@@ -207,6 +209,29 @@ def test_delta_rule(device, dtype, H, G, K, V, taps):
         if sizes == [61]:
             whole = S[slot % 3].clone()
     close(S[(len(PORTIONS)) % 3], whole.cpu(), dtype)
+    fault_free(device)
+
+
+@pytest.mark.parametrize("device,dtype", PLACES)
+@pytest.mark.parametrize("shift", [0.0, 8.0, 60.0])
+def test_long_prompts_and_strong_decays(device, dtype, shift):
+    """Many chunks in one portion, and decays down to nothing within a token (cumulated over a chunk they are beyond fp32's range)."""
+    T = 300 if device == "cuda" else 90
+    k = space_case(2, 64, 128, 1, 4, T, 7, shift)
+    put = lambda t: t.to(device, dtype).contiguous()  # noqa: E731
+    C = k.raw.shape[1]
+    ring, S, _ = state_record(4, C, (2, 64, 128), dtype, device)
+    rows = put(torch.cat([k.raw, k.dt], 1))
+    got = [ops.state_space(rows[a:b, :C], ops.ShortConv(put(k.w), put(k.b), ring), rows[a:b, C:], k.dt_bias.to(device), k.A.to(device),
+                           k.D.to(device), S, 1, step_of([(a, b - a, 1)], None, device)).float().cpu() for a, b in ((0, T - 70), (T - 70, T))]
+    close(torch.cat(got), k.want, dtype, LOOSE[dtype] * max(1.0, float(k.want.abs().max())))
+    k = delta_case(2, 1, 128, 128, 4, T, 9, shift)
+    C = k.raw.shape[1]
+    ring, S, _ = state_record(4, C, (2, 128, 128), dtype, device)
+    rows, decay = put(torch.cat([k.raw, k.beta], 1)), put(k.decay)
+    got = [ops.delta_rule(rows[a:b, :C], ops.ShortConv(put(k.w), None, ring), rows[a:b, C:], decay[a:b], k.bias.to(device), k.A.to(device), S, 1,
+                          128 ** -0.5, step_of([(a, b - a, 1)], None, device)).float().cpu() for a, b in ((0, T - 70), (T - 70, T))]
+    close(torch.cat(got), k.want, dtype, LOOSE[dtype] * max(1.0, float(k.want.abs().max())))
     fault_free(device)
 
 
