@@ -18,7 +18,8 @@ def enabled() -> bool:
     return os.environ.get("KSANA_CHECK_INPUTS", "0") not in ("", "0", "false", "False")
 
 
-def step_violations(step, num_blocks: int, block_tokens: int, vocab_size: int, max_positions: int) -> List[str]:
+def step_violations(step, num_blocks: int, block_tokens: int, vocab_size: int, max_positions: int,
+                    num_state_slots: int = 0) -> List[str]:
     """All violations found in a StepInput (empty list = consistent)."""
     bad: List[str] = []
     T = int(step.input_ids.shape[0])
@@ -74,6 +75,12 @@ def step_violations(step, num_blocks: int, block_tokens: int, vocab_size: int, m
             if sl != int(table[s, p // block_tokens]) * block_tokens + p % block_tokens:
                 bad.append(f"sequence {s}: row {r} writes slot {sl}, its block table says otherwise")
                 break
+    if getattr(step, "state_slots", None) is not None:
+        held = step.state_slots.long().cpu()
+        if held.numel() != nseq or (nseq and (int(held.min()) < 0 or int(held.max()) >= num_state_slots)):
+            bad.append(f"not one state slot in [0, {num_state_slots}) per sequence")
+        elif held.unique().numel() != held.numel():
+            bad.append("two sequences hold the same state slot")
     if step.logits_rows is not None and step.logits_rows.numel():
         lr = step.logits_rows.long().cpu()
         if int(lr.min()) < 0 or int(lr.max()) >= T:
@@ -88,6 +95,7 @@ def step_violations(step, num_blocks: int, block_tokens: int, vocab_size: int, m
 def check_step(step, model) -> None:
     cache = model.kv_cache
     bad = step_violations(step, int(cache.shape[0]), model.block_tokens, model.cfg.vocab_size,
-                          int(model.cos_sin.shape[0]) if model.cos_sin is not None else 1 << 30)
+                          int(model.cos_sin.shape[0]) if model.cos_sin is not None else 1 << 30,
+                          int(model.state.shape[0]) if getattr(model, "state", None) is not None else 0)
     if bad:
         raise RuntimeError("inconsistent step metadata: " + "; ".join(bad))

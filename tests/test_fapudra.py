@@ -304,6 +304,25 @@ def test_positions_end_with_the_table():
     assert eng.add_request(t + t, greedy(1)).status_code != 0
 
 
+def test_checked_steps(monkeypatch):
+    """The engine's own bounds checks cover the state slots."""
+    from ksanallm_b200.ops import checks
+    monkeypatch.setenv("KSANA_CHECK_INPUTS", "1")
+    eng = engine("plain", "cpu", torch.float32, max_batch_size=2)
+    t, want = truth("plain", 150)
+    check(hlp.run_portions(eng, t[:40], [9, 1, 30]), want[:40], torch.float32, "cpu")
+    seen = []
+    monkeypatch.setattr(checks, "check_step", lambda step, model: seen.append(step))
+    a, b = eng.open_given(), eng.open_given()
+    eng.step_given([(a, t[:5], []), (b, t[:3], [])])
+    args = (eng.model.kv_cache.shape[0], eng.model.block_tokens, 96, 512, 2)
+    (step,) = seen
+    assert checks.step_violations(step, *args) == []
+    for slots in ([0, 0], [0, 2], [-1, 0], [0]):
+        step.state_slots = torch.tensor(slots, dtype=torch.int32)
+        assert any("state slot" in m for m in checks.step_violations(step, *args))
+
+
 def test_more_requests_than_slots_wait():
     """A given sequence beyond the state slots is refused until another one ends; generation queues."""
     eng = engine("plain", "cpu", torch.float32, max_batch_size=2)
