@@ -265,7 +265,7 @@ __global__ void space_step_kernel(const SpaceParams<T> p) {
   pdl_trigger();
   pdl_wait();
   constexpr int KP = J * kLanes * 4;
-  __shared__ __align__(16) float Bs[KP], Cs[KP], xs[64];
+  __shared__ __align__(16) float Bs[KP], Cs[KP], xs[32];
   __shared__ float step, decay;
   const int slab = blockDim.x / kLanes, s = blockIdx.z, h = blockIdx.y, p0 = blockIdx.x * slab, np = min(slab, p.P - p0);
   const int slot = slot_of(p.ref, s), pos = p.ref.kv_lens[s] - 1;
@@ -448,7 +448,7 @@ __global__ void delta_step_kernel(const DeltaParams<T> p) {
   pdl_trigger();
   pdl_wait();
   constexpr int KP = J * kLanes * 4;
-  __shared__ __align__(16) float qs[KP], ks[KP], gs[KP], vs[64];
+  __shared__ __align__(16) float qs[KP], ks[KP], gs[KP], vs[32];
   const int slab = blockDim.x / kLanes, s = blockIdx.z, h = blockIdx.y, p0 = blockIdx.x * slab, np = min(slab, p.V - p0);
   const int slot = slot_of(p.ref, s), pos = p.ref.kv_lens[s] - 1;
   const int lane = threadIdx.x & (kLanes - 1), col = threadIdx.x / kLanes, g = h / (p.H / p.G);
@@ -531,7 +531,7 @@ __global__ void delta_step_kernel(const DeltaParams<T> p) {
 // ------------------------------------------------------------------------------------------------ host
 static int launched(cudaError_t e) { return e == cudaSuccess ? 0 : -4; }
 static int column_vectors(int keys) { const int j = (keys + 31) / 32; return j <= 1 ? 1 : j <= 2 ? 2 : j <= 4 ? 4 : j <= 8 ? 8 : 0; }
-static int step_threads(int cols) { return (cols < 64 ? (cols + 7) / 8 * 8 : 64) * kLanes; }
+static int step_threads(int cols) { return (cols < 32 ? (cols + 7) / 8 * 8 : 32) * kLanes; }
 
 template <typename T>
 static int launch_conv(const ConvRef<T>& v, const StateRef& r, T* out, long long ldo, const int* cu_q, int B, int max_q, cudaStream_t st) {
