@@ -11,7 +11,7 @@ def space(heads, vdim, state, groups, conv, norm_groups):
     return "mamba2", {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "conv": conv, "norm_groups": norm_groups}
 
 
-def both(left, mask, right, scales=(1.2, 0.8), bias_max=40, scale=None):
+def both(left, mask, right, scales=(1.25, 0.8), bias_max=40, scale=None):
     """left: heads, kv_heads, dim; right: heads, kv_heads, dim, vdim, conv."""
     H, G, d = left
     names = ("heads", "kv_heads", "dim", "vdim", "conv")
@@ -20,12 +20,12 @@ def both(left, mask, right, scales=(1.2, 0.8), bias_max=40, scale=None):
                         "right": dict(zip(names, right)), "left_scale": scales[0], "right_scale": scales[1]}
 
 
-def moe(experts, top, groups, ff, limit=1.5):
+def moe(experts, top, groups, ff, limit=1.3):
     return {"kind": "moe", "router": {"experts": experts, "top": top, "groups": dict(zip(("count", "keep"), groups)) if groups else None},
             "expert": {"ff": ff, "limit": limit}}
 
 
-def config(width, vocab, layers, cap=30.0, scale=3.0, eps=1e-5, max_positions=512):
+def config(width, vocab, layers, cap=24.0, scale=3.0, eps=1e-5, max_positions=512):
     return {"architecture": "Fapudra", "width": width, "vocab": vocab, "max_positions": max_positions, "norm": {"eps": eps},
             "embedding": {"scale": scale}, "logit_softcap": cap,
             "layers": [{"type": t, "mixer": m, "mlp": ff} for (t, m), ff in layers]}
@@ -33,7 +33,7 @@ def config(width, vocab, layers, cap=30.0, scale=3.0, eps=1e-5, max_positions=51
 
 CONFIGS = {
     # both mixers with and without experts, groups of heads, a norm of several parts, unequal key and value sizes
-    "unequal": config(72, 203, [(space(6, 16, 24, 2, 3, 3), moe(12, 3, (3, 2), 24)), (both((6, 2, 24), (20, 5), (4, 2, 16, 24, 4)), None),
+    "unequal": config(72, 203, [(space(6, 16, 24, 2, 3, 3), moe(15, 4, (5, 3), 24)), (both((6, 2, 24), (20, 5), (4, 2, 16, 24, 4)), None),
                                 (space(4, 24, 16, 4, 4, 1), None), (both((4, 4, 16), (33, 0), (2, 2, 24, 8, 2), (0.7, 1.4), 25), moe(10, 2, None, 16, 0.8))]),
     # nothing is a multiple of 8, norm parts that cross heads
     "odd": config(70, 101, [(both((3, 1, 10), (17, 3), (3, 3, 10, 6, 3), (0.5, 2.0), 23, 0.4), moe(9, 2, (3, 1), 13, 1.1)),

@@ -92,7 +92,7 @@ def test_gated_norm(device, dtype, heads, real, parts):
 
 
 @pytest.mark.parametrize("device", ["cpu", pytest.param("cuda", marks=pytest.mark.gpu)])
-@pytest.mark.parametrize("cap", [0.5, 30.0])
+@pytest.mark.parametrize("cap", [0.5, 24.0])
 def test_softcap(device, cap):
     z = torch.cat([rand(0, 3, 100) * 40, rand(1, 3, 100) * 1e-3])
     want = cap * torch.tanh(z.double() / cap)
@@ -281,7 +281,7 @@ def test_recurrence_cases_notice():
 
 
 # ------------------------------------------------------------------------------------------------ attention
-@pytest.mark.parametrize("count,far", [(16, 40), (32, 120), (10, 23), (32, 1000), (4, 9), (2, 5), (64, 65), (1, 10), (32, 128), (32, 256)])
+@pytest.mark.parametrize("count,far", [(16, 40), (32, 110), (10, 23), (32, 1000), (4, 9), (2, 5), (64, 65), (1, 10), (32, 128), (32, 256)])
 def test_distance_buckets(count, far):
     rel = rand(0, count, 3)
     got = distance_biases(rel, far)
@@ -316,7 +316,7 @@ def plain_attention(q, k, rel, pb, gate, scale, far, window, keep, factor):
     return torch.cat(out, 1)
 
 
-HEADS = [(1, 1, 8), (6, 2, 24), (8, 1, 64), (4, 4, 128), (6, 3, 96), (2, 1, 136), (40, 2, 16), (4, 2, 200), (3, 1, 256)]
+HEADS = [(1, 1, 8), (6, 2, 24), (8, 1, 64), (4, 4, 128), (6, 3, 88), (2, 1, 136), (40, 2, 16), (4, 2, 200), (3, 1, 256)]
 MASKS = [(0, 0), (33, 0), (64, 20), (1, 1), (17, 130), (100, 5)]
 
 
@@ -417,7 +417,7 @@ def apart(E, T, seed, top, count, keep):
 
 
 @pytest.mark.parametrize("device", ["cpu", pytest.param("cuda", marks=pytest.mark.gpu)])
-@pytest.mark.parametrize("E,top,count,keep", [(12, 3, 3, 2), (10, 2, 1, 1), (9, 2, 3, 1), (5, 5, 1, 1), (64, 6, 8, 3), (40, 8, 40, 12), (1, 1, 1, 1), (2, 1, 2, 1),
+@pytest.mark.parametrize("E,top,count,keep", [(15, 4, 5, 3), (10, 2, 1, 1), (9, 2, 3, 1), (5, 5, 1, 1), (64, 6, 8, 3), (40, 8, 40, 12), (1, 1, 1, 1), (2, 1, 2, 1),
                                               (512, 10, 64, 4)])
 def test_choice_of_experts(device, E, top, count, keep):
     z = apart(E, 37, E + top, top, count, keep)
@@ -440,7 +440,7 @@ def test_group_score_matters():
 
 
 @pytest.mark.parametrize("device,dtype", PLACES)
-@pytest.mark.parametrize("T,E,top,H,ff", [(1, 4, 2, 64, 24), (37, 12, 3, 72, 24), (300, 6, 2, 128, 40)])
+@pytest.mark.parametrize("T,E,top,H,ff", [(1, 4, 2, 64, 24), (37, 14, 3, 72, 24), (300, 6, 2, 128, 40)])
 def test_clamped_experts_beside_a_mixer(device, dtype, T, E, top, H, ff):
     """Expert outputs through the clamped unit, and their weighted sum plus the mixer's result (weight one) on the stream."""
     limit = 1.1
